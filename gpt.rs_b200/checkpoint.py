@@ -1,4 +1,4 @@
-"""GPTRSCHK v2 checkpoints -> a model resident on the GPU.
+"""GPTRSCHK v2 checkpoints and safetensors model folders -> a model resident on the GPU.
 
 Mirrors the reference's streaming load path for the decode models:
   * the file format (crates/gpt-rs/src/checkpoint/loader.rs:34-201, docs/formats.md): magic, version 2,
@@ -10,6 +10,9 @@ Mirrors the reference's streaming load path for the decode models:
     every tensor fetched by name when the model asks for it, derived layouts memoised by the stable
     id ParamKey(namespace, base id) -- here the memo lives in the CUDA library, so loading the same
     checkpoint twice into one namespace quantises nothing the second time.
+
+A folder with config.json and model.safetensors is read the same way (`open_model`); the "architecture" of its config.json
+picks the model kind from `ARCHITECTURES`.
 
 Extension over the reference reader (which rejects them, loader.rs:194-196): payloads tagged f16 (1)
 and bf16 (2) are accepted and widened to f32 on the way in.
@@ -133,6 +136,55 @@ class CheckpointReader:
         if base_id not in self.by_base_id:
             raise BackendError(3, f"tensor id {base_id:#x} not found in checkpoint")
         return self._read(self.entries[self.by_base_id[base_id]])
+
+
+# "architecture" of a model folder's config.json -> model kind of `engine_config`
+ARCHITECTURES = {"Bevosun": "bevosun"}
+
+
+class ModelFolder:
+    """config.json + model.safetensors (8-byte length, JSON header of name -> dtype, shape, data_offsets, payload), with the
+    interface of CheckpointReader; payloads are read on demand."""
+
+    TAGS = {"F32": TAG_F32, "F16": TAG_F16, "BF16": TAG_BF16, "I32": TAG_I32}
+
+    def __init__(self, path):
+        self.folder = Path(path)
+        config = json.loads((self.folder / "config.json").read_text())
+        arch = config.get("architecture")
+        if arch not in ARCHITECTURES:
+            raise BackendError(2, f"architecture {arch!r} is not a decode model of this backend")
+        self.model_config = {"kind": ARCHITECTURES[arch], "config": config}
+        self.path = self.folder / "model.safetensors"
+        with open(self.path, "rb") as f:
+            head = f.read(8)
+            if len(head) != 8:
+                raise BackendError(3, "safetensors file is truncated")
+            (n,) = struct.unpack("<Q", head)
+            self.file_size = f.seek(0, 2)
+            if 8 + n > self.file_size:
+                raise BackendError(3, "safetensors header is truncated")
+            f.seek(8)
+            header = json.loads(f.read(n).decode("utf-8"))
+        self.entries: list[Entry] = []
+        self.by_name: dict[str, int] = {}
+        for name, t in header.items():
+            if name == "__metadata__":
+                continue
+            if t["dtype"] not in self.TAGS:
+                raise BackendError(3, f"tensor {name} has dtype {t['dtype']}, which this reader does not know")
+            lo, hi = t["data_offsets"]
+            self.by_name[name] = len(self.entries)
+            self.entries.append(Entry(name, gm.base_param_id(name), tuple(t["shape"]), self.TAGS[t["dtype"]], 8 + n + lo, hi - lo))
+
+    kind = CheckpointReader.kind
+    _read = CheckpointReader._read
+    get = CheckpointReader.get
+
+
+def open_model(path):
+    """A reader for a model folder or a GPTRSCHK file."""
+    return ModelFolder(path) if Path(path).is_dir() else CheckpointReader(path)
 
 
 def save(path, kind: str, config: dict, tensors: dict[str, np.ndarray], store_base_ids: bool = False,
@@ -268,14 +320,33 @@ def engine_config(model_config: dict, weight_mode: int = gm.MODE_F32, **engine_k
                              int(c["rotary_dim"]), weight_mode=weight_mode, **engine_kw)
         scaling = c.get("rope_scaling") or {"kind": "none"}
         return cfg, (scaling if scaling.get("kind", "none") != "none" else None)
+    if kind == "bevosun":
+        return bevosun_config(c, weight_mode=weight_mode, **engine_kw), None
     raise BackendError(2, f"model kind {kind!r} is not a decode model of this backend")
+
+
+def bevosun_config(c: dict, context_length: int = 4096, **engine_kw) -> gm.ModelConfig:
+    """Bevosun's config object -> the layered kind. The design bounds no context: `context_length` is the caller's (rotation
+    tables, token history)."""
+    layers = []
+    for i, layer in enumerate(c["layers"]):
+        if layer["type"] != "latent_attention":
+            raise BackendError(2, f"layer {i}: mixer {layer['type']!r} is not built")
+        m, mlp = layer["mixer"], layer.get("mlp")
+        if mlp and mlp.get("kind") != "dense":
+            raise BackendError(2, f"layer {i}: feed-forward {mlp.get('kind')!r} is not built")
+        layers.append(gm.LayerConfig(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"]), int(m["mask"]["size"]),
+                                     float(m["scale"]), float(m["rot"]["base"]), int(m["rot"]["dims"]),
+                                     mlp=gm.MLP_DENSE_XIELU if mlp else gm.MLP_NONE, d_ff=int(mlp["ff"]) if mlp else 0))
+    return gm.ModelConfig.layered(layers, int(c["width"]), int(c["vocab"]), context_length, float(c["norm"]["eps"]), int(c["canon"]["taps"]),
+                                  float(c.get("logit_softcap") or 0.0), **engine_kw)
 
 
 def load_model(path, weight_mode: int = gm.MODE_F32, namespace: int | None = None, **engine_kw) -> gm.LoadedModel:
     """Opens a checkpoint, creates the engine model it describes and streams every parameter the
     model names to the GPU, one tensor at a time (quantising / repacking on the device when
     `weight_mode` asks for it)."""
-    reader = CheckpointReader(path)
+    reader = open_model(path)
     cfg, scaling = engine_config(reader.model_config, weight_mode, **engine_kw)
     ns = next_namespace() if namespace is None else namespace
     model = gm.LoadedModel(cfg, namespace=ns)

@@ -5,6 +5,9 @@
     python gpt.rs_b200/cli.py generate --checkpoint model.gptrschk --prompt-ids 464,2068,286 --max-tokens 64
     python gpt.rs_b200/cli.py inspect  --checkpoint model.gptrschk
     python gpt.rs_b200/cli.py export-random --out tiny.gptrschk --kind gpt --config '{"vocab_size":64,...}'
+    python gpt.rs_b200/cli.py trace    --model DIR --dtype bfloat16 --out DIR --max-tokens 4096 < steps.jsonl
+
+A checkpoint is a GPTRSCHK file or a folder with config.json and model.safetensors.
 
 `generate` prints the generated ids (one line, comma separated) on stdout and the reference's timing
 report on stderr: total tokens/s, the steady-state rate without the first token, and the wall time.
@@ -43,16 +46,18 @@ def cmd_generate(args) -> int:
     from gptrs_b200 import checkpoint as ck
     from gptrs_b200 import model as gm
     prompt = _ids(args)
-    mode = {"f32": gm.MODE_F32, "w4a16": gm.MODE_W4A16, "w8a16": gm.MODE_W8A16}[args.weight_mode]
+    mode = {"f32": gm.MODE_F32, "w4a16": gm.MODE_W4A16, "w8a16": gm.MODE_W8A16, "bf16": gm.MODE_BF16}[args.weight_mode]
     if args.top_k is not None and args.top_k < 1:
         raise SystemExit("--top-k must be at least 1")
-    reader = ck.CheckpointReader(args.checkpoint)
-    ctx_cap = int(reader.model_config["config"]["context_length"])
+    reader = ck.open_model(args.checkpoint)
+    layered = reader.kind == "bevosun"
     need = len(prompt) + args.max_tokens
+    ctx_cap = need if layered else int(reader.model_config["config"]["context_length"])
     if need > ctx_cap:
         raise SystemExit(f"prompt + max-tokens = {need} exceeds the model's context_length {ctx_cap}")
-    kw = dict(max_seqs=1, max_tokens=min(max(len(prompt), 16), 1024), max_logit_rows=1, use_pdl=1)
-    if mode != gm.MODE_F32:
+    kw = dict(context_length=ctx_cap) if layered else {}
+    kw.update(max_seqs=1, max_tokens=min(max(len(prompt), 16), 1024), max_logit_rows=1, use_pdl=1)
+    if mode != gm.MODE_F32 or layered:
         pages = (need + 15) // 16 + 1
         kw.update(kv_pages=pages + 4, max_pages_per_seq=pages)
     t_load = time.perf_counter()
@@ -65,7 +70,10 @@ def cmd_generate(args) -> int:
     if args.temperature > 0:
         model.set_top_k(args.top_k)  # kept on the device, unlike the reference's host-only top-k (inference/sampler.rs:74-81)
         n = len(prompt)
-        _, first = model.forward_with_decode_cache(prompt, [0] * n, list(range(n)), [n - 1], want_logits=False,
+        head = (n - 1) // model.config.max_tokens * model.config.max_tokens   # full chunks in front of the last one
+        if head:
+            model.prefill(0, prompt[:head])
+        _, first = model.forward_with_decode_cache(prompt[head:], [0] * (n - head), list(range(head, n)), [n - head - 1], want_logits=False,
                                                    temperature=args.temperature, seed=args.seed)
         out.append(int(first[0]))
         first_s = time.perf_counter() - t0
@@ -95,7 +103,7 @@ def cmd_generate(args) -> int:
 def cmd_inspect(args) -> int:
     _package()
     from gptrs_b200 import checkpoint as ck
-    r = ck.CheckpointReader(args.checkpoint)
+    r = ck.open_model(args.checkpoint)
     print(json.dumps(r.model_config))
     names = {ck.TAG_F32: "f32", ck.TAG_F16: "f16", ck.TAG_BF16: "bf16", ck.TAG_I32: "i32"}
     for e in r.entries:
@@ -114,15 +122,21 @@ def cmd_export_random(args) -> int:
     rng = np.random.default_rng(args.seed)
     tensors = {}
     for name, shape in cfg.param_shapes().items():
-        if name.endswith("gamma"):
+        if name.endswith("gamma") or "norm" in name.rsplit(".", 1)[-1]:
             tensors[name] = np.ones(shape, np.float32)
-        elif name.endswith("beta") or ".b_" in name:
+        elif name.endswith(("beta", ".b", ".act")) or ".b_" in name:
             tensors[name] = np.zeros(shape, np.float32)
         else:
             tensors[name] = (rng.standard_normal(size=shape, dtype=np.float32) * np.float32(args.std))
     ck.save(args.out, args.kind, config, tensors)
     print(f"wrote {args.out}: {len(tensors)} tensors", file=sys.stderr)
     return 0
+
+
+def cmd_trace(args) -> int:
+    _package()
+    from gptrs_b200 import trace
+    return trace.run(args.model, args.dtype, args.out, args.max_tokens, sys.stdin, sys.stdout)
 
 
 def main(argv=None) -> int:
@@ -137,8 +151,8 @@ def main(argv=None) -> int:
     g.add_argument("--temperature", type=float, default=0.0)
     g.add_argument("--top-k", type=int, default=None)
     g.add_argument("--seed", type=int, default=0)
-    g.add_argument("--weight-mode", default="f32", choices=["f32", "w4a16", "w8a16"],
-                   help="w4a16 / w8a16 quantise the linear weights on the device while loading (ministral kind)")
+    g.add_argument("--weight-mode", default="f32", choices=["f32", "w4a16", "w8a16", "bf16"],
+                   help="w4a16 / w8a16 quantise the linear weights on the device while loading (ministral kind); bf16: bevosun kind")
     g.add_argument("--no-graph", action="store_true", help="launch kernels one by one instead of replaying a CUDA graph")
     g.set_defaults(fn=cmd_generate)
     i = sub.add_parser("inspect", help="print the config and tensor index of a checkpoint")
@@ -146,11 +160,17 @@ def main(argv=None) -> int:
     i.set_defaults(fn=cmd_inspect)
     x = sub.add_parser("export-random", help="write a checkpoint with random weights for a config")
     x.add_argument("--out", required=True)
-    x.add_argument("--kind", required=True, choices=["gpt", "ministral"])
+    x.add_argument("--kind", required=True, choices=["gpt", "ministral", "bevosun"])
     x.add_argument("--config", required=True, help="the model's config JSON object")
     x.add_argument("--seed", type=int, default=0)
     x.add_argument("--std", type=float, default=0.02)
     x.set_defaults(fn=cmd_export_random)
+    t = sub.add_parser("trace", help="replay given token ids through a model step by step and write logits")
+    t.add_argument("--model", required=True, help="folder with config.json and model.safetensors, or a GPTRSCHK file")
+    t.add_argument("--dtype", default="bfloat16", choices=["bfloat16", "float32"])
+    t.add_argument("--out", required=True, help="folder for <step>.f32 (little-endian f32 [wanted][vocab])")
+    t.add_argument("--max-tokens", type=int, required=True, help="tokens the cache pool holds over all live requests")
+    t.set_defaults(fn=cmd_trace)
     args = ap.parse_args(argv)
     return args.fn(args)
 

@@ -11,7 +11,7 @@
 // each load instruction of a warp is one contiguous 128-byte row segment and no alignment of
 // N is needed), warps split the K rows, partial sums meet in shared memory and, when K is
 // split across a thread-block cluster, through distributed shared memory.
-#include "common.cuh"
+#include "matmul_common.cuh"
 
 namespace gptrs {
 namespace {
@@ -33,6 +33,11 @@ struct SgemmParams {
     const float* norm_gamma;  // [K]
     const float* norm_beta;   // [K] (LayerNorm)
     float norm_eps;
+    // strided and batched form: row strides of x and y, and the steps between the matrices of a batch (blockIdx.z counts
+    // row tiles x batch); act.kind / softcap replace `act`
+    int64_t ldx, ldy, x_step, y_step;
+    int m_tiles;
+    DenseAct dense;
 };
 
 template <int MT>
@@ -44,14 +49,16 @@ __global__ void __launch_bounds__(kSgWarps * 32) sgemm_smallm_kernel(const Sgemm
     const int col0 = blockIdx.x * kSgCols + lane;
     const int kb = blockIdx.y * p.k_per_cta;
     const int kn = min(p.k_per_cta, p.K - kb);
-    const int m0 = blockIdx.z * MT;
+    const int m0 = (blockIdx.z % p.m_tiles) * MT, batch = blockIdx.z / p.m_tiles;
+    const float* px = p.x + batch * p.x_step;
+    const float* pw = p.w + (size_t)batch * p.K * p.N;
 
     pdl_launch_dependents();  // dependents still wait for this whole grid before reading its results
     pdl_wait();
     if (p.norm_kind == 0) {
         for (int i = tid; i < MT * kn; i += kSgWarps * 32) {
             int m = i / kn, k = i % kn;
-            xs[m * p.k_per_cta + k] = (m0 + m < p.M) ? p.x[(size_t)(m0 + m) * p.K + kb + k] : 0.f;
+            xs[m * p.k_per_cta + k] = (m0 + m < p.M) ? px[(size_t)(m0 + m) * p.ldx + kb + k] : 0.f;
         }
     } else {
         // Row statistics over the FULL K of every row of this CTA (a few KB per row, L2 resident), two passes as
@@ -69,7 +76,7 @@ __global__ void __launch_bounds__(kSgWarps * 32) sgemm_smallm_kernel(const Sgemm
             for (int m = 0; m < MT; ++m) {
                 part[m] = 0.f;
                 if (m0 + m < p.M) {
-                    const float* row = p.x + (size_t)(m0 + m) * p.K;
+                    const float* row = px + (size_t)(m0 + m) * p.ldx;
                     const float mu = pass ? mean_s[m] : 0.f;
                     for (int k = tid; k < p.K; k += kSgWarps * 32) {
                         const float v = row[k] - mu;
@@ -93,7 +100,7 @@ __global__ void __launch_bounds__(kSgWarps * 32) sgemm_smallm_kernel(const Sgemm
             int m = i / kn, k = i % kn;
             float v = 0.f;
             if (m0 + m < p.M) {
-                v = (p.x[(size_t)(m0 + m) * p.K + kb + k] - mean_s[m]) * inv_s[m] * p.norm_gamma[kb + k];
+                v = (px[(size_t)(m0 + m) * p.ldx + kb + k] - mean_s[m]) * inv_s[m] * p.norm_gamma[kb + k];
                 if (p.norm_beta) v += p.norm_beta[kb + k];
             }
             xs[m * p.k_per_cta + k] = v;
@@ -116,7 +123,7 @@ __global__ void __launch_bounds__(kSgWarps * 32) sgemm_smallm_kernel(const Sgemm
         float wv[U][4];
 #pragma unroll
         for (int u = 0; u < U; ++u) {
-            const float* wr = p.w + (size_t)(kb + k + u * kSgWarps) * p.N + col0;
+            const float* wr = pw + (size_t)(kb + k + u * kSgWarps) * p.N + col0;
 #pragma unroll
             for (int j = 0; j < 4; ++j) wv[u][j] = cv[j] ? __ldg(wr + 32 * j) : 0.f;
         }
@@ -130,7 +137,7 @@ __global__ void __launch_bounds__(kSgWarps * 32) sgemm_smallm_kernel(const Sgemm
             }
     }
     for (; k < kn; k += kSgWarps) {
-        const float* wr = p.w + (size_t)(kb + k) * p.N + col0;
+        const float* wr = pw + (size_t)(kb + k) * p.N + col0;
         float wv[4];
 #pragma unroll
         for (int j = 0; j < 4; ++j) wv[j] = cv[j] ? __ldg(wr + 32 * j) : 0.f;
@@ -179,8 +186,9 @@ __global__ void __launch_bounds__(kSgWarps * 32) sgemm_smallm_kernel(const Sgemm
         }
         if (p.bias) v += p.bias[col];
         if (p.act == 1) v = (0.5f * v) * (1.f + erff(v / 1.4142135f));
+        v = dense_act(p.dense, v);
         if (p.residual) v += p.residual[(size_t)row * p.N + col];
-        p.y[(size_t)row * p.N + col] = v;
+        p.y[batch * p.y_step + (size_t)row * p.ldy + col] = v;
     }
     if (S > 1) cluster_sync_all();
 }
@@ -312,7 +320,7 @@ int pick_split_f32(int n_blocks, int K) {
 }
 
 template <int MT>
-int launch_sgemm(SgemmParams p, cudaStream_t st) {
+int launch_sgemm(SgemmParams p, int batch, cudaStream_t st) {
     const int n_blocks = ceil_div(p.N, kSgCols);
     p.n_split = pick_split_f32(n_blocks, p.K);
     p.k_per_cta = p.K / p.n_split;
@@ -320,8 +328,17 @@ int launch_sgemm(SgemmParams p, cudaStream_t st) {
     if (smem > 200 * 1024) return fail(GPTRS_UNIMPLEMENTED, "f32 matmul: K too large for the shared-memory x tile");
     void (*kern)(SgemmParams) = sgemm_smallm_kernel<MT>;
     GPTRS_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-    dim3 grid(n_blocks, p.n_split, ceil_div(p.M, MT));
+    p.m_tiles = ceil_div(p.M, MT);
+    if ((int64_t)p.m_tiles * batch > 65535) return fail(GPTRS_UNIMPLEMENTED, "f32 matmul: too many rows in one launch");
+    dim3 grid(n_blocks, p.n_split, p.m_tiles * batch);
     return launch_kernel(kern, grid, dim3(kSgWarps * 32), smem, st, p.n_split, p);
+}
+
+int run_sgemm(const SgemmParams& p, int batch, cudaStream_t st) {
+    if (p.M == 1) return launch_sgemm<1>(p, batch, st);
+    if (p.M == 2) return launch_sgemm<2>(p, batch, st);
+    if (p.M <= 4) return launch_sgemm<4>(p, batch, st);
+    return launch_sgemm<8>(p, batch, st);
 }
 
 }  // namespace
@@ -348,11 +365,23 @@ int gptrs_cuda_norm_matmul_f32(const float* d_x, int norm_kind, const float* d_g
     p.x = d_x; p.w = d_w; p.bias = d_bias; p.residual = d_residual; p.y = d_y;
     p.M = (int)m; p.N = (int)n; p.K = (int)k; p.act = gelu ? 1 : 0;
     p.norm_kind = norm_kind; p.norm_gamma = d_gamma; p.norm_beta = norm_kind == 1 ? d_beta : nullptr; p.norm_eps = eps;
-    cudaStream_t st = as_stream(stream);
-    if (m == 1) return launch_sgemm<1>(p, st);
-    if (m == 2) return launch_sgemm<2>(p, st);
-    if (m <= 4) return launch_sgemm<4>(p, st);
-    return launch_sgemm<8>(p, st);
+    p.ldx = k; p.ldy = n;
+    return run_sgemm(p, 1, as_stream(stream));
+}
+
+int gptrs_cuda_dense_f32(const float* d_x, const float* d_w, float* d_y, int64_t m, int64_t n, int64_t k, const gptrs_dense_epilogue* ep, void* stream) {
+    GPTRS_REQUIRE(d_x && d_w && d_y && ep, "null pointer");
+    GPTRS_REQUIRE(m >= 0 && n > 0 && k > 0 && n < (1ll << 31) && k < (1ll << 31) && m < (1ll << 31), "bad shape");
+    GPTRS_REQUIRE(ep->act == 0 || ep->act == 1, "activation: 0 none, 1 xIELU");
+    GPTRS_REQUIRE(!ep->d_best_val, "the fused greedy head is part of the bf16 path");
+    if (m == 0) return GPTRS_OK;
+    SgemmParams p = {};
+    p.x = d_x; p.w = d_w; p.bias = ep->d_bias; p.y = d_y;
+    p.M = (int)m; p.N = (int)n; p.K = (int)k;
+    p.ldx = ep->ldx ? ep->ldx : k; p.ldy = ep->ldy ? ep->ldy : n;
+    p.x_step = ep->x_step; p.y_step = ep->y_step;
+    p.dense = {ep->act, ep->act_pos, ep->act_neg, ep->softcap};
+    return run_sgemm(p, ep->batch > 1 ? (int)ep->batch : 1, as_stream(stream));
 }
 
 int gptrs_cuda_kv_append_f32(const float* d_qkv, const int32_t* d_positions, const int32_t* d_slot, float* d_k_cache,

@@ -21,155 +21,11 @@
 #include <tuple>
 #include <vector>
 
-#include "nccl_dl.h"
-#include "peer_allreduce.h"
-#include "gpt_decode_mega.h"
-#include "tensor.h"
+#include "engine.h"
 
 namespace gptrs {
 
 int sample_rows_with_values(const float* d_logits, int64_t rows, int64_t vocab, int32_t* d_tokens, float* d_values, cudaStream_t st);  // norm_embed_sample.cu
-
-namespace {
-
-enum { kKindGpt = 0, kKindMinistral = 1 };
-enum { kModeF32 = 0, kModeW4 = 1, kModeW8 = 2 };
-constexpr int kPage = 16;
-
-struct DevBuf {
-    void* p = nullptr;
-    size_t n = 0;
-    int alloc(size_t bytes, bool zero = false) {
-        release();
-        if (bytes == 0) return GPTRS_OK;
-        cudaError_t e = cudaMalloc(&p, bytes);
-        if (e != cudaSuccess) return fail(GPTRS_EXECUTION, std::string("cudaMalloc(") + std::to_string(bytes) + "): " + cudaGetErrorString(e));
-        n = bytes;
-        if (zero) cudaMemset(p, 0, bytes);
-        return GPTRS_OK;
-    }
-    void release() { if (p) cudaFree(p); p = nullptr; n = 0; }
-    ~DevBuf() { release(); }
-    template <typename T> T* as() const { return static_cast<T*>(p); }
-};
-
-struct Weight {        // one Linear
-    Tensor* f32 = nullptr;     // [in][out] (f32 mode)
-    Tensor* packed = nullptr;  // quantised + repacked (W4/W8 modes)
-    Tensor* bias = nullptr;    // optional [out]
-    int64_t in = 0, out = 0;
-};
-
-struct Layer {
-    Tensor *ln1_g = nullptr, *ln1_b = nullptr, *ln2_g = nullptr, *ln2_b = nullptr;
-    Weight qkv, attn_out, mlp_in, mlp_gate, mlp_up, mlp_gate_up, mlp_out;
-};
-
-struct GraphKey {
-    int batch, chunk_pages, splits;
-    bool operator<(const GraphKey& o) const {
-        return std::tie(batch, chunk_pages, splits) < std::tie(o.batch, o.chunk_pages, o.splits);
-    }
-};
-
-}  // namespace
-
-struct Model {
-    gptrs_model_config cfg;
-    bool finalized = false;
-    std::map<std::string, Tensor*> raw;  // name -> f32 leaf (retained)
-    std::map<std::string, std::pair<uint64_t, uint64_t>> ids;
-    Tensor *tok_emb = nullptr, *pos_emb = nullptr, *final_g = nullptr, *final_b = nullptr;
-    Weight lm_head;
-    std::vector<Layer> layers;
-    int quantised_now = 0, memo_hits = 0;
-
-    // activations
-    DevBuf hidden, xn, qkv, q_rot, attn, mlp_h, mlp_g, mlp_u, logits, xn_rows;
-    DevBuf d_tokens, d_slot, d_pos, d_ctx, d_rows, d_sampled, d_status, attn_scratch;
-    DevBuf sumsq;  // [d_model / 128][max_tokens] row sums of squares of the folded RMSNorm
-    DevBuf history;  // [max_seqs][context_length] token ids by position (the generator re-windows from it)
-    bool fold_norm = true, fold_rope = true;
-    DevBuf cos_tab, sin_tab;
-    int n_rope_pos = 0;
-    // KV
-    DevBuf kv_pool;                 // bf16 modes: [layer][page][kv_head][K|V][16][128]
-    size_t pool_layer_bytes = 0;
-    DevBuf k_cache, v_cache;        // f32 mode: [layer][slot][kv_head][capacity][hd]
-    size_t cache_layer_elems = 0;
-    DevBuf d_page_table;
-    int32_t* h_page_table = nullptr;  // pinned mirror [max_seqs][max_pages_per_seq]
-    bool table_dirty = true;
-    std::vector<int32_t> free_pages;
-    std::vector<int> seq_pages, seq_len;
-    // staging (pinned)
-    int32_t* h_stage = nullptr;  // 6 * max_tokens int32
-    float* h_logits = nullptr;
-    cudaStream_t stream = nullptr;
-    // Optional (GPTRS_LANES=2): decode steps of >= 32 sequences run as two half-batches ("lanes") on two
-    // streams, meant to overlap the HBM-bound attention of one half with the latency-bound projections of
-    // the other. Off by default: on B200 the grids of both lanes fill every SM, the work distributor runs
-    // them back to back, and the doubled weight traffic made a batch-64 step 15 % slower.
-    cudaStream_t stream2 = nullptr;
-    cudaEvent_t ev_fork = nullptr, ev_join = nullptr;
-    std::vector<cudaEvent_t> ev_a, ev_b;  // per layer: attention of lane A / lane B finished
-    int n_lanes = 1;
-    bool lane_order = true;  // lanes take turns at the attention kernel
-    int lane_priority = 0;   // launch priority of everything but attention in a two-lane step (0 = off)
-    struct GraphEntry { cudaGraphExec_t exec; int64_t kernels; };
-    std::map<GraphKey, GraphEntry> graphs;
-    // tensor parallelism: cfg holds the LOCAL head / MLP sizes; the full sizes are kept here
-    int tp = 1, tp_rank = 0, full_q = 0, full_kv = 0, full_mlp = 0, vocab_l = 0;
-    NcclComm comm = nullptr;
-    // one-shot all-reduce over peer memory (decode-sized messages); the regions of the peers are IPC mappings
-    void* peer_region = nullptr;
-    void* peer_maps[kMaxPeers] = {};
-    PeerView peer = {};
-    bool peer_on = false;
-    bool fuse_peer_push = true;   // GPTRS_TP_FUSED_PUSH=0: a copy kernel pushes the tile instead of the matmul epilogue
-    DevBuf partial, tp_vals, tp_idx, tp_gvals, tp_gidx;  // row-parallel partial sums; (max, argmax) exchange
-    // greedy head of the quantised engine: per-tile (max, argmax) candidates from the lm_head epilogue
-    DevBuf best_val, best_idx;
-    bool fuse_pick = true;   // GPTRS_FUSE_PICK=0: logits + sampling kernel
-    // f32 GPT kind, one sequence: the whole decode step as one cooperative kernel (gpt_decode_mega.cu)
-    bool mega_on = false;
-    DevBuf mega_wt, mega_scratch;   // transposed weights [out][in]; vectors + barrier word
-    MegaParams mega = {};
-    int gen_batch = 0;  // slots 0..gen_batch-1 are driven by generator_step
-    int64_t launches = 0;
-    uint32_t sample_seed = 0;
-    int64_t top_k = 0;  // 0 = no top-k filter in temperature sampling
-
-    int QKV() const { return (cfg.n_q_heads + 2 * cfg.n_kv_heads) * cfg.head_dim; }
-    int QD() const { return cfg.n_q_heads * cfg.head_dim; }
-    bool f32() const { return cfg.weight_mode == kModeF32; }
-
-    ~Model() {
-        for (auto& g : graphs) cudaGraphExecDestroy(g.second.exec);
-        for (auto& r : raw) tensor_release(r.second);
-        auto relw = [](Weight& w) { tensor_release(w.f32); tensor_release(w.packed); tensor_release(w.bias); };
-        for (auto& l : layers) {
-            for (Tensor* t : {l.ln1_g, l.ln1_b, l.ln2_g, l.ln2_b}) tensor_release(t);
-            for (Weight* w : {&l.qkv, &l.attn_out, &l.mlp_in, &l.mlp_gate, &l.mlp_up, &l.mlp_gate_up, &l.mlp_out}) relw(*w);
-        }
-        relw(lm_head);
-        for (Tensor* t : {tok_emb, pos_emb, final_g, final_b}) tensor_release(t);
-        if (h_page_table) cudaFreeHost(h_page_table);
-        if (h_stage) cudaFreeHost(h_stage);
-        if (h_logits) cudaFreeHost(h_logits);
-        for (void* p : peer_maps) if (p) cudaIpcCloseMemHandle(p);
-        if (peer_region) cudaFree(peer_region);
-        if (comm) { std::string e; if (const NcclApi* api = nccl_api(&e)) api->CommDestroy(comm); }
-        for (cudaEvent_t e : ev_a) cudaEventDestroy(e);
-        for (cudaEvent_t e : ev_b) cudaEventDestroy(e);
-        if (ev_fork) cudaEventDestroy(ev_fork);
-        if (ev_join) cudaEventDestroy(ev_join);
-        if (stream2) cudaStreamDestroy(stream2);
-        if (stream) cudaStreamDestroy(stream);
-    }
-};
-
-namespace {
 
 // Derived-parameter id: FNV-1a mix of the leaf id and a layout tag, top bit set (derived ids
 // never collide with blake3-derived leaf ids in practice; the reference uses the same idea,
@@ -192,6 +48,36 @@ int get_raw(Model& m, const std::string& name, std::vector<int64_t> want_dims, T
     *out = it->second;
     return GPTRS_OK;
 }
+
+// Device arrays of a step (token ids, slots, positions, ...), their pinned staging area of `stage_arrays` rows-long arrays, the
+// token history and the per-slot bookkeeping.
+int alloc_step_buffers(Model& m, int stage_arrays) {
+    const auto& c = m.cfg;
+    int rc;
+    if ((rc = m.history.alloc((size_t)c.max_seqs * c.context_length * 4, true))) return rc;
+    for (DevBuf* b : {&m.d_tokens, &m.d_slot, &m.d_pos, &m.d_ctx, &m.d_rows, &m.d_sampled})
+        if ((rc = b->alloc((size_t)m.stage_stride() * 4, true))) return rc;
+    if ((rc = m.d_status.alloc(4, true))) return rc;
+    GPTRS_CUDA_OK(cudaMallocHost(&m.h_stage, (size_t)stage_arrays * m.stage_stride() * 4));
+    GPTRS_CUDA_OK(cudaMallocHost(&m.h_logits, (size_t)m.max_rows() * m.vocab_l * 4));
+    m.seq_pages.assign(c.max_seqs, 0);
+    m.seq_first_page.assign(c.max_seqs, 0);
+    m.seq_len.assign(c.max_seqs, 0);
+    return GPTRS_OK;
+}
+
+int alloc_page_tables(Model& m) {
+    const auto& c = m.cfg;
+    const size_t tbytes = (size_t)c.max_seqs * c.max_pages_per_seq * 4;
+    int rc = m.d_page_table.alloc(tbytes, true);
+    if (rc) return rc;
+    GPTRS_CUDA_OK(cudaMallocHost(&m.h_page_table, tbytes));
+    memset(m.h_page_table, 0, tbytes);
+    for (int64_t p = c.kv_pages - 1; p >= 0; --p) m.free_pages.push_back((int32_t)p);
+    return GPTRS_OK;
+}
+
+namespace {
 
 // Copies rows [row0, row0+rows) and the listed column ranges of an f32 leaf [R][C] into a new tensor.
 int slice_leaf(Model& m, Tensor* full, int64_t row0, int64_t rows, const std::vector<std::pair<int64_t, int64_t>>& cols,
@@ -391,7 +277,7 @@ __global__ void tp_pick_kernel(const TpPickParams p) {
 
 // End of a generator step: the token a slot consumed goes into its history at the position it had, the sampled id
 // becomes the slot's next input, position and visible length advance.
-struct AdvanceParams { int* tokens; const int* sampled; int* pos; int* ctx; int* history; int n, context_length; };
+struct AdvanceParams { int* tokens; const int* sampled; int* pos; int* ctx; int* history; int n, context_length; int* parity; };
 __global__ void advance_kernel(const AdvanceParams p) {
     pdl_launch_dependents();  // dependents still wait for this whole grid before reading its results
     pdl_wait();
@@ -402,6 +288,7 @@ __global__ void advance_kernel(const AdvanceParams p) {
         p.tokens[i] = p.sampled[i];
         p.pos[i] = at + 1;
         p.ctx[i] += 1;
+        if (p.parity) p.parity[i] ^= 1;   // the half of the convolution state that the next step reads
     }
 }
 
@@ -421,6 +308,7 @@ int attention_plan(const Model& m, int T, int max_ctx, size_t scratch_bytes, int
 // or all T rows in order when rows_identity).
 int enqueue_forward(Model& m, int T, int max_ctx, int chunk_pages, int n_rows, bool rows_identity, float temperature,
                     int prefill_groups = 0, bool skip_logits = false) {
+    if (m.layered()) return layered_forward(m, T, max_ctx, n_rows, rows_identity, temperature, skip_logits);
     const auto& c = m.cfg;
     const int D = c.d_model;
     cudaStream_t st = m.stream;
@@ -700,8 +588,17 @@ int enqueue_forward(Model& m, int T, int max_ctx, int chunk_pages, int n_rows, b
     return launch_kernel(tp_pick_kernel, dim3((n_rows + 127) / 128), dim3(128), 0, st, 1, pp);
 }
 
+// Pages that no layer's window reaches from position `next_pos` on go back to the pool (models with windows in every layer).
+void release_passed_pages(Model& m, int slot, int next_pos) {
+    if (!m.layered()) return;
+    const int first_visible = std::max(0, next_pos - m.lay->max_window + 1);
+    const int keep = std::min(first_visible / kPage, m.seq_pages[slot]);
+    for (; m.seq_first_page[slot] < keep; ++m.seq_first_page[slot])
+        m.free_pages.push_back(m.h_page_table[(size_t)slot * m.cfg.max_pages_per_seq + m.seq_first_page[slot]]);
+}
+
 int ensure_pages(Model& m, int slot, int upto_pos) {
-    if (m.f32()) return GPTRS_OK;
+    if (!m.paged()) return GPTRS_OK;
     const int need = upto_pos / kPage + 1;
     if (need > m.cfg.max_pages_per_seq) return fail(GPTRS_SPEC_VIOLATION, "sequence exceeds max_pages_per_seq");
     while (m.seq_pages[slot] < need) {
@@ -715,7 +612,7 @@ int ensure_pages(Model& m, int slot, int upto_pos) {
 }
 
 int sync_page_table(Model& m) {
-    if (m.f32() || !m.table_dirty) return GPTRS_OK;
+    if (!m.paged() || !m.table_dirty) return GPTRS_OK;
     GPTRS_CUDA_OK(cudaMemcpyAsync(m.d_page_table.p, m.h_page_table, m.d_page_table.n, cudaMemcpyHostToDevice, m.stream));
     m.table_dirty = false;
     return GPTRS_OK;
@@ -846,7 +743,7 @@ int check_status(Model& m) {
     if (st != 0) {
         cudaMemsetAsync(m.d_status.p, 0, 4, m.stream);
         return fail(GPTRS_EXECUTION, st == 2   ? "token or position id out of range"
-                                     : st == 3 ? "a bounded wait inside a tensor-core kernel (matmul or prefill attention) gave up"
+                                     : st == 3 ? "a bounded wait inside a tensor-core kernel (matmul or attention) gave up"
                                      : st == 4 ? "a tensor-parallel peer did not deliver its partial sums in time"
                                                : "a bounded wait inside the attention kernel gave up");
     }
@@ -854,7 +751,7 @@ int check_status(Model& m) {
 }
 
 int attention_plan(const Model& m, int T, int max_ctx, size_t scratch_bytes, int* chunk_pages) {
-    if (m.f32()) { *chunk_pages = 1; return GPTRS_OK; }
+    if (m.f32() || m.layered()) { *chunk_pages = 1; return GPTRS_OK; }
     int chunk = gptrs_cuda_attention_chunk_pages(max_ctx, T, m.cfg.n_kv_heads);
     // grow the chunk until the split partials fit the scratch buffer
     while (chunk < 128 && gptrs_cuda_attention_scratch_bytes(T, m.cfg.n_q_heads, max_ctx, chunk) > scratch_bytes) chunk *= 2;
@@ -872,7 +769,18 @@ extern "C" {
 int gptrs_cuda_model_create(const gptrs_model_config* cfg, gptrs_model** out) {
     GPTRS_REQUIRE(cfg && out, "null pointer");
     const auto& c = *cfg;
-    GPTRS_REQUIRE(c.kind == kKindGpt || c.kind == kKindMinistral, "unknown model kind");
+    GPTRS_REQUIRE(c.kind == kKindGpt || c.kind == kKindMinistral || c.kind == kKindLayered, "unknown model kind");
+    if (c.kind == kKindLayered) {
+        int rc = layered_check_config(c);
+        if (rc) return rc;
+        auto m = std::make_unique<Model>();
+        m->cfg = c;
+        m->vocab_l = c.vocab;
+        m->lay = std::make_unique<Layered>();
+        GPTRS_CUDA_OK(cudaStreamCreateWithFlags(&m->stream, cudaStreamNonBlocking));
+        *out = reinterpret_cast<gptrs_model*>(m.release());
+        return GPTRS_OK;
+    }
     GPTRS_REQUIRE(c.weight_mode >= kModeF32 && c.weight_mode <= kModeW8, "unknown weight mode");
     GPTRS_REQUIRE(c.n_layers > 0 && c.d_model > 0 && c.n_q_heads > 0 && c.n_kv_heads > 0 && c.head_dim > 0 &&
                       c.d_mlp > 0 && c.vocab > 0 && c.context_length > 0, "bad model dimensions");
@@ -994,10 +902,48 @@ int gptrs_cuda_model_tp_allreduce_kind(gptrs_model* h) {
     return m.tp <= 1 ? 0 : (m.peer_on ? 2 : 1);
 }
 
+int gptrs_cuda_model_set_layers(gptrs_model* h, const gptrs_layered_config* common, const gptrs_layer_config* layers, int n_layers) {
+    GPTRS_REQUIRE(h && common && layers, "null pointer");
+    Model& m = *reinterpret_cast<Model*>(h);
+    GPTRS_REQUIRE(m.layered() && !m.finalized, "per-layer configurations belong to the layered kind, before finalize");
+    GPTRS_REQUIRE(n_layers == m.cfg.n_layers, "one configuration per layer");
+    GPTRS_REQUIRE(common->conv_taps >= 1 && common->conv_taps <= 16, "short convolutions of 1 to 16 taps");
+    m.lay->cfg = *common;
+    m.lay->layers.clear();
+    m.lay->layers.resize(n_layers);
+    for (int l = 0; l < n_layers; ++l) {
+        const gptrs_layer_config& c = layers[l];
+        if (c.mixer != GPTRS_MIXER_LATENT_ATTENTION) return fail(GPTRS_UNIMPLEMENTED, "unknown mixer");
+        if (c.mlp != GPTRS_MLP_NONE && c.mlp != GPTRS_MLP_DENSE_XIELU) return fail(GPTRS_UNIMPLEMENTED, "unknown feed-forward kind");
+        GPTRS_REQUIRE(c.mlp == GPTRS_MLP_NONE || c.d_ff > 0, "feed-forward size");
+        LayeredLayer& L = m.lay->layers[l];
+        L.cfg = c;
+        L.att.dtype = m.f32() ? GPTRS_F32 : GPTRS_BF16;
+        L.att.heads = c.heads; L.att.dim = c.dim; L.att.rot_dim = c.rot_dim; L.att.vdim = c.vdim; L.att.kv_rank = c.kv_rank;
+        L.att.window = c.window; L.att.rot_dims = c.rot_dims; L.att.scale = c.scale;
+        int rc = gptrs_cuda_latent_layout(&L.att);
+        if (rc) return rc;
+    }
+    return GPTRS_OK;
+}
+
+int gptrs_cuda_debug_layer_residuals(gptrs_model* h, float* h_out) {
+    GPTRS_REQUIRE(h, "null pointer");
+    Model& m = *reinterpret_cast<Model*>(h);
+    GPTRS_REQUIRE(m.layered(), "residuals are captured for the layered kind");
+    m.lay->h_residuals = h_out;
+    return GPTRS_OK;
+}
+
 int gptrs_cuda_model_finalize(gptrs_model* h, int drop_f32_leaves) {
     GPTRS_REQUIRE(h, "null pointer");
     Model& m = *reinterpret_cast<Model*>(h);
     GPTRS_REQUIRE(!m.finalized, "model already finalized");
+    if (m.layered()) {
+        int lrc = layered_finalize(m, drop_f32_leaves != 0);
+        if (!lrc) m.finalized = true;
+        return lrc;
+    }
     const auto& c = m.cfg;
     const int64_t D = c.d_model, QKV = m.QKV(), QD = m.QD(), MLP = c.d_mlp;
     const int64_t QKVf = (int64_t)(m.full_q + 2 * m.full_kv) * c.head_dim, QDf = (int64_t)m.full_q * c.head_dim, MLPf = m.full_mlp;
@@ -1083,17 +1029,10 @@ int gptrs_cuda_model_finalize(gptrs_model* h, int drop_f32_leaves) {
     }
     if (m.tp > 1 && ((rc = m.partial.alloc((size_t)T * D * 4)) || (rc = m.tp_vals.alloc((size_t)max_rows * 4)) || (rc = m.tp_idx.alloc((size_t)max_rows * 4)) ||
                      (rc = m.tp_gvals.alloc((size_t)m.tp * max_rows * 4)) || (rc = m.tp_gidx.alloc((size_t)m.tp * max_rows * 4)))) return rc;
-    if ((rc = m.history.alloc((size_t)c.max_seqs * c.context_length * 4, true))) return rc;
     if (m.tp > 1 && (rc = setup_peer_allreduce(m, std::min(T, 256)))) return rc;
-    for (DevBuf* b : {&m.d_tokens, &m.d_slot, &m.d_pos, &m.d_ctx, &m.d_rows, &m.d_sampled})
-        if ((rc = b->alloc((size_t)std::max(T, max_rows) * 4, true))) return rc;
-    if ((rc = m.d_status.alloc(4, true))) return rc;
-    GPTRS_CUDA_OK(cudaMallocHost(&m.h_stage, (size_t)6 * std::max(T, max_rows) * 4));
-    GPTRS_CUDA_OK(cudaMallocHost(&m.h_logits, (size_t)max_rows * m.vocab_l * 4));
+    if ((rc = alloc_step_buffers(m, 6))) return rc;
 
     // KV storage
-    m.seq_pages.assign(c.max_seqs, 0);
-    m.seq_len.assign(c.max_seqs, 0);
     if (m.f32()) {
         m.cache_layer_elems = (size_t)c.max_seqs * c.n_kv_heads * c.context_length * c.head_dim;
         if ((rc = m.k_cache.alloc(m.cache_layer_elems * c.n_layers * 4, true)) ||
@@ -1102,11 +1041,7 @@ int gptrs_cuda_model_finalize(gptrs_model* h, int drop_f32_leaves) {
         m.pool_layer_bytes = gptrs_cuda_kv_pool_bytes(c.kv_pages, c.n_kv_heads, c.head_dim);
         if ((rc = m.kv_pool.alloc(m.pool_layer_bytes * c.n_layers))) return rc;
         GPTRS_CUDA_OK(cudaMemsetAsync(m.kv_pool.p, 0, m.kv_pool.n, m.stream));
-        const size_t tbytes = (size_t)c.max_seqs * c.max_pages_per_seq * 4;
-        if ((rc = m.d_page_table.alloc(tbytes, true))) return rc;
-        GPTRS_CUDA_OK(cudaMallocHost(&m.h_page_table, tbytes));
-        memset(m.h_page_table, 0, tbytes);
-        for (int64_t p = c.kv_pages - 1; p >= 0; --p) m.free_pages.push_back((int32_t)p);
+        if ((rc = alloc_page_tables(m))) return rc;
         // scratch for the split partials at the worst case of a step
         const int64_t max_ctx = (int64_t)c.max_pages_per_seq * kPage;
         size_t worst = 0;
@@ -1145,9 +1080,10 @@ int gptrs_cuda_model_reset_sequence(gptrs_model* h, int slot) {
     Model& m = *reinterpret_cast<Model*>(h);
     GPTRS_REQUIRE(m.finalized && slot >= 0 && slot < m.cfg.max_seqs, "bad slot");
     GPTRS_CUDA_OK(cudaStreamSynchronize(m.stream));
-    for (int i = 0; i < m.seq_pages[slot]; ++i)
+    for (int i = m.seq_first_page[slot]; i < m.seq_pages[slot]; ++i)
         m.free_pages.push_back(m.h_page_table[(size_t)slot * m.cfg.max_pages_per_seq + i]);
     m.seq_pages[slot] = 0;
+    m.seq_first_page[slot] = 0;
     m.seq_len[slot] = 0;
     return GPTRS_OK;
 }
@@ -1174,18 +1110,22 @@ int gptrs_cuda_model_forward_with_decode_cache(gptrs_model* h, const int32_t* h_
     const int T = n_tokens;
     int max_ctx = 1;
     int32_t* st = m.h_stage;
-    const int stride = std::max(c.max_tokens, max_rows);
+    const int stride = m.stage_stride();
     for (int i = 0; i < T; ++i) {
         GPTRS_REQUIRE(h_slots[i] >= 0 && h_slots[i] < c.max_seqs, "slot out of range");
         GPTRS_REQUIRE(h_positions[i] >= 0 && h_positions[i] < c.context_length, "position beyond context_length");
         GPTRS_REQUIRE(h_tokens[i] >= 0 && h_tokens[i] < c.vocab, "token id out of range");
+    }
+    if (m.layered()) { int lrc = layered_stage_rows(m, h_slots, h_positions, T); if (lrc) return lrc; }
+    for (int i = 0; i < T; ++i) {
+        if (i == 0 || h_slots[i] != h_slots[i - 1]) release_passed_pages(m, h_slots[i], h_positions[i]);
         int rc = ensure_pages(m, h_slots[i], h_positions[i]);
         if (rc) return rc;
         st[i] = h_tokens[i]; st[stride + i] = h_slots[i]; st[2 * stride + i] = h_positions[i];
         st[3 * stride + i] = h_positions[i] + 1;
         max_ctx = std::max(max_ctx, h_positions[i] + 1);
-        m.seq_len[h_slots[i]] = std::max(m.seq_len[h_slots[i]], h_positions[i] + 1);
     }
+    for (int i = 0; i < T; ++i) m.seq_len[h_slots[i]] = std::max(m.seq_len[h_slots[i]], h_positions[i] + 1);
     for (int i = 0; i < n_logit_rows; ++i) {
         GPTRS_REQUIRE(h_logit_rows[i] >= 0 && h_logit_rows[i] < T, "logit row out of range");
         st[4 * stride + i] = h_logit_rows[i];
@@ -1206,7 +1146,7 @@ int gptrs_cuda_model_forward_with_decode_cache(gptrs_model* h, const int32_t* h_
     // stream, and four warps that share one ring wait for each other.
     int prefill_groups = 0;
     int attn_rows = T;
-    if (!m.f32() && T >= 2) {
+    if (!m.f32() && !m.layered() && T >= 2) {
         const int grp = c.n_q_heads / c.n_kv_heads;
         if (grp == 1 || grp == 2 || grp == 4 || grp == 8) {
             const int tq = 16 / grp;
@@ -1231,7 +1171,7 @@ int gptrs_cuda_model_forward_with_decode_cache(gptrs_model* h, const int32_t* h_
     int chunk = 1;
     attention_plan(m, attn_rows, max_ctx, m.attn_scratch.n, &chunk);
     // the split partials are indexed by token row: the scratch must hold T rows at this chunk size
-    while (chunk < 128 && gptrs_cuda_attention_scratch_bytes(T, c.n_q_heads, max_ctx, chunk) > m.attn_scratch.n) chunk *= 2;
+    while (!m.layered() && chunk < 128 && gptrs_cuda_attention_scratch_bytes(T, c.n_q_heads, max_ctx, chunk) > m.attn_scratch.n) chunk *= 2;
     m.sample_seed = seed;
     // with no requested rows the pass still runs (it fills the KV cache); logits of row 0 are discarded
     const int rows = n_logit_rows > 0 ? n_logit_rows : 1;
@@ -1243,6 +1183,7 @@ int gptrs_cuda_model_forward_with_decode_cache(gptrs_model* h, const int32_t* h_
     }
     rc = enqueue_forward(m, T, max_ctx, chunk, rows, false, temperature, prefill_groups);
     if (rc) return rc;
+    if (m.layered()) for (size_t r = 0; r < m.lay->runs.size(); r += 2) m.lay->parity[h_slots[m.lay->runs[r]]] ^= 1;
     if (h_logits && n_logit_rows)
         GPTRS_CUDA_OK(cudaMemcpyAsync(m.h_logits, m.logits.p, (size_t)n_logit_rows * m.vocab_l * 4, cudaMemcpyDeviceToHost, s));
     if (h_sampled && n_logit_rows)
@@ -1259,7 +1200,7 @@ int gptrs_cuda_generator_begin(gptrs_model* h, int batch, const int32_t* h_first
     Model& m = *reinterpret_cast<Model*>(h);
     const auto& c = m.cfg;
     GPTRS_REQUIRE(m.finalized && batch > 0 && batch <= c.max_seqs && batch <= c.max_tokens, "bad batch");
-    const int stride = std::max(c.max_tokens, c.max_logit_rows > 0 ? c.max_logit_rows : c.max_seqs);
+    const int stride = m.stage_stride();
     int32_t* st = m.h_stage;
     for (int b = 0; b < batch; ++b) {
         GPTRS_REQUIRE(h_first_tokens[b] >= 0 && h_first_tokens[b] < c.vocab, "token id out of range");
@@ -1271,6 +1212,7 @@ int gptrs_cuda_generator_begin(gptrs_model* h, int batch, const int32_t* h_first
     GPTRS_CUDA_OK(cudaMemcpyAsync(m.d_slot.p, st + stride, (size_t)batch * 4, cudaMemcpyHostToDevice, s));
     GPTRS_CUDA_OK(cudaMemcpyAsync(m.d_pos.p, st + 2 * stride, (size_t)batch * 4, cudaMemcpyHostToDevice, s));
     GPTRS_CUDA_OK(cudaMemcpyAsync(m.d_ctx.p, st + 3 * stride, (size_t)batch * 4, cudaMemcpyHostToDevice, s));
+    if (m.layered()) { int lrc = layered_stage_generator(m, batch); if (lrc) return lrc; }
     GPTRS_CUDA_OK(cudaStreamSynchronize(s));
     m.gen_batch = batch;
     return GPTRS_OK;
@@ -1307,13 +1249,14 @@ int slide_windows(Model& m, gptrs_model* h, int B, const int32_t* h_tokens_in) {
         }
     }
     // the generator's rows again: slot b at its (new) length
-    const int stride = std::max(c.max_tokens, c.max_logit_rows > 0 ? c.max_logit_rows : c.max_seqs);
+    const int stride = m.stage_stride();
     int32_t* st = m.h_stage;
     for (int b = 0; b < B; ++b) { st[b] = cur[b]; st[stride + b] = b; st[2 * stride + b] = m.seq_len[b]; st[3 * stride + b] = m.seq_len[b] + 1; }
     GPTRS_CUDA_OK(cudaMemcpyAsync(m.d_tokens.p, st, (size_t)B * 4, cudaMemcpyHostToDevice, s));
     GPTRS_CUDA_OK(cudaMemcpyAsync(m.d_slot.p, st + stride, (size_t)B * 4, cudaMemcpyHostToDevice, s));
     GPTRS_CUDA_OK(cudaMemcpyAsync(m.d_pos.p, st + 2 * stride, (size_t)B * 4, cudaMemcpyHostToDevice, s));
     GPTRS_CUDA_OK(cudaMemcpyAsync(m.d_ctx.p, st + 3 * stride, (size_t)B * 4, cudaMemcpyHostToDevice, s));
+    if (m.layered()) { int lrc = layered_stage_generator(m, B); if (lrc) return lrc; }
     GPTRS_CUDA_OK(cudaStreamSynchronize(s));
     return GPTRS_OK;
 }
@@ -1338,6 +1281,7 @@ int gptrs_cuda_generator_step(gptrs_model* h, const int32_t* h_tokens_in, int32_
     int max_ctx = 1;
     for (int b = 0; b < B; ++b) {
         GPTRS_REQUIRE(m.seq_len[b] < c.context_length, "sequence reached context_length");
+        release_passed_pages(m, b, m.seq_len[b]);
         int rc = ensure_pages(m, b, m.seq_len[b]);
         if (rc) return rc;
         max_ctx = std::max(max_ctx, m.seq_len[b] + 1);
@@ -1352,17 +1296,18 @@ int gptrs_cuda_generator_step(gptrs_model* h, const int32_t* h_tokens_in, int32_
     }
     // The launch geometry is fixed per graph: bucket the visible length (multiples of 512 tokens)
     // so that graph keys change rarely.
-    const int cap = m.f32() ? c.context_length : c.max_pages_per_seq * kPage;
-    const int bucket = m.f32() ? c.context_length : std::min(cap, ((max_ctx + 511) / 512) * 512);
+    const int cap = m.paged() ? c.max_pages_per_seq * kPage : c.context_length;
+    int bucket = m.paged() ? std::min(cap, ((max_ctx + 511) / 512) * 512) : c.context_length;
+    if (m.layered()) bucket = layered_graph_bucket(m, bucket);
     int chunk = 1;
     attention_plan(m, B, bucket, m.attn_scratch.n, &chunk);
-    const int splits = m.f32() ? 1 : (bucket + chunk * kPage - 1) / (chunk * kPage);
+    const int splits = m.layered() ? bucket : m.f32() ? 1 : (bucket + chunk * kPage - 1) / (chunk * kPage);
     auto body = [&]() -> int {
         int r = enqueue_forward(m, B, bucket, chunk, B, true, 0.f, false, true);
         if (r) return r;
         // next step: the consumed ids go into the history, the sampled ids become the inputs, positions advance
         AdvanceParams ap = {m.d_tokens.as<int>(), m.d_sampled.as<int>(), m.d_pos.as<int>(), m.d_ctx.as<int>(), m.history.as<int>(), B,
-                            c.context_length};
+                            c.context_length, m.layered() ? m.lay->d_parity.as<int>() : nullptr};
         ++m.launches;
         return launch_kernel(advance_kernel, dim3((B + 127) / 128), dim3(128), 0, s, 1, ap);
     };
@@ -1395,6 +1340,7 @@ int gptrs_cuda_generator_step(gptrs_model* h, const int32_t* h_tokens_in, int32_
         if (r) return r;
     }
     for (int b = 0; b < B; ++b) ++m.seq_len[b];
+    if (m.layered()) for (int b = 0; b < B; ++b) m.lay->parity[b] ^= 1;
     if (h_tokens_out) {
         GPTRS_CUDA_OK(cudaMemcpyAsync(m.h_stage + B, m.d_sampled.p, (size_t)B * 4, cudaMemcpyDeviceToHost, s));
         rc = check_status(m);

@@ -32,6 +32,19 @@ __host__ __device__ inline size_t w8_layout_b_bytes(int64_t n, int64_t k) {
 
 constexpr int kRedStride = kCtaN + 4; // row stride (floats) of the partial tile in shared memory
 
+// What a dense matmul does to an output element after the bias: xIELU (for z > 0 pos * z^2 + z / 2, else
+// neg * (exp(z) - 1 - z) + z / 2), then a soft cap c * tanh(z / c).
+struct DenseAct {
+    int kind;          // 0 none, 1 xIELU
+    float pos, neg;
+    float softcap;     // 0 = none
+};
+__device__ __forceinline__ float dense_act(const DenseAct& a, float z) {
+    if (a.kind == 1) z = z > 0.f ? fmaf(a.pos * z, z, 0.5f * z) : fmaf(a.neg, expm1f(z) - z, 0.5f * z);
+    if (a.softcap > 0.f) z = a.softcap * tanhf(z / a.softcap);
+    return z;
+}
+
 struct MatmulParams {
     const __nv_bfloat16* x;  // [M][K]
     const uint4* wq;         // tile-interleaved weights (layout A)
@@ -80,6 +93,9 @@ struct MatmulParams {
     float* best_val;   // [N / 128][M]
     int* best_idx;
     int skip_store;    // with best_val: the outputs themselves are not written
+    // dense bf16 matmuls (split_reduce_finish<.., true>): row stride of y, activation, soft cap
+    DenseAct act;
+    int64_t ldy;
 };
 
 // ---- split-K reduction across the CTAs of a cluster: push, one barrier, local sum -------------------
@@ -132,7 +148,7 @@ struct SplitReduce {
 };
 
 // Second half: barrier, local sum over the S slots, bias / residual / SwiGLU, store. All threads of the CTA.
-template <int MPAD>
+template <int MPAD, bool kDense = false>
 __device__ __forceinline__ void split_reduce_finish(const MatmulParams& p, const SplitReduce& sr, const float* slots, int tid,
                                                     int n_threads, int m0, int n_cta0, int tile_cols = kCtaN,
                                                     bool cluster_barrier = true) {
@@ -225,6 +241,9 @@ __device__ __forceinline__ void split_reduce_finish(const MatmulParams& p, const
                 float4 b = *reinterpret_cast<const float4*>(p.residual + (size_t)m * p.N + n);
                 v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
             }
+            if constexpr (kDense) {
+                if (p.act.kind || p.act.softcap > 0.f) { v.x = dense_act(p.act, v.x); v.y = dense_act(p.act, v.y); v.z = dense_act(p.act, v.z); v.w = dense_act(p.act, v.w); }
+            }
             if (p.best_val) {
                 // the 32 lanes of a warp hold one row of the 128-column tile
                 float bv = -INFINITY;
@@ -247,9 +266,10 @@ __device__ __forceinline__ void split_reduce_finish(const MatmulParams& p, const
                 }
             }
             if (live && !(p.best_val && p.skip_store)) {
+                const size_t at = kDense ? (size_t)m * p.ldy + n : (size_t)m * p.N + n;
                 if (p.out_f32) {
-                    *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.y) + (size_t)m * p.N + n) = v;
-                    if (p.peer_on) {
+                    *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.y) + at) = v;
+                    if (!kDense && p.peer_on) {
                         const uint32_t call = *reinterpret_cast<volatile uint32_t*>(p.peer.calls) + 1u;   // advanced by the consumer of the previous call
                         const size_t unit = ((size_t)((call - 1u) & 1u) * p.peer.tp + p.peer.rank) * p.peer.cap_floats + (size_t)m * p.N + n;
                         const uint4 lo = make_uint4(__float_as_uint(v.x), call, __float_as_uint(v.y), call);
@@ -262,7 +282,7 @@ __device__ __forceinline__ void split_reduce_finish(const MatmulParams& p, const
                     }
                 } else {
                     uint2 o = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
-                    *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(p.y) + (size_t)m * p.N + n) = o;
+                    *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(p.y) + at) = o;
                 }
             }
             if (p.sumsq_out) {

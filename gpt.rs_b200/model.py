@@ -18,8 +18,10 @@ import numpy as np
 
 from . import check, lib
 
-KIND_GPT, KIND_MINISTRAL = 0, 1
-MODE_F32, MODE_W4A16, MODE_W8A16 = 0, 1, 2
+KIND_GPT, KIND_MINISTRAL, KIND_LAYERED = 0, 1, 2
+MODE_F32, MODE_W4A16, MODE_W8A16, MODE_BF16 = 0, 1, 2, 3
+MIXER_LATENT_ATTENTION = 0
+MLP_NONE, MLP_DENSE_XIELU = 0, 1
 
 
 class _ModelConfig(ctypes.Structure):
@@ -33,6 +35,39 @@ class _ModelConfig(ctypes.Structure):
         ("kv_pages", ctypes.c_int64), ("max_pages_per_seq", ctypes.c_int), ("use_pdl", ctypes.c_int),
         ("tp_size", ctypes.c_int), ("tp_rank", ctypes.c_int),
     ]
+
+
+class _LayerConfig(ctypes.Structure):
+    _fields_ = [
+        ("mixer", ctypes.c_int), ("heads", ctypes.c_int), ("dim", ctypes.c_int), ("rot_dim", ctypes.c_int), ("rot_dims", ctypes.c_int),
+        ("vdim", ctypes.c_int), ("kv_rank", ctypes.c_int), ("window", ctypes.c_int), ("scale", ctypes.c_float),
+        ("rope_base", ctypes.c_double), ("mlp", ctypes.c_int), ("d_ff", ctypes.c_int),
+    ]
+
+
+class _LayeredConfig(ctypes.Structure):
+    _fields_ = [("conv_taps", ctypes.c_int), ("logit_softcap", ctypes.c_float)]
+
+
+@dataclass
+class LayerConfig:
+    """One layer of a model of the layered kind: its mixer (latent attention in a sliding window) and its feed-forward."""
+    heads: int
+    dim: int            # query / key dimensions of a head that are not rotated
+    rot_dim: int        # and those that are (shared key part)
+    vdim: int
+    kv_rank: int
+    window: int
+    scale: float
+    rope_base: float = 10000.0
+    rot_dims: int = 0   # rotated dimensions of the rot_dim part (0 = all)
+    mixer: int = MIXER_LATENT_ATTENTION
+    mlp: int = MLP_DENSE_XIELU
+    d_ff: int = 0
+
+    def _struct(self):
+        return _LayerConfig(self.mixer, self.heads, self.dim, self.rot_dim, self.rot_dims or self.rot_dim, self.vdim, self.kv_rank, self.window,
+                            self.scale, self.rope_base, self.mlp, self.d_ff)
 
 
 @dataclass
@@ -58,6 +93,14 @@ class ModelConfig:
     use_pdl: int = 0
     tp_size: int = 1
     tp_rank: int = 0
+    layers: list | None = None     # layered kind: one LayerConfig per layer (the head and MLP sizes above are unused)
+    conv_taps: int = 1
+    logit_softcap: float = 0.0
+
+    @staticmethod
+    def layered(layers, d_model: int, vocab: int, context_length: int, norm_eps: float, conv_taps: int, logit_softcap: float = 0.0, **kw):
+        return ModelConfig(KIND_LAYERED, len(layers), d_model, 0, 0, 0, 0, vocab, context_length, norm_eps, layers=list(layers),
+                           conv_taps=conv_taps, logit_softcap=logit_softcap, **kw)
 
     @staticmethod
     def gpt2_small(**kw):
@@ -76,6 +119,8 @@ class ModelConfig:
     def param_shapes(self) -> dict[str, tuple[int, ...]]:
         """Parameter names and shapes in the reference's layout (model/gpt.rs:222-291,
         model/ministral.rs:376-421); Linear weights are [in, out]."""
+        if self.kind == KIND_LAYERED:
+            return self._layered_shapes()
         d, qd = self.d_model, self.n_q_heads * self.head_dim
         qkv = (self.n_q_heads + 2 * self.n_kv_heads) * self.head_dim
         out: dict[str, tuple[int, ...]] = {"tok_embeddings.weight": (self.vocab, d)}
@@ -109,6 +154,32 @@ class ModelConfig:
         out["lm_head"] = (d, self.vocab)
         return out
 
+    def _layered_shapes(self) -> dict[str, tuple[int, ...]]:
+        """Names and shapes of the layered kind; Linear weights are [out, in]."""
+        d = self.d_model
+        out: dict[str, tuple[int, ...]] = {"embed": (self.vocab, d), "embed.norm": (d,)}
+        for l, c in enumerate(self.layers):
+            p = f"l{l}"
+            out[f"{p}.norm1"] = (d,)
+            out[f"{p}.canon1"] = (d, self.conv_taps)
+            out[f"{p}.mix.q"] = (c.heads * (c.dim + c.rot_dim), d)
+            out[f"{p}.mix.dkv"] = (c.kv_rank + c.rot_dim, d)
+            out[f"{p}.mix.dkv.norm"] = (c.kv_rank,)
+            out[f"{p}.mix.uk"] = (c.heads * c.dim, c.kv_rank)
+            out[f"{p}.mix.uv"] = (c.heads * c.vdim, c.kv_rank)
+            out[f"{p}.mix.o"] = (d, c.heads * c.vdim)
+            if c.mlp != MLP_NONE:
+                out[f"{p}.norm2"] = (d,)
+                out[f"{p}.canon2"] = (d, self.conv_taps)
+                out[f"{p}.mlp.up"] = (c.d_ff, d)
+                out[f"{p}.mlp.up.b"] = (c.d_ff,)
+                out[f"{p}.mlp.down"] = (d, c.d_ff)
+                out[f"{p}.mlp.down.b"] = (d,)
+                out[f"{p}.mlp.act"] = (2,)
+        out["final.norm"] = (d,)
+        out["head"] = (self.vocab, d)
+        return out
+
 
 def base_param_id(name: str) -> int:
     """first 16 bytes of blake3(name), little endian (crates/gpt-rs/src/params.rs:29-36)."""
@@ -135,6 +206,10 @@ class LoadedModel:
         c = _ModelConfig(**{f: getattr(config, f) for f, _ in _ModelConfig._fields_})
         self._h = ctypes.c_void_p()
         check(lib().gptrs_cuda_model_create(ctypes.byref(c), ctypes.byref(self._h)))
+        if config.kind == KIND_LAYERED:
+            rows = (_LayerConfig * len(config.layers))(*[l._struct() for l in config.layers])
+            common = _LayeredConfig(config.conv_taps, config.logit_softcap)
+            check(lib().gptrs_cuda_model_set_layers(self._h, ctypes.byref(common), rows, len(config.layers)))
         self._finalized = False
 
     def close(self):
@@ -219,6 +294,16 @@ class LoadedModel:
             float(temperature), int(seed)))
         return logits, sampled
 
+    def layer_residuals(self, tokens, slots, positions) -> np.ndarray:
+        """Debug, layered kind: one forward pass that returns the residual stream after every layer [layer][row][d_model]."""
+        out = np.empty((self.config.n_layers, len(tokens), self.config.d_model), dtype=np.float32)
+        check(lib().gptrs_cuda_debug_layer_residuals(self._h, out.ctypes.data))
+        try:
+            self.forward_with_decode_cache(tokens, slots, positions)
+        finally:
+            check(lib().gptrs_cuda_debug_layer_residuals(self._h, None))
+        return out
+
     def prefill(self, slot: int, tokens, chunk: int | None = None, want_logits: bool = False):
         """Appends a prompt to `slot` in chunks of at most `chunk` tokens; returns the logits
         (optional) and greedy id of the LAST prompt row (the generator's first sampled token)."""
@@ -248,7 +333,9 @@ class LoadedModel:
         align = max(16 // group, 1)
         # passes the engine gives to the tensor-core prefill attention (the rule of gptrs_cuda_model_forward: paged bf16
         # cache, heads of 128, at least two 256-row tiles) need no alignment: a tile may hold two sequences
-        if (cfg.weight_mode != MODE_F32 and cfg.head_dim == 128 and group in (1, 2, 4, 8) and chunk >= 2 * (256 // group)
+        if cfg.kind == KIND_LAYERED:   # query tiles are cut at sequence boundaries
+            align = 1
+        elif (cfg.weight_mode != MODE_F32 and cfg.head_dim == 128 and group in (1, 2, 4, 8) and chunk >= 2 * (256 // group)
                 and os.environ.get("GPTRS_PREFILL_TC", "1") != "0"):
             align = 1
         max_rows = cfg.max_logit_rows if cfg.max_logit_rows > 0 else cfg.max_seqs

@@ -189,6 +189,110 @@ int gptrs_cuda_matmul_status(int32_t* h_status);
 int gptrs_cuda_debug_matmul_fault(int starve, uint32_t spin_limit);
 
 /* ==============================================================================================
+ * Dense (unquantised) linear layers with strided rows and batches, f32 and bf16 (functional::matmul + add_bias,
+ * crates/gpt-rs/src/ops/functional/linalg.rs:109-127, tensor_ops.rs:42-56; the activations and the soft cap have no
+ * counterpart in gpt.rs).
+ * ============================================================================================ */
+typedef struct {
+    int out_dtype;             /* bf16 kernel: GPTRS_BF16 or GPTRS_F32 */
+    const float* d_bias;       /* optional [n] */
+    int act;                   /* 0 = none, 1 = xIELU: z > 0: act_pos z^2 + z/2, else act_neg (exp(z) - 1 - z) + z/2 */
+    float act_pos, act_neg;
+    float softcap;             /* > 0: y = softcap * tanh(y / softcap), after the activation */
+    int64_t ldx, ldy;          /* row strides in elements (0 = k and n) */
+    int64_t batch;             /* matrices of a batch (0 or 1 = one): weight b, x + b x_step, y + b y_step */
+    int64_t x_step, y_step;
+    /* bf16 kernel, up to 128 rows, f32 output: greedy candidates per 128-column tile (see gptrs_matmul_epilogue) */
+    float* d_best_val;
+    int32_t* d_best_idx;
+    int skip_store;
+    int32_t* d_status;         /* bf16 kernel: receives 3 when a bounded wait gives up (required) */
+} gptrs_dense_epilogue;
+/* y[m][n] = act(x[m][k] . w[b][k][n] + bias), everything f32 (weights [in, out], nn/layers/linear.rs:14). */
+int gptrs_cuda_dense_f32(const float* d_x, const float* d_w, float* d_y, int64_t m, int64_t n, int64_t k,
+                         const gptrs_dense_epilogue* ep, void* stream);
+/* y[m][n] = act(x[m][k] . w[b][n][k]^T + bias), bf16 operands on the tcgen05 tensor cores, f32 accumulation. n, k, the
+ * strides and the steps are multiples of 8; pointers are 16-byte aligned. */
+int gptrs_cuda_dense_bf16(const void* d_x, const void* d_w, void* d_y, int64_t m, int64_t n, int64_t k,
+                          const gptrs_dense_epilogue* ep, void* stream);
+
+/* ==============================================================================================
+ * Step between two sublayers of a model with norms on the sublayers' outputs and short-convolution inputs (no counterpart
+ * in gpt.rs): for every row
+ *     x_out = x + y / sqrt(mean(y^2) + eps) * gamma          (d_x NULL: without x;  d_embed set: y = embed[token])
+ *     h     = x_out + sum_j conv[:, j] * x_out(t - taps + 1 + j)
+ * Rows come in runs of consecutive positions of one sequence: run_first / run_last give the first and the last row of the
+ * run of every row. The taps - 1 values of x_out in front of a run come from d_state [slots][2][taps - 1][dim] (value of
+ * position q at index q % (taps - 1); zeros before position 0): half `parity` is read, the other one written. Without
+ * d_conv only x_out is produced. The residual is read from one buffer and written to another.
+ * ============================================================================================ */
+typedef struct {
+    const float* d_x;
+    float* d_x_out;
+    const void* d_y;
+    int y_dtype;
+    int64_t ldy;
+    const float* d_embed;
+    const int32_t* d_tokens;
+    int64_t vocab;
+    const float* d_gamma;
+    float eps;
+    const float* d_conv;       /* [dim][taps], the newest input under the last tap */
+    int64_t taps;
+    float* d_state;
+    const int32_t* d_slot;
+    const int32_t* d_pos;
+    const int32_t* d_run_first;
+    const int32_t* d_run_last;
+    const int32_t* d_parity;
+    void* d_h;
+    int h_dtype;
+    int64_t ldh;
+    int32_t* d_status;         /* receives 2 for a token id out of range */
+    int64_t rows, dim;
+} gptrs_conv_step;
+int gptrs_cuda_post_norm_conv(const gptrs_conv_step* step, void* stream);
+/* The end of such a model for the listed rows (NULL = rows 0 ..): out[i] = rms_norm(x[r] + rms_norm(y[r]) gamma) final_gamma. */
+int gptrs_cuda_post_norm_final(const float* d_x, const void* d_y, int y_dtype, int64_t ldy, const float* d_gamma,
+                               const float* d_final_gamma, float eps, const int32_t* d_rows, void* d_out, int out_dtype, int64_t ldo,
+                               int64_t n_rows, int64_t dim, void* stream);
+
+/* ==============================================================================================
+ * Latent attention (no counterpart in gpt.rs): the cache holds one normed latent of kv_rank values and one rotated key part
+ * of rot_dim values per token, shared by all heads; the per-head key and value projections are absorbed into the query
+ * (W_uk^T q, a batched gptrs_cuda_dense_* in front) and the output (W_uv o, one behind). Sliding window: position i sees
+ * i - window + 1 .. i. Pages of 16 tokens, addressed through page_table[slot][page index] like the KV pool below.
+ * ============================================================================================ */
+typedef struct {
+    int dtype;                 /* GPTRS_F32 or GPTRS_BF16: activations and cache */
+    int heads, dim, rot_dim, vdim, kv_rank, window;
+    int rot_dims;              /* rotated dimensions of the rot_dim part: pairs (2i, 2i + 1) */
+    float scale;
+    /* filled in by gptrs_cuda_latent_layout (elements): */
+    int q_head_stride, q_rot_offset, dkv_offset, rot_offset, q_row; /* projection row: heads x [dim | rot], latent, rotated key */
+    int qa_head_stride, qa_rot_offset;                              /* absorbed query of a head: [kv_rank | rot] */
+    int lat_head_stride;                                            /* attention output of a head, [kv_rank] */
+    int out_head_stride;                                            /* the same after W_uv, [vdim] */
+    int64_t page_bytes;
+} gptrs_latent_attention;
+int gptrs_cuda_latent_layout(gptrs_latent_attention* a);
+/* Rows of projections -> the latent (RMS-normed with d_norm_w) and the rotated key part in the token's page, and the
+ * rotated query parts in d_qa (the absorbed parts are written by the batched product). cos / sin [position][rot_dims / 2]. */
+int gptrs_cuda_latent_append(const gptrs_latent_attention* a, const void* d_qkv, const int32_t* d_positions, const int32_t* d_slot,
+                             const int32_t* d_page_table, int64_t max_pages, const float* d_norm_w, float eps, const float* d_cos,
+                             const float* d_sin, void* d_qa, void* d_pool, int64_t n_tokens, void* stream);
+/* Tokens of a query tile of the tensor-core kernel (0: these sizes use the plain kernel), key splits for a launch, scratch. */
+int gptrs_cuda_latent_tile_tokens(const gptrs_latent_attention* a);
+int gptrs_cuda_latent_splits(const gptrs_latent_attention* a, int64_t n_tiles, int64_t max_ctx_len);
+size_t gptrs_cuda_latent_scratch_bytes(const gptrs_latent_attention* a, int64_t n_tiles, int splits);
+/* out[T][heads][lat_head_stride] = softmax over the visible cache rows . latents. n_tiles = 0: the plain kernel; else tile i
+ * is the rows tile_row[i] .. + tile_rows[i] (at most gptrs_cuda_latent_tile_tokens, consecutive positions of one sequence). */
+int gptrs_cuda_latent_attention(const gptrs_latent_attention* a, const void* d_qa, const void* d_pool, const int32_t* d_page_table,
+                                int64_t max_pages, const int32_t* d_slot, const int32_t* d_ctx_len, const int32_t* d_tile_row,
+                                const int32_t* d_tile_rows, int64_t n_tiles, int splits, void* d_out, void* d_scratch,
+                                size_t scratch_bytes, int32_t* d_status, int64_t n_tokens, void* stream);
+
+/* ==============================================================================================
  * Paged bf16 KV cache and decode attention (split-K flash decoding).
  * Stand in for functional::apply_rope_qkv_packed (crates/gpt-rs/src/ops/functional/rotary.rs:430-536)
  * followed by functional::attention_decode_cache (crates/gpt-rs/src/ops/functional/attention.rs:657-779).
@@ -448,8 +552,8 @@ int gptrs_cuda_param_set(uint64_t id_lo, uint64_t id_hi, gptrs_tensor* h);
  * ============================================================================================ */
 typedef struct gptrs_model gptrs_model;
 typedef struct {
-    int kind;            /* 0 = gpt (LayerNorm, learned positions, GELU MLP, biases), 1 = ministral */
-    int weight_mode;     /* 0 = f32, 1 = W4A16, 2 = W8A16 */
+    int kind;            /* 0 = gpt (LayerNorm, learned positions, GELU MLP, biases), 1 = ministral, 2 = layered (below) */
+    int weight_mode;     /* 0 = f32, 1 = W4A16, 2 = W8A16, 3 = bf16 (layered kind: 0 and 3) */
     int n_layers, d_model, n_q_heads, n_kv_heads, head_dim, d_mlp, vocab, context_length;
     float norm_eps;
     float rope_theta;    /* ministral */
@@ -464,7 +568,33 @@ typedef struct {
     int tp_rank;
 } gptrs_model_config;
 
+/* Layered kind (no counterpart in gpt.rs): every layer has a configuration of its own. Norms sit on the outputs of the
+ * sublayers, x <- x + rms(mixer(h)), x <- x + rms(ff(h)), and a sublayer reads h = x + conv(x), a causal convolution over the
+ * last conv_taps positions of every channel whose last conv_taps - 1 inputs are part of a sequence's state. The embedding is
+ * normed, the logits are soft-capped. Of gptrs_model_config the fields n_layers, d_model, vocab, context_length, norm_eps,
+ * max_*, kv_pages and use_pdl apply. Both weight modes keep the cache in pages; rows of a sequence must arrive in order. Pages
+ * that the windows of all layers have passed return to the pool. Parameter names ([out, in] weights): embed, embed.norm,
+ * l<i>.norm1, .norm2, .canon1, .canon2, .mix.{q,dkv,dkv.norm,uk,uv,o}, .mlp.{up,up.b,down,down.b,act}, final.norm, head. */
+enum { GPTRS_MIXER_LATENT_ATTENTION = 0 };
+enum { GPTRS_MLP_NONE = 0, GPTRS_MLP_DENSE_XIELU = 1 };
+typedef struct {
+    int mixer;
+    int heads, dim, rot_dim, rot_dims, vdim, kv_rank, window;
+    float scale;
+    double rope_base;
+    int mlp, d_ff;
+} gptrs_layer_config;
+typedef struct {
+    int conv_taps;
+    float logit_softcap;   /* 0 = none */
+} gptrs_layered_config;
+
 int gptrs_cuda_model_create(const gptrs_model_config* cfg, gptrs_model** out);
+/* Layered kind: the layers, between create and finalize. */
+int gptrs_cuda_model_set_layers(gptrs_model* m, const gptrs_layered_config* common, const gptrs_layer_config* layers, int n_layers);
+/* Debug, layered kind: the next forward_with_decode_cache also leaves the residual stream after every layer in h_out
+ * [n_layers][rows][d_model] (NULL switches it off again). */
+int gptrs_cuda_debug_layer_residuals(gptrs_model* m, float* h_out);
 void gptrs_cuda_model_destroy(gptrs_model* m);
 /* Hands one f32 parameter to the model under the reference's name (model/gpt.rs:222-291,
  * model/ministral.rs:376-421) and stable id (params.rs:29-48, two 64-bit halves). `data` is a host

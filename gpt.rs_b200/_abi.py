@@ -56,6 +56,35 @@ class MatmulEpilogue(ctypes.Structure):
     ]
 
 
+class DenseEpilogue(ctypes.Structure):
+    """gptrs_dense_epilogue."""
+    _fields_ = [
+        ("out_dtype", ctypes.c_int), ("d_bias", ctypes.c_void_p), ("act", ctypes.c_int), ("act_pos", ctypes.c_float), ("act_neg", ctypes.c_float),
+        ("softcap", ctypes.c_float), ("ldx", ctypes.c_int64), ("ldy", ctypes.c_int64), ("batch", ctypes.c_int64), ("x_step", ctypes.c_int64),
+        ("y_step", ctypes.c_int64), ("d_best_val", ctypes.c_void_p), ("d_best_idx", ctypes.c_void_p), ("skip_store", ctypes.c_int),
+        ("d_status", ctypes.c_void_p),
+    ]
+
+
+class ConvStep(ctypes.Structure):
+    """gptrs_conv_step."""
+    _fields_ = [
+        ("d_x", ctypes.c_void_p), ("d_x_out", ctypes.c_void_p), ("d_y", ctypes.c_void_p), ("y_dtype", ctypes.c_int), ("ldy", ctypes.c_int64),
+        ("d_embed", ctypes.c_void_p), ("d_tokens", ctypes.c_void_p), ("vocab", ctypes.c_int64), ("d_gamma", ctypes.c_void_p),
+        ("eps", ctypes.c_float), ("d_conv", ctypes.c_void_p), ("taps", ctypes.c_int64), ("d_state", ctypes.c_void_p), ("d_slot", ctypes.c_void_p),
+        ("d_pos", ctypes.c_void_p), ("d_run_first", ctypes.c_void_p), ("d_run_last", ctypes.c_void_p), ("d_parity", ctypes.c_void_p),
+        ("d_h", ctypes.c_void_p), ("h_dtype", ctypes.c_int), ("ldh", ctypes.c_int64), ("d_status", ctypes.c_void_p), ("rows", ctypes.c_int64),
+        ("dim", ctypes.c_int64),
+    ]
+
+
+class LatentAttention(ctypes.Structure):
+    """gptrs_latent_attention."""
+    _fields_ = [(n, ctypes.c_int) for n in ("dtype", "heads", "dim", "rot_dim", "vdim", "kv_rank", "window", "rot_dims")] + [("scale", ctypes.c_float)] + \
+        [(n, ctypes.c_int) for n in ("q_head_stride", "q_rot_offset", "dkv_offset", "rot_offset", "q_row", "qa_head_stride", "qa_rot_offset",
+                                     "lat_head_stride", "out_head_stride")] + [("page_bytes", ctypes.c_int64)]
+
+
 def prototypes(header_text: str | None = None) -> dict[str, tuple[str, list[str]]]:
     """Returns {name: (return type, [parameter declarations])} for every exported function."""
     text = header_text if header_text is not None else HEADER.read_text()

@@ -327,7 +327,7 @@ __device__ __forceinline__ float ex2f(float x) {
 
 __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams p) {
     extern __shared__ unsigned char smem_raw[];
-    __shared__ __align__(8) uint64_t k_full[kMaxStages], k_empty[kMaxStages], s_full[2], p_full[2], o_done, q_full;
+    __shared__ __align__(8) uint64_t k_full[kMaxStages], k_empty[kMaxStages], s_full[2], p_full[2], o_done, o_last, q_full;
     __shared__ uint32_t tmem_holder;
     const Geometry& g = p.g;
     const uint32_t smem = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -344,6 +344,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
         for (int i = 0; i < p.stages; ++i) { mbar_init(&k_full[i], 1); mbar_init(&k_empty[i], 1); }
         for (int i = 0; i < 2; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], (uint32_t)live_warps * 32); }
         mbar_init(&o_done, 1);
+        mbar_init(&o_last, 1);
         mbar_init(&q_full, 128);
         mbar_fence_init();
     }
@@ -446,7 +447,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
                             umma_bf16_ts(tmem + kOCol, pa + (uint32_t)(half * (kKeys / 2) + 8 * ks), vd + (uint64_t)(ks * (2 * group_stride >> 4)), idesc_o,
                                          (it > 0 || half > 0 || ks > 0) ? 1u : 0u);
                     umma_commit(&k_empty[st]);
-                    umma_commit(&o_done);
+                    umma_commit(it + 1 < n_blocks ? &o_done : &o_last);
                 }
                 __syncwarp();
             }
@@ -497,7 +498,9 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
                     m_run = m_blk;
                 }
                 if (it > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
-                    if (!wait(&o_done, (uint32_t)(it - 1) & 1u)) break;   // the product of the block before is complete
+                    // the product of the block before is complete (the one before that is: its MMAs precede these scores', so the
+                    // barrier is at most one phase behind and the parity says which)
+                    if (!wait(&o_done, (uint32_t)(it - 1) & 1u)) break;
                     tc_fence_after();
 #pragma unroll 1
                     for (int c = 0; c < g.nbc * 2; ++c) {
@@ -526,7 +529,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
                 tc_fence_before();
                 mbar_arrive_addr(smem_u32(&p_full[it & 1]));
             }
-            if (n_blocks > 0 && !failed) wait(&o_done, (uint32_t)(n_blocks - 1) & 1u);
+            if (n_blocks > 0 && !failed) wait(&o_last, 0);
             tc_fence_after();
             const size_t token_head = (size_t)(row0 + r / heads_n) * g.heads + heads0 + r % heads_n;
             if (p.splits > 1) {

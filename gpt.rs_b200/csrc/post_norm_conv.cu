@@ -84,10 +84,10 @@ __global__ void __launch_bounds__(kThreads) post_norm_conv_kernel(const StepPara
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     const int T = (int)a.rows, D = (int)a.dim;
     const int r0 = blockIdx.x * p.tile, r1 = min(r0 + p.tile, T);
-    const int keep = (int)a.taps - 1;       // values of state per channel
+    const bool conv = a.d_conv != nullptr;
+    const int keep = conv ? (int)a.taps - 1 : 0;   // values of state per channel
     pdl_launch_dependents();
     pdl_wait();
-    const bool conv = a.d_conv != nullptr;
     const int first0 = conv ? a.d_run_first[r0] : r0;
     const int i0 = max(r0 - keep, first0);  // the first row whose x this CTA needs
     const int n = r1 - i0;

@@ -375,3 +375,106 @@ def dequantize_w8(q, scales, n, k, transposed=False):
     w = torch.empty((n, k) if transposed else (k, n), dtype=torch.float32, device=q.device)
     check(lib().gptrs_cuda_dequantize_w8(_ptr(q), _ptr(scales), k, n, int(transposed), _ptr(w), _stream()))
     return w
+
+
+# ---- dense matmuls, output norm + short convolution, latent attention (layered models) ---------------------
+def _status(dev, status):
+    return torch.zeros(1, dtype=torch.int32, device=dev) if status is None else status
+
+
+def _dense_epilogue(x, bias, xielu, softcap, strides, status):
+    ep = _abi.DenseEpilogue()
+    ep.d_bias = _ptr(bias)
+    if xielu is not None:
+        ep.act, ep.act_pos, ep.act_neg = 1, *xielu
+    ep.softcap = softcap
+    for name, v in strides.items():   # ldx, ldy, batch, x_step, y_step
+        setattr(ep, name, v)
+    ep.d_status = _ptr(status)
+    return ep
+
+
+def dense_bf16(x, w, m, n, k, out=None, out_f32=False, bias=None, xielu=None, softcap=0.0, status=None, best=None, **strides):
+    """y = act(x[m][k] . w[batch][n][k]^T + bias); `xielu` = (factor of z^2 for z > 0, factor of exp(z) - 1 - z below)."""
+    status = _status(x.device, status)
+    ep = _dense_epilogue(x, bias, xielu, softcap, strides, status)
+    ep.out_dtype = F32 if out_f32 else BF16
+    if best is not None:
+        ep.d_best_val, ep.d_best_idx, ep.skip_store = _ptr(best[0]), _ptr(best[1]), 1
+    if out is None:
+        out = torch.empty((m, n), dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device)
+    check(lib().gptrs_cuda_dense_bf16(_ptr(x), _ptr(w), _ptr(out), m, n, k, ctypes.byref(ep), _stream()))
+    return out
+
+
+def dense_f32(x, w, m, n, k, out=None, bias=None, xielu=None, softcap=0.0, **strides):
+    """The same in f32 with weights [batch][k][n]."""
+    ep = _dense_epilogue(x, bias, xielu, softcap, strides, None)
+    if out is None:
+        out = torch.empty((m, n), dtype=torch.float32, device=x.device)
+    check(lib().gptrs_cuda_dense_f32(_ptr(x), _ptr(w), _ptr(out), m, n, k, ctypes.byref(ep), _stream()))
+    return out
+
+
+def post_norm_conv(gamma, eps, rows, dim, x=None, y=None, embed=None, tokens=None, conv=None, state=None, runs=None, out_dtype=torch.float32,
+                   ldh=None, status=None):
+    """x_out = x + rms_norm(y) gamma (or the normed embedding rows) and h = x_out + conv(x_out). `conv` [dim][taps];
+    `runs` = (slot, pos, run_first, run_last, parity), int32 each. Returns (x_out, h or None)."""
+    dev = gamma.device
+    status = _status(dev, status)
+    s = _abi.ConvStep()
+    s.d_gamma, s.eps, s.rows, s.dim, s.d_status = _ptr(gamma), eps, rows, dim, _ptr(status)
+    s.d_x = _ptr(x)
+    if embed is not None:
+        s.d_embed, s.d_tokens, s.vocab, s.ldy = _ptr(embed), _ptr(tokens), embed.shape[0], dim
+    else:
+        s.d_y, s.y_dtype, s.ldy = _ptr(y), _dt(y), y.shape[1]
+    x_out = torch.empty((rows, dim), dtype=torch.float32, device=dev)
+    s.d_x_out = _ptr(x_out)
+    h = None
+    if conv is not None:
+        ldh = ldh or dim
+        h = torch.empty((rows, ldh), dtype=out_dtype, device=dev)
+        s.d_conv, s.taps, s.d_state, s.d_h, s.h_dtype, s.ldh = _ptr(conv), conv.shape[1], _ptr(state), _ptr(h), _dt(h), ldh
+        s.d_slot, s.d_pos, s.d_run_first, s.d_run_last, s.d_parity = (_ptr(t) for t in runs)
+    check(lib().gptrs_cuda_post_norm_conv(ctypes.byref(s), _stream()))
+    return x_out, h
+
+
+def post_norm_final(x, y, gamma, final_gamma, eps, rows=None, out_dtype=torch.float32):
+    n, dim = (x.shape[0] if rows is None else rows.shape[0]), x.shape[1]
+    out = torch.empty((n, dim), dtype=out_dtype, device=x.device)
+    check(lib().gptrs_cuda_post_norm_final(_ptr(x), _ptr(y), _dt(y), y.shape[1], _ptr(gamma), _ptr(final_gamma), eps, _ptr(rows), _ptr(out), _dt(out),
+                                           dim, n, dim, _stream()))
+    return out
+
+
+def latent_layout(heads, dim, rot_dim, vdim, kv_rank, window, scale, rot_dims=None, bf16=True):
+    a = _abi.LatentAttention(BF16 if bf16 else F32, heads, dim, rot_dim, vdim, kv_rank, window, rot_dim if rot_dims is None else rot_dims, scale)
+    check(lib().gptrs_cuda_latent_layout(ctypes.byref(a)))
+    return a
+
+
+def latent_append(a, qkv, positions, slot, page_table, norm_w, eps, cos, sin, qa, pool):
+    check(lib().gptrs_cuda_latent_append(ctypes.byref(a), _ptr(qkv), _ptr(positions), _ptr(slot), _ptr(page_table), page_table.shape[1], _ptr(norm_w), eps,
+                                         _ptr(cos), _ptr(sin), _ptr(qa), _ptr(pool), qkv.shape[0], _stream()))
+
+
+def latent_attention(a, qa, pool, page_table, slot, ctx_len, max_ctx_len, tiles=None, splits=None, status=None):
+    """out [T][heads][lat_head_stride]; `tiles` = (first rows, row counts) for the tensor-core kernel, None for the plain one."""
+    status = _status(qa.device, status)
+    n = slot.shape[0]
+    out = torch.empty((n, a.heads, a.lat_head_stride), dtype=qa.dtype, device=qa.device)
+    n_tiles = 0 if tiles is None else tiles[0].shape[0]
+    if splits is None:
+        splits = lib().gptrs_cuda_latent_splits(ctypes.byref(a), n_tiles, max_ctx_len) if n_tiles else 1
+    nbytes = lib().gptrs_cuda_latent_scratch_bytes(ctypes.byref(a), n_tiles, splits)
+    scratch = torch.empty(max(nbytes, 1), dtype=torch.uint8, device=qa.device)
+    check(lib().gptrs_cuda_latent_attention(ctypes.byref(a), _ptr(qa), _ptr(pool), _ptr(page_table), page_table.shape[1], _ptr(slot), _ptr(ctx_len),
+                                            None if tiles is None else _ptr(tiles[0]), None if tiles is None else _ptr(tiles[1]), n_tiles, splits, _ptr(out),
+                                            _ptr(scratch), nbytes, _ptr(status), n, _stream()))
+    return out, status
+
+
+def latent_tile_tokens(a) -> int:
+    return lib().gptrs_cuda_latent_tile_tokens(ctypes.byref(a))

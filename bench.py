@@ -271,6 +271,229 @@ def time_gemv(ops, torch, dev, n=9216, k=3072, m=1, n_mats=64, iters=3, bits=4, 
     return us, alg
 
 
+# ---- layered models (Bevosun) beside the closest existing model -----------------------------------------------------------
+# name -> (width, heads, dim, rot_dim, vdim, kv_rank, window, ff, vocab; q heads and kv heads of the Ministral-shaped model of
+# the same width and feed-forward size, which has heads of 128)
+LAYERED_SIZES = {
+    "w1024": (1024, 16, 64, 32, 64, 128, 1024, 3072, 32768, 8, 2),
+    "w2048": (2048, 16, 128, 64, 128, 256, 4096, 6144, 32768, 16, 4),
+    "w3072": (3072, 32, 96, 32, 96, 256, 4096, 9216, 32768, 32, 8),
+}
+
+
+def _layered_model(gm, torch, dev, size, n_layers, ctx, pdl, chunk, batch):
+    w, heads, dim, rot, vdim, rank, window, ff, vocab = size[:9]
+    layer = gm.LayerConfig(heads, dim, rot, vdim, rank, window, (dim + rot) ** -0.5, 1e6, d_ff=ff)
+    pages = (ctx + 15) // 16
+    cfg = gm.ModelConfig.layered([layer] * n_layers, w, vocab, ctx, 1e-6, 3, 30.0, weight_mode=gm.MODE_BF16, max_seqs=batch, max_tokens=chunk,
+                                 max_logit_rows=batch, kv_pages=batch * pages + 8, max_pages_per_seq=pages, use_pdl=pdl)
+    return _random_model(gm, torch, dev, cfg, 71)
+
+
+def _ministral_model(gm, torch, dev, size, n_layers, ctx, pdl, chunk, batch):
+    pages = (ctx + 15) // 16
+    cfg = gm.ModelConfig(gm.KIND_MINISTRAL, n_layers, size[0], size[9], size[10], 128, size[7], size[8], ctx, 1e-5, 1e6, 128, weight_mode=gm.MODE_W4A16,
+                         max_seqs=batch, max_tokens=chunk, max_logit_rows=batch, kv_pages=batch * pages + 8, max_pages_per_seq=pages, use_pdl=pdl)
+    return _random_model(gm, torch, dev, cfg, 72)
+
+
+def _random_model(gm, torch, dev, cfg, namespace):
+    from gptrs_b200 import checkpoint as ck
+    m = gm.LoadedModel(cfg, namespace=ck.next_namespace() * 1000 + namespace)
+    g = torch.Generator(device=dev).manual_seed(0)
+    for name, shape in cfg.param_shapes().items():
+        if name.endswith("gamma") or "norm" in name.rsplit(".", 1)[-1]:
+            t = torch.ones(shape, device=dev)
+        else:
+            t = torch.empty(shape, device=dev).normal_(0.0, 0.02, generator=g)
+        m.load_param(name, t)
+    m.finalize()
+    return m
+
+
+def _model_speed(gm, torch, np, dev, model, prompt_len, batch, steps, warmup, prefill_seqs=8):
+    """Prefill tokens/s (prompts packed into passes of max_tokens rows) and decode tokens/s of a batch (CUDA graph, device-resident
+    ids) of one model: CUDA events on the model's stream."""
+    stream = torch.cuda.ExternalStream(lib_stream(model), device=dev)
+    rng = np.random.default_rng(7)
+    prompts = [rng.integers(0, model.config.vocab, prompt_len) for _ in range(batch)]
+    first = model.prefill_many(list(range(batch)), prompts)      # also the warm-up
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    for s in range(prefill_seqs):
+        model.reset_sequence(s)
+    torch.cuda.synchronize()
+    e0.record(stream)
+    first[:prefill_seqs] = model.prefill_many(list(range(prefill_seqs)), prompts[:prefill_seqs])
+    e1.record(stream)
+    torch.cuda.synchronize()
+    prefill_ms = e0.elapsed_time(e1)
+    gen = gm.Generator(model, first)
+    for _ in range(warmup):
+        gen.step(read_back=False)
+    gen.sync()
+    launches = model.stats()["kernel_launches"]
+    e0.record(stream)
+    for _ in range(steps):
+        gen.step(read_back=False)
+    e1.record(stream)
+    gen.sync()
+    ms = e0.elapsed_time(e1) / steps
+    return {"prefill_tokens_per_s": round(prefill_seqs * prompt_len / prefill_ms * 1e3), "prefill_ms": round(prefill_ms, 2),
+            "decode_tokens_per_s": round(batch / ms * 1e3), "decode_ms_per_step": round(ms, 4), "launches_per_step": (model.stats()["kernel_launches"] - launches) // steps}
+
+
+def run_layered(args, out, gm, torch, np):
+    """Prefill and decode of Bevosun at sizes that resemble a real model's layers (random weights, bf16), beside the Ministral-shaped
+    W4A16 model of the same width, feed-forward size and depth. Not the default line."""
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    n_layers, batch, prompt = 4, BATCH, PROMPT_LEN
+    ctx = prompt + args.steps + args.warmup + 32
+    rec = {"workload": "bevosun", "layers": n_layers, "batch": batch, "prompt_tokens": prompt, "steps": args.steps, "warmup": args.warmup, "data": "synthetic", "sizes": {}}
+    sampler = ClockSampler(None)
+    sampler.start()
+    for name, size in LAYERED_SIZES.items():
+        row = {"bevosun": dict(zip(("width", "heads", "dim", "rot_dim", "vdim", "kv_rank", "window", "ff", "vocab"), size)),
+               "ministral": {"width": size[0], "q_heads": size[9], "kv_heads": size[10], "head_dim": 128, "ff": size[7]}}
+        for kind, build in (("bevosun", _layered_model), ("ministral", _ministral_model)):
+            m = build(gm, torch, dev, size, n_layers, ctx, args.pdl, args.prefill_chunk if kind == "ministral" else 2048, batch)
+            row[kind].update(_model_speed(gm, torch, np, dev, m, prompt, batch, args.steps, args.warmup))
+            m.close()
+            torch.cuda.empty_cache()
+        rec["sizes"][name] = row
+    rec["clocks"] = sampler.stop()
+    print(json.dumps(rec), file=out)
+
+
+def _graph_us(torch, calls, iters=3):
+    """Mean time of a launch in a CUDA graph that runs `calls` (distinct buffers, so that nothing stays in L2 unless it would in
+    use) back to back."""
+    for f in calls[:2]:
+        f()
+    torch.cuda.synchronize()
+    graph, side = torch.cuda.CUDAGraph(), torch.cuda.Stream()
+    with torch.cuda.stream(side):
+        graph.capture_begin()
+        for f in calls:
+            f()
+        graph.capture_end()
+    graph.replay()
+    torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record()
+    for _ in range(iters):
+        graph.replay()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1) * 1e3 / iters / len(calls)
+
+
+def time_layered_kernels(ops, torch, dev, size, rows, ctx_len=PROMPT_LEN):
+    """Every kernel of a Bevosun layer by itself at `rows` tokens: rows <= 128 is a decode step (one token per sequence, context
+    ctx_len), more is a pass over whole prompts of ctx_len tokens. Bytes and FLOPs are the algorithmic ones (each operand once;
+    attention: the cache rows a sequence sees, or 2 x (key + value dimensions) per visible pair and head of the kernel's own
+    absorbed form)."""
+    w, heads, dim, rot, vdim, rank, window, ff = size[:8]
+    decode = rows <= 128
+    hbm, tf = _peaks()[0], _tensor_peak()
+    a = ops.latent_layout(heads, dim, rot, vdim, rank, window, (dim + rot) ** -0.5)
+    res = {}
+
+    def put(name, us, nbytes, flops):
+        t_mem, t_tc = nbytes / hbm / 1e3, flops / tf / 1e6   # us at the measured peaks
+        res[name] = {"us": round(us, 2), "roofline_us": round(max(t_mem, t_tc), 2), "bound": "hbm" if t_mem > t_tc else "tensor", "frac": round(max(t_mem, t_tc) / us, 3)}
+
+    bf = torch.bfloat16
+    status = torch.zeros(1, dtype=torch.int32, device=dev)
+
+    def gemm(name, n, k, batch=1, ldx=None, x_step=0, ldy=None, y_step=0, out_f32=False, **kw):
+        n8, k8 = (n + 7) // 8 * 8, (k + 7) // 8 * 8
+        per = batch * n8 * k8 * 2
+        mats = [torch.randn(batch, n8, k8, device=dev).mul_(k8 ** -0.5).to(bf) for _ in range(max(2, min(24, (300 << 20) // per)))]
+        x = torch.randn(rows, ldx or k8, device=dev).to(bf)
+        y = torch.empty(rows, ldy or n8, device=dev, dtype=torch.float32 if out_f32 else bf)
+        st = dict(ldx=ldx or k8, ldy=ldy or n8, batch=batch, x_step=x_step, y_step=y_step) if batch > 1 else {}
+        us = _graph_us(torch, [lambda m=m: ops.dense_bf16(x, m, rows, n8, k8, out=y, out_f32=out_f32, status=status, **st, **kw) for m in mats])
+        put(name, us, per + rows * batch * (k8 + n8) * 2, 2.0 * rows * n8 * k8 * batch)
+
+    gemm("qkv", a.q_row, w)
+    gemm("absorb_q", a.lat_head_stride, dim, heads, a.q_row, a.q_head_stride, heads * a.qa_head_stride, a.qa_head_stride)
+    gemm("absorb_v", a.out_head_stride, a.lat_head_stride, heads, heads * a.lat_head_stride, a.lat_head_stride, heads * a.out_head_stride, a.out_head_stride)
+    gemm("out", w, heads * a.out_head_stride)
+    gemm("up", ff, w, bias=torch.zeros(ff, device=dev), xielu=(0.7, 1.2))
+    gemm("down", w, ff, bias=torch.zeros(w, device=dev))
+    if decode:
+        gemm("head", size[8], w, out_f32=True, softcap=30.0)
+
+    seqs = rows if decode else rows // ctx_len
+    pages = (ctx_len + 15) // 16
+    copies = 4 if decode else 1
+    pools = [torch.randn(seqs * pages * a.page_bytes // 2, device=dev).to(bf) for _ in range(copies)]
+    table = torch.randperm(seqs * pages, device=dev, dtype=torch.int32).view(seqs, pages).contiguous()
+    slot = torch.arange(seqs, dtype=torch.int32, device=dev).repeat_interleave(rows // seqs).contiguous()
+    pos = (torch.full((rows,), ctx_len - 1, device=dev) if decode else torch.arange(ctx_len, device=dev).repeat(seqs)).to(torch.int32)
+    ctx = (pos + 1).to(torch.int32)
+    qa = torch.randn(rows, heads, a.qa_head_stride, device=dev).to(bf)
+    t = 1 if decode else ops.latent_tile_tokens(a)
+    first = torch.cat([torch.arange(0, rows // seqs, t, device=dev) + s * (rows // seqs) for s in range(seqs)]).to(torch.int32)
+    count = torch.minimum(torch.full_like(first, t), (rows // seqs) - first % (rows // seqs)).to(torch.int32)
+    us = _graph_us(torch, [lambda p=p: ops.latent_attention(a, qa, p, table, slot, ctx, ctx_len, tiles=(first, count), status=status) for p in pools] * (4 if decode else 2))
+    seen = torch.minimum(ctx, torch.full_like(ctx, window)).double()
+    cache = float(seen.sum()) if decode else seqs * ctx_len
+    put("attention", us, cache * (rank + rot) * 2 + rows * heads * (2 * rank + rot) * 2, 2.0 * heads * (2 * rank + rot) * float(seen.sum()))
+    if not decode:   # the same pairs with per-head keys and values instead of latents
+        flops = 2.0 * heads * (dim + rot + vdim) * float(seen.sum())
+        res["attention"]["frac_of_unabsorbed_flops"] = round(flops / tf / 1e6 / us, 3)
+    qkv = torch.randn(rows, a.q_row, device=dev).to(bf)
+    half = rot // 2
+    cs, sn = torch.randn(ctx_len, half, device=dev), torch.randn(ctx_len, half, device=dev)
+    nw = torch.ones(rank, device=dev)
+    us = _graph_us(torch, [lambda p=p: ops.latent_append(a, qkv, pos, slot, table, nw, 1e-6, cs, sn, qa, p) for p in pools] * 4)
+    put("append", us, rows * (a.q_row + a.qa_head_stride + heads * rot) * 2, 0)
+    x = torch.randn(rows, w, device=dev)
+    y = torch.randn(rows, w, device=dev).to(bf)
+    gamma, conv = torch.ones(w, device=dev), torch.randn(w, 3, device=dev)
+    state = torch.zeros(seqs, 2, 2, w, device=dev)
+    lo = torch.arange(rows, device=dev) // (rows // seqs) * (rows // seqs)
+    runs = (slot, pos, lo.to(torch.int32), (lo + rows // seqs - 1).to(torch.int32), torch.zeros_like(slot))
+    us = _graph_us(torch, [lambda: ops.post_norm_conv(gamma, 1e-6, rows, w, x=x, y=y, conv=conv, state=state, runs=runs, out_dtype=bf, status=status)] * 8)
+    put("post_norm_conv", us, rows * w * (4 + 2 + 4 + 2) + min(rows, 2 * seqs) * w * 16, 0)
+    assert int(status) == 0
+    return res
+
+
+def time_like_kernels(ops, torch, dev, size, rows, ctx_len=PROMPT_LEN):
+    """The like kernels of the Ministral-shaped W4A16 model of the same width at the same number of rows."""
+    w, ff, n_q, n_kv = size[0], size[7], size[9], size[10]
+    hbm, tf = _peaks()[0], _tensor_peak()
+    res = {}
+    for name, n, k in (("qkv", (n_q + 2 * n_kv) * 128, w), ("out", w, n_q * 128), ("gate_up", 2 * ff, w), ("down", w, ff)):
+        per = n * k // 2 + n * (k // 128) * 2
+        us, _ = time_gemv(ops, torch, dev, n=n, k=k, m=rows, n_mats=max(2, min(24, (300 << 20) // per)), iters=1)
+        t_mem, t_tc = (per + rows * (n + k) * 2) / hbm / 1e3, 2.0 * rows * n * k / tf / 1e6
+        res[name] = {"us": round(us, 2), "roofline_us": round(max(t_mem, t_tc), 2), "bound": "hbm" if t_mem > t_tc else "tensor", "frac": round(max(t_mem, t_tc) / us, 3)}
+    x = torch.randn(rows, w, device=dev)
+    gamma = torch.ones(w, device=dev)
+    us = _graph_us(torch, [lambda: ops.add_rms_norm(x, gamma, 1e-6)] * 8)
+    t = rows * w * (4 + 2) / hbm / 1e3
+    res["rms_norm"] = {"us": round(us, 2), "roofline_us": round(t, 2), "bound": "hbm", "frac": round(t / us, 3)}
+    return res
+
+
+def run_layered_kernels(args, out, ops, torch):
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    rec = {"microbench": "layered", "decode_rows": BATCH, "ctx": PROMPT_LEN, "prefill_rows": 4 * PROMPT_LEN, "sizes": {}}
+    for name, size in LAYERED_SIZES.items():
+        rec["sizes"][name] = {"decode": time_layered_kernels(ops, torch, dev, size, BATCH), "prefill": time_layered_kernels(ops, torch, dev, size, 4 * PROMPT_LEN),
+                              "like_decode": time_like_kernels(ops, torch, dev, size, BATCH), "like_prefill": time_like_kernels(ops, torch, dev, size, 1536)}
+    ms, nbytes, _ = time_attention_kernel(ops, torch, dev, PROMPT_LEN, launches=5)
+    rec["like_decode_attention"] = {"us": round(ms * 1e3, 1), "frac": round(nbytes / ms / 1e6 / _peaks()[0], 3)}
+    pre, flops = time_prefill_attention(ops, torch, dev, PROMPT_LEN)
+    rec["like_prefill_attention"] = {"us": pre["paged_prefill_tc_kernel"]["us"], "frac": round(pre["paged_prefill_tc_kernel"]["tflops"] / _tensor_peak(), 3)}
+    print(json.dumps(rec), file=out)
+
+
 def run_reference_arm(args):
     """CPU arm: the gpt.rs C backend's kernel library (oracle/_ref) driving the restated f32 decode
     step on the host. The reference's kernels are single-threaded and requests are independent, so one
@@ -696,13 +919,14 @@ def _main(out):
     ap.add_argument("--pdl", type=int, default=int(os.environ.get("GPTRS_PDL", "1")))
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-extras", action="store_true", help="skip the kernel microbenchmarks")
-    ap.add_argument("--microbench", default=None, choices=["attention", "attention-ragged", "gemv", "gemv-lm-head", "gemm64", "quant-linear", "prefill", "prefill-attention"],
+    ap.add_argument("--microbench", default=None, choices=["attention", "attention-ragged", "gemv", "gemv-lm-head", "gemm64", "quant-linear", "prefill", "prefill-attention", "layered"],
                     help="run only one kernel microbenchmark (used for ncu captures) and print its JSON")
     ap.add_argument("--ctx", type=int, default=PROMPT_LEN + 20, help="context length for --microbench attention")
-    ap.add_argument("--workload", default="ministral3b-w4", choices=["ministral3b-w4", "gpt2-fp32", "dp512"],
+    ap.add_argument("--workload", default="ministral3b-w4", choices=["ministral3b-w4", "gpt2-fp32", "dp512", "bevosun"],
                     help="gpt2-fp32 = the reference's CPU-runnable case (one sequence, 32-token prompt, 64 greedy tokens); "
                          "dp512 = 512 requests with prompt lengths U{256..4096}, 256 decode steps each, partitioned over the ranks "
-                         "(total work fixed: strong scaling; not the default line)")
+                         "(total work fixed: strong scaling; not the default line); "
+                         "bevosun = prefill and decode of the layered kind at three sizes beside the Ministral-shaped model of equal size")
     ap.add_argument("--path", default="engine", choices=["engine", "run_program"],
                     help="gpt2-fp32 only: engine = the model-level ABI (default); run_program = every decode step one "
                          "PortableBackend::run_program call on the captured decode program")
@@ -732,6 +956,12 @@ def _main(out):
         return
     if args.workload == "dp512":
         run_dp512(args, out, gm, torch, np)
+        return
+    if args.microbench == "layered":
+        run_layered_kernels(args, out, ops, torch)
+        return
+    if args.workload == "bevosun":
+        run_layered(args, out, gm, torch, np)
         return
     if args.microbench == "prefill":
         # chunked prefill of a few 2048-token prompts through the engine (used for the ncu launch list of the prefill path)

@@ -268,22 +268,25 @@ __global__ void __launch_bounds__(kPlainThreads) latent_attention_kernel(const A
 // A CTA takes a tile of up to 128 query rows = consecutive tokens of one sequence x all heads (more than 128 heads: one token
 // x 128 heads), all reading the same cache rows, and walks its share of the visible keys in blocks of 64 (4 pages):
 //   S[128 x 64]  = Q . K^T        A = Q tile, B = key block, both K-major in shared memory; accumulator in tensor memory,
-//                                 two buffers: the scores of the next block are computed under the softmax of this one
+//                                 three buffers: the scores of the next blocks are computed under the softmax of this one
 //   softmax                       thread r owns row r: scaled scores, mask by position and window, running maximum with a lazy
 //                                 rescale; the weights go back over the scores as two bf16 terms, P = P_hi + P_lo, so that
 //                                 the weights keep 16 significant bits in the second product
 //   O[128 x rank] += P . C        A = P_hi then P_lo from tensor memory, B = the latent columns of the SAME key block
 //                                 (contraction index as rows: MN-major operand)
-// Warps 0-3 softmax, warp 4 MMA issue and tensor memory, warp 5 page requests (one bulk copy per page). A decode step is the
-// case of one token per tile, with the keys split over the y dimension of the grid; latent_combine_kernel merges the parts.
+// Warps 0-3 softmax, warp 4 score MMAs and tensor memory, warp 5 page requests (one bulk copy per page), warp 6 output MMAs: a
+// commit holds up its thread until the MMAs in front of it are under way, so one thread for both products would leave the
+// tensor pipe idle between them. A decode step is the case of one token per tile, with the keys split over the y dimension of the grid; latent_combine_kernel merges the parts.
 // Every wait is bounded (status 3).
 constexpr int kRows = 128;
 constexpr int kKeys = 64;
-constexpr int kTcThreads = 192;
+constexpr int kTcThreads = 224;
+constexpr int kScores = 3;           // score buffers in tensor memory
 constexpr int kMaxStages = 6;
+constexpr int kMaxBlocks = 6;        // 64-column blocks of a cache row
 constexpr uint32_t kWaitLimit = 1u << 16;
 constexpr float kRescaleStep = 8.f;
-constexpr uint32_t kOCol = 2 * kKeys;
+constexpr uint32_t kOCol = kScores * kKeys;
 
 struct TcParams {
     Geometry g;
@@ -319,6 +322,12 @@ __device__ __forceinline__ uint64_t desc_mn_major(uint32_t addr, uint32_t group_
     d |= (uint64_t)2 << 61;
     return d;
 }
+// true in one lane of a converged warp; unlike a test of the lane number it leaves the branch known to be warp-uniform
+__device__ __forceinline__ bool elect_one() {
+    uint32_t p;
+    asm volatile("{\n .reg .pred p;\n elect.sync _|p, 0xffffffff;\n selp.u32 %0, 1, 0, p;\n}\n" : "=r"(p));
+    return p != 0;
+}
 __device__ __forceinline__ float ex2f(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
@@ -327,7 +336,7 @@ __device__ __forceinline__ float ex2f(float x) {
 
 __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams p) {
     extern __shared__ unsigned char smem_raw[];
-    __shared__ __align__(8) uint64_t k_full[kMaxStages], k_empty[kMaxStages], s_full[2], p_full[2], o_done, o_last, q_full;
+    __shared__ __align__(8) uint64_t k_full[kMaxStages], k_empty[kMaxStages], s_full[kScores], p_full[kScores], q_full;
     __shared__ uint32_t tmem_holder;
     const Geometry& g = p.g;
     const uint32_t smem = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -342,9 +351,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
     const int live_warps = (live + 31) / 32;
     if (tid == 0) {
         for (int i = 0; i < p.stages; ++i) { mbar_init(&k_full[i], 1); mbar_init(&k_empty[i], 1); }
-        for (int i = 0; i < 2; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], (uint32_t)live_warps * 32); }
-        mbar_init(&o_done, 1);
-        mbar_init(&o_last, 1);
+        for (int i = 0; i < kScores; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], (uint32_t)live_warps * 32); }
         mbar_init(&q_full, 128);
         mbar_fence_init();
     }
@@ -378,9 +385,15 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
         // ================= pages ===================================================================================================
         const int* pt = p.page_table + (size_t)slot0 * p.max_pages;
         const uint32_t page_bytes = (uint32_t)g.page_bytes;
-        int n_req = 0;
+        auto page_of = [&](int it) {   // lane j: the j-th page of block `it`
+            const int key0 = key_base + it * kKeys;
+            return it < n_blocks && lane < (min(kKeys, hi - key0) + kPageTok - 1) / kPageTok ? __ldg(pt + key0 / kPageTok + lane) : 0;
+        };
+        int n_req = 0, page_next = page_of(0);
         for (int it = 0; it < n_blocks; ++it) {
             const int st = it % p.stages, lap = it / p.stages;
+            const int page = page_next;
+            page_next = page_of(it + 1);
             if (lap > 0 && !wait(&k_empty[st], (uint32_t)(lap - 1) & 1u)) break;
             const int key0 = key_base + it * kKeys;
             const int pages = (min(kKeys, hi - key0) + kPageTok - 1) / kPageTok;
@@ -388,7 +401,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
             if (lane == 0) mbar_expect_tx_addr(bar, (uint32_t)pages * page_bytes);
             __syncwarp();
             if (lane < pages)
-                bulk_g2s_addr(sK + st * stage_bytes + lane * page_bytes, p.pool + (size_t)pt[key0 / kPageTok + lane] * page_bytes, page_bytes, bar);
+                bulk_g2s_addr(sK + st * stage_bytes + lane * page_bytes, p.pool + (size_t)page * page_bytes, page_bytes, bar);
             __syncwarp();
             n_req = it + 1;
         }
@@ -397,60 +410,69 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
             if (!mbar_wait_parked(smem_u32(&k_full[it % p.stages]), (uint32_t)(it / p.stages) & 1u, kWaitLimit)) failed = true;
         if (failed && lane == 0) atomicExch(p.status, 3);
     } else if (warp == 4) {
-        // ================= MMA issue ===============================================================================================
+        // ================= scores ==================================================================================================
         const uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(kKeys >> 3) << 17) | ((uint32_t)(kRows >> 4) << 24);
-        const uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(g.nbc * 64 >> 3) << 17) | ((uint32_t)(kRows >> 4) << 24);
-        auto issue_s = [&](int it) {
-            if (lane == 0) {
-                const uint64_t qd = desc_k_major(sQ, 1024), kd = desc_k_major(sK + (it % p.stages) * stage_bytes, group_stride);
-                uint32_t acc = 0;
-                for (int b = 0; b < g.nb; ++b) {
-                    const int cols = b < g.nbc ? g.rank - b * 64 : g.rot - (b - g.nbc) * 64;   // columns past these are zero
-                    for (int ks = 0; ks < 4 && ks * 16 < cols; ++ks) {
-                        umma_bf16(tmem + (uint32_t)(it & 1) * kKeys, qd + (uint64_t)(b * (kRows * 128 >> 4) + 2 * ks), kd + (uint64_t)(b * (1024 >> 4) + 2 * ks),
-                                  idesc_s, acc);
-                        acc = 1;
+        // 16-column steps of every block that hold data (the columns behind them are zero). The loops are unrolled with constant
+        // descriptor offsets: an MMA of 64 keys takes about 45 cycles, so its issue must not take longer.
+        int steps[kMaxBlocks];
+#pragma unroll
+        for (int b = 0; b < kMaxBlocks; ++b) {
+            const int cols = b < g.nbc ? g.rank - b * 64 : g.rot - (b - g.nbc) * 64;
+            steps[b] = b < g.nb ? min((cols + 15) / 16, 4) : 0;
+        }
+        const uint64_t q_desc = desc_k_major(sQ, 1024);
+        if (n_blocks > 0) wait(&q_full, 0);
+        for (int it = 0; it < n_blocks && !failed; ++it) {
+            const int st = it % p.stages;
+            if (!wait(&k_full[st], (uint32_t)(it / p.stages) & 1u)) break;
+            // the weights that were in this buffer have been used up; with three stages or fewer the pages just waited for were
+            // requested after that
+            if (it >= kScores && p.stages > kScores && !wait(&k_empty[(it - kScores) % p.stages], (uint32_t)((it - kScores) / p.stages) & 1u)) break;
+            tc_fence_after();
+            const uint64_t kd = desc_k_major(sK + st * stage_bytes, group_stride);
+            const uint32_t d = tmem + (uint32_t)(it % kScores) * kKeys;
+            if (elect_one()) {
+#pragma unroll
+                for (int b = 0; b < kMaxBlocks; ++b)
+                    if (b < g.nb) {
+#pragma unroll
+                        for (int ks = 0; ks < 4; ++ks)
+                            if (ks < steps[b])
+                                umma_bf16(d, q_desc + (uint64_t)(b * (kRows * 128 >> 4) + 2 * ks), kd + (uint64_t)(b * (1024 >> 4) + 2 * ks), idesc_s, (b > 0 || ks > 0) ? 1u : 0u);
                     }
-                }
-                umma_commit(&s_full[it & 1]);
+                umma_commit(&s_full[it % kScores]);
             }
             __syncwarp();
-        };
-        if (n_blocks > 0 && wait(&q_full, 0) && wait(&k_full[0], 0)) {
-            tc_fence_after();
-            issue_s(0);
-            for (int it = 0; it < n_blocks; ++it) {
-                const int st = it % p.stages;
-                if (it + 1 < n_blocks) {
-                    if (!wait(&k_full[(it + 1) % p.stages], (uint32_t)((it + 1) / p.stages) & 1u)) break;
-                    tc_fence_after();
-                    issue_s(it + 1);
-                }
-                if (!wait(&p_full[it & 1], (uint32_t)(it >> 1) & 1u)) break;
-                const int keys = hi - (key_base + it * kKeys);
-                if (keys < kKeys) {
-                    // cache rows past the last visible key may hold anything; their weights are 0, but 0 x NaN is not
-                    for (int r = keys; r < kKeys; ++r)
-                        for (int c = lane; c < g.nbc * 8; c += 32)
-                            st_shared_v4(sK + st * stage_bytes + (r >> 3) * group_stride + (c >> 3) * 1024 + (r & 7) * 128 + ((c & 7) << 4), 0, 0, 0, 0);
-                    fence_proxy_async();
-                    __syncwarp();
-                }
-                tc_fence_after();
-                if (lane == 0) {
-                    const uint64_t vd = desc_mn_major(sK + st * stage_bytes, group_stride);
-                    const uint32_t pa = tmem + (uint32_t)(it & 1) * kKeys;
-#pragma unroll
-                    for (int half = 0; half < 2; ++half)
-#pragma unroll
-                        for (int ks = 0; ks < kKeys / 16; ++ks)
-                            umma_bf16_ts(tmem + kOCol, pa + (uint32_t)(half * (kKeys / 2) + 8 * ks), vd + (uint64_t)(ks * (2 * group_stride >> 4)), idesc_o,
-                                         (it > 0 || half > 0 || ks > 0) ? 1u : 0u);
-                    umma_commit(&k_empty[st]);
-                    umma_commit(it + 1 < n_blocks ? &o_done : &o_last);
-                }
+        }
+        if (failed && lane == 0) atomicExch(p.status, 3);
+    } else if (warp == 6) {
+        // ================= outputs =================================================================================================
+        const uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(g.nbc * 64 >> 3) << 17) | ((uint32_t)(kRows >> 4) << 24);
+        for (int it = 0; it < n_blocks; ++it) {
+            const int st = it % p.stages;
+            if (!wait(&p_full[it % kScores], (uint32_t)(it / kScores) & 1u)) break;
+            const int keys = hi - (key_base + it * kKeys);
+            if (keys < kKeys) {
+                // cache rows past the last visible key may hold anything; their weights are 0, but 0 x NaN is not
+                for (int r = keys; r < kKeys; ++r)
+                    for (int c = lane; c < g.nbc * 8; c += 32)
+                        st_shared_v4(sK + st * stage_bytes + (r >> 3) * group_stride + (c >> 3) * 1024 + (r & 7) * 128 + ((c & 7) << 4), 0, 0, 0, 0);
+                fence_proxy_async();
                 __syncwarp();
             }
+            tc_fence_after();
+            const uint64_t vd = desc_mn_major(sK + st * stage_bytes, group_stride);
+            const uint32_t pa = tmem + (uint32_t)(it % kScores) * kKeys;
+            if (elect_one()) {
+#pragma unroll
+                for (int half = 0; half < 2; ++half)
+#pragma unroll
+                    for (int ks = 0; ks < kKeys / 16; ++ks)
+                        umma_bf16_ts(tmem + kOCol, pa + (uint32_t)(half * (kKeys / 2) + 8 * ks), vd + (uint64_t)((uint32_t)ks * (group_stride >> 3)), idesc_o,
+                                     (it > 0 || half > 0 || ks > 0) ? 1u : 0u);
+                umma_commit(&k_empty[st]);
+            }
+            __syncwarp();
         }
         if (failed && lane == 0) atomicExch(p.status, 3);
     } else {
@@ -475,9 +497,10 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
         float m_run = -1e30f, l_run = 0.f;
         if (warp < live_warps) {
             for (int it = 0; it < n_blocks; ++it) {
-                if (!wait(&s_full[it & 1], (uint32_t)(it >> 1) & 1u)) break;
+                const int buf = it % kScores;
+                if (!wait(&s_full[buf], (uint32_t)(it / kScores) & 1u)) break;
                 tc_fence_after();
-                const uint32_t t_s = t_lane + (uint32_t)(it & 1) * kKeys;
+                const uint32_t t_s = t_lane + (uint32_t)buf * kKeys;
                 float s[kKeys];
                 tmem_ld_32(t_s, *reinterpret_cast<float(*)[32]>(&s[0]));
                 tmem_ld_32(t_s + 32u, *reinterpret_cast<float(*)[32]>(&s[32]));
@@ -498,9 +521,8 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
                     m_run = m_blk;
                 }
                 if (it > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
-                    // the product of the block before is complete (the one before that is: its MMAs precede these scores', so the
-                    // barrier is at most one phase behind and the parity says which)
-                    if (!wait(&o_done, (uint32_t)(it - 1) & 1u)) break;
+                    // the product of the block before must be complete
+                    if (!wait(&k_empty[(it - 1) % p.stages], (uint32_t)((it - 1) / p.stages) & 1u)) break;
                     tc_fence_after();
 #pragma unroll 1
                     for (int c = 0; c < g.nbc * 2; ++c) {
@@ -527,9 +549,9 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
                 l_run += (sum[0] + sum[1]) + (sum[2] + sum[3]);
                 asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
                 tc_fence_before();
-                mbar_arrive_addr(smem_u32(&p_full[it & 1]));
+                mbar_arrive_addr(smem_u32(&p_full[buf]));
             }
-            if (n_blocks > 0 && !failed) wait(&o_last, 0);
+            if (n_blocks > 0 && !failed) wait(&k_empty[(n_blocks - 1) % p.stages], (uint32_t)((n_blocks - 1) / p.stages) & 1u);
             tc_fence_after();
             const size_t token_head = (size_t)(row0 + r / heads_n) * g.heads + heads0 + r % heads_n;
             if (p.splits > 1) {
@@ -612,7 +634,7 @@ int tc_stages(int nb) {
     const int n = left > 0 ? left / stage : 0;
     return n > kMaxStages ? kMaxStages : n;
 }
-bool tc_fits(const Geometry& g) { return g.nbc <= 4 && g.nb <= 6 && tc_stages(g.nb) >= 2; }
+bool tc_fits(const Geometry& g) { return g.nbc <= 4 && g.nb <= kMaxBlocks && tc_stages(g.nb) >= 2; }
 
 }  // namespace
 }  // namespace gptrs

@@ -121,7 +121,6 @@ __global__ void __launch_bounds__(192, 1) dense_rows_kernel(const __grid_constan
             tc_fence_after();
             const int m = m0 + warp * 32 + lane;
             const int64_t row = b * p.y_step + (int64_t)m * p.ldy;
-            const bool act = p.act.kind != 0 || p.act.softcap > 0.f;
 #pragma unroll 1
             for (int c0 = 0; c0 < BN && n0 + c0 < p.N; c0 += 32) {
                 float v[32];
@@ -135,9 +134,15 @@ __global__ void __launch_bounds__(192, 1) dense_rows_kernel(const __grid_constan
                             v[4 * i] += bb.x; v[4 * i + 1] += bb.y; v[4 * i + 2] += bb.z; v[4 * i + 3] += bb.w;
                         }
                 }
-                if (act) {
+                if (p.act.softcap > 0.f) {
+#pragma unroll 4
+                    for (int i = 0; i < 32; ++i) v[i] = dense_act<true>(p.act, v[i]);
+                } else if (p.act.kind == 1) {
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) v[i] = dense_act(p.act, v[i]);
+                    for (int i = 0; i < 32; ++i) {
+                        const float e = expm1_minus_fast(fminf(v[i], 0.f));
+                        v[i] = v[i] > 0.f ? fmaf(p.act.pos * v[i], v[i], 0.5f * v[i]) : fmaf(p.act.neg, e, 0.5f * v[i]);
+                    }
                 }
                 if (m < p.M) {
                     if (p.out_f32) {

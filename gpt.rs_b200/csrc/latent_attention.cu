@@ -277,7 +277,9 @@ __global__ void __launch_bounds__(kPlainThreads) latent_attention_kernel(const A
 // Warps 0-3 softmax, warp 4 score MMAs and tensor memory, warp 5 page requests (one bulk copy per page), warp 6 output MMAs: a
 // commit holds up its thread until the MMAs in front of it are under way, so one thread for both products would leave the
 // tensor pipe idle between them. A decode step is the case of one token per tile, with the keys split over the y dimension of the grid; latent_combine_kernel merges the parts.
-// Every wait is bounded (status 3).
+// Tiles of up to 64 rows (decode steps of up to 64 heads) hold every row twice: rows 64 .. 127 repeat the queries, hence the
+// scores and the softmax, and put P_lo where the first copy puts P_hi, so that one product serves both terms; the two halves of
+// O are added at the end. Every wait is bounded (status 3).
 constexpr int kRows = 128;
 constexpr int kKeys = 64;
 constexpr int kTcThreads = 224;
@@ -289,8 +291,8 @@ constexpr float kRescaleStep = 8.f;
 constexpr uint32_t kOCol = kScores * kKeys;
 
 struct TcParams {
+    CUtensorMap q_map;                 // absorbed queries: [64 columns][nb blocks][T x heads rows], 128-byte swizzle
     Geometry g;
-    const __nv_bfloat16* qa;
     const unsigned char* pool;
     const int *page_table, *slot, *ctx_len;
     const int *tile_row, *tile_rows;   // first row and number of rows of every tile
@@ -303,6 +305,11 @@ struct TcParams {
     float scale_log2;
 };
 
+__device__ __forceinline__ void tma_q(uint32_t dst, const CUtensorMap* map, int block, int row, uint32_t bar) {
+    asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];\n" ::"r"(dst), "l"(map),
+                 "r"(0), "r"(block), "r"(row), "r"(bar)
+                 : "memory");
+}
 __device__ __forceinline__ uint64_t desc_k_major(uint32_t addr, uint32_t group_stride) {
     uint64_t d = 0;
     d |= (uint64_t)((addr & 0x3FFFF) >> 4);
@@ -334,7 +341,7 @@ __device__ __forceinline__ float ex2f(float x) {
     return y;
 }
 
-__global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams p) {
+__global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const __grid_constant__ TcParams p) {
     extern __shared__ unsigned char smem_raw[];
     __shared__ __align__(8) uint64_t k_full[kMaxStages], k_empty[kMaxStages], s_full[kScores], p_full[kScores], q_full;
     __shared__ uint32_t tmem_holder;
@@ -343,21 +350,23 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
     const uint32_t stage_bytes = (uint32_t)(kKeys * 128) * g.nb, group_stride = (uint32_t)g.nb * 1024u;
     const uint32_t sQ = smem, sK = smem + (uint32_t)g.nb * (kRows * 128);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    if (warp == 4) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(smem_u32(&tmem_holder)), "r"(p.tmem_cols) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::: "memory");
+    }
+    if (tid == 32 * 5) asm volatile("prefetch.tensormap [%0];\n" ::"l"(&p.q_map) : "memory");
     pdl_wait();
     const int tile = (int)gridDim.x - 1 - (int)blockIdx.x;   // long contexts come last in a token list: start them first
     const int row0 = p.tile_row[tile], n_tok = p.tile_rows[tile], hb = blockIdx.z;
     const int heads0 = hb * kRows, heads_n = min(p.rows_per_token, g.heads - heads0);   // heads of this CTA per token
     const int live = n_tok * heads_n;
     const int live_warps = (live + 31) / 32;
+    const bool dup = live <= kRows / 2;
     if (tid == 0) {
         for (int i = 0; i < p.stages; ++i) { mbar_init(&k_full[i], 1); mbar_init(&k_empty[i], 1); }
-        for (int i = 0; i < kScores; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], (uint32_t)live_warps * 32); }
-        mbar_init(&q_full, 128);
+        for (int i = 0; i < kScores; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], (uint32_t)live_warps * (dup ? 64 : 32)); }
+        mbar_init(&q_full, 1);
         mbar_fence_init();
-    }
-    if (warp == 4) {
-        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n" ::"r"(smem_u32(&tmem_holder)), "r"(p.tmem_cols) : "memory");
-        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::: "memory");
     }
     tc_fence_before();
     __syncthreads();
@@ -382,7 +391,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
     };
 
     if (warp == 5) {
-        // ================= pages ===================================================================================================
+        // ================= pages and queries =======================================================================================
         const int* pt = p.page_table + (size_t)slot0 * p.max_pages;
         const uint32_t page_bytes = (uint32_t)g.page_bytes;
         auto page_of = [&](int it) {   // lane j: the j-th page of block `it`
@@ -390,6 +399,19 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
             return it < n_blocks && lane < (min(kKeys, hi - key0) + kPageTok - 1) / kPageTok ? __ldg(pt + key0 / kPageTok + lane) : 0;
         };
         int n_req = 0, page_next = page_of(0);
+        auto request_queries = [&]() {   // 32 rows x 64 columns per copy; rows past the live ones are other queries, whose results nobody reads
+            if (lane == 0) {
+                const uint32_t bar = smem_u32(&q_full);
+                mbar_expect_tx_addr(bar, (uint32_t)(live_warps * (dup ? 2 : 1) * g.nb) * 4096u);
+                for (int w = 0; w < live_warps; ++w)
+                    for (int b = 0; b < g.nb; ++b) {
+                        const uint32_t dst = sQ + (uint32_t)(b * kRows + w * 32) * 128u;
+                        tma_q(dst, &p.q_map, b, row0 * g.heads + heads0 + w * 32, bar);
+                        if (dup) tma_q(dst + (kRows / 2) * 128u, &p.q_map, b, row0 * g.heads + heads0 + w * 32, bar);
+                    }
+            }
+            __syncwarp();
+        };
         for (int it = 0; it < n_blocks; ++it) {
             const int st = it % p.stages, lap = it / p.stages;
             const int page = page_next;
@@ -404,8 +426,10 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
                 bulk_g2s_addr(sK + st * stage_bytes + lane * page_bytes, p.pool + (size_t)page * page_bytes, page_bytes, bar);
             __syncwarp();
             n_req = it + 1;
+            if (it == 0) request_queries();   // behind the first pages, which come from further away
         }
         // copies still in flight write this CTA's shared memory: wait for them (bounded) before leaving
+        if (n_blocks > 0 && !mbar_wait_parked(smem_u32(&q_full), 0, kWaitLimit)) failed = true;
         for (int it = max(n_req - p.stages, 0); it < n_req; ++it)
             if (!mbar_wait_parked(smem_u32(&k_full[it % p.stages]), (uint32_t)(it / p.stages) & 1u, kWaitLimit)) failed = true;
         if (failed && lane == 0) atomicExch(p.status, 3);
@@ -466,27 +490,20 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
             if (elect_one()) {
 #pragma unroll
                 for (int half = 0; half < 2; ++half)
+                    if (half == 0 || !dup)
 #pragma unroll
-                    for (int ks = 0; ks < kKeys / 16; ++ks)
-                        umma_bf16_ts(tmem + kOCol, pa + (uint32_t)(half * (kKeys / 2) + 8 * ks), vd + (uint64_t)((uint32_t)ks * (group_stride >> 3)), idesc_o,
-                                     (it > 0 || half > 0 || ks > 0) ? 1u : 0u);
+                        for (int ks = 0; ks < kKeys / 16; ++ks)
+                            umma_bf16_ts(tmem + kOCol, pa + (uint32_t)(half * (kKeys / 2) + 8 * ks), vd + (uint64_t)((uint32_t)ks * (group_stride >> 3)), idesc_o,
+                                         (it > 0 || half > 0 || ks > 0) ? 1u : 0u);
                 umma_commit(&k_empty[st]);
             }
             __syncwarp();
         }
         if (failed && lane == 0) atomicExch(p.status, 3);
     } else {
-        // ================= warps 0-3: queries to shared memory, softmax, output ========================================================
-        const int chunks = g.nb * 8;
-        for (int i = tid; i < live * chunks; i += kRows) {
-            const int r = i / chunks, c = i % chunks;
-            const size_t src = ((size_t)(row0 + r / heads_n) * g.heads + heads0 + r % heads_n) * g.qa_head_stride + c * 8;
-            const uint4 v = __ldg(reinterpret_cast<const uint4*>(p.qa + src));
-            st_shared_v4(sQ + (c >> 3) * (kRows * 128) + r * 128 + (((c & 7) ^ (r & 7)) << 4), v.x, v.y, v.z, v.w);
-        }
-        fence_proxy_async();
-        mbar_arrive_addr(smem_u32(&q_full));
-        const int r = tid;
+        // ================= warps 0-3: softmax, output ==============================================================================
+        const int r = dup ? tid & (kRows / 2 - 1) : tid;   // row of the tile
+        const bool lo_half = dup && warp >= 2;             // this copy of the row carries P_lo
         int my_len = 0;
         if (r < live) {
             my_len = p.ctx_len[row0 + r / heads_n];
@@ -495,7 +512,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
         const int my_lo = max(my_len - g.window, 0);
         const uint32_t t_lane = tmem + ((uint32_t)(warp * 32) << 16);
         float m_run = -1e30f, l_run = 0.f;
-        if (warp < live_warps) {
+        if ((dup ? warp & 1 : warp) < live_warps) {
             for (int it = 0; it < n_blocks; ++it) {
                 const int buf = it % kScores;
                 if (!wait(&s_full[buf], (uint32_t)(it / kScores) & 1u)) break;
@@ -544,8 +561,14 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
                     hi_w[i] = pack_bf16x2(p0, p1);
                     lo_w[i] = pack_bf16x2(p0 - bf16_lo(hi_w[i]), p1 - bf16_hi(hi_w[i]));
                 }
-                tmem_st_32(t_s, hi_w);
-                tmem_st_32(t_s + 32u, lo_w);
+                if (!dup) {
+                    tmem_st_32(t_s, hi_w);
+                    tmem_st_32(t_s + 32u, lo_w);
+                } else if (lo_half) {
+                    tmem_st_32(t_s, lo_w);
+                } else {
+                    tmem_st_32(t_s, hi_w);
+                }
                 l_run += (sum[0] + sum[1]) + (sum[2] + sum[3]);
                 asm volatile("tcgen05.wait::st.sync.aligned;\n" ::: "memory");
                 tc_fence_before();
@@ -553,38 +576,49 @@ __global__ void __launch_bounds__(kTcThreads, 1) latent_tc_kernel(const TcParams
             }
             if (n_blocks > 0 && !failed) wait(&k_empty[(n_blocks - 1) % p.stages], (uint32_t)((n_blocks - 1) / p.stages) & 1u);
             tc_fence_after();
-            const size_t token_head = (size_t)(row0 + r / heads_n) * g.heads + heads0 + r % heads_n;
-            if (p.splits > 1) {
-                const size_t part = (((size_t)tile * p.head_blocks + hb) * p.splits + blockIdx.y) * kRows + r;
-                if (r < live) p.part_ml[part] = make_float2(m_run, failed ? 0.f : l_run);
-                if (n_blocks > 0 && !failed) {
+            const int cols = g.nbc * 64;
+            const bool any = n_blocks > 0 && !failed;
+            float* add = reinterpret_cast<float*>(smem_raw + (sK - smem_u32(smem_raw)));   // dup: the P_lo half of O, [row][cols + 4]; every page has been used
+            if (dup) {
+                if (lo_half && any)
 #pragma unroll 1
-                    for (int c = 0; c < g.nbc * 2; ++c) {
+                    for (int c = 0; c < cols; c += 32) {
                         float o[32];
-                        tmem_ld_32(t_lane + kOCol + 32u * c, o);
-                        if (r < live) {
-                            float4* dst = reinterpret_cast<float4*>(p.part_o + part * (g.nbc * 64) + 32 * c);
+                        tmem_ld_32(t_lane + kOCol + (uint32_t)c, o);
+                        float4* dst = reinterpret_cast<float4*>(add + r * (cols + 4) + c);
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) dst[i] = make_float4(o[4 * i], o[4 * i + 1], o[4 * i + 2], o[4 * i + 3]);
+                    }
+                asm volatile("bar.sync 1, %0;\n" ::"r"(live_warps * 64) : "memory");
+            }
+            if (!lo_half) {
+                const size_t token_head = (size_t)(row0 + r / heads_n) * g.heads + heads0 + r % heads_n;
+                const size_t part = (((size_t)tile * p.head_blocks + hb) * p.splits + blockIdx.y) * kRows + r;
+                if (p.splits > 1 && r < live) p.part_ml[part] = make_float2(m_run, failed ? 0.f : l_run);
+                const float inv = p.splits > 1 ? 1.f : l_run > 0.f ? 1.f / l_run : 0.f;
+                if (any)
+#pragma unroll 1
+                    for (int c = 0; c < cols; c += 32) {
+                        float o[32];
+                        tmem_ld_32(t_lane + kOCol + (uint32_t)c, o);
+                        if (dup) {
+                            const float4* src = reinterpret_cast<const float4*>(add + r * (cols + 4) + c);
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) { const float4 v = src[i]; o[4 * i] += v.x; o[4 * i + 1] += v.y; o[4 * i + 2] += v.z; o[4 * i + 3] += v.w; }
+                        }
+                        if (r < live && p.splits > 1) {
+                            float4* dst = reinterpret_cast<float4*>(p.part_o + part * cols + c);
 #pragma unroll
                             for (int i = 0; i < 8; ++i) dst[i] = make_float4(o[4 * i], o[4 * i + 1], o[4 * i + 2], o[4 * i + 3]);
+                        } else if (r < live) {
+                            uint4* dst = reinterpret_cast<uint4*>(p.out + token_head * g.lat_stride + c);
+#pragma unroll
+                            for (int i = 0; i < 4; ++i)
+                                if (c + 8 * i < g.lat_stride)
+                                    dst[i] = make_uint4(pack_bf16x2(o[8 * i] * inv, o[8 * i + 1] * inv), pack_bf16x2(o[8 * i + 2] * inv, o[8 * i + 3] * inv),
+                                                        pack_bf16x2(o[8 * i + 4] * inv, o[8 * i + 5] * inv), pack_bf16x2(o[8 * i + 6] * inv, o[8 * i + 7] * inv));
                         }
                     }
-                }
-            } else if (n_blocks > 0 && !failed) {
-                const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-                __nv_bfloat16* dst = p.out + token_head * g.lat_stride;
-#pragma unroll 1
-                for (int c = 0; c < g.nbc * 2; ++c) {
-                    float o[32];
-                    tmem_ld_32(t_lane + kOCol + 32u * c, o);
-                    if (r < live) {
-#pragma unroll
-                        for (int i = 0; i < 4; ++i)
-                            if (32 * c + 8 * i < g.lat_stride)
-                                *reinterpret_cast<uint4*>(dst + 32 * c + 8 * i) =
-                                    make_uint4(pack_bf16x2(o[8 * i] * inv, o[8 * i + 1] * inv), pack_bf16x2(o[8 * i + 2] * inv, o[8 * i + 3] * inv),
-                                               pack_bf16x2(o[8 * i + 4] * inv, o[8 * i + 5] * inv), pack_bf16x2(o[8 * i + 6] * inv, o[8 * i + 7] * inv));
-                    }
-                }
             }
             if (failed && lane == 0) atomicExch(p.status, 3);
         }
@@ -627,6 +661,19 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const CombineParams
         }
         *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(a * inv, b * inv);
     }
+}
+
+int encode_queries(const void* qa, const Geometry& g, int64_t n_tokens, CUtensorMap* map) {
+    EncodeTiledFn enc = encode_fn();
+    if (!enc) return fail(GPTRS_EXECUTION, "cuTensorMapEncodeTiled is not available");
+    cuuint64_t dims[3] = {64, (cuuint64_t)g.nb, (cuuint64_t)(n_tokens * g.heads)};
+    cuuint64_t strides[2] = {128, (cuuint64_t)g.qa_head_stride * 2};
+    cuuint32_t box[3] = {64, 1, 32};
+    cuuint32_t estr[3] = {1, 1, 1};
+    CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(qa), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                     CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) return fail(GPTRS_EXECUTION, "cuTensorMapEncodeTiled failed for latent attention (" + std::to_string((int)r) + ")");
+    return GPTRS_OK;
 }
 
 int tc_stages(int nb) {
@@ -731,7 +778,8 @@ int gptrs_cuda_latent_attention(const gptrs_latent_attention* a, const void* d_q
     GPTRS_REQUIRE(need == 0 || (d_scratch && scratch_bytes >= need), "latent attention: scratch too small");
     TcParams p = {};
     p.g = g;
-    p.qa = static_cast<const __nv_bfloat16*>(d_qa);
+    int erc = encode_queries(d_qa, g, n_tokens, &p.q_map);
+    if (erc) return erc;
     p.pool = static_cast<const unsigned char*>(d_pool);
     p.page_table = d_page_table; p.slot = d_slot; p.ctx_len = d_ctx_len; p.tile_row = d_tile_row; p.tile_rows = d_tile_rows;
     p.out = static_cast<__nv_bfloat16*>(d_out);

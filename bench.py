@@ -133,7 +133,7 @@ def _tensor_peak():
     return 1590.0
 
 
-def time_attention_kernel(ops, torch, dev, ctx_len: int, launches: int = 20, ragged_seed=None):
+def time_attention_kernel(ops, torch, dev, ctx_len: int, launches: int = 20, ragged_seed=None, copies: int = 1):
     """CUDA-event time of the dominant kernel (paged decode attention of ONE layer) on a synthetic
     pool of the bench geometry; every launch streams the whole pool (> L2). With `ragged_seed` the
     context lengths are drawn uniformly from 512..ctx_len and the physical pages are a random permutation."""
@@ -145,7 +145,9 @@ def time_attention_kernel(ops, torch, dev, ctx_len: int, launches: int = 20, rag
         import numpy as np
         lens_host = [int(v) for v in np.random.default_rng(ragged_seed).integers(512, ctx_len + 1, size=BATCH)]
     total = BATCH * pages_per
-    pool = torch.randn(total * n_kv * 2 * 16 * 128, dtype=torch.bfloat16, device=dev).view(torch.uint8)
+    # `copies` pools take turns where one alone would stay in L2
+    pools = [torch.randn(total * n_kv * 2 * 16 * 128, dtype=torch.bfloat16, device=dev).view(torch.uint8) for _ in range(copies)]
+    pool = pools[0]
     table = torch.randperm(total, device=dev, dtype=torch.int32).view(BATCH, pages_per).contiguous()
     q = torch.randn((BATCH, n_q, 128), dtype=torch.bfloat16, device=dev)
     slot = torch.arange(BATCH, dtype=torch.int32, device=dev)
@@ -158,10 +160,10 @@ def time_attention_kernel(ops, torch, dev, ctx_len: int, launches: int = 20, rag
     nbytes = lib().gptrs_cuda_attention_scratch_bytes(BATCH, n_q, min(bucket, pages_per * 16), chunk)
     scratch = torch.empty(max(nbytes, 16), dtype=torch.uint8, device=dev)
 
-    def launch():
+    def launch(i=0):
         from gptrs_b200 import check
         check(lib().gptrs_cuda_paged_attention_decode(
-            q.data_ptr(), pool.data_ptr(), table.data_ptr(), pages_per, slot.data_ptr(), lens.data_ptr(), out.data_ptr(),
+            q.data_ptr(), pools[i % copies].data_ptr(), table.data_ptr(), pages_per, slot.data_ptr(), lens.data_ptr(), out.data_ptr(),
             scratch.data_ptr(), nbytes, status.data_ptr(), BATCH, n_q, n_kv, 128, min(bucket, pages_per * 16), chunk,
             torch.cuda.current_stream().cuda_stream))
 
@@ -172,8 +174,8 @@ def time_attention_kernel(ops, torch, dev, ctx_len: int, launches: int = 20, rag
     side = torch.cuda.Stream()
     with torch.cuda.stream(side):
         graph.capture_begin()
-        for _ in range(launches):
-            launch()
+        for i in range(launches):
+            launch(i)
         graph.capture_end()
     torch.cuda.synchronize()
     graph.replay()
@@ -388,7 +390,7 @@ def _graph_us(torch, calls, iters=3):
     return e0.elapsed_time(e1) * 1e3 / iters / len(calls)
 
 
-def time_layered_kernels(ops, torch, dev, size, rows, ctx_len=PROMPT_LEN):
+def time_layered_kernels(ops, torch, dev, size, rows, ctx_len=PROMPT_LEN, only_attention=False):
     """Every kernel of a Bevosun layer by itself at `rows` tokens: rows <= 128 is a decode step (one token per sequence, context
     ctx_len), more is a pass over whole prompts of ctx_len tokens. Bytes and FLOPs are the algorithmic ones (each operand once;
     attention: the cache rows a sequence sees, or 2 x (key + value dimensions) per visible pair and head of the kernel's own
@@ -416,14 +418,15 @@ def time_layered_kernels(ops, torch, dev, size, rows, ctx_len=PROMPT_LEN):
         us = _graph_us(torch, [lambda m=m: ops.dense_bf16(x, m, rows, n8, k8, out=y, out_f32=out_f32, status=status, **st, **kw) for m in mats])
         put(name, us, per + rows * batch * (k8 + n8) * 2, 2.0 * rows * n8 * k8 * batch)
 
-    gemm("qkv", a.q_row, w)
-    gemm("absorb_q", a.lat_head_stride, dim, heads, a.q_row, a.q_head_stride, heads * a.qa_head_stride, a.qa_head_stride)
-    gemm("absorb_v", a.out_head_stride, a.lat_head_stride, heads, heads * a.lat_head_stride, a.lat_head_stride, heads * a.out_head_stride, a.out_head_stride)
-    gemm("out", w, heads * a.out_head_stride)
-    gemm("up", ff, w, bias=torch.zeros(ff, device=dev), xielu=(0.7, 1.2))
-    gemm("down", w, ff, bias=torch.zeros(w, device=dev))
-    if decode:
-        gemm("head", size[8], w, out_f32=True, softcap=30.0)
+    if not only_attention:
+        gemm("qkv", a.q_row, w)
+        gemm("absorb_q", a.lat_head_stride, dim, heads, a.q_row, a.q_head_stride, heads * a.qa_head_stride, a.qa_head_stride)
+        gemm("absorb_v", a.out_head_stride, a.lat_head_stride, heads, heads * a.lat_head_stride, a.lat_head_stride, heads * a.out_head_stride, a.out_head_stride)
+        gemm("out", w, heads * a.out_head_stride)
+        gemm("up", ff, w, bias=torch.zeros(ff, device=dev), xielu=(0.7, 1.2))
+        gemm("down", w, ff, bias=torch.zeros(w, device=dev))
+        if decode:
+            gemm("head", size[8], w, out_f32=True, softcap=30.0)
 
     seqs = rows if decode else rows // ctx_len
     pages = (ctx_len + 15) // 16
@@ -444,6 +447,8 @@ def time_layered_kernels(ops, torch, dev, size, rows, ctx_len=PROMPT_LEN):
     if not decode:   # the same pairs with per-head keys and values instead of latents
         flops = 2.0 * heads * (dim + rot + vdim) * float(seen.sum())
         res["attention"]["frac_of_unabsorbed_flops"] = round(flops / tf / 1e6 / us, 3)
+    if only_attention:
+        return res
     qkv = torch.randn(rows, a.q_row, device=dev).to(bf)
     half = rot // 2
     cs, sn = torch.randn(ctx_len, half, device=dev), torch.randn(ctx_len, half, device=dev)
@@ -489,6 +494,13 @@ def run_layered_kernels(args, out, ops, torch):
                               "like_decode": time_like_kernels(ops, torch, dev, size, BATCH), "like_prefill": time_like_kernels(ops, torch, dev, size, 1536)}
     ms, nbytes, _ = time_attention_kernel(ops, torch, dev, PROMPT_LEN, launches=5)
     rec["like_decode_attention"] = {"us": round(ms * 1e3, 1), "frac": round(nbytes / ms / 1e6 / _peaks()[0], 3)}
+    for name, size in LAYERED_SIZES.items():   # the same kernel where it reads as many bytes as the latent cache of that size
+        eq = min(PROMPT_LEN, size[6]) * (size[5] + size[3]) * 2 // 4096
+        ms, nbytes, _ = time_attention_kernel(ops, torch, dev, eq, launches=16, copies=8)
+        rec["like_decode_attention"][f"equal_bytes_{name}"] = {"us": round(ms * 1e3, 1), "frac": round(nbytes / ms / 1e6 / _peaks()[0], 3)}
+    for ctx in (8192, 32768):   # long contexts: 64 and 16 sequences
+        size = LAYERED_SIZES["w3072"][:6] + (1 << 20,) + LAYERED_SIZES["w3072"][7:]
+        rec[f"latent_decode_attention_ctx{ctx}"] = time_layered_kernels(ops, torch, dev, size, 64 if ctx == 8192 else 16, ctx, only_attention=True)["attention"]
     pre, flops = time_prefill_attention(ops, torch, dev, PROMPT_LEN)
     rec["like_prefill_attention"] = {"us": pre["paged_prefill_tc_kernel"]["us"], "frac": round(pre["paged_prefill_tc_kernel"]["tflops"] / _tensor_peak(), 3)}
     print(json.dumps(rec), file=out)

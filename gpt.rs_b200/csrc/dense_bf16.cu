@@ -4,7 +4,7 @@
 // past the end zero-filled by the copy engine. Two kernels share that plan:
 //   dense_rows_kernel      more than 128 rows (prompts): persistent CTAs walk over 128 x BN output tiles, x rows are the M side
 //                          of the MMA. Warp 5 requests stages, warp 4 issues the MMAs into one of two accumulators in tensor
-//                          memory while warps 0-3 (thread = row) turn the other one into bias + activation + stores.
+//                          memory while warps 0-3 and 8-11 (thread = row, half of the columns) turn the other one into bias + activation + stores.
 //   dense_channels_kernel  up to 128 rows (decode steps): 128 output channels are the M side, the rows the N side (16 .. 128);
 //                          the weights of the first stages are requested before griddepcontrol.wait; K is split over a thread
 //                          block cluster and the partial tiles meet in the owner's shared memory (matmul_common.cuh).
@@ -42,8 +42,10 @@ struct RowsParams {
     int64_t ldy, y_step;
 };
 
-template <int BN, int STAGES>
-__global__ void __launch_bounds__(192, 1) dense_rows_kernel(const __grid_constant__ RowsParams p) {
+constexpr int kRowsThreads = 384;    // warps 0-3 and 8-11 epilogue, 4 MMA + tensor memory, 5 loader
+// ACT: 0 none, 1 xIELU, 2 whatever p.act says (with a soft cap)
+template <int BN, int STAGES, int ACT>
+__global__ void __launch_bounds__(kRowsThreads, 1) dense_rows_kernel(const __grid_constant__ RowsParams p) {
     constexpr int kStageBytes = kATile + BN * 128;
     constexpr uint32_t kCols = 2 * BN < 32 ? 32 : 2 * BN;
     constexpr uint32_t kIdesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(BN >> 3) << 17) | ((uint32_t)(kTileM >> 4) << 24);
@@ -54,7 +56,7 @@ __global__ void __launch_bounds__(192, 1) dense_rows_kernel(const __grid_constan
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     if (tid == 0) {
         for (int s = 0; s < STAGES; ++s) { mbar_init(&full[s], 1); mbar_init(&empty[s], 1); }
-        for (int i = 0; i < 2; ++i) { mbar_init(&acc_full[i], 1); mbar_init(&acc_empty[i], 128); }
+        for (int i = 0; i < 2; ++i) { mbar_init(&acc_full[i], 1); mbar_init(&acc_empty[i], 256); }
         mbar_fence_init();
     }
     if (warp == 4) tmem_alloc(&tmem_holder, kCols);
@@ -112,19 +114,20 @@ __global__ void __launch_bounds__(192, 1) dense_rows_kernel(const __grid_constan
                 __syncwarp();
             }
         }
-    } else {
+    } else if (warp < 4 || warp >= 8) {
+        const int quarter = warp & 3, c_lo = warp < 4 ? 0 : BN / 2;   // lane quarter and half of the columns
         int n = 0;
         for (int t = blockIdx.x; t < tiles && !failed; t += gridDim.x, ++n) {
             const int buf = n & 1;
             const int m0 = (t % p.m_tiles) * kTileM, rest = t / p.m_tiles, n0 = (rest % p.n_tiles) * BN, b = rest / p.n_tiles;
             if (!wait(&acc_full[buf], (uint32_t)(n / 2) & 1u)) break;
             tc_fence_after();
-            const int m = m0 + warp * 32 + lane;
+            const int m = m0 + quarter * 32 + lane;
             const int64_t row = b * p.y_step + (int64_t)m * p.ldy;
 #pragma unroll 1
-            for (int c0 = 0; c0 < BN && n0 + c0 < p.N; c0 += 32) {
+            for (int c0 = c_lo; c0 < c_lo + BN / 2 && n0 + c0 < p.N; c0 += 32) {
                 float v[32];
-                tmem_ld_32(tmem + ((uint32_t)(warp * 32) << 16) + (uint32_t)(buf * BN + c0), v);
+                tmem_ld_32(tmem + ((uint32_t)(quarter * 32) << 16) + (uint32_t)(buf * BN + c0), v);
                 const int left = p.N - (n0 + c0);   // a multiple of 8
                 if (p.bias) {
 #pragma unroll
@@ -134,15 +137,12 @@ __global__ void __launch_bounds__(192, 1) dense_rows_kernel(const __grid_constan
                             v[4 * i] += bb.x; v[4 * i + 1] += bb.y; v[4 * i + 2] += bb.z; v[4 * i + 3] += bb.w;
                         }
                 }
-                if (p.act.softcap > 0.f) {
-#pragma unroll 4
-                    for (int i = 0; i < 32; ++i) v[i] = dense_act<true>(p.act, v[i]);
-                } else if (p.act.kind == 1) {
+                if constexpr (ACT == 1) {
 #pragma unroll
-                    for (int i = 0; i < 32; ++i) {
-                        const float e = expm1_minus_fast(fminf(v[i], 0.f));
-                        v[i] = v[i] > 0.f ? fmaf(p.act.pos * v[i], v[i], 0.5f * v[i]) : fmaf(p.act.neg, e, 0.5f * v[i]);
-                    }
+                    for (int i = 0; i < 32; ++i) v[i] = dense_act<true>({1, p.act.pos, p.act.neg, 0.f}, v[i]);
+                } else if constexpr (ACT == 2) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) v[i] = dense_act<true>(p.act, v[i]);
                 }
                 if (m < p.M) {
                     if (p.out_f32) {
@@ -321,10 +321,12 @@ int launch_rows(const Call& c, cudaStream_t st) {
     p.x_step = (int)c.x_step; p.w_rows = c.N; p.ldy = c.ldy; p.y_step = c.y_step;
     const int64_t tiles = (int64_t)p.m_tiles * p.n_tiles * p.batch;
     constexpr size_t smem = (size_t)STAGES * (kATile + BN * 128) + 1024;
-    void (*kern)(RowsParams) = dense_rows_kernel<BN, STAGES>;
+    void (*kerns[3])(RowsParams) = {dense_rows_kernel<BN, STAGES, 0>, dense_rows_kernel<BN, STAGES, 1>, dense_rows_kernel<BN, STAGES, 2>};
     static PerDeviceOnce attr_once;
-    if (attr_once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    return launch_kernel(kern, dim3((unsigned)(tiles < sm_count() ? tiles : sm_count())), dim3(192), smem, st, 1, p);
+    if (attr_once.first_time())
+        for (auto k : kerns) GPTRS_CUDA_OK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    const auto kern = kerns[c.ep->softcap > 0.f ? 2 : c.ep->act];
+    return launch_kernel(kern, dim3((unsigned)(tiles < sm_count() ? tiles : sm_count())), dim3(kRowsThreads), smem, st, 1, p);
 }
 
 template <int BN, int STAGES>

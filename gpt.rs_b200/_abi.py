@@ -62,8 +62,48 @@ class DenseEpilogue(ctypes.Structure):
         ("out_dtype", ctypes.c_int), ("d_bias", ctypes.c_void_p), ("act", ctypes.c_int), ("act_pos", ctypes.c_float), ("act_neg", ctypes.c_float),
         ("softcap", ctypes.c_float), ("ldx", ctypes.c_int64), ("ldy", ctypes.c_int64), ("batch", ctypes.c_int64), ("x_step", ctypes.c_int64),
         ("y_step", ctypes.c_int64), ("d_best_val", ctypes.c_void_p), ("d_best_idx", ctypes.c_void_p), ("skip_store", ctypes.c_int),
-        ("d_status", ctypes.c_void_p),
+        ("d_status", ctypes.c_void_p), ("d_tiles", ctypes.c_void_p), ("d_n_tiles", ctypes.c_void_p), ("max_tiles", ctypes.c_int64),
+        ("tile_rows", ctypes.c_int64), ("swiglu", ctypes.c_int),
     ]
+
+
+class NormStep(ctypes.Structure):
+    """gptrs_norm_step."""
+    _fields_ = [
+        ("d_x", ctypes.c_void_p), ("d_y", ctypes.c_void_p), ("y_dtype", ctypes.c_int), ("ldy", ctypes.c_int64), ("d_pair", ctypes.c_void_p),
+        ("d_pair_weight", ctypes.c_void_p), ("top", ctypes.c_int64), ("d_embed", ctypes.c_void_p), ("d_pos_embed", ctypes.c_void_p),
+        ("d_tokens", ctypes.c_void_p), ("d_pos", ctypes.c_void_p), ("vocab", ctypes.c_int64), ("positions", ctypes.c_int64), ("d_gamma_out", ctypes.c_void_p),
+        ("d_gamma_in", ctypes.c_void_p), ("eps", ctypes.c_float), ("d_rows", ctypes.c_void_p), ("d_h", ctypes.c_void_p), ("h_dtype", ctypes.c_int),
+        ("ldh", ctypes.c_int64), ("d_status", ctypes.c_void_p), ("rows", ctypes.c_int64), ("dim", ctypes.c_int64),
+    ]
+
+
+class GroupedAttention(ctypes.Structure):
+    """gptrs_grouped_attention."""
+    _fields_ = [(n, ctypes.c_int) for n in ("dtype", "heads", "kv_heads", "dim", "vdim", "mask", "mask_size")] + \
+        [("scale", ctypes.c_float), ("softcap", ctypes.c_float), ("distance_bias", ctypes.c_int)] + \
+        [(n, ctypes.c_int) for n in ("q_head_stride", "k_offset", "k_head_stride", "v_offset", "v_head_stride", "q_row", "out_head_stride")] + \
+        [("page_bytes", ctypes.c_int64)]
+
+
+class DeltaRule(ctypes.Structure):
+    """gptrs_delta_rule."""
+    _fields_ = [(n, ctypes.c_int) for n in ("dtype", "heads", "kv_heads", "dim", "vdim", "taps", "decay_rank", "gate_rank")] + [("eps", ctypes.c_float)] + \
+        [(n, ctypes.c_int) for n in ("q_offset", "k_offset", "v_offset", "beta_offset", "a_offset", "g_offset", "row", "decay_row", "gate_row",
+                                     "out_head_stride", "conv_channels")] + \
+        [(n, ctypes.c_int64) for n in ("state_floats", "conv_floats", "scratch_floats")]
+
+
+class DeltaStep(ctypes.Structure):
+    """gptrs_delta_step."""
+    _fields_ = [(n, ctypes.c_void_p) for n in ("d_proj", "d_decay", "d_gate", "d_conv", "d_a_log", "d_dt_bias", "d_norm", "d_state", "d_conv_state", "d_slot",
+                                               "d_pos", "d_run_first", "d_run_last", "d_parity", "d_runs")] + \
+        [("n_runs", ctypes.c_int64), ("d_out", ctypes.c_void_p), ("d_scratch", ctypes.c_void_p), ("rows", ctypes.c_int64)]
+
+
+class Moe(ctypes.Structure):
+    """gptrs_moe."""
+    _fields_ = [(n, ctypes.c_int) for n in ("experts", "top", "groups", "keep", "tile_rows")]
 
 
 class ConvStep(ctypes.Structure):

@@ -139,7 +139,8 @@ class CheckpointReader:
 
 
 # "architecture" of a model folder's config.json -> model kind of `engine_config`
-ARCHITECTURES = {"Bevosun": "bevosun"}
+ARCHITECTURES = {"Bevosun": "bevosun", "Felepel": "felepel"}
+LAYERED_KINDS = ("bevosun", "felepel")   # kinds whose layers are configured one by one
 
 
 class ModelFolder:
@@ -301,9 +302,14 @@ def next_namespace() -> int:
     return next(_namespaces)
 
 
-def engine_config(model_config: dict, weight_mode: int = gm.MODE_F32, **engine_kw) -> tuple[gm.ModelConfig, dict | None]:
+def shapes_of(reader) -> dict[str, tuple[int, ...]]:
+    return {e.name: e.dims for e in reader.entries}
+
+
+def engine_config(model_config: dict, weight_mode: int = gm.MODE_F32, shapes: dict | None = None, **engine_kw) -> tuple[gm.ModelConfig, dict | None]:
     """ModelConfig of the engine for a checkpoint's {kind, config} object; also returns the rope
-    scaling object when the tables must come from `rope_tables`."""
+    scaling object when the tables must come from `rope_tables`. `shapes` (of the checkpoint's tensors) gives the sizes that a
+    kind's config leaves to them."""
     kind, c = model_config["kind"], model_config["config"]
     if kind == "gpt":
         d, heads = int(c["embed_dim"]), int(c["num_heads"])
@@ -322,6 +328,8 @@ def engine_config(model_config: dict, weight_mode: int = gm.MODE_F32, **engine_k
         return cfg, (scaling if scaling.get("kind", "none") != "none" else None)
     if kind == "bevosun":
         return bevosun_config(c, weight_mode=weight_mode, **engine_kw), None
+    if kind == "felepel":
+        return felepel_config(c, shapes, weight_mode=weight_mode, **engine_kw), None
     raise BackendError(2, f"model kind {kind!r} is not a decode model of this backend")
 
 
@@ -342,12 +350,52 @@ def bevosun_config(c: dict, context_length: int = 4096, **engine_kw) -> gm.Model
                                   float(c.get("logit_softcap") or 0.0), **engine_kw)
 
 
+def felepel_config(c: dict, shapes: dict | None = None, context_length: int | None = None, **engine_kw) -> gm.ModelConfig:
+    """Felepel's config object -> the layered kind. The ranks of the decay and gate bottlenecks are those of the tensors in `shapes`
+    (a config without tensors may name them in the mixer: decay_rank, gate_rank). The context is bounded by the position table."""
+    layers = []
+    for i, layer in enumerate(c["layers"]):
+        m, mlp, of = layer["mixer"], layer.get("mlp"), layer.get("weights_of")
+        if of is not None and any(layer.get(k) != c["layers"][of].get(k) for k in ("type", "mixer", "mlp")):
+            raise BackendError(1, f"layer {i} reuses the weights of layer {of} but differs from it")
+        kw = dict(heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), mlp=gm.MLP_NONE,
+                  weights_of=-1 if of is None else int(of))
+        if layer["type"] == "attention":
+            mask = m.get("mask")
+            kw.update(mixer=gm.MIXER_GROUPED_ATTENTION, scale=float(m["scale"]), softcap=float(m.get("softcap") or 0.0), distance_bias=1, proj_bias=1,
+                      mask=gm.MASK_CHUNK if mask else gm.MASK_CAUSAL, mask_size=int(mask["size"]) if mask else 0)
+        elif layer["type"] == "channel_delta":
+            owner = f"l{i if of is None else of}.mix."
+
+            def rank(name, key):
+                if shapes and owner + name in shapes:
+                    return int(shapes[owner + name][0])
+                if key in m:
+                    return int(m[key])
+                raise BackendError(1, f"layer {i}: neither a tensor {owner}{name} nor {key} gives the rank of a bottleneck")
+
+            kw.update(mixer=gm.MIXER_CHANNEL_DELTA, taps=int(m["conv"]), decay_rank=rank("a1", "decay_rank"), gate_rank=rank("g1", "gate_rank"))
+        else:
+            raise BackendError(2, f"layer {i}: mixer {layer['type']!r} is not built")
+        if mlp:
+            if mlp.get("kind") != "moe":
+                raise BackendError(2, f"layer {i}: feed-forward {mlp.get('kind')!r} is not built")
+            r = mlp["router"]
+            groups = r.get("groups") or {"count": 1, "keep": 1}
+            kw.update(mlp=gm.MLP_EXPERTS, d_ff=int(mlp["expert"]["ff"]), experts=int(r["experts"]), top=int(r["top"]), groups=int(groups["count"]),
+                      keep=int(groups["keep"]))
+        layers.append(gm.LayerConfig(**kw))
+    positions = int(c["max_positions"])
+    return gm.ModelConfig.layered(layers, int(c["width"]), int(c["vocab"]), min(context_length or positions, positions), float(c["norm"]["eps"]),
+                                  block=gm.BLOCK_SANDWICH, learned_positions=positions, **engine_kw)
+
+
 def load_model(path, weight_mode: int = gm.MODE_F32, namespace: int | None = None, **engine_kw) -> gm.LoadedModel:
     """Opens a checkpoint, creates the engine model it describes and streams every parameter the
     model names to the GPU, one tensor at a time (quantising / repacking on the device when
     `weight_mode` asks for it)."""
     reader = open_model(path)
-    cfg, scaling = engine_config(reader.model_config, weight_mode, **engine_kw)
+    cfg, scaling = engine_config(reader.model_config, weight_mode, shapes_of(reader), **engine_kw)
     ns = next_namespace() if namespace is None else namespace
     model = gm.LoadedModel(cfg, namespace=ns)
     for name, shape in cfg.param_shapes().items():

@@ -50,12 +50,13 @@ def cmd_generate(args) -> int:
     if args.top_k is not None and args.top_k < 1:
         raise SystemExit("--top-k must be at least 1")
     reader = ck.open_model(args.checkpoint)
-    layered = reader.kind == "bevosun"
+    layered = reader.kind in ck.LAYERED_KINDS
     need = len(prompt) + args.max_tokens
-    ctx_cap = need if layered else int(reader.model_config["config"]["context_length"])
+    config = reader.model_config["config"]
+    ctx_cap = int(config.get("max_positions", need)) if layered else int(config["context_length"])
     if need > ctx_cap:
         raise SystemExit(f"prompt + max-tokens = {need} exceeds the model's context_length {ctx_cap}")
-    kw = dict(context_length=ctx_cap) if layered else {}
+    kw = dict(context_length=need) if layered else {}
     kw.update(max_seqs=1, max_tokens=min(max(len(prompt), 16), 1024), max_logit_rows=1, use_pdl=1)
     if mode != gm.MODE_F32 or layered:
         pages = (need + 15) // 16 + 1
@@ -152,7 +153,7 @@ def main(argv=None) -> int:
     g.add_argument("--top-k", type=int, default=None)
     g.add_argument("--seed", type=int, default=0)
     g.add_argument("--weight-mode", default="f32", choices=["f32", "w4a16", "w8a16", "bf16"],
-                   help="w4a16 / w8a16 quantise the linear weights on the device while loading (ministral kind); bf16: bevosun kind")
+                   help="w4a16 / w8a16 quantise the linear weights on the device while loading (ministral kind); bf16: the layered kinds, bevosun and felepel")
     g.add_argument("--no-graph", action="store_true", help="launch kernels one by one instead of replaying a CUDA graph")
     g.set_defaults(fn=cmd_generate)
     i = sub.add_parser("inspect", help="print the config and tensor index of a checkpoint")
@@ -160,7 +161,7 @@ def main(argv=None) -> int:
     i.set_defaults(fn=cmd_inspect)
     x = sub.add_parser("export-random", help="write a checkpoint with random weights for a config")
     x.add_argument("--out", required=True)
-    x.add_argument("--kind", required=True, choices=["gpt", "ministral", "bevosun"])
+    x.add_argument("--kind", required=True, choices=["gpt", "ministral", "bevosun", "felepel"])
     x.add_argument("--config", required=True, help="the model's config JSON object")
     x.add_argument("--seed", type=int, default=0)
     x.add_argument("--std", type=float, default=0.02)

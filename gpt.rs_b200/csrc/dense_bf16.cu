@@ -40,11 +40,14 @@ struct RowsParams {
     int m_tiles, n_tiles;
     int x_step, w_rows;          // x columns between batches; weight rows between batches
     int64_t ldy, y_step;
+    const gptrs_row_tile* tiles; // grouped form
+    const int* n_row_tiles;
 };
 
 constexpr int kRowsThreads = 384;    // warps 0-3 and 8-11 epilogue, 4 MMA + tensor memory, 5 loader
-// ACT: 0 none, 1 xIELU, 2 whatever p.act says (with a soft cap)
-template <int BN, int STAGES, int ACT>
+// ACT: 0 none, 1 xIELU, 2 whatever p.act says (with a soft cap), 3 silu(gate) partner (8 gates, then their 8 partners).
+// GROUPED: the row tiles come from a list in device memory, each with the weight matrix that it meets.
+template <int BN, int STAGES, int ACT, bool GROUPED = false>
 __global__ void __launch_bounds__(kRowsThreads, 1) dense_rows_kernel(const __grid_constant__ RowsParams p) {
     constexpr int kStageBytes = kATile + BN * 128;
     constexpr uint32_t kCols = 2 * BN < 32 ? 32 : 2 * BN;
@@ -67,25 +70,37 @@ __global__ void __launch_bounds__(kRowsThreads, 1) dense_rows_kernel(const __gri
     pdl_launch_dependents();
     pdl_wait();
     const int n_k = (p.K + kBK - 1) / kBK;
-    const int tiles = p.m_tiles * p.n_tiles * p.batch;
+    const int tiles = GROUPED ? *p.n_row_tiles * p.n_tiles : p.m_tiles * p.n_tiles * p.batch;
     bool failed = false;
+    struct Tile { int m0, m_end, n0, b; };
+    auto tile_of = [&](int t) {
+        Tile r;
+        if constexpr (GROUPED) {   // column tile fastest: the rows are read once, an expert's weights stay in L2 for its row tiles
+            const gptrs_row_tile g = p.tiles[t / p.n_tiles];
+            r = {g.row0, g.row0 + g.rows, (t % p.n_tiles) * BN, g.group};
+        } else {                   // row tile fastest, so that the CTAs running at one time share weight tiles
+            const int rest = t / p.m_tiles;
+            r = {(t % p.m_tiles) * kTileM, p.M, (rest % p.n_tiles) * BN, rest / p.n_tiles};
+        }
+        return r;
+    };
     auto wait = [&](uint64_t* bar, uint32_t parity) {
         if (!failed && !mbar_wait_relaxed(bar, parity)) failed = true;
         failed = __any_sync(0xffffffffu, failed);
         return !failed;
     };
-    // tile -> (row tile fastest, so that the CTAs running at one time share weight tiles)
     if (warp == 5) {
         int it = 0, last_it = 0;
         for (int t = blockIdx.x; t < tiles && !failed; t += gridDim.x) {
-            const int m0 = (t % p.m_tiles) * kTileM, rest = t / p.m_tiles, n0 = (rest % p.n_tiles) * BN, b = rest / p.n_tiles;
+            const Tile tl = tile_of(t);
+            const int m0 = tl.m0, n0 = tl.n0, b = tl.b;
             for (int k = 0; k < n_k; ++k, ++it) {
                 const int s = it % STAGES;
                 if (it >= STAGES && !wait(&empty[s], (uint32_t)(it / STAGES - 1) & 1u)) break;
                 if (lane == 0) {
                     const uint32_t bar = smem_u32(&full[s]);
                     mbar_expect_tx_addr(bar, kStageBytes);
-                    tma_load_2d(smem + s * kStageBytes, &p.x_map, b * p.x_step + k * kBK, m0, bar);
+                    tma_load_2d(smem + s * kStageBytes, &p.x_map, (GROUPED ? 0 : b * p.x_step) + k * kBK, m0, bar);
                     tma_load_2d(smem + s * kStageBytes + kATile, &p.w_map, k * kBK, b * p.w_rows + n0, bar);
                 }
                 __syncwarp();
@@ -119,11 +134,12 @@ __global__ void __launch_bounds__(kRowsThreads, 1) dense_rows_kernel(const __gri
         int n = 0;
         for (int t = blockIdx.x; t < tiles && !failed; t += gridDim.x, ++n) {
             const int buf = n & 1;
-            const int m0 = (t % p.m_tiles) * kTileM, rest = t / p.m_tiles, n0 = (rest % p.n_tiles) * BN, b = rest / p.n_tiles;
+            const Tile tl = tile_of(t);
+            const int m0 = tl.m0, n0 = tl.n0;
             if (!wait(&acc_full[buf], (uint32_t)(n / 2) & 1u)) break;
             tc_fence_after();
             const int m = m0 + quarter * 32 + lane;
-            const int64_t row = b * p.y_step + (int64_t)m * p.ldy;
+            const int64_t row = (GROUPED ? 0 : tl.b * p.y_step) + (int64_t)m * p.ldy;
 #pragma unroll 1
             for (int c0 = c_lo; c0 < c_lo + BN / 2 && n0 + c0 < p.N; c0 += 32) {
                 float v[32];
@@ -144,7 +160,22 @@ __global__ void __launch_bounds__(kRowsThreads, 1) dense_rows_kernel(const __gri
 #pragma unroll
                     for (int i = 0; i < 32; ++i) v[i] = dense_act<true>(p.act, v[i]);
                 }
-                if (m < p.M) {
+                if constexpr (ACT == 3) {
+                    if (m < tl.m_end) {
+                        float o[16];
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) {
+                            const float gt = v[(i >> 3) * 16 + (i & 7)];
+                            o[i] = __fdividef(gt, 1.f + __expf(-gt)) * v[(i >> 3) * 16 + (i & 7) + 8];
+                        }
+                        uint4* dst = reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(p.y) + row + ((n0 + c0) >> 1));
+#pragma unroll
+                        for (int i = 0; i < 2; ++i)
+                            if (16 * i < left)
+                                dst[i] = make_uint4(pack_bf16x2(o[8 * i], o[8 * i + 1]), pack_bf16x2(o[8 * i + 2], o[8 * i + 3]),
+                                                    pack_bf16x2(o[8 * i + 4], o[8 * i + 5]), pack_bf16x2(o[8 * i + 6], o[8 * i + 7]));
+                    }
+                } else if (m < tl.m_end) {
                     if (p.out_f32) {
                         float4* dst = reinterpret_cast<float4*>(static_cast<float*>(p.y) + row + n0 + c0);
 #pragma unroll
@@ -177,10 +208,12 @@ struct ChannelsParams {
     int batch_m_tiles;           // row tiles per batch entry (blockIdx.z = batch * row tiles + row tile)
     int x_step, w_rows;
     int64_t y_step;
+    const gptrs_row_tile* tiles; // grouped form: blockIdx.z counts the row tiles of the list
+    const int* n_row_tiles;
 };
 constexpr int kChThreads = 320;  // warps 0-7 epilogue, 8 loader, 9 MMA + tensor memory
 
-template <int BN, int STAGES>
+template <int BN, int STAGES, bool GROUPED = false>
 __global__ void __launch_bounds__(kChThreads, BN <= 64 ? 2 : 1) dense_channels_kernel(const __grid_constant__ ChannelsParams cp) {
     constexpr int kStageBytes = kATile + BN * 128;
     constexpr uint32_t kCols = BN < 32 ? 32 : BN;
@@ -192,7 +225,15 @@ __global__ void __launch_bounds__(kChThreads, BN <= 64 ? 2 : 1) dense_channels_k
     unsigned char* smem = smem_raw + ((1024 - (smem_u32(smem_raw) & 1023)) & 1023);
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     MatmulParams p = cp.p;
-    const int b = blockIdx.z / cp.batch_m_tiles, m0 = (blockIdx.z % cp.batch_m_tiles) * BN, n0 = blockIdx.x * kTileM;
+    int b = blockIdx.z / cp.batch_m_tiles, m0 = (blockIdx.z % cp.batch_m_tiles) * BN;
+    const int n0 = blockIdx.x * kTileM;
+    if constexpr (GROUPED) {   // which weights to read is a result of the kernels in front
+        pdl_wait();
+        if ((int)blockIdx.z >= *cp.n_row_tiles) return;   // the whole cluster
+        const gptrs_row_tile t = cp.tiles[blockIdx.z];
+        b = t.group; m0 = t.row0;
+        p.M = t.row0 + t.rows;
+    }
     SplitReduce sr;
     sr.begin(p, false);
     const int k_tiles = (p.K + kBK - 1) / kBK;
@@ -219,7 +260,7 @@ __global__ void __launch_bounds__(kChThreads, BN <= 64 ? 2 : 1) dense_channels_k
     tc_fence_after();
     const uint32_t tmem = tmem_holder;
     pdl_launch_dependents();   // every CTA of this grid holds its tensor memory before a dependent grid may start
-    pdl_wait();
+    if constexpr (!GROUPED) pdl_wait();
     bool failed = false;
     if (warp == 8) {
         for (int it = 0; it < n_k; ++it) {
@@ -231,7 +272,7 @@ __global__ void __launch_bounds__(kChThreads, BN <= 64 ? 2 : 1) dense_channels_k
                     mbar_expect_tx_addr(bar, kStageBytes);
                     tma_load_2d(smem + s * kStageBytes, &cp.w_map, (k0 + it) * kBK, b * cp.w_rows + n0, bar);
                 }
-                tma_load_2d(smem + s * kStageBytes + kATile, &cp.x_map, b * cp.x_step + (k0 + it) * kBK, m0, bar);
+                tma_load_2d(smem + s * kStageBytes + kATile, &cp.x_map, (GROUPED ? 0 : b * cp.x_step) + (k0 + it) * kBK, m0, bar);
             }
             __syncwarp();
         }
@@ -282,8 +323,10 @@ __global__ void __launch_bounds__(kChThreads, BN <= 64 ? 2 : 1) dense_channels_k
     tc_fence_before();
     __syncthreads();
     if (warp == 9) tmem_free(tmem, kCols);
-    if (p.out_f32) p.y = static_cast<float*>(p.y) + b * cp.y_step;
-    else p.y = static_cast<__nv_bfloat16*>(p.y) + b * cp.y_step;
+    if constexpr (!GROUPED) {
+        if (p.out_f32) p.y = static_cast<float*>(p.y) + b * cp.y_step;
+        else p.y = static_cast<__nv_bfloat16*>(p.y) + b * cp.y_step;
+    }
     split_reduce_finish<BN, true>(p, sr, slots, tid, kChThreads, m0, n0);
 }
 
@@ -319,13 +362,15 @@ int launch_rows(const Call& c, cudaStream_t st) {
     p.M = c.M; p.N = c.N; p.K = c.K; p.batch = c.batch; p.out_f32 = c.ep->out_dtype == GPTRS_F32;
     p.m_tiles = ceil_div(c.M, kTileM); p.n_tiles = ceil_div(c.N, BN);
     p.x_step = (int)c.x_step; p.w_rows = c.N; p.ldy = c.ldy; p.y_step = c.y_step;
-    const int64_t tiles = (int64_t)p.m_tiles * p.n_tiles * p.batch;
+    p.tiles = c.ep->d_tiles; p.n_row_tiles = c.ep->d_n_tiles;
+    const int64_t tiles = (p.tiles ? c.ep->max_tiles : (int64_t)p.m_tiles * p.batch) * p.n_tiles;
     constexpr size_t smem = (size_t)STAGES * (kATile + BN * 128) + 1024;
-    void (*kerns[3])(RowsParams) = {dense_rows_kernel<BN, STAGES, 0>, dense_rows_kernel<BN, STAGES, 1>, dense_rows_kernel<BN, STAGES, 2>};
+    void (*kerns[5])(RowsParams) = {dense_rows_kernel<BN, STAGES, 0>, dense_rows_kernel<BN, STAGES, 1>, dense_rows_kernel<BN, STAGES, 2>,
+                                    dense_rows_kernel<BN, STAGES, 0, true>, dense_rows_kernel<BN, STAGES, 3, true>};
     static PerDeviceOnce attr_once;
     if (attr_once.first_time())
         for (auto k : kerns) GPTRS_CUDA_OK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    const auto kern = kerns[c.ep->softcap > 0.f ? 2 : c.ep->act];
+    const auto kern = kerns[p.tiles ? (c.ep->swiglu ? 4 : 3) : c.ep->softcap > 0.f ? 2 : c.ep->act];
     return launch_kernel(kern, dim3((unsigned)(tiles < sm_count() ? tiles : sm_count())), dim3(kRowsThreads), smem, st, 1, p);
 }
 
@@ -342,9 +387,13 @@ int launch_channels(const Call& c, cudaStream_t st) {
     p.ldy = c.ldy;
     p.best_val = c.ep->d_best_val; p.best_idx = c.ep->d_best_idx; p.skip_store = c.ep->skip_store;
     cp.batch_m_tiles = ceil_div(c.M, BN);
+    cp.tiles = c.ep->d_tiles; cp.n_row_tiles = c.ep->d_n_tiles;
+    p.swiglu = c.ep->swiglu;
+    const int64_t z = cp.tiles ? c.ep->max_tiles : (int64_t)cp.batch_m_tiles * c.batch;
+    GPTRS_REQUIRE(z <= 65535, "dense bf16 matmul: too many row tiles in one launch");
     cp.x_step = (int)c.x_step; cp.w_rows = c.N; cp.y_step = c.y_step;
     const int n_tiles = ceil_div(c.N, kTileM), k_tiles = ceil_div(c.K, kBK);
-    const int64_t ctas = (int64_t)n_tiles * cp.batch_m_tiles * c.batch;
+    const int64_t ctas = (int64_t)n_tiles * z;
     // fill the SMs (two CTAs each up to 64 rows) with at least two stages of K per CTA; clusters above 4 pack badly once
     // most of the slots are taken
     const int64_t slots = (int64_t)sm_count() * (BN <= 64 ? 2 : 1);
@@ -354,10 +403,11 @@ int launch_channels(const Call& c, cudaStream_t st) {
     while (split > 3 && ctas * split * 100 > slots * 85) --split;
     p.n_split = (int)(split < 1 ? 1 : split);
     constexpr size_t smem = (size_t)STAGES * (kATile + BN * 128) + 1024;
-    void (*kern)(ChannelsParams) = dense_channels_kernel<BN, STAGES>;
+    void (*kerns[2])(ChannelsParams) = {dense_channels_kernel<BN, STAGES>, dense_channels_kernel<BN, STAGES, true>};
     static PerDeviceOnce attr_once;
-    if (attr_once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    return launch_kernel(kern, dim3((unsigned)n_tiles, (unsigned)p.n_split, (unsigned)(cp.batch_m_tiles * c.batch)), dim3(kChThreads), smem, st, p.n_split, cp);
+    if (attr_once.first_time())
+        for (auto k : kerns) GPTRS_CUDA_OK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    return launch_kernel(kerns[cp.tiles ? 1 : 0], dim3((unsigned)n_tiles, (unsigned)p.n_split, (unsigned)z), dim3(kChThreads), smem, st, p.n_split, cp);
 }
 
 }  // namespace
@@ -371,15 +421,27 @@ extern "C" int gptrs_cuda_dense_bf16(const void* d_x, const void* d_w, void* d_y
     GPTRS_REQUIRE(m >= 0 && n > 0 && k > 0 && m < (1ll << 30) && n < (1ll << 30) && k < (1ll << 30), "bad shape");
     Call c = {d_x, d_w, d_y, (int)m, (int)n, (int)k, ep->batch > 1 ? (int)ep->batch : 1, ep->ldx ? ep->ldx : k, ep->ldy ? ep->ldy : n,
               ep->x_step, ep->y_step, ep};
+    if (ep->swiglu && !ep->ldy) c.ldy = n / 2;
     GPTRS_REQUIRE(((n | k | c.ldx | c.ldy | c.x_step | c.y_step) & 7) == 0, "dense bf16 matmul: sizes, strides and steps must be multiples of 8");
     GPTRS_REQUIRE(((reinterpret_cast<uintptr_t>(d_x) | reinterpret_cast<uintptr_t>(d_w) | reinterpret_cast<uintptr_t>(d_y)) & 15) == 0, "16-byte alignment");
-    GPTRS_REQUIRE(c.ldx >= k && c.ldy >= n && c.ldx < (1ll << 30), "row strides shorter than the rows");
-    GPTRS_REQUIRE((int64_t)c.batch * n < (1ll << 31) && (c.batch == 1 || (c.x_step > 0 && c.y_step > 0)), "batch");
+    GPTRS_REQUIRE(c.ldx >= k && c.ldy >= (ep->swiglu ? n / 2 : n) && c.ldx < (1ll << 30), "row strides shorter than the rows");
+    GPTRS_REQUIRE((int64_t)c.batch * n < (1ll << 31) && (c.batch == 1 || ep->d_tiles || (c.x_step > 0 && c.y_step > 0)), "batch");
     GPTRS_REQUIRE(ep->out_dtype == GPTRS_BF16 || ep->out_dtype == GPTRS_F32, "out_dtype must be bf16 or f32");
     GPTRS_REQUIRE(ep->act == 0 || ep->act == 1, "activation: 0 none, 1 xIELU");
     GPTRS_REQUIRE(!ep->d_best_val || (m <= 128 && c.batch == 1 && ep->out_dtype == GPTRS_F32 && ep->d_best_idx), "fused greedy head: up to 128 rows, f32");
+    GPTRS_REQUIRE(!ep->swiglu || (ep->d_tiles && ep->out_dtype == GPTRS_BF16 && n % 16 == 0 && c.ldy == n / 2), "swiglu: grouped form, compact bf16 output");
     if (m == 0) return GPTRS_OK;
     cudaStream_t st = as_stream(stream);
+    if (ep->d_tiles) {
+        GPTRS_REQUIRE(ep->d_n_tiles && ep->max_tiles > 0 && !ep->d_bias && !ep->act && ep->softcap == 0.f && !ep->d_best_val, "grouped form: tile list, no other epilogue");
+        if (ep->tile_rows == 16) return launch_channels<16, 5>(c, st);
+        if (ep->tile_rows == 32) return launch_channels<32, 5>(c, st);
+        if (ep->tile_rows == 64) return launch_channels<64, 4>(c, st);
+        GPTRS_REQUIRE(ep->tile_rows == kTileM, "grouped form: tiles of 16, 32, 64 or 128 rows");
+        if (n <= 64) return launch_rows<64, 8>(c, st);
+        if (n > 128 && ep->max_tiles * ceil_div(n, 256) >= sm_count()) return launch_rows<256, 4>(c, st);
+        return launch_rows<128, 6>(c, st);
+    }
     if (m <= 16) return launch_channels<16, 5>(c, st);
     if (m <= 32) return launch_channels<32, 5>(c, st);
     if (m <= 64) return launch_channels<64, 4>(c, st);

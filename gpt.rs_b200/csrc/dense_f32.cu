@@ -38,10 +38,13 @@ struct SgemmParams {
     int64_t ldx, ldy, x_step, y_step;
     int m_tiles;
     DenseAct dense;
+    const gptrs_row_tile* tiles;   // grouped form: blockIdx.z counts the row tiles of the list
+    const int* n_row_tiles;
 };
 
 template <int MT>
-__global__ void __launch_bounds__(kSgWarps * 32) sgemm_smallm_kernel(const SgemmParams p) {
+__global__ void __launch_bounds__(kSgWarps * 32) sgemm_smallm_kernel(const SgemmParams pp) {
+    SgemmParams p = pp;
     extern __shared__ __align__(16) float sg_smem[];
     float* xs = sg_smem;                          // [MT][k_per_cta]
     float* red = sg_smem + MT * p.k_per_cta;      // [warps][MT][128]
@@ -49,12 +52,17 @@ __global__ void __launch_bounds__(kSgWarps * 32) sgemm_smallm_kernel(const Sgemm
     const int col0 = blockIdx.x * kSgCols + lane;
     const int kb = blockIdx.y * p.k_per_cta;
     const int kn = min(p.k_per_cta, p.K - kb);
-    const int m0 = (blockIdx.z % p.m_tiles) * MT, batch = blockIdx.z / p.m_tiles;
-    const float* px = p.x + batch * p.x_step;
-    const float* pw = p.w + (size_t)batch * p.K * p.N;
+    int m0 = (blockIdx.z % p.m_tiles) * MT, batch = blockIdx.z / p.m_tiles;
 
     pdl_launch_dependents();  // dependents still wait for this whole grid before reading its results
     pdl_wait();
+    if (p.tiles) {
+        if ((int)blockIdx.z >= *p.n_row_tiles) return;   // the whole cluster
+        const gptrs_row_tile t = p.tiles[blockIdx.z];
+        m0 = t.row0; batch = t.group; p.M = t.row0 + t.rows;
+    }
+    const float* px = p.x + batch * p.x_step;
+    const float* pw = p.w + (size_t)batch * p.K * p.N;
     if (p.norm_kind == 0) {
         for (int i = tid; i < MT * kn; i += kSgWarps * 32) {
             int m = i / kn, k = i % kn;
@@ -329,8 +337,9 @@ int launch_sgemm(SgemmParams p, int batch, cudaStream_t st) {
     void (*kern)(SgemmParams) = sgemm_smallm_kernel<MT>;
     GPTRS_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     p.m_tiles = ceil_div(p.M, MT);
-    if ((int64_t)p.m_tiles * batch > 65535) return fail(GPTRS_UNIMPLEMENTED, "f32 matmul: too many rows in one launch");
-    dim3 grid(n_blocks, p.n_split, p.m_tiles * batch);
+    const int64_t z = p.tiles ? batch : (int64_t)p.m_tiles * batch;   // grouped form: `batch` is the most tiles there can be
+    if (z > 65535) return fail(GPTRS_UNIMPLEMENTED, "f32 matmul: too many rows in one launch");
+    dim3 grid(n_blocks, p.n_split, (unsigned)z);
     return launch_kernel(kern, grid, dim3(kSgWarps * 32), smem, st, p.n_split, p);
 }
 
@@ -381,6 +390,12 @@ int gptrs_cuda_dense_f32(const float* d_x, const float* d_w, float* d_y, int64_t
     p.ldx = ep->ldx ? ep->ldx : k; p.ldy = ep->ldy ? ep->ldy : n;
     p.x_step = ep->x_step; p.y_step = ep->y_step;
     p.dense = {ep->act, ep->act_pos, ep->act_neg, ep->softcap};
+    if (ep->d_tiles) {
+        GPTRS_REQUIRE(ep->d_n_tiles && ep->max_tiles > 0 && ep->tile_rows == 8 && !ep->d_bias && !ep->swiglu, "grouped form: tile list with tiles of 8 rows, no bias");
+        p.tiles = ep->d_tiles; p.n_row_tiles = ep->d_n_tiles;
+        p.x_step = p.y_step = 0;
+        return launch_sgemm<8>(p, (int)ep->max_tiles, as_stream(stream));
+    }
     return run_sgemm(p, ep->batch > 1 ? (int)ep->batch : 1, as_stream(stream));
 }
 

@@ -588,11 +588,10 @@ int enqueue_forward(Model& m, int T, int max_ctx, int chunk_pages, int n_rows, b
     return launch_kernel(tp_pick_kernel, dim3((n_rows + 127) / 128), dim3(128), 0, st, 1, pp);
 }
 
-// Pages that no layer's window reaches from position `next_pos` on go back to the pool (models with windows in every layer).
+// Pages that no layer's mask reaches from position `next_pos` on go back to the pool.
 void release_passed_pages(Model& m, int slot, int next_pos) {
     if (!m.layered()) return;
-    const int first_visible = std::max(0, next_pos - m.lay->max_window + 1);
-    const int keep = std::min(first_visible / kPage, m.seq_pages[slot]);
+    const int keep = std::min(layered_first_visible(m, next_pos) / kPage, m.seq_pages[slot]);
     for (; m.seq_first_page[slot] < keep; ++m.seq_first_page[slot])
         m.free_pages.push_back(m.h_page_table[(size_t)slot * m.cfg.max_pages_per_seq + m.seq_first_page[slot]]);
 }
@@ -907,24 +906,7 @@ int gptrs_cuda_model_set_layers(gptrs_model* h, const gptrs_layered_config* comm
     Model& m = *reinterpret_cast<Model*>(h);
     GPTRS_REQUIRE(m.layered() && !m.finalized, "per-layer configurations belong to the layered kind, before finalize");
     GPTRS_REQUIRE(n_layers == m.cfg.n_layers, "one configuration per layer");
-    GPTRS_REQUIRE(common->conv_taps >= 1 && common->conv_taps <= 16, "short convolutions of 1 to 16 taps");
-    m.lay->cfg = *common;
-    m.lay->layers.clear();
-    m.lay->layers.resize(n_layers);
-    for (int l = 0; l < n_layers; ++l) {
-        const gptrs_layer_config& c = layers[l];
-        if (c.mixer != GPTRS_MIXER_LATENT_ATTENTION) return fail(GPTRS_UNIMPLEMENTED, "unknown mixer");
-        if (c.mlp != GPTRS_MLP_NONE && c.mlp != GPTRS_MLP_DENSE_XIELU) return fail(GPTRS_UNIMPLEMENTED, "unknown feed-forward kind");
-        GPTRS_REQUIRE(c.mlp == GPTRS_MLP_NONE || c.d_ff > 0, "feed-forward size");
-        LayeredLayer& L = m.lay->layers[l];
-        L.cfg = c;
-        L.att.dtype = m.f32() ? GPTRS_F32 : GPTRS_BF16;
-        L.att.heads = c.heads; L.att.dim = c.dim; L.att.rot_dim = c.rot_dim; L.att.vdim = c.vdim; L.att.kv_rank = c.kv_rank;
-        L.att.window = c.window; L.att.rot_dims = c.rot_dims; L.att.scale = c.scale;
-        int rc = gptrs_cuda_latent_layout(&L.att);
-        if (rc) return rc;
-    }
-    return GPTRS_OK;
+    return layered_set_layers(m, *common, layers);
 }
 
 int gptrs_cuda_debug_layer_residuals(gptrs_model* h, float* h_out) {

@@ -65,16 +65,31 @@ struct DenseWeight {   // [batch][n][k] bf16 with n and k padded to 8, or [batch
     Tensor* bias = nullptr;
     int64_t n = 0, k = 0, batch = 1;
 };
+// What a layer multiplies with; layers that reuse another one's weights share the object.
+struct LayerWeights {
+    Tensor *norm1 = nullptr, *norm2 = nullptr, *norm1b = nullptr, *norm2b = nullptr, *conv1 = nullptr, *conv2 = nullptr, *latent_norm = nullptr;
+    Tensor *r1 = nullptr, *r2 = nullptr;                                                              // distance penalty
+    Tensor *delta_conv = nullptr, *a_log = nullptr, *dt_bias = nullptr, *delta_norm = nullptr;        // delta rule
+    DenseWeight qkv, uk, uv, out, up, down, decay, gate, router;   // up: the experts' gates and ups too
+    float act_pos = 0.f, act_neg = 0.f;
+    ~LayerWeights() {
+        for (Tensor* t : {norm1, norm2, norm1b, norm2b, conv1, conv2, latent_norm, r1, r2, delta_conv, a_log, dt_bias, delta_norm}) tensor_release(t);
+        for (DenseWeight* w : {&qkv, &uk, &uv, &out, &up, &down, &decay, &gate, &router}) { tensor_release(w->w); tensor_release(w->bias); }
+    }
+};
 struct LayeredLayer {
     gptrs_layer_config cfg = {};
-    gptrs_latent_attention att = {};
-    Tensor *norm1 = nullptr, *norm2 = nullptr, *conv1 = nullptr, *conv2 = nullptr, *latent_norm = nullptr;
-    DenseWeight qkv, uk, uv, out, up, down;
-    float act_pos = 0.f, act_neg = 0.f;
+    gptrs_latent_attention att = {};      // the mixer, whichever it is
+    gptrs_grouped_attention gatt = {};
+    gptrs_delta_rule delta = {};
+    gptrs_moe moe = {};
+    std::shared_ptr<LayerWeights> w;
     size_t pool_off = 0;   // byte offset of the layer's pages in Model::kv_pool
-    int rope = 0;          // index into Layered::ropes
+    int rope = -1;         // index into Layered::ropes
     int tiles = -1;        // index into Layered::tile_sets, -1 = plain attention kernel
-    int state1 = 0, state2 = 0;   // convolution states of the two sublayers
+    int state1 = 0, state2 = 0;                      // convolution states of the two sublayers
+    size_t delta_state_off = 0, delta_conv_off = 0;  // floats
+    bool attends() const { return cfg.mixer != GPTRS_MIXER_CHANNEL_DELTA; }
 };
 struct Layered {
     gptrs_layered_config cfg = {};
@@ -88,17 +103,16 @@ struct Layered {
     std::vector<std::unique_ptr<TileSet>> tile_sets;
     int32_t* h_tiles = nullptr;   // pinned staging of one tile list (rows, then counts)
     DevBuf x2, h, qkv, qa, lat, attn, up, y, logits_pad, state, scratch;
-    DevBuf d_run_first, d_run_last, d_parity;
+    DevBuf d_run_first, d_run_last, d_parity, d_runs;
+    DevBuf decay, gate, delta_state, delta_conv, delta_scratch;   // delta rule
+    // experts: logits, sorted rows and what comes of them, the place of every (row, choice) among them, row tiles
+    DevBuf router, sorted, gate_up, expert_y, pair, pair_weight, row_tiles, n_row_tiles, moe_work;
     std::vector<int> parity;      // per slot: the half of the convolution state the next step reads
+    int n_runs = 0;               // runs of the rows that are staged
     std::vector<int32_t> runs;    // host scratch: (first row, rows) of every run of the current call
     size_t state_stride = 0;      // floats of one sublayer's state
-    int max_window = 0;
     float* h_residuals = nullptr; // debug: where the next forward pass leaves the residual stream after every layer
     ~Layered() {
-        for (auto& l : layers) {
-            for (Tensor* t : {l.norm1, l.norm2, l.conv1, l.conv2, l.latent_norm}) tensor_release(t);
-            for (DenseWeight* w : {&l.qkv, &l.uk, &l.uv, &l.out, &l.up, &l.down}) { tensor_release(w->w); tensor_release(w->bias); }
-        }
         tensor_release(embed_norm);
         tensor_release(head.w);
         if (h_tiles) cudaFreeHost(h_tiles);
@@ -216,6 +230,8 @@ int layered_check_config(const gptrs_model_config& c);
 int layered_finalize(Model& m, bool drop_leaves);
 int layered_stage_rows(Model& m, const int32_t* slots, const int32_t* positions, int n);
 int layered_stage_generator(Model& m, int batch);
+int layered_set_layers(Model& m, const gptrs_layered_config& common, const gptrs_layer_config* layers);
+int layered_first_visible(const Model& m, int pos);
 int layered_graph_bucket(const Model& m, int bucket);
 int layered_forward(Model& m, int rows, int max_ctx, int n_rows, bool rows_identity, float temperature, bool skip_logits);
 

@@ -1,7 +1,9 @@
 // Models whose layers are configured one by one (engine kind "layered"): weight packing, cache and state set-up and the forward
-// pass. A layer is a mixer (latent attention over the paged cache, latent_attention.cu) and an optional feed-forward; the step
-// between two sublayers (output norm, residual sum, short convolution with its per-sequence state) is post_norm_conv.cu, the
-// matmuls are dense_bf16.cu or, in f32 mode, dense_f32.cu. Slots, pages, graphs, sampling and the generator are the engine's.
+// pass. A layer is a mixer (latent attention, latent_attention.cu; attention with grouped key / value heads, grouped_attention.cu; a
+// gated delta rule, delta_rule.cu) and an optional feed-forward (dense xIELU; a mixture of experts, moe_route.cu). The step between
+// two sublayers is post_norm_conv.cu (output norm, residual sum, short convolution with its per-sequence state) or norm_step.cu (norms
+// on both sides of a sublayer), the matmuls are dense_bf16.cu or, in f32 mode, dense_f32.cu. Slots, pages, graphs, sampling and the
+// generator are the engine's.
 #include <cmath>
 #include <cstdlib>
 #include <cstring>
@@ -30,6 +32,11 @@ __global__ void pack_kernel(const PackParams p) {
         else static_cast<float*>(p.dst)[at] = v;
     }
 }
+int launch_pack(Model& m, const PackParams& pp) {
+    const int64_t blocks = (pp.total + 255) / 256;
+    pack_kernel<<<(unsigned)(blocks < 4096 ? blocks : 4096), 256, 0, m.stream>>>(pp);
+    return cudaGetLastError() == cudaSuccess ? GPTRS_OK : fail(GPTRS_EXECUTION, "packing a weight failed");
+}
 
 // One block of a source leaf and where it goes in the packed weight: rows n (with a step between batches) and columns k.
 struct Piece {
@@ -38,30 +45,62 @@ struct Piece {
     int64_t row, row_b;         // first output channel in the packed weight, step between batches
     int64_t col, col_b;         // first input column, step between batches
     int64_t mat_b;              // step between batches in whole matrices (1: a batch entry is a matrix of its own)
+    int64_t mat = 0;            // matrix of the first batch entry
 };
+struct Leaf {
+    std::string name;
+    std::vector<int64_t> dims;
+    std::vector<Piece> pieces;
+    std::string bias;           // optional [dims[0]], placed like the pieces' rows
+};
+// a leaf [n][k] whose rows go to the rows from `row` on
+Leaf rows_of(const std::string& name, int64_t n, int64_t k, int64_t row, const std::string& bias = "") {
+    return {name, {n, k}, {{1, n, k, 0, 0, k, 1, row, 0, 0, 0, 0}}, bias};
+}
+// the same in `heads` groups of rows, `stride` rows apart
+Leaf heads_of(const std::string& name, int64_t heads, int64_t n, int64_t k, int64_t row, int64_t stride, const std::string& bias = "") {
+    return {name, {heads * n, k}, {{heads, n, k, 0, n * k, k, 1, row, stride, 0, 0, 0}}, bias};
+}
 
-// Packs the pieces of the leaves `names` (name i holds pieces[i]) into a weight of `batch` matrices n x k: bf16 [n][k] with
-// both sizes padded to 8 and zeros in between, or f32 [k][n]. Memoised by the stable ids of the leaves like every derived layout.
-int pack_weight(Model& m, const std::vector<std::string>& names, const std::vector<std::vector<int64_t>>& dims, const std::vector<std::vector<Piece>>& pieces,
-                int64_t batch, int64_t n, int64_t k, const std::string& bias, const std::string& tag, DenseWeight* w) {
+// Packs the pieces of the leaves into a weight of `batch` matrices n x k: bf16 [n][k] with both sizes padded to 8 and zeros in
+// between, or f32 [k][n]; biases into one vector of n. Memoised by the stable ids of the leaves like every derived layout. The
+// names of the leaves are added to `used`.
+int pack_weight(Model& m, const std::vector<Leaf>& leaves, int64_t batch, int64_t n, int64_t k, const std::string& tag, DenseWeight* w,
+                std::vector<std::string>* used) {
     const bool bf16 = !m.f32();
     w->batch = batch; w->n = bf16 ? pad8(n) : n; w->k = bf16 ? pad8(k) : k;
     int rc = GPTRS_OK;
-    if (!bias.empty()) {
-        Tensor* raw = nullptr;
-        if ((rc = get_raw(m, bias, {n}, &raw))) return rc;
-        int64_t bd[1] = {w->n};
-        if (!(rc = tensor_alloc(GPTRS_F32, 1, bd, true, &w->bias)))
-            if (cudaMemcpy(w->bias->data, raw->data, (size_t)n * 4, cudaMemcpyDeviceToDevice) != cudaSuccess) rc = fail(GPTRS_EXECUTION, "bias copy failed");
-        tensor_release(raw);
-        if (rc) return rc;
+    std::vector<Tensor*> raw(leaves.size(), nullptr);
+    auto drop = [&]() { for (Tensor* t : raw) tensor_release(t); };
+    for (size_t i = 0; i < leaves.size(); ++i) {
+        if ((rc = get_raw(m, leaves[i].name, leaves[i].dims, &raw[i]))) { drop(); return rc; }
+        if (used) used->push_back(leaves[i].name);
     }
-    std::vector<Tensor*> leaves(names.size(), nullptr);
-    auto drop = [&]() { for (Tensor* t : leaves) tensor_release(t); };
-    for (size_t i = 0; i < names.size(); ++i)
-        if ((rc = get_raw(m, names[i], dims[i], &leaves[i]))) { drop(); return rc; }
-    std::pair<uint64_t, uint64_t> key = m.ids[names[0]];
-    for (size_t i = 1; i < names.size(); ++i) { key.first ^= m.ids[names[i]].first * 31; key.second ^= m.ids[names[i]].second * 131; }
+    for (size_t i = 0; i < leaves.size(); ++i) {
+        if (leaves[i].bias.empty()) continue;
+        if (!w->bias) {
+            int64_t bd[1] = {w->n};
+            if ((rc = tensor_alloc(GPTRS_F32, 1, bd, true, &w->bias))) { drop(); return rc; }
+            if (cudaDeviceSynchronize() != cudaSuccess) { drop(); return fail(GPTRS_EXECUTION, "packing a bias failed"); }   // the zero fill is done
+        }
+        Tensor* b = nullptr;
+        if ((rc = get_raw(m, leaves[i].bias, {leaves[i].dims[0]}, &b))) { drop(); return rc; }
+        for (const Piece& p : leaves[i].pieces) {
+            PackParams pp = {};
+            pp.src = static_cast<const float*>(b->data); pp.dst = static_cast<float*>(w->bias->data) + p.row;
+            pp.n = p.n; pp.k = 1; pp.total = p.batch * p.n;
+            pp.sb = p.n; pp.sn = 1; pp.db = p.row_b; pp.dn = 1;
+            if (!rc) rc = launch_pack(m, pp);
+        }
+        if (cudaStreamSynchronize(m.stream) != cudaSuccess && !rc) rc = fail(GPTRS_EXECUTION, "packing a bias failed");
+        tensor_release(b);
+        if (rc) { drop(); return rc; }
+    }
+    std::pair<uint64_t, uint64_t> key = m.ids[leaves[0].name];
+    for (size_t i = 1; i < leaves.size(); ++i) {
+        const auto id = m.ids[leaves[i].name];
+        key.first = key.first * 3 ^ id.first * 31; key.second = key.second * 5 ^ id.second * 131;
+    }
     const auto did = derived_id(key, (bf16 ? "dense_bf16:" : "dense_f32:") + tag + ":" + std::to_string(batch) + "x" + std::to_string(w->n) + "x" + std::to_string(w->k));
     const size_t need = (size_t)batch * w->n * w->k * (bf16 ? 2 : 4);
     if (Tensor* hit = param_lookup(did.first, did.second)) {
@@ -71,20 +110,20 @@ int pack_weight(Model& m, const std::vector<std::string>& names, const std::vect
     int64_t wd[3] = {batch, bf16 ? w->n : w->k, bf16 ? w->k : w->n};
     if ((rc = tensor_alloc(bf16 ? GPTRS_BF16 : GPTRS_F32, 3, wd, true, &w->w))) { drop(); return rc; }
     if (cudaDeviceSynchronize() != cudaSuccess) { drop(); return fail(GPTRS_EXECUTION, "packing a weight failed"); }   // the zero fill is done
-    for (size_t i = 0; i < names.size(); ++i)
-        for (const Piece& p : pieces[i]) {
+    for (size_t i = 0; i < leaves.size() && !rc; ++i)
+        for (const Piece& p : leaves[i].pieces) {
+            if (p.batch * p.n * p.k == 0) continue;
             PackParams pp = {};
             const int64_t dn = bf16 ? w->k : 1, dk = bf16 ? 1 : w->n;
-            pp.src = static_cast<const float*>(leaves[i]->data) + p.src;
-            pp.dst = static_cast<unsigned char*>(w->w->data) + (p.row * dn + p.col * dk) * (bf16 ? 2 : 4);
+            pp.src = static_cast<const float*>(raw[i]->data) + p.src;
+            pp.dst = static_cast<unsigned char*>(w->w->data) + (p.mat * w->n * w->k + p.row * dn + p.col * dk) * (bf16 ? 2 : 4);
             pp.n = p.n; pp.k = p.k; pp.total = p.batch * p.n * p.k;
             pp.sb = p.sb; pp.sn = p.sn; pp.sk = p.sk;
             pp.db = p.row_b * dn + p.col_b * dk + p.mat_b * w->n * w->k; pp.dn = dn; pp.dk = dk;
             pp.bf16 = bf16;
-            const int64_t blocks = (pp.total + 255) / 256;
-            pack_kernel<<<(unsigned)(blocks < 4096 ? blocks : 4096), 256, 0, m.stream>>>(pp);
+            if ((rc = launch_pack(m, pp))) break;
         }
-    if (cudaGetLastError() != cudaSuccess || cudaStreamSynchronize(m.stream) != cudaSuccess) rc = fail(GPTRS_EXECUTION, "packing a weight failed");
+    if (cudaStreamSynchronize(m.stream) != cudaSuccess && !rc) rc = fail(GPTRS_EXECUTION, "packing a weight failed");
     drop();
     if (rc) return rc;
     param_store(did.first, did.second, w->w);
@@ -92,8 +131,8 @@ int pack_weight(Model& m, const std::vector<std::string>& names, const std::vect
     return GPTRS_OK;
 }
 // a plain [out][in] leaf
-int pack_plain(Model& m, const std::string& name, int64_t n, int64_t k, const std::string& bias, DenseWeight* w) {
-    return pack_weight(m, {name}, {{n, k}}, {{{1, n, k, 0, 0, k, 1, 0, 0, 0, 0, 0}}}, 1, n, k, bias, "plain", w);
+int pack_plain(Model& m, const std::string& name, int64_t n, int64_t k, const std::string& bias, DenseWeight* w, std::vector<std::string>* used = nullptr) {
+    return pack_weight(m, {rows_of(name, n, k, 0, bias)}, 1, n, k, "plain", w, used);
 }
 
 // rows of `ld` floats -> rows of `n` (a vocabulary that is no multiple of 8 is computed with padding columns)
@@ -110,8 +149,13 @@ struct DenseOpts {
     float pos = 0.f, neg = 0.f, softcap = 0.f;
     int64_t ldx = 0, ldy = 0, x_step = 0, y_step = 0;
     bool pick = false;
+    // grouped form
+    const gptrs_row_tile* tiles = nullptr;
+    const int32_t* n_tiles = nullptr;
+    int64_t max_tiles = 0, tile_rows = 0;
+    bool swiglu = false;
 };
-int dense(Model& m, const DenseWeight& w, const void* x, void* y, int rows, const DenseOpts& o) {
+int dense(Model& m, const DenseWeight& w, const void* x, void* y, int64_t rows, const DenseOpts& o) {
     ++m.launches;
     gptrs_dense_epilogue ep = {};
     ep.out_dtype = (m.f32() || o.out_f32) ? GPTRS_F32 : GPTRS_BF16;
@@ -120,12 +164,258 @@ int dense(Model& m, const DenseWeight& w, const void* x, void* y, int rows, cons
     ep.ldx = o.ldx; ep.ldy = o.ldy; ep.batch = w.batch; ep.x_step = o.x_step; ep.y_step = o.y_step;
     if (o.pick) { ep.d_best_val = m.best_val.as<float>(); ep.d_best_idx = m.best_idx.as<int32_t>(); ep.skip_store = 1; }
     ep.d_status = m.d_status.as<int32_t>();
+    ep.d_tiles = o.tiles; ep.d_n_tiles = o.n_tiles; ep.max_tiles = o.max_tiles; ep.tile_rows = o.tile_rows; ep.swiglu = o.swiglu;
     if (m.f32())
         return gptrs_cuda_dense_f32(static_cast<const float*>(x), static_cast<const float*>(w.w->data), static_cast<float*>(y), rows, w.n, w.k, &ep, m.stream);
     return gptrs_cuda_dense_bf16(x, w.w->data, y, rows, w.n, w.k, &ep, m.stream);
 }
 
 float softplus(float x) { return x > 20.f ? x : (float)std::log1p(std::exp((double)x)); }
+
+// Rows of a tile of the experts' matmuls for a launch of `rows` rows: small tiles (weights on the M side of the MMA) while an
+// expert has few rows on average, whole 128-row tiles beyond.
+int expert_tile_rows(const Model& m, const gptrs_moe& a, int64_t rows) {
+    if (m.f32()) return 8;
+    const double mean = (double)rows * a.top / a.experts;
+    return mean <= 8 ? 16 : mean <= 24 ? 32 : mean <= 48 ? 64 : 128;
+}
+
+// what the buffers of a forward pass must hold, over all layers (elements per row unless said otherwise)
+struct Widths {
+    int64_t qkv = 0, qa = 0, lat = 0, attn = 0, up = 0, decay = 0, gate = 0;
+    int64_t delta_scratch = 0, router = 0, sorted = 0, expert_up = 0, expert_y = 0, top = 0, work = 0, row_tiles = 0;
+    size_t pool = 0, delta_state = 0, delta_conv = 0;
+    int n_state = 0;
+};
+
+int build_latent(Model& m, LayeredLayer& L, const std::string& x, std::vector<std::string>* used) {
+    const gptrs_latent_attention& a = L.att;
+    LayerWeights& w = *L.w;
+    const int64_t W = m.cfg.d_model, H = a.heads, dim = a.dim, rot = a.rot_dim, rank = a.kv_rank, vd = a.vdim;
+    int rc;
+    if ((rc = get_raw(m, x + "dkv.norm", {rank}, &w.latent_norm))) return rc;
+    // queries and the down-projection in one weight, laid out as the attention kernels expect a projection row
+    if ((rc = pack_weight(m, {{x + "q", {H * (dim + rot), W}, {{H, dim, W, 0, (dim + rot) * W, W, 1, 0, a.q_head_stride, 0, 0, 0},
+                                                              {H, rot, W, dim * W, (dim + rot) * W, W, 1, a.q_rot_offset, a.q_head_stride, 0, 0, 0}}, ""},
+                              {x + "dkv", {rank + rot, W}, {{1, rank, W, 0, 0, W, 1, a.dkv_offset, 0, 0, 0, 0}, {1, rot, W, rank * W, 0, W, 1, a.rot_offset, 0, 0, 0, 0}}, ""}},
+                          1, a.q_row, W, "latent_qkv", &w.qkv, used))) return rc;
+    // absorbed query: per head [rank] <- [dim], the stored key projection transposed
+    if ((rc = pack_weight(m, {{x + "uk", {H * dim, rank}, {{H, rank, dim, 0, dim * rank, 1, rank, 0, 0, 0, 0, 1}}, ""}}, H, rank, dim, "latent_uk", &w.uk, used))) return rc;
+    if ((rc = pack_weight(m, {{x + "uv", {H * vd, rank}, {{H, vd, rank, 0, vd * rank, rank, 1, 0, 0, 0, 0, 1}}, ""}}, H, vd, rank, "latent_uv", &w.uv, used))) return rc;
+    return pack_weight(m, {{x + "o", {W, H * vd}, {{H, W, vd, 0, vd, H * vd, 1, 0, 0, 0, a.out_head_stride, 0}}, ""}}, 1, W, H * a.out_head_stride, "latent_o", &w.out, used);
+}
+
+int build_grouped(Model& m, LayeredLayer& L, const std::string& x, std::vector<std::string>* used) {
+    const gptrs_grouped_attention& a = L.gatt;
+    LayerWeights& w = *L.w;
+    const int64_t W = m.cfg.d_model, H = a.heads, G = a.kv_heads;
+    auto bias = [&](const char* n) { return L.cfg.proj_bias ? x + n + ".b" : std::string(); };
+    int rc;
+    if (a.distance_bias && ((rc = get_raw(m, x + "r1", {H}, &w.r1)) || (rc = get_raw(m, x + "r2", {H}, &w.r2)))) return rc;
+    if ((rc = pack_weight(m, {heads_of(x + "q", H, a.dim, W, 0, a.q_head_stride, bias("q")), heads_of(x + "k", G, a.dim, W, a.k_offset, a.k_head_stride, bias("k")),
+                              heads_of(x + "v", G, a.vdim, W, a.v_offset, a.v_head_stride, bias("v"))}, 1, a.q_row, W, "grouped_qkv", &w.qkv, used))) return rc;
+    return pack_weight(m, {{x + "o", {W, H * a.vdim}, {{H, W, a.vdim, 0, a.vdim, H * a.vdim, 1, 0, 0, 0, a.out_head_stride, 0}}, ""}}, 1, W, H * a.out_head_stride, "heads_o", &w.out, used);
+}
+
+// bias of a weight whose rows are not placed by heads
+int add_bias(Model& m, const std::string& name, int64_t n, DenseWeight* w) {
+    Tensor* b = nullptr;
+    int rc = get_raw(m, name, {n}, &b);
+    if (rc) return rc;
+    int64_t bd[1] = {w->n};
+    if (!(rc = tensor_alloc(GPTRS_F32, 1, bd, true, &w->bias)) &&
+        (cudaDeviceSynchronize() != cudaSuccess || cudaMemcpy(w->bias->data, b->data, (size_t)n * 4, cudaMemcpyDeviceToDevice) != cudaSuccess))
+        rc = fail(GPTRS_EXECUTION, "bias copy failed");
+    tensor_release(b);
+    return rc;
+}
+
+int build_delta(Model& m, LayeredLayer& L, const std::string& x, std::vector<std::string>* used) {
+    const gptrs_delta_rule& a = L.delta;
+    LayerWeights& w = *L.w;
+    const int64_t W = m.cfg.d_model, H = a.heads, kq = (int64_t)a.kv_heads * a.dim, hv = H * a.vdim, hd = H * a.dim;
+    int rc;
+    if ((rc = get_raw(m, x + "A_log", {H}, &w.a_log)) || (rc = get_raw(m, x + "dt_bias", {hd}, &w.dt_bias)) || (rc = get_raw(m, x + "norm", {a.vdim}, &w.delta_norm))) return rc;
+    if ((rc = pack_weight(m, {rows_of(x + "q", kq, W, a.q_offset), rows_of(x + "k", kq, W, a.k_offset), rows_of(x + "v", hv, W, a.v_offset), rows_of(x + "b", H, W, a.beta_offset),
+                              rows_of(x + "a1", a.decay_rank, W, a.a_offset), rows_of(x + "g1", a.gate_rank, W, a.g_offset)}, 1, a.row, W, "delta_proj", &w.qkv, used))) return rc;
+    if ((rc = pack_plain(m, x + "a2", hd, a.decay_rank, "", &w.decay, used)) || (rc = pack_plain(m, x + "g2", hv, a.gate_rank, "", &w.gate, used))) return rc;
+    if ((rc = pack_weight(m, {{x + "o", {W, hv}, {{H, W, a.vdim, 0, a.vdim, hv, 1, 0, 0, 0, a.out_head_stride, 0}}, ""}}, 1, W, H * a.out_head_stride, "heads_o", &w.out, used))) return rc;
+    // the three convolutions behind one another
+    int64_t cd[2] = {a.conv_channels, a.taps};
+    if ((rc = tensor_alloc(GPTRS_F32, 2, cd, false, &w.delta_conv))) return rc;
+    float* dst = static_cast<float*>(w.delta_conv->data);
+    for (const auto& part : {std::make_pair("q.conv", kq), std::make_pair("k.conv", kq), std::make_pair("v.conv", hv)}) {
+        Tensor* t = nullptr;
+        if ((rc = get_raw(m, x + part.first, {part.second, a.taps}, &t))) return rc;
+        const cudaError_t e = cudaMemcpy(dst, t->data, (size_t)part.second * a.taps * 4, cudaMemcpyDeviceToDevice);
+        tensor_release(t);
+        GPTRS_CUDA_OK(e);
+        dst += part.second * a.taps;
+    }
+    return GPTRS_OK;
+}
+
+int build_experts(Model& m, LayeredLayer& L, const std::string& x, std::vector<std::string>* used) {
+    LayerWeights& w = *L.w;
+    const int64_t W = m.cfg.d_model, F = L.cfg.d_ff, Fp = pad8(F), E = L.moe.experts;
+    std::vector<Leaf> up, down;
+    for (int64_t e = 0; e < E; ++e) {
+        const std::string n = x + "e" + std::to_string(e) + ".";
+        for (int part = 0; part < 2; ++part) {   // 8 gates, then their 8 partners
+            const int64_t full = F / 8, rest = F % 8;
+            Leaf l = {n + (part ? "up" : "gate"), {F, W}, {{full, 8, W, 0, 8 * W, W, 1, part * 8, 16, 0, 0, 0, e}}, ""};
+            if (rest) l.pieces.push_back({1, rest, W, full * 8 * W, 0, W, 1, full * 16 + part * 8, 0, 0, 0, 0, e});
+            up.push_back(l);
+        }
+        down.push_back({n + "down", {W, F}, {{1, W, F, 0, 0, F, 1, 0, 0, 0, 0, 0, e}}, ""});
+    }
+    int rc;
+    if ((rc = pack_weight(m, up, E, 2 * Fp, W, "experts_up", &w.up, used)) || (rc = pack_weight(m, down, E, W, Fp, "experts_down", &w.down, used))) return rc;
+    return pack_plain(m, x + "router", E, W, "", &w.router, used);
+}
+
+int build_weights(Model& m, LayeredLayer& L, int l, bool drop_leaves) {
+    const int64_t W = m.cfg.d_model, taps = m.lay->cfg.conv_taps;
+    const bool sandwich = m.lay->cfg.block == GPTRS_BLOCK_SANDWICH;
+    const std::string p = "l" + std::to_string(l) + ".", x = p + "mix.", f = p + "mlp.";
+    L.w = std::make_shared<LayerWeights>();
+    LayerWeights& w = *L.w;
+    std::vector<std::string> used;
+    int rc;
+    if ((rc = get_raw(m, p + "norm1", {W}, &w.norm1))) return rc;
+    if ((rc = sandwich ? get_raw(m, p + "norm1b", {W}, &w.norm1b) : get_raw(m, p + "canon1", {W, taps}, &w.conv1))) return rc;
+    if (L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION) rc = build_latent(m, L, x, &used);
+    else if (L.cfg.mixer == GPTRS_MIXER_GROUPED_ATTENTION) rc = build_grouped(m, L, x, &used);
+    else rc = build_delta(m, L, x, &used);
+    if (rc) return rc;
+    if (L.cfg.mixer == GPTRS_MIXER_GROUPED_ATTENTION && L.cfg.proj_bias && (rc = add_bias(m, x + "o.b", W, &w.out))) return rc;
+    if (L.cfg.mlp != GPTRS_MLP_NONE) {
+        if ((rc = get_raw(m, p + "norm2", {W}, &w.norm2))) return rc;
+        if ((rc = sandwich ? get_raw(m, p + "norm2b", {W}, &w.norm2b) : get_raw(m, p + "canon2", {W, taps}, &w.conv2))) return rc;
+    }
+    if (L.cfg.mlp == GPTRS_MLP_DENSE_XIELU) {
+        const int64_t F = L.cfg.d_ff;
+        if ((rc = pack_plain(m, f + "up", F, W, f + "up.b", &w.up, &used)) || (rc = pack_plain(m, f + "down", W, F, f + "down.b", &w.down, &used))) return rc;
+        Tensor* pq = nullptr;
+        float v[2];
+        if ((rc = get_raw(m, f + "act", {2}, &pq))) return rc;
+        const cudaError_t e = cudaMemcpy(v, pq->data, 8, cudaMemcpyDeviceToHost);
+        tensor_release(pq);
+        GPTRS_CUDA_OK(e);
+        w.act_pos = softplus(v[0]);
+        w.act_neg = 0.5f + softplus(v[1]);
+    } else if (L.cfg.mlp == GPTRS_MLP_EXPERTS) {
+        if ((rc = build_experts(m, L, f, &used))) return rc;
+    }
+    if (drop_leaves)
+        for (const std::string& n : used) {
+            auto it = m.raw.find(n);
+            if (it != m.raw.end()) { tensor_release(it->second); m.raw.erase(it); }
+        }
+    return GPTRS_OK;
+}
+
+// rotation tables, one pair per distinct (base, dims); angles in double, rounded once
+int add_rope(Model& m, LayeredLayer& L) {
+    Layered& y = *m.lay;
+    const auto& c = m.cfg;
+    const gptrs_latent_attention& a = L.att;
+    for (size_t i = 0; i < y.ropes.size(); ++i)
+        if (y.ropes[i]->base == L.cfg.rope_base && y.ropes[i]->dims == a.rot_dims) L.rope = (int)i;
+    if (L.rope >= 0) return GPTRS_OK;
+    auto r = std::make_unique<Layered::Rope>();
+    r->base = L.cfg.rope_base; r->dims = a.rot_dims;
+    const int half = a.rot_dims / 2;
+    std::vector<float> cs((size_t)c.context_length * half), sn(cs.size());
+    for (int i = 0; i < half; ++i) {
+        const double f = std::pow(r->base, -2.0 * i / a.rot_dims);
+        for (int q = 0; q < c.context_length; ++q) {
+            cs[(size_t)q * half + i] = (float)std::cos(q * f);
+            sn[(size_t)q * half + i] = (float)std::sin(q * f);
+        }
+    }
+    int rc;
+    if (half > 0) {
+        if ((rc = r->cos_t.alloc(cs.size() * 4)) || (rc = r->sin_t.alloc(sn.size() * 4))) return rc;
+        GPTRS_CUDA_OK(cudaMemcpy(r->cos_t.p, cs.data(), cs.size() * 4, cudaMemcpyHostToDevice));
+        GPTRS_CUDA_OK(cudaMemcpy(r->sin_t.p, sn.data(), sn.size() * 4, cudaMemcpyHostToDevice));
+    }
+    L.rope = (int)y.ropes.size();
+    y.ropes.push_back(std::move(r));
+    return GPTRS_OK;
+}
+
+// query tiles of the tensor-core attention (GPTRS_LATENT_TC=0 / GPTRS_GROUPED_TC=0 keep the plain kernels)
+int add_tiles(Model& m, LayeredLayer& L) {
+    Layered& y = *m.lay;
+    static const bool latent_on = [] { const char* e = getenv("GPTRS_LATENT_TC"); return !e || atoi(e) != 0; }();
+    static const bool grouped_on = [] { const char* e = getenv("GPTRS_GROUPED_TC"); return !e || atoi(e) != 0; }();
+    const int tokens = L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION ? (latent_on ? gptrs_cuda_latent_tile_tokens(&L.att) : 0)
+                                                                   : (grouped_on ? gptrs_cuda_grouped_tile_tokens(&L.gatt) : 0);
+    L.tiles = -1;
+    if (tokens <= 0) return GPTRS_OK;
+    for (size_t i = 0; i < y.tile_sets.size(); ++i)
+        if (y.tile_sets[i]->tokens == tokens) L.tiles = (int)i;
+    if (L.tiles >= 0) return GPTRS_OK;
+    auto t = std::make_unique<Layered::TileSet>();
+    t->tokens = tokens;
+    int rc;
+    if ((rc = t->row.alloc((size_t)m.cfg.max_tokens * 4, true)) || (rc = t->rows.alloc((size_t)m.cfg.max_tokens * 4, true))) return rc;
+    L.tiles = (int)y.tile_sets.size();
+    y.tile_sets.push_back(std::move(t));
+    return GPTRS_OK;
+}
+
+void count_widths(const Model& m, LayeredLayer& L, Widths* n) {
+    const auto& c = m.cfg;
+    const LayerWeights& w = *L.w;
+    n->qkv = std::max(n->qkv, w.qkv.n);
+    n->attn = std::max(n->attn, w.out.k);
+    L.pool_off = n->pool;
+    if (L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION) {
+        n->qa = std::max(n->qa, (int64_t)L.att.heads * L.att.qa_head_stride);
+        n->lat = std::max(n->lat, (int64_t)L.att.heads * L.att.lat_head_stride);
+        n->pool += (size_t)c.kv_pages * L.att.page_bytes;
+    } else if (L.cfg.mixer == GPTRS_MIXER_GROUPED_ATTENTION) {
+        n->pool += (size_t)c.kv_pages * L.gatt.page_bytes;
+    } else {
+        n->decay = std::max(n->decay, (int64_t)L.delta.decay_row);
+        n->gate = std::max(n->gate, (int64_t)L.delta.gate_row);
+        n->delta_scratch = std::max(n->delta_scratch, L.delta.scratch_floats);
+        L.delta_state_off = n->delta_state;
+        L.delta_conv_off = n->delta_conv;
+        n->delta_state += (size_t)c.max_seqs * L.delta.state_floats;
+        n->delta_conv += (size_t)c.max_seqs * L.delta.conv_floats;
+    }
+    n->pool = (n->pool + 255) / 256 * 256;
+    n->delta_state = (n->delta_state + 63) / 64 * 64;
+    if (m.lay->cfg.block == GPTRS_BLOCK_OUTPUT_NORM) {
+        L.state1 = n->n_state++;
+        if (L.cfg.mlp != GPTRS_MLP_NONE) L.state2 = n->n_state++;
+    }
+    if (L.cfg.mlp == GPTRS_MLP_DENSE_XIELU) n->up = std::max(n->up, w.up.n);
+    if (L.cfg.mlp == GPTRS_MLP_EXPERTS) {
+        const int64_t T = c.max_tokens, top = L.moe.top;
+        n->top = std::max(n->top, top);
+        n->router = std::max(n->router, w.router.n);
+        n->sorted = std::max(n->sorted, top * w.up.k);
+        n->expert_up = std::max(n->expert_up, top * w.up.n);
+        n->expert_y = std::max(n->expert_y, top * w.down.n);
+        n->work = std::max(n->work, gptrs_cuda_moe_work_ints(&L.moe, T));
+        gptrs_moe smallest = L.moe;   // most tiles: the smallest tile that a launch of this many rows, or of one, may get
+        smallest.tile_rows = m.f32() ? 8 : 16;
+        n->row_tiles = std::max(n->row_tiles, gptrs_cuda_moe_max_tiles(&smallest, T));
+    }
+}
+
+bool same_shape(const gptrs_layer_config& a, const gptrs_layer_config& b) {
+    auto key = [](const gptrs_layer_config& c) {
+        return std::make_tuple(std::make_tuple(c.mixer, c.heads, c.dim, c.rot_dim, c.rot_dims, c.vdim, c.kv_rank, c.window, c.scale, c.rope_base, c.mlp, c.d_ff),
+                               std::make_tuple(c.kv_heads, c.mask, c.mask_size, c.distance_bias, c.proj_bias, c.softcap, c.taps, c.decay_rank, c.gate_rank),
+                               std::make_tuple(c.experts, c.top, c.groups, c.keep));
+    };
+    return key(a) == key(b);
+}
 
 }  // namespace
 
@@ -137,103 +427,79 @@ int layered_check_config(const gptrs_model_config& c) {
     return GPTRS_OK;
 }
 
+int layered_set_layers(Model& m, const gptrs_layered_config& common, const gptrs_layer_config* layers) {
+    const int n = m.cfg.n_layers;
+    GPTRS_REQUIRE(common.block == GPTRS_BLOCK_OUTPUT_NORM || common.block == GPTRS_BLOCK_SANDWICH, "unknown block form");
+    GPTRS_REQUIRE(common.block != GPTRS_BLOCK_OUTPUT_NORM || (common.conv_taps >= 1 && common.conv_taps <= 16), "short convolutions of 1 to 16 taps");
+    GPTRS_REQUIRE(common.learned_positions == 0 || (common.block == GPTRS_BLOCK_SANDWICH && common.learned_positions >= m.cfg.context_length),
+                  "learned positions: for the block form with norms on both sides, one for every position of the context");
+    m.lay->cfg = common;
+    m.lay->layers.clear();
+    m.lay->layers.resize(n);
+    const int dtype = m.f32() ? GPTRS_F32 : GPTRS_BF16;
+    for (int l = 0; l < n; ++l) {
+        const gptrs_layer_config& c = layers[l];
+        GPTRS_REQUIRE(c.mlp == GPTRS_MLP_NONE || c.d_ff > 0, "feed-forward size");
+        GPTRS_REQUIRE(c.weights_of < n && (c.weights_of < 0 || layers[c.weights_of].weights_of < 0), "weights_of names a layer that has weights of its own");
+        LayeredLayer& L = m.lay->layers[l];
+        L.cfg = c;
+        int rc;
+        if (c.mixer == GPTRS_MIXER_LATENT_ATTENTION) {
+            L.att.dtype = dtype;
+            L.att.heads = c.heads; L.att.dim = c.dim; L.att.rot_dim = c.rot_dim; L.att.vdim = c.vdim; L.att.kv_rank = c.kv_rank;
+            L.att.window = c.window; L.att.rot_dims = c.rot_dims; L.att.scale = c.scale;
+            rc = gptrs_cuda_latent_layout(&L.att);
+        } else if (c.mixer == GPTRS_MIXER_GROUPED_ATTENTION) {
+            L.gatt.dtype = dtype;
+            L.gatt.heads = c.heads; L.gatt.kv_heads = c.kv_heads; L.gatt.dim = c.dim; L.gatt.vdim = c.vdim; L.gatt.mask = c.mask; L.gatt.mask_size = c.mask_size;
+            L.gatt.scale = c.scale; L.gatt.softcap = c.softcap; L.gatt.distance_bias = c.distance_bias;
+            rc = gptrs_cuda_grouped_layout(&L.gatt);
+        } else if (c.mixer == GPTRS_MIXER_CHANNEL_DELTA) {
+            L.delta.dtype = dtype;
+            L.delta.heads = c.heads; L.delta.kv_heads = c.kv_heads; L.delta.dim = c.dim; L.delta.vdim = c.vdim; L.delta.taps = c.taps;
+            L.delta.decay_rank = c.decay_rank; L.delta.gate_rank = c.gate_rank; L.delta.eps = m.cfg.norm_eps;
+            rc = gptrs_cuda_delta_layout(&L.delta);
+        } else {
+            return fail(GPTRS_UNIMPLEMENTED, "unknown mixer");
+        }
+        if (rc) return rc;
+        if (c.mlp == GPTRS_MLP_EXPERTS) {
+            GPTRS_REQUIRE(common.block == GPTRS_BLOCK_SANDWICH, "experts: for the block form with norms on both sides");
+            L.moe = {c.experts, c.top, c.groups, c.keep, 16};
+            GPTRS_REQUIRE(c.experts > 0 && c.top > 0 && c.groups > 0 && c.keep > 0 && c.experts % c.groups == 0 && c.keep <= c.groups &&
+                              c.top <= c.keep * (c.experts / c.groups), "experts: groups must be equal and hold enough experts");
+            if (c.experts > 1024) return fail(GPTRS_UNIMPLEMENTED, "experts: more than 1024");
+        } else if (c.mlp != GPTRS_MLP_NONE && c.mlp != GPTRS_MLP_DENSE_XIELU) {
+            return fail(GPTRS_UNIMPLEMENTED, "unknown feed-forward kind");
+        }
+    }
+    return GPTRS_OK;
+}
+
 int layered_finalize(Model& m, bool drop_leaves) {
     Layered& y = *m.lay;
     const auto& c = m.cfg;
     GPTRS_REQUIRE(!y.layers.empty(), "call gptrs_cuda_model_set_layers before finalize");
     const int64_t W = c.d_model, V = c.vocab, taps = y.cfg.conv_taps;
+    const bool sandwich = y.cfg.block == GPTRS_BLOCK_SANDWICH;
     int rc;
-    if ((rc = get_raw(m, "embed", {V, W}, &m.tok_emb)) || (rc = get_raw(m, "embed.norm", {W}, &y.embed_norm)) ||
-        (rc = get_raw(m, "final.norm", {W}, &m.final_g))) return rc;
+    if ((rc = get_raw(m, "embed", {V, W}, &m.tok_emb)) || (rc = get_raw(m, "final.norm", {W}, &m.final_g))) return rc;
+    if (!sandwich && (rc = get_raw(m, "embed.norm", {W}, &y.embed_norm))) return rc;
+    if (y.cfg.learned_positions > 0 && (rc = get_raw(m, "pos", {y.cfg.learned_positions, W}, &m.pos_emb))) return rc;
     if ((rc = pack_plain(m, "head", V, W, "", &y.head))) return rc;
     const size_t act = m.f32() ? 4 : 2;
-    int64_t qkv_w = 0, qa_w = 0, lat_w = 0, attn_w = 0, up_w = 0;
-    size_t pool = 0;
-    int n_state = 0;
+    Widths n;
+    for (int l = 0; l < c.n_layers; ++l)
+        if (y.layers[l].cfg.weights_of < 0 && (rc = build_weights(m, y.layers[l], l, drop_leaves))) return rc;
     for (int l = 0; l < c.n_layers; ++l) {
         LayeredLayer& L = y.layers[l];
-        const gptrs_latent_attention& a = L.att;
-        const std::string p = "l" + std::to_string(l) + ".", x = p + "mix.";
-        const int64_t H = a.heads, dim = a.dim, rot = a.rot_dim, rank = a.kv_rank, vd = a.vdim;
-        if ((rc = get_raw(m, p + "norm1", {W}, &L.norm1)) || (rc = get_raw(m, p + "canon1", {W, taps}, &L.conv1)) ||
-            (rc = get_raw(m, x + "dkv.norm", {rank}, &L.latent_norm))) return rc;
-        // queries and the down-projection in one weight, laid out as the attention kernels expect a projection row
-        if ((rc = pack_weight(m, {x + "q", x + "dkv"}, {{H * (dim + rot), W}, {rank + rot, W}},
-                              {{{H, dim, W, 0, (dim + rot) * W, W, 1, 0, a.q_head_stride, 0, 0, 0},
-                                {H, rot, W, dim * W, (dim + rot) * W, W, 1, a.q_rot_offset, a.q_head_stride, 0, 0, 0}},
-                               {{1, rank, W, 0, 0, W, 1, a.dkv_offset, 0, 0, 0, 0}, {1, rot, W, rank * W, 0, W, 1, a.rot_offset, 0, 0, 0, 0}}},
-                              1, a.q_row, W, "", "latent_qkv", &L.qkv))) return rc;
-        // absorbed query: per head [rank] <- [dim], the stored key projection transposed
-        if ((rc = pack_weight(m, {x + "uk"}, {{H * dim, rank}}, {{{H, rank, dim, 0, dim * rank, 1, rank, 0, 0, 0, 0, 1}}}, H, rank, dim, "", "latent_uk", &L.uk))) return rc;
-        if ((rc = pack_weight(m, {x + "uv"}, {{H * vd, rank}}, {{{H, vd, rank, 0, vd * rank, rank, 1, 0, 0, 0, 0, 1}}}, H, vd, rank, "", "latent_uv", &L.uv))) return rc;
-        if ((rc = pack_weight(m, {x + "o"}, {{W, H * vd}}, {{{H, W, vd, 0, vd, H * vd, 1, 0, 0, 0, a.out_head_stride, 0}}}, 1, W, H * a.out_head_stride, "", "latent_o", &L.out))) return rc;
-        L.state1 = n_state++;
-        if (L.cfg.mlp == GPTRS_MLP_DENSE_XIELU) {
-            const int64_t F = L.cfg.d_ff;
-            if ((rc = get_raw(m, p + "norm2", {W}, &L.norm2)) || (rc = get_raw(m, p + "canon2", {W, taps}, &L.conv2))) return rc;
-            if ((rc = pack_plain(m, p + "mlp.up", F, W, p + "mlp.up.b", &L.up)) || (rc = pack_plain(m, p + "mlp.down", W, F, p + "mlp.down.b", &L.down))) return rc;
-            Tensor* pq = nullptr;
-            float v[2];
-            if ((rc = get_raw(m, p + "mlp.act", {2}, &pq))) return rc;
-            const cudaError_t e = cudaMemcpy(v, pq->data, 8, cudaMemcpyDeviceToHost);
-            tensor_release(pq);
-            GPTRS_CUDA_OK(e);
-            L.act_pos = softplus(v[0]);
-            L.act_neg = 0.5f + softplus(v[1]);
-            L.state2 = n_state++;
-            up_w = std::max(up_w, L.up.n);
+        if (L.cfg.weights_of >= 0) {
+            GPTRS_REQUIRE(same_shape(L.cfg, y.layers[L.cfg.weights_of].cfg), "a layer that reuses another one's weights has an equal configuration");
+            L.w = y.layers[L.cfg.weights_of].w;
         }
-        if (drop_leaves)
-            for (const char* s : {"mix.q", "mix.dkv", "mix.uk", "mix.uv", "mix.o", "mlp.up", "mlp.down"}) {
-                auto it = m.raw.find(p + s);
-                if (it != m.raw.end()) { tensor_release(it->second); m.raw.erase(it); }
-            }
-        qkv_w = std::max(qkv_w, L.qkv.n);
-        qa_w = std::max(qa_w, H * (int64_t)a.qa_head_stride);
-        lat_w = std::max(lat_w, H * (int64_t)a.lat_head_stride);
-        attn_w = std::max(attn_w, L.out.k);
-        L.pool_off = pool;
-        pool += (size_t)c.kv_pages * a.page_bytes;
-        y.max_window = std::max(y.max_window, a.window);
-        // rotation tables, one pair per distinct (base, dims); angles in double, rounded once
-        L.rope = -1;
-        for (size_t i = 0; i < y.ropes.size(); ++i)
-            if (y.ropes[i]->base == L.cfg.rope_base && y.ropes[i]->dims == a.rot_dims) L.rope = (int)i;
-        if (L.rope < 0) {
-            auto r = std::make_unique<Layered::Rope>();
-            r->base = L.cfg.rope_base; r->dims = a.rot_dims;
-            const int half = a.rot_dims / 2;
-            std::vector<float> cs((size_t)c.context_length * half), sn(cs.size());
-            for (int i = 0; i < half; ++i) {
-                const double f = std::pow(r->base, -2.0 * i / a.rot_dims);
-                for (int q = 0; q < c.context_length; ++q) {
-                    cs[(size_t)q * half + i] = (float)std::cos(q * f);
-                    sn[(size_t)q * half + i] = (float)std::sin(q * f);
-                }
-            }
-            if (half > 0) {
-                if ((rc = r->cos_t.alloc(cs.size() * 4)) || (rc = r->sin_t.alloc(sn.size() * 4))) return rc;
-                GPTRS_CUDA_OK(cudaMemcpy(r->cos_t.p, cs.data(), cs.size() * 4, cudaMemcpyHostToDevice));
-                GPTRS_CUDA_OK(cudaMemcpy(r->sin_t.p, sn.data(), sn.size() * 4, cudaMemcpyHostToDevice));
-            }
-            L.rope = (int)y.ropes.size();
-            y.ropes.push_back(std::move(r));
-        }
-        // GPTRS_LATENT_TC=0 keeps the plain attention kernel
-        static const bool tc_on = [] { const char* e = getenv("GPTRS_LATENT_TC"); return !e || atoi(e) != 0; }();
-        const int tokens = tc_on ? gptrs_cuda_latent_tile_tokens(&a) : 0;
-        L.tiles = -1;
-        if (tokens > 0) {
-            for (size_t i = 0; i < y.tile_sets.size(); ++i)
-                if (y.tile_sets[i]->tokens == tokens) L.tiles = (int)i;
-            if (L.tiles < 0) {
-                auto t = std::make_unique<Layered::TileSet>();
-                t->tokens = tokens;
-                if ((rc = t->row.alloc((size_t)c.max_tokens * 4, true)) || (rc = t->rows.alloc((size_t)c.max_tokens * 4, true))) return rc;
-                L.tiles = (int)y.tile_sets.size();
-                y.tile_sets.push_back(std::move(t));
-            }
-        }
+        count_widths(m, L, &n);
+        if (L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION && (rc = add_rope(m, L))) return rc;
+        if (L.attends() && (rc = add_tiles(m, L))) return rc;
     }
     if (drop_leaves) {
         auto it = m.raw.find("head");
@@ -241,29 +507,40 @@ int layered_finalize(Model& m, bool drop_leaves) {
     }
     // activations (zeroed: padding columns that no kernel writes are multiplied by zero weights and must be finite)
     const size_t T = c.max_tokens, Wp = m.f32() ? W : pad8(W), Vp = y.head.n, rows = m.max_rows();
-    if ((rc = m.hidden.alloc(T * W * 4, true)) || (rc = y.x2.alloc(T * W * 4, true)) || (rc = y.h.alloc(T * Wp * act, true)) ||
-        (rc = y.y.alloc(T * Wp * act, true)) || (rc = y.qkv.alloc(T * qkv_w * act, true)) || (rc = y.qa.alloc(T * qa_w * act, true)) ||
-        (rc = y.lat.alloc(T * lat_w * act, true)) || (rc = y.attn.alloc(T * attn_w * act, true)) || (rc = y.up.alloc(T * up_w * act, true)) ||
+    if ((rc = m.hidden.alloc(T * W * 4, true)) || (rc = y.x2.alloc(sandwich ? 0 : T * W * 4, true)) || (rc = y.h.alloc(T * Wp * act, true)) ||
+        (rc = y.y.alloc(T * Wp * act, true)) || (rc = y.qkv.alloc(T * n.qkv * act, true)) || (rc = y.qa.alloc(T * n.qa * act, true)) ||
+        (rc = y.lat.alloc(T * n.lat * act, true)) || (rc = y.attn.alloc(T * n.attn * act, true)) || (rc = y.up.alloc(T * std::max(n.up, n.expert_up / 2) * act, true)) ||
         (rc = m.xn_rows.alloc(rows * Wp * act, true)) || (rc = m.logits.alloc(rows * V * 4, true))) return rc;
+    if ((rc = y.decay.alloc(T * n.decay * 4, true)) || (rc = y.gate.alloc(T * n.gate * act, true)) || (rc = y.delta_scratch.alloc(T * n.delta_scratch * 4, true)) ||
+        (rc = y.delta_state.alloc(n.delta_state * 4, true)) || (rc = y.delta_conv.alloc(n.delta_conv * 4, true))) return rc;
+    if ((rc = y.router.alloc(T * n.router * 4, true)) || (rc = y.sorted.alloc(T * n.sorted * act, true)) || (rc = y.gate_up.alloc(m.f32() ? T * n.expert_up * 4 : 0, true)) ||
+        (rc = y.expert_y.alloc(T * n.expert_y * act, true)) || (rc = y.pair.alloc(T * n.top * 4, true)) || (rc = y.pair_weight.alloc(T * n.top * 4, true)) ||
+        (rc = y.row_tiles.alloc(n.row_tiles * sizeof(gptrs_row_tile), true)) || (rc = y.n_row_tiles.alloc(4, true)) || (rc = y.moe_work.alloc(n.work * 4, true))) return rc;
     if ((int64_t)Vp != V && (rc = y.logits_pad.alloc(rows * Vp * 4, true))) return rc;
     if (!m.f32()) {
         const size_t tiles = (Vp + 127) / 128, r = std::min<size_t>(rows, 128);
         if ((rc = m.best_val.alloc(tiles * r * 4)) || (rc = m.best_idx.alloc(tiles * r * 4))) return rc;
         if (const char* e = getenv("GPTRS_FUSE_PICK")) m.fuse_pick = atoi(e) != 0;
     }
-    y.state_stride = (size_t)c.max_seqs * 2 * (taps - 1) * W;
-    if ((rc = y.state.alloc(std::max<size_t>(1, (size_t)n_state * y.state_stride) * 4, true))) return rc;
-    for (DevBuf* b : {&y.d_run_first, &y.d_run_last, &y.d_parity})
+    y.state_stride = sandwich ? 0 : (size_t)c.max_seqs * 2 * (taps - 1) * W;
+    if ((rc = y.state.alloc(std::max<size_t>(1, (size_t)n.n_state * y.state_stride) * 4, true))) return rc;
+    for (DevBuf* b : {&y.d_run_first, &y.d_run_last, &y.d_parity, &y.d_runs})
         if ((rc = b->alloc(T * 4, true))) return rc;
     GPTRS_CUDA_OK(cudaMallocHost(&y.h_tiles, T * 2 * 4));
     y.parity.assign(c.max_seqs, 0);
-    if ((rc = alloc_step_buffers(m, 9))) return rc;
-    if ((rc = m.kv_pool.alloc(pool, true))) return rc;
+    if ((rc = alloc_step_buffers(m, 10))) return rc;
+    if ((rc = m.kv_pool.alloc(n.pool, true))) return rc;
     if ((rc = alloc_page_tables(m))) return rc;
     // partial outputs of split keys: a launch splits only while its CTAs number at most the SMs
     size_t scratch = 0;
-    for (const LayeredLayer& L : y.layers)
-        if (L.tiles >= 0) scratch = std::max(scratch, gptrs_cuda_latent_scratch_bytes(&L.att, 1, sm_count() + 1));
+    for (const LayeredLayer& L : y.layers) {
+        if (L.tiles < 0) continue;
+        if (L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION) scratch = std::max(scratch, gptrs_cuda_latent_scratch_bytes(&L.att, 1, sm_count() + 1));
+        else {
+            const int per_split = L.gatt.kv_heads * ((L.gatt.heads / L.gatt.kv_heads + 127) / 128);
+            scratch = std::max(scratch, gptrs_cuda_grouped_scratch_bytes(&L.gatt, 1, sm_count() / per_split + 2));
+        }
+    }
     if ((rc = y.scratch.alloc(scratch))) return rc;
     GPTRS_CUDA_OK(cudaDeviceSynchronize());
     return GPTRS_OK;
@@ -281,7 +558,7 @@ int copy_tiles(Model& m, Layered::TileSet& t) {
 }  // namespace
 
 // Host rows -> runs (consecutive positions of one sequence), the halves of the convolution state they read, and query tiles.
-// Convolution state and cache move forward only, so a run must start where its sequence stands.
+// State and cache move forward only, so a run must start where its sequence stands.
 int layered_stage_rows(Model& m, const int32_t* slots, const int32_t* positions, int n) {
     Layered& y = *m.lay;
     y.runs.clear();
@@ -298,15 +575,21 @@ int layered_stage_rows(Model& m, const int32_t* slots, const int32_t* positions,
     }
     int32_t* st = m.h_stage;
     const int stride = m.stage_stride();
-    for (size_t r = 0; r < y.runs.size(); r += 2)
-        for (int i = y.runs[r]; i < y.runs[r] + y.runs[r + 1]; ++i) {
-            st[6 * stride + i] = y.runs[r];
-            st[7 * stride + i] = y.runs[r] + y.runs[r + 1] - 1;
+    const int n_runs = (int)y.runs.size() / 2;
+    for (int r = 0; r < n_runs; ++r) {
+        const int first = y.runs[2 * r], len = y.runs[2 * r + 1];
+        for (int i = first; i < first + len; ++i) {
+            st[6 * stride + i] = first;
+            st[7 * stride + i] = first + len - 1;
             st[8 * stride + i] = y.parity[slots[i]];
         }
+        st[9 * stride + r] = first;
+    }
     GPTRS_CUDA_OK(cudaMemcpyAsync(y.d_run_first.p, st + 6 * stride, (size_t)n * 4, cudaMemcpyHostToDevice, m.stream));
     GPTRS_CUDA_OK(cudaMemcpyAsync(y.d_run_last.p, st + 7 * stride, (size_t)n * 4, cudaMemcpyHostToDevice, m.stream));
     GPTRS_CUDA_OK(cudaMemcpyAsync(y.d_parity.p, st + 8 * stride, (size_t)n * 4, cudaMemcpyHostToDevice, m.stream));
+    GPTRS_CUDA_OK(cudaMemcpyAsync(y.d_runs.p, st + 9 * stride, (size_t)n_runs * 4, cudaMemcpyHostToDevice, m.stream));
+    y.n_runs = n_runs;
     for (auto& t : y.tile_sets) {
         t->n = 0;
         for (size_t r = 0; r < y.runs.size(); r += 2)
@@ -329,7 +612,9 @@ int layered_stage_generator(Model& m, int batch) {
     for (int b = 0; b < batch; ++b) { st[6 * stride + b] = b; st[8 * stride + b] = y.parity[b]; }
     GPTRS_CUDA_OK(cudaMemcpyAsync(y.d_run_first.p, st + 6 * stride, (size_t)batch * 4, cudaMemcpyHostToDevice, m.stream));
     GPTRS_CUDA_OK(cudaMemcpyAsync(y.d_run_last.p, st + 6 * stride, (size_t)batch * 4, cudaMemcpyHostToDevice, m.stream));
+    GPTRS_CUDA_OK(cudaMemcpyAsync(y.d_runs.p, st + 6 * stride, (size_t)batch * 4, cudaMemcpyHostToDevice, m.stream));
     GPTRS_CUDA_OK(cudaMemcpyAsync(y.d_parity.p, st + 8 * stride, (size_t)batch * 4, cudaMemcpyHostToDevice, m.stream));
+    y.n_runs = batch;
     for (int b = 0; b < batch; ++b) { y.h_tiles[b] = b; y.h_tiles[m.cfg.max_tokens + b] = 1; }
     for (auto& t : y.tile_sets) {
         t->n = batch;
@@ -339,98 +624,293 @@ int layered_stage_generator(Model& m, int batch) {
     return GPTRS_OK;
 }
 
-// Beyond the widest window a longer context changes nothing about the launches of a decode step.
-int layered_graph_bucket(const Model& m, int bucket) { return std::min(bucket, (m.lay->max_window + 511) / 512 * 512); }
+// The first position whose cached keys some layer still reads from position `pos` on.
+int layered_first_visible(const Model& m, int pos) {
+    int first = pos;
+    for (const LayeredLayer& L : m.lay->layers) {
+        if (!L.attends()) continue;
+        int f = 0;
+        if (L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION) f = pos - L.att.window + 1;
+        else if (L.gatt.mask == GPTRS_MASK_WINDOW) f = pos - L.gatt.mask_size + 1;
+        else if (L.gatt.mask == GPTRS_MASK_CHUNK) f = pos / L.gatt.mask_size * L.gatt.mask_size;
+        first = std::min(first, std::max(f, 0));
+    }
+    return first;
+}
 
-int layered_forward(Model& m, int T, int max_ctx, int n_rows, bool rows_identity, float temperature, bool skip_logits) {
-    Layered& y = *m.lay;
+// Beyond the widest mask a longer context changes nothing about the launches of a decode step.
+int layered_graph_bucket(const Model& m, int bucket) {
+    int widest = 1;
+    for (const LayeredLayer& L : m.lay->layers) {
+        if (!L.attends()) continue;
+        const int span = L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION ? L.att.window : L.gatt.mask == GPTRS_MASK_CAUSAL ? bucket : L.gatt.mask_size;
+        widest = std::max(widest, span);
+    }
+    return (int)std::min<int64_t>(bucket, ((int64_t)widest + 511) / 512 * 512);
+}
+
+namespace {
+
+// One forward pass: what its parts share.
+struct Pass {
+    Model& m;
+    Layered& y;
+    int T, max_ctx, act_dt;
+    int64_t ldw;
+    cudaStream_t st;
+    static const float* fp(Tensor* t) { return t ? static_cast<const float*>(t->data) : nullptr; }
+
+    unsigned char* pool(const LayeredLayer& L) const { return m.kv_pool.as<unsigned char>() + L.pool_off; }
+    const int32_t* slot() const { return m.d_slot.as<int32_t>(); }
+    const int32_t* pos() const { return m.d_pos.as<int32_t>(); }
+    const int32_t* pages() const { return m.d_page_table.as<int32_t>(); }
+
+    int latent(LayeredLayer& L) {
+        const gptrs_latent_attention& a = L.att;
+        const LayerWeights& w = *L.w;
+        const Layered::Rope& rope = *y.ropes[L.rope];
+        int rc;
+        if ((rc = dense(m, w.qkv, y.h.p, y.qkv.p, T, {}))) return rc;
+        DenseOpts ok;
+        ok.ldx = w.qkv.n; ok.x_step = a.q_head_stride; ok.ldy = (int64_t)a.heads * a.qa_head_stride; ok.y_step = a.qa_head_stride;
+        if ((rc = dense(m, w.uk, y.qkv.p, y.qa.p, T, ok))) return rc;
+        ++m.launches;
+        if ((rc = gptrs_cuda_latent_append(&a, y.qkv.p, pos(), slot(), pages(), m.cfg.max_pages_per_seq, fp(w.latent_norm), m.cfg.norm_eps,
+                                           rope.cos_t.as<float>(), rope.sin_t.as<float>(), y.qa.p, pool(L), T, st))) return rc;
+        const Layered::TileSet* t = L.tiles >= 0 ? y.tile_sets[L.tiles].get() : nullptr;
+        const int splits = t ? gptrs_cuda_latent_splits(&a, t->n, max_ctx) : 1;
+        m.launches += splits > 1 ? 2 : 1;
+        if ((rc = gptrs_cuda_latent_attention(&a, y.qa.p, pool(L), pages(), m.cfg.max_pages_per_seq, slot(), m.d_ctx.as<int32_t>(),
+                                              t ? t->row.as<int32_t>() : nullptr, t ? t->rows.as<int32_t>() : nullptr, t ? t->n : 0, splits, y.lat.p, y.scratch.p,
+                                              y.scratch.n, m.d_status.as<int32_t>(), T, st))) return rc;
+        DenseOpts ov;
+        ov.ldx = (int64_t)a.heads * a.lat_head_stride; ov.x_step = a.lat_head_stride; ov.ldy = w.out.k; ov.y_step = a.out_head_stride;
+        if ((rc = dense(m, w.uv, y.lat.p, y.attn.p, T, ov))) return rc;
+        return dense(m, w.out, y.attn.p, y.y.p, T, {});
+    }
+
+    int grouped(LayeredLayer& L) {
+        const gptrs_grouped_attention& a = L.gatt;
+        const LayerWeights& w = *L.w;
+        int rc;
+        if ((rc = dense(m, w.qkv, y.h.p, y.qkv.p, T, {}))) return rc;
+        ++m.launches;
+        if ((rc = gptrs_cuda_grouped_append(&a, y.qkv.p, pos(), slot(), pages(), m.cfg.max_pages_per_seq, pool(L), T, st))) return rc;
+        const Layered::TileSet* t = L.tiles >= 0 ? y.tile_sets[L.tiles].get() : nullptr;
+        const int splits = t ? gptrs_cuda_grouped_splits(&a, t->n, max_ctx) : 1;
+        m.launches += splits > 1 ? 2 : 1;
+        if ((rc = gptrs_cuda_grouped_attention(&a, y.qkv.p, pool(L), pages(), m.cfg.max_pages_per_seq, slot(), m.d_ctx.as<int32_t>(), fp(w.r1), fp(w.r2),
+                                               t ? t->row.as<int32_t>() : nullptr, t ? t->rows.as<int32_t>() : nullptr, t ? t->n : 0, splits, y.attn.p, y.scratch.p,
+                                               y.scratch.n, m.d_status.as<int32_t>(), T, st))) return rc;
+        return dense(m, w.out, y.attn.p, y.y.p, T, {});
+    }
+
+    int delta(LayeredLayer& L) {
+        const gptrs_delta_rule& a = L.delta;
+        const LayerWeights& w = *L.w;
+        const size_t act = m.f32() ? 4 : 2;
+        int rc;
+        if ((rc = dense(m, w.qkv, y.h.p, y.qkv.p, T, {}))) return rc;
+        auto column = [&](int off) { return y.qkv.as<unsigned char>() + off * act; };
+        DenseOpts od;
+        od.out_f32 = true; od.ldx = w.qkv.n; od.ldy = a.decay_row;
+        if ((rc = dense(m, w.decay, column(a.a_offset), y.decay.p, T, od))) return rc;
+        DenseOpts og;
+        og.ldx = w.qkv.n; og.ldy = a.gate_row;
+        if ((rc = dense(m, w.gate, column(a.g_offset), y.gate.p, T, og))) return rc;
+        gptrs_delta_step s = {};
+        s.d_proj = y.qkv.p; s.d_decay = y.decay.as<float>(); s.d_gate = y.gate.p;
+        s.d_conv = fp(w.delta_conv); s.d_a_log = fp(w.a_log); s.d_dt_bias = fp(w.dt_bias); s.d_norm = fp(w.delta_norm);
+        s.d_state = y.delta_state.as<float>() + L.delta_state_off;
+        s.d_conv_state = y.delta_conv.as<float>() + L.delta_conv_off;
+        s.d_slot = slot(); s.d_pos = pos();
+        s.d_run_first = y.d_run_first.as<int32_t>(); s.d_run_last = y.d_run_last.as<int32_t>(); s.d_parity = y.d_parity.as<int32_t>();
+        s.d_runs = y.d_runs.as<int32_t>(); s.n_runs = y.n_runs;
+        s.d_out = y.attn.p; s.d_scratch = y.delta_scratch.as<float>(); s.rows = T;
+        m.launches += y.n_runs == T ? 1 : 3;
+        if ((rc = gptrs_cuda_delta_rule(&a, &s, st))) return rc;
+        return dense(m, w.out, y.attn.p, y.y.p, T, {});
+    }
+
+    // leaves the experts' outputs in expert_y; the step behind sums them up
+    int experts(LayeredLayer& L) {
+        const LayerWeights& w = *L.w;
+        gptrs_moe a = L.moe;
+        a.tile_rows = expert_tile_rows(m, a, T);
+        int rc;
+        DenseOpts orr;
+        orr.out_f32 = true;
+        if ((rc = dense(m, w.router, y.h.p, y.router.p, T, orr))) return rc;
+        m.launches += T > 128 ? 3 : 2;
+        gptrs_row_tile* tiles = y.row_tiles.as<gptrs_row_tile>();
+        int32_t* n_tiles = y.n_row_tiles.as<int32_t>();
+        if ((rc = gptrs_cuda_moe_route(&a, y.router.as<float>(), w.router.n, y.h.p, act_dt, ldw, y.pair.as<int32_t>(), y.pair_weight.as<float>(), tiles, n_tiles,
+                                       y.sorted.p, y.moe_work.as<int32_t>(), T, st))) return rc;
+        DenseOpts o;
+        o.tiles = tiles; o.n_tiles = n_tiles; o.tile_rows = a.tile_rows; o.max_tiles = gptrs_cuda_moe_max_tiles(&a, T);
+        const int64_t pairs = (int64_t)T * a.top;
+        DenseOpts ou = o;
+        ou.swiglu = !m.f32();
+        if ((rc = dense(m, w.up, y.sorted.p, m.f32() ? y.gate_up.p : y.up.p, pairs, ou))) return rc;
+        if (m.f32()) {
+            ++m.launches;
+            if ((rc = gptrs_cuda_swiglu_pairs_f32(y.gate_up.as<float>(), y.up.as<float>(), pairs, w.up.n / 2, st))) return rc;
+        }
+        return dense(m, w.down, y.up.p, y.expert_y.p, pairs, o);
+    }
+
+    int mixer(LayeredLayer& L) {
+        return L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION ? latent(L) : L.cfg.mixer == GPTRS_MIXER_GROUPED_ATTENTION ? grouped(L) : delta(L);
+    }
+    int feed_forward(LayeredLayer& L) {
+        if (L.cfg.mlp == GPTRS_MLP_EXPERTS) return experts(L);
+        DenseOpts ou;
+        ou.act = 1; ou.pos = L.w->act_pos; ou.neg = L.w->act_neg;
+        int rc = dense(m, L.w->up, y.h.p, y.up.p, T, ou);
+        return rc ? rc : dense(m, L.w->down, y.up.p, y.y.p, T, {});
+    }
+};
+
+struct Capture {   // debug: the residual stream after every layer
+    DevBuf buf;
+    int begin(Model& m, int T) { return m.lay->h_residuals ? buf.alloc((size_t)m.cfg.n_layers * T * m.cfg.d_model * 4) : GPTRS_OK; }
+    int take(Model& m, int l, const float* x, int T) {
+        const size_t n = (size_t)T * m.cfg.d_model;
+        if (buf.p) GPTRS_CUDA_OK(cudaMemcpyAsync(buf.as<float>() + l * n, x, n * 4, cudaMemcpyDeviceToDevice, m.stream));
+        return GPTRS_OK;
+    }
+    int end(Model& m) {
+        if (!buf.p) return GPTRS_OK;
+        GPTRS_CUDA_OK(cudaMemcpyAsync(m.lay->h_residuals, buf.p, buf.n, cudaMemcpyDeviceToHost, m.stream));
+        GPTRS_CUDA_OK(cudaStreamSynchronize(m.stream));
+        m.lay->h_residuals = nullptr;
+        return GPTRS_OK;
+    }
+};
+
+// norms on the outputs, sublayers that read the stream through short convolutions
+int forward_output_norm(Pass& f, Capture& cap, int n_rows, bool rows_identity) {
+    Model& m = f.m;
+    Layered& y = f.y;
     const auto& c = m.cfg;
-    const int W = c.d_model, taps = y.cfg.conv_taps;
-    const int act_dt = m.f32() ? GPTRS_F32 : GPTRS_BF16;
-    const int64_t ldw = m.f32() ? W : pad8(W);
-    cudaStream_t st = m.stream;
+    const int W = c.d_model, T = f.T;
     float* x = m.hidden.as<float>();
     float* x_other = y.x2.as<float>();
     int rc;
     gptrs_conv_step base = {};
-    base.y_dtype = act_dt; base.d_y = y.y.p; base.ldy = ldw;
-    base.eps = c.norm_eps; base.taps = taps;
-    base.d_slot = m.d_slot.as<int32_t>(); base.d_pos = m.d_pos.as<int32_t>();
+    base.y_dtype = f.act_dt; base.d_y = y.y.p; base.ldy = f.ldw;
+    base.eps = c.norm_eps; base.taps = y.cfg.conv_taps;
+    base.d_slot = f.slot(); base.d_pos = f.pos();
     base.d_run_first = y.d_run_first.as<int32_t>(); base.d_run_last = y.d_run_last.as<int32_t>(); base.d_parity = y.d_parity.as<int32_t>();
-    base.d_h = y.h.p; base.h_dtype = act_dt; base.ldh = ldw;
+    base.d_h = y.h.p; base.h_dtype = f.act_dt; base.ldh = f.ldw;
     base.d_status = m.d_status.as<int32_t>();
     base.rows = T; base.dim = W;
-    auto fp = [](Tensor* t) { return static_cast<const float*>(t->data); };
     // closes a sublayer with its output norm (or opens the model with the normed embedding) and prepares the next one's input
     auto step = [&](Tensor* gamma, bool embed, Tensor* conv, int state) -> int {
         gptrs_conv_step s = base;
-        if (embed) { s.d_embed = fp(m.tok_emb); s.d_tokens = m.d_tokens.as<int32_t>(); s.vocab = c.vocab; s.ldy = W; s.y_dtype = GPTRS_F32; }
+        if (embed) { s.d_embed = f.fp(m.tok_emb); s.d_tokens = m.d_tokens.as<int32_t>(); s.vocab = c.vocab; s.ldy = W; s.y_dtype = GPTRS_F32; }
         else s.d_x = x;
         s.d_x_out = x_other;
-        s.d_gamma = fp(gamma);
-        if (conv) { s.d_conv = fp(conv); s.d_state = y.state.as<float>() + (size_t)state * y.state_stride; }
+        s.d_gamma = f.fp(gamma);
+        if (conv) { s.d_conv = f.fp(conv); s.d_state = y.state.as<float>() + (size_t)state * y.state_stride; }
         ++m.launches;
-        int r = gptrs_cuda_post_norm_conv(&s, st);
+        int r = gptrs_cuda_post_norm_conv(&s, f.st);
         std::swap(x, x_other);
         return r;
     };
-    DevBuf captured;
-    if (y.h_residuals && (rc = captured.alloc((size_t)c.n_layers * T * W * 4))) return rc;
-    auto capture = [&](int l) -> int {
-        if (captured.p) GPTRS_CUDA_OK(cudaMemcpyAsync(captured.as<float>() + (size_t)l * T * W, x, (size_t)T * W * 4, cudaMemcpyDeviceToDevice, st));
-        return GPTRS_OK;
-    };
-
-    if ((rc = step(y.embed_norm, true, y.layers[0].conv1, y.layers[0].state1))) return rc;
+    if ((rc = step(y.embed_norm, true, y.layers[0].w->conv1, y.layers[0].state1))) return rc;
     for (int l = 0; l < c.n_layers; ++l) {
         LayeredLayer& L = y.layers[l];
-        const gptrs_latent_attention& a = L.att;
-        const Layered::Rope& rope = *y.ropes[L.rope];
-        unsigned char* pool = m.kv_pool.as<unsigned char>() + L.pool_off;
-        DenseOpts o;
-        if ((rc = dense(m, L.qkv, y.h.p, y.qkv.p, T, o))) return rc;
-        DenseOpts ok;
-        ok.ldx = L.qkv.n; ok.x_step = a.q_head_stride; ok.ldy = (int64_t)a.heads * a.qa_head_stride; ok.y_step = a.qa_head_stride;
-        if ((rc = dense(m, L.uk, y.qkv.p, y.qa.p, T, ok))) return rc;
-        ++m.launches;
-        if ((rc = gptrs_cuda_latent_append(&a, y.qkv.p, base.d_pos, base.d_slot, m.d_page_table.as<int32_t>(), c.max_pages_per_seq, fp(L.latent_norm), c.norm_eps,
-                                           rope.cos_t.as<float>(), rope.sin_t.as<float>(), y.qa.p, pool, T, st))) return rc;
-        const Layered::TileSet* t = L.tiles >= 0 ? y.tile_sets[L.tiles].get() : nullptr;
-        const int splits = t ? gptrs_cuda_latent_splits(&a, t->n, max_ctx) : 1;
-        m.launches += splits > 1 ? 2 : 1;
-        if ((rc = gptrs_cuda_latent_attention(&a, y.qa.p, pool, m.d_page_table.as<int32_t>(), c.max_pages_per_seq, base.d_slot, m.d_ctx.as<int32_t>(),
-                                              t ? t->row.as<int32_t>() : nullptr, t ? t->rows.as<int32_t>() : nullptr, t ? t->n : 0, splits, y.lat.p, y.scratch.p,
-                                              y.scratch.n, base.d_status, T, st))) return rc;
-        DenseOpts ov;
-        ov.ldx = (int64_t)a.heads * a.lat_head_stride; ov.x_step = a.lat_head_stride; ov.ldy = L.out.k; ov.y_step = a.out_head_stride;
-        if ((rc = dense(m, L.uv, y.lat.p, y.attn.p, T, ov))) return rc;
-        if ((rc = dense(m, L.out, y.attn.p, y.y.p, T, o))) return rc;
+        if ((rc = f.mixer(L))) return rc;
         const bool last = l + 1 == c.n_layers;
-        Tensor* next = last ? nullptr : y.layers[l + 1].conv1;
+        Tensor* next = last ? nullptr : y.layers[l + 1].w->conv1;
         const int next_state = last ? 0 : y.layers[l + 1].state1;
-        Tensor* gamma = L.norm1;
-        if (L.cfg.mlp == GPTRS_MLP_DENSE_XIELU) {
-            if ((rc = step(L.norm1, false, L.conv2, L.state2))) return rc;
-            DenseOpts ou;
-            ou.act = 1; ou.pos = L.act_pos; ou.neg = L.act_neg;
-            if ((rc = dense(m, L.up, y.h.p, y.up.p, T, ou))) return rc;
-            if ((rc = dense(m, L.down, y.up.p, y.y.p, T, o))) return rc;
-            gamma = L.norm2;
+        Tensor* gamma = L.w->norm1;
+        if (L.cfg.mlp != GPTRS_MLP_NONE) {
+            if ((rc = step(L.w->norm1, false, L.w->conv2, L.state2)) || (rc = f.feed_forward(L))) return rc;
+            gamma = L.w->norm2;
         }
         if (!last) {
-            if ((rc = step(gamma, false, next, next_state)) || (rc = capture(l))) return rc;
+            if ((rc = step(gamma, false, next, next_state)) || (rc = cap.take(m, l, x, T))) return rc;
             continue;
         }
         ++m.launches;
-        if ((rc = gptrs_cuda_post_norm_final(x, y.y.p, act_dt, ldw, fp(gamma), fp(m.final_g), c.norm_eps, rows_identity ? nullptr : m.d_rows.as<int32_t>(),
-                                             m.xn_rows.p, act_dt, ldw, n_rows, W, st))) return rc;
-        if (captured.p && ((rc = step(gamma, false, nullptr, 0)) || (rc = capture(l)))) return rc;
+        if ((rc = gptrs_cuda_post_norm_final(x, y.y.p, f.act_dt, f.ldw, f.fp(gamma), f.fp(m.final_g), c.norm_eps, rows_identity ? nullptr : m.d_rows.as<int32_t>(),
+                                             m.xn_rows.p, f.act_dt, f.ldw, n_rows, W, f.st))) return rc;
+        if (cap.buf.p && ((rc = step(gamma, false, nullptr, 0)) || (rc = cap.take(m, l, x, T)))) return rc;
     }
-    if (captured.p) {
-        GPTRS_CUDA_OK(cudaMemcpyAsync(y.h_residuals, captured.p, captured.n, cudaMemcpyDeviceToHost, st));
-        GPTRS_CUDA_OK(cudaStreamSynchronize(st));
-        y.h_residuals = nullptr;
+    return GPTRS_OK;
+}
+
+// norms on both sides of every sublayer
+int forward_sandwich(Pass& f, Capture& cap, int n_rows, bool rows_identity) {
+    Model& m = f.m;
+    Layered& y = f.y;
+    const auto& c = m.cfg;
+    float* x = m.hidden.as<float>();
+    gptrs_norm_step base = {};
+    base.d_x = x; base.y_dtype = f.act_dt; base.eps = c.norm_eps;
+    base.d_h = y.h.p; base.h_dtype = f.act_dt; base.ldh = f.ldw;
+    base.d_status = m.d_status.as<int32_t>();
+    base.rows = f.T; base.dim = c.d_model;
+    auto launch = [&](const gptrs_norm_step& s) { ++m.launches; return gptrs_cuda_norm_step(&s, f.st); };
+    // the output of the sublayer that has just run, normed by `gamma`
+    auto closing = [&](const LayeredLayer& L, bool ff, Tensor* gamma) {
+        gptrs_norm_step s = base;
+        s.d_gamma_out = f.fp(gamma);
+        if (ff && L.cfg.mlp == GPTRS_MLP_EXPERTS) {
+            s.d_y = y.expert_y.p; s.ldy = L.w->down.n;
+            s.d_pair = y.pair.as<int32_t>(); s.d_pair_weight = y.pair_weight.as<float>(); s.top = L.moe.top;
+        } else {
+            s.d_y = y.y.p; s.ldy = f.ldw;
+        }
+        return s;
+    };
+    gptrs_norm_step open = base;
+    open.d_embed = f.fp(m.tok_emb); open.d_pos_embed = f.fp(m.pos_emb);
+    open.d_tokens = m.d_tokens.as<int32_t>(); open.d_pos = f.pos();
+    open.vocab = c.vocab; open.positions = y.cfg.learned_positions;
+    open.d_gamma_in = f.fp(y.layers[0].w->norm1);
+    int rc = launch(open);
+    if (rc) return rc;
+    for (int l = 0; l < c.n_layers; ++l) {
+        LayeredLayer& L = y.layers[l];
+        const bool last = l + 1 == c.n_layers, ff = L.cfg.mlp != GPTRS_MLP_NONE;
+        if ((rc = f.mixer(L))) return rc;
+        if (ff) {
+            gptrs_norm_step s = closing(L, false, L.w->norm1b);
+            s.d_gamma_in = f.fp(L.w->norm2);
+            if ((rc = launch(s)) || (rc = f.feed_forward(L))) return rc;
+        }
+        gptrs_norm_step s = closing(L, ff, ff ? L.w->norm2b : L.w->norm1b);
+        if (!last || cap.buf.p) {
+            s.d_gamma_in = last ? nullptr : f.fp(y.layers[l + 1].w->norm1);
+            if ((rc = launch(s)) || (rc = cap.take(m, l, x, f.T))) return rc;
+        }
+        if (last) {
+            if (cap.buf.p) s.d_y = nullptr;   // the stream already holds it
+            s.d_gamma_in = f.fp(m.final_g);
+            s.d_rows = rows_identity ? nullptr : m.d_rows.as<int32_t>();
+            s.d_h = m.xn_rows.p;
+            s.rows = n_rows;
+            if ((rc = launch(s))) return rc;
+        }
     }
+    return GPTRS_OK;
+}
+
+}  // namespace
+
+int layered_forward(Model& m, int T, int max_ctx, int n_rows, bool rows_identity, float temperature, bool skip_logits) {
+    Layered& y = *m.lay;
+    const auto& c = m.cfg;
+    Pass f = {m, y, T, max_ctx, m.f32() ? GPTRS_F32 : GPTRS_BF16, m.f32() ? (int64_t)c.d_model : pad8(c.d_model), m.stream};
+    cudaStream_t st = m.stream;
+    Capture cap;
+    int rc = cap.begin(m, T);
+    if (!rc) rc = y.cfg.block == GPTRS_BLOCK_SANDWICH ? forward_sandwich(f, cap, n_rows, rows_identity) : forward_output_norm(f, cap, n_rows, rows_identity);
+    if (!rc) rc = cap.end(m);
+    if (rc) return rc;
     const bool padded = y.head.n != c.vocab;
     const bool pick = skip_logits && m.fuse_pick && temperature <= 0.f && !m.f32() && !padded && n_rows <= 128;
     DenseOpts oh;

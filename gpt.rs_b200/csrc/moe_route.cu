@@ -1,0 +1,259 @@
+// Mixture of experts: which experts a row goes to, and the order of rows in which the grouped matmuls (dense_bf16.cu, dense_f32.cu)
+// find every expert's rows next to one another (no counterpart in gpt.rs).
+//   moe_choose_kernel   a warp per row: softmax over all experts, best groups, best experts of those; counts per expert
+//   moe_plan            row offsets of the experts and the tile list of the grouped matmuls; with few rows the tail of the kernel above,
+//                       otherwise a kernel of its own
+//   moe_gather_kernel   copies every row to its places
+// Where a row lies among its expert's rows depends on the order of atomic additions; no value depends on it.
+#include "common.cuh"
+
+namespace gptrs {
+namespace {
+
+struct Params {
+    gptrs_moe a;
+    const float* logits;
+    int64_t ld;
+    const unsigned char* h;
+    unsigned char* sorted;
+    int row_bytes;
+    int* pair;
+    float* weight;
+    gptrs_row_tile* tiles;
+    int* n_tiles;
+    int *counts, *offsets, *id, *place;   // [experts], [experts], [rows][top], [rows][top]
+    int rows, per_cta;
+};
+constexpr int kMaxExperts = 1024;
+constexpr int kWarps = 32;
+
+// order-preserving map of floats to signed integers
+__device__ __forceinline__ int order_of(float v) {
+    const int b = __float_as_int(v);
+    return b ^ ((b >> 31) & 0x7fffffff);
+}
+
+// inclusive sum over the 1024 threads of a CTA
+__device__ __forceinline__ int cta_scan(int v, int* sh) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) { const int u = __shfl_up_sync(0xffffffffu, v, o); if (lane >= o) v += u; }
+    __syncthreads();
+    if (lane == 31) sh[warp] = v;
+    __syncthreads();
+    if (warp == 0) {
+        int w = sh[lane];
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) { const int u = __shfl_up_sync(0xffffffffu, w, o); if (lane >= o) w += u; }
+        sh[lane] = w;
+    }
+    __syncthreads();
+    return v + (warp > 0 ? sh[warp - 1] : 0);
+}
+
+__device__ __forceinline__ void moe_plan(const Params& p, int* sh) {
+    const int e = threadIdx.x;
+    const int n = e < p.a.experts ? p.counts[e] : 0, nt = (n + p.a.tile_rows - 1) / p.a.tile_rows;
+    const int end = cta_scan(n, sh), t_end = cta_scan(nt, sh);
+    if (e < p.a.experts) {
+        const int r0 = end - n;
+        p.offsets[e] = r0;
+        p.counts[e] = 0;   // for the next call
+        for (int t = 0; t < nt; ++t) {
+            const gptrs_row_tile tile = {e, r0 + t * p.a.tile_rows, min(p.a.tile_rows, n - t * p.a.tile_rows), 0};
+            p.tiles[t_end - nt + t] = tile;
+        }
+    }
+    if (e == kWarps * 32 - 1) *p.n_tiles = t_end;
+}
+
+template <int VPL>
+__global__ void __launch_bounds__(kWarps * 32) moe_choose_kernel(const Params p) {
+    __shared__ int hist[kMaxExperts], sh[32];
+    extern __shared__ int mc_groups[];   // [warps][groups]: best score of every group, then whether it takes part
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int E = p.a.experts, G = p.a.groups, size = E / G;
+    int* gm = mc_groups + warp * G;
+    pdl_launch_dependents();
+    pdl_wait();
+    for (int e = tid; e < E; e += kWarps * 32) hist[e] = 0;
+    __syncthreads();
+    const int r_lo = blockIdx.x * p.per_cta, r_hi = min(r_lo + p.per_cta, p.rows);
+    for (int row = r_lo + warp; row < r_hi; row += kWarps) {
+        float z[VPL];
+        float mx = -INFINITY;
+#pragma unroll
+        for (int i = 0; i < VPL; ++i) {
+            const int e = i * 32 + lane;
+            z[i] = e < E ? p.logits[(size_t)row * p.ld + e] : -INFINITY;
+            mx = fmaxf(mx, z[i]);
+        }
+        mx = warp_max(mx);
+        float sum = 0.f;
+#pragma unroll
+        for (int i = 0; i < VPL; ++i) sum += i * 32 + lane < E ? expf(z[i] - mx) : 0.f;
+        sum = warp_sum(sum);
+        if (p.a.keep < G) {
+            const int none = (int)0x80000000;
+            for (int g = lane; g < G; g += 32) gm[g] = none;
+            __syncwarp();
+#pragma unroll
+            for (int i = 0; i < VPL; ++i)
+                if (i * 32 + lane < E) atomicMax(gm + (i * 32 + lane) / size, order_of(z[i]));
+            __syncwarp();
+            for (int n = 0; n < p.a.keep; ++n) {
+                int best = none, at = 0x7fffffff;
+                for (int g = lane; g < G; g += 32)
+                    if (gm[g] != 0x7fffffff && (gm[g] > best || at == 0x7fffffff)) { best = gm[g]; at = g; }
+#pragma unroll
+                for (int o = 16; o > 0; o >>= 1) {
+                    const int ob = __shfl_xor_sync(0xffffffffu, best, o), oa = __shfl_xor_sync(0xffffffffu, at, o);
+                    if (oa != 0x7fffffff && (at == 0x7fffffff || ob > best || (ob == best && oa < at))) { best = ob; at = oa; }
+                }
+                __syncwarp();
+                if (lane == 0 && at < G) gm[at] = 0x7fffffff;   // taken
+                __syncwarp();
+            }
+#pragma unroll
+            for (int i = 0; i < VPL; ++i)
+                if (i * 32 + lane < E && gm[(i * 32 + lane) / size] != 0x7fffffff) z[i] = -INFINITY;
+            __syncwarp();
+        }
+        for (int k = 0; k < p.a.top; ++k) {
+            float best = -INFINITY;
+            int at = 0x7fffffff;
+#pragma unroll
+            for (int i = 0; i < VPL; ++i)
+                if (z[i] > best) { best = z[i]; at = i * 32 + lane; }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+                const int oa = __shfl_xor_sync(0xffffffffu, at, o);
+                if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
+            }
+            if (at >= E) at = 0;   // only where logits are not numbers
+#pragma unroll
+            for (int i = 0; i < VPL; ++i)
+                if (i * 32 + lane == at) z[i] = -INFINITY;
+            if (lane == 0) {
+                const size_t o = (size_t)row * p.a.top + k;
+                p.weight[o] = expf(best - mx) / sum;
+                p.id[o] = at;
+                p.place[o] = atomicAdd(hist + at, 1);
+            }
+        }
+    }
+    __syncthreads();
+    if (gridDim.x == 1) {   // few rows: this CTA has seen them all
+        for (int e = tid; e < E; e += kWarps * 32) p.counts[e] = hist[e];
+        __syncthreads();
+        moe_plan(p, sh);
+        return;
+    }
+    for (int e = tid; e < E; e += kWarps * 32) hist[e] = hist[e] > 0 ? atomicAdd(p.counts + e, hist[e]) : 0;   // first place of this CTA's rows
+    __syncthreads();
+    for (int i = r_lo * p.a.top + tid; i < r_hi * p.a.top; i += kWarps * 32) p.place[i] += hist[p.id[i]];
+}
+
+__global__ void __launch_bounds__(kWarps * 32) moe_plan_kernel(const Params p) {
+    __shared__ int sh[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    moe_plan(p, sh);
+}
+
+// a CTA per (row, k)
+__global__ void __launch_bounds__(128) moe_gather_kernel(const Params p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int row = blockIdx.x, k = blockIdx.y;
+    const size_t o = (size_t)row * p.a.top + k;
+    const int dst = p.offsets[p.id[o]] + p.place[o];
+    if (threadIdx.x == 0) p.pair[o] = dst;
+    const unsigned char* s = p.h + (size_t)row * p.row_bytes;
+    unsigned char* d = p.sorted + (size_t)dst * p.row_bytes;
+    if (p.row_bytes % 16 == 0)
+        for (int i = threadIdx.x * 16; i < p.row_bytes; i += 128 * 16) *reinterpret_cast<uint4*>(d + i) = *reinterpret_cast<const uint4*>(s + i);
+    else
+        for (int i = threadIdx.x * 4; i < p.row_bytes; i += 128 * 4) *reinterpret_cast<uint32_t*>(d + i) = *reinterpret_cast<const uint32_t*>(s + i);
+}
+
+struct PairParams { const float* x; float* y; int n; };
+__global__ void __launch_bounds__(128) swiglu_pairs_kernel(const PairParams p) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const float* x = p.x + (size_t)blockIdx.x * 2 * p.n;
+    for (int i = threadIdx.x; i < p.n; i += 128) {
+        const int c = (i >> 3) * 16 + (i & 7);
+        const float g = x[c];
+        p.y[(size_t)blockIdx.x * p.n + i] = g / (1.f + expf(-g)) * x[c + 8];
+    }
+}
+
+template <int VPL>
+int launch_choose(const Params& p, int ctas, size_t smem, cudaStream_t st) {
+    if (smem > 40 * 1024) GPTRS_CUDA_OK(cudaFuncSetAttribute(moe_choose_kernel<VPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    return launch_kernel(moe_choose_kernel<VPL>, dim3((unsigned)ctas), dim3(kWarps * 32), smem, st, 1, p);
+}
+
+int check(const gptrs_moe* a) {
+    GPTRS_REQUIRE(a && a->experts > 0 && a->top > 0 && a->groups > 0 && a->keep > 0 && a->tile_rows > 0, "experts: sizes must be positive");
+    GPTRS_REQUIRE(a->experts % a->groups == 0 && a->keep <= a->groups && a->top <= a->keep * (a->experts / a->groups), "experts: groups must be equal and hold enough experts");
+    if (a->experts > kMaxExperts) return fail(GPTRS_UNIMPLEMENTED, "experts: more than 1024");
+    return GPTRS_OK;
+}
+
+}  // namespace
+}  // namespace gptrs
+
+using namespace gptrs;
+
+extern "C" {
+
+int64_t gptrs_cuda_moe_max_tiles(const gptrs_moe* a, int64_t rows) {
+    if (!a || a->tile_rows < 1 || rows < 0) return 0;
+    const int64_t pairs = rows * a->top;
+    return (pairs < a->experts ? pairs : a->experts) + pairs / a->tile_rows;
+}
+
+int64_t gptrs_cuda_moe_work_ints(const gptrs_moe* a, int64_t rows) { return a ? 2 * (int64_t)a->experts + 2 * rows * a->top : 0; }
+
+int gptrs_cuda_moe_route(const gptrs_moe* a, const float* d_logits, int64_t ld, const void* d_h, int h_dtype, int64_t ldh, int32_t* d_pair, float* d_weight,
+                         gptrs_row_tile* d_tiles, int32_t* d_n_tiles, void* d_sorted, int32_t* d_work, int64_t rows, void* stream) {
+    int rc = check(a);
+    if (rc) return rc;
+    GPTRS_REQUIRE(d_logits && d_h && d_pair && d_weight && d_tiles && d_n_tiles && d_sorted && d_work, "null pointer");
+    GPTRS_REQUIRE(ld >= a->experts && ldh > 0 && rows >= 0 && rows * a->top < (1ll << 30), "bad shape");
+    GPTRS_REQUIRE(h_dtype == GPTRS_F32 || (h_dtype == GPTRS_BF16 && ldh % 2 == 0), "rows of f32, or of an even number of bf16");
+    if (rows == 0) return GPTRS_OK;
+    Params p = {};
+    p.a = *a; p.logits = d_logits; p.ld = ld;
+    p.h = static_cast<const unsigned char*>(d_h); p.sorted = static_cast<unsigned char*>(d_sorted);
+    p.row_bytes = (int)(ldh * (h_dtype == GPTRS_F32 ? 4 : 2));
+    p.pair = d_pair; p.weight = d_weight; p.tiles = d_tiles; p.n_tiles = d_n_tiles;
+    p.counts = d_work; p.offsets = d_work + a->experts; p.id = p.offsets + a->experts; p.place = p.id + rows * a->top;
+    p.rows = (int)rows;
+    p.per_cta = rows <= 128 ? (int)rows : 64;
+    const int ctas = ceil_div(rows, p.per_cta);
+    cudaStream_t st = as_stream(stream);
+    const size_t smem = (size_t)kWarps * a->groups * 4;
+    const int vpl = ceil_div(a->experts, 32);
+    if (vpl <= 1) rc = launch_choose<1>(p, ctas, smem, st);
+    else if (vpl <= 2) rc = launch_choose<2>(p, ctas, smem, st);
+    else if (vpl <= 4) rc = launch_choose<4>(p, ctas, smem, st);
+    else if (vpl <= 8) rc = launch_choose<8>(p, ctas, smem, st);
+    else rc = launch_choose<32>(p, ctas, smem, st);
+    if (!rc && ctas > 1) rc = launch_kernel(moe_plan_kernel, dim3(1), dim3(kWarps * 32), 0, st, 1, p);
+    if (rc) return rc;
+    return launch_kernel(moe_gather_kernel, dim3((unsigned)rows, (unsigned)a->top), dim3(128), 0, st, 1, p);
+}
+
+int gptrs_cuda_swiglu_pairs_f32(const float* d_gate_up, float* d_y, int64_t rows, int64_t n, void* stream) {
+    GPTRS_REQUIRE(d_gate_up && d_y, "null pointer");
+    GPTRS_REQUIRE(rows >= 0 && rows < (1ll << 31) && n > 0 && n % 8 == 0 && n < (1ll << 30), "bad shape");
+    if (rows == 0) return GPTRS_OK;
+    const PairParams p = {d_gate_up, d_y, (int)n};
+    return launch_kernel(swiglu_pairs_kernel, dim3((unsigned)rows), dim3(128), 0, as_stream(stream), 1, p);
+}
+
+}  // extern "C"

@@ -20,8 +20,10 @@ from . import check, lib
 
 KIND_GPT, KIND_MINISTRAL, KIND_LAYERED = 0, 1, 2
 MODE_F32, MODE_W4A16, MODE_W8A16, MODE_BF16 = 0, 1, 2, 3
-MIXER_LATENT_ATTENTION = 0
-MLP_NONE, MLP_DENSE_XIELU = 0, 1
+MIXER_LATENT_ATTENTION, MIXER_GROUPED_ATTENTION, MIXER_CHANNEL_DELTA = 0, 1, 2
+MLP_NONE, MLP_DENSE_XIELU, MLP_EXPERTS = 0, 1, 2
+BLOCK_OUTPUT_NORM, BLOCK_SANDWICH = 0, 1
+MASK_CAUSAL, MASK_WINDOW, MASK_CHUNK = 0, 1, 2
 
 
 class _ModelConfig(ctypes.Structure):
@@ -42,32 +44,89 @@ class _LayerConfig(ctypes.Structure):
         ("mixer", ctypes.c_int), ("heads", ctypes.c_int), ("dim", ctypes.c_int), ("rot_dim", ctypes.c_int), ("rot_dims", ctypes.c_int),
         ("vdim", ctypes.c_int), ("kv_rank", ctypes.c_int), ("window", ctypes.c_int), ("scale", ctypes.c_float),
         ("rope_base", ctypes.c_double), ("mlp", ctypes.c_int), ("d_ff", ctypes.c_int),
+        ("kv_heads", ctypes.c_int), ("mask", ctypes.c_int), ("mask_size", ctypes.c_int), ("distance_bias", ctypes.c_int), ("proj_bias", ctypes.c_int),
+        ("softcap", ctypes.c_float), ("taps", ctypes.c_int), ("decay_rank", ctypes.c_int), ("gate_rank", ctypes.c_int),
+        ("experts", ctypes.c_int), ("top", ctypes.c_int), ("groups", ctypes.c_int), ("keep", ctypes.c_int), ("weights_of", ctypes.c_int),
     ]
 
 
 class _LayeredConfig(ctypes.Structure):
-    _fields_ = [("conv_taps", ctypes.c_int), ("logit_softcap", ctypes.c_float)]
+    _fields_ = [("conv_taps", ctypes.c_int), ("logit_softcap", ctypes.c_float), ("block", ctypes.c_int), ("learned_positions", ctypes.c_int)]
 
 
 @dataclass
 class LayerConfig:
-    """One layer of a model of the layered kind: its mixer (latent attention in a sliding window) and its feed-forward."""
+    """One layer of a model of the layered kind: its mixer and its feed-forward. Latent attention (in a sliding window) takes heads
+    .. rot_dims; attention with grouped key / value heads takes heads, dim, vdim, scale and kv_heads .. softcap; the delta rule takes
+    heads, dim, vdim, kv_heads and taps .. gate_rank. Experts have the size d_ff each."""
     heads: int
-    dim: int            # query / key dimensions of a head that are not rotated
-    rot_dim: int        # and those that are (shared key part)
-    vdim: int
-    kv_rank: int
-    window: int
-    scale: float
+    dim: int            # query / key dimensions of a head (latent attention: those that are not rotated)
+    rot_dim: int = 0    # and those that are (shared key part)
+    vdim: int = 0
+    kv_rank: int = 0
+    window: int = 0
+    scale: float = 1.0
     rope_base: float = 10000.0
     rot_dims: int = 0   # rotated dimensions of the rot_dim part (0 = all)
     mixer: int = MIXER_LATENT_ATTENTION
     mlp: int = MLP_DENSE_XIELU
     d_ff: int = 0
+    kv_heads: int = 0
+    mask: int = MASK_CAUSAL
+    mask_size: int = 0
+    distance_bias: int = 0   # a penalty r1 ln(1 + r2 distance) per head
+    proj_bias: int = 0       # biases on the four projections
+    softcap: float = 0.0     # of the scores
+    taps: int = 0
+    decay_rank: int = 0
+    gate_rank: int = 0
+    experts: int = 0
+    top: int = 0
+    groups: int = 1
+    keep: int = 1
+    weights_of: int = -1     # layer whose weights this one uses
 
     def _struct(self):
-        return _LayerConfig(self.mixer, self.heads, self.dim, self.rot_dim, self.rot_dims or self.rot_dim, self.vdim, self.kv_rank, self.window,
-                            self.scale, self.rope_base, self.mlp, self.d_ff)
+        values = {f: getattr(self, f) for f, _ in _LayerConfig._fields_}
+        values["rot_dims"] = self.rot_dims or self.rot_dim
+        return _LayerConfig(**values)
+
+    def shapes(self, p: str, d: int, sandwich: bool, conv_taps: int) -> dict[str, tuple[int, ...]]:
+        """Names and shapes of the layer's parameters (prefix `p`, width `d`)."""
+        if self.weights_of >= 0:
+            return {}
+        out: dict[str, tuple[int, ...]] = {f"{p}.norm1": (d,)}
+        out.update({f"{p}.norm1b": (d,)} if sandwich else {f"{p}.canon1": (d, conv_taps)})
+        x, qk, v = f"{p}.mix", self.heads * self.dim, self.heads * self.vdim
+        if self.mixer == MIXER_LATENT_ATTENTION:
+            out.update({f"{x}.q": (self.heads * (self.dim + self.rot_dim), d), f"{x}.dkv": (self.kv_rank + self.rot_dim, d), f"{x}.dkv.norm": (self.kv_rank,),
+                        f"{x}.uk": (qk, self.kv_rank), f"{x}.uv": (v, self.kv_rank), f"{x}.o": (d, v)})
+        elif self.mixer == MIXER_GROUPED_ATTENTION:
+            rows = {"q": qk, "k": self.kv_heads * self.dim, "v": self.kv_heads * self.vdim}
+            out.update({f"{x}.{n}": (r, d) for n, r in rows.items()})
+            out[f"{x}.o"] = (d, v)
+            if self.proj_bias:
+                out.update({f"{x}.{n}.b": (r,) for n, r in {**rows, "o": d}.items()})
+            if self.distance_bias:
+                out.update({f"{x}.r1": (self.heads,), f"{x}.r2": (self.heads,)})
+        else:
+            kq = self.kv_heads * self.dim
+            for n, r in (("q", kq), ("k", kq), ("v", v)):
+                out.update({f"{x}.{n}": (r, d), f"{x}.{n}.conv": (r, self.taps)})
+            out.update({f"{x}.b": (self.heads, d), f"{x}.A_log": (self.heads,), f"{x}.a1": (self.decay_rank, d), f"{x}.a2": (qk, self.decay_rank),
+                        f"{x}.dt_bias": (qk,), f"{x}.g1": (self.gate_rank, d), f"{x}.g2": (v, self.gate_rank), f"{x}.norm": (self.vdim,), f"{x}.o": (d, v)})
+        if self.mlp == MLP_NONE:
+            return out
+        f = f"{p}.mlp"
+        out[f"{p}.norm2"] = (d,)
+        out.update({f"{p}.norm2b": (d,)} if sandwich else {f"{p}.canon2": (d, conv_taps)})
+        if self.mlp == MLP_DENSE_XIELU:
+            out.update({f"{f}.up": (self.d_ff, d), f"{f}.up.b": (self.d_ff,), f"{f}.down": (d, self.d_ff), f"{f}.down.b": (d,), f"{f}.act": (2,)})
+        else:
+            for e in range(self.experts):
+                out.update({f"{f}.e{e}.gate": (self.d_ff, d), f"{f}.e{e}.up": (self.d_ff, d), f"{f}.e{e}.down": (d, self.d_ff)})
+            out[f"{f}.router"] = (self.experts, d)
+        return out
 
 
 @dataclass
@@ -96,9 +155,11 @@ class ModelConfig:
     layers: list | None = None     # layered kind: one LayerConfig per layer (the head and MLP sizes above are unused)
     conv_taps: int = 1
     logit_softcap: float = 0.0
+    block: int = BLOCK_OUTPUT_NORM
+    learned_positions: int = 0     # position vectors added to the embedding
 
     @staticmethod
-    def layered(layers, d_model: int, vocab: int, context_length: int, norm_eps: float, conv_taps: int, logit_softcap: float = 0.0, **kw):
+    def layered(layers, d_model: int, vocab: int, context_length: int, norm_eps: float, conv_taps: int = 1, logit_softcap: float = 0.0, **kw):
         return ModelConfig(KIND_LAYERED, len(layers), d_model, 0, 0, 0, 0, vocab, context_length, norm_eps, layers=list(layers),
                            conv_taps=conv_taps, logit_softcap=logit_softcap, **kw)
 
@@ -156,26 +217,14 @@ class ModelConfig:
 
     def _layered_shapes(self) -> dict[str, tuple[int, ...]]:
         """Names and shapes of the layered kind; Linear weights are [out, in]."""
-        d = self.d_model
-        out: dict[str, tuple[int, ...]] = {"embed": (self.vocab, d), "embed.norm": (d,)}
+        d, sandwich = self.d_model, self.block == BLOCK_SANDWICH
+        out: dict[str, tuple[int, ...]] = {"embed": (self.vocab, d)}
+        if not sandwich:
+            out["embed.norm"] = (d,)
+        if self.learned_positions:
+            out["pos"] = (self.learned_positions, d)
         for l, c in enumerate(self.layers):
-            p = f"l{l}"
-            out[f"{p}.norm1"] = (d,)
-            out[f"{p}.canon1"] = (d, self.conv_taps)
-            out[f"{p}.mix.q"] = (c.heads * (c.dim + c.rot_dim), d)
-            out[f"{p}.mix.dkv"] = (c.kv_rank + c.rot_dim, d)
-            out[f"{p}.mix.dkv.norm"] = (c.kv_rank,)
-            out[f"{p}.mix.uk"] = (c.heads * c.dim, c.kv_rank)
-            out[f"{p}.mix.uv"] = (c.heads * c.vdim, c.kv_rank)
-            out[f"{p}.mix.o"] = (d, c.heads * c.vdim)
-            if c.mlp != MLP_NONE:
-                out[f"{p}.norm2"] = (d,)
-                out[f"{p}.canon2"] = (d, self.conv_taps)
-                out[f"{p}.mlp.up"] = (c.d_ff, d)
-                out[f"{p}.mlp.up.b"] = (c.d_ff,)
-                out[f"{p}.mlp.down"] = (d, c.d_ff)
-                out[f"{p}.mlp.down.b"] = (d,)
-                out[f"{p}.mlp.act"] = (2,)
+            out.update(c.shapes(f"l{l}", d, sandwich, self.conv_taps))
         out["final.norm"] = (d,)
         out["head"] = (self.vocab, d)
         return out
@@ -208,7 +257,7 @@ class LoadedModel:
         check(lib().gptrs_cuda_model_create(ctypes.byref(c), ctypes.byref(self._h)))
         if config.kind == KIND_LAYERED:
             rows = (_LayerConfig * len(config.layers))(*[l._struct() for l in config.layers])
-            common = _LayeredConfig(config.conv_taps, config.logit_softcap)
+            common = _LayeredConfig(config.conv_taps, config.logit_softcap, config.block, config.learned_positions)
             check(lib().gptrs_cuda_model_set_layers(self._h, ctypes.byref(common), rows, len(config.layers)))
         self._finalized = False
 

@@ -71,9 +71,9 @@ class Replay:
 def load(model_dir, dtype: str, max_tokens: int) -> gm.LoadedModel:
     mode = gm.MODE_BF16 if dtype == "bfloat16" else gm.MODE_F32
     pool = (max_tokens + 63) // 64 * 64
-    described = ck.open_model(model_dir).model_config
-    kw = dict(context_length=pool) if described["kind"] == "bevosun" else {}   # the other kinds name theirs
-    vocab = ck.engine_config(described, mode, **kw)[0].vocab
+    reader = ck.open_model(model_dir)
+    kw = dict(context_length=pool) if reader.kind in ck.LAYERED_KINDS else {}   # the other kinds name theirs
+    vocab = ck.engine_config(reader.model_config, mode, ck.shapes_of(reader), **kw)[0].vocab
     logit_rows = max(1, min(pool, 2 ** 26 // vocab))
     return ck.load_model(model_dir, weight_mode=mode, max_seqs=SLOTS, max_tokens=min(pool, 8192), max_logit_rows=logit_rows, kv_pages=pool // PAGE,
                          max_pages_per_seq=pool // PAGE, **kw)

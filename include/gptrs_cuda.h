@@ -193,6 +193,7 @@ int gptrs_cuda_debug_matmul_fault(int starve, uint32_t spin_limit);
  * crates/gpt-rs/src/ops/functional/linalg.rs:109-127, tensor_ops.rs:42-56; the activations and the soft cap have no
  * counterpart in gpt.rs).
  * ============================================================================================ */
+typedef struct gptrs_row_tile { int32_t group, row0, rows, pad; } gptrs_row_tile;
 typedef struct {
     int out_dtype;             /* bf16 kernel: GPTRS_BF16 or GPTRS_F32 */
     const float* d_bias;       /* optional [n] */
@@ -207,6 +208,13 @@ typedef struct {
     int32_t* d_best_idx;
     int skip_store;
     int32_t* d_status;         /* bf16 kernel: receives 3 when a bounded wait gives up (required) */
+    /* grouped form (experts): rows [tile.row0, tile.row0 + tile.rows) of x meet matrix tile.group of the `batch` matrices, for
+     * the *d_n_tiles entries of d_tiles (gptrs_cuda_moe_route writes both); max_tiles bounds their number, tile_rows is the most
+     * rows a tile has. m is the number of rows behind x, the steps between matrices are those of the weights only. */
+    const struct gptrs_row_tile* d_tiles;
+    const int32_t* d_n_tiles;
+    int64_t max_tiles, tile_rows;
+    int swiglu;                /* bf16 kernel: 16 channels = 8 gates, then their 8 partners; y[m][n / 2] = silu(gate) partner */
 } gptrs_dense_epilogue;
 /* y[m][n] = act(x[m][k] . w[b][k][n] + bias), everything f32 (weights [in, out], nn/layers/linear.rs:14). */
 int gptrs_cuda_dense_f32(const float* d_x, const float* d_w, float* d_y, int64_t m, int64_t n, int64_t k,
@@ -291,6 +299,131 @@ int gptrs_cuda_latent_attention(const gptrs_latent_attention* a, const void* d_q
                                 int64_t max_pages, const int32_t* d_slot, const int32_t* d_ctx_len, const int32_t* d_tile_row,
                                 const int32_t* d_tile_rows, int64_t n_tiles, int splits, void* d_out, void* d_scratch,
                                 size_t scratch_bytes, int32_t* d_status, int64_t n_tokens, void* stream);
+
+/* ==============================================================================================
+ * Step between two sublayers of a model with a norm in front of and behind every sublayer (no counterpart in gpt.rs): for
+ * every row
+ *     x <- x + y / sqrt(mean(y^2) + eps) * gamma_out        h = x / sqrt(mean(x^2) + eps) * gamma_in
+ * d_embed set: x = embed[token] + pos_embed[position] instead (no first norm). d_y NULL: x stays. d_pair set: y is the sum over
+ * k < top of pair_weight[row][k] * d_y[pair[row][k]] (what the experts of a row put out). d_rows set: row i of the launch is row
+ * d_rows[i] of x and y, h is compact, and x is not written (the end of the model).
+ * ============================================================================================ */
+typedef struct {
+    float* d_x;
+    const void* d_y;
+    int y_dtype;
+    int64_t ldy;
+    const int32_t* d_pair;     /* [rows][top] */
+    const float* d_pair_weight;
+    int64_t top;
+    const float* d_embed;
+    const float* d_pos_embed;  /* optional [positions][dim] */
+    const int32_t* d_tokens;
+    const int32_t* d_pos;
+    int64_t vocab, positions;
+    const float* d_gamma_out;
+    const float* d_gamma_in;   /* NULL: no h */
+    float eps;
+    const int32_t* d_rows;
+    void* d_h;
+    int h_dtype;
+    int64_t ldh;               /* columns past dim are zeroed */
+    int32_t* d_status;         /* receives 2 for a token id or position out of range */
+    int64_t rows, dim;
+} gptrs_norm_step;
+int gptrs_cuda_norm_step(const gptrs_norm_step* step, void* stream);
+
+/* ==============================================================================================
+ * Attention with grouped key / value heads of any size over a paged cache (no counterpart in gpt.rs; the kernels further down
+ * serve gpt.rs' own attention): query head h reads key / value head h / (heads / kv_heads); scores are soft-capped, then
+ * r1[h] ln(1 + r2[h] (i - j)) is taken off; a mask says where the keys of position i begin. Pages of 16 tokens hold the
+ * [value | key] rows of every kv head.
+ * ============================================================================================ */
+enum { GPTRS_MASK_CAUSAL = 0, GPTRS_MASK_WINDOW = 1, GPTRS_MASK_CHUNK = 2 };   /* from 0; i - size + 1; floor(i / size) size */
+typedef struct {
+    int dtype;                 /* GPTRS_F32 or GPTRS_BF16: activations and cache */
+    int heads, kv_heads, dim, vdim;
+    int mask, mask_size;
+    float scale, softcap;      /* softcap 0 = none */
+    int distance_bias;         /* 1: r1 and r2 are given */
+    /* filled in by gptrs_cuda_grouped_layout (elements): */
+    int q_head_stride, k_offset, k_head_stride, v_offset, v_head_stride, q_row;   /* projection row: queries, keys, values */
+    int out_head_stride;       /* attention output of a head */
+    int64_t page_bytes;
+} gptrs_grouped_attention;
+int gptrs_cuda_grouped_layout(gptrs_grouped_attention* a);
+/* Keys and values of projection rows -> the tokens' pages. */
+int gptrs_cuda_grouped_append(const gptrs_grouped_attention* a, const void* d_qkv, const int32_t* d_positions, const int32_t* d_slot,
+                              const int32_t* d_page_table, int64_t max_pages, void* d_pool, int64_t n_tokens, void* stream);
+/* As for latent attention above: tokens of a query tile of the tensor-core kernel (0: these sizes use the plain kernel), key
+ * splits, scratch. */
+int gptrs_cuda_grouped_tile_tokens(const gptrs_grouped_attention* a);
+int gptrs_cuda_grouped_splits(const gptrs_grouped_attention* a, int64_t n_tiles, int64_t max_ctx_len);
+size_t gptrs_cuda_grouped_scratch_bytes(const gptrs_grouped_attention* a, int64_t n_tiles, int splits);
+/* out[T][heads][out_head_stride]; n_tiles = 0: the plain kernel. d_ctx_len[t] = position + 1. */
+int gptrs_cuda_grouped_attention(const gptrs_grouped_attention* a, const void* d_qkv, const void* d_pool, const int32_t* d_page_table,
+                                 int64_t max_pages, const int32_t* d_slot, const int32_t* d_ctx_len, const float* d_r1, const float* d_r2,
+                                 const int32_t* d_tile_row, const int32_t* d_tile_rows, int64_t n_tiles, int splits, void* d_out,
+                                 void* d_scratch, size_t scratch_bytes, int32_t* d_status, int64_t n_tokens, void* stream);
+
+/* ==============================================================================================
+ * Gated delta rule with a decay per key channel (no counterpart in gpt.rs). Per head a state S[dim][vdim] in f32:
+ *     S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+ * q, k (kv_heads x dim, shared by heads / kv_heads heads) and v come from short causal convolutions over time with silu; q and k
+ * are unit vectors, q times dim^(-1/2); g = exp(-exp(A_log_h) softplus(a + dt_bias)) per head and key channel; the output is
+ * o / rms(o) * norm * sigmoid(gate). Rows come in runs of consecutive positions of one sequence (run_first / run_last as above).
+ * The recurrent state is updated in place, the taps - 1 last inputs of the convolutions have two halves (parity as above).
+ * ============================================================================================ */
+typedef struct {
+    int dtype;                 /* GPTRS_F32 or GPTRS_BF16: projections and output */
+    int heads, kv_heads, dim, vdim, taps, decay_rank, gate_rank;
+    float eps;
+    /* filled in by gptrs_cuda_delta_layout (elements): */
+    int q_offset, k_offset, v_offset, beta_offset, a_offset, g_offset, row;   /* projection row: q, k, v, beta, decay and gate bottlenecks */
+    int decay_row, gate_row;   /* rows of the expanded decay (f32) and gate */
+    int out_head_stride;
+    int conv_channels;         /* 2 kv_heads dim + heads vdim: rows of d_conv, channels of the convolution state */
+    int64_t state_floats;      /* recurrent state of a slot: heads dim vdim */
+    int64_t conv_floats;       /* convolution state of a slot: 2 (taps - 1) conv_channels */
+    int64_t scratch_floats;    /* per row, for prompts */
+} gptrs_delta_rule;
+int gptrs_cuda_delta_layout(gptrs_delta_rule* a);
+typedef struct {
+    const void* d_proj;        /* [T][row] */
+    const float* d_decay;      /* [T][decay_row] */
+    const void* d_gate;        /* [T][gate_row] */
+    const float* d_conv;       /* [conv_channels][taps], the newest input under the last tap */
+    const float *d_a_log, *d_dt_bias, *d_norm;
+    float* d_state;            /* [slots][heads][dim][vdim] */
+    float* d_conv_state;       /* [slots][2][taps - 1][conv_channels] */
+    const int32_t *d_slot, *d_pos, *d_run_first, *d_run_last, *d_parity;
+    const int32_t* d_runs;     /* first row of every run */
+    int64_t n_runs;            /* n_runs = rows: every row is a run of its own (a decode step) */
+    void* d_out;               /* [T][heads][out_head_stride] */
+    float* d_scratch;          /* rows * scratch_floats, unless n_runs = rows */
+    int64_t rows;
+} gptrs_delta_step;
+int gptrs_cuda_delta_rule(const gptrs_delta_rule* a, const gptrs_delta_step* step, void* stream);
+
+/* ==============================================================================================
+ * Mixture of experts: routing and the row order of the grouped matmuls (no counterpart in gpt.rs). Scores are the softmax of the
+ * logits over all experts; the experts form `groups` equal groups of neighbours, those of the `keep` groups with the largest best
+ * score may be chosen; a row goes to its `top` best experts with their scores as weights.
+ * ============================================================================================ */
+typedef struct {
+    int experts, top, groups, keep;
+    int tile_rows;             /* rows of a tile of the grouped matmuls */
+} gptrs_moe;
+/* logits [rows][ld] -> d_pair[rows][top]: the row of x_sorted that belongs to (row, k), sorted by expert; d_weight[rows][top]; the
+ * tiles of every expert's rows (at most gptrs_cuda_moe_max_tiles) and their number; d_work: gptrs_cuda_moe_work_ints ints, zeroed
+ * before the first call. h [rows][ldh] -> d_sorted [rows * top][ldh]. */
+int64_t gptrs_cuda_moe_max_tiles(const gptrs_moe* a, int64_t rows);
+int64_t gptrs_cuda_moe_work_ints(const gptrs_moe* a, int64_t rows);
+int gptrs_cuda_moe_route(const gptrs_moe* a, const float* d_logits, int64_t ld, const void* d_h, int h_dtype, int64_t ldh, int32_t* d_pair,
+                         float* d_weight, gptrs_row_tile* d_tiles, int32_t* d_n_tiles, void* d_sorted, int32_t* d_work, int64_t rows,
+                         void* stream);
+/* f32 mode: y[r][i] = silu(gate) partner over rows of 2 n f32 in the order of the swiglu epilogue, for the first rows of d_tiles. */
+int gptrs_cuda_swiglu_pairs_f32(const float* d_gate_up, float* d_y, int64_t rows, int64_t n, void* stream);
 
 /* ==============================================================================================
  * Paged bf16 KV cache and decode attention (split-K flash decoding).
@@ -568,25 +701,42 @@ typedef struct {
     int tp_rank;
 } gptrs_model_config;
 
-/* Layered kind (no counterpart in gpt.rs): every layer has a configuration of its own. Norms sit on the outputs of the
- * sublayers, x <- x + rms(mixer(h)), x <- x + rms(ff(h)), and a sublayer reads h = x + conv(x), a causal convolution over the
- * last conv_taps positions of every channel whose last conv_taps - 1 inputs are part of a sequence's state. The embedding is
- * normed, the logits are soft-capped. Of gptrs_model_config the fields n_layers, d_model, vocab, context_length, norm_eps,
- * max_*, kv_pages and use_pdl apply. Both weight modes keep the cache in pages; rows of a sequence must arrive in order. Pages
- * that the windows of all layers have passed return to the pool. Parameter names ([out, in] weights): embed, embed.norm,
- * l<i>.norm1, .norm2, .canon1, .canon2, .mix.{q,dkv,dkv.norm,uk,uv,o}, .mlp.{up,up.b,down,down.b,act}, final.norm, head. */
-enum { GPTRS_MIXER_LATENT_ATTENTION = 0 };
-enum { GPTRS_MLP_NONE = 0, GPTRS_MLP_DENSE_XIELU = 1 };
+/* Layered kind (no counterpart in gpt.rs): every layer has a configuration of its own, a mixer and an optional feed-forward, in
+ * one of two block forms:
+ *   GPTRS_BLOCK_OUTPUT_NORM  norms on the outputs of the sublayers, x <- x + rms(mixer(h)), x <- x + rms(ff(h)); a sublayer reads
+ *                            h = x + conv(x), a causal convolution over the last conv_taps positions of every channel whose last
+ *                            conv_taps - 1 inputs are part of a sequence's state; the embedding is normed.
+ *   GPTRS_BLOCK_SANDWICH     norms on both sides, x <- x + rms(mixer(rms(x))), x <- x + rms(ff(rms(x))); with learned_positions a
+ *                            position vector is added to the embedding.
+ * The logits may be soft-capped. Of gptrs_model_config the fields n_layers, d_model, vocab, context_length, norm_eps, max_*,
+ * kv_pages and use_pdl apply. Both weight modes keep the cache in pages; rows of a sequence must arrive in order. Pages that the
+ * masks of all layers have passed return to the pool. A layer with weights_of >= 0 uses the weights of that layer (an equal
+ * configuration) with a cache and state of its own. Parameter names ([out, in] weights): embed, embed.norm | pos,
+ * l<i>.norm1, .norm2, .canon1, .canon2 | .norm1b, .norm2b, final.norm, head, and per mixer and feed-forward l<i>.mix. and l<i>.mlp.
+ *   latent attention   q, dkv, dkv.norm, uk, uv, o
+ *   grouped attention  q, q.b, k, k.b, v, v.b, r1, r2, o, o.b
+ *   channel delta      q, q.conv, k, k.conv, v, v.conv, b, A_log, a1, a2, dt_bias, g1, g2, norm, o
+ *   dense xIELU        up, up.b, down, down.b, act
+ *   experts            e<j>.gate, e<j>.up, e<j>.down, router */
+enum { GPTRS_MIXER_LATENT_ATTENTION = 0, GPTRS_MIXER_GROUPED_ATTENTION = 1, GPTRS_MIXER_CHANNEL_DELTA = 2 };
+enum { GPTRS_MLP_NONE = 0, GPTRS_MLP_DENSE_XIELU = 1, GPTRS_MLP_EXPERTS = 2 };
+enum { GPTRS_BLOCK_OUTPUT_NORM = 0, GPTRS_BLOCK_SANDWICH = 1 };
 typedef struct {
     int mixer;
     int heads, dim, rot_dim, rot_dims, vdim, kv_rank, window;
     float scale;
     double rope_base;
     int mlp, d_ff;
+    int kv_heads, mask, mask_size, distance_bias, proj_bias;   /* grouped attention */
+    float softcap;
+    int taps, decay_rank, gate_rank;                           /* channel delta (kv_heads too) */
+    int experts, top, groups, keep;                            /* experts of size d_ff */
+    int weights_of;                                            /* -1 = weights of its own */
 } gptrs_layer_config;
 typedef struct {
     int conv_taps;
     float logit_softcap;   /* 0 = none */
+    int block, learned_positions;
 } gptrs_layered_config;
 
 int gptrs_cuda_model_create(const gptrs_model_config* cfg, gptrs_model** out);

@@ -167,7 +167,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) flash_tc_kernel(const __grid_co
     const int heads0 = kvh * g.group + head_block * kRows;
     const int live = n_tok * heads_n;
     const int live_warps = (live + 31) / 32;
-    const bool dup = live <= kRows / 2 && (!GROUPED || n_tok == 1);
+    const bool dup = live <= kRows / 2 && (!GROUPED || (n_tok == 1 && p.rows_per_token <= kRows / 2));   // a box of queries lands twice
     if (tid == 0) {
         for (int i = 0; i < p.stages; ++i) { mbar_init(&k_full[i], 1); mbar_init(&k_empty[i], 1); }
         for (int i = 0; i < kScores; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], (uint32_t)live_warps * (dup ? 64 : 32)); }

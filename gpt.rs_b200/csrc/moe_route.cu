@@ -21,7 +21,7 @@ struct Params {
     float* weight;
     gptrs_row_tile* tiles;
     int* n_tiles;
-    int *counts, *offsets, *id, *place;   // [experts], [experts], [rows][top], [rows][top]
+    int *counts, *offsets, *id, *place;   // [kMaxExperts] each, [rows][top] each
     int rows, per_cta;
 };
 constexpr int kMaxExperts = 1024;
@@ -216,7 +216,7 @@ int64_t gptrs_cuda_moe_max_tiles(const gptrs_moe* a, int64_t rows) {
     return (pairs < a->experts ? pairs : a->experts) + pairs / a->tile_rows;
 }
 
-int64_t gptrs_cuda_moe_work_ints(const gptrs_moe* a, int64_t rows) { return a ? 2 * (int64_t)a->experts + 2 * rows * a->top : 0; }
+int64_t gptrs_cuda_moe_work_ints(const gptrs_moe* a, int64_t rows) { return a ? 2 * (int64_t)kMaxExperts + 2 * rows * a->top : 0; }
 
 int gptrs_cuda_moe_route(const gptrs_moe* a, const float* d_logits, int64_t ld, const void* d_h, int h_dtype, int64_t ldh, int32_t* d_pair, float* d_weight,
                          gptrs_row_tile* d_tiles, int32_t* d_n_tiles, void* d_sorted, int32_t* d_work, int64_t rows, void* stream) {
@@ -231,7 +231,8 @@ int gptrs_cuda_moe_route(const gptrs_moe* a, const float* d_logits, int64_t ld, 
     p.h = static_cast<const unsigned char*>(d_h); p.sorted = static_cast<unsigned char*>(d_sorted);
     p.row_bytes = (int)(ldh * (h_dtype == GPTRS_F32 ? 4 : 2));
     p.pair = d_pair; p.weight = d_weight; p.tiles = d_tiles; p.n_tiles = d_n_tiles;
-    p.counts = d_work; p.offsets = d_work + a->experts; p.id = p.offsets + a->experts; p.place = p.id + rows * a->top;
+    // the same places for every number of experts: the counts stay zero in between
+    p.counts = d_work; p.offsets = d_work + kMaxExperts; p.id = p.offsets + kMaxExperts; p.place = p.id + rows * a->top;
     p.rows = (int)rows;
     p.per_cta = rows <= 128 ? (int)rows : 64;
     const int ctas = ceil_div(rows, p.per_cta);

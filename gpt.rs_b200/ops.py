@@ -388,7 +388,9 @@ def _dense_epilogue(x, bias, xielu, softcap, strides, status):
     if xielu is not None:
         ep.act, ep.act_pos, ep.act_neg = 1, *xielu
     ep.softcap = softcap
-    for name, v in strides.items():   # ldx, ldy, batch, x_step, y_step
+    for name, v in strides.items():   # ldx, ldy, batch, x_step, y_step; tiles, n_tiles, max_tiles, tile_rows, swiglu
+        if name in ("tiles", "n_tiles"):
+            name, v = "d_" + name, _ptr(v)
         setattr(ep, name, v)
     ep.d_status = _ptr(status)
     return ep
@@ -402,7 +404,7 @@ def dense_bf16(x, w, m, n, k, out=None, out_f32=False, bias=None, xielu=None, so
     if best is not None:
         ep.d_best_val, ep.d_best_idx, ep.skip_store = _ptr(best[0]), _ptr(best[1]), 1
     if out is None:
-        out = torch.empty((m, n), dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device)
+        out = torch.empty((m, n // 2 if strides.get("swiglu") else n), dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device)
     check(lib().gptrs_cuda_dense_bf16(_ptr(x), _ptr(w), _ptr(out), m, n, k, ctypes.byref(ep), _stream()))
     return out
 
@@ -478,3 +480,102 @@ def latent_attention(a, qa, pool, page_table, slot, ctx_len, max_ctx_len, tiles=
 
 def latent_tile_tokens(a) -> int:
     return lib().gptrs_cuda_latent_tile_tokens(ctypes.byref(a))
+
+
+# ---- norms on both sides of a sublayer, grouped attention, delta rule, experts (layered models) ------------------------------
+def norm_step(x, eps, y=None, gamma_out=None, gamma_in=None, pair=None, pair_weight=None, embed=None, pos_embed=None, tokens=None, positions=None,
+              rows=None, out_dtype=torch.float32, ldh=None, status=None):
+    """x (f32, in place) <- x + rms_norm(y) gamma_out, or embedding rows; returns h = rms_norm(x) gamma_in (or None). `pair` and
+    `pair_weight` [rows][top]: y of a row is a weighted sum of rows of `y`."""
+    dev, (n, dim) = x.device, x.shape
+    s = _abi.NormStep()
+    s.d_x, s.eps, s.dim, s.d_status = _ptr(x), eps, dim, _ptr(_status(dev, status))
+    s.rows = n if rows is None else rows.shape[0]
+    s.d_rows = _ptr(rows)
+    if y is not None:
+        s.d_y, s.y_dtype, s.ldy, s.d_gamma_out = _ptr(y), _dt(y), y.shape[1], _ptr(gamma_out)
+    if pair is not None:
+        s.d_pair, s.d_pair_weight, s.top = _ptr(pair), _ptr(pair_weight), pair.shape[1]
+    if embed is not None:
+        s.d_embed, s.d_tokens, s.vocab = _ptr(embed), _ptr(tokens), embed.shape[0]
+        if pos_embed is not None:
+            s.d_pos_embed, s.d_pos, s.positions = _ptr(pos_embed), _ptr(positions), pos_embed.shape[0]
+    h = None
+    if gamma_in is not None:
+        h = torch.empty((s.rows, ldh or dim), dtype=out_dtype, device=dev)
+        s.d_gamma_in, s.d_h, s.h_dtype, s.ldh = _ptr(gamma_in), _ptr(h), _dt(h), h.shape[1]
+    check(lib().gptrs_cuda_norm_step(ctypes.byref(s), _stream()))
+    return h
+
+
+def grouped_layout(heads, kv_heads, dim, vdim, mask, mask_size, scale, softcap=0.0, distance_bias=False, bf16=True):
+    a = _abi.GroupedAttention(BF16 if bf16 else F32, heads, kv_heads, dim, vdim, mask, mask_size, scale, softcap, int(distance_bias))
+    check(lib().gptrs_cuda_grouped_layout(ctypes.byref(a)))
+    return a
+
+
+def grouped_append(a, qkv, positions, slot, page_table, pool):
+    check(lib().gptrs_cuda_grouped_append(ctypes.byref(a), _ptr(qkv), _ptr(positions), _ptr(slot), _ptr(page_table), page_table.shape[1], _ptr(pool),
+                                          qkv.shape[0], _stream()))
+
+
+def grouped_tile_tokens(a) -> int:
+    return lib().gptrs_cuda_grouped_tile_tokens(ctypes.byref(a))
+
+
+def grouped_attention(a, qkv, pool, page_table, slot, ctx_len, max_ctx_len, r1=None, r2=None, tiles=None, splits=None, status=None):
+    """out [T][heads][out_head_stride]; `tiles` = (first rows, row counts) for the tensor-core kernel, None for the plain one."""
+    status = _status(qkv.device, status)
+    n = slot.shape[0]
+    out = torch.empty((n, a.heads, a.out_head_stride), dtype=qkv.dtype, device=qkv.device)
+    n_tiles = 0 if tiles is None else tiles[0].shape[0]
+    if splits is None:
+        splits = lib().gptrs_cuda_grouped_splits(ctypes.byref(a), n_tiles, max_ctx_len) if n_tiles else 1
+    nbytes = lib().gptrs_cuda_grouped_scratch_bytes(ctypes.byref(a), n_tiles, splits)
+    scratch = torch.empty(max(nbytes, 1), dtype=torch.uint8, device=qkv.device)
+    check(lib().gptrs_cuda_grouped_attention(ctypes.byref(a), _ptr(qkv), _ptr(pool), _ptr(page_table), page_table.shape[1], _ptr(slot), _ptr(ctx_len), _ptr(r1),
+                                             _ptr(r2), None if tiles is None else _ptr(tiles[0]), None if tiles is None else _ptr(tiles[1]), n_tiles, splits,
+                                             _ptr(out), _ptr(scratch), nbytes, _ptr(status), n, _stream()))
+    return out, status
+
+
+def delta_layout(heads, kv_heads, dim, vdim, taps, decay_rank, gate_rank, eps, bf16=True):
+    a = _abi.DeltaRule(BF16 if bf16 else F32, heads, kv_heads, dim, vdim, taps, decay_rank, gate_rank, eps)
+    check(lib().gptrs_cuda_delta_layout(ctypes.byref(a)))
+    return a
+
+
+def delta_rule(a, proj, decay, gate, conv, a_log, dt_bias, norm, state, conv_state, runs, first_rows, n_runs=None):
+    """`runs` = (slot, pos, run_first, run_last, parity) per row, `first_rows` = first row of every run; states are updated in place."""
+    n = proj.shape[0]
+    out = torch.empty((n, a.heads, a.out_head_stride), dtype=proj.dtype, device=proj.device)
+    s = _abi.DeltaStep()
+    s.d_proj, s.d_decay, s.d_gate, s.d_conv, s.d_a_log, s.d_dt_bias, s.d_norm = (_ptr(t) for t in (proj, decay, gate, conv, a_log, dt_bias, norm))
+    s.d_state, s.d_conv_state = _ptr(state), _ptr(conv_state)
+    s.d_slot, s.d_pos, s.d_run_first, s.d_run_last, s.d_parity = (_ptr(t) for t in runs)
+    s.d_runs, s.n_runs, s.rows, s.d_out = _ptr(first_rows), first_rows.shape[0] if n_runs is None else n_runs, n, _ptr(out)
+    scratch = torch.empty(max(n * a.scratch_floats, 1), dtype=torch.float32, device=proj.device)
+    s.d_scratch = _ptr(scratch)
+    check(lib().gptrs_cuda_delta_rule(ctypes.byref(a), ctypes.byref(s), _stream()))
+    return out
+
+
+def moe_route(experts, top, groups, keep, tile_rows, logits, h, work=None):
+    """Returns (pair, weight, tiles, n_tiles, sorted rows, most tiles): see gptrs_cuda_moe_route."""
+    a = _abi.Moe(experts, top, groups, keep, tile_rows)
+    n, dev = logits.shape[0], logits.device
+    most = lib().gptrs_cuda_moe_max_tiles(ctypes.byref(a), n)
+    pair, weight = torch.empty((n, top), dtype=torch.int32, device=dev), torch.empty((n, top), device=dev)
+    tiles, n_tiles = torch.zeros((max(most, 1), 4), dtype=torch.int32, device=dev), torch.zeros(1, dtype=torch.int32, device=dev)
+    out = torch.empty((n * top, h.shape[1]), dtype=h.dtype, device=dev)
+    if work is None:
+        work = torch.zeros(lib().gptrs_cuda_moe_work_ints(ctypes.byref(a), n), dtype=torch.int32, device=dev)
+    check(lib().gptrs_cuda_moe_route(ctypes.byref(a), _ptr(logits), logits.shape[1], _ptr(h), _dt(h), h.shape[1], _ptr(pair), _ptr(weight), _ptr(tiles),
+                                     _ptr(n_tiles), _ptr(out), _ptr(work), n, _stream()))
+    return pair, weight, tiles, n_tiles, out, most
+
+
+def swiglu_pairs_f32(gate_up, n):
+    out = torch.empty((gate_up.shape[0], n), device=gate_up.device)
+    check(lib().gptrs_cuda_swiglu_pairs_f32(_ptr(gate_up), _ptr(out), gate_up.shape[0], n, _stream()))
+    return out

@@ -416,7 +416,7 @@ typedef struct {
 } gptrs_moe;
 /* logits [rows][ld] -> d_pair[rows][top]: the row of x_sorted that belongs to (row, k), sorted by expert; d_weight[rows][top]; the
  * tiles of every expert's rows (at most gptrs_cuda_moe_max_tiles) and their number; d_work: gptrs_cuda_moe_work_ints ints, zeroed
- * before the first call. h [rows][ldh] -> d_sorted [rows * top][ldh]. */
+ * before the first call (calls of different configurations may share it). h [rows][ldh] -> d_sorted [rows * top][ldh]. */
 int64_t gptrs_cuda_moe_max_tiles(const gptrs_moe* a, int64_t rows);
 int64_t gptrs_cuda_moe_work_ints(const gptrs_moe* a, int64_t rows);
 int gptrs_cuda_moe_route(const gptrs_moe* a, const float* d_logits, int64_t ld, const void* d_h, int h_dtype, int64_t ldh, int32_t* d_pair,

@@ -12,6 +12,7 @@ may reuse an earlier layer's weights. Nothing under gpt.rs_b200/ may import this
 """
 from __future__ import annotations
 
+import copy
 import json
 import struct
 from pathlib import Path
@@ -206,7 +207,7 @@ def delta_layer(heads=4, kv_heads=2, dim=16, vdim=24, conv=3, mlp=moe()):
 
 def again(layers, j):
     """The entry of a layer that reuses layer j's weights."""
-    return {**layers[j], "weights_of": j}
+    return {**copy.deepcopy(layers[j]), "weights_of": j}
 
 
 def model_config(layers, width=40, vocab=72, eps=1e-5, positions=1024):
@@ -271,6 +272,50 @@ def random_tensors(cfg, seed=0, **ranks):
             w = rng.standard_normal(shape) / np.sqrt(shape[-1])
         out[name] = to_bf16(w.astype(np.float32))
     return out
+
+
+CODE = 8   # width reserved by `steady_routing`
+
+
+def steady_routing(cfg, tensors, seed=0, margin=0.12):
+    """Weights whose routers read the last CODE channels of the stream only, where every token keeps a code of its own that no layer
+    adds to, drawn so that no choice of experts or groups is close: rounding then never changes an expert."""
+    rng = np.random.default_rng(seed)
+    t = {n: w.copy() for n, w in tensors.items()}
+    routers = []
+    t["pos"][:, -CODE:] = 0
+    for i, layer in enumerate(cfg["layers"]):
+        if "weights_of" in layer:
+            continue
+        t[f"l{i}.norm1b"][-CODE:] = 0
+        if not layer["mlp"]:
+            continue
+        t[f"l{i}.norm2b"][-CODE:] = 0
+        t[f"l{i}.norm2"][-CODE:] = 1
+        w = t[f"l{i}.mlp.router"]
+        w[:, :-CODE] = 0
+        w[:, -CODE:] = to_bf16(rng.standard_normal((w.shape[0], CODE)).astype(np.float32))
+        r = layer["mlp"]["router"]
+        routers.append((w[:, -CODE:].astype(D), r["top"], r["groups"]["count"], r["groups"]["keep"]))
+
+    def decided(z, top, count, keep):
+        best = np.sort(z.reshape(count, -1).max(axis=1))[::-1]
+        if keep < count and best[keep - 1] - best[keep] < margin * np.abs(z).max():
+            return False
+        chosen, _ = route(z, top, count, keep)
+        allowed = np.isin(np.arange(len(z)) // (len(z) // count), np.argsort(-z.reshape(count, -1).max(axis=1), kind="stable")[:keep])
+        rest = np.setdiff1d(np.nonzero(allowed)[0], chosen)
+        return len(rest) == 0 or z[chosen].min() - z[rest].max() >= margin * np.abs(z).max()
+
+    for v in range(cfg["vocab"]):
+        for _ in range(20000):
+            code = to_bf16((1.5 * rng.standard_normal(CODE)).astype(np.float32))
+            if all(decided(w @ code, *r) for w, *r in routers):
+                break
+        else:
+            raise ValueError("no code with this margin")
+        t["embed"][v, -CODE:] = code
+    return t
 
 
 def write_model(folder, cfg, tensors):

@@ -304,8 +304,11 @@ def _random_model(gm, torch, dev, cfg, namespace):
     m = gm.LoadedModel(cfg, namespace=ck.next_namespace() * 1000 + namespace)
     g = torch.Generator(device=dev).manual_seed(0)
     for name, shape in cfg.param_shapes().items():
-        if name.endswith("gamma") or "norm" in name.rsplit(".", 1)[-1]:
+        last = name.rsplit(".", 1)[-1]
+        if name.endswith("gamma") or "norm" in last:
             t = torch.ones(shape, device=dev)
+        elif last in ("r1", "r2", "dt_bias"):   # distance penalties are positive, decays slow
+            t = torch.full(shape, -3.0 if last == "dt_bias" else 0.3, device=dev)
         else:
             t = torch.empty(shape, device=dev).normal_(0.0, 0.02, generator=g)
         m.load_param(name, t)
@@ -503,6 +506,168 @@ def run_layered_kernels(args, out, ops, torch):
         rec[f"latent_decode_attention_ctx{ctx}"] = time_layered_kernels(ops, torch, dev, size, 64 if ctx == 8192 else 16, ctx, only_attention=True)["attention"]
     pre, flops = time_prefill_attention(ops, torch, dev, PROMPT_LEN)
     rec["like_prefill_attention"] = {"us": pre["paged_prefill_tc_kernel"]["us"], "frac": round(pre["paged_prefill_tc_kernel"]["tflops"] / _tensor_peak(), 3)}
+    print(json.dumps(rec), file=out)
+
+
+# ---- Felepel beside Bevosun -------------------------------------------------------------------------------------------------------
+# name -> attention (heads, kv heads, dim, vdim, chunk), delta rule (heads, q/k heads, dim, vdim, taps, ranks), experts (number, top,
+# groups, kept groups, size); the width, the vocabulary and the active feed-forward size (top x size) are those of LAYERED_SIZES
+FELEPEL_SIZES = {
+    "w1024": ((8, 2, 128, 128, 1024), (8, 8, 128, 128, 4, 64), (16, 4, 4, 2, 768)),
+    "w2048": ((16, 4, 128, 128, 2048), (16, 16, 128, 128, 4, 128), (32, 6, 4, 2, 1024)),
+    "w3072": ((32, 8, 128, 128, 4096), (24, 24, 128, 128, 4, 128), (64, 6, 8, 4, 1536)),
+}
+
+
+def _felepel_model(gm, torch, dev, name, n_layers, ctx, pdl, chunk, batch):
+    width, vocab = LAYERED_SIZES[name][0], LAYERED_SIZES[name][8]
+    (h, g, d, v, size), (dh, dg, dd, dv, taps, rank), (experts, top, groups, keep, ff) = FELEPEL_SIZES[name]
+    moe = dict(mlp=gm.MLP_EXPERTS, d_ff=ff, experts=experts, top=top, groups=groups, keep=keep)
+    att = gm.LayerConfig(heads=h, kv_heads=g, dim=d, vdim=v, scale=d ** -0.5, softcap=30.0, mask=gm.MASK_CHUNK, mask_size=size, distance_bias=1, proj_bias=1,
+                         mixer=gm.MIXER_GROUPED_ATTENTION, **moe)
+    delta = gm.LayerConfig(heads=dh, kv_heads=dg, dim=dd, vdim=dv, taps=taps, decay_rank=rank, gate_rank=rank, mixer=gm.MIXER_CHANNEL_DELTA, **moe)
+    pages = (ctx + 15) // 16
+    cfg = gm.ModelConfig.layered([att, delta] * (n_layers // 2), width, vocab, ctx, 1e-6, block=gm.BLOCK_SANDWICH, learned_positions=ctx, weight_mode=gm.MODE_BF16,
+                                 max_seqs=batch, max_tokens=chunk, max_logit_rows=batch, kv_pages=batch * pages + 8, max_pages_per_seq=pages, use_pdl=pdl)
+    return _random_model(gm, torch, dev, cfg, 73)
+
+
+def run_felepel(args, out, gm, torch, np):
+    """Prefill and decode of Felepel (attention and delta-rule layers in turn, experts; random weights, bf16) beside Bevosun of the same
+    width, depth and active feed-forward size. Not the default line."""
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    n_layers, batch, prompt = 4, BATCH, PROMPT_LEN
+    ctx = prompt + args.steps + args.warmup + 32
+    rec = {"workload": "felepel", "layers": n_layers, "batch": batch, "prompt_tokens": prompt, "steps": args.steps, "warmup": args.warmup, "data": "synthetic", "sizes": {}}
+    sampler = ClockSampler(None)
+    sampler.start()
+    for name in args.sizes.split(","):
+        row = {"felepel": dict(zip(("attention", "delta", "experts"), FELEPEL_SIZES[name])), "bevosun": {"width": LAYERED_SIZES[name][0]}}
+        for kind, build in (("felepel", lambda *a: _felepel_model(gm, torch, dev, name, *a)), ("bevosun", lambda *a: _layered_model(gm, torch, dev, LAYERED_SIZES[name], *a))):
+            m = build(n_layers, ctx, args.pdl, 8192 if kind == "felepel" else 2048, batch)
+            row[kind].update(_model_speed(gm, torch, np, dev, m, prompt, batch, args.steps, args.warmup))
+            m.close()
+            torch.cuda.empty_cache()
+        rec["sizes"][name] = row
+    rec["clocks"] = sampler.stop()
+    print(json.dumps(rec), file=out)
+
+
+def time_felepel_kernels(ops, torch, dev, name, rows, ctx_len=PROMPT_LEN, only=None):
+    """Every kernel of Felepel's layers by itself at `rows` tokens, as time_layered_kernels does it. The delta rule's FLOPs are those of
+    the recurrence (8 per element of the state and token) at the f32 rate of the CUDA cores; `frac_hbm` is against its bytes alone."""
+    w = LAYERED_SIZES[name][0]
+    (heads, kv, dim, vdim, size), (dh, dg, dd, dv, taps, rank), (experts, top, groups, keep, ff) = FELEPEL_SIZES[name]
+    decode = rows <= 128
+    hbm, tf, f32_tf = _peaks()[0], _tensor_peak(), 148 * 128 * 2 * 1.965e-3
+    res = {}
+
+    def put(label, us, nbytes, flops, peak=tf):
+        t_mem, t_op = nbytes / hbm / 1e3, flops / peak / 1e6
+        res[label] = {"us": round(us, 2), "roofline_us": round(max(t_mem, t_op), 2), "bound": "hbm" if t_mem > t_op else ("f32" if peak == f32_tf else "tensor"),
+                      "frac": round(max(t_mem, t_op) / us, 3)}
+
+    bf, i32 = torch.bfloat16, torch.int32
+    status = torch.zeros(1, dtype=i32, device=dev)
+    want = lambda label: only is None or label in only  # noqa: E731
+
+    def gemm(label, n, k, ldx=None, out_f32=False, **kw):
+        if not want(label):
+            return
+        n8, k8 = (n + 7) // 8 * 8, (k + 7) // 8 * 8
+        per = n8 * k8 * 2
+        mats = [torch.randn(n8, k8, device=dev).mul_(k8 ** -0.5).to(bf) for _ in range(max(2, min(24, (300 << 20) // per)))]
+        x = torch.randn(rows, ldx or k8, device=dev).to(bf)
+        y = torch.empty(rows, n8, device=dev, dtype=torch.float32 if out_f32 else bf)
+        us = _graph_us(torch, [lambda m=m: ops.dense_bf16(x, m, rows, n8, k8, out=y, out_f32=out_f32, status=status, **({"ldx": ldx} if ldx else {}), **kw) for m in mats])
+        put(label, us, per + rows * (k8 + n8 * (2 if out_f32 else 1)) * 2, 2.0 * rows * n8 * k8)
+
+    a = ops.grouped_layout(heads, kv, dim, vdim, 2, size, dim ** -0.5, 30.0, True)
+    d = ops.delta_layout(dh, dg, dd, dv, taps, rank, rank, 1e-6)
+    gemm("qkv", a.q_row, w, bias=torch.zeros(a.q_row, device=dev))
+    gemm("out", w, heads * a.out_head_stride, bias=torch.zeros(w, device=dev))
+    gemm("delta_proj", d.row, w)
+    gemm("delta_decay", d.decay_row, rank, ldx=d.row, out_f32=True)
+    gemm("delta_gate", d.gate_row, rank, ldx=d.row)
+    gemm("delta_out", w, dh * d.out_head_stride)
+    gemm("router", experts, w, out_f32=True)
+
+    seqs = rows if decode else rows // ctx_len
+    per_seq = rows // seqs
+    slot = torch.arange(seqs, dtype=i32, device=dev).repeat_interleave(per_seq).contiguous()
+    pos = (torch.full((rows,), ctx_len - 1, device=dev) if decode else torch.arange(ctx_len, device=dev).repeat(seqs)).to(i32)
+    ctx = (pos + 1).to(i32)
+    if want("attention") or want("append"):
+        pages = (ctx_len + 15) // 16
+        pools = [torch.randn(seqs * pages * a.page_bytes // 2, device=dev).to(bf) for _ in range(4 if decode else 1)]
+        table = torch.randperm(seqs * pages, device=dev, dtype=i32).view(seqs, pages).contiguous()
+        qkv = torch.randn(rows, a.q_row, device=dev).to(bf)
+        r1, r2 = torch.full((heads,), 0.5, device=dev), torch.full((heads,), 0.2, device=dev)
+        t = 1 if decode else ops.grouped_tile_tokens(a)
+        first = torch.cat([torch.arange(0, per_seq, t, device=dev) + s * per_seq for s in range(seqs)]).to(i32)
+        count = torch.minimum(torch.full_like(first, t), per_seq - first % per_seq).to(i32)
+        us = _graph_us(torch, [lambda p=p: ops.grouped_attention(a, qkv, p, table, slot, ctx, ctx_len, r1, r2, tiles=(first, count), status=status) for p in pools] * (4 if decode else 2))
+        seen = (pos % size + 1).double()
+        cache = float(seen.sum()) if decode else rows
+        put("attention", us, cache * kv * (dim + vdim) * 2 + rows * heads * (dim + vdim) * 2, 2.0 * heads * (dim + vdim) * float(seen.sum()))
+        us = _graph_us(torch, [lambda p=p: ops.grouped_append(a, qkv, pos, slot, table, p) for p in pools] * 4)
+        put("append", us, rows * kv * (dim + vdim) * 4, 0)
+    if want("delta_rule"):
+        lo = torch.arange(rows, device=dev) // per_seq * per_seq
+        runs = (slot, pos, lo.to(i32), (lo + per_seq - 1).to(i32), torch.zeros_like(slot))
+        starts = (torch.arange(seqs, device=dev) * per_seq).to(i32)
+        proj, gate = torch.randn(rows, d.row, device=dev).to(bf), torch.randn(rows, d.gate_row, device=dev).to(bf)
+        decay = torch.randn(rows, d.decay_row, device=dev)
+        consts = [torch.randn(d.conv_channels, taps, device=dev), torch.zeros(dh, device=dev), torch.full((dh * dd,), -3.0, device=dev), torch.ones(dv, device=dev)]
+        copies = 4 if decode else 1
+        states = [(torch.zeros(seqs, d.state_floats, device=dev), torch.zeros(seqs, max(d.conv_floats, 1), device=dev)) for _ in range(copies)]
+        us = _graph_us(torch, [lambda s=s: ops.delta_rule(d, proj, decay, gate, *consts, *s, runs, starts) for s in states] * (4 if decode else 1))
+        state_bytes = seqs * (d.state_floats * 8 + d.conv_floats * 4)
+        row_bytes = rows * ((d.conv_channels + dh) * 2 + dh * dd * 4 + 2 * dh * dv * 2)
+        put("delta_rule", us, state_bytes + row_bytes, 8.0 * rows * dh * dd * dv, f32_tf)
+        res["delta_rule"]["frac_hbm"] = round((state_bytes + row_bytes) / hbm / 1e3 / us, 3)
+    x, y = torch.randn(rows, w, device=dev), torch.randn(rows, w, device=dev).to(bf)
+    gamma = torch.ones(w, device=dev)
+    if want("norm_step"):
+        us = _graph_us(torch, [lambda: ops.norm_step(x, 1e-6, y=y, gamma_out=gamma, gamma_in=gamma, out_dtype=bf, status=status)] * 8)
+        put("norm_step", us, rows * w * (4 + 2 + 4 + 2), 0)
+    if want("experts") or want("route"):
+        mean = rows * top / experts
+        tile = 16 if mean <= 8 else 32 if mean <= 24 else 64 if mean <= 48 else 128
+        z = torch.randn(rows, experts, device=dev)
+        us = _graph_us(torch, [lambda: ops.moe_route(experts, top, groups, keep, tile, z, y)] * 4)
+        put("route", us, rows * experts * 4 + rows * w * 2 * (1 + top), 0)
+        pair, weight, tiles, n_tiles, srt, most = ops.moe_route(experts, top, groups, keep, tile, z, y)
+        per = experts * 3 * ff * w * 2
+        active = int((torch.zeros(experts, device=dev).index_add_(0, tiles[:int(n_tiles), 0].long(), torch.ones(int(n_tiles), device=dev)) > 0).sum())
+        ups = [torch.randn(experts, 2 * ff, w, device=dev).mul_(w ** -0.5).to(bf) for _ in range(2 if per > (100 << 20) else 6)]
+        kw = dict(tiles=tiles, n_tiles=n_tiles, max_tiles=most, tile_rows=tile, batch=experts, status=status)
+        mid = torch.empty(rows * top, ff, device=dev, dtype=bf)
+        us = _graph_us(torch, [lambda m=m: ops.dense_bf16(srt, m, rows * top, 2 * ff, w, out=mid, swiglu=1, **kw) for m in ups] * 2)
+        put("experts_up", us, active * 2 * ff * w * 2 + rows * top * (w + ff) * 2, 4.0 * rows * top * ff * w)
+        del ups
+        downs = [torch.randn(experts, w, ff, device=dev).mul_(ff ** -0.5).to(bf) for _ in range(2 if per > (100 << 20) else 6)]
+        ey = torch.empty(rows * top, w, device=dev, dtype=bf)
+        us = _graph_us(torch, [lambda m=m: ops.dense_bf16(mid, m, rows * top, w, ff, out=ey, **kw) for m in downs] * 2)
+        put("experts_down", us, active * ff * w * 2 + rows * top * (w + ff) * 2, 2.0 * rows * top * ff * w)
+        us = _graph_us(torch, [lambda: ops.norm_step(x, 1e-6, y=ey, gamma_out=gamma, gamma_in=gamma, pair=pair, pair_weight=weight, out_dtype=bf, status=status)] * 4)
+        put("norm_step_experts", us, rows * w * (4 + 2 * top + 4 + 2), 0)
+    assert int(status) == 0
+    return res
+
+
+def run_felepel_kernels(args, out, ops, torch):
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    rec = {"microbench": "felepel", "decode_rows": BATCH, "ctx": PROMPT_LEN, "prefill_rows": 4 * PROMPT_LEN, "sizes": {}}
+    only = args.only.split(",") if args.only else None
+    for name in args.sizes.split(","):
+        rec["sizes"][name] = {"decode": time_felepel_kernels(ops, torch, dev, name, BATCH, only=only), "prefill": time_felepel_kernels(ops, torch, dev, name, 4 * PROMPT_LEN, only=only)}
+        if only is None:   # the like kernels of Bevosun
+            rec["sizes"][name].update(like_decode=time_layered_kernels(ops, torch, dev, LAYERED_SIZES[name], BATCH),
+                                      like_prefill=time_layered_kernels(ops, torch, dev, LAYERED_SIZES[name], 4 * PROMPT_LEN))
+        torch.cuda.empty_cache()
     print(json.dumps(rec), file=out)
 
 
@@ -931,14 +1096,17 @@ def _main(out):
     ap.add_argument("--pdl", type=int, default=int(os.environ.get("GPTRS_PDL", "1")))
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-extras", action="store_true", help="skip the kernel microbenchmarks")
-    ap.add_argument("--microbench", default=None, choices=["attention", "attention-ragged", "gemv", "gemv-lm-head", "gemm64", "quant-linear", "prefill", "prefill-attention", "layered"],
+    ap.add_argument("--microbench", default=None, choices=["attention", "attention-ragged", "gemv", "gemv-lm-head", "gemm64", "quant-linear", "prefill", "prefill-attention", "layered", "felepel"],
                     help="run only one kernel microbenchmark (used for ncu captures) and print its JSON")
     ap.add_argument("--ctx", type=int, default=PROMPT_LEN + 20, help="context length for --microbench attention")
-    ap.add_argument("--workload", default="ministral3b-w4", choices=["ministral3b-w4", "gpt2-fp32", "dp512", "bevosun"],
+    ap.add_argument("--workload", default="ministral3b-w4", choices=["ministral3b-w4", "gpt2-fp32", "dp512", "bevosun", "felepel"],
                     help="gpt2-fp32 = the reference's CPU-runnable case (one sequence, 32-token prompt, 64 greedy tokens); "
                          "dp512 = 512 requests with prompt lengths U{256..4096}, 256 decode steps each, partitioned over the ranks "
                          "(total work fixed: strong scaling; not the default line); "
-                         "bevosun = prefill and decode of the layered kind at three sizes beside the Ministral-shaped model of equal size")
+                         "bevosun = prefill and decode of the layered kind at three sizes beside the Ministral-shaped model of equal size; "
+                         "felepel = the same for Felepel beside Bevosun")
+    ap.add_argument("--sizes", default="w1024,w2048,w3072", help="felepel: comma list of sizes")
+    ap.add_argument("--only", default="", help="--microbench felepel: comma list of kernels (attention, append, delta_rule, norm_step, experts, route, or a matmul)")
     ap.add_argument("--path", default="engine", choices=["engine", "run_program"],
                     help="gpt2-fp32 only: engine = the model-level ABI (default); run_program = every decode step one "
                          "PortableBackend::run_program call on the captured decode program")
@@ -974,6 +1142,12 @@ def _main(out):
         return
     if args.workload == "bevosun":
         run_layered(args, out, gm, torch, np)
+        return
+    if args.microbench == "felepel":
+        run_felepel_kernels(args, out, ops, torch)
+        return
+    if args.workload == "felepel":
+        run_felepel(args, out, gm, torch, np)
         return
     if args.microbench == "prefill":
         # chunked prefill of a few 2048-token prompts through the engine (used for the ncu launch list of the prefill path)

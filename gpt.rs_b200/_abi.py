@@ -91,7 +91,7 @@ class DeltaRule(ctypes.Structure):
     _fields_ = [(n, ctypes.c_int) for n in ("dtype", "heads", "kv_heads", "dim", "vdim", "taps", "decay_rank", "gate_rank")] + [("eps", ctypes.c_float)] + \
         [(n, ctypes.c_int) for n in ("q_offset", "k_offset", "v_offset", "beta_offset", "a_offset", "g_offset", "row", "decay_row", "gate_row",
                                      "out_head_stride", "conv_channels")] + \
-        [(n, ctypes.c_int64) for n in ("state_floats", "conv_floats", "scratch_floats")]
+        [(n, ctypes.c_int64) for n in ("state_floats", "conv_floats")]
 
 
 class DeltaStep(ctypes.Structure):

@@ -3,10 +3,19 @@
 //   S <- g S (rows of S are key channels);   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
 //
 // with q, k, v behind short causal convolutions and silu, q and k of unit length, and o normed and gated. The columns of S are
-// independent of one another. With S' = g S one pass over S' gives S'^T k and S'^T q, hence u, and o = S'^T q + (q . k) u.
-//   delta_prepare_kernel   prompts: convolutions with their state, unit norms, decays, step sizes -> f32 planes, a CTA per row
-//   delta_scan_kernel      prompts: a warp keeps 16 columns of a head's S in registers over a whole run; tokens arrive in stages of
-//                          shared memory; the two sums over the key channels meet in one transposing warp reduction
+// independent of one another. Prompts take the recurrence in blocks of four tokens, which is exact algebra, not an approximation:
+// with p_t the product of the block's decays up to token t (per key channel) and S0 the state in front of the block,
+//
+//   r_t = S0^T (p_t k_t)      u_t = beta_t (v_t - r_t - sum_{s<t} A_ts u_s)        A_ts = sum_d k_t k_s (decays of s+1 .. t)
+//   w_t = S0^T (p_t q_t)      o_t = w_t + sum_{s<=t} B_ts u_s                      B_ts = sum_d q_t k_s (decays of s+1 .. t)
+//   S4  = p_3 S0 + sum_t c_t u_t^T,   c_t = k_t (decays of t+1 .. 3)
+//
+// so that a block costs 13 multiply-adds per element of S instead of 16 and one reduction over the key channels instead of four.
+// Every factor is a product of decays, at most 1.
+//   delta_prepare_kernel   prompts: a CTA per block, a warp per head: convolutions with their state, unit norms, decays, the vectors
+//                          p_t k_t, p_t q_t, c_t, p_3 and the numbers A, B of the block
+//   delta_scan_kernel      prompts: a warp keeps 16 columns of a head's S in registers over a whole run (packed pairs of key channels,
+//                          fma.rn.f32x2); blocks arrive in a ring of shared-memory stages; the sums meet in a transposing reduction
 //   delta_output_kernel    prompts: norm and gate of the read-outs
 //   delta_decode_kernel    rows that are runs of their own: all of the above in one launch, a CTA per (head, row), S is read and
 //                          written once
@@ -29,18 +38,21 @@ Geo geo(const gptrs_delta_rule& a) {
              a.out_head_stride, a.conv_channels, pad4(a.dim), pad4(a.vdim), a.eps, 1.f / sqrtf((float)a.dim)};
     return g;
 }
-// f32 planes of a prompt's rows behind one another in the scratch: q, k, v, decay, step size, q . k, read-out
-struct Planes { float *q, *k, *v, *g, *beta, *qk, *o; };
-int64_t plane_floats(const Geo& g) { return (int64_t)2 * g.kv_heads * g.dp + (int64_t)g.heads * (2 * g.vp + g.dp) + pad4(g.heads) + pad4(g.kv_heads); }
-Planes planes(const Geo& g, float* s, int64_t rows) {
+constexpr int kBlock = 4;        // tokens of a block
+constexpr int kVecs = 13;        // per block, head and key channel: p_t k_t (4), p_t q_t (4), c_t (4), p_3
+constexpr int kNums = 24;        // per block and head: beta (4), A10 A20 A21 A30 A31 A32 (+ 2), B00 B10 B11 B20 B21 B22 B30 .. B33 (+ 2)
+// Scratch of a prompt's blocks: vectors [block][head][13][dp], values [block][head][4][vp], numbers [block][head][24]; then the
+// read-outs [row][head][vp]. Run i with first row r keeps its blocks from number r / 4 + i on.
+struct Planes { float *vec, *v, *num, *o; };
+int64_t block_floats(const Geo& g) { return (int64_t)g.heads * (kVecs * g.dp + kBlock * g.vp + kNums); }
+int64_t max_blocks(int64_t rows, int64_t runs) { return rows / kBlock + runs; }
+Planes planes(const Geo& g, float* s, int64_t rows, int64_t runs) {
+    const int64_t n = max_blocks(rows, runs);
     Planes p;
-    p.q = s; s += rows * g.kv_heads * g.dp;
-    p.k = s; s += rows * g.kv_heads * g.dp;
-    p.v = s; s += rows * g.heads * g.vp;
-    p.g = s; s += rows * g.heads * g.dp;
-    p.o = s; s += rows * g.heads * g.vp;
-    p.beta = s; s += rows * pad4(g.heads);
-    p.qk = s;
+    p.vec = s; s += n * g.heads * kVecs * g.dp;
+    p.v = s; s += n * g.heads * kBlock * g.vp;
+    p.num = s; s += n * g.heads * kNums;
+    p.o = s;
     return p;
 }
 
@@ -102,205 +114,348 @@ __device__ __forceinline__ float conv_channel(const Params& p, const RowState& r
     return silu(fmaf(w[keep], now, acc));
 }
 
-constexpr int kPrepThreads = 256;
 constexpr int kMaxDim = 512;
+constexpr int kPrepThreads = 256;
 
-template <typename T>
+// What a block's channels need: the first row of the block, its live tokens, the convolution state of the sequence.
+struct BlockState { int row, n, first, last, pos; const float* old; float* fresh; };
+// silu(convolution) of channel `ch` (column `col` of the projection rows) for the tokens of a block; tokens that are not there give 0.
+// TAPS 0: any number. `keep_state`: this thread also passes the channel's inputs on to the next step.
+template <typename T, int TAPS>
+__device__ __forceinline__ void conv_block(const Params& p, const BlockState& b, int ch, int col, bool keep_state, float (&out)[kBlock]) {
+    const int taps = TAPS ? TAPS : p.g.taps, keep = taps - 1;
+    const T* x = static_cast<const T*>(p.s.d_proj) + (size_t)b.row * p.g.row + col;
+    const float* w = p.s.d_conv + (size_t)ch * taps;
+    auto input = [&](int k) -> float {   // k rows after the block's first one (k < 0: before it)
+        if (b.row + k >= b.first) return ld(x + (int64_t)k * p.g.row);
+        const int at = b.pos + k;
+        return at >= 0 ? b.old[(size_t)(at % keep) * p.g.channels + ch] : 0.f;
+    };
+    if constexpr (TAPS > 0) {
+        float in[TAPS - 1 + kBlock], wt[TAPS];
+#pragma unroll
+        for (int k = 0; k < TAPS - 1 + kBlock; ++k) in[k] = k - (TAPS - 1) < b.n ? input(k - (TAPS - 1)) : 0.f;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) wt[j] = __ldg(w + j);
+#pragma unroll
+        for (int t = 0; t < kBlock; ++t) {
+            float acc = 0.f;
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) acc = fmaf(wt[j], in[t + j], acc);
+            out[t] = t < b.n ? silu(acc) : 0.f;
+        }
+    } else {
+        for (int t = 0; t < kBlock; ++t) {
+            float acc = 0.f;
+            if (t < b.n)
+                for (int j = 0; j < taps; ++j) acc = fmaf(w[j], input(t + j - keep), acc);
+            out[t] = t < b.n ? silu(acc) : 0.f;
+        }
+    }
+    if (!keep_state || keep == 0) return;
+    if (b.row == b.first)   // a run shorter than the state: what it does not push out stays
+        for (int k = 1; k <= keep; ++k) {
+            const int at = b.pos - k;
+            if (at >= 0 && at > b.pos + (b.last - b.row) - keep) b.fresh[(size_t)(at % keep) * p.g.channels + ch] = b.old[(size_t)(at % keep) * p.g.channels + ch];
+        }
+    for (int t = 0; t < b.n; ++t)
+        if (b.last - (b.row + t) < keep) b.fresh[(size_t)((b.pos + t) % keep) * p.g.channels + ch] = ld(x + (int64_t)t * p.g.row);
+}
+
+// sums of 32 values over the warp: lane i gets the sum of v[i]
+__device__ __forceinline__ float transpose_sum(float (&v)[32]) {
+    const int lane = threadIdx.x & 31;
+#pragma unroll
+    for (int h = 16; h >= 1; h >>= 1)
+#pragma unroll
+        for (int i = 0; i < h; ++i) {
+            const float give = (lane & h) ? v[i] : v[i + h], keep = (lane & h) ? v[i + h] : v[i];
+            v[i] = keep + __shfl_xor_sync(0xffffffffu, give, h);
+        }
+    return v[0];
+}
+
+// NI: groups of 32 key channels
+template <typename T, int NI, int TAPS>
 __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Params p) {
     const Geo& g = p.g;
-    const int row = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, blk = blockIdx.x;
     pdl_launch_dependents();
     pdl_wait();
-    const RowState r = row_state(p, row);
-    const int v_jobs = (g.heads * g.vp + 127) / 128, g_jobs = (g.heads * g.dp + 127) / 128;
-    const int jobs = g.kv_heads + v_jobs + g_jobs + 1;
-    for (int job = warp; job < jobs; job += kPrepThreads / 32) {
-        if (job < g.kv_heads) {   // q and k of one head
-            float q[kMaxDim / 32], k[kMaxDim / 32], qq = 0.f, kk = 0.f, qk = 0.f;
-            const int c0 = job * g.dim;
-#pragma unroll
-            for (int i = 0; i < kMaxDim / 32; ++i) {
-                const int d = i * 32 + lane;
-                q[i] = k[i] = 0.f;
-                if (d < g.dim) {
-                    q[i] = conv_channel<T>(p, r, row, c0 + d, g.q_off + c0 + d, true);
-                    k[i] = conv_channel<T>(p, r, row, g.kv_heads * g.dim + c0 + d, g.k_off + c0 + d, true);
-                }
-                qq = fmaf(q[i], q[i], qq); kk = fmaf(k[i], k[i], kk); qk = fmaf(q[i], k[i], qk);
-            }
-            const float qs = g.q_scale / sqrtf(warp_sum(qq) + 1e-6f), ks = 1.f / sqrtf(warp_sum(kk) + 1e-6f);
-            qk = warp_sum(qk);
-            float *dq = p.w.q + ((size_t)row * g.kv_heads + job) * g.dp, *dk = p.w.k + ((size_t)row * g.kv_heads + job) * g.dp;
-#pragma unroll
-            for (int i = 0; i < kMaxDim / 32; ++i) {
-                const int d = i * 32 + lane;
-                if (d < g.dp) { dq[d] = q[i] * qs; dk[d] = k[i] * ks; }
-            }
-            if (lane == 0) p.w.qk[(size_t)row * g.kv_heads + job] = qk * qs * ks;
-        } else if (job < g.kv_heads + v_jobs) {
+    int run = 0;   // the last run whose blocks start at or before this one
+    for (int lo = 0, hi = (int)p.s.n_runs; lo < hi;) {
+        const int mid = (lo + hi) / 2;
+        if (p.s.d_runs[mid] / kBlock + mid <= blk) { run = mid; lo = mid + 1; }
+        else hi = mid;
+    }
+    BlockState b;
+    b.first = p.s.d_runs[run];
+    b.last = p.s.d_run_last[b.first];
+    b.row = b.first + (blk - (b.first / kBlock + run)) * kBlock;
+    if (b.row > b.last) return;
+    b.n = min(kBlock, b.last - b.row + 1);
+    b.pos = p.s.d_pos[b.row];
+    {
+        const size_t half = (size_t)(g.taps - 1) * g.channels;
+        float* state = p.s.d_conv_state + (size_t)p.s.d_slot[b.row] * 2 * half;
+        const int par = p.s.d_parity[b.row] & 1;
+        b.old = state + par * half; b.fresh = state + (par ^ 1) * half;
+    }
+    const int v_jobs = (g.heads * g.vp + 127) / 128;
+    for (int job = warp; job < g.heads + v_jobs; job += kPrepThreads / 32) {
+        if (job >= g.heads) {
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-                const int e = (job - g.kv_heads) * 128 + i * 32 + lane, h = e / g.vp, c = e % g.vp;
+                const int e = (job - g.heads) * 128 + i * 32 + lane, h = e / g.vp, c = e % g.vp;
                 if (h >= g.heads) continue;
-                float v = 0.f;
-                if (c < g.vdim) v = conv_channel<T>(p, r, row, 2 * g.kv_heads * g.dim + h * g.vdim + c, g.v_off + h * g.vdim + c, true);
-                p.w.v[(size_t)row * g.heads * g.vp + e] = v;
-            }
-        } else if (job < jobs - 1) {
+                float v[kBlock] = {0.f, 0.f, 0.f, 0.f};
+                if (c < g.vdim) conv_block<T, TAPS>(p, b, 2 * g.kv_heads * g.dim + h * g.vdim + c, g.v_off + h * g.vdim + c, true, v);
+                float* dst = p.w.v + ((size_t)blk * g.heads + h) * kBlock * g.vp + c;
 #pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int e = (job - g.kv_heads - v_jobs) * 128 + i * 32 + lane, h = e / g.dp, d = e % g.dp;
-                if (h >= g.heads) continue;
-                p.w.g[(size_t)row * g.heads * g.dp + e] = d < g.dim ? decay_of(p, row, h, d) : 0.f;
+                for (int t = 0; t < kBlock; ++t) dst[(size_t)t * g.vp] = v[t];
             }
-        } else {
-            for (int h = lane; h < g.heads; h += 32)
-                p.w.beta[(size_t)row * g.heads + h] = sigmoid(ld(static_cast<const T*>(p.s.d_proj) + (size_t)row * g.row + g.beta_off + h));
+            continue;
         }
+        const int head = job, kvh = head / g.group;
+        const bool own = head % g.group == 0;   // heads that share q and k: the first passes their convolution state on
+        float q[NI][kBlock], k[NI][kBlock];
+        float sums[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) sums[i] = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int d = i * 32 + lane;
+#pragma unroll
+            for (int t = 0; t < kBlock; ++t) q[i][t] = k[i][t] = 0.f;
+            if (d < g.dim) {
+                conv_block<T, TAPS>(p, b, kvh * g.dim + d, g.q_off + kvh * g.dim + d, own, q[i]);
+                conv_block<T, TAPS>(p, b, (g.kv_heads + kvh) * g.dim + d, g.k_off + kvh * g.dim + d, own, k[i]);
+            }
+#pragma unroll
+            for (int t = 0; t < kBlock; ++t) { sums[t] = fmaf(q[i][t], q[i][t], sums[t]); sums[4 + t] = fmaf(k[i][t], k[i][t], sums[4 + t]); }
+        }
+        float norm = 1.f / sqrtf(transpose_sum(sums) + 1e-6f);
+        if (lane < 4) norm *= g.q_scale;
+#pragma unroll
+        for (int t = 0; t < kBlock; ++t) {
+            const float qs = __shfl_sync(0xffffffffu, norm, t), ks = __shfl_sync(0xffffffffu, norm, 4 + t);
+#pragma unroll
+            for (int i = 0; i < NI; ++i) { q[i][t] *= qs; k[i][t] *= ks; }
+        }
+        const float rate = -expf(p.s.d_a_log[head]);
+        float* vec = p.w.vec + ((size_t)blk * g.heads + head) * kVecs * g.dp;
+        float num[32];   // A in 0 .. 5, B in 8 .. 17
+#pragma unroll
+        for (int i = 0; i < 32; ++i) num[i] = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int d = i * 32 + lane;
+            float gd[kBlock] = {1.f, 1.f, 1.f, 1.f};
+            if (d < g.dim) {
+                const float bias = p.s.d_dt_bias[head * g.dim + d];
+#pragma unroll
+                for (int t = 0; t < kBlock; ++t)
+                    if (t < b.n) gd[t] = expf(rate * softplus(p.s.d_decay[(size_t)(b.row + t) * g.decay_row + head * g.dim + d] + bias));
+            }
+            const float g10 = gd[1], g21 = gd[2], g32 = gd[3], g20 = g21 * g10, g31 = g32 * g21, g30 = g31 * g10;   // decays of s+1 .. t
+            const float* kk = k[i];
+            const float* qq = q[i];
+            num[0] = fmaf(kk[1] * kk[0], g10, num[0]);
+            num[1] = fmaf(kk[2] * kk[0], g20, num[1]);
+            num[2] = fmaf(kk[2] * kk[1], g21, num[2]);
+            num[3] = fmaf(kk[3] * kk[0], g30, num[3]);
+            num[4] = fmaf(kk[3] * kk[1], g31, num[4]);
+            num[5] = fmaf(kk[3] * kk[2], g32, num[5]);
+            num[8] = fmaf(qq[0], kk[0], num[8]);
+            num[9] = fmaf(qq[1] * kk[0], g10, num[9]);
+            num[10] = fmaf(qq[1], kk[1], num[10]);
+            num[11] = fmaf(qq[2] * kk[0], g20, num[11]);
+            num[12] = fmaf(qq[2] * kk[1], g21, num[12]);
+            num[13] = fmaf(qq[2], kk[2], num[13]);
+            num[14] = fmaf(qq[3] * kk[0], g30, num[14]);
+            num[15] = fmaf(qq[3] * kk[1], g31, num[15]);
+            num[16] = fmaf(qq[3] * kk[2], g32, num[16]);
+            num[17] = fmaf(qq[3], kk[3], num[17]);
+            if (d < g.dp) {
+                const float p0 = gd[0], p1 = p0 * gd[1], p2 = p1 * gd[2], p3 = p2 * gd[3];
+                float* o = vec + d;
+                o[0] = p0 * kk[0]; o[g.dp] = p1 * kk[1]; o[2 * g.dp] = p2 * kk[2]; o[3 * g.dp] = p3 * kk[3];
+                o[4 * g.dp] = p0 * qq[0]; o[5 * g.dp] = p1 * qq[1]; o[6 * g.dp] = p2 * qq[2]; o[7 * g.dp] = p3 * qq[3];
+                o[8 * g.dp] = kk[0] * g30; o[9 * g.dp] = kk[1] * g31; o[10 * g.dp] = kk[2] * g32; o[11 * g.dp] = kk[3];
+                o[12 * g.dp] = p3;
+            }
+        }
+        const float mine = transpose_sum(num);
+        float* dst = p.w.num + ((size_t)blk * g.heads + head) * kNums;
+        if (lane < 18) dst[4 + lane] = mine;
+        if (lane < kBlock)
+            dst[lane] = lane < b.n ? sigmoid(ld(static_cast<const T*>(p.s.d_proj) + (size_t)(b.row + lane) * g.row + g.beta_off + head)) : 0.f;
     }
 }
 
 // ---- the scan ------------------------------------------------------------------------------------------------------------------
 constexpr int kScanWarps = 4;
-__device__ __forceinline__ void cp_async_4(uint32_t dst, const void* src) {
-    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(dst), "l"(src));
-}
 
 // Eight lanes share a column: lane l holds the channels (8 i + l) 4 + e, i < NI, of CPL neighbouring columns; four such groups
 // make a warp. dim <= 32 NI.
-template <int NI, int CPL, int TB>
+template <int NI, int CPL, int STAGES>
 __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Params p) {
-    constexpr int W = 32 * NI;                       // channels with padding
-    constexpr int COLS = kScanWarps * 4 * CPL;       // columns of the CTA
-    constexpr int kStage = TB * (3 * W + COLS + 2);  // floats: k, q, g, v, beta, qk
-    constexpr int M = 2 * CPL, SH = M == 8 ? 0 : M == 4 ? 1 : 2;
+    constexpr int W = 32 * NI;                                      // channels with padding
+    constexpr int COLS = kScanWarps * 4 * CPL;                      // columns of the CTA
+    constexpr int kStage = kVecs * W + kBlock * COLS + kNums;       // floats
+    constexpr int SH = CPL == 4 ? 0 : CPL == 2 ? 1 : 2;             // lane bits that are left after (column, k or q)
     extern __shared__ __align__(16) float ds_smem[];
     const Geo& g = p.g;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = lane & 7, cg = lane >> 3;
-    const int head = blockIdx.y, kvh = head / g.group;
+    const int head = blockIdx.y;
     const int c_blk = blockIdx.x * COLS, col0 = c_blk + (warp * 4 + cg) * CPL;
+    for (int i = tid; i < STAGES * kStage; i += kScanWarps * 32) ds_smem[i] = 0.f;   // the padding stays zero
     pdl_launch_dependents();
     pdl_wait();
-    const int r0 = p.s.d_runs[blockIdx.z], r1 = p.s.d_run_last[r0] + 1;
+    const int run = blockIdx.z, r0 = p.s.d_runs[run], r1 = p.s.d_run_last[r0] + 1;
+    const int blk0 = r0 / kBlock + run, n_blk = (r1 - r0 + kBlock - 1) / kBlock;
     float* state = p.s.d_state + ((size_t)p.s.d_slot[r0] * g.heads + head) * g.dim * g.vdim;
     const bool fresh = p.s.d_pos[r0] == 0;
-    float S[NI][4][CPL];
+    uint64_t S[NI][2][CPL];
 #pragma unroll
     for (int i = 0; i < NI; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
+        for (int e = 0; e < 2; ++e)
 #pragma unroll
             for (int j = 0; j < CPL; ++j) {
-                const int d = (8 * i + l) * 4 + e;
-                S[i][e][j] = (!fresh && d < g.dim && col0 + j < g.vdim) ? state[(size_t)d * g.vdim + col0 + j] : 0.f;
+                const int d = (8 * i + l) * 4 + 2 * e;
+                const bool in = !fresh && col0 + j < g.vdim;
+                S[i][e][j] = pair_of(in && d < g.dim ? state[(size_t)d * g.vdim + col0 + j] : 0.f, in && d + 1 < g.dim ? state[(size_t)(d + 1) * g.vdim + col0 + j] : 0.f);
             }
-    for (int i = tid; i < 2 * kStage; i += kScanWarps * 32) ds_smem[i] = 0.f;   // the padding stays zero
     __syncthreads();
-    const int kq4 = g.dp / 4, v4 = min(COLS, g.vp - c_blk) / 4;
-    auto request = [&](int t0, int buf) {   // rows t0 .. t0 + TB of the run
-        float* sm = ds_smem + buf * kStage;
-        const int n = min(TB, r1 - t0);
-        for (int i = tid; i < n * kq4; i += kScanWarps * 32) {
-            const int t = i / kq4, c = (i % kq4) * 4;
-            const size_t kv = ((size_t)(t0 + t) * g.kv_heads + kvh) * g.dp + c, hd = ((size_t)(t0 + t) * g.heads + head) * g.dp + c;
-            cp_async_16(sm + t * W + c, p.w.k + kv, true);
-            cp_async_16(sm + (TB + t) * W + c, p.w.q + kv, true);
-            cp_async_16(sm + (2 * TB + t) * W + c, p.w.g + hd, true);
-        }
-        for (int i = tid; i < n * v4; i += kScanWarps * 32) {
-            const int t = i / v4, c = (i % v4) * 4;
-            cp_async_16(sm + 3 * TB * W + t * COLS + c, p.w.v + ((size_t)(t0 + t) * g.heads + head) * g.vp + c_blk + c, true);
-        }
-        for (int t = tid; t < n; t += kScanWarps * 32) {
-            cp_async_4(smem_u32(sm + TB * (3 * W + COLS) + t), p.w.beta + (size_t)(t0 + t) * g.heads + head);
-            cp_async_4(smem_u32(sm + TB * (3 * W + COLS + 1) + t), p.w.qk + (size_t)(t0 + t) * g.kv_heads + kvh);
+    const int d4 = g.dp / 4, v4 = min(COLS, g.vp - c_blk) / 4;
+    auto request = [&](int b) {   // block b of the run; always one group of copies
+        if (b < n_blk) {
+            float* sm = ds_smem + (b % STAGES) * kStage;
+            const size_t at = (size_t)(blk0 + b) * g.heads + head;
+            for (int i = tid; i < kVecs * d4; i += kScanWarps * 32) {
+                const int x = i / d4, c = (i % d4) * 4;
+                cp_async_16(sm + x * W + c, p.w.vec + (at * kVecs + x) * g.dp + c, true);
+            }
+            for (int i = tid; i < kBlock * v4; i += kScanWarps * 32) {
+                const int t = i / v4, c = (i % v4) * 4;
+                cp_async_16(sm + kVecs * W + t * COLS + c, p.w.v + (at * kBlock + t) * g.vp + c_blk + c, true);
+            }
+            if (tid < kNums / 4) cp_async_16(sm + kVecs * W + kBlock * COLS + tid * 4, p.w.num + at * kNums + tid * 4, true);
         }
         cp_async_commit();
     };
-    request(r0, 0);
-    int buf = 0;
-    for (int t0 = r0; t0 < r1; t0 += TB, buf ^= 1) {
-        if (t0 + TB < r1) { request(t0 + TB, buf ^ 1); cp_async_wait<1>(); }
-        else cp_async_wait<0>();
-        __syncthreads();
-        const float* sm = ds_smem + buf * kStage;
-        const int n = min(TB, r1 - t0);
+#pragma unroll
+    for (int b = 0; b < STAGES - 1; ++b) request(b);
 #pragma unroll 1
-        for (int t = 0; t < n; ++t) {
-            float r[M];
+    for (int b = 0; b < n_blk; ++b) {
+        cp_async_wait<STAGES - 2>();
+        __syncthreads();          // block b is there, and everyone is done with block b - 1
+        request(b + STAGES - 1);
+        const float* sm = ds_smem + (b % STAGES) * kStage;
+        const float* lanes = sm + l * 4;
+        uint64_t acc[8][CPL];     // p_t k_t, then p_t q_t
 #pragma unroll
-            for (int j = 0; j < M; ++j) r[j] = 0.f;
-            float4 kk[NI];
+        for (int x = 0; x < 8; ++x)
 #pragma unroll
-            for (int i = 0; i < NI; ++i) {
-                kk[i] = *reinterpret_cast<const float4*>(sm + t * W + (8 * i + l) * 4);
-                const float4 qv = *reinterpret_cast<const float4*>(sm + (TB + t) * W + (8 * i + l) * 4);
-                const float4 gv = *reinterpret_cast<const float4*>(sm + (2 * TB + t) * W + (8 * i + l) * 4);
-                const float ka[4] = {kk[i].x, kk[i].y, kk[i].z, kk[i].w}, qa[4] = {qv.x, qv.y, qv.z, qv.w}, ga[4] = {gv.x, gv.y, gv.z, gv.w};
+            for (int j = 0; j < CPL; ++j) acc[x][j] = 0;
 #pragma unroll
-                for (int e = 0; e < 4; ++e)
+        for (int i = 0; i < NI; ++i)
 #pragma unroll
-                    for (int j = 0; j < CPL; ++j) {
-                        const float s = S[i][e][j] * ga[e];
-                        S[i][e][j] = s;
-                        r[2 * j] = fmaf(s, ka[e], r[2 * j]);
-                        r[2 * j + 1] = fmaf(s, qa[e], r[2 * j + 1]);
-                    }
+            for (int x = 0; x < 8; ++x) {
+                const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(lanes + x * W + 32 * i);
+#pragma unroll
+                for (int j = 0; j < CPL; ++j) acc[x][j] = fma2(S[i][1][j], v.y, fma2(S[i][0][j], v.x, acc[x][j]));
             }
-            // transposing reduction over the eight lanes: afterwards this lane holds the sum number l >> SH
-            if constexpr (M == 8) {
+        // transposing reduction over the eight lanes: this lane ends up with the four sums of (column j_mine, k or q)
+        float r[CPL][2][kBlock];
 #pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    const float give = (l & 4) ? r[j] : r[j + 4], keep = (l & 4) ? r[j + 4] : r[j];
-                    r[j] = keep + __shfl_xor_sync(0xffffffffu, give, 4);
+        for (int j = 0; j < CPL; ++j)
+#pragma unroll
+            for (int x = 0; x < 8; ++x) { const float2 h = split(acc[x][j]); r[j][x >> 2][x & 3] = h.x + h.y; }
+        if constexpr (CPL == 4) {
+#pragma unroll
+            for (int j = 0; j < 2; ++j)
+#pragma unroll
+                for (int x = 0; x < 8; ++x) {
+                    float &a = r[j][x >> 2][x & 3], &c = r[j + 2][x >> 2][x & 3];
+                    const float give = (l & 4) ? a : c, keep = (l & 4) ? c : a;
+                    a = keep + __shfl_xor_sync(0xffffffffu, give, 4);
                 }
-            }
-            if constexpr (M >= 4) {
-                constexpr int bit = M == 8 ? 2 : 4;
+        }
+        if constexpr (CPL >= 2) {
+            constexpr int bit = CPL == 4 ? 2 : 4;
 #pragma unroll
-                for (int j = 0; j < 2; ++j) {
-                    const float give = (l & bit) ? r[j] : r[j + 2], keep = (l & bit) ? r[j + 2] : r[j];
-                    r[j] = keep + __shfl_xor_sync(0xffffffffu, give, bit);
-                }
-            }
-            {
-                constexpr int bit = 1 << SH;
-                const float give = (l & bit) ? r[0] : r[1], keep = (l & bit) ? r[1] : r[0];
-                r[0] = keep + __shfl_xor_sync(0xffffffffu, give, bit);
-            }
-#pragma unroll
-            for (int b = (1 << SH) >> 1; b > 0; b >>= 1) r[0] += __shfl_xor_sync(0xffffffffu, r[0], b);
-            const int m = l >> SH, j_mine = m >> 1;
-            const float beta = sm[TB * (3 * W + COLS) + t], qk = sm[TB * (3 * W + COLS + 1) + t];
-            const float v = sm[3 * TB * W + t * COLS + col0 - c_blk + j_mine];
-            const float u_mine = beta * (v - r[0]);   // meaningful where m is even
-            float u[CPL];
-#pragma unroll
-            for (int j = 0; j < CPL; ++j) u[j] = __shfl_sync(0xffffffffu, u_mine, (lane & 24) + ((2 * j) << SH));
-            float uo = u[0];
-#pragma unroll
-            for (int j = 1; j < CPL; ++j) uo = j_mine == j ? u[j] : uo;
-            if ((m & 1) && (l & ((1 << SH) - 1)) == 0 && col0 + j_mine < g.vdim)
-                p.w.o[((size_t)(t0 + t) * g.heads + head) * g.vp + col0 + j_mine] = fmaf(qk, uo, r[0]);
-#pragma unroll
-            for (int i = 0; i < NI; ++i) {
-                const float ka[4] = {kk[i].x, kk[i].y, kk[i].z, kk[i].w};
-#pragma unroll
-                for (int e = 0; e < 4; ++e)
-#pragma unroll
-                    for (int j = 0; j < CPL; ++j) S[i][e][j] = fmaf(ka[e], u[j], S[i][e][j]);
+            for (int x = 0; x < 8; ++x) {
+                float &a = r[0][x >> 2][x & 3], &c = r[1][x >> 2][x & 3];
+                const float give = (l & bit) ? a : c, keep = (l & bit) ? c : a;
+                a = keep + __shfl_xor_sync(0xffffffffu, give, bit);
             }
         }
-        __syncthreads();
+        float y[kBlock];
+#pragma unroll
+        for (int t = 0; t < kBlock; ++t) {
+            constexpr int bit = 1 << SH;
+            const float a = r[0][0][t], c = r[0][1][t];
+            const float give = (l & bit) ? a : c, keep = (l & bit) ? c : a;
+            y[t] = keep + __shfl_xor_sync(0xffffffffu, give, bit);
+#pragma unroll
+            for (int o = (1 << SH) >> 1; o > 0; o >>= 1) y[t] += __shfl_xor_sync(0xffffffffu, y[t], o);
+        }
+        const int m = l >> SH, j_mine = m >> 1;
+        const float* num = sm + kVecs * W + kBlock * COLS;
+        const float4 beta = *reinterpret_cast<const float4*>(num), a0 = *reinterpret_cast<const float4*>(num + 4), a1 = *reinterpret_cast<const float4*>(num + 8);
+        const float* vs = sm + kVecs * W + col0 - c_blk + j_mine;
+        float u[kBlock];          // meaningful in the lanes of the k sums
+        u[0] = beta.x * (vs[0] - y[0]);
+        u[1] = beta.y * (vs[COLS] - fmaf(a0.x, u[0], y[1]));
+        u[2] = beta.z * (vs[2 * COLS] - fmaf(a0.z, u[1], fmaf(a0.y, u[0], y[2])));
+        u[3] = beta.w * (vs[3 * COLS] - fmaf(a1.y, u[2], fmaf(a1.x, u[1], fmaf(a0.w, u[0], y[3]))));
+        uint64_t uu[CPL][kBlock];
+#pragma unroll
+        for (int j = 0; j < CPL; ++j)
+#pragma unroll
+            for (int t = 0; t < kBlock; ++t) {
+                const float x = __shfl_sync(0xffffffffu, u[t], (lane & 24) + ((2 * j) << SH));
+                uu[j][t] = pair_of(x, x);
+            }
+        float uo[kBlock];
+#pragma unroll
+        for (int t = 0; t < kBlock; ++t) uo[t] = __shfl_xor_sync(0xffffffffu, u[t], 1 << SH);
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const ulonglong2 gv = *reinterpret_cast<const ulonglong2*>(lanes + 12 * W + 32 * i);
+#pragma unroll
+            for (int j = 0; j < CPL; ++j) { S[i][0][j] = mul2(S[i][0][j], gv.x); S[i][1][j] = mul2(S[i][1][j], gv.y); }
+#pragma unroll
+            for (int t = 0; t < kBlock; ++t) {
+                const ulonglong2 c = *reinterpret_cast<const ulonglong2*>(lanes + (8 + t) * W + 32 * i);
+#pragma unroll
+                for (int j = 0; j < CPL; ++j) { S[i][0][j] = fma2(c.x, uu[j][t], S[i][0][j]); S[i][1][j] = fma2(c.y, uu[j][t], S[i][1][j]); }
+            }
+        }
+        if ((m & 1) && (l & ((1 << SH) - 1)) == 0 && col0 + j_mine < g.vdim) {
+            const float4 b0 = *reinterpret_cast<const float4*>(num + 12), b1 = *reinterpret_cast<const float4*>(num + 16), b2 = *reinterpret_cast<const float4*>(num + 20);
+            const int row = r0 + b * kBlock;
+            float* o = p.w.o + ((size_t)row * g.heads + head) * g.vp + col0 + j_mine;
+            const size_t step = (size_t)g.heads * g.vp;
+            o[0] = fmaf(b0.x, uo[0], y[0]);
+            if (row + 1 < r1) o[step] = fmaf(b0.z, uo[1], fmaf(b0.y, uo[0], y[1]));
+            if (row + 2 < r1) o[2 * step] = fmaf(b1.y, uo[2], fmaf(b1.x, uo[1], fmaf(b0.w, uo[0], y[2])));
+            if (row + 3 < r1) o[3 * step] = fmaf(b2.y, uo[3], fmaf(b2.x, uo[2], fmaf(b1.w, uo[1], fmaf(b1.z, uo[0], y[3]))));
+        }
     }
+    cp_async_wait<0>();
 #pragma unroll
     for (int i = 0; i < NI; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
+        for (int e = 0; e < 2; ++e)
 #pragma unroll
             for (int j = 0; j < CPL; ++j) {
-                const int d = (8 * i + l) * 4 + e;
-                if (d < g.dim && col0 + j < g.vdim) state[(size_t)d * g.vdim + col0 + j] = S[i][e][j];
+                const int d = (8 * i + l) * 4 + 2 * e;
+                const float2 x = split(S[i][e][j]);
+                if (col0 + j < g.vdim && d < g.dim) state[(size_t)d * g.vdim + col0 + j] = x.x;
+                if (col0 + j < g.vdim && d + 1 < g.dim) state[(size_t)(d + 1) * g.vdim + col0 + j] = x.y;
             }
 }
 
@@ -315,11 +470,28 @@ __global__ void __launch_bounds__(256) delta_output_kernel(const Params p) {
     if (job >= (int64_t)p.s.rows * g.heads) return;
     const int row = (int)(job / g.heads), head = (int)(job % g.heads);
     const float* o = p.w.o + job * g.vp;
+    const T* gate = static_cast<const T*>(p.s.d_gate) + (size_t)row * g.gate_row + head * g.vdim;
+    T* out = static_cast<T*>(p.s.d_out) + job * g.out_stride;
+    if constexpr (sizeof(T) == 2) {
+        if (g.vdim % 4 == 0 && g.vdim <= 128) {   // the row in one register each
+            const int c = lane * 4;
+            const bool in = c < g.vdim;
+            const float4 v = in ? *reinterpret_cast<const float4*>(o + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            const float inv = 1.f / sqrtf(warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w) / (float)g.vdim + g.eps);
+            if (in) {
+                const uint2 gu = *reinterpret_cast<const uint2*>(gate + c);
+                const float4 w = *reinterpret_cast<const float4*>(p.s.d_norm + c);
+                *reinterpret_cast<uint2*>(out + c) = make_uint2(pack_bf16x2(v.x * inv * w.x * sigmoid(bf16_lo(gu.x)), v.y * inv * w.y * sigmoid(bf16_hi(gu.x))),
+                                                                pack_bf16x2(v.z * inv * w.z * sigmoid(bf16_lo(gu.y)), v.w * inv * w.w * sigmoid(bf16_hi(gu.y))));
+            } else if (c < g.out_stride) {
+                *reinterpret_cast<uint2*>(out + c) = make_uint2(0, 0);
+            }
+            return;
+        }
+    }
     float ss = 0.f;
     for (int c = lane; c < g.vdim; c += 32) ss = fmaf(o[c], o[c], ss);
     const float inv = 1.f / sqrtf(warp_sum(ss) / (float)g.vdim + g.eps);
-    const T* gate = static_cast<const T*>(p.s.d_gate) + (size_t)row * g.gate_row + head * g.vdim;
-    T* out = static_cast<T*>(p.s.d_out) + job * g.out_stride;
     for (int c = lane; c < g.out_stride; c += 32) st(out + c, c < g.vdim ? o[c] * inv * p.s.d_norm[c] * sigmoid(ld(gate + c)) : 0.f);
 }
 
@@ -443,13 +615,19 @@ __global__ void __launch_bounds__(kDecThreads) delta_decode_kernel(const Params 
     for (int c = tid; c < g.out_stride; c += kDecThreads) st(out + c, c < g.vdim ? o[c] * inv * p.s.d_norm[c] * sigmoid(ld(gate + c)) : 0.f);
 }
 
-template <int NI, int CPL, int TB>
+template <int NI, int CPL, int STAGES>
 int launch_scan(const Params& p, cudaStream_t s) {
     constexpr int cols = kScanWarps * 4 * CPL;
-    constexpr size_t smem = (size_t)2 * TB * (3 * 32 * NI + cols + 2) * 4;
+    constexpr size_t smem = (size_t)STAGES * (kVecs * 32 * NI + kBlock * cols + kNums) * 4;
     static PerDeviceOnce once;
-    if (once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(delta_scan_kernel<NI, CPL, TB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    return launch_kernel(delta_scan_kernel<NI, CPL, TB>, dim3((unsigned)ceil_div(p.g.vdim, cols), (unsigned)p.g.heads, (unsigned)p.s.n_runs), dim3(kScanWarps * 32), smem, s, 1, p);
+    if (once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(delta_scan_kernel<NI, CPL, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    return launch_kernel(delta_scan_kernel<NI, CPL, STAGES>, dim3((unsigned)ceil_div(p.g.vdim, cols), (unsigned)p.g.heads, (unsigned)p.s.n_runs), dim3(kScanWarps * 32), smem, s, 1, p);
+}
+template <typename T, int NI>
+int launch_prepare(const Params& p, cudaStream_t s) {
+    const dim3 grid((unsigned)max_blocks(p.s.rows, p.s.n_runs));
+    if (p.g.taps == 4) return launch_kernel(delta_prepare_kernel<T, NI, 4>, grid, dim3(kPrepThreads), 0, s, 1, p);
+    return launch_kernel(delta_prepare_kernel<T, NI, 0>, grid, dim3(kPrepThreads), 0, s, 1, p);
 }
 template <typename T, int NR, int VEC>
 int launch_decode(const Params& p, cudaStream_t s) {
@@ -468,13 +646,12 @@ int run(const Params& p, cudaStream_t s) {
         if (g.dim <= 128) return launch_decode<T, 16, 1>(p, s);
         return launch_decode<T, 64, 1>(p, s);
     }
-    int rc = launch_kernel(delta_prepare_kernel<T>, dim3((unsigned)p.s.rows), dim3(kPrepThreads), 0, s, 1, p);
-    if (rc) return rc;
-    if (g.dim <= 32) rc = launch_scan<1, 4, 16>(p, s);
-    else if (g.dim <= 64) rc = launch_scan<2, 4, 16>(p, s);
-    else if (g.dim <= 128) rc = launch_scan<4, 4, 16>(p, s);
-    else if (g.dim <= 256) rc = launch_scan<8, 2, 8>(p, s);
-    else rc = launch_scan<16, 1, 8>(p, s);
+    int rc = GPTRS_OK;
+    if (g.dim <= 32) { if (!(rc = launch_prepare<T, 1>(p, s))) rc = launch_scan<1, 4, 4>(p, s); }
+    else if (g.dim <= 64) { if (!(rc = launch_prepare<T, 2>(p, s))) rc = launch_scan<2, 4, 4>(p, s); }
+    else if (g.dim <= 128) { if (!(rc = launch_prepare<T, 4>(p, s))) rc = launch_scan<4, 4, 4>(p, s); }
+    else if (g.dim <= 256) { if (!(rc = launch_prepare<T, 8>(p, s))) rc = launch_scan<8, 2, 4>(p, s); }
+    else { if (!(rc = launch_prepare<T, 16>(p, s))) rc = launch_scan<16, 1, 4>(p, s); }
     if (rc) return rc;
     return launch_kernel(delta_output_kernel<T>, dim3((unsigned)ceil_div(p.s.rows * g.heads, 8)), dim3(256), 0, s, 1, p);
 }
@@ -506,8 +683,13 @@ int gptrs_cuda_delta_layout(gptrs_delta_rule* a) {
     a->conv_channels = 2 * a->kv_heads * a->dim + a->heads * a->vdim;
     a->state_floats = (int64_t)a->heads * a->dim * a->vdim;
     a->conv_floats = (int64_t)2 * (a->taps - 1) * a->conv_channels;
-    a->scratch_floats = plane_floats(geo(*a));
     return GPTRS_OK;
+}
+
+int64_t gptrs_cuda_delta_scratch_floats(const gptrs_delta_rule* a, int64_t rows, int64_t n_runs) {
+    if (!a || n_runs == rows) return 0;
+    const Geo g = geo(*a);
+    return max_blocks(rows, n_runs) * block_floats(g) + rows * g.heads * g.vp;
 }
 
 int gptrs_cuda_delta_rule(const gptrs_delta_rule* a, const gptrs_delta_step* step, void* stream) {
@@ -519,7 +701,7 @@ int gptrs_cuda_delta_rule(const gptrs_delta_rule* a, const gptrs_delta_step* ste
     if (s.rows == 0) return GPTRS_OK;
     GPTRS_REQUIRE(s.n_runs == s.rows || (s.n_runs > 0 && s.d_runs && s.d_scratch && (reinterpret_cast<uintptr_t>(s.d_scratch) & 15) == 0), "delta rule: run list and scratch");
     Params p = {s, geo(*a), {}};
-    if (s.n_runs != s.rows) p.w = planes(p.g, s.d_scratch, s.rows);
+    if (s.n_runs != s.rows) p.w = planes(p.g, s.d_scratch, s.rows, s.n_runs);
     return a->dtype == GPTRS_BF16 ? run<__nv_bfloat16>(p, as_stream(stream)) : run<float>(p, as_stream(stream));
 }
 

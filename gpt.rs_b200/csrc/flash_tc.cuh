@@ -117,29 +117,76 @@ __device__ __forceinline__ float ex2f(float x) {
     return y;
 }
 
-// Raw products of a row -> scores in log2 units: cap tanh(scale s / cap) - r1 ln(1 + r2 d), all times log2(e). d is the distance of
-// column 0 (a column on the far side of the row's own position is masked later; its logarithm is kept finite).
+// Raw products of a row -> scores in log2 units: cap tanh(scale s / cap) - r1 ln(1 + r2 d), all times log2(e). d0 is the distance of
+// column 0 (a column on the far side of the row's own position is masked later; its logarithm is kept finite). The tanh is its Taylor
+// series while the whole warp's arguments are at most 1/2 (7 terms, error below 2e-7), the logarithms of eight neighbouring columns
+// are one logarithm in their middle and the series of ln(1 - y) around it while |y| <= 1/8 (5 terms, error below 1e-6): the
+// multi-function unit, which would otherwise give four results per score, is what bounds this kernel.
 __device__ __forceinline__ void score_log2(float (&s)[kKeys], float scale_log2, float cap_log2, float r1, float r2, int d0) {
-    if (cap_log2 > 0.f) {   // tanh(x) = 1 - 2 / (exp(2x) + 1)
+    if (cap_log2 > 0.f) {
+        const float cx = scale_log2 * (0.5f / kLog2e);   // scale / cap
+        float mx[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-        for (int j = 0; j < kKeys; ++j) {
-            const float e = ex2f(s[j] * scale_log2) + 1.f;
-            float inv;
-            asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(inv) : "f"(e));
-            s[j] = fmaf(-2.f * cap_log2, inv, cap_log2);
+        for (int j = 0; j < kKeys; ++j) mx[j & 3] = fmaxf(mx[j & 3], fabsf(s[j]));
+        const float m = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * cx;
+        if (__all_sync(0xffffffffu, m <= 0.5f)) {
+            const float k0 = cap_log2;
+            const uint64_t c0 = pair_of(k0, k0), c1 = pair_of(k0 * (-1.f / 3.f), k0 * (-1.f / 3.f)), c2 = pair_of(k0 * (2.f / 15.f), k0 * (2.f / 15.f)),
+                           c3 = pair_of(k0 * (-17.f / 315.f), k0 * (-17.f / 315.f)), c4 = pair_of(k0 * (62.f / 2835.f), k0 * (62.f / 2835.f)),
+                           c5 = pair_of(k0 * (-1382.f / 155925.f), k0 * (-1382.f / 155925.f)), c6 = pair_of(k0 * (21844.f / 6081075.f), k0 * (21844.f / 6081075.f)),
+                           cc = pair_of(cx, cx);
+#pragma unroll
+            for (int j = 0; j < kKeys; j += 2) {
+                const uint64_t x = mul2(pair_of(s[j], s[j + 1]), cc), z = mul2(x, x);
+                uint64_t t = fma2(z, c6, c5);
+                t = fma2(z, t, c4);
+                t = fma2(z, t, c3);
+                t = fma2(z, t, c2);
+                t = fma2(z, t, c1);
+                t = fma2(z, t, c0);
+                const float2 v = split(mul2(x, t));
+                s[j] = v.x; s[j + 1] = v.y;
+            }
+        } else {   // tanh(x) = 1 - 2 / (exp(2x) + 1)
+#pragma unroll
+            for (int j = 0; j < kKeys; ++j) {
+                const float e = ex2f(s[j] * scale_log2) + 1.f;
+                float inv;
+                asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(inv) : "f"(e));
+                s[j] = fmaf(-2.f * cap_log2, inv, cap_log2);
+            }
         }
     } else {
 #pragma unroll
         for (int j = 0; j < kKeys; ++j) s[j] *= scale_log2;
     }
-    if (r1 != 0.f) {
-        const float first = fmaf(r2, (float)d0, 1.f);
+    auto lg2f = [](float x) {
+        float l;
+        asm("lg2.approx.ftz.f32 %0, %1;\n" : "=f"(l) : "f"(x));
+        return l;
+    };
+    if (!__any_sync(0xffffffffu, r1 != 0.f)) return;
+    const float first = fmaf(r2, (float)d0, 1.f);
+    if (__all_sync(0xffffffffu, fmaf(-r2, (float)(kKeys - 1), first) >= fmaxf(28.f * r2, 1e-3f))) {
 #pragma unroll
-        for (int j = 0; j < kKeys; ++j) {
-            float l;
-            asm("lg2.approx.ftz.f32 %0, %1;\n" : "=f"(l) : "f"(fmaxf(fmaf(-r2, (float)j, first), 1e-30f)));
-            s[j] = fmaf(-r1, l, s[j]);
+        for (int j0 = 0; j0 < kKeys; j0 += 8) {
+            const float a = fmaf(-r2, (float)j0 + 3.5f, first);   // 1 + r2 distance in the middle
+            float w;
+            asm("rcp.approx.ftz.f32 %0, %1;\n" : "=f"(w) : "f"(a));
+            w *= r2;
+            // - r1 log2(1 - w o) at the offsets o = -3.5 .. 3.5
+            const float b1 = r1 * kLog2e * w, b2 = b1 * w * 0.5f, b3 = b1 * w * w * (1.f / 3.f), b4 = b2 * w * w * 0.5f, b5 = b3 * w * w * 0.6f, b0 = -r1 * lg2f(a);
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float o = 3.5f - i;
+                const float even = fmaf(b4, o * o * o * o, fmaf(b2, o * o, b0)), odd = fmaf(b5, o * o * o * o * o, fmaf(b3, o * o * o, b1 * o));
+                s[j0 + i] += even - odd;
+                s[j0 + 7 - i] += even + odd;
+            }
         }
+    } else {
+#pragma unroll
+        for (int j = 0; j < kKeys; ++j) s[j] = fmaf(-r1, lg2f(fmaxf(fmaf(-r2, (float)j, first), 1e-30f)), s[j]);
     }
 }
 

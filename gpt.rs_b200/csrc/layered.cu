@@ -381,7 +381,8 @@ void count_widths(const Model& m, LayeredLayer& L, Widths* n) {
     } else {
         n->decay = std::max(n->decay, (int64_t)L.delta.decay_row);
         n->gate = std::max(n->gate, (int64_t)L.delta.gate_row);
-        n->delta_scratch = std::max(n->delta_scratch, L.delta.scratch_floats);
+        // a pass that is not one token per sequence: at most one run per slot
+        n->delta_scratch = std::max(n->delta_scratch, gptrs_cuda_delta_scratch_floats(&L.delta, c.max_tokens, std::min(c.max_seqs, c.max_tokens - 1)));
         L.delta_state_off = n->delta_state;
         L.delta_conv_off = n->delta_conv;
         n->delta_state += (size_t)c.max_seqs * L.delta.state_floats;
@@ -511,7 +512,7 @@ int layered_finalize(Model& m, bool drop_leaves) {
         (rc = y.y.alloc(T * Wp * act, true)) || (rc = y.qkv.alloc(T * n.qkv * act, true)) || (rc = y.qa.alloc(T * n.qa * act, true)) ||
         (rc = y.lat.alloc(T * n.lat * act, true)) || (rc = y.attn.alloc(T * n.attn * act, true)) || (rc = y.up.alloc(T * std::max(n.up, n.expert_up / 2) * act, true)) ||
         (rc = m.xn_rows.alloc(rows * Wp * act, true)) || (rc = m.logits.alloc(rows * V * 4, true))) return rc;
-    if ((rc = y.decay.alloc(T * n.decay * 4, true)) || (rc = y.gate.alloc(T * n.gate * act, true)) || (rc = y.delta_scratch.alloc(T * n.delta_scratch * 4, true)) ||
+    if ((rc = y.decay.alloc(T * n.decay * 4, true)) || (rc = y.gate.alloc(T * n.gate * act, true)) || (rc = y.delta_scratch.alloc(n.delta_scratch * 4, true)) ||
         (rc = y.delta_state.alloc(n.delta_state * 4, true)) || (rc = y.delta_conv.alloc(n.delta_conv * 4, true))) return rc;
     if ((rc = y.router.alloc(T * n.router * 4, true)) || (rc = y.sorted.alloc(T * n.sorted * act, true)) || (rc = y.gate_up.alloc(m.f32() ? T * n.expert_up * 4 : 0, true)) ||
         (rc = y.expert_y.alloc(T * n.expert_y * act, true)) || (rc = y.pair.alloc(T * n.top * 4, true)) || (rc = y.pair_weight.alloc(T * n.top * 4, true)) ||

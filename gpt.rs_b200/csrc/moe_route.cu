@@ -33,6 +33,8 @@ __device__ __forceinline__ int order_of(float v) {
     return b ^ ((b >> 31) & 0x7fffffff);
 }
 
+__device__ __forceinline__ float value_of(int order) { return __int_as_float(order ^ ((order >> 31) & 0x7fffffff)); }
+
 // inclusive sum over the 1024 threads of a CTA
 __device__ __forceinline__ int cta_scan(int v, int* sh) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -80,12 +82,15 @@ __global__ void __launch_bounds__(kWarps * 32) moe_choose_kernel(const Params p)
     __syncthreads();
     const int r_lo = blockIdx.x * p.per_cta, r_hi = min(r_lo + p.per_cta, p.rows);
     for (int row = r_lo + warp; row < r_hi; row += kWarps) {
+        constexpr int kNone = (int)0x80000000;
         float z[VPL];
+        int key[VPL];   // order of the logits; kNone: not to be chosen (any more)
         float mx = -INFINITY;
 #pragma unroll
         for (int i = 0; i < VPL; ++i) {
             const int e = i * 32 + lane;
             z[i] = e < E ? p.logits[(size_t)row * p.ld + e] : -INFINITY;
+            key[i] = e < E ? max(order_of(z[i]), kNone + 1) : kNone;
             mx = fmaxf(mx, z[i]);
         }
         mx = warp_max(mx);
@@ -93,53 +98,53 @@ __global__ void __launch_bounds__(kWarps * 32) moe_choose_kernel(const Params p)
 #pragma unroll
         for (int i = 0; i < VPL; ++i) sum += i * 32 + lane < E ? expf(z[i] - mx) : 0.f;
         sum = warp_sum(sum);
+        // largest key of `v` and the lowest index that has it
+        auto best_of = [&](int v, int index, int* at) {
+            const int best = __reduce_max_sync(0xffffffffu, v);
+            *at = __reduce_min_sync(0xffffffffu, v == best ? index : 0x7fffffff);
+            return best;
+        };
         if (p.a.keep < G) {
-            const int none = (int)0x80000000;
-            for (int g = lane; g < G; g += 32) gm[g] = none;
+            for (int g = lane; g < G; g += 32) gm[g] = kNone;
             __syncwarp();
 #pragma unroll
             for (int i = 0; i < VPL; ++i)
-                if (i * 32 + lane < E) atomicMax(gm + (i * 32 + lane) / size, order_of(z[i]));
+                if (i * 32 + lane < E) atomicMax(gm + (i * 32 + lane) / size, key[i]);
             __syncwarp();
             for (int n = 0; n < p.a.keep; ++n) {
-                int best = none, at = 0x7fffffff;
+                int best = kNone, index = 0x7fffffff, at;
                 for (int g = lane; g < G; g += 32)
-                    if (gm[g] != 0x7fffffff && (gm[g] > best || at == 0x7fffffff)) { best = gm[g]; at = g; }
-#pragma unroll
-                for (int o = 16; o > 0; o >>= 1) {
-                    const int ob = __shfl_xor_sync(0xffffffffu, best, o), oa = __shfl_xor_sync(0xffffffffu, at, o);
-                    if (oa != 0x7fffffff && (at == 0x7fffffff || ob > best || (ob == best && oa < at))) { best = ob; at = oa; }
-                }
+                    if (gm[g] != 0x7fffffff && gm[g] > best) { best = gm[g]; index = g; }
+                best_of(best, index, &at);
                 __syncwarp();
                 if (lane == 0 && at < G) gm[at] = 0x7fffffff;   // taken
                 __syncwarp();
             }
 #pragma unroll
             for (int i = 0; i < VPL; ++i)
-                if (i * 32 + lane < E && gm[(i * 32 + lane) / size] != 0x7fffffff) z[i] = -INFINITY;
+                if (i * 32 + lane < E && gm[(i * 32 + lane) / size] != 0x7fffffff) key[i] = kNone;
             __syncwarp();
         }
+        int mine = 0, chosen = 0;   // lane k: the k-th choice (of the current 32)
         for (int k = 0; k < p.a.top; ++k) {
-            float best = -INFINITY;
-            int at = 0x7fffffff;
+            int best = kNone, index = 0x7fffffff, at;
 #pragma unroll
             for (int i = 0; i < VPL; ++i)
-                if (z[i] > best) { best = z[i]; at = i * 32 + lane; }
-#pragma unroll
-            for (int o = 16; o > 0; o >>= 1) {
-                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-                const int oa = __shfl_xor_sync(0xffffffffu, at, o);
-                if (ob > best || (ob == best && oa < at)) { best = ob; at = oa; }
-            }
+                if (key[i] > best) { best = key[i]; index = i * 32 + lane; }
+            best = best_of(best, index, &at);
             if (at >= E) at = 0;   // only where logits are not numbers
 #pragma unroll
             for (int i = 0; i < VPL; ++i)
-                if (i * 32 + lane == at) z[i] = -INFINITY;
-            if (lane == 0) {
-                const size_t o = (size_t)row * p.a.top + k;
-                p.weight[o] = expf(best - mx) / sum;
-                p.id[o] = at;
-                p.place[o] = atomicAdd(hist + at, 1);
+                if (i * 32 + lane == at) key[i] = kNone;
+            if (lane == (k & 31)) { mine = best; chosen = at; }
+            if ((k & 31) == 31 || k + 1 == p.a.top) {
+                const int k0 = k & ~31;
+                if (lane <= k - k0) {
+                    const size_t o = (size_t)row * p.a.top + k0 + lane;
+                    p.weight[o] = expf(value_of(mine) - mx) / sum;
+                    p.id[o] = chosen;
+                    p.place[o] = atomicAdd(hist + chosen, 1);
+                }
             }
         }
     }

@@ -554,7 +554,7 @@ def delta_rule(a, proj, decay, gate, conv, a_log, dt_bias, norm, state, conv_sta
     s.d_state, s.d_conv_state = _ptr(state), _ptr(conv_state)
     s.d_slot, s.d_pos, s.d_run_first, s.d_run_last, s.d_parity = (_ptr(t) for t in runs)
     s.d_runs, s.n_runs, s.rows, s.d_out = _ptr(first_rows), first_rows.shape[0] if n_runs is None else n_runs, n, _ptr(out)
-    scratch = torch.empty(max(n * a.scratch_floats, 1), dtype=torch.float32, device=proj.device)
+    scratch = torch.empty(max(lib().gptrs_cuda_delta_scratch_floats(ctypes.byref(a), n, s.n_runs), 1), dtype=torch.float32, device=proj.device)
     s.d_scratch = _ptr(scratch)
     check(lib().gptrs_cuda_delta_rule(ctypes.byref(a), ctypes.byref(s), _stream()))
     return out

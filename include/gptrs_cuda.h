@@ -385,9 +385,9 @@ typedef struct {
     int conv_channels;         /* 2 kv_heads dim + heads vdim: rows of d_conv, channels of the convolution state */
     int64_t state_floats;      /* recurrent state of a slot: heads dim vdim */
     int64_t conv_floats;       /* convolution state of a slot: 2 (taps - 1) conv_channels */
-    int64_t scratch_floats;    /* per row, for prompts */
 } gptrs_delta_rule;
 int gptrs_cuda_delta_layout(gptrs_delta_rule* a);
+int64_t gptrs_cuda_delta_scratch_floats(const gptrs_delta_rule* a, int64_t rows, int64_t n_runs);
 typedef struct {
     const void* d_proj;        /* [T][row] */
     const float* d_decay;      /* [T][decay_row] */
@@ -400,7 +400,7 @@ typedef struct {
     const int32_t* d_runs;     /* first row of every run */
     int64_t n_runs;            /* n_runs = rows: every row is a run of its own (a decode step) */
     void* d_out;               /* [T][heads][out_head_stride] */
-    float* d_scratch;          /* rows * scratch_floats, unless n_runs = rows */
+    float* d_scratch;          /* gptrs_cuda_delta_scratch_floats of them (0 when n_runs = rows) */
     int64_t rows;
 } gptrs_delta_step;
 int gptrs_cuda_delta_rule(const gptrs_delta_rule* a, const gptrs_delta_step* step, void* stream);

@@ -75,6 +75,14 @@ __device__ __forceinline__ void st(T* p, float v) {
     if constexpr (sizeof(T) == 2) *p = __float2bfloat16_rn(v);
     else *p = v;
 }
+// silu of a convolution that is rounded to bf16 anyway; exp(rate softplus(x)) with the hardware's exponential and logarithm, the latter
+// as the series of ln(1 + e) where 1 + e would lose e
+__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f + __expf(-x)); }
+__device__ __forceinline__ float decay_fast(float x, float rate) {
+    const float e = __expf(-fabsf(x));
+    const float series = e * fmaf(e, fmaf(e, fmaf(e, -0.25f, 1.f / 3.f), -0.5f), 1.f);
+    return __expf(rate * (fmaxf(x, 0.f) + (e < 0.02f ? series : __logf(1.f + e))));
+}
 __device__ __forceinline__ float decay_of(const Params& p, int row, int head, int d) {
     const int c = head * p.g.dim + d;
     return expf(-expf(p.s.d_a_log[head]) * softplus(p.s.d_decay[(size_t)row * p.g.decay_row + c] + p.s.d_dt_bias[c]));
@@ -118,7 +126,7 @@ constexpr int kMaxDim = 512;
 constexpr int kPrepThreads = 256;
 
 // What a block's channels need: the first row of the block, its live tokens, the convolution state of the sequence.
-struct BlockState { int row, n, first, last, pos; const float* old; float* fresh; };
+struct BlockState { bool inner; int row, n, first, last, pos; const float* old; float* fresh; };
 // silu(convolution) of channel `ch` (column `col` of the projection rows) for the tokens of a block; tokens that are not there give 0.
 // TAPS 0: any number. `keep_state`: this thread also passes the channel's inputs on to the next step.
 template <typename T, int TAPS>
@@ -134,15 +142,20 @@ __device__ __forceinline__ void conv_block(const Params& p, const BlockState& b,
     if constexpr (TAPS > 0) {
         float in[TAPS - 1 + kBlock], wt[TAPS];
 #pragma unroll
-        for (int k = 0; k < TAPS - 1 + kBlock; ++k) in[k] = k - (TAPS - 1) < b.n ? input(k - (TAPS - 1)) : 0.f;
-#pragma unroll
         for (int j = 0; j < TAPS; ++j) wt[j] = __ldg(w + j);
+        if (b.inner) {   // a whole block away from the start of its run: all inputs are rows of this pass
+#pragma unroll
+            for (int k = 0; k < TAPS - 1 + kBlock; ++k) in[k] = ld(x + (int64_t)(k - (TAPS - 1)) * p.g.row);
+        } else {
+#pragma unroll
+            for (int k = 0; k < TAPS - 1 + kBlock; ++k) in[k] = k - (TAPS - 1) < b.n ? input(k - (TAPS - 1)) : 0.f;
+        }
 #pragma unroll
         for (int t = 0; t < kBlock; ++t) {
             float acc = 0.f;
 #pragma unroll
             for (int j = 0; j < TAPS; ++j) acc = fmaf(wt[j], in[t + j], acc);
-            out[t] = t < b.n ? silu(acc) : 0.f;
+            out[t] = t < b.n ? (sizeof(T) == 2 ? silu_fast(acc) : silu(acc)) : 0.f;
         }
     } else {
         for (int t = 0; t < kBlock; ++t) {
@@ -152,7 +165,7 @@ __device__ __forceinline__ void conv_block(const Params& p, const BlockState& b,
             out[t] = t < b.n ? silu(acc) : 0.f;
         }
     }
-    if (!keep_state || keep == 0) return;
+    if (!keep_state || keep == 0 || (b.inner && b.last - (b.row + kBlock - 1) >= keep)) return;
     if (b.row == b.first)   // a run shorter than the state: what it does not push out stays
         for (int k = 1; k <= keep; ++k) {
             const int at = b.pos - k;
@@ -195,6 +208,7 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Param
     if (b.row > b.last) return;
     b.n = min(kBlock, b.last - b.row + 1);
     b.pos = p.s.d_pos[b.row];
+    b.inner = b.n == kBlock && b.row - b.first >= g.taps - 1;
     {
         const size_t half = (size_t)(g.taps - 1) * g.channels;
         float* state = p.s.d_conv_state + (size_t)p.s.d_slot[b.row] * 2 * half;
@@ -218,7 +232,14 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Param
         }
         const int head = job, kvh = head / g.group;
         const bool own = head % g.group == 0;   // heads that share q and k: the first passes their convolution state on
-        float q[NI][kBlock], k[NI][kBlock];
+        float q[NI][kBlock], k[NI][kBlock], dec[NI][kBlock];
+#pragma unroll
+        for (int i = 0; i < NI; ++i)   // travels while the convolutions are computed
+#pragma unroll
+            for (int t = 0; t < kBlock; ++t) {
+                const int d = i * 32 + lane;
+                dec[i][t] = t < b.n && d < g.dim ? p.s.d_decay[(size_t)(b.row + t) * g.decay_row + head * g.dim + d] : 0.f;
+            }
         float sums[32];
 #pragma unroll
         for (int i = 0; i < 32; ++i) sums[i] = 0.f;
@@ -255,7 +276,10 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Param
                 const float bias = p.s.d_dt_bias[head * g.dim + d];
 #pragma unroll
                 for (int t = 0; t < kBlock; ++t)
-                    if (t < b.n) gd[t] = expf(rate * softplus(p.s.d_decay[(size_t)(b.row + t) * g.decay_row + head * g.dim + d] + bias));
+                    if (t < b.n) {
+                        const float x = dec[i][t] + bias;
+                        gd[t] = sizeof(T) == 2 ? decay_fast(x, rate) : expf(rate * softplus(x));
+                    }
             }
             const float g10 = gd[1], g21 = gd[2], g32 = gd[3], g20 = g21 * g10, g31 = g32 * g21, g30 = g31 * g10;   // decays of s+1 .. t
             const float* kk = k[i];

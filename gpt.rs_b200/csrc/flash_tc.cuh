@@ -39,12 +39,11 @@ __device__ __forceinline__ int page_chunk(int t, int chunk, int nb) {
 constexpr int kRows = 128;
 constexpr int kKeys = 64;
 constexpr int kTcThreads = 224;
-constexpr int kScores = 3;           // score buffers in tensor memory
+constexpr int kMaxScores = 3;        // score buffers in tensor memory: three with one CTA per SM, two with two
 constexpr int kMaxStages = 6;
 constexpr int kMaxBlocks = 6;        // 64-column blocks of a query
 constexpr uint32_t kWaitLimit = 1u << 16;
 constexpr float kRescaleStep = 8.f;
-constexpr uint32_t kOCol = kScores * kKeys;
 
 // What a kernel's keys, values and queries look like. A cache row is `blocks` blocks of 64 columns: the first value_blocks are the
 // values, the query_blocks from key_block on are the key (latent attention: the key is the whole row and contains the value).
@@ -191,8 +190,11 @@ __device__ __forceinline__ void score_log2(float (&s)[kKeys], float scale_log2, 
 }
 
 // GROUPED: kv heads of their own, soft cap, distance penalty; otherwise one latent row for all heads
-template <bool GROUPED>
-__global__ void __launch_bounds__(kTcThreads, 1) flash_tc_kernel(const __grid_constant__ TcParams p) {
+// kScores 2: two CTAs share an SM (tensor memory, shared memory and registers for half of one each), so that the softmax of one runs
+// under the waits of the other.
+template <bool GROUPED, int kScores>
+__global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_kernel(const __grid_constant__ TcParams p) {
+    constexpr uint32_t kOCol = kScores * kKeys;
     extern __shared__ unsigned char smem_raw[];
     __shared__ __align__(8) uint64_t k_full[kMaxStages], k_empty[kMaxStages], s_full[kScores], p_full[kScores], q_full;
     __shared__ uint32_t tmem_holder;
@@ -307,7 +309,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) flash_tc_kernel(const __grid_co
         for (int it = 0; it < n_blocks && !failed; ++it) {
             const int st = it % p.stages;
             if (!wait(&k_full[st], (uint32_t)(it / p.stages) & 1u)) break;
-            // the weights that were in this buffer have been used up; with three stages or fewer the pages just waited for were
+            // the weights that were in this buffer have been used up; with as many stages or fewer the pages just waited for were
             // requested after that
             if (it >= kScores && p.stages > kScores && !wait(&k_empty[(it - kScores) % p.stages], (uint32_t)((it - kScores) / p.stages) & 1u)) break;
             tc_fence_after();
@@ -526,34 +528,37 @@ __global__ void __launch_bounds__(128) flash_combine_kernel(const CombineParams 
     }
 }
 
-int tc_stages(int query_blocks, int blocks) {
-    const int left = 220 * 1024 - 1024 - query_blocks * kRows * 128, stage = blocks * kKeys * 128;
+int tc_stages(int query_blocks, int blocks, int smem_kb = 220) {
+    const int left = smem_kb * 1024 - 1024 - query_blocks * kRows * 128, stage = blocks * kKeys * 128;
     const int n = left > 0 ? left / stage : 0;
     return n > kMaxStages ? kMaxStages : n;
 }
 bool tc_fits(int query_blocks, int value_blocks, int blocks) {
     return value_blocks <= 4 && query_blocks <= kMaxBlocks && tc_stages(query_blocks, blocks) >= 2;
 }
+// two CTAs per SM: 256 columns of tensor memory and 112 KB of shared memory each
+constexpr int kHalfSmemKb = 112;
+bool tc_fits_twice(int query_blocks, int value_blocks, int blocks) { return value_blocks <= 2 && tc_stages(query_blocks, blocks, kHalfSmemKb) >= 2; }
 size_t tc_scratch_bytes(int64_t n_tiles, int z_blocks, int splits, int value_blocks) {
     return (size_t)n_tiles * z_blocks * splits * kRows * ((size_t)value_blocks * 64 * 4 + 8);
 }
 
 // Launches the kernel and, with key splits, the merge. The caller has filled in everything but the fields set here.
-template <bool GROUPED>
+template <bool GROUPED, int kScores>
 int launch_flash(TcParams& p, int64_t n_tiles, void* d_scratch, cudaStream_t st) {
     const FlashShape& g = p.g;
-    p.stages = tc_stages(g.query_blocks, g.blocks);
+    p.stages = tc_stages(g.query_blocks, g.blocks, kScores == 2 ? kHalfSmemKb : 220);
     p.head_blocks = ceil_div(g.group, kRows);
     p.rows_per_token = g.group < kRows ? g.group : kRows;
-    p.tmem_cols = kOCol + g.value_blocks * 64 <= 256 ? 256 : 512;
+    p.tmem_cols = kScores * kKeys + g.value_blocks * 64 <= 256 ? 256 : 512;
     const int z = g.kv_heads * p.head_blocks;
     const size_t rows = (size_t)n_tiles * z * p.splits * kRows;
     p.part_o = static_cast<float*>(d_scratch);
     p.part_ml = reinterpret_cast<float2*>(p.part_o + rows * (g.value_blocks * 64));
     static PerDeviceOnce attr_once;
-    if (attr_once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(flash_tc_kernel<GROUPED>, cudaFuncAttributeMaxDynamicSharedMemorySize, 221 * 1024));
+    if (attr_once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(flash_tc_kernel<GROUPED, kScores>, cudaFuncAttributeMaxDynamicSharedMemorySize, 221 * 1024));
     const size_t smem = (size_t)g.query_blocks * kRows * 128 + (size_t)p.stages * g.blocks * kKeys * 128 + 1024;
-    int rc = launch_kernel(flash_tc_kernel<GROUPED>, dim3((unsigned)n_tiles, (unsigned)p.splits, (unsigned)z), dim3(kTcThreads), smem, st, 1, p);
+    int rc = launch_kernel(flash_tc_kernel<GROUPED, kScores>, dim3((unsigned)n_tiles, (unsigned)p.splits, (unsigned)z), dim3(kTcThreads), smem, st, 1, p);
     if (rc || p.splits == 1) return rc;
     CombineParams c = {p.part_o, p.part_ml, p.tile_row, p.tile_rows, p.out, g.heads, g.group, p.rows_per_token, p.head_blocks, p.splits, g.value_blocks * 64, g.out_stride};
     // 32 CTAs of four warps cover the 128 rows of a tile

@@ -258,7 +258,8 @@ int gptrs_cuda_grouped_splits(const gptrs_grouped_attention* a, int64_t n_tiles,
     const int64_t limit = a->mask == GPTRS_MASK_CAUSAL ? max_ctx_len : (int64_t)a->mask_size + tokens - 1;
     const int64_t span = max_ctx_len < limit ? max_ctx_len : limit;
     const int64_t blocks = (span + kPageTok - 1 + kKeys - 1) / kKeys;
-    int64_t s = sm_count() / (n_tiles * a->kv_heads * ceil_div(a->heads / a->kv_heads, kRows));
+    const Shape g = shape_of(*a);
+    int64_t s = (tc_fits_twice(g.nb - g.nbv, g.nbv, g.nb) ? 2 : 1) * sm_count() / (n_tiles * a->kv_heads * ceil_div(g.group, kRows));
     if (s > blocks) s = blocks;
     return (int)(s < 1 ? 1 : s);
 }
@@ -316,7 +317,7 @@ int gptrs_cuda_grouped_attention(const gptrs_grouped_attention* a, const void* d
     p.r1 = r1; p.r2 = r2;
     p.scale_log2 = g.softcap > 0.f ? 2.f * kLog2e * g.scale / g.softcap : kLog2e * g.scale;
     p.cap_log2 = g.softcap > 0.f ? kLog2e * g.softcap : 0.f;
-    return launch_flash<true>(p, n_tiles, d_scratch, st);
+    return tc_fits_twice(f.query_blocks, f.value_blocks, f.blocks) ? launch_flash<true, 2>(p, n_tiles, d_scratch, st) : launch_flash<true, 3>(p, n_tiles, d_scratch, st);
 }
 
 }  // extern "C"

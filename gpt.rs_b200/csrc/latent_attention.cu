@@ -378,7 +378,7 @@ int gptrs_cuda_latent_attention(const gptrs_latent_attention* a, const void* d_q
     p.status = d_status;
     p.max_pages = (int)max_pages; p.splits = splits;
     p.scale_log2 = kLog2e * g.scale;
-    return launch_flash<false>(p, n_tiles, d_scratch, st);
+    return launch_flash<false, 3>(p, n_tiles, d_scratch, st);
 }
 
 }  // extern "C"

@@ -539,7 +539,7 @@ int layered_finalize(Model& m, bool drop_leaves) {
         if (L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION) scratch = std::max(scratch, gptrs_cuda_latent_scratch_bytes(&L.att, 1, sm_count() + 1));
         else {
             const int per_split = L.gatt.kv_heads * ((L.gatt.heads / L.gatt.kv_heads + 127) / 128);
-            scratch = std::max(scratch, gptrs_cuda_grouped_scratch_bytes(&L.gatt, 1, sm_count() / per_split + 2));
+            scratch = std::max(scratch, gptrs_cuda_grouped_scratch_bytes(&L.gatt, 1, 2 * sm_count() / per_split + 2));
         }
     }
     if ((rc = y.scratch.alloc(scratch))) return rc;

@@ -98,7 +98,7 @@ class DeltaStep(ctypes.Structure):
     """gptrs_delta_step."""
     _fields_ = [(n, ctypes.c_void_p) for n in ("d_proj", "d_decay", "d_gate", "d_conv", "d_a_log", "d_dt_bias", "d_norm", "d_state", "d_conv_state", "d_slot",
                                                "d_pos", "d_run_first", "d_run_last", "d_parity", "d_runs")] + \
-        [("n_runs", ctypes.c_int64), ("d_out", ctypes.c_void_p), ("d_scratch", ctypes.c_void_p), ("rows", ctypes.c_int64)]
+        [("n_runs", ctypes.c_int64), ("d_out", ctypes.c_void_p), ("d_scratch", ctypes.c_void_p), ("rows", ctypes.c_int64), ("d_status", ctypes.c_void_p)]
 
 
 class Moe(ctypes.Structure):

@@ -14,14 +14,14 @@
 // Every factor is a product of decays, at most 1.
 //   delta_prepare_kernel   prompts: a CTA per block, a warp per head: convolutions with their state, unit norms, decays, the vectors
 //                          p_t k_t, p_t q_t, c_t, p_3 and the numbers A, B of the block
-//   delta_scan_kernel      prompts: a warp keeps 16 columns of a head's S in registers over a whole run (packed pairs of key channels,
-//                          fma.rn.f32x2); blocks arrive in a ring of shared-memory stages; the sums meet in a transposing reduction
+//   delta_scan_kernel      prompts: a warp keeps a few columns of a head's S in registers over a whole run (packed pairs of key channels,
+//                          fma.rn.f32x2); blocks arrive by bulk copies in a ring of shared-memory stages (bounded waits, status 3); the sums meet in a transposing reduction
 //   delta_output_kernel    prompts: norm and gate of the read-outs
 //   delta_decode_kernel    rows that are runs of their own: all of the above in one launch, a CTA per (head, row), S is read and
 //                          written once
 // Everything that enters the recurrence, and S itself, is f32. S is updated in place (one CTA owns a column of a slot's state);
 // the convolution state has two halves like the one of post_norm_conv.cu.
-#include "common.cuh"
+#include "umma_common.cuh"
 
 namespace gptrs {
 namespace {
@@ -175,22 +175,25 @@ __device__ __forceinline__ void conv_block(const Params& p, const BlockState& b,
         if (b.last - (b.row + t) < keep) b.fresh[(size_t)((b.pos + t) % keep) * p.g.channels + ch] = ld(x + (int64_t)t * p.g.row);
 }
 
-// sums of 32 values over the warp: lane i gets the sum of v[i]
-__device__ __forceinline__ float transpose_sum(float (&v)[32]) {
+// sums of N values over the warp: lane i gets the sum of v[i mod N]
+template <int N>
+__device__ __forceinline__ float transpose_sum(float (&v)[N]) {
     const int lane = threadIdx.x & 31;
 #pragma unroll
-    for (int h = 16; h >= 1; h >>= 1)
+    for (int h = N / 2; h >= 1; h >>= 1)
 #pragma unroll
         for (int i = 0; i < h; ++i) {
             const float give = (lane & h) ? v[i] : v[i + h], keep = (lane & h) ? v[i + h] : v[i];
             v[i] = keep + __shfl_xor_sync(0xffffffffu, give, h);
         }
+#pragma unroll
+    for (int h = N; h < 32; h <<= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], h);
     return v[0];
 }
 
 // NI: groups of 32 key channels
 template <typename T, int NI, int TAPS>
-__global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Params p) {
+__global__ void __launch_bounds__(kPrepThreads, NI <= 4 ? 3 : 1) delta_prepare_kernel(const Params p) {
     const Geo& g = p.g;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, blk = blockIdx.x;
     pdl_launch_dependents();
@@ -240,9 +243,9 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Param
                 const int d = i * 32 + lane;
                 dec[i][t] = t < b.n && d < g.dim ? p.s.d_decay[(size_t)(b.row + t) * g.decay_row + head * g.dim + d] : 0.f;
             }
-        float sums[32];
+        float sums[8];
 #pragma unroll
-        for (int i = 0; i < 32; ++i) sums[i] = 0.f;
+        for (int i = 0; i < 8; ++i) sums[i] = 0.f;
 #pragma unroll
         for (int i = 0; i < NI; ++i) {
             const int d = i * 32 + lane;
@@ -265,9 +268,9 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Param
         }
         const float rate = -expf(p.s.d_a_log[head]);
         float* vec = p.w.vec + ((size_t)blk * g.heads + head) * kVecs * g.dp;
-        float num[32];   // A in 0 .. 5, B in 8 .. 17
+        float num[16];   // A in 0 .. 5, B in 6 .. 15
 #pragma unroll
-        for (int i = 0; i < 32; ++i) num[i] = 0.f;
+        for (int i = 0; i < 16; ++i) num[i] = 0.f;
 #pragma unroll
         for (int i = 0; i < NI; ++i) {
             const int d = i * 32 + lane;
@@ -290,16 +293,16 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Param
             num[3] = fmaf(kk[3] * kk[0], g30, num[3]);
             num[4] = fmaf(kk[3] * kk[1], g31, num[4]);
             num[5] = fmaf(kk[3] * kk[2], g32, num[5]);
-            num[8] = fmaf(qq[0], kk[0], num[8]);
-            num[9] = fmaf(qq[1] * kk[0], g10, num[9]);
-            num[10] = fmaf(qq[1], kk[1], num[10]);
-            num[11] = fmaf(qq[2] * kk[0], g20, num[11]);
-            num[12] = fmaf(qq[2] * kk[1], g21, num[12]);
-            num[13] = fmaf(qq[2], kk[2], num[13]);
-            num[14] = fmaf(qq[3] * kk[0], g30, num[14]);
-            num[15] = fmaf(qq[3] * kk[1], g31, num[15]);
-            num[16] = fmaf(qq[3] * kk[2], g32, num[16]);
-            num[17] = fmaf(qq[3], kk[3], num[17]);
+            num[6] = fmaf(qq[0], kk[0], num[6]);
+            num[7] = fmaf(qq[1] * kk[0], g10, num[7]);
+            num[8] = fmaf(qq[1], kk[1], num[8]);
+            num[9] = fmaf(qq[2] * kk[0], g20, num[9]);
+            num[10] = fmaf(qq[2] * kk[1], g21, num[10]);
+            num[11] = fmaf(qq[2], kk[2], num[11]);
+            num[12] = fmaf(qq[3] * kk[0], g30, num[12]);
+            num[13] = fmaf(qq[3] * kk[1], g31, num[13]);
+            num[14] = fmaf(qq[3] * kk[2], g32, num[14]);
+            num[15] = fmaf(qq[3], kk[3], num[15]);
             if (d < g.dp) {
                 const float p0 = gd[0], p1 = p0 * gd[1], p2 = p1 * gd[2], p3 = p2 * gd[3];
                 float* o = vec + d;
@@ -311,29 +314,35 @@ __global__ void __launch_bounds__(kPrepThreads) delta_prepare_kernel(const Param
         }
         const float mine = transpose_sum(num);
         float* dst = p.w.num + ((size_t)blk * g.heads + head) * kNums;
-        if (lane < 18) dst[4 + lane] = mine;
+        if (lane < 16) dst[lane < 6 ? 4 + lane : 6 + lane] = mine;
         if (lane < kBlock)
             dst[lane] = lane < b.n ? sigmoid(ld(static_cast<const T*>(p.s.d_proj) + (size_t)(b.row + lane) * g.row + g.beta_off + head)) : 0.f;
     }
 }
 
 // ---- the scan ------------------------------------------------------------------------------------------------------------------
-constexpr int kScanWarps = 4;
+constexpr int kScanWarps = 8;
 
-// Eight lanes share a column: lane l holds the channels (8 i + l) 4 + e, i < NI, of CPL neighbouring columns; four such groups
-// make a warp. dim <= 32 NI.
-template <int NI, int CPL, int STAGES>
+// LPC lanes share a column: lane l holds the channels (LPC i + l) 4 + e, i < NI, of CPL neighbouring columns; 32 / LPC such groups
+// make a warp. dim <= 4 LPC NI. 
+template <int NI, int CPL, int LPC, int STAGES>
 __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Params p) {
-    constexpr int W = 32 * NI;                                      // channels with padding
-    constexpr int COLS = kScanWarps * 4 * CPL;                      // columns of the CTA
+    constexpr int W = 4 * LPC * NI;                                 // channels with padding
+    constexpr int GROUPS = 32 / LPC, COLS = kScanWarps * GROUPS * CPL;
     constexpr int kStage = kVecs * W + kBlock * COLS + kNums;       // floats
-    constexpr int SH = CPL == 4 ? 0 : CPL == 2 ? 1 : 2;             // lane bits that are left after (column, k or q)
+    constexpr int SH = (LPC == 16 ? 4 : 3) - (CPL == 4 ? 2 : CPL == 2 ? 1 : 0) - 1;   // lane bits that are left after (column, k or q)
     extern __shared__ __align__(16) float ds_smem[];
+    __shared__ __align__(8) uint64_t full[STAGES];
     const Geo& g = p.g;
-    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = lane & 7, cg = lane >> 3;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, l = lane & (LPC - 1), cg = lane / LPC;
     const int head = blockIdx.y;
-    const int c_blk = blockIdx.x * COLS, col0 = c_blk + (warp * 4 + cg) * CPL;
+    const int c_blk = blockIdx.x * COLS, col0 = c_blk + (warp * GROUPS + cg) * CPL;
     for (int i = tid; i < STAGES * kStage; i += kScanWarps * 32) ds_smem[i] = 0.f;   // the padding stays zero
+    if (tid == 0) {
+        for (int i = 0; i < STAGES; ++i) mbar_init(&full[i], 1);
+        mbar_fence_init();
+    }
+    fence_proxy_async();
     pdl_launch_dependents();
     pdl_wait();
     const int run = blockIdx.z, r0 = p.s.d_runs[run], r1 = p.s.d_run_last[r0] + 1;
@@ -347,35 +356,40 @@ __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Param
         for (int e = 0; e < 2; ++e)
 #pragma unroll
             for (int j = 0; j < CPL; ++j) {
-                const int d = (8 * i + l) * 4 + 2 * e;
+                const int d = (LPC * i + l) * 4 + 2 * e;
                 const bool in = !fresh && col0 + j < g.vdim;
                 S[i][e][j] = pair_of(in && d < g.dim ? state[(size_t)d * g.vdim + col0 + j] : 0.f, in && d + 1 < g.dim ? state[(size_t)(d + 1) * g.vdim + col0 + j] : 0.f);
             }
     __syncthreads();
-    const int d4 = g.dp / 4, v4 = min(COLS, g.vp - c_blk) / 4;
-    auto request = [&](int b) {   // block b of the run; always one group of copies
-        if (b < n_blk) {
-            float* sm = ds_smem + (b % STAGES) * kStage;
-            const size_t at = (size_t)(blk0 + b) * g.heads + head;
-            for (int i = tid; i < kVecs * d4; i += kScanWarps * 32) {
-                const int x = i / d4, c = (i % d4) * 4;
-                cp_async_16(sm + x * W + c, p.w.vec + (at * kVecs + x) * g.dp + c, true);
-            }
-            for (int i = tid; i < kBlock * v4; i += kScanWarps * 32) {
-                const int t = i / v4, c = (i % v4) * 4;
-                cp_async_16(sm + kVecs * W + t * COLS + c, p.w.v + (at * kBlock + t) * g.vp + c_blk + c, true);
-            }
-            if (tid < kNums / 4) cp_async_16(sm + kVecs * W + kBlock * COLS + tid * 4, p.w.num + at * kNums + tid * 4, true);
-        }
-        cp_async_commit();
+    // the copies of a block, one per lane of warp 0: 13 vectors (a single one where they need no padding), 4 rows of values, the numbers
+    const bool packed = g.dp == W;
+    const uint32_t vec_bytes = (uint32_t)(packed ? kVecs : 1) * g.dp * 4, v_bytes = (uint32_t)min(COLS, g.vp - c_blk) * 4;
+    const float* src = nullptr;   // of block 0
+    uint32_t dst = 0, bytes = 0;
+    size_t step = 0;
+    if (warp == 0) {
+        const size_t at = (size_t)blk0 * g.heads + head;
+        if (lane < kVecs && (lane == 0 || !packed)) { src = p.w.vec + (at * kVecs + lane) * g.dp; dst = lane * W; bytes = vec_bytes; step = (size_t)g.heads * kVecs * g.dp; }
+        else if (lane >= 16 && lane < 16 + kBlock) { src = p.w.v + (at * kBlock + lane - 16) * g.vp + c_blk; dst = kVecs * W + (lane - 16) * COLS; bytes = v_bytes; step = (size_t)g.heads * kBlock * g.vp; }
+        else if (lane == 20) { src = p.w.num + at * kNums; dst = kVecs * W + kBlock * COLS; bytes = kNums * 4; step = (size_t)g.heads * kNums; }
+    }
+    const uint32_t total = (uint32_t)kVecs * g.dp * 4 + kBlock * v_bytes + kNums * 4, smem0 = smem_u32(ds_smem);
+    auto request = [&](int b) {   // warp 0: block b of the run
+        if (b >= n_blk) return;
+        const uint32_t bar = smem_u32(&full[b % STAGES]);
+        if (lane == 0) mbar_expect_tx_addr(bar, total);
+        __syncwarp();
+        if (bytes) bulk_g2s_addr(smem0 + ((b % STAGES) * kStage + dst) * 4, src + b * step, bytes, bar);
     };
+    if (warp == 0)
 #pragma unroll
-    for (int b = 0; b < STAGES - 1; ++b) request(b);
+        for (int b = 0; b < STAGES - 1; ++b) request(b);
+    bool failed = false;
 #pragma unroll 1
     for (int b = 0; b < n_blk; ++b) {
-        cp_async_wait<STAGES - 2>();
-        __syncthreads();          // block b is there, and everyone is done with block b - 1
-        request(b + STAGES - 1);
+        __syncthreads();          // everyone is done with block b - 1
+        if (warp == 0) request(b + STAGES - 1);
+        if (!failed && !mbar_wait_relaxed(&full[b % STAGES], (uint32_t)(b / STAGES) & 1u)) failed = true;   // bounded: reported below
         const float* sm = ds_smem + (b % STAGES) * kStage;
         const float* lanes = sm + l * 4;
         uint64_t acc[8][CPL];     // p_t k_t, then p_t q_t
@@ -387,11 +401,11 @@ __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Param
         for (int i = 0; i < NI; ++i)
 #pragma unroll
             for (int x = 0; x < 8; ++x) {
-                const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(lanes + x * W + 32 * i);
+                const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(lanes + x * W + 4 * LPC * i);
 #pragma unroll
                 for (int j = 0; j < CPL; ++j) acc[x][j] = fma2(S[i][1][j], v.y, fma2(S[i][0][j], v.x, acc[x][j]));
             }
-        // transposing reduction over the eight lanes: this lane ends up with the four sums of (column j_mine, k or q)
+        // transposing reduction over the lanes of a column: this lane ends up with the four sums of (column j_mine, k or q)
         float r[CPL][2][kBlock];
 #pragma unroll
         for (int j = 0; j < CPL; ++j)
@@ -403,12 +417,13 @@ __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Param
 #pragma unroll
                 for (int x = 0; x < 8; ++x) {
                     float &a = r[j][x >> 2][x & 3], &c = r[j + 2][x >> 2][x & 3];
-                    const float give = (l & 4) ? a : c, keep = (l & 4) ? c : a;
-                    a = keep + __shfl_xor_sync(0xffffffffu, give, 4);
+                    constexpr int bit = LPC / 2;
+                    const float give = (l & bit) ? a : c, keep = (l & bit) ? c : a;
+                    a = keep + __shfl_xor_sync(0xffffffffu, give, bit);
                 }
         }
         if constexpr (CPL >= 2) {
-            constexpr int bit = CPL == 4 ? 2 : 4;
+            constexpr int bit = CPL == 4 ? LPC / 4 : LPC / 2;
 #pragma unroll
             for (int x = 0; x < 8; ++x) {
                 float &a = r[0][x >> 2][x & 3], &c = r[1][x >> 2][x & 3];
@@ -440,7 +455,7 @@ __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Param
         for (int j = 0; j < CPL; ++j)
 #pragma unroll
             for (int t = 0; t < kBlock; ++t) {
-                const float x = __shfl_sync(0xffffffffu, u[t], (lane & 24) + ((2 * j) << SH));
+                const float x = __shfl_sync(0xffffffffu, u[t], (lane & ~(LPC - 1)) + ((2 * j) << SH));
                 uu[j][t] = pair_of(x, x);
             }
         float uo[kBlock];
@@ -448,12 +463,12 @@ __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Param
         for (int t = 0; t < kBlock; ++t) uo[t] = __shfl_xor_sync(0xffffffffu, u[t], 1 << SH);
 #pragma unroll
         for (int i = 0; i < NI; ++i) {
-            const ulonglong2 gv = *reinterpret_cast<const ulonglong2*>(lanes + 12 * W + 32 * i);
+            const ulonglong2 gv = *reinterpret_cast<const ulonglong2*>(lanes + 12 * W + 4 * LPC * i);
 #pragma unroll
             for (int j = 0; j < CPL; ++j) { S[i][0][j] = mul2(S[i][0][j], gv.x); S[i][1][j] = mul2(S[i][1][j], gv.y); }
 #pragma unroll
             for (int t = 0; t < kBlock; ++t) {
-                const ulonglong2 c = *reinterpret_cast<const ulonglong2*>(lanes + (8 + t) * W + 32 * i);
+                const ulonglong2 c = *reinterpret_cast<const ulonglong2*>(lanes + (8 + t) * W + 4 * LPC * i);
 #pragma unroll
                 for (int j = 0; j < CPL; ++j) { S[i][0][j] = fma2(c.x, uu[j][t], S[i][0][j]); S[i][1][j] = fma2(c.y, uu[j][t], S[i][1][j]); }
             }
@@ -469,14 +484,17 @@ __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Param
             if (row + 3 < r1) o[3 * step] = fmaf(b2.y, uo[3], fmaf(b2.x, uo[2], fmaf(b1.w, uo[1], fmaf(b1.z, uo[0], y[3]))));
         }
     }
-    cp_async_wait<0>();
+    if (failed) {
+        for (int b = max(n_blk - STAGES, 0); b < n_blk; ++b) mbar_wait_relaxed(&full[b % STAGES], (uint32_t)(b / STAGES) & 1u);   // copies in flight land in this CTA
+        atomicExch(p.s.d_status, 3);
+    }
 #pragma unroll
     for (int i = 0; i < NI; ++i)
 #pragma unroll
         for (int e = 0; e < 2; ++e)
 #pragma unroll
             for (int j = 0; j < CPL; ++j) {
-                const int d = (8 * i + l) * 4 + 2 * e;
+                const int d = (LPC * i + l) * 4 + 2 * e;
                 const float2 x = split(S[i][e][j]);
                 if (col0 + j < g.vdim && d < g.dim) state[(size_t)d * g.vdim + col0 + j] = x.x;
                 if (col0 + j < g.vdim && d + 1 < g.dim) state[(size_t)(d + 1) * g.vdim + col0 + j] = x.y;
@@ -639,13 +657,14 @@ __global__ void __launch_bounds__(kDecThreads) delta_decode_kernel(const Params 
     for (int c = tid; c < g.out_stride; c += kDecThreads) st(out + c, c < g.vdim ? o[c] * inv * p.s.d_norm[c] * sigmoid(ld(gate + c)) : 0.f);
 }
 
-template <int NI, int CPL, int STAGES>
+template <int NI, int CPL, int LPC, int STAGES>
 int launch_scan(const Params& p, cudaStream_t s) {
-    constexpr int cols = kScanWarps * 4 * CPL;
-    constexpr size_t smem = (size_t)STAGES * (kVecs * 32 * NI + kBlock * cols + kNums) * 4;
+    constexpr int cols = kScanWarps * 32 / LPC * CPL;
+    constexpr size_t smem = (size_t)STAGES * (kVecs * 4 * LPC * NI + kBlock * cols + kNums) * 4;
     static PerDeviceOnce once;
-    if (once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(delta_scan_kernel<NI, CPL, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    return launch_kernel(delta_scan_kernel<NI, CPL, STAGES>, dim3((unsigned)ceil_div(p.g.vdim, cols), (unsigned)p.g.heads, (unsigned)p.s.n_runs), dim3(kScanWarps * 32), smem, s, 1, p);
+    if (once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(delta_scan_kernel<NI, CPL, LPC, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    return launch_kernel(delta_scan_kernel<NI, CPL, LPC, STAGES>, dim3((unsigned)ceil_div(p.g.vdim, cols), (unsigned)p.g.heads, (unsigned)p.s.n_runs), dim3(kScanWarps * 32), smem,
+                         s, 1, p);
 }
 template <typename T, int NI>
 int launch_prepare(const Params& p, cudaStream_t s) {
@@ -671,11 +690,11 @@ int run(const Params& p, cudaStream_t s) {
         return launch_decode<T, 64, 1>(p, s);
     }
     int rc = GPTRS_OK;
-    if (g.dim <= 32) { if (!(rc = launch_prepare<T, 1>(p, s))) rc = launch_scan<1, 4, 4>(p, s); }
-    else if (g.dim <= 64) { if (!(rc = launch_prepare<T, 2>(p, s))) rc = launch_scan<2, 4, 4>(p, s); }
-    else if (g.dim <= 128) { if (!(rc = launch_prepare<T, 4>(p, s))) rc = launch_scan<4, 4, 4>(p, s); }
-    else if (g.dim <= 256) { if (!(rc = launch_prepare<T, 8>(p, s))) rc = launch_scan<8, 2, 4>(p, s); }
-    else { if (!(rc = launch_prepare<T, 16>(p, s))) rc = launch_scan<16, 1, 4>(p, s); }
+    if (g.dim <= 32) { if (!(rc = launch_prepare<T, 1>(p, s))) rc = launch_scan<1, 2, 8, 4>(p, s); }
+    else if (g.dim <= 64) { if (!(rc = launch_prepare<T, 2>(p, s))) rc = launch_scan<1, 4, 16, 4>(p, s); }
+    else if (g.dim <= 128) { if (!(rc = launch_prepare<T, 4>(p, s))) rc = launch_scan<2, 4, 16, 4>(p, s); }
+    else if (g.dim <= 256) { if (!(rc = launch_prepare<T, 8>(p, s))) rc = launch_scan<4, 4, 16, 4>(p, s); }
+    else { if (!(rc = launch_prepare<T, 16>(p, s))) rc = launch_scan<8, 2, 16, 4>(p, s); }
     if (rc) return rc;
     return launch_kernel(delta_output_kernel<T>, dim3((unsigned)ceil_div(p.s.rows * g.heads, 8)), dim3(256), 0, s, 1, p);
 }
@@ -723,7 +742,7 @@ int gptrs_cuda_delta_rule(const gptrs_delta_rule* a, const gptrs_delta_step* ste
     GPTRS_REQUIRE(s.d_slot && s.d_pos && s.d_run_first && s.d_run_last && s.d_parity, "null pointer");
     GPTRS_REQUIRE(s.rows >= 0 && s.rows < (1ll << 31) && s.n_runs >= 0 && s.n_runs <= s.rows && s.n_runs <= 65535, "delta rule: rows and runs");
     if (s.rows == 0) return GPTRS_OK;
-    GPTRS_REQUIRE(s.n_runs == s.rows || (s.n_runs > 0 && s.d_runs && s.d_scratch && (reinterpret_cast<uintptr_t>(s.d_scratch) & 15) == 0), "delta rule: run list and scratch");
+    GPTRS_REQUIRE(s.n_runs == s.rows || (s.n_runs > 0 && s.d_runs && s.d_status && s.d_scratch && (reinterpret_cast<uintptr_t>(s.d_scratch) & 15) == 0), "delta rule: run list and scratch");
     Params p = {s, geo(*a), {}};
     if (s.n_runs != s.rows) p.w = planes(p.g, s.d_scratch, s.rows, s.n_runs);
     return a->dtype == GPTRS_BF16 ? run<__nv_bfloat16>(p, as_stream(stream)) : run<float>(p, as_stream(stream));

@@ -373,7 +373,10 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
         float r1 = 0.f, r2 = 0.f;
         if (GROUPED && p.r1 && r < live) { r1 = p.r1[heads0 + r % heads_n]; r2 = p.r2[heads0 + r % heads_n]; }
         const uint32_t t_lane = tmem + ((uint32_t)(warp * 32) << 16);
-        float m_run = -1e30f, l_run = 0.f;
+        // capped scores of up to 60 in log2 units need no running maximum: every row sees itself at no distance, so its largest weight lies
+        // between 2^-60 and 2^60
+        const bool fixed = GROUPED && p.cap_log2 > 0.f && p.cap_log2 <= 60.f;
+        float m_run = fixed ? 0.f : -1e30f, l_run = 0.f;
         if ((dup ? warp & 1 : warp) < live_warps) {
             for (int it = 0; it < n_blocks; ++it) {
                 const int buf = it % kScores;
@@ -392,38 +395,57 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
                     for (int j = 0; j < kKeys; ++j)
                         if (j < v_lo || j >= v_hi) s[j] = -INFINITY;
                 }
-                float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+                if (!fixed) {
+                    float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-                for (int j = 0; j < kKeys; ++j) mx[j & 3] = fmaxf(mx[j & 3], s[j]);
-                const float m_blk = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * mul;   // the scale is positive
-                float alpha = 1.f;
-                if (m_blk > m_run + kRescaleStep) {   // always at a row's first visible key
-                    alpha = ex2f(m_run - m_blk);
-                    m_run = m_blk;
-                }
-                if (it > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
-                    // the product of the block before must be complete
-                    if (!wait(&k_empty[(it - 1) % p.stages], (uint32_t)((it - 1) / p.stages) & 1u)) break;
-                    tc_fence_after();
-#pragma unroll 1
-                    for (int c = 0; c < g.value_blocks * 2; ++c) {
-                        float o[32];
-                        tmem_ld_32(t_lane + kOCol + 32u * c, o);
-#pragma unroll
-                        for (int i = 0; i < 32; ++i) o[i] *= alpha;
-                        tmem_st_32(t_lane + kOCol + 32u * c, *reinterpret_cast<uint32_t(*)[32]>(&o[0]));
+                    for (int j = 0; j < kKeys; ++j) mx[j & 3] = fmaxf(mx[j & 3], s[j]);
+                    const float m_blk = fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])) * mul;   // the scale is positive
+                    float alpha = 1.f;
+                    if (m_blk > m_run + kRescaleStep) {   // always at a row's first visible key
+                        alpha = ex2f(m_run - m_blk);
+                        m_run = m_blk;
                     }
+                    if (it > 0 && __any_sync(0xffffffffu, alpha != 1.f)) {
+                        // the product of the block before must be complete
+                        if (!wait(&k_empty[(it - 1) % p.stages], (uint32_t)((it - 1) / p.stages) & 1u)) break;
+                        tc_fence_after();
+#pragma unroll 1
+                        for (int c = 0; c < g.value_blocks * 2; ++c) {
+                            float o[32];
+                            tmem_ld_32(t_lane + kOCol + 32u * c, o);
+#pragma unroll
+                            for (int i = 0; i < 32; ++i) o[i] *= alpha;
+                            tmem_st_32(t_lane + kOCol + 32u * c, *reinterpret_cast<uint32_t(*)[32]>(&o[0]));
+                        }
+                    }
+                    l_run *= alpha;
                 }
-                l_run *= alpha;
                 const float neg_m = -m_run;
                 float sum[4] = {0.f, 0.f, 0.f, 0.f};
                 uint32_t hi_w[kKeys / 2], lo_w[kKeys / 2];
+                if constexpr (GROUPED) {
+                    const uint64_t nm = pair_of(neg_m, neg_m), one = pair_of(1.f, 1.f), minus = pair_of(-1.f, -1.f);
+                    uint64_t acc[2] = {0, 0};
 #pragma unroll
-                for (int i = 0; i < kKeys / 2; ++i) {
-                    const float p0 = ex2f(fmaf(s[2 * i], mul, neg_m)), p1 = ex2f(fmaf(s[2 * i + 1], mul, neg_m));
-                    sum[i & 3] += p0 + p1;
-                    hi_w[i] = pack_bf16x2(p0, p1);
-                    lo_w[i] = pack_bf16x2(p0 - bf16_lo(hi_w[i]), p1 - bf16_hi(hi_w[i]));
+                    for (int i = 0; i < kKeys / 2; ++i) {
+                        const float2 x = split(fma2(pair_of(s[2 * i], s[2 * i + 1]), one, nm));
+                        const float p0 = ex2f(x.x), p1 = ex2f(x.y);
+                        const uint64_t pp = pair_of(p0, p1);
+                        acc[i & 1] = fma2(pp, one, acc[i & 1]);
+                        hi_w[i] = pack_bf16x2(p0, p1);
+                        const float2 lo = split(fma2(pair_of(bf16_lo(hi_w[i]), bf16_hi(hi_w[i])), minus, pp));
+                        lo_w[i] = pack_bf16x2(lo.x, lo.y);
+                    }
+                    const float2 a0 = split(acc[0]), a1 = split(acc[1]);
+                    sum[0] = a0.x; sum[1] = a0.y; sum[2] = a1.x; sum[3] = a1.y;
+                } else {
+#pragma unroll
+                    for (int i = 0; i < kKeys / 2; ++i) {
+                        const float p0 = ex2f(fmaf(s[2 * i], mul, neg_m)), p1 = ex2f(fmaf(s[2 * i + 1], mul, neg_m));
+                        sum[i & 3] += p0 + p1;
+                        hi_w[i] = pack_bf16x2(p0, p1);
+                        lo_w[i] = pack_bf16x2(p0 - bf16_lo(hi_w[i]), p1 - bf16_hi(hi_w[i]));
+                    }
                 }
                 if (!dup) {
                     tmem_st_32(t_s, hi_w);

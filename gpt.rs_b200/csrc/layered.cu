@@ -727,7 +727,7 @@ struct Pass {
         s.d_slot = slot(); s.d_pos = pos();
         s.d_run_first = y.d_run_first.as<int32_t>(); s.d_run_last = y.d_run_last.as<int32_t>(); s.d_parity = y.d_parity.as<int32_t>();
         s.d_runs = y.d_runs.as<int32_t>(); s.n_runs = y.n_runs;
-        s.d_out = y.attn.p; s.d_scratch = y.delta_scratch.as<float>(); s.rows = T;
+        s.d_out = y.attn.p; s.d_scratch = y.delta_scratch.as<float>(); s.rows = T; s.d_status = m.d_status.as<int32_t>();
         m.launches += y.n_runs == T ? 1 : 3;
         if ((rc = gptrs_cuda_delta_rule(&a, &s, st))) return rc;
         return dense(m, w.out, y.attn.p, y.y.p, T, {});

@@ -545,7 +545,7 @@ def delta_layout(heads, kv_heads, dim, vdim, taps, decay_rank, gate_rank, eps, b
     return a
 
 
-def delta_rule(a, proj, decay, gate, conv, a_log, dt_bias, norm, state, conv_state, runs, first_rows, n_runs=None):
+def delta_rule(a, proj, decay, gate, conv, a_log, dt_bias, norm, state, conv_state, runs, first_rows, n_runs=None, status=None):
     """`runs` = (slot, pos, run_first, run_last, parity) per row, `first_rows` = first row of every run; states are updated in place."""
     n = proj.shape[0]
     out = torch.empty((n, a.heads, a.out_head_stride), dtype=proj.dtype, device=proj.device)
@@ -555,7 +555,8 @@ def delta_rule(a, proj, decay, gate, conv, a_log, dt_bias, norm, state, conv_sta
     s.d_slot, s.d_pos, s.d_run_first, s.d_run_last, s.d_parity = (_ptr(t) for t in runs)
     s.d_runs, s.n_runs, s.rows, s.d_out = _ptr(first_rows), first_rows.shape[0] if n_runs is None else n_runs, n, _ptr(out)
     scratch = torch.empty(max(lib().gptrs_cuda_delta_scratch_floats(ctypes.byref(a), n, s.n_runs), 1), dtype=torch.float32, device=proj.device)
-    s.d_scratch = _ptr(scratch)
+    status = _status(proj.device, status)
+    s.d_scratch, s.d_status = _ptr(scratch), _ptr(status)
     check(lib().gptrs_cuda_delta_rule(ctypes.byref(a), ctypes.byref(s), _stream()))
     return out
 

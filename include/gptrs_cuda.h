@@ -402,6 +402,7 @@ typedef struct {
     void* d_out;               /* [T][heads][out_head_stride] */
     float* d_scratch;          /* gptrs_cuda_delta_scratch_floats of them (0 when n_runs = rows) */
     int64_t rows;
+    int32_t* d_status;         /* receives 3 when a bounded wait gives up (required unless n_runs = rows) */
 } gptrs_delta_step;
 int gptrs_cuda_delta_rule(const gptrs_delta_rule* a, const gptrs_delta_step* step, void* stream);
 

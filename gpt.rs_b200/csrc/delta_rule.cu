@@ -88,37 +88,57 @@ __device__ __forceinline__ float decay_of(const Params& p, int row, int head, in
     return expf(-expf(p.s.d_a_log[head]) * softplus(p.s.d_decay[(size_t)row * p.g.decay_row + c] + p.s.d_dt_bias[c]));
 }
 
-// A row's place in its run, and the convolution state it reads and writes.
-struct RowState { int pos, first, len_before, last; const float* old; float* fresh; };
+// The convolution state that a single-token run reads and writes; place: where in the ring of taps - 1 inputs the last one lies.
+struct RowState { int pos, place; const float* old; float* fresh; };
 __device__ __forceinline__ RowState row_state(const Params& p, int row) {
     RowState r;
-    r.pos = p.s.d_pos[row]; r.first = p.s.d_run_first[row]; r.last = p.s.d_run_last[row];
-    r.len_before = row - r.first;
-    const size_t half = (size_t)(p.g.taps - 1) * p.g.channels;
+    const int keep = p.g.taps - 1;
+    r.pos = p.s.d_pos[row];
+    r.place = keep > 0 && r.pos > 0 ? (r.pos - 1) % keep : 0;
+    const size_t half = (size_t)keep * p.g.channels;
     float* state = p.s.d_conv_state + (size_t)p.s.d_slot[row] * 2 * half;
     const int par = p.s.d_parity[row] & 1;
     r.old = state + par * half; r.fresh = state + (par ^ 1) * half;
     return r;
 }
-// silu(convolution) of channel `ch` (column `col` of the projection row); `keep_state`: this thread also passes the channel's
-// inputs on to the next step
+// silu(convolution) of channel `ch` (column `col` of the projection row) where the row is a run of its own; `keep_state`: this thread
+// also passes the channel's inputs on to the next step. The loads of four taps or fewer are all under way at once.
 template <typename T>
 __device__ __forceinline__ float conv_channel(const Params& p, const RowState& r, int row, int ch, int col, bool keep_state) {
     const int keep = p.g.taps - 1;
-    const T* x = static_cast<const T*>(p.s.d_proj) + (size_t)row * p.g.row + col;
+    const float now = ld(static_cast<const T*>(p.s.d_proj) + (size_t)row * p.g.row + col);
     const float* w = p.s.d_conv + (size_t)ch * p.g.taps;
     float acc = 0.f;
-    for (int k = keep; k >= 1; --k) {   // the input k positions back
-        const int at = r.pos - k;
-        float v = 0.f;
-        if (k <= r.len_before) v = ld(x - (size_t)k * p.g.row);
-        else if (at >= 0) v = r.old[(size_t)(at % keep) * p.g.channels + ch];
-        acc = fmaf(w[keep - k], v, acc);
-        // first row of a run shorter than the state: what the run does not push out stays
-        if (keep_state && row == r.first && at >= 0 && at > r.pos + (r.last - row) - keep) r.fresh[(size_t)(at % keep) * p.g.channels + ch] = v;
+    if (keep <= 3) {
+        float v[3] = {0.f, 0.f, 0.f}, wt[3] = {0.f, 0.f, 0.f};
+        int at[3];
+#pragma unroll
+        for (int k = 0; k < 3; ++k) {   // the input k + 1 positions back lies at r.place - k of the ring
+            at[k] = r.place - k < 0 ? r.place - k + keep : r.place - k;
+            if (k < keep) {
+                wt[k] = __ldg(w + keep - 1 - k);
+                if (r.pos - 1 - k >= 0) v[k] = r.old[(size_t)at[k] * p.g.channels + ch];
+            }
+        }
+        const float w_now = __ldg(w + keep);
+#pragma unroll
+        for (int k = 2; k >= 0; --k) acc = fmaf(wt[k], v[k], acc);
+        if (keep_state && keep > 0) {
+#pragma unroll
+            for (int k = 0; k < 2; ++k)   // the oldest one leaves
+                if (k < keep - 1 && r.pos - 1 - k >= 0) r.fresh[(size_t)at[k] * p.g.channels + ch] = v[k];
+            r.fresh[(size_t)(r.pos % keep) * p.g.channels + ch] = now;
+        }
+        return silu(fmaf(w_now, now, acc));
     }
-    const float now = ld(x);
-    if (keep_state && keep > 0 && r.last - row < keep) r.fresh[(size_t)(r.pos % keep) * p.g.channels + ch] = now;
+    for (int k = keep; k >= 1; --k) {
+        const int q = r.pos - k;
+        if (q < 0) continue;
+        const float v = r.old[(size_t)(q % keep) * p.g.channels + ch];
+        acc = fmaf(w[keep - k], v, acc);
+        if (keep_state && k < keep) r.fresh[(size_t)(q % keep) * p.g.channels + ch] = v;
+    }
+    if (keep_state) r.fresh[(size_t)(r.pos % keep) * p.g.channels + ch] = now;
     return silu(fmaf(w[keep], now, acc));
 }
 
@@ -193,7 +213,7 @@ __device__ __forceinline__ float transpose_sum(float (&v)[N]) {
 
 // NI: groups of 32 key channels
 template <typename T, int NI, int TAPS>
-__global__ void __launch_bounds__(kPrepThreads, NI <= 4 ? 3 : 1) delta_prepare_kernel(const Params p) {
+__global__ void __launch_bounds__(kPrepThreads, NI <= 4 ? 4 : 1) delta_prepare_kernel(const Params p) {
     const Geo& g = p.g;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, blk = blockIdx.x;
     pdl_launch_dependents();
@@ -218,13 +238,14 @@ __global__ void __launch_bounds__(kPrepThreads, NI <= 4 ? 3 : 1) delta_prepare_k
         const int par = p.s.d_parity[b.row] & 1;
         b.old = state + par * half; b.fresh = state + (par ^ 1) * half;
     }
-    const int v_jobs = (g.heads * g.vp + 127) / 128;
-    for (int job = warp; job < g.heads + v_jobs; job += kPrepThreads / 32) {
+    const int v_groups = (g.vp + 127) / 128;   // of 128 value columns of a head
+    for (int job = warp; job < g.heads * (1 + v_groups); job += kPrepThreads / 32) {
         if (job >= g.heads) {
+            const int h = (job - g.heads) / v_groups, c0 = (job - g.heads) % v_groups * 128 + lane;
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
-                const int e = (job - g.heads) * 128 + i * 32 + lane, h = e / g.vp, c = e % g.vp;
-                if (h >= g.heads) continue;
+                const int c = c0 + i * 32;
+                if (c >= g.vp) break;
                 float v[kBlock] = {0.f, 0.f, 0.f, 0.f};
                 if (c < g.vdim) conv_block<T, TAPS>(p, b, 2 * g.kv_heads * g.dim + h * g.vdim + c, g.v_off + h * g.vdim + c, true, v);
                 float* dst = p.w.v + ((size_t)blk * g.heads + h) * kBlock * g.vp + c;
@@ -542,7 +563,7 @@ constexpr int kDecThreads = 256, kDecWarps = 8;
 
 // Warp w holds the key channels w, w + 8, .. of 32 VEC columns at a time. dim <= 8 NR.
 template <typename T, int NR, int VEC>
-__global__ void __launch_bounds__(kDecThreads) delta_decode_kernel(const Params p) {
+__global__ void __launch_bounds__(kDecThreads, NR * VEC <= 64 ? 2 : 1) delta_decode_kernel(const Params p) {
     extern __shared__ __align__(16) float dd_smem[];
     __shared__ float sh_sum[3], sh_ss[kDecWarps];
     const Geo& g = p.g;
@@ -560,7 +581,7 @@ __global__ void __launch_bounds__(kDecThreads) delta_decode_kernel(const Params 
         const int c = cb + lane * VEC;
 #pragma unroll
         for (int i = 0; i < NR; ++i) {
-            const int d = warp + 8 * i;
+            const int d = warp + kDecWarps * i;
 #pragma unroll
             for (int e = 0; e < VEC; ++e) S[i][e] = 0.f;
             if (!fresh && d < g.dim && c < g.vdim) {
@@ -574,13 +595,14 @@ __global__ void __launch_bounds__(kDecThreads) delta_decode_kernel(const Params 
         }
     };
     load_state(0);   // travels while the vectors are prepared
+    const float beta_raw = ld(static_cast<const T*>(p.s.d_proj) + (size_t)row * g.row + g.beta_off + head);
+    for (int d = tid; d < g.dim; d += kDecThreads) gd[d] = decay_of(p, row, head, d);
     const bool own = head % g.group == 0;   // heads that share q and k: the first passes their convolution state on
     for (int i = tid; i < 2 * g.dim + g.vdim; i += kDecThreads) {
         if (i < g.dim) q[i] = conv_channel<T>(p, r, row, kvh * g.dim + i, g.q_off + kvh * g.dim + i, own);
         else if (i < 2 * g.dim) k[i - g.dim] = conv_channel<T>(p, r, row, g.kv_heads * g.dim + kvh * g.dim + i - g.dim, g.k_off + kvh * g.dim + i - g.dim, own);
         else v[i - 2 * g.dim] = conv_channel<T>(p, r, row, 2 * g.kv_heads * g.dim + head * g.vdim + i - 2 * g.dim, g.v_off + head * g.vdim + i - 2 * g.dim, true);
     }
-    for (int d = tid; d < g.dim; d += kDecThreads) gd[d] = decay_of(p, row, head, d);
     __syncthreads();
     if (warp < 3) {
         const float *a = warp == 1 ? k : q, *b = warp == 0 ? q : k;   // q.q, k.k, q.k
@@ -591,7 +613,7 @@ __global__ void __launch_bounds__(kDecThreads) delta_decode_kernel(const Params 
     }
     __syncthreads();
     const float qs = g.q_scale / sqrtf(sh_sum[0] + 1e-6f), ks = 1.f / sqrtf(sh_sum[1] + 1e-6f), qk = sh_sum[2] * qs * ks;
-    const float beta = sigmoid(ld(static_cast<const T*>(p.s.d_proj) + (size_t)row * g.row + g.beta_off + head));
+    const float beta = sigmoid(beta_raw);
     for (int cb = 0; cb < g.vdim; cb += CB) {
         if (cb > 0) load_state(cb);
         const int c = cb + lane * VEC;
@@ -600,7 +622,7 @@ __global__ void __launch_bounds__(kDecThreads) delta_decode_kernel(const Params 
         for (int e = 0; e < VEC; ++e) t1[e] = t2[e] = 0.f;
 #pragma unroll
         for (int i = 0; i < NR; ++i) {
-            const int d = warp + 8 * i;
+            const int d = warp + kDecWarps * i;
             if (d >= g.dim) break;
             const float gv = gd[d], kv = k[d] * ks, qv = q[d] * qs;
 #pragma unroll
@@ -632,7 +654,7 @@ __global__ void __launch_bounds__(kDecThreads) delta_decode_kernel(const Params 
                 }
 #pragma unroll
         for (int i = 0; i < NR; ++i) {
-            const int d = warp + 8 * i;
+            const int d = warp + kDecWarps * i;
             if (d >= g.dim || c >= g.vdim) break;
             const float kv = k[d] * ks;
             if constexpr (VEC == 4)
@@ -675,6 +697,8 @@ int launch_prepare(const Params& p, cudaStream_t s) {
 template <typename T, int NR, int VEC>
 int launch_decode(const Params& p, cudaStream_t s) {
     const size_t smem = ((size_t)3 * p.g.dp + 2 * p.g.vp + kDecWarps * 2 * 32 * VEC) * 4;
+    static PerDeviceOnce once;
+    if (once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(delta_decode_kernel<T, NR, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 64 * 1024));
     return launch_kernel(delta_decode_kernel<T, NR, VEC>, dim3((unsigned)p.g.heads, (unsigned)p.s.rows), dim3(kDecThreads), smem, s, 1, p);
 }
 template <typename T>

@@ -78,11 +78,25 @@ class NormStep(ctypes.Structure):
     ]
 
 
+class StreamStep(ctypes.Structure):
+    """gptrs_stream_step."""
+    _fields_ = [
+        ("d_x", ctypes.c_void_p), ("streams", ctypes.c_int), ("d_y", ctypes.c_void_p), ("y_dtype", ctypes.c_int), ("ldy", ctypes.c_int64),
+        ("d_pair", ctypes.c_void_p), ("d_pair_weight", ctypes.c_void_p), ("top", ctypes.c_int64), ("d_add", ctypes.c_void_p), ("ld_add", ctypes.c_int64),
+        ("d_embed", ctypes.c_void_p), ("embed_scale", ctypes.c_float), ("d_tokens", ctypes.c_void_p), ("vocab", ctypes.c_int64), ("d_mix", ctypes.c_void_p),
+        ("d_out", ctypes.c_void_p), ("d_in", ctypes.c_void_p), ("d_gamma_in", ctypes.c_void_p), ("eps", ctypes.c_float), ("d_rows", ctypes.c_void_p),
+        ("d_h", ctypes.c_void_p), ("h_dtype", ctypes.c_int), ("ldh", ctypes.c_int64), ("d_sum", ctypes.c_void_p), ("d_status", ctypes.c_void_p),
+        ("rows", ctypes.c_int64), ("dim", ctypes.c_int64),
+    ]
+
+
 class GroupedAttention(ctypes.Structure):
     """gptrs_grouped_attention."""
     _fields_ = [(n, ctypes.c_int) for n in ("dtype", "heads", "kv_heads", "dim", "vdim", "mask", "mask_size")] + \
         [("scale", ctypes.c_float), ("softcap", ctypes.c_float), ("distance_bias", ctypes.c_int)] + \
-        [(n, ctypes.c_int) for n in ("q_head_stride", "k_offset", "k_head_stride", "v_offset", "v_head_stride", "q_row", "out_head_stride")] + \
+        [(n, ctypes.c_int) for n in ("maps", "gate", "shared_kv")] + [(n, ctypes.c_float) for n in ("lambda_", "head_scale", "head_eps")] + \
+        [(n, ctypes.c_int) for n in ("q_head_stride", "k_offset", "k_head_stride", "v_offset", "v_head_stride", "q_row", "map_stride", "g_offset",
+                                     "g_head_stride", "out_head_stride")] + \
         [("page_bytes", ctypes.c_int64)]
 
 
@@ -103,7 +117,7 @@ class DeltaStep(ctypes.Structure):
 
 class Moe(ctypes.Structure):
     """gptrs_moe."""
-    _fields_ = [(n, ctypes.c_int) for n in ("experts", "top", "groups", "keep", "tile_rows")]
+    _fields_ = [(n, ctypes.c_int) for n in ("experts", "top", "groups", "keep", "tile_rows", "scores", "group_best")] + [("weight_scale", ctypes.c_float)]
 
 
 class ConvStep(ctypes.Structure):
@@ -121,7 +135,7 @@ class ConvStep(ctypes.Structure):
 class LatentAttention(ctypes.Structure):
     """gptrs_latent_attention."""
     _fields_ = [(n, ctypes.c_int) for n in ("dtype", "heads", "dim", "rot_dim", "vdim", "kv_rank", "window", "rot_dims")] + [("scale", ctypes.c_float)] + \
-        [(n, ctypes.c_int) for n in ("q_head_stride", "q_rot_offset", "dkv_offset", "rot_offset", "q_row", "qa_head_stride", "qa_rot_offset",
+        [(n, ctypes.c_int) for n in ("q_rank", "q_head_stride", "q_rot_offset", "dkv_offset", "rot_offset", "q_row", "kv_row", "q_latent_row", "qa_head_stride", "qa_rot_offset",
                                      "lat_head_stride", "out_head_stride")] + [("page_bytes", ctypes.c_int64)]
 
 

@@ -139,8 +139,8 @@ class CheckpointReader:
 
 
 # "architecture" of a model folder's config.json -> model kind of `engine_config`
-ARCHITECTURES = {"Bevosun": "bevosun", "Felepel": "felepel"}
-LAYERED_KINDS = ("bevosun", "felepel")   # kinds whose layers are configured one by one
+ARCHITECTURES = {"Bevosun": "bevosun", "Felepel": "felepel", "Kozapel": "kozapel"}
+LAYERED_KINDS = ("bevosun", "felepel", "kozapel")   # kinds whose layers are configured one by one
 
 
 class ModelFolder:
@@ -330,6 +330,8 @@ def engine_config(model_config: dict, weight_mode: int = gm.MODE_F32, shapes: di
         return bevosun_config(c, weight_mode=weight_mode, **engine_kw), None
     if kind == "felepel":
         return felepel_config(c, shapes, weight_mode=weight_mode, **engine_kw), None
+    if kind == "kozapel":
+        return kozapel_config(c, weight_mode=weight_mode, **engine_kw), None
     raise BackendError(2, f"model kind {kind!r} is not a decode model of this backend")
 
 
@@ -388,6 +390,37 @@ def felepel_config(c: dict, shapes: dict | None = None, context_length: int | No
     positions = int(c["max_positions"])
     return gm.ModelConfig.layered(layers, int(c["width"]), int(c["vocab"]), min(context_length or positions, positions), float(c["norm"]["eps"]),
                                   block=gm.BLOCK_SANDWICH, learned_positions=positions, **engine_kw)
+
+
+def kozapel_config(c: dict, context_length: int = 4096, **engine_kw) -> gm.ModelConfig:
+    """Kozapel's config object -> the layered kind. The design bounds no context: `context_length` is the caller's."""
+    layers = []
+    for i, layer in enumerate(c["layers"]):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        kw = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), scale=float(m["scale"]), mlp=gm.MLP_NONE)
+        mask = m.get("mask")
+        if layer["type"] == "latent_attention":
+            kw.update(mixer=gm.MIXER_LATENT_ATTENTION, rot_dim=int(m["rot_dim"]), kv_rank=int(m["kv_rank"]), q_rank=int(m["q_rank"]),
+                      rope_base=float(m["rot"]["base"]), rot_dims=int(m["rot"]["dims"]), window=int(mask["size"]) if mask else 0)
+        elif layer["type"] == "attention":
+            of = m.get("kv_from")
+            kw.update(mixer=gm.MIXER_GROUPED_ATTENTION, kv_heads=int(m["kv_heads"]), maps=2, out_gate=1, diff=float(m["diff"]),
+                      mask=gm.MASK_WINDOW if mask else gm.MASK_CAUSAL, mask_size=int(mask["size"]) if mask else 0, kv_from=-1 if of is None else int(of))
+        else:
+            raise BackendError(2, f"layer {i}: mixer {layer['type']!r} is not built")
+        if mlp and mlp["kind"] == "dense":
+            kw.update(mlp=gm.MLP_DENSE_GELU, d_ff=int(mlp["ff"]))
+        elif mlp and mlp["kind"] == "moe":
+            r = mlp["router"]
+            groups, shared = r.get("groups") or {"count": 1, "keep": 1}, mlp.get("shared")
+            kw.update(mlp=gm.MLP_EXPERTS, expert_form=gm.EXPERT_RELU2, d_ff=int(mlp["expert"]["ff"]), experts=int(r["experts"]), top=int(r["top"]),
+                      groups=int(groups["count"]), keep=int(groups["keep"]), route=gm.ROUTE_SIGMOID, group_best=2, correction=1,
+                      weight_scale=float(r["scale"]), shared_ff=int(shared["ff"]) if shared else 0)
+        elif mlp:
+            raise BackendError(2, f"layer {i}: feed-forward {mlp['kind']!r} is not built")
+        layers.append(gm.LayerConfig(**kw))
+    return gm.ModelConfig.layered(layers, int(c["width"]), int(c["vocab"]), context_length, float(c["norm"]["eps"]), block=gm.BLOCK_PRE_NORM,
+                                  streams=int(c.get("streams") or 0), embed_scale=float(c["embedding"]["scale"]), **engine_kw)
 
 
 def load_model(path, weight_mode: int = gm.MODE_F32, namespace: int | None = None, **engine_kw) -> gm.LoadedModel:

@@ -125,8 +125,10 @@ def cmd_export_random(args) -> int:
     for name, shape in cfg.param_shapes().items():
         if name.endswith("gamma") or "norm" in name.rsplit(".", 1)[-1]:
             tensors[name] = np.ones(shape, np.float32)
-        elif name.endswith(("beta", ".b", ".act")) or ".b_" in name:
+        elif name.endswith(("beta", ".b", ".act", ".correction")) or ".b_" in name:
             tensors[name] = np.zeros(shape, np.float32)
+        elif ".hc" in name:   # streams that stay as they are, read as their mean
+            tensors[name] = np.eye(*shape, dtype=np.float32) if len(shape) == 2 else np.full(shape, 1.0 / shape[0] if name.endswith(".in") else 1.0, np.float32)
         else:
             tensors[name] = (rng.standard_normal(size=shape, dtype=np.float32) * np.float32(args.std))
     ck.save(args.out, args.kind, config, tensors)
@@ -153,7 +155,7 @@ def main(argv=None) -> int:
     g.add_argument("--top-k", type=int, default=None)
     g.add_argument("--seed", type=int, default=0)
     g.add_argument("--weight-mode", default="f32", choices=["f32", "w4a16", "w8a16", "bf16"],
-                   help="w4a16 / w8a16 quantise the linear weights on the device while loading (ministral kind); bf16: the layered kinds, bevosun and felepel")
+                   help="w4a16 / w8a16 quantise the linear weights on the device while loading (ministral kind); bf16: the layered kinds, bevosun, felepel and kozapel")
     g.add_argument("--no-graph", action="store_true", help="launch kernels one by one instead of replaying a CUDA graph")
     g.set_defaults(fn=cmd_generate)
     i = sub.add_parser("inspect", help="print the config and tensor index of a checkpoint")
@@ -161,7 +163,7 @@ def main(argv=None) -> int:
     i.set_defaults(fn=cmd_inspect)
     x = sub.add_parser("export-random", help="write a checkpoint with random weights for a config")
     x.add_argument("--out", required=True)
-    x.add_argument("--kind", required=True, choices=["gpt", "ministral", "bevosun", "felepel"])
+    x.add_argument("--kind", required=True, choices=["gpt", "ministral", "bevosun", "felepel", "kozapel"])
     x.add_argument("--config", required=True, help="the model's config JSON object")
     x.add_argument("--seed", type=int, default=0)
     x.add_argument("--std", type=float, default=0.02)

@@ -36,6 +36,7 @@ struct RowsParams {
     const float* bias;
     int* status;
     DenseAct act;
+    int gate;                    // GPTRS_GATE_*
     int M, N, K, batch, out_f32;
     int m_tiles, n_tiles;
     int x_step, w_rows;          // x columns between batches; weight rows between batches
@@ -45,7 +46,7 @@ struct RowsParams {
 };
 
 constexpr int kRowsThreads = 384;    // warps 0-3 and 8-11 epilogue, 4 MMA + tensor memory, 5 loader
-// ACT: 0 none, 1 xIELU, 2 whatever p.act says (with a soft cap), 3 silu(gate) partner (8 gates, then their 8 partners).
+// ACT: 0 none, 1 xIELU, 2 whatever p.act says (with a soft cap), 3 act(gate) partner (8 gates, then their 8 partners), 4 squared relu.
 // GROUPED: the row tiles come from a list in device memory, each with the weight matrix that it meets.
 template <int BN, int STAGES, int ACT, bool GROUPED = false>
 __global__ void __launch_bounds__(kRowsThreads, 1) dense_rows_kernel(const __grid_constant__ RowsParams p) {
@@ -159,14 +160,19 @@ __global__ void __launch_bounds__(kRowsThreads, 1) dense_rows_kernel(const __gri
                 } else if constexpr (ACT == 2) {
 #pragma unroll
                     for (int i = 0; i < 32; ++i) v[i] = dense_act<true>(p.act, v[i]);
+                } else if constexpr (ACT == 4) {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) v[i] = dense_act<true>({2, 0.f, 0.f, 0.f}, v[i]);
                 }
                 if constexpr (ACT == 3) {
                     if (m < tl.m_end) {
                         float o[16];
+                        if (p.gate == GPTRS_GATE_GELU_TANH) {
 #pragma unroll
-                        for (int i = 0; i < 16; ++i) {
-                            const float gt = v[(i >> 3) * 16 + (i & 7)];
-                            o[i] = __fdividef(gt, 1.f + __expf(-gt)) * v[(i >> 3) * 16 + (i & 7) + 8];
+                            for (int i = 0; i < 16; ++i) o[i] = gelu_tanh_fast(v[(i >> 3) * 16 + (i & 7)]) * v[(i >> 3) * 16 + (i & 7) + 8];
+                        } else {
+#pragma unroll
+                            for (int i = 0; i < 16; ++i) o[i] = silu_fast(v[(i >> 3) * 16 + (i & 7)]) * v[(i >> 3) * 16 + (i & 7) + 8];
                         }
                         uint4* dst = reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(p.y) + row + ((n0 + c0) >> 1));
 #pragma unroll
@@ -359,18 +365,20 @@ int launch_rows(const Call& c, cudaStream_t st) {
     if (rc) return rc;
     p.y = c.y; p.bias = c.ep->d_bias; p.status = c.ep->d_status;
     p.act = {c.ep->act, c.ep->act_pos, c.ep->act_neg, c.ep->softcap};
+    p.gate = c.ep->swiglu;
     p.M = c.M; p.N = c.N; p.K = c.K; p.batch = c.batch; p.out_f32 = c.ep->out_dtype == GPTRS_F32;
     p.m_tiles = ceil_div(c.M, kTileM); p.n_tiles = ceil_div(c.N, BN);
     p.x_step = (int)c.x_step; p.w_rows = c.N; p.ldy = c.ldy; p.y_step = c.y_step;
     p.tiles = c.ep->d_tiles; p.n_row_tiles = c.ep->d_n_tiles;
     const int64_t tiles = (p.tiles ? c.ep->max_tiles : (int64_t)p.m_tiles * p.batch) * p.n_tiles;
     constexpr size_t smem = (size_t)STAGES * (kATile + BN * 128) + 1024;
-    void (*kerns[5])(RowsParams) = {dense_rows_kernel<BN, STAGES, 0>, dense_rows_kernel<BN, STAGES, 1>, dense_rows_kernel<BN, STAGES, 2>,
-                                    dense_rows_kernel<BN, STAGES, 0, true>, dense_rows_kernel<BN, STAGES, 3, true>};
+    void (*kerns[8])(RowsParams) = {dense_rows_kernel<BN, STAGES, 0>, dense_rows_kernel<BN, STAGES, 1>, dense_rows_kernel<BN, STAGES, 4>,
+                                    dense_rows_kernel<BN, STAGES, 2>, dense_rows_kernel<BN, STAGES, 3>, dense_rows_kernel<BN, STAGES, 0, true>,
+                                    dense_rows_kernel<BN, STAGES, 4, true>, dense_rows_kernel<BN, STAGES, 3, true>};
     static PerDeviceOnce attr_once;
     if (attr_once.first_time())
         for (auto k : kerns) GPTRS_CUDA_OK(cudaFuncSetAttribute(k, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    const auto kern = kerns[p.tiles ? (c.ep->swiglu ? 4 : 3) : c.ep->softcap > 0.f ? 2 : c.ep->act];
+    const auto kern = kerns[p.tiles ? (c.ep->swiglu ? 7 : c.ep->act == 2 ? 6 : 5) : c.ep->swiglu ? 4 : c.ep->softcap > 0.f ? 3 : c.ep->act];
     return launch_kernel(kern, dim3((unsigned)(tiles < sm_count() ? tiles : sm_count())), dim3(kRowsThreads), smem, st, 1, p);
 }
 
@@ -427,13 +435,15 @@ extern "C" int gptrs_cuda_dense_bf16(const void* d_x, const void* d_w, void* d_y
     GPTRS_REQUIRE(c.ldx >= k && c.ldy >= (ep->swiglu ? n / 2 : n) && c.ldx < (1ll << 30), "row strides shorter than the rows");
     GPTRS_REQUIRE((int64_t)c.batch * n < (1ll << 31) && (c.batch == 1 || ep->d_tiles || (c.x_step > 0 && c.y_step > 0)), "batch");
     GPTRS_REQUIRE(ep->out_dtype == GPTRS_BF16 || ep->out_dtype == GPTRS_F32, "out_dtype must be bf16 or f32");
-    GPTRS_REQUIRE(ep->act == 0 || ep->act == 1, "activation: 0 none, 1 xIELU");
+    GPTRS_REQUIRE(ep->act >= 0 && ep->act <= 2, "activation: 0 none, 1 xIELU, 2 squared relu");
     GPTRS_REQUIRE(!ep->d_best_val || (m <= 128 && c.batch == 1 && ep->out_dtype == GPTRS_F32 && ep->d_best_idx), "fused greedy head: up to 128 rows, f32");
-    GPTRS_REQUIRE(!ep->swiglu || (ep->d_tiles && ep->out_dtype == GPTRS_BF16 && n % 16 == 0 && c.ldy == n / 2), "swiglu: grouped form, compact bf16 output");
+    GPTRS_REQUIRE(!ep->swiglu || ((ep->swiglu == GPTRS_GATE_SILU || ep->swiglu == GPTRS_GATE_GELU_TANH) && ep->out_dtype == GPTRS_BF16 && n % 16 == 0 &&
+                                  c.ldy == n / 2 && (c.batch == 1 || ep->d_tiles) && !ep->d_bias && !ep->act && ep->softcap == 0.f && !ep->d_best_val),
+                  "gated output: compact bf16 rows, no other epilogue");
     if (m == 0) return GPTRS_OK;
     cudaStream_t st = as_stream(stream);
     if (ep->d_tiles) {
-        GPTRS_REQUIRE(ep->d_n_tiles && ep->max_tiles > 0 && !ep->d_bias && !ep->act && ep->softcap == 0.f && !ep->d_best_val, "grouped form: tile list, no other epilogue");
+        GPTRS_REQUIRE(ep->d_n_tiles && ep->max_tiles > 0 && !ep->d_bias && ep->act != 1 && ep->softcap == 0.f && !ep->d_best_val, "grouped form: tile list, squared relu or no activation");
         if (ep->tile_rows == 16) return launch_channels<16, 5>(c, st);
         if (ep->tile_rows == 32) return launch_channels<32, 5>(c, st);
         if (ep->tile_rows == 64) return launch_channels<64, 4>(c, st);

@@ -381,7 +381,8 @@ int gptrs_cuda_norm_matmul_f32(const float* d_x, int norm_kind, const float* d_g
 int gptrs_cuda_dense_f32(const float* d_x, const float* d_w, float* d_y, int64_t m, int64_t n, int64_t k, const gptrs_dense_epilogue* ep, void* stream) {
     GPTRS_REQUIRE(d_x && d_w && d_y && ep, "null pointer");
     GPTRS_REQUIRE(m >= 0 && n > 0 && k > 0 && n < (1ll << 31) && k < (1ll << 31) && m < (1ll << 31), "bad shape");
-    GPTRS_REQUIRE(ep->act == 0 || ep->act == 1, "activation: 0 none, 1 xIELU");
+    GPTRS_REQUIRE(ep->act >= 0 && ep->act <= 2, "activation: 0 none, 1 xIELU, 2 squared relu");
+    GPTRS_REQUIRE(!ep->swiglu, "gated outputs are a pass of their own in f32");
     GPTRS_REQUIRE(!ep->d_best_val, "the fused greedy head is part of the bf16 path");
     if (m == 0) return GPTRS_OK;
     SgemmParams p = {};
@@ -391,7 +392,7 @@ int gptrs_cuda_dense_f32(const float* d_x, const float* d_w, float* d_y, int64_t
     p.x_step = ep->x_step; p.y_step = ep->y_step;
     p.dense = {ep->act, ep->act_pos, ep->act_neg, ep->softcap};
     if (ep->d_tiles) {
-        GPTRS_REQUIRE(ep->d_n_tiles && ep->max_tiles > 0 && ep->tile_rows == 8 && !ep->d_bias && !ep->swiglu, "grouped form: tile list with tiles of 8 rows, no bias");
+        GPTRS_REQUIRE(ep->d_n_tiles && ep->max_tiles > 0 && ep->tile_rows == 8 && !ep->d_bias, "grouped form: tile list with tiles of 8 rows, no bias");
         p.tiles = ep->d_tiles; p.n_row_tiles = ep->d_n_tiles;
         p.x_step = p.y_step = 0;
         return launch_sgemm<8>(p, (int)ep->max_tiles, as_stream(stream));

@@ -69,12 +69,16 @@ struct DenseWeight {   // [batch][n][k] bf16 with n and k padded to 8, or [batch
 struct LayerWeights {
     Tensor *norm1 = nullptr, *norm2 = nullptr, *norm1b = nullptr, *norm2b = nullptr, *conv1 = nullptr, *conv2 = nullptr, *latent_norm = nullptr;
     Tensor *r1 = nullptr, *r2 = nullptr;                                                              // distance penalty
+    Tensor *q_norm = nullptr, *correction = nullptr;                                                  // query latent; experts' choice
+    struct Streams { Tensor *in = nullptr, *out = nullptr, *mix = nullptr; } streams[2];              // of the two sublayers
     Tensor *delta_conv = nullptr, *a_log = nullptr, *dt_bias = nullptr, *delta_norm = nullptr;        // delta rule
-    DenseWeight qkv, uk, uv, out, up, down, decay, gate, router;   // up: the experts' gates and ups too
+    DenseWeight qkv, uq, uk, uv, out, up, down, decay, gate, router, shared_up, shared_down;   // up: gates and ups of a gated layer or experts
     float act_pos = 0.f, act_neg = 0.f;
+    float lambda = 0.f;   // differential attention
     ~LayerWeights() {
-        for (Tensor* t : {norm1, norm2, norm1b, norm2b, conv1, conv2, latent_norm, r1, r2, delta_conv, a_log, dt_bias, delta_norm}) tensor_release(t);
-        for (DenseWeight* w : {&qkv, &uk, &uv, &out, &up, &down, &decay, &gate, &router}) { tensor_release(w->w); tensor_release(w->bias); }
+        for (Tensor* t : {norm1, norm2, norm1b, norm2b, conv1, conv2, latent_norm, r1, r2, q_norm, correction, delta_conv, a_log, dt_bias, delta_norm}) tensor_release(t);
+        for (Streams& s : streams) for (Tensor* t : {s.in, s.out, s.mix}) tensor_release(t);
+        for (DenseWeight* w : {&qkv, &uq, &uk, &uv, &out, &up, &down, &decay, &gate, &router, &shared_up, &shared_down}) { tensor_release(w->w); tensor_release(w->bias); }
     }
 };
 struct LayeredLayer {
@@ -90,6 +94,19 @@ struct LayeredLayer {
     int state1 = 0, state2 = 0;                      // convolution states of the two sublayers
     size_t delta_state_off = 0, delta_conv_off = 0;  // floats
     bool attends() const { return cfg.mixer != GPTRS_MIXER_CHANNEL_DELTA; }
+    // the first position that `pos` sees
+    int first_visible(int pos) const {
+        int f = 0;
+        if (cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION) f = att.window > 0 ? pos - att.window + 1 : 0;
+        else if (gatt.mask == GPTRS_MASK_WINDOW) f = pos - gatt.mask_size + 1;
+        else if (gatt.mask == GPTRS_MASK_CHUNK) f = pos / gatt.mask_size * gatt.mask_size;
+        return f > 0 ? f : 0;
+    }
+    // most positions that one sees, of a sequence of `len`
+    int span(int len) const {
+        const int size = cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION ? att.window : gatt.mask == GPTRS_MASK_CAUSAL ? 0 : gatt.mask_size;
+        return size > 0 ? size : len;
+    }
 };
 struct Layered {
     gptrs_layered_config cfg = {};
@@ -102,7 +119,7 @@ struct Layered {
     struct TileSet { int tokens = 1, n = 0; DevBuf row, rows; };
     std::vector<std::unique_ptr<TileSet>> tile_sets;
     int32_t* h_tiles = nullptr;   // pinned staging of one tile list (rows, then counts)
-    DevBuf x2, h, qkv, qa, lat, attn, up, y, logits_pad, state, scratch;
+    DevBuf x2, h, qkv, q, q_latent, qa, lat, attn, up, y, logits_pad, state, scratch;
     DevBuf d_run_first, d_run_last, d_parity, d_runs;
     DevBuf decay, gate, delta_state, delta_conv, delta_scratch;   // delta rule
     // experts: logits, sorted rows and what comes of them, the place of every (row, choice) among them, row tiles

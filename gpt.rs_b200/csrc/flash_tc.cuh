@@ -36,6 +36,10 @@ __device__ __forceinline__ int page_chunk(int t, int chunk, int nb) {
 // Tiles of up to 64 rows (decode steps of up to 64 heads) hold every row twice: rows 64 .. 127 repeat the queries, hence the
 // scores and the softmax, and put P_lo where the first copy puts P_hi, so that one product serves both terms; the two halves of
 // O are added at the end. Every wait is bounded (status 3).
+// Differential attention (TWO): two attentions of one head, with a query and a key part each, over the same values. A tile is 64 rows;
+// rows 0 .. 63 carry the first part of the queries, rows 64 .. 127 the second one, each with zeros in the columns of the other part, so
+// that one product with the whole key block gives the scores of both (an MMA of 64 rows would take as long as one of 128) and keys and
+// values are read once. At the end the halves of O meet in shared memory: difference, norm over the head, gate.
 constexpr int kRows = 128;
 constexpr int kKeys = 64;
 constexpr int kTcThreads = 224;
@@ -53,16 +57,31 @@ struct FlashShape {
     int steps[kMaxBlocks];             // 16-column steps of every query block that hold data
     int mask, mask_size;               // GPTRS_MASK_*
     int out_stride;                    // output elements of a head
+    int vdim;                          // of them data
+    int map_blocks;                    // query blocks of one part (query_blocks without a second one)
     uint32_t block_bytes;              // (page, kv head): 16 rows
     long long page_bytes;
 };
+// What happens to the output of a head behind the softmax.
+struct HeadOutput {
+    float lambda, scale, eps;          // two parts: d = a1 - lambda a2, then d / sqrt(mean(d^2) + eps) scale
+    const __nv_bfloat16* gate;         // times sigmoid(gate[row][head][..]), or null
+    int gate_row, gate_stride;
+};
+// eight values times sigmoid of their gates
+__device__ __forceinline__ void apply_gate(const __nv_bfloat16* g, float (&v)[8]) {
+    const uint4 u = __ldg(reinterpret_cast<const uint4*>(g));
+    const float z[8] = {bf16_lo(u.x), bf16_hi(u.x), bf16_lo(u.y), bf16_hi(u.y), bf16_lo(u.z), bf16_hi(u.z), bf16_lo(u.w), bf16_hi(u.w)};
+#pragma unroll
+    for (int i = 0; i < 8; ++i) v[i] = __fdividef(v[i], 1.f + __expf(-z[i]));
+}
 // first key that position `pos` sees
 __device__ __forceinline__ int first_visible(int mask, int size, int pos) {
     return mask == GPTRS_MASK_WINDOW ? max(pos - size + 1, 0) : mask == GPTRS_MASK_CHUNK ? pos - pos % size : 0;
 }
 
 struct TcParams {
-    // queries, 128-byte swizzle. Latent: [64 columns][blocks][T x heads rows], boxes of 32 rows. Grouped: [dim][heads][T], a box
+    // queries, 128-byte swizzle. Latent: [64 columns][blocks][T x heads rows], boxes of 32 rows. Grouped: [dim][parts][heads][T], a box
     // holds the heads of a kv head for the tokens of a tile (q_map) or for one token (q_one)
     CUtensorMap q_map, q_one;
     FlashShape g;
@@ -78,11 +97,17 @@ struct TcParams {
     float scale_log2;                  // log2(e) scale; with a soft cap, 2 log2(e) scale / cap
     float cap_log2;                    // log2(e) cap, 0 = none
     const float *r1, *r2;              // distance penalty r1[h] ln(1 + r2[h] d), or null
+    HeadOutput head_out;
 };
 
 __device__ __forceinline__ void tma_3d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, uint32_t bar) {
     asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];\n" ::"r"(dst), "l"(map),
                  "r"(x), "r"(y), "r"(z), "r"(bar)
+                 : "memory");
+}
+__device__ __forceinline__ void tma_4d(uint32_t dst, const CUtensorMap* map, int x, int y, int z, int w, uint32_t bar) {
+    asm volatile("cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4, %5}], [%6];\n" ::"r"(dst), "l"(map),
+                 "r"(x), "r"(y), "r"(z), "r"(w), "r"(bar)
                  : "memory");
 }
 __device__ __forceinline__ uint64_t desc_k_major(uint32_t addr, uint32_t group_stride) {
@@ -192,9 +217,11 @@ __device__ __forceinline__ void score_log2(float (&s)[kKeys], float scale_log2, 
 // GROUPED: kv heads of their own, soft cap, distance penalty; otherwise one latent row for all heads
 // kScores 2: two CTAs share an SM (tensor memory, shared memory and registers for half of one each), so that the softmax of one runs
 // under the waits of the other.
-template <bool GROUPED, int kScores>
+// TWO: two query and key parts per head.
+template <bool GROUPED, int kScores, bool TWO = false>
 __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_kernel(const __grid_constant__ TcParams p) {
     constexpr uint32_t kOCol = kScores * kKeys;
+    constexpr int kTileRows = TWO ? kRows / 2 : kRows;
     extern __shared__ unsigned char smem_raw[];
     __shared__ __align__(8) uint64_t k_full[kMaxStages], k_empty[kMaxStages], s_full[kScores], p_full[kScores], q_full;
     __shared__ uint32_t tmem_holder;
@@ -208,18 +235,26 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;\n" ::: "memory");
     }
     if (tid == 32 * 5) asm volatile("prefetch.tensormap [%0];\n" ::"l"(&p.q_map) : "memory");
+    if constexpr (TWO) {   // zeros in the columns of the other part; the copies of the queries fill the rest
+        for (int i = tid; i < g.query_blocks * (kRows / 2) * 8; i += kTcThreads) {
+            const int b = i / (kRows / 2 * 8), o = i % (kRows / 2 * 8);
+            st_shared_v4(sQ + (uint32_t)(b * kRows + (b < g.map_blocks ? kRows / 2 : 0)) * 128u + (uint32_t)o * 16u, 0, 0, 0, 0);
+        }
+        fence_proxy_async();
+    }
     pdl_wait();
     const int tile = (int)gridDim.x - 1 - (int)blockIdx.x;   // long contexts come last in a token list: start them first
     const int row0 = p.tile_row[tile], n_tok = p.tile_rows[tile], hb = blockIdx.z;
     const int kvh = GROUPED ? hb / p.head_blocks : 0, head_block = GROUPED ? hb % p.head_blocks : hb;
-    const int heads_n = min(p.rows_per_token, g.group - head_block * kRows);   // heads of this CTA per token
-    const int heads0 = kvh * g.group + head_block * kRows;
+    const int heads_n = min(p.rows_per_token, g.group - head_block * kTileRows);   // heads of this CTA per token
+    const int heads0 = kvh * g.group + head_block * kTileRows;
     const int live = n_tok * heads_n;
     const int live_warps = (live + 31) / 32;
-    const bool dup = live <= kRows / 2 && (!GROUPED || (n_tok == 1 && p.rows_per_token <= kRows / 2));   // a box of queries lands twice
+    const bool dup = !TWO && live <= kRows / 2 && (!GROUPED || (n_tok == 1 && p.rows_per_token <= kRows / 2));   // a box of queries lands twice
+    const bool halves = dup || TWO;   // rows 64 .. 127 belong to the same tokens and heads as rows 0 .. 63
     if (tid == 0) {
         for (int i = 0; i < p.stages; ++i) { mbar_init(&k_full[i], 1); mbar_init(&k_empty[i], 1); }
-        for (int i = 0; i < kScores; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], (uint32_t)live_warps * (dup ? 64 : 32)); }
+        for (int i = 0; i < kScores; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_full[i], (uint32_t)live_warps * (halves ? 64 : 32)); }
         mbar_init(&q_full, 1);
         mbar_fence_init();
     }
@@ -263,8 +298,13 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
                     mbar_expect_tx_addr(bar, (uint32_t)g.query_blocks * (one ? p.q_one_bytes * (dup ? 2u : 1u) : p.q_box_bytes));
                     for (int b = 0; b < g.query_blocks; ++b) {
                         const uint32_t dst = sQ + (uint32_t)(b * kRows) * 128u;
-                        tma_3d(dst, one ? &p.q_one : &p.q_map, b * 64, heads0, row0, bar);
-                        if (dup) tma_3d(dst + (kRows / 2) * 128u, &p.q_one, b * 64, heads0, row0, bar);
+                        if constexpr (TWO) {
+                            const int part = b >= g.map_blocks;
+                            tma_4d(dst + (uint32_t)(part * (kRows / 2)) * 128u, one ? &p.q_one : &p.q_map, (b - part * g.map_blocks) * 64, part, heads0, row0, bar);
+                        } else {
+                            tma_4d(dst, one ? &p.q_one : &p.q_map, b * 64, 0, heads0, row0, bar);
+                            if (dup) tma_4d(dst + (kRows / 2) * 128u, &p.q_one, b * 64, 0, heads0, row0, bar);
+                        }
                     }
                 } else {
                     mbar_expect_tx_addr(bar, (uint32_t)(live_warps * (dup ? 2 : 1) * g.query_blocks) * 4096u);
@@ -362,8 +402,8 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
         if (failed && lane == 0) atomicExch(p.status, 3);
     } else {
         // ================= warps 0-3: softmax, output ==============================================================================
-        const int r = dup ? tid & (kRows / 2 - 1) : tid;   // row of the tile
-        const bool lo_half = dup && warp >= 2;             // this copy of the row carries P_lo
+        const int r = halves ? tid & (kRows / 2 - 1) : tid;   // row of the tile
+        const bool lo_half = halves && warp >= 2;             // this copy of the row carries P_lo, or the second part
         int my_len = 0;
         if (r < live) {
             my_len = p.ctx_len[row0 + r / heads_n];
@@ -377,7 +417,7 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
         // between 2^-60 and 2^60
         const bool fixed = GROUPED && p.cap_log2 > 0.f && p.cap_log2 <= 60.f;
         float m_run = fixed ? 0.f : -1e30f, l_run = 0.f;
-        if ((dup ? warp & 1 : warp) < live_warps) {
+        if ((halves ? warp & 1 : warp) < live_warps) {
             for (int it = 0; it < n_blocks; ++it) {
                 const int buf = it % kScores;
                 if (!wait(&s_full[buf], (uint32_t)(it / kScores) & 1u)) break;
@@ -464,7 +504,51 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
             tc_fence_after();
             const int cols = g.value_blocks * 64;
             const bool any = n_blocks > 0 && !failed;
-            float* add = reinterpret_cast<float*>(smem_raw + (sK - smem_u32(smem_raw)));   // dup: the P_lo half of O, [row][cols + 4]; every page has been used
+            float* add = reinterpret_cast<float*>(smem_raw + (sK - smem_u32(smem_raw)));   // the other half of O, [row][cols + 4]; every page has been used
+            const HeadOutput& ho = p.head_out;
+            if (TWO && p.splits == 1) {
+                const float inv = any && l_run > 0.f ? 1.f / l_run : 0.f;
+                float4* mine = reinterpret_cast<float4*>(add + r * (cols + 4));
+                if (lo_half && any) {
+                    const float f = -ho.lambda * inv;
+#pragma unroll 1
+                    for (int c = 0; c < cols; c += 32) {
+                        float o[32];
+                        tmem_ld_32(t_lane + kOCol + (uint32_t)c, o);
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) mine[c / 4 + i] = make_float4(f * o[4 * i], f * o[4 * i + 1], f * o[4 * i + 2], f * o[4 * i + 3]);
+                    }
+                }
+                asm volatile("bar.sync 1, %0;\n" ::"r"(live_warps * 64) : "memory");
+                if (!lo_half && any) {
+                    float ss[4] = {0.f, 0.f, 0.f, 0.f};   // columns past vdim are zero
+#pragma unroll 1
+                    for (int c = 0; c < cols; c += 32) {
+                        float o[32];
+                        tmem_ld_32(t_lane + kOCol + (uint32_t)c, o);
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) {
+                            float4 v = mine[c / 4 + i];
+                            v.x = fmaf(o[4 * i], inv, v.x); v.y = fmaf(o[4 * i + 1], inv, v.y); v.z = fmaf(o[4 * i + 2], inv, v.z); v.w = fmaf(o[4 * i + 3], inv, v.w);
+                            ss[0] = fmaf(v.x, v.x, ss[0]); ss[1] = fmaf(v.y, v.y, ss[1]); ss[2] = fmaf(v.z, v.z, ss[2]); ss[3] = fmaf(v.w, v.w, ss[3]);
+                            mine[c / 4 + i] = v;
+                        }
+                    }
+                    const float f = ho.scale / sqrtf(((ss[0] + ss[1]) + (ss[2] + ss[3])) / (float)g.vdim + ho.eps);
+                    if (r < live) {
+                        const int row = row0 + r / heads_n, head = heads0 + r % heads_n;
+                        uint4* dst = reinterpret_cast<uint4*>(p.out + ((size_t)row * g.heads + head) * g.out_stride);
+                        const __nv_bfloat16* gate = ho.gate ? ho.gate + (size_t)row * ho.gate_row + (size_t)head * ho.gate_stride : nullptr;
+#pragma unroll 4
+                        for (int c = 0; c < g.out_stride; c += 8) {
+                            const float4 a = mine[c / 4], b = mine[c / 4 + 1];
+                            float v[8] = {a.x * f, a.y * f, a.z * f, a.w * f, b.x * f, b.y * f, b.z * f, b.w * f};
+                            if (gate) apply_gate(gate + c, v);
+                            dst[c / 8] = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+                        }
+                    }
+                }
+            }
             if (dup) {
                 if (lo_half && any)
 #pragma unroll 1
@@ -477,9 +561,9 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
                     }
                 asm volatile("bar.sync 1, %0;\n" ::"r"(live_warps * 64) : "memory");
             }
-            if (!lo_half) {
+            if (TWO ? p.splits > 1 : !lo_half) {
                 const size_t token_head = (size_t)(row0 + r / heads_n) * g.heads + heads0 + r % heads_n;
-                const size_t part = (((size_t)tile * gridDim.z + hb) * p.splits + blockIdx.y) * kRows + r;
+                const size_t part = (((size_t)tile * gridDim.z + hb) * p.splits + blockIdx.y) * kRows + (TWO ? tid : r);
                 if (p.splits > 1 && r < live) p.part_ml[part] = make_float2(m_run, failed ? 0.f : l_run);
                 const float inv = p.splits > 1 ? 1.f : l_run > 0.f ? 1.f / l_run : 0.f;
                 if (any)
@@ -496,13 +580,18 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
                             float4* dst = reinterpret_cast<float4*>(p.part_o + part * cols + c);
 #pragma unroll
                             for (int i = 0; i < 8; ++i) dst[i] = make_float4(o[4 * i], o[4 * i + 1], o[4 * i + 2], o[4 * i + 3]);
-                        } else if (r < live) {
+                        } else if (!TWO && r < live) {
                             uint4* dst = reinterpret_cast<uint4*>(p.out + token_head * g.out_stride + c);
+                            const __nv_bfloat16* gate = GROUPED && ho.gate ? ho.gate + (size_t)(row0 + r / heads_n) * ho.gate_row + (size_t)(heads0 + r % heads_n) * ho.gate_stride + c : nullptr;
 #pragma unroll
                             for (int i = 0; i < 4; ++i)
-                                if (c + 8 * i < g.out_stride)
-                                    dst[i] = make_uint4(pack_bf16x2(o[8 * i] * inv, o[8 * i + 1] * inv), pack_bf16x2(o[8 * i + 2] * inv, o[8 * i + 3] * inv),
-                                                        pack_bf16x2(o[8 * i + 4] * inv, o[8 * i + 5] * inv), pack_bf16x2(o[8 * i + 6] * inv, o[8 * i + 7] * inv));
+                                if (c + 8 * i < g.out_stride) {
+                                    float v[8];
+#pragma unroll
+                                    for (int e = 0; e < 8; ++e) v[e] = o[8 * i + e] * inv;
+                                    if (GROUPED && gate) apply_gate(gate + 8 * i, v);
+                                    dst[i] = make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+                                }
                         }
                     }
             }
@@ -514,39 +603,72 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
     if (warp == 4) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;\n" ::"r"(tmem), "r"(p.tmem_cols) : "memory");
 }
 
-// One warp per (row of a tile): out = sum_s 2^(m_s - m) O_s / sum_s 2^(m_s - m) l_s
+// One warp per (row of a tile): out = sum_s 2^(m_s - m) O_s / sum_s 2^(m_s - m) l_s, of both parts where there are two
 struct CombineParams {
     const float* part_o;
     const float2* part_ml;
     const int *tile_row, *tile_rows;
     __nv_bfloat16* out;
-    int heads, group, rows_per_token, head_blocks, splits, cols, out_stride;
+    int heads, group, rows_per_token, head_blocks, splits, cols, out_stride, vdim;
+    HeadOutput head_out;
 };
+template <bool TWO>
 __global__ void __launch_bounds__(128) flash_combine_kernel(const CombineParams p) {
+    constexpr int kTileRows = TWO ? kRows / 2 : kRows, kParts = TWO ? 2 : 1;
     pdl_launch_dependents();
     pdl_wait();
     const int tile = blockIdx.x, hb = blockIdx.z, r = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     const int kvh = hb / p.head_blocks, head_block = hb % p.head_blocks;
-    const int heads_n = min(p.rows_per_token, p.group - head_block * kRows), heads0 = kvh * p.group + head_block * kRows;
+    const int heads_n = min(p.rows_per_token, p.group - head_block * kTileRows), heads0 = kvh * p.group + head_block * kTileRows;
     if (r >= p.tile_rows[tile] * heads_n) return;
-    const size_t part = ((size_t)tile * gridDim.z + hb) * p.splits * kRows + r;
-    float m = -1e30f;
-    for (int s = 0; s < p.splits; ++s) m = fmaxf(m, p.part_ml[part + (size_t)s * kRows].x);
-    float l = 0.f;
-    for (int s = 0; s < p.splits; ++s) { const float2 v = p.part_ml[part + (size_t)s * kRows]; l += v.y * ex2f(v.x - m); }
-    const float inv = l > 0.f ? 1.f / l : 0.f;
-    __nv_bfloat16* dst = p.out + ((size_t)(p.tile_row[tile] + r / heads_n) * p.heads + heads0 + r % heads_n) * p.out_stride;
-    for (int c = lane * 2; c < p.out_stride; c += 64) {
-        float a = 0.f, b = 0.f;
+    const int row = p.tile_row[tile] + r / heads_n, head = heads0 + r % heads_n;
+    const HeadOutput& ho = p.head_out;
+    constexpr int kSteps = 4;   // 64-column steps: values of up to 256 columns
+    float2 acc[kSteps];
+#pragma unroll
+    for (int i = 0; i < kSteps; ++i) acc[i] = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int q = 0; q < kParts; ++q) {
+        const size_t part = ((size_t)tile * gridDim.z + hb) * p.splits * kRows + q * (kRows / 2) + r;
+        float m = -1e30f;
+        for (int s = 0; s < p.splits; ++s) m = fmaxf(m, p.part_ml[part + (size_t)s * kRows].x);
+        float l = 0.f;
+        for (int s = 0; s < p.splits; ++s) { const float2 v = p.part_ml[part + (size_t)s * kRows]; l += v.y * ex2f(v.x - m); }
+        const float inv = (l > 0.f ? 1.f / l : 0.f) * (q ? -ho.lambda : 1.f);
         for (int s = 0; s < p.splits; ++s) {
             const float2 v = p.part_ml[part + (size_t)s * kRows];
             if (v.y == 0.f) continue;   // a split without a visible key left no output
-            const float w = ex2f(v.x - m);
-            const float2 o = *reinterpret_cast<const float2*>(p.part_o + (part + (size_t)s * kRows) * p.cols + c);
-            a = fmaf(w, o.x, a);
-            b = fmaf(w, o.y, b);
+            const float w = ex2f(v.x - m) * inv;
+            const float* src = p.part_o + (part + (size_t)s * kRows) * p.cols + lane * 2;
+#pragma unroll
+            for (int i = 0; i < kSteps; ++i)
+                if (i * 64 < p.cols) {
+                    const float2 o = *reinterpret_cast<const float2*>(src + i * 64);
+                    acc[i].x = fmaf(w, o.x, acc[i].x);
+                    acc[i].y = fmaf(w, o.y, acc[i].y);
+                }
         }
-        *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(a * inv, b * inv);
+    }
+    float f = 1.f;
+    if (TWO) {
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < kSteps; ++i) ss = fmaf(acc[i].x, acc[i].x, fmaf(acc[i].y, acc[i].y, ss));
+        f = ho.scale / sqrtf(warp_sum(ss) / (float)p.vdim + ho.eps);
+    }
+    __nv_bfloat16* dst = p.out + ((size_t)row * p.heads + head) * p.out_stride;
+    const __nv_bfloat16* gate = ho.gate ? ho.gate + (size_t)row * ho.gate_row + (size_t)head * ho.gate_stride : nullptr;
+#pragma unroll
+    for (int i = 0; i < kSteps; ++i) {
+        const int c = i * 64 + lane * 2;
+        if (c >= p.out_stride) break;
+        float a = acc[i].x * f, b = acc[i].y * f;
+        if (gate) {
+            const uint32_t z = __ldg(reinterpret_cast<const uint32_t*>(gate + c));
+            a = __fdividef(a, 1.f + __expf(-bf16_lo(z)));
+            b = __fdividef(b, 1.f + __expf(-bf16_hi(z)));
+        }
+        *reinterpret_cast<uint32_t*>(dst + c) = pack_bf16x2(a, b);
     }
 }
 
@@ -566,25 +688,26 @@ size_t tc_scratch_bytes(int64_t n_tiles, int z_blocks, int splits, int value_blo
 }
 
 // Launches the kernel and, with key splits, the merge. The caller has filled in everything but the fields set here.
-template <bool GROUPED, int kScores>
+template <bool GROUPED, int kScores, bool TWO = false>
 int launch_flash(TcParams& p, int64_t n_tiles, void* d_scratch, cudaStream_t st) {
+    constexpr int kTileRows = TWO ? kRows / 2 : kRows;
     const FlashShape& g = p.g;
     p.stages = tc_stages(g.query_blocks, g.blocks, kScores == 2 ? kHalfSmemKb : 220);
-    p.head_blocks = ceil_div(g.group, kRows);
-    p.rows_per_token = g.group < kRows ? g.group : kRows;
+    p.head_blocks = ceil_div(g.group, kTileRows);
+    p.rows_per_token = g.group < kTileRows ? g.group : kTileRows;
     p.tmem_cols = kScores * kKeys + g.value_blocks * 64 <= 256 ? 256 : 512;
     const int z = g.kv_heads * p.head_blocks;
     const size_t rows = (size_t)n_tiles * z * p.splits * kRows;
     p.part_o = static_cast<float*>(d_scratch);
     p.part_ml = reinterpret_cast<float2*>(p.part_o + rows * (g.value_blocks * 64));
     static PerDeviceOnce attr_once;
-    if (attr_once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(flash_tc_kernel<GROUPED, kScores>, cudaFuncAttributeMaxDynamicSharedMemorySize, 221 * 1024));
+    if (attr_once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(flash_tc_kernel<GROUPED, kScores, TWO>, cudaFuncAttributeMaxDynamicSharedMemorySize, 221 * 1024));
     const size_t smem = (size_t)g.query_blocks * kRows * 128 + (size_t)p.stages * g.blocks * kKeys * 128 + 1024;
-    int rc = launch_kernel(flash_tc_kernel<GROUPED, kScores>, dim3((unsigned)n_tiles, (unsigned)p.splits, (unsigned)z), dim3(kTcThreads), smem, st, 1, p);
+    int rc = launch_kernel(flash_tc_kernel<GROUPED, kScores, TWO>, dim3((unsigned)n_tiles, (unsigned)p.splits, (unsigned)z), dim3(kTcThreads), smem, st, 1, p);
     if (rc || p.splits == 1) return rc;
-    CombineParams c = {p.part_o, p.part_ml, p.tile_row, p.tile_rows, p.out, g.heads, g.group, p.rows_per_token, p.head_blocks, p.splits, g.value_blocks * 64, g.out_stride};
-    // 32 CTAs of four warps cover the 128 rows of a tile
-    return launch_kernel(flash_combine_kernel, dim3((unsigned)n_tiles, kRows / 4, (unsigned)z), dim3(128), 0, st, 1, c);
+    CombineParams c = {p.part_o, p.part_ml, p.tile_row, p.tile_rows, p.out, g.heads, g.group, p.rows_per_token, p.head_blocks, p.splits, g.value_blocks * 64, g.out_stride, g.vdim, p.head_out};
+    // CTAs of four warps cover the rows of a tile
+    return launch_kernel(flash_combine_kernel<TWO>, dim3((unsigned)n_tiles, kTileRows / 4, (unsigned)z), dim3(128), 0, st, 1, c);
 }
 
 }  // namespace

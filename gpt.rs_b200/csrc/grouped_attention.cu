@@ -5,11 +5,14 @@
 //   o_ih = softmax over the visible j . v_jg
 //
 // A mask says where the keys of position i begin: at 0, at i - size + 1 (window) or at the last multiple of size (chunks).
+// Differential attention gives every query and key head two parts, each a softmax attention of its own over the same values; the output
+// of a head is their difference a1 - lambda a2, brought to unit root mean square. An output gate multiplies by sigmoid(gate). A layer may
+// read keys and values that another layer has put into the cache.
 //   grouped_append_kernel       key / value part of a projection row -> the token's page
 //   grouped_attention_kernel    plain CUDA-core attention, f32 or bf16 cache, any sizes (the f32 path)
 //   flash_tc_kernel<true>       tcgen05 flash attention (flash_tc.cuh), bf16, prompts and decode steps alike
-// A page holds, kv head by kv head, 16 rows of [value | key]; in bf16 both parts are padded to whole 64-column blocks in the
-// layout of flash_tc.cuh, in f32 the rows are plain.
+// A page holds, kv head by kv head, 16 rows of [value | key] or [value | key part 1 | key part 2]; in bf16 all are padded to whole
+// 64-column blocks in the layout of flash_tc.cuh, in f32 the rows are plain.
 #include "flash_tc.cuh"
 
 namespace gptrs {
@@ -18,9 +21,10 @@ namespace {
 struct Shape {
     int heads, kv_heads, group, dim, vdim, mask, mask_size;
     int q_head_stride, k_off, k_head_stride, v_off, v_head_stride, q_row, out_stride;
-    int nb, nbv;            // 64-column blocks of a cache row (bf16); of them values
+    int maps, map_stride, g_off, g_head_stride;   // parts of a head; gate (g_head_stride 0: none)
+    int nb, nbv, nbk;       // 64-column blocks of a cache row (bf16); of them values; of one key part
     long long page_bytes, block_bytes;
-    float scale, softcap;
+    float scale, softcap, lambda, head_scale, head_eps;
 };
 Shape shape_of(const gptrs_grouped_attention& a) {
     Shape g = {};
@@ -28,10 +32,13 @@ Shape shape_of(const gptrs_grouped_attention& a) {
     g.mask = a.mask; g.mask_size = a.mask_size;
     g.q_head_stride = a.q_head_stride; g.k_off = a.k_offset; g.k_head_stride = a.k_head_stride; g.v_off = a.v_offset; g.v_head_stride = a.v_head_stride;
     g.q_row = a.q_row; g.out_stride = a.out_head_stride;
+    g.maps = a.maps > 1 ? a.maps : 1; g.map_stride = a.map_stride; g.g_off = a.g_offset; g.g_head_stride = a.g_head_stride;
     g.nbv = up(a.vdim, 64) / 64;
-    g.nb = g.nbv + up(a.dim, 64) / 64;
+    g.nbk = up(a.dim, 64) / 64;
+    g.nb = g.nbv + g.maps * g.nbk;
     g.page_bytes = a.page_bytes; g.block_bytes = a.page_bytes / a.kv_heads;
     g.scale = a.scale; g.softcap = a.softcap;
+    g.lambda = a.lambda_; g.head_scale = a.head_scale; g.head_eps = a.head_eps;
     return g;
 }
 
@@ -59,8 +66,9 @@ __global__ void __launch_bounds__(kAppendThreads) grouped_append_kernel(const Ap
         for (int j = tid; j < g.kv_heads * per_head; j += kAppendThreads) {
             const int h = j / per_head, c = j % per_head;
             const bool val = c < g.nbv * 8;
-            const int col = (val ? c : c - g.nbv * 8) * 8, n = val ? g.vdim : g.dim;
-            const __nv_bfloat16* s = src + (val ? g.v_off + h * g.v_head_stride : g.k_off + h * g.k_head_stride) + col;
+            const int kc = c - g.nbv * 8, part = val ? 0 : kc / (g.nbk * 8);
+            const int col = (val ? c : kc - part * g.nbk * 8) * 8, n = val ? g.vdim : g.dim;
+            const __nv_bfloat16* s = src + (val ? g.v_off + h * g.v_head_stride : g.k_off + h * g.k_head_stride + part * g.map_stride) + col;
             uint4 v = make_uint4(0, 0, 0, 0);
             if (col + 8 <= n) {
                 v = *reinterpret_cast<const uint4*>(s);
@@ -74,7 +82,7 @@ __global__ void __launch_bounds__(kAppendThreads) grouped_append_kernel(const Ap
         }
     } else {
         const float* src = static_cast<const float*>(p.qkv) + (size_t)row * g.q_row;
-        const int width = g.vdim + g.dim;
+        const int width = g.vdim + g.maps * g.dim;   // the parts of a key lie next to one another
         for (int j = tid; j < g.kv_heads * width; j += kAppendThreads) {
             const int h = j / width, c = j % width;
             reinterpret_cast<float*>(page + h * g.block_bytes)[(size_t)t * width + c] =
@@ -112,103 +120,127 @@ __global__ void __launch_bounds__(kPlainThreads) grouped_attention_kernel(const 
     int len = p.ctx_len[row];
     if (len < 0 || len > p.max_pages * kPageTok) { if (tid == 0) atomicExch(p.status, 2); len = len < 0 ? 0 : p.max_pages * kPageTok; }
     const int lo = first_visible(g.mask, g.mask_size, max(len - 1, 0));
-    const int kvh = head / g.group;
+    const int kvh = head / g.group, width = g.vdim + g.maps * g.dim;
     const int* pt = p.page_table + (size_t)p.slot[row] * p.max_pages;
-    const size_t qo = (size_t)row * g.q_row + (size_t)head * g.q_head_stride;
-    for (int c = tid; c < dim_pad; c += kPlainThreads) {
-        float v = 0.f;
-        if (c < g.dim) v = BF16 ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.qkv)[qo + c]) : static_cast<const float*>(p.qkv)[qo + c];
-        qs[c] = v;
-    }
-    __syncthreads();
     const float r1 = p.r1 ? p.r1[head] : 0.f, r2 = p.r1 ? p.r2[head] : 0.f;
-    float acc[kPlainCols];
-#pragma unroll
-    for (int i = 0; i < kPlainCols; ++i) acc[i] = 0.f;
-    float m = -INFINITY, l = 0.f;
-    for (int j0 = lo; j0 < len; j0 += kPlainThreads) {
-        const int n = min(kPlainThreads, len - j0);
-        float s = -INFINITY;
-        if (tid < n) {
-            const int j = j0 + tid;
-            const long long base = (long long)pt[j / kPageTok] * g.page_bytes + kvh * g.block_bytes;
-            s_row[tid] = base;
-            s = 0.f;
-            if constexpr (BF16) {
-                const unsigned char* pg = p.pool + base;
-                for (int k = 0; k < dim_pad / 8; ++k) {
-                    const uint4 u = __ldg(reinterpret_cast<const uint4*>(pg + page_chunk(j % kPageTok, g.nbv * 8 + k, g.nb)));
-                    const float* qk = qs + k * 8;
-                    s = fmaf(qk[0], bf16_lo(u.x), s); s = fmaf(qk[1], bf16_hi(u.x), s);
-                    s = fmaf(qk[2], bf16_lo(u.y), s); s = fmaf(qk[3], bf16_hi(u.y), s);
-                    s = fmaf(qk[4], bf16_lo(u.z), s); s = fmaf(qk[5], bf16_hi(u.z), s);
-                    s = fmaf(qk[6], bf16_lo(u.w), s); s = fmaf(qk[7], bf16_hi(u.w), s);
-                }
-            } else {
-                const float* kv = reinterpret_cast<const float*>(p.pool + base) + (size_t)(j % kPageTok) * (g.vdim + g.dim) + g.vdim;
-                for (int c = 0; c < g.dim; ++c) s = fmaf(qs[c], __ldg(kv + c), s);
-            }
-            s *= g.scale;
-            if (g.softcap > 0.f) s = g.softcap * tanhf(s / g.softcap);
-            if (p.r1) s -= r1 * log1pf(r2 * (float)(len - 1 - j));
+    float o[kPlainCols], acc[kPlainCols];
+    float m, l;
+    for (int part = 0; part < g.maps; ++part) {
+        const size_t qo = (size_t)row * g.q_row + (size_t)head * g.q_head_stride + (size_t)part * g.map_stride;
+        for (int c = tid; c < dim_pad; c += kPlainThreads) {
+            float v = 0.f;
+            if (c < g.dim) v = BF16 ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.qkv)[qo + c]) : static_cast<const float*>(p.qkv)[qo + c];
+            qs[c] = v;
         }
-        const float wm = warp_max(s);
-        if ((tid & 31) == 0) sh[tid >> 5] = wm;
         __syncthreads();
-        const float m_new = fmaxf(m, fmaxf(fmaxf(sh[0], sh[1]), fmaxf(sh[2], sh[3])));
-        const float e = tid < n ? expf(s - m_new) : 0.f;
-        ps[tid] = e;
-        const float ws = warp_sum(e);
-        if ((tid & 31) == 0) sh[4 + (tid >> 5)] = ws;
-        __syncthreads();
-        const float alpha = expf(m - m_new);   // 0 for the first round
-        l = l * alpha + ((sh[4] + sh[5]) + (sh[6] + sh[7]));
-        m = m_new;
+#pragma unroll
+        for (int i = 0; i < kPlainCols; ++i) acc[i] = 0.f;
+        m = -INFINITY; l = 0.f;
+        for (int j0 = lo; j0 < len; j0 += kPlainThreads) {
+            const int n = min(kPlainThreads, len - j0);
+            float s = -INFINITY;
+            if (tid < n) {
+                const int j = j0 + tid;
+                const long long base = (long long)pt[j / kPageTok] * g.page_bytes + kvh * g.block_bytes;
+                s_row[tid] = base;
+                s = 0.f;
+                if constexpr (BF16) {
+                    const unsigned char* pg = p.pool + base;
+                    for (int k = 0; k < dim_pad / 8; ++k) {
+                        const uint4 u = __ldg(reinterpret_cast<const uint4*>(pg + page_chunk(j % kPageTok, (g.nbv + part * g.nbk) * 8 + k, g.nb)));
+                        const float* qk = qs + k * 8;
+                        s = fmaf(qk[0], bf16_lo(u.x), s); s = fmaf(qk[1], bf16_hi(u.x), s);
+                        s = fmaf(qk[2], bf16_lo(u.y), s); s = fmaf(qk[3], bf16_hi(u.y), s);
+                        s = fmaf(qk[4], bf16_lo(u.z), s); s = fmaf(qk[5], bf16_hi(u.z), s);
+                        s = fmaf(qk[6], bf16_lo(u.w), s); s = fmaf(qk[7], bf16_hi(u.w), s);
+                    }
+                } else {
+                    const float* kv = reinterpret_cast<const float*>(p.pool + base) + (size_t)(j % kPageTok) * width + g.vdim + part * g.dim;
+                    for (int c = 0; c < g.dim; ++c) s = fmaf(qs[c], __ldg(kv + c), s);
+                }
+                s *= g.scale;
+                if (g.softcap > 0.f) s = g.softcap * tanhf(s / g.softcap);
+                if (p.r1) s -= r1 * log1pf(r2 * (float)(len - 1 - j));
+            }
+            const float wm = warp_max(s);
+            if ((tid & 31) == 0) sh[tid >> 5] = wm;
+            __syncthreads();
+            const float m_new = fmaxf(m, fmaxf(fmaxf(sh[0], sh[1]), fmaxf(sh[2], sh[3])));
+            const float e = tid < n ? expf(s - m_new) : 0.f;
+            ps[tid] = e;
+            const float ws = warp_sum(e);
+            if ((tid & 31) == 0) sh[4 + (tid >> 5)] = ws;
+            __syncthreads();
+            const float alpha = expf(m - m_new);   // 0 for the first round
+            l = l * alpha + ((sh[4] + sh[5]) + (sh[6] + sh[7]));
+            m = m_new;
+#pragma unroll
+            for (int i = 0; i < kPlainCols; ++i) {
+                const int c = tid + i * kPlainThreads;
+                if (c >= g.vdim) break;
+                float a = acc[i] * alpha;
+                for (int k = 0; k < n; ++k) {
+                    const int t = (j0 + k) % kPageTok;
+                    float v;
+                    if constexpr (BF16)
+                        v = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(p.pool + s_row[k] + page_chunk(t, c >> 3, g.nb) + (c & 7) * 2));
+                    else
+                        v = __ldg(reinterpret_cast<const float*>(p.pool + s_row[k]) + (size_t)t * width + c);
+                    a = fmaf(ps[k], v, a);
+                }
+                acc[i] = a;
+            }
+            __syncthreads();
+        }
+        const float inv = l > 0.f ? 1.f / l : 0.f;
 #pragma unroll
         for (int i = 0; i < kPlainCols; ++i) {
-            const int c = tid + i * kPlainThreads;
-            if (c >= g.vdim) break;
-            float a = acc[i] * alpha;
-            for (int k = 0; k < n; ++k) {
-                const int t = (j0 + k) % kPageTok;
-                float v;
-                if constexpr (BF16)
-                    v = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(p.pool + s_row[k] + page_chunk(t, c >> 3, g.nb) + (c & 7) * 2));
-                else
-                    v = __ldg(reinterpret_cast<const float*>(p.pool + s_row[k]) + (size_t)t * (g.vdim + g.dim) + c);
-                a = fmaf(ps[k], v, a);
-            }
-            acc[i] = a;
+            const float v = tid + i * kPlainThreads < g.vdim ? acc[i] * inv : 0.f;
+            o[i] = part == 0 ? v : fmaf(-g.lambda, v, o[i]);
         }
-        __syncthreads();
     }
-    const size_t oo = ((size_t)row * g.heads + head) * g.out_stride;
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    float f = 1.f;
+    if (g.maps > 1) {
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < kPlainCols; ++i) ss = fmaf(o[i], o[i], ss);
+        ss = warp_sum(ss);
+        __syncthreads();
+        if ((tid & 31) == 0) sh[tid >> 5] = ss;
+        __syncthreads();
+        f = g.head_scale / sqrtf(((sh[0] + sh[1]) + (sh[2] + sh[3])) / (float)g.vdim + g.head_eps);
+    }
+    const size_t oo = ((size_t)row * g.heads + head) * g.out_stride, go = (size_t)row * g.q_row + g.g_off + (size_t)head * g.g_head_stride;
 #pragma unroll
     for (int i = 0; i < kPlainCols; ++i) {
         const int c = tid + i * kPlainThreads;
         if (c >= g.out_stride) break;
-        const float v = c < g.vdim ? acc[i] * inv : 0.f;
+        float v = o[i] * f;
+        if (g.g_head_stride > 0 && c < g.vdim) {
+            const float z = BF16 ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.qkv)[go + c]) : static_cast<const float*>(p.qkv)[go + c];
+            v /= 1.f + expf(-z);
+        }
         if (BF16) static_cast<__nv_bfloat16*>(p.out)[oo + c] = __float2bfloat16_rn(v);
         else static_cast<float*>(p.out)[oo + c] = v;
     }
 }
 
-// queries [dim][heads][T] of projection rows; a box is 64 columns of `heads` heads of `tokens` tokens
+// queries [dim][parts][heads][T] of projection rows; a box is 64 columns of one part of `heads` heads of `tokens` tokens
 int encode_queries(const void* qkv, const Shape& g, int64_t n_tokens, int heads, int tokens, CUtensorMap* map) {
     EncodeTiledFn enc = encode_fn();
     if (!enc) return fail(GPTRS_EXECUTION, "cuTensorMapEncodeTiled is not available");
-    cuuint64_t dims[3] = {(cuuint64_t)g.q_head_stride, (cuuint64_t)g.heads, (cuuint64_t)n_tokens};
-    cuuint64_t strides[2] = {(cuuint64_t)g.q_head_stride * 2, (cuuint64_t)g.q_row * 2};
-    cuuint32_t box[3] = {64, (cuuint32_t)heads, (cuuint32_t)tokens};
-    cuuint32_t estr[3] = {1, 1, 1};
-    CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(qkv), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+    cuuint64_t dims[4] = {(cuuint64_t)g.map_stride, (cuuint64_t)g.maps, (cuuint64_t)g.heads, (cuuint64_t)n_tokens};
+    cuuint64_t strides[3] = {(cuuint64_t)g.map_stride * 2, (cuuint64_t)g.q_head_stride * 2, (cuuint64_t)g.q_row * 2};
+    cuuint32_t box[4] = {64, 1, (cuuint32_t)heads, (cuuint32_t)tokens};
+    cuuint32_t estr[4] = {1, 1, 1, 1};
+    CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(qkv), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                      CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     if (r != CUDA_SUCCESS) return fail(GPTRS_EXECUTION, "cuTensorMapEncodeTiled failed for grouped attention (" + std::to_string((int)r) + ")");
     return GPTRS_OK;
 }
 
-int tile_tokens(const Shape& g) { return g.group >= kRows ? 1 : kRows / g.group; }
+int tile_rows(const Shape& g) { return g.maps > 1 ? kRows / 2 : kRows; }   // rows of a tile that are (token, head) pairs of their own
+int tile_tokens(const Shape& g) { return g.group >= tile_rows(g) ? 1 : tile_rows(g) / g.group; }
 
 }  // namespace
 }  // namespace gptrs
@@ -224,14 +256,19 @@ int gptrs_cuda_grouped_layout(gptrs_grouped_attention* a) {
     GPTRS_REQUIRE(a->mask == GPTRS_MASK_CAUSAL || ((a->mask == GPTRS_MASK_WINDOW || a->mask == GPTRS_MASK_CHUNK) && a->mask_size > 0), "grouped attention: mask");
     GPTRS_REQUIRE(a->scale > 0.f && a->softcap >= 0.f, "grouped attention: the scale must be positive, the soft cap not negative");
     GPTRS_REQUIRE(a->dtype == GPTRS_F32 || a->dtype == GPTRS_BF16, "grouped attention: f32 or bf16");
+    GPTRS_REQUIRE(a->maps >= 0 && a->maps <= 2, "grouped attention: one or two parts of a head");
     if (a->vdim > kPlainThreads * kPlainCols || a->dim > 8192) return fail(GPTRS_UNIMPLEMENTED, "grouped attention: vdim above 1024 or dim above 8192");
     const bool bf16 = a->dtype == GPTRS_BF16;
-    a->q_head_stride = a->k_head_stride = bf16 ? up(a->dim, 8) : a->dim;
+    const int maps = a->maps > 1 ? a->maps : 1;
+    a->map_stride = bf16 ? up(a->dim, 8) : a->dim;
+    a->q_head_stride = a->k_head_stride = maps * a->map_stride;
     a->v_head_stride = a->out_head_stride = bf16 ? up(a->vdim, 8) : a->vdim;
     a->k_offset = a->heads * a->q_head_stride;
-    a->v_offset = a->k_offset + a->kv_heads * a->k_head_stride;
-    a->q_row = a->v_offset + a->kv_heads * a->v_head_stride;
-    a->page_bytes = (int64_t)a->kv_heads * kPageTok * (bf16 ? (up(a->dim, 64) + up(a->vdim, 64)) * 2 : (a->dim + a->vdim) * 4);
+    a->v_offset = a->k_offset + (a->shared_kv ? 0 : a->kv_heads * a->k_head_stride);
+    a->g_offset = a->v_offset + (a->shared_kv ? 0 : a->kv_heads * a->v_head_stride);
+    a->g_head_stride = a->gate ? a->out_head_stride : 0;
+    a->q_row = a->g_offset + a->heads * a->g_head_stride;
+    a->page_bytes = (int64_t)a->kv_heads * kPageTok * (bf16 ? (maps * up(a->dim, 64) + up(a->vdim, 64)) * 2 : (maps * a->dim + a->vdim) * 4);
     return GPTRS_OK;
 }
 
@@ -239,6 +276,7 @@ int gptrs_cuda_grouped_append(const gptrs_grouped_attention* a, const void* d_qk
                               const int32_t* d_page_table, int64_t max_pages, void* d_pool, int64_t n_tokens, void* stream) {
     GPTRS_REQUIRE(a && d_qkv && d_positions && d_slot && d_page_table && d_pool, "null pointer");
     GPTRS_REQUIRE(a->q_row > 0 && max_pages > 0, "grouped attention: layout not filled in");
+    GPTRS_REQUIRE(!a->shared_kv, "grouped attention: these rows hold no keys and values");
     if (n_tokens == 0) return GPTRS_OK;
     AppendParams p = {shape_of(*a), d_qkv, d_positions, d_slot, d_page_table, static_cast<unsigned char*>(d_pool), (int)max_pages};
     const dim3 grid((unsigned)n_tokens);
@@ -259,14 +297,15 @@ int gptrs_cuda_grouped_splits(const gptrs_grouped_attention* a, int64_t n_tiles,
     const int64_t span = max_ctx_len < limit ? max_ctx_len : limit;
     const int64_t blocks = (span + kPageTok - 1 + kKeys - 1) / kKeys;
     const Shape g = shape_of(*a);
-    int64_t s = (tc_fits_twice(g.nb - g.nbv, g.nbv, g.nb) ? 2 : 1) * sm_count() / (n_tiles * a->kv_heads * ceil_div(g.group, kRows));
+    int64_t s = (tc_fits_twice(g.nb - g.nbv, g.nbv, g.nb) ? 2 : 1) * sm_count() / (n_tiles * a->kv_heads * ceil_div(g.group, tile_rows(g)));
     if (s > blocks) s = blocks;
     return (int)(s < 1 ? 1 : s);
 }
 
 size_t gptrs_cuda_grouped_scratch_bytes(const gptrs_grouped_attention* a, int64_t n_tiles, int splits) {
     if (!a || splits <= 1) return 0;
-    return tc_scratch_bytes(n_tiles, a->kv_heads * ceil_div(a->heads / a->kv_heads, kRows), splits, up(a->vdim, 64) / 64);
+    const Shape g = shape_of(*a);
+    return tc_scratch_bytes(n_tiles, g.kv_heads * ceil_div(g.group, tile_rows(g)), splits, g.nbv);
 }
 
 int gptrs_cuda_grouped_attention(const gptrs_grouped_attention* a, const void* d_qkv, const void* d_pool, const int32_t* d_page_table, int64_t max_pages,
@@ -296,7 +335,7 @@ int gptrs_cuda_grouped_attention(const gptrs_grouped_attention* a, const void* d
     const size_t need = gptrs_cuda_grouped_scratch_bytes(a, n_tiles, splits);
     GPTRS_REQUIRE(need == 0 || (d_scratch && scratch_bytes >= need), "grouped attention: scratch too small");
     TcParams p = {};
-    const int box_heads = g.group < kRows ? g.group : kRows;
+    const int box_heads = g.group < tile_rows(g) ? g.group : tile_rows(g);
     int rc = encode_queries(d_qkv, g, n_tokens, box_heads, tokens, &p.q_map);
     if (!rc) rc = encode_queries(d_qkv, g, n_tokens, box_heads, 1, &p.q_one);
     if (rc) return rc;
@@ -305,9 +344,13 @@ int gptrs_cuda_grouped_attention(const gptrs_grouped_attention* a, const void* d
     FlashShape& f = p.g;
     f.heads = g.heads; f.kv_heads = g.kv_heads; f.group = g.group;
     f.blocks = g.nb; f.value_blocks = f.key_block = g.nbv; f.query_blocks = g.nb - g.nbv;
-    for (int b = 0; b < f.query_blocks; ++b) f.steps[b] = g.dim - b * 64 >= 64 ? 4 : (g.dim - b * 64 + 15) / 16;
+    f.map_blocks = g.nbk;
+    for (int b = 0; b < f.query_blocks; ++b) {
+        const int left = g.dim - b % g.nbk * 64;
+        f.steps[b] = left >= 64 ? 4 : (left + 15) / 16;
+    }
     f.mask = g.mask; f.mask_size = g.mask_size;
-    f.out_stride = g.out_stride;
+    f.out_stride = g.out_stride; f.vdim = g.vdim;
     f.page_bytes = g.page_bytes; f.block_bytes = (uint32_t)g.block_bytes;
     p.pool = static_cast<const unsigned char*>(d_pool);
     p.page_table = d_page_table; p.slot = d_slot; p.ctx_len = d_ctx_len; p.tile_row = d_tile_row; p.tile_rows = d_tile_rows;
@@ -317,7 +360,10 @@ int gptrs_cuda_grouped_attention(const gptrs_grouped_attention* a, const void* d
     p.r1 = r1; p.r2 = r2;
     p.scale_log2 = g.softcap > 0.f ? 2.f * kLog2e * g.scale / g.softcap : kLog2e * g.scale;
     p.cap_log2 = g.softcap > 0.f ? kLog2e * g.softcap : 0.f;
-    return tc_fits_twice(f.query_blocks, f.value_blocks, f.blocks) ? launch_flash<true, 2>(p, n_tiles, d_scratch, st) : launch_flash<true, 3>(p, n_tiles, d_scratch, st);
+    p.head_out = {g.lambda, g.head_scale, g.head_eps, g.g_head_stride > 0 ? static_cast<const __nv_bfloat16*>(d_qkv) + g.g_off : nullptr, g.q_row, g.g_head_stride};
+    const bool twice = tc_fits_twice(f.query_blocks, f.value_blocks, f.blocks);
+    if (g.maps > 1) return twice ? launch_flash<true, 2, true>(p, n_tiles, d_scratch, st) : launch_flash<true, 3, true>(p, n_tiles, d_scratch, st);
+    return twice ? launch_flash<true, 2>(p, n_tiles, d_scratch, st) : launch_flash<true, 3>(p, n_tiles, d_scratch, st);
 }
 
 }  // extern "C"

@@ -5,9 +5,10 @@
 //   score(i, j, h) = ((W_uk,h^T q_ih) . c_j + rot(q'_ih) . k'_j) * scale,      o_ih = W_uv,h (sum_j p_ijh c_j)
 //
 // so attention itself is multi-query attention with kv_rank + rot_dim key dimensions whose values are the first kv_rank of
-// them, over a sliding window (position i sees i - window + 1 .. i). The two absorbed products are batched matmuls in front
-// of and behind the kernels of this file:
-//   latent_append_kernel        norm of the latent, rotation of the shared key part and of the queries, page write
+// them, over a sliding window (position i sees i - window + 1 .. i) or all of 0 .. i. The two absorbed products are batched matmuls in
+// front of and behind the kernels of this file. Where queries come through a latent of their own, the first projection gives both
+// latents, and the kernel that writes the page also norms the query latent for the second projection:
+//   latent_append_kernel        norm of the latent(s), rotation of the shared key part and of the queries, page write
 //   latent_attention_kernel     plain CUDA-core attention, f32 or bf16 cache, any sizes (the f32 path)
 //   flash_tc_kernel             tcgen05 flash attention (flash_tc.cuh), bf16, prompts and decode steps alike, kv_rank up to 256
 //
@@ -22,15 +23,17 @@ namespace {
 
 struct Geometry {
     int heads, dim, rot, rank, window, rot_pairs;
-    int q_head_stride, dkv_off, rot_off, q_row;
+    int q_head_stride, dkv_off, rot_off, q_row, kv_row, q_rank, q_latent_row;
     int qa_head_stride, qa_rot_off, lat_stride;
     int nb, nbc;            // 64-column blocks of a cache row (bf16); of them latent
     long long page_bytes;
     float scale;
 };
+int window_of(const gptrs_latent_attention& a) { return a.window > 0 ? a.window : 1 << 30; }
 Geometry geometry(const gptrs_latent_attention& a) {
     Geometry g = {};
-    g.heads = a.heads; g.dim = a.dim; g.rot = a.rot_dim; g.rank = a.kv_rank; g.window = a.window; g.rot_pairs = a.rot_dims / 2;
+    g.heads = a.heads; g.dim = a.dim; g.rot = a.rot_dim; g.rank = a.kv_rank; g.window = window_of(a); g.rot_pairs = a.rot_dims / 2;
+    g.kv_row = a.kv_row; g.q_rank = a.q_rank; g.q_latent_row = a.q_latent_row;
     g.q_head_stride = a.q_head_stride; g.dkv_off = a.dkv_offset; g.rot_off = a.rot_offset; g.q_row = a.q_row;
     g.qa_head_stride = a.qa_head_stride; g.qa_rot_off = a.qa_rot_offset; g.lat_stride = a.lat_head_stride;
     g.nbc = up(a.kv_rank, 64) / 64;
@@ -42,9 +45,11 @@ Geometry geometry(const gptrs_latent_attention& a) {
 
 struct AppendParams {
     Geometry g;
-    const void* qkv;            // [T][q_row]
+    const void* kv;             // [T][kv_row]
+    const void* q;              // [T][q_row]
     const int *pos, *slot, *page_table;
-    const float* norm_w;        // [kv_rank]
+    const float *norm_w, *q_norm_w;   // [kv_rank], [q_rank]
+    void* q_latent;             // [T][q_latent_row]
     const float *cos_t, *sin_t; // [positions][rot_pairs]
     void* qa;                   // [T][heads][qa_head_stride]
     unsigned char* pool;
@@ -79,50 +84,75 @@ __device__ __forceinline__ uint4 pack8(const float (&v)[8]) {
     return make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
 }
 
-template <bool BF16>
+// KEYS: the page (and the query latent, where there is one); QUERIES: the rotated query parts. Both at once where one projection gives
+// everything.
+template <bool BF16, bool KEYS, bool QUERIES>
 __global__ void __launch_bounds__(kAppendThreads) latent_append_kernel(const AppendParams p) {
     using T = typename std::conditional<BF16, __nv_bfloat16, float>::type;
-    __shared__ float sh[kAppendThreads / 32];
+    __shared__ float2 sh[kAppendThreads / 32];
     const Geometry& g = p.g;
     const int row = blockIdx.x, tid = threadIdx.x;
     pdl_launch_dependents();
     pdl_wait();
-    const T* q = static_cast<const T*>(p.qkv) + (size_t)row * g.q_row;
-    const T* lat = q + g.dkv_off;
-    const T* kr = q + g.rot_off;
+    const T* kv = static_cast<const T*>(p.kv) + (size_t)row * g.kv_row;
+    const T* q = static_cast<const T*>(p.q) + (size_t)row * g.q_row;
+    const T* lat = kv + g.dkv_off;
+    const T* kr = kv + g.rot_off;
     const int pos = p.pos[row];
     const float* cs = p.cos_t + (size_t)pos * g.rot_pairs;
     const float* sn = p.sin_t + (size_t)pos * g.rot_pairs;
-    float ss = 0.f;
-    for (int c = tid; c < g.rank; c += kAppendThreads) { const float v = ld_val(lat + c); ss = fmaf(v, v, ss); }
-    ss = warp_sum(ss);
-    if ((tid & 31) == 0) sh[tid >> 5] = ss;
-    __syncthreads();
-    ss = 0.f;
-#pragma unroll
-    for (int w = 0; w < kAppendThreads / 32; ++w) ss += sh[w];
-    const float inv = 1.f / sqrtf(ss / (float)g.rank + p.eps);
-    unsigned char* page = p.pool + (size_t)p.page_table[(size_t)p.slot[row] * p.max_pages + pos / kPageTok] * g.page_bytes;
+    unsigned char* page = nullptr;
+    float inv = 0.f;
     const int t = pos % kPageTok;
+    if constexpr (KEYS) {
+        page = p.pool + (size_t)p.page_table[(size_t)p.slot[row] * p.max_pages + pos / kPageTok] * g.page_bytes;
+        const int q_rank = QUERIES ? 0 : g.q_rank;   // the query latent is at the start of the row
+        float ss = 0.f, qs = 0.f;
+        for (int c = tid; c < g.rank; c += kAppendThreads) { const float v = ld_val(lat + c); ss = fmaf(v, v, ss); }
+        for (int c = tid; c < q_rank; c += kAppendThreads) { const float v = ld_val(kv + c); qs = fmaf(v, v, qs); }
+        ss = warp_sum(ss);
+        if (!QUERIES) qs = warp_sum(qs);
+        if ((tid & 31) == 0) sh[tid >> 5] = make_float2(ss, qs);
+        __syncthreads();
+        ss = qs = 0.f;
+#pragma unroll
+        for (int w = 0; w < kAppendThreads / 32; ++w) { ss += sh[w].x; qs += sh[w].y; }
+        inv = 1.f / sqrtf(ss / (float)g.rank + p.eps);
+        if constexpr (!QUERIES) {
+            const float q_inv = 1.f / sqrtf(qs / (float)q_rank + p.eps);
+            T* ql = static_cast<T*>(p.q_latent) + (size_t)row * g.q_latent_row;
+            if constexpr (BF16) {
+                for (int c0 = tid * 8; c0 < g.q_latent_row; c0 += kAppendThreads * 8) {
+                    float v[8];
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) v[e] = c0 + e < q_rank ? ld_val(kv + c0 + e) * q_inv * p.q_norm_w[c0 + e] : 0.f;
+                    *reinterpret_cast<uint4*>(ql + c0) = pack8(v);
+                }
+            } else {
+                for (int c = tid; c < q_rank; c += kAppendThreads) ql[c] = ld_val(kv + c) * q_inv * p.q_norm_w[c];
+            }
+        }
+    }
     T* qa = static_cast<T*>(p.qa) + (size_t)row * g.heads * g.qa_head_stride;
     if constexpr (BF16) {
         const int rb = g.nb - g.nbc;   // blocks of the rotated part
-        for (int j = tid; j < g.nb * 8; j += kAppendThreads) {
-            float v[8];
-            if (j < g.nbc * 8) {
+        if constexpr (KEYS)
+            for (int j = tid; j < g.nb * 8; j += kAppendThreads) {
+                float v[8];
+                if (j < g.nbc * 8) {
 #pragma unroll
-                for (int e = 0; e < 8; ++e) {
-                    const int c = j * 8 + e;
-                    v[e] = c < g.rank ? ld_val(lat + c) * inv * p.norm_w[c] : 0.f;
+                    for (int e = 0; e < 8; ++e) {
+                        const int c = j * 8 + e;
+                        v[e] = c < g.rank ? ld_val(lat + c) * inv * p.norm_w[c] : 0.f;
+                    }
+                } else {
+                    rotated8(kr, j - g.nbc * 8, g.rot, g.rot_pairs, cs, sn, v);
                 }
-            } else {
-                rotated8(kr, j - g.nbc * 8, g.rot, g.rot_pairs, cs, sn, v);
+                *reinterpret_cast<uint4*>(page + page_chunk(t, j, g.nb)) = pack8(v);
             }
-            *reinterpret_cast<uint4*>(page + page_chunk(t, j, g.nb)) = pack8(v);
-        }
         // queries: the rotated part, and zeros in the columns between the absorbed part and it
         const int z0 = up(g.rank, 8) / 8, zn = g.nbc * 8 - z0, per_head = zn + rb * 8;
-        for (int j = tid; j < g.heads * per_head; j += kAppendThreads) {
+        for (int j = tid; QUERIES && j < g.heads * per_head; j += kAppendThreads) {
             const int h = j / per_head, e = j % per_head;
             float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
             int chunk = z0 + e;
@@ -133,16 +163,18 @@ __global__ void __launch_bounds__(kAppendThreads) latent_append_kernel(const App
             *reinterpret_cast<uint4*>(qa + (size_t)h * g.qa_head_stride + chunk * 8) = pack8(v);
         }
     } else {
-        float* dst = reinterpret_cast<float*>(page) + (size_t)t * (g.rank + g.rot);
-        for (int c = tid; c < g.rank; c += kAppendThreads) dst[c] = ld_val(lat + c) * inv * p.norm_w[c];
         auto rotate = [&](const T* src, float* out, int c) {
             const int i = c >> 1;
             float v = ld_val(src + c);
             if (i < g.rot_pairs) v = (c & 1) ? v * cs[i] + ld_val(src + c - 1) * sn[i] : v * cs[i] - ld_val(src + c + 1) * sn[i];
             out[c] = v;
         };
-        for (int c = tid; c < g.rot; c += kAppendThreads) rotate(kr, dst + g.rank, c);
-        for (int j = tid; j < g.heads * g.rot; j += kAppendThreads) {
+        if constexpr (KEYS) {
+            float* dst = reinterpret_cast<float*>(page) + (size_t)t * (g.rank + g.rot);
+            for (int c = tid; c < g.rank; c += kAppendThreads) dst[c] = ld_val(lat + c) * inv * p.norm_w[c];
+            for (int c = tid; c < g.rot; c += kAppendThreads) rotate(kr, dst + g.rank, c);
+        }
+        for (int j = tid; QUERIES && j < g.heads * g.rot; j += kAppendThreads) {
             const int h = j / g.rot, c = j % g.rot;
             rotate(q + h * g.q_head_stride + g.dim, reinterpret_cast<float*>(qa) + (size_t)h * g.qa_head_stride + g.qa_rot_off, c);
         }
@@ -264,6 +296,13 @@ int encode_queries(const void* qa, const Geometry& g, int64_t n_tokens, CUtensor
     return GPTRS_OK;
 }
 
+template <bool KEYS, bool QUERIES>
+int launch_append(const gptrs_latent_attention* a, const AppendParams& p, int64_t n_tokens, void* stream) {
+    const dim3 grid((unsigned)n_tokens);
+    return a->dtype == GPTRS_BF16 ? launch_kernel(latent_append_kernel<true, KEYS, QUERIES>, grid, dim3(kAppendThreads), 0, as_stream(stream), 1, p)
+                                  : launch_kernel(latent_append_kernel<false, KEYS, QUERIES>, grid, dim3(kAppendThreads), 0, as_stream(stream), 1, p);
+}
+
 bool fits(const Geometry& g) { return tc_fits(g.nb, g.nbc, g.nb); }
 
 }  // namespace
@@ -275,16 +314,17 @@ extern "C" {
 
 int gptrs_cuda_latent_layout(gptrs_latent_attention* a) {
     GPTRS_REQUIRE(a, "null pointer");
-    GPTRS_REQUIRE(a->heads > 0 && a->dim > 0 && a->rot_dim > 0 && a->vdim > 0 && a->kv_rank > 0 && a->window > 0, "latent attention: sizes must be positive");
+    GPTRS_REQUIRE(a->heads > 0 && a->dim > 0 && a->rot_dim > 0 && a->vdim > 0 && a->kv_rank > 0 && a->window >= 0 && a->q_rank >= 0, "latent attention: sizes must be positive");
     GPTRS_REQUIRE(a->rot_dims >= 0 && a->rot_dims <= a->rot_dim && a->rot_dims % 2 == 0, "latent attention: rotated dimensions");
     GPTRS_REQUIRE(a->scale > 0.f, "latent attention: the scale must be positive");
     GPTRS_REQUIRE(a->dtype == GPTRS_F32 || a->dtype == GPTRS_BF16, "latent attention: f32 or bf16");
     if (a->kv_rank > kPlainThreads * kPlainCols) return fail(GPTRS_UNIMPLEMENTED, "latent attention: kv_rank above 1024");
     if (a->dtype == GPTRS_F32) {
         a->q_head_stride = a->dim + a->rot_dim;
-        a->dkv_offset = a->heads * a->q_head_stride;
+        a->q_latent_row = a->q_rank;
+        a->dkv_offset = a->q_rank > 0 ? a->q_latent_row : a->heads * a->q_head_stride;
         a->rot_offset = a->dkv_offset + a->kv_rank;
-        a->q_row = a->rot_offset + a->rot_dim;
+        a->kv_row = a->rot_offset + a->rot_dim;
         a->q_rot_offset = a->dim;
         a->qa_head_stride = a->kv_rank + a->rot_dim;
         a->qa_rot_offset = a->kv_rank;
@@ -294,15 +334,17 @@ int gptrs_cuda_latent_layout(gptrs_latent_attention* a) {
     } else {
         a->q_rot_offset = up(a->dim, 8);
         a->q_head_stride = a->q_rot_offset + up(a->rot_dim, 8);
-        a->dkv_offset = a->heads * a->q_head_stride;
+        a->q_latent_row = up(a->q_rank, 8);
+        a->dkv_offset = a->q_rank > 0 ? a->q_latent_row : a->heads * a->q_head_stride;
         a->rot_offset = a->dkv_offset + up(a->kv_rank, 8);
-        a->q_row = a->rot_offset + up(a->rot_dim, 8);
+        a->kv_row = a->rot_offset + up(a->rot_dim, 8);
         a->qa_rot_offset = up(a->kv_rank, 64);
         a->qa_head_stride = a->qa_rot_offset + up(a->rot_dim, 64);
         a->lat_head_stride = up(a->kv_rank, 8);
         a->out_head_stride = up(a->vdim, 8);
         a->page_bytes = (int64_t)kPageTok * a->qa_head_stride * 2;
     }
+    a->q_row = a->q_rank > 0 ? a->heads * a->q_head_stride : a->kv_row;
     return GPTRS_OK;
 }
 
@@ -311,11 +353,34 @@ int gptrs_cuda_latent_append(const gptrs_latent_attention* a, const void* d_qkv,
                              void* d_qa, void* d_pool, int64_t n_tokens, void* stream) {
     GPTRS_REQUIRE(a && d_qkv && d_positions && d_slot && d_page_table && d_norm_w && d_qa && d_pool, "null pointer");
     GPTRS_REQUIRE(a->q_row > 0 && max_pages > 0 && (a->rot_dims == 0 || (d_cos && d_sin)), "latent attention: layout not filled in, or no rotation tables");
+    GPTRS_REQUIRE(a->q_rank == 0, "latent attention: queries with a latent of their own are appended in two steps");
     if (n_tokens == 0) return GPTRS_OK;
-    AppendParams p = {geometry(*a), d_qkv, d_positions, d_slot, d_page_table, d_norm_w, d_cos, d_sin, d_qa, static_cast<unsigned char*>(d_pool), (int)max_pages, eps};
-    const dim3 grid((unsigned)n_tokens);
-    return a->dtype == GPTRS_BF16 ? launch_kernel(latent_append_kernel<true>, grid, dim3(kAppendThreads), 0, as_stream(stream), 1, p)
-                                  : launch_kernel(latent_append_kernel<false>, grid, dim3(kAppendThreads), 0, as_stream(stream), 1, p);
+    AppendParams p = {};
+    p.g = geometry(*a); p.kv = p.q = d_qkv; p.pos = d_positions; p.slot = d_slot; p.page_table = d_page_table; p.norm_w = d_norm_w; p.cos_t = d_cos; p.sin_t = d_sin;
+    p.qa = d_qa; p.pool = static_cast<unsigned char*>(d_pool); p.max_pages = (int)max_pages; p.eps = eps;
+    return launch_append<true, true>(a, p, n_tokens, stream);
+}
+
+int gptrs_cuda_latent_append_keys(const gptrs_latent_attention* a, const void* d_kv, const int32_t* d_positions, const int32_t* d_slot, const int32_t* d_page_table,
+                                  int64_t max_pages, const float* d_norm_w, const float* d_q_norm_w, float eps, const float* d_cos, const float* d_sin,
+                                  void* d_q_latent, void* d_pool, int64_t n_tokens, void* stream) {
+    GPTRS_REQUIRE(a && d_kv && d_positions && d_slot && d_page_table && d_norm_w && d_q_norm_w && d_q_latent && d_pool, "null pointer");
+    GPTRS_REQUIRE(a->q_rank > 0 && a->q_row > 0 && max_pages > 0 && (a->rot_dims == 0 || (d_cos && d_sin)), "latent attention: layout not filled in, or no rotation tables");
+    if (n_tokens == 0) return GPTRS_OK;
+    AppendParams p = {};
+    p.g = geometry(*a); p.kv = d_kv; p.pos = d_positions; p.slot = d_slot; p.page_table = d_page_table; p.norm_w = d_norm_w; p.q_norm_w = d_q_norm_w;
+    p.cos_t = d_cos; p.sin_t = d_sin; p.q_latent = d_q_latent; p.pool = static_cast<unsigned char*>(d_pool); p.max_pages = (int)max_pages; p.eps = eps;
+    return launch_append<true, false>(a, p, n_tokens, stream);
+}
+
+int gptrs_cuda_latent_rotate_queries(const gptrs_latent_attention* a, const void* d_q, const int32_t* d_positions, const float* d_cos, const float* d_sin, void* d_qa,
+                                     int64_t n_tokens, void* stream) {
+    GPTRS_REQUIRE(a && d_q && d_positions && d_qa, "null pointer");
+    GPTRS_REQUIRE(a->q_row > 0 && (a->rot_dims == 0 || (d_cos && d_sin)), "latent attention: layout not filled in, or no rotation tables");
+    if (n_tokens == 0) return GPTRS_OK;
+    AppendParams p = {};
+    p.g = geometry(*a); p.q = d_q; p.pos = d_positions; p.cos_t = d_cos; p.sin_t = d_sin; p.qa = d_qa;
+    return launch_append<false, true>(a, p, n_tokens, stream);
 }
 
 int gptrs_cuda_latent_tile_tokens(const gptrs_latent_attention* a) {
@@ -325,7 +390,7 @@ int gptrs_cuda_latent_tile_tokens(const gptrs_latent_attention* a) {
 
 int gptrs_cuda_latent_splits(const gptrs_latent_attention* a, int64_t n_tiles, int64_t max_ctx_len) {
     if (!a || n_tiles <= 0 || gptrs_cuda_latent_tile_tokens(a) == 0) return 1;
-    const int64_t span = (max_ctx_len < (int64_t)a->window + gptrs_cuda_latent_tile_tokens(a) ? max_ctx_len : (int64_t)a->window + gptrs_cuda_latent_tile_tokens(a));
+    const int64_t widest = (int64_t)window_of(*a) + gptrs_cuda_latent_tile_tokens(a), span = max_ctx_len < widest ? max_ctx_len : widest;
     const int64_t blocks = (span + kPageTok - 1 + kKeys - 1) / kKeys;
     int64_t s = sm_count() / (n_tiles * ceil_div(a->heads, kRows));
     if (s > blocks) s = blocks;

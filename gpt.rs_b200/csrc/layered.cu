@@ -1,8 +1,8 @@
 // Models whose layers are configured one by one (engine kind "layered"): weight packing, cache and state set-up and the forward
 // pass. A layer is a mixer (latent attention, latent_attention.cu; attention with grouped key / value heads, grouped_attention.cu; a
-// gated delta rule, delta_rule.cu) and an optional feed-forward (dense xIELU; a mixture of experts, moe_route.cu). The step between
-// two sublayers is post_norm_conv.cu (output norm, residual sum, short convolution with its per-sequence state) or norm_step.cu (norms
-// on both sides of a sublayer), the matmuls are dense_bf16.cu or, in f32 mode, dense_f32.cu. Slots, pages, graphs, sampling and the
+// gated delta rule, delta_rule.cu) and an optional feed-forward (dense xIELU or gated gelu; a mixture of experts, moe_route.cu). The step
+// between two sublayers is post_norm_conv.cu (output norm, residual sum, short convolution with its per-sequence state), norm_step.cu
+// (norms on both sides of a sublayer) or stream_step.cu (norms in front, several residual streams), the matmuls are dense_bf16.cu or, in f32 mode, dense_f32.cu. Slots, pages, graphs, sampling and the
 // generator are the engine's.
 #include <cmath>
 #include <cstdlib>
@@ -153,7 +153,7 @@ struct DenseOpts {
     const gptrs_row_tile* tiles = nullptr;
     const int32_t* n_tiles = nullptr;
     int64_t max_tiles = 0, tile_rows = 0;
-    bool swiglu = false;
+    int gate = 0;   // GPTRS_GATE_*
 };
 int dense(Model& m, const DenseWeight& w, const void* x, void* y, int64_t rows, const DenseOpts& o) {
     ++m.launches;
@@ -164,7 +164,7 @@ int dense(Model& m, const DenseWeight& w, const void* x, void* y, int64_t rows, 
     ep.ldx = o.ldx; ep.ldy = o.ldy; ep.batch = w.batch; ep.x_step = o.x_step; ep.y_step = o.y_step;
     if (o.pick) { ep.d_best_val = m.best_val.as<float>(); ep.d_best_idx = m.best_idx.as<int32_t>(); ep.skip_store = 1; }
     ep.d_status = m.d_status.as<int32_t>();
-    ep.d_tiles = o.tiles; ep.d_n_tiles = o.n_tiles; ep.max_tiles = o.max_tiles; ep.tile_rows = o.tile_rows; ep.swiglu = o.swiglu;
+    ep.d_tiles = o.tiles; ep.d_n_tiles = o.n_tiles; ep.max_tiles = o.max_tiles; ep.tile_rows = o.tile_rows; ep.swiglu = o.gate;
     if (m.f32())
         return gptrs_cuda_dense_f32(static_cast<const float*>(x), static_cast<const float*>(w.w->data), static_cast<float*>(y), rows, w.n, w.k, &ep, m.stream);
     return gptrs_cuda_dense_bf16(x, w.w->data, y, rows, w.n, w.k, &ep, m.stream);
@@ -182,8 +182,8 @@ int expert_tile_rows(const Model& m, const gptrs_moe& a, int64_t rows) {
 
 // what the buffers of a forward pass must hold, over all layers (elements per row unless said otherwise)
 struct Widths {
-    int64_t qkv = 0, qa = 0, lat = 0, attn = 0, up = 0, decay = 0, gate = 0;
-    int64_t delta_scratch = 0, router = 0, sorted = 0, expert_up = 0, expert_y = 0, top = 0, work = 0, row_tiles = 0;
+    int64_t qkv = 0, q = 0, q_latent = 0, qa = 0, lat = 0, attn = 0, up = 0, gate_up = 0, decay = 0, gate = 0;
+    int64_t delta_scratch = 0, router = 0, sorted = 0, expert_y = 0, top = 0, work = 0, row_tiles = 0;
     size_t pool = 0, delta_state = 0, delta_conv = 0;
     int n_state = 0;
 };
@@ -194,15 +194,38 @@ int build_latent(Model& m, LayeredLayer& L, const std::string& x, std::vector<st
     const int64_t W = m.cfg.d_model, H = a.heads, dim = a.dim, rot = a.rot_dim, rank = a.kv_rank, vd = a.vdim;
     int rc;
     if ((rc = get_raw(m, x + "dkv.norm", {rank}, &w.latent_norm))) return rc;
-    // queries and the down-projection in one weight, laid out as the attention kernels expect a projection row
-    if ((rc = pack_weight(m, {{x + "q", {H * (dim + rot), W}, {{H, dim, W, 0, (dim + rot) * W, W, 1, 0, a.q_head_stride, 0, 0, 0},
-                                                              {H, rot, W, dim * W, (dim + rot) * W, W, 1, a.q_rot_offset, a.q_head_stride, 0, 0, 0}}, ""},
+    // queries (or the query latent) and the down-projection in one weight, laid out as the attention kernels expect a projection row
+    auto queries = [&](const char* name, int64_t k) {
+        return Leaf{x + name, {H * (dim + rot), k}, {{H, dim, k, 0, (dim + rot) * k, k, 1, 0, a.q_head_stride, 0, 0, 0},
+                                                    {H, rot, k, dim * k, (dim + rot) * k, k, 1, a.q_rot_offset, a.q_head_stride, 0, 0, 0}}, ""};
+    };
+    if ((rc = pack_weight(m, {a.q_rank > 0 ? rows_of(x + "dq", a.q_rank, W, 0) : queries("q", W),
                               {x + "dkv", {rank + rot, W}, {{1, rank, W, 0, 0, W, 1, a.dkv_offset, 0, 0, 0, 0}, {1, rot, W, rank * W, 0, W, 1, a.rot_offset, 0, 0, 0, 0}}, ""}},
-                          1, a.q_row, W, "latent_qkv", &w.qkv, used))) return rc;
+                          1, a.kv_row, W, "latent_qkv", &w.qkv, used))) return rc;
+    if (a.q_rank > 0 && ((rc = get_raw(m, x + "dq.norm", {a.q_rank}, &w.q_norm)) || (rc = pack_weight(m, {queries("uq", a.q_rank)}, 1, a.q_row, a.q_rank, "latent_uq", &w.uq, used)))) return rc;
     // absorbed query: per head [rank] <- [dim], the stored key projection transposed
     if ((rc = pack_weight(m, {{x + "uk", {H * dim, rank}, {{H, rank, dim, 0, dim * rank, 1, rank, 0, 0, 0, 0, 1}}, ""}}, H, rank, dim, "latent_uk", &w.uk, used))) return rc;
     if ((rc = pack_weight(m, {{x + "uv", {H * vd, rank}, {{H, vd, rank, 0, vd * rank, rank, 1, 0, 0, 0, 0, 1}}, ""}}, H, vd, rank, "latent_uv", &w.uv, used))) return rc;
     return pack_weight(m, {{x + "o", {W, H * vd}, {{H, W, vd, 0, vd, H * vd, 1, 0, 0, 0, a.out_head_stride, 0}}, ""}}, 1, W, H * a.out_head_stride, "latent_o", &w.out, used);
+}
+
+// lambda of differential attention: exp(lq1 . lk1) - exp(lq2 . lk2) + diff
+int read_lambda(Model& m, const std::string& x, int64_t dim, float diff, float* lambda) {
+    std::vector<float> v[4];
+    const char* names[4] = {"lq1", "lk1", "lq2", "lk2"};
+    for (int i = 0; i < 4; ++i) {
+        Tensor* t = nullptr;
+        int rc = get_raw(m, x + names[i], {dim}, &t);
+        if (rc) return rc;
+        v[i].resize(dim);
+        const cudaError_t e = cudaMemcpy(v[i].data(), t->data, (size_t)dim * 4, cudaMemcpyDeviceToHost);
+        tensor_release(t);
+        GPTRS_CUDA_OK(e);
+    }
+    double s1 = 0., s2 = 0.;
+    for (int64_t i = 0; i < dim; ++i) { s1 += (double)v[0][i] * v[1][i]; s2 += (double)v[2][i] * v[3][i]; }
+    *lambda = (float)(std::exp(s1) - std::exp(s2) + diff);
+    return GPTRS_OK;
 }
 
 int build_grouped(Model& m, LayeredLayer& L, const std::string& x, std::vector<std::string>* used) {
@@ -212,8 +235,15 @@ int build_grouped(Model& m, LayeredLayer& L, const std::string& x, std::vector<s
     auto bias = [&](const char* n) { return L.cfg.proj_bias ? x + n + ".b" : std::string(); };
     int rc;
     if (a.distance_bias && ((rc = get_raw(m, x + "r1", {H}, &w.r1)) || (rc = get_raw(m, x + "r2", {H}, &w.r2)))) return rc;
-    if ((rc = pack_weight(m, {heads_of(x + "q", H, a.dim, W, 0, a.q_head_stride, bias("q")), heads_of(x + "k", G, a.dim, W, a.k_offset, a.k_head_stride, bias("k")),
-                              heads_of(x + "v", G, a.vdim, W, a.v_offset, a.v_head_stride, bias("v"))}, 1, a.q_row, W, "grouped_qkv", &w.qkv, used))) return rc;
+    const int64_t maps = a.maps > 1 ? a.maps : 1;
+    if (maps > 1 && (rc = read_lambda(m, x, a.dim, L.cfg.diff, &w.lambda))) return rc;
+    std::vector<Leaf> in = {heads_of(x + "q", H * maps, a.dim, W, 0, a.map_stride, bias("q"))};
+    if (!a.shared_kv) {
+        in.push_back(heads_of(x + "k", G * maps, a.dim, W, a.k_offset, a.map_stride, bias("k")));
+        in.push_back(heads_of(x + "v", G, a.vdim, W, a.v_offset, a.v_head_stride, bias("v")));
+    }
+    if (a.gate) in.push_back(heads_of(x + "g", H, a.vdim, W, a.g_offset, a.g_head_stride));
+    if ((rc = pack_weight(m, in, 1, a.q_row, W, "grouped_qkv", &w.qkv, used))) return rc;
     return pack_weight(m, {{x + "o", {W, H * a.vdim}, {{H, W, a.vdim, 0, a.vdim, H * a.vdim, 1, 0, 0, 0, a.out_head_stride, 0}}, ""}}, 1, W, H * a.out_head_stride, "heads_o", &w.out, used);
 }
 
@@ -255,44 +285,65 @@ int build_delta(Model& m, LayeredLayer& L, const std::string& x, std::vector<std
     return GPTRS_OK;
 }
 
+// gate and up of a gated feed-forward [F][W] as one matrix: 8 gates, then their 8 partners (matrix `mat` of a batch)
+void add_gated(std::vector<Leaf>* leaves, const std::string& x, int64_t F, int64_t W, int64_t mat) {
+    for (int part = 0; part < 2; ++part) {
+        const int64_t full = F / 8, rest = F % 8;
+        Leaf l = {x + (part ? "up" : "gate"), {F, W}, {{full, 8, W, 0, 8 * W, W, 1, part * 8, 16, 0, 0, 0, mat}}, ""};
+        if (rest) l.pieces.push_back({1, rest, W, full * 8 * W, 0, W, 1, full * 16 + part * 8, 0, 0, 0, 0, mat});
+        leaves->push_back(l);
+    }
+}
+
 int build_experts(Model& m, LayeredLayer& L, const std::string& x, std::vector<std::string>* used) {
     LayerWeights& w = *L.w;
-    const int64_t W = m.cfg.d_model, F = L.cfg.d_ff, Fp = pad8(F), E = L.moe.experts;
+    const bool gated = L.cfg.expert_form == GPTRS_EXPERT_SWIGLU;
+    const int64_t W = m.cfg.d_model, F = L.cfg.d_ff, Fp = pad8(F), E = L.moe.experts, S = L.cfg.shared_ff;
     std::vector<Leaf> up, down;
     for (int64_t e = 0; e < E; ++e) {
         const std::string n = x + "e" + std::to_string(e) + ".";
-        for (int part = 0; part < 2; ++part) {   // 8 gates, then their 8 partners
-            const int64_t full = F / 8, rest = F % 8;
-            Leaf l = {n + (part ? "up" : "gate"), {F, W}, {{full, 8, W, 0, 8 * W, W, 1, part * 8, 16, 0, 0, 0, e}}, ""};
-            if (rest) l.pieces.push_back({1, rest, W, full * 8 * W, 0, W, 1, full * 16 + part * 8, 0, 0, 0, 0, e});
-            up.push_back(l);
-        }
+        if (gated) add_gated(&up, n, F, W, e);
+        else up.push_back({n + "up", {F, W}, {{1, F, W, 0, 0, W, 1, 0, 0, 0, 0, 0, e}}, ""});
         down.push_back({n + "down", {W, F}, {{1, W, F, 0, 0, F, 1, 0, 0, 0, 0, 0, e}}, ""});
     }
     int rc;
-    if ((rc = pack_weight(m, up, E, 2 * Fp, W, "experts_up", &w.up, used)) || (rc = pack_weight(m, down, E, W, Fp, "experts_down", &w.down, used))) return rc;
+    if ((rc = pack_weight(m, up, E, gated ? 2 * Fp : F, W, "experts_up", &w.up, used)) ||
+        (rc = pack_weight(m, down, E, W, gated ? Fp : F, "experts_down", &w.down, used))) return rc;
+    if (S > 0 && ((rc = pack_plain(m, x + "shared.up", S, W, "", &w.shared_up, used)) || (rc = pack_plain(m, x + "shared.down", W, S, "", &w.shared_down, used)))) return rc;
+    if (L.cfg.correction && (rc = get_raw(m, x + "correction", {E}, &w.correction))) return rc;
     return pack_plain(m, x + "router", E, W, "", &w.router, used);
 }
 
+// what stands beside the norms of a sublayer (0: mixer, 1: feed-forward), depending on the block form
+int build_block(Model& m, LayerWeights& w, const std::string& p, int sub) {
+    const gptrs_layered_config& c = m.lay->cfg;
+    const int64_t W = m.cfg.d_model;
+    const std::string n = std::to_string(sub + 1);
+    int rc;
+    if ((rc = get_raw(m, p + "norm" + n, {W}, sub ? &w.norm2 : &w.norm1))) return rc;
+    if (c.block == GPTRS_BLOCK_SANDWICH) return get_raw(m, p + "norm" + n + "b", {W}, sub ? &w.norm2b : &w.norm1b);
+    if (c.block == GPTRS_BLOCK_OUTPUT_NORM) return get_raw(m, p + "canon" + n, {W, c.conv_taps}, sub ? &w.conv2 : &w.conv1);
+    if (c.streams == 0) return GPTRS_OK;
+    const std::string h = p + "hc" + n + ".";
+    LayerWeights::Streams& s = w.streams[sub];
+    if ((rc = get_raw(m, h + "in", {c.streams}, &s.in)) || (rc = get_raw(m, h + "out", {c.streams}, &s.out))) return rc;
+    return get_raw(m, h + "mix", {c.streams, c.streams}, &s.mix);
+}
+
 int build_weights(Model& m, LayeredLayer& L, int l, bool drop_leaves) {
-    const int64_t W = m.cfg.d_model, taps = m.lay->cfg.conv_taps;
-    const bool sandwich = m.lay->cfg.block == GPTRS_BLOCK_SANDWICH;
+    const int64_t W = m.cfg.d_model;
     const std::string p = "l" + std::to_string(l) + ".", x = p + "mix.", f = p + "mlp.";
     L.w = std::make_shared<LayerWeights>();
     LayerWeights& w = *L.w;
     std::vector<std::string> used;
     int rc;
-    if ((rc = get_raw(m, p + "norm1", {W}, &w.norm1))) return rc;
-    if ((rc = sandwich ? get_raw(m, p + "norm1b", {W}, &w.norm1b) : get_raw(m, p + "canon1", {W, taps}, &w.conv1))) return rc;
+    if ((rc = build_block(m, w, p, 0))) return rc;
     if (L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION) rc = build_latent(m, L, x, &used);
     else if (L.cfg.mixer == GPTRS_MIXER_GROUPED_ATTENTION) rc = build_grouped(m, L, x, &used);
     else rc = build_delta(m, L, x, &used);
     if (rc) return rc;
     if (L.cfg.mixer == GPTRS_MIXER_GROUPED_ATTENTION && L.cfg.proj_bias && (rc = add_bias(m, x + "o.b", W, &w.out))) return rc;
-    if (L.cfg.mlp != GPTRS_MLP_NONE) {
-        if ((rc = get_raw(m, p + "norm2", {W}, &w.norm2))) return rc;
-        if ((rc = sandwich ? get_raw(m, p + "norm2b", {W}, &w.norm2b) : get_raw(m, p + "canon2", {W, taps}, &w.conv2))) return rc;
-    }
+    if (L.cfg.mlp != GPTRS_MLP_NONE && (rc = build_block(m, w, p, 1))) return rc;
     if (L.cfg.mlp == GPTRS_MLP_DENSE_XIELU) {
         const int64_t F = L.cfg.d_ff;
         if ((rc = pack_plain(m, f + "up", F, W, f + "up.b", &w.up, &used)) || (rc = pack_plain(m, f + "down", W, F, f + "down.b", &w.down, &used))) return rc;
@@ -304,6 +355,12 @@ int build_weights(Model& m, LayeredLayer& L, int l, bool drop_leaves) {
         GPTRS_CUDA_OK(e);
         w.act_pos = softplus(v[0]);
         w.act_neg = 0.5f + softplus(v[1]);
+    } else if (L.cfg.mlp == GPTRS_MLP_DENSE_GELU) {
+        const int64_t F = L.cfg.d_ff;
+        std::vector<Leaf> up;
+        add_gated(&up, f, F, W, 0);
+        if ((rc = pack_weight(m, up, 1, 2 * pad8(F), W, "gated_up", &w.up, &used)) ||
+            (rc = pack_weight(m, {rows_of(f + "down", W, F, 0)}, 1, W, pad8(F), "gated_down", &w.down, &used))) return rc;
     } else if (L.cfg.mlp == GPTRS_MLP_EXPERTS) {
         if ((rc = build_experts(m, L, f, &used))) return rc;
     }
@@ -375,9 +432,14 @@ void count_widths(const Model& m, LayeredLayer& L, Widths* n) {
     if (L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION) {
         n->qa = std::max(n->qa, (int64_t)L.att.heads * L.att.qa_head_stride);
         n->lat = std::max(n->lat, (int64_t)L.att.heads * L.att.lat_head_stride);
+        if (L.att.q_rank > 0) {
+            n->q = std::max(n->q, (int64_t)L.att.q_row);
+            n->q_latent = std::max(n->q_latent, (int64_t)L.att.q_latent_row);
+        }
         n->pool += (size_t)c.kv_pages * L.att.page_bytes;
     } else if (L.cfg.mixer == GPTRS_MIXER_GROUPED_ATTENTION) {
-        n->pool += (size_t)c.kv_pages * L.gatt.page_bytes;
+        if (L.cfg.kv_from >= 0) L.pool_off = m.lay->layers[L.cfg.kv_from].pool_off;
+        else n->pool += (size_t)c.kv_pages * L.gatt.page_bytes;
     } else {
         n->decay = std::max(n->decay, (int64_t)L.delta.decay_row);
         n->gate = std::max(n->gate, (int64_t)L.delta.gate_row);
@@ -395,12 +457,18 @@ void count_widths(const Model& m, LayeredLayer& L, Widths* n) {
         if (L.cfg.mlp != GPTRS_MLP_NONE) L.state2 = n->n_state++;
     }
     if (L.cfg.mlp == GPTRS_MLP_DENSE_XIELU) n->up = std::max(n->up, w.up.n);
+    if (L.cfg.mlp == GPTRS_MLP_DENSE_GELU) {
+        n->up = std::max(n->up, w.up.n / 2);
+        n->gate_up = std::max(n->gate_up, w.up.n);
+    }
     if (L.cfg.mlp == GPTRS_MLP_EXPERTS) {
         const int64_t T = c.max_tokens, top = L.moe.top;
         n->top = std::max(n->top, top);
         n->router = std::max(n->router, w.router.n);
         n->sorted = std::max(n->sorted, top * w.up.k);
-        n->expert_up = std::max(n->expert_up, top * w.up.n);
+        const bool gated = L.cfg.expert_form == GPTRS_EXPERT_SWIGLU;
+        n->up = std::max({n->up, gated ? top * w.up.n / 2 : top * w.up.n, w.shared_up.n});
+        if (gated) n->gate_up = std::max(n->gate_up, top * w.up.n);
         n->expert_y = std::max(n->expert_y, top * w.down.n);
         n->work = std::max(n->work, gptrs_cuda_moe_work_ints(&L.moe, T));
         gptrs_moe smallest = L.moe;   // most tiles: the smallest tile that a launch of this many rows, or of one, may get
@@ -413,7 +481,8 @@ bool same_shape(const gptrs_layer_config& a, const gptrs_layer_config& b) {
     auto key = [](const gptrs_layer_config& c) {
         return std::make_tuple(std::make_tuple(c.mixer, c.heads, c.dim, c.rot_dim, c.rot_dims, c.vdim, c.kv_rank, c.window, c.scale, c.rope_base, c.mlp, c.d_ff),
                                std::make_tuple(c.kv_heads, c.mask, c.mask_size, c.distance_bias, c.proj_bias, c.softcap, c.taps, c.decay_rank, c.gate_rank),
-                               std::make_tuple(c.experts, c.top, c.groups, c.keep));
+                               std::make_tuple(c.experts, c.top, c.groups, c.keep, c.expert_form, c.shared_ff, c.route, c.group_best, c.correction, c.weight_scale),
+                               std::make_tuple(c.q_rank, c.maps, c.out_gate, c.kv_from, c.diff));
     };
     return key(a) == key(b);
 }
@@ -430,7 +499,9 @@ int layered_check_config(const gptrs_model_config& c) {
 
 int layered_set_layers(Model& m, const gptrs_layered_config& common, const gptrs_layer_config* layers) {
     const int n = m.cfg.n_layers;
-    GPTRS_REQUIRE(common.block == GPTRS_BLOCK_OUTPUT_NORM || common.block == GPTRS_BLOCK_SANDWICH, "unknown block form");
+    GPTRS_REQUIRE(common.block == GPTRS_BLOCK_OUTPUT_NORM || common.block == GPTRS_BLOCK_SANDWICH || common.block == GPTRS_BLOCK_PRE_NORM, "unknown block form");
+    GPTRS_REQUIRE(common.streams >= 0 && (common.streams == 0 || common.block == GPTRS_BLOCK_PRE_NORM), "residual streams: for the block form with norms in front");
+    if (common.streams > GPTRS_MAX_STREAMS) return fail(GPTRS_UNIMPLEMENTED, "more than 16 residual streams");
     GPTRS_REQUIRE(common.block != GPTRS_BLOCK_OUTPUT_NORM || (common.conv_taps >= 1 && common.conv_taps <= 16), "short convolutions of 1 to 16 taps");
     GPTRS_REQUIRE(common.learned_positions == 0 || (common.block == GPTRS_BLOCK_SANDWICH && common.learned_positions >= m.cfg.context_length),
                   "learned positions: for the block form with norms on both sides, one for every position of the context");
@@ -448,12 +519,20 @@ int layered_set_layers(Model& m, const gptrs_layered_config& common, const gptrs
         if (c.mixer == GPTRS_MIXER_LATENT_ATTENTION) {
             L.att.dtype = dtype;
             L.att.heads = c.heads; L.att.dim = c.dim; L.att.rot_dim = c.rot_dim; L.att.vdim = c.vdim; L.att.kv_rank = c.kv_rank;
-            L.att.window = c.window; L.att.rot_dims = c.rot_dims; L.att.scale = c.scale;
+            L.att.window = c.window; L.att.rot_dims = c.rot_dims; L.att.scale = c.scale; L.att.q_rank = c.q_rank;
             rc = gptrs_cuda_latent_layout(&L.att);
         } else if (c.mixer == GPTRS_MIXER_GROUPED_ATTENTION) {
             L.gatt.dtype = dtype;
             L.gatt.heads = c.heads; L.gatt.kv_heads = c.kv_heads; L.gatt.dim = c.dim; L.gatt.vdim = c.vdim; L.gatt.mask = c.mask; L.gatt.mask_size = c.mask_size;
             L.gatt.scale = c.scale; L.gatt.softcap = c.softcap; L.gatt.distance_bias = c.distance_bias;
+            L.gatt.maps = c.maps; L.gatt.gate = c.out_gate; L.gatt.shared_kv = c.kv_from >= 0;
+            L.gatt.head_scale = 1.f - c.diff; L.gatt.head_eps = m.cfg.norm_eps;
+            if (c.kv_from >= 0) {
+                GPTRS_REQUIRE(c.kv_from < l && !c.proj_bias, "kv_from names an earlier layer (projections without biases)");
+                const gptrs_layer_config& o = layers[c.kv_from];
+                GPTRS_REQUIRE(o.mixer == c.mixer && o.kv_from < 0 && o.kv_heads == c.kv_heads && o.dim == c.dim && o.vdim == c.vdim && std::max(o.maps, 1) == std::max(c.maps, 1),
+                              "kv_from names a layer with keys and values of its own and the same heads");
+            }
             rc = gptrs_cuda_grouped_layout(&L.gatt);
         } else if (c.mixer == GPTRS_MIXER_CHANNEL_DELTA) {
             L.delta.dtype = dtype;
@@ -465,12 +544,15 @@ int layered_set_layers(Model& m, const gptrs_layered_config& common, const gptrs
         }
         if (rc) return rc;
         if (c.mlp == GPTRS_MLP_EXPERTS) {
-            GPTRS_REQUIRE(common.block == GPTRS_BLOCK_SANDWICH, "experts: for the block form with norms on both sides");
-            L.moe = {c.experts, c.top, c.groups, c.keep, 16};
+            GPTRS_REQUIRE(common.block != GPTRS_BLOCK_OUTPUT_NORM, "experts: for the block forms with norms in front of the sublayers");
+            GPTRS_REQUIRE(c.shared_ff >= 0 && (c.shared_ff == 0 || (common.block == GPTRS_BLOCK_PRE_NORM && c.expert_form == GPTRS_EXPERT_RELU2)),
+                          "shared expert: of squared-relu form, for the block form with norms in front only");
+            GPTRS_REQUIRE(c.expert_form == GPTRS_EXPERT_SWIGLU || c.expert_form == GPTRS_EXPERT_RELU2, "unknown form of the experts");
+            L.moe = {c.experts, c.top, c.groups, c.keep, 16, c.route, c.group_best, c.weight_scale};
             GPTRS_REQUIRE(c.experts > 0 && c.top > 0 && c.groups > 0 && c.keep > 0 && c.experts % c.groups == 0 && c.keep <= c.groups &&
                               c.top <= c.keep * (c.experts / c.groups), "experts: groups must be equal and hold enough experts");
             if (c.experts > 1024) return fail(GPTRS_UNIMPLEMENTED, "experts: more than 1024");
-        } else if (c.mlp != GPTRS_MLP_NONE && c.mlp != GPTRS_MLP_DENSE_XIELU) {
+        } else if (c.mlp != GPTRS_MLP_NONE && c.mlp != GPTRS_MLP_DENSE_XIELU && c.mlp != GPTRS_MLP_DENSE_GELU) {
             return fail(GPTRS_UNIMPLEMENTED, "unknown feed-forward kind");
         }
     }
@@ -482,10 +564,11 @@ int layered_finalize(Model& m, bool drop_leaves) {
     const auto& c = m.cfg;
     GPTRS_REQUIRE(!y.layers.empty(), "call gptrs_cuda_model_set_layers before finalize");
     const int64_t W = c.d_model, V = c.vocab, taps = y.cfg.conv_taps;
-    const bool sandwich = y.cfg.block == GPTRS_BLOCK_SANDWICH;
+    const bool convs = y.cfg.block == GPTRS_BLOCK_OUTPUT_NORM;
+    const int64_t streams = std::max(y.cfg.streams, 1);
     int rc;
     if ((rc = get_raw(m, "embed", {V, W}, &m.tok_emb)) || (rc = get_raw(m, "final.norm", {W}, &m.final_g))) return rc;
-    if (!sandwich && (rc = get_raw(m, "embed.norm", {W}, &y.embed_norm))) return rc;
+    if (convs && (rc = get_raw(m, "embed.norm", {W}, &y.embed_norm))) return rc;
     if (y.cfg.learned_positions > 0 && (rc = get_raw(m, "pos", {y.cfg.learned_positions, W}, &m.pos_emb))) return rc;
     if ((rc = pack_plain(m, "head", V, W, "", &y.head))) return rc;
     const size_t act = m.f32() ? 4 : 2;
@@ -498,6 +581,7 @@ int layered_finalize(Model& m, bool drop_leaves) {
             GPTRS_REQUIRE(same_shape(L.cfg, y.layers[L.cfg.weights_of].cfg), "a layer that reuses another one's weights has an equal configuration");
             L.w = y.layers[L.cfg.weights_of].w;
         }
+        L.gatt.lambda_ = L.w->lambda;
         count_widths(m, L, &n);
         if (L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION && (rc = add_rope(m, L))) return rc;
         if (L.attends() && (rc = add_tiles(m, L))) return rc;
@@ -508,13 +592,14 @@ int layered_finalize(Model& m, bool drop_leaves) {
     }
     // activations (zeroed: padding columns that no kernel writes are multiplied by zero weights and must be finite)
     const size_t T = c.max_tokens, Wp = m.f32() ? W : pad8(W), Vp = y.head.n, rows = m.max_rows();
-    if ((rc = m.hidden.alloc(T * W * 4, true)) || (rc = y.x2.alloc(sandwich ? 0 : T * W * 4, true)) || (rc = y.h.alloc(T * Wp * act, true)) ||
-        (rc = y.y.alloc(T * Wp * act, true)) || (rc = y.qkv.alloc(T * n.qkv * act, true)) || (rc = y.qa.alloc(T * n.qa * act, true)) ||
-        (rc = y.lat.alloc(T * n.lat * act, true)) || (rc = y.attn.alloc(T * n.attn * act, true)) || (rc = y.up.alloc(T * std::max(n.up, n.expert_up / 2) * act, true)) ||
+    if ((rc = m.hidden.alloc(T * streams * W * 4, true)) || (rc = y.x2.alloc(convs ? T * W * 4 : 0, true)) || (rc = y.h.alloc(T * Wp * act, true)) ||
+        (rc = y.y.alloc(T * Wp * act, true)) || (rc = y.qkv.alloc(T * n.qkv * act, true)) || (rc = y.q.alloc(T * n.q * act, true)) ||
+        (rc = y.q_latent.alloc(T * n.q_latent * act, true)) || (rc = y.qa.alloc(T * n.qa * act, true)) ||
+        (rc = y.lat.alloc(T * n.lat * act, true)) || (rc = y.attn.alloc(T * n.attn * act, true)) || (rc = y.up.alloc(T * n.up * act, true)) ||
         (rc = m.xn_rows.alloc(rows * Wp * act, true)) || (rc = m.logits.alloc(rows * V * 4, true))) return rc;
     if ((rc = y.decay.alloc(T * n.decay * 4, true)) || (rc = y.gate.alloc(T * n.gate * act, true)) || (rc = y.delta_scratch.alloc(n.delta_scratch * 4, true)) ||
         (rc = y.delta_state.alloc(n.delta_state * 4, true)) || (rc = y.delta_conv.alloc(n.delta_conv * 4, true))) return rc;
-    if ((rc = y.router.alloc(T * n.router * 4, true)) || (rc = y.sorted.alloc(T * n.sorted * act, true)) || (rc = y.gate_up.alloc(m.f32() ? T * n.expert_up * 4 : 0, true)) ||
+    if ((rc = y.router.alloc(T * n.router * 4, true)) || (rc = y.sorted.alloc(T * n.sorted * act, true)) || (rc = y.gate_up.alloc(m.f32() ? T * n.gate_up * 4 : 0, true)) ||
         (rc = y.expert_y.alloc(T * n.expert_y * act, true)) || (rc = y.pair.alloc(T * n.top * 4, true)) || (rc = y.pair_weight.alloc(T * n.top * 4, true)) ||
         (rc = y.row_tiles.alloc(n.row_tiles * sizeof(gptrs_row_tile), true)) || (rc = y.n_row_tiles.alloc(4, true)) || (rc = y.moe_work.alloc(n.work * 4, true))) return rc;
     if ((int64_t)Vp != V && (rc = y.logits_pad.alloc(rows * Vp * 4, true))) return rc;
@@ -523,7 +608,7 @@ int layered_finalize(Model& m, bool drop_leaves) {
         if ((rc = m.best_val.alloc(tiles * r * 4)) || (rc = m.best_idx.alloc(tiles * r * 4))) return rc;
         if (const char* e = getenv("GPTRS_FUSE_PICK")) m.fuse_pick = atoi(e) != 0;
     }
-    y.state_stride = sandwich ? 0 : (size_t)c.max_seqs * 2 * (taps - 1) * W;
+    y.state_stride = convs ? (size_t)c.max_seqs * 2 * (taps - 1) * W : 0;
     if ((rc = y.state.alloc(std::max<size_t>(1, (size_t)n.n_state * y.state_stride) * 4, true))) return rc;
     for (DevBuf* b : {&y.d_run_first, &y.d_run_last, &y.d_parity, &y.d_runs})
         if ((rc = b->alloc(T * 4, true))) return rc;
@@ -538,7 +623,7 @@ int layered_finalize(Model& m, bool drop_leaves) {
         if (L.tiles < 0) continue;
         if (L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION) scratch = std::max(scratch, gptrs_cuda_latent_scratch_bytes(&L.att, 1, sm_count() + 1));
         else {
-            const int per_split = L.gatt.kv_heads * ((L.gatt.heads / L.gatt.kv_heads + 127) / 128);
+            const int tile_rows = L.gatt.maps > 1 ? 64 : 128, per_split = L.gatt.kv_heads * ((L.gatt.heads / L.gatt.kv_heads + tile_rows - 1) / tile_rows);
             scratch = std::max(scratch, gptrs_cuda_grouped_scratch_bytes(&L.gatt, 1, 2 * sm_count() / per_split + 2));
         }
     }
@@ -629,12 +714,7 @@ int layered_stage_generator(Model& m, int batch) {
 int layered_first_visible(const Model& m, int pos) {
     int first = pos;
     for (const LayeredLayer& L : m.lay->layers) {
-        if (!L.attends()) continue;
-        int f = 0;
-        if (L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION) f = pos - L.att.window + 1;
-        else if (L.gatt.mask == GPTRS_MASK_WINDOW) f = pos - L.gatt.mask_size + 1;
-        else if (L.gatt.mask == GPTRS_MASK_CHUNK) f = pos / L.gatt.mask_size * L.gatt.mask_size;
-        first = std::min(first, std::max(f, 0));
+        if (L.attends()) first = std::min(first, L.first_visible(pos));
     }
     return first;
 }
@@ -643,9 +723,7 @@ int layered_first_visible(const Model& m, int pos) {
 int layered_graph_bucket(const Model& m, int bucket) {
     int widest = 1;
     for (const LayeredLayer& L : m.lay->layers) {
-        if (!L.attends()) continue;
-        const int span = L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION ? L.att.window : L.gatt.mask == GPTRS_MASK_CAUSAL ? bucket : L.gatt.mask_size;
-        widest = std::max(widest, span);
+        if (L.attends()) widest = std::max(widest, L.span(bucket));
     }
     return (int)std::min<int64_t>(bucket, ((int64_t)widest + 511) / 512 * 512);
 }
@@ -672,11 +750,21 @@ struct Pass {
         const Layered::Rope& rope = *y.ropes[L.rope];
         int rc;
         if ((rc = dense(m, w.qkv, y.h.p, y.qkv.p, T, {}))) return rc;
+        const bool two_steps = a.q_rank > 0;
+        const void* q = two_steps ? y.q.p : y.qkv.p;
+        if (two_steps) {
+            ++m.launches;
+            if ((rc = gptrs_cuda_latent_append_keys(&a, y.qkv.p, pos(), slot(), pages(), m.cfg.max_pages_per_seq, fp(w.latent_norm), fp(w.q_norm), m.cfg.norm_eps,
+                                                    rope.cos_t.as<float>(), rope.sin_t.as<float>(), y.q_latent.p, pool(L), T, st))) return rc;
+            if ((rc = dense(m, w.uq, y.q_latent.p, y.q.p, T, {}))) return rc;
+        }
         DenseOpts ok;
-        ok.ldx = w.qkv.n; ok.x_step = a.q_head_stride; ok.ldy = (int64_t)a.heads * a.qa_head_stride; ok.y_step = a.qa_head_stride;
-        if ((rc = dense(m, w.uk, y.qkv.p, y.qa.p, T, ok))) return rc;
+        ok.ldx = a.q_row; ok.x_step = a.q_head_stride; ok.ldy = (int64_t)a.heads * a.qa_head_stride; ok.y_step = a.qa_head_stride;
+        if ((rc = dense(m, w.uk, q, y.qa.p, T, ok))) return rc;
         ++m.launches;
-        if ((rc = gptrs_cuda_latent_append(&a, y.qkv.p, pos(), slot(), pages(), m.cfg.max_pages_per_seq, fp(w.latent_norm), m.cfg.norm_eps,
+        if (two_steps) {
+            if ((rc = gptrs_cuda_latent_rotate_queries(&a, q, pos(), rope.cos_t.as<float>(), rope.sin_t.as<float>(), y.qa.p, T, st))) return rc;
+        } else if ((rc = gptrs_cuda_latent_append(&a, y.qkv.p, pos(), slot(), pages(), m.cfg.max_pages_per_seq, fp(w.latent_norm), m.cfg.norm_eps,
                                            rope.cos_t.as<float>(), rope.sin_t.as<float>(), y.qa.p, pool(L), T, st))) return rc;
         const Layered::TileSet* t = L.tiles >= 0 ? y.tile_sets[L.tiles].get() : nullptr;
         const int splits = t ? gptrs_cuda_latent_splits(&a, t->n, max_ctx) : 1;
@@ -695,8 +783,8 @@ struct Pass {
         const LayerWeights& w = *L.w;
         int rc;
         if ((rc = dense(m, w.qkv, y.h.p, y.qkv.p, T, {}))) return rc;
-        ++m.launches;
-        if ((rc = gptrs_cuda_grouped_append(&a, y.qkv.p, pos(), slot(), pages(), m.cfg.max_pages_per_seq, pool(L), T, st))) return rc;
+        if (!a.shared_kv) ++m.launches;
+        if (!a.shared_kv && (rc = gptrs_cuda_grouped_append(&a, y.qkv.p, pos(), slot(), pages(), m.cfg.max_pages_per_seq, pool(L), T, st))) return rc;
         const Layered::TileSet* t = L.tiles >= 0 ? y.tile_sets[L.tiles].get() : nullptr;
         const int splits = t ? gptrs_cuda_grouped_splits(&a, t->n, max_ctx) : 1;
         m.launches += splits > 1 ? 2 : 1;
@@ -739,25 +827,41 @@ struct Pass {
         gptrs_moe a = L.moe;
         a.tile_rows = expert_tile_rows(m, a, T);
         int rc;
+        if (L.cfg.shared_ff > 0) {   // its output is a second one for the step behind
+            DenseOpts os;
+            os.act = 2;
+            if ((rc = dense(m, w.shared_up, y.h.p, y.up.p, T, os)) || (rc = dense(m, w.shared_down, y.up.p, y.y.p, T, {}))) return rc;
+        }
         DenseOpts orr;
         orr.out_f32 = true;
         if ((rc = dense(m, w.router, y.h.p, y.router.p, T, orr))) return rc;
         m.launches += T > 128 ? 3 : 2;
         gptrs_row_tile* tiles = y.row_tiles.as<gptrs_row_tile>();
         int32_t* n_tiles = y.n_row_tiles.as<int32_t>();
-        if ((rc = gptrs_cuda_moe_route(&a, y.router.as<float>(), w.router.n, y.h.p, act_dt, ldw, y.pair.as<int32_t>(), y.pair_weight.as<float>(), tiles, n_tiles,
+        if ((rc = gptrs_cuda_moe_route(&a, y.router.as<float>(), w.router.n, fp(w.correction), y.h.p, act_dt, ldw, y.pair.as<int32_t>(), y.pair_weight.as<float>(), tiles, n_tiles,
                                        y.sorted.p, y.moe_work.as<int32_t>(), T, st))) return rc;
         DenseOpts o;
         o.tiles = tiles; o.n_tiles = n_tiles; o.tile_rows = a.tile_rows; o.max_tiles = gptrs_cuda_moe_max_tiles(&a, T);
         const int64_t pairs = (int64_t)T * a.top;
-        DenseOpts ou = o;
-        ou.swiglu = !m.f32();
-        if ((rc = dense(m, w.up, y.sorted.p, m.f32() ? y.gate_up.p : y.up.p, pairs, ou))) return rc;
-        if (m.f32()) {
-            ++m.launches;
-            if ((rc = gptrs_cuda_swiglu_pairs_f32(y.gate_up.as<float>(), y.up.as<float>(), pairs, w.up.n / 2, st))) return rc;
+        if (L.cfg.expert_form == GPTRS_EXPERT_RELU2) {
+            DenseOpts ou = o;
+            ou.act = 2;
+            rc = dense(m, w.up, y.sorted.p, y.up.p, pairs, ou);
+        } else {
+            rc = gated(w.up, y.sorted.p, pairs, GPTRS_GATE_SILU, o);
         }
-        return dense(m, w.down, y.up.p, y.expert_y.p, pairs, o);
+        return rc ? rc : dense(m, w.down, y.up.p, y.expert_y.p, pairs, o);
+    }
+
+    // act(gate) up of a gated feed-forward -> y.up
+    int gated(const DenseWeight& w, const void* x, int64_t rows, int gate, DenseOpts o) {
+        if (!m.f32()) {
+            o.gate = gate;
+            return dense(m, w, x, y.up.p, rows, o);
+        }
+        const int rc = dense(m, w, x, y.gate_up.p, rows, o);
+        ++m.launches;
+        return rc ? rc : gptrs_cuda_gated_pairs_f32(y.gate_up.as<float>(), y.up.as<float>(), rows, w.n / 2, gate, st);
     }
 
     int mixer(LayeredLayer& L) {
@@ -765,6 +869,10 @@ struct Pass {
     }
     int feed_forward(LayeredLayer& L) {
         if (L.cfg.mlp == GPTRS_MLP_EXPERTS) return experts(L);
+        if (L.cfg.mlp == GPTRS_MLP_DENSE_GELU) {
+            const int rg = gated(L.w->up, y.h.p, T, GPTRS_GATE_GELU_TANH, {});
+            return rg ? rg : dense(m, L.w->down, y.up.p, y.y.p, T, {});
+        }
         DenseOpts ou;
         ou.act = 1; ou.pos = L.w->act_pos; ou.neg = L.w->act_neg;
         int rc = dense(m, L.w->up, y.h.p, y.up.p, T, ou);
@@ -775,6 +883,7 @@ struct Pass {
 struct Capture {   // debug: the residual stream after every layer
     DevBuf buf;
     int begin(Model& m, int T) { return m.lay->h_residuals ? buf.alloc((size_t)m.cfg.n_layers * T * m.cfg.d_model * 4) : GPTRS_OK; }
+    float* at(Model& m, int l, int T) { return buf.p ? buf.as<float>() + (size_t)l * T * m.cfg.d_model : nullptr; }
     int take(Model& m, int l, const float* x, int T) {
         const size_t n = (size_t)T * m.cfg.d_model;
         if (buf.p) GPTRS_CUDA_OK(cudaMemcpyAsync(buf.as<float>() + l * n, x, n * 4, cudaMemcpyDeviceToDevice, m.stream));
@@ -900,6 +1009,68 @@ int forward_sandwich(Pass& f, Capture& cap, int n_rows, bool rows_identity) {
     return GPTRS_OK;
 }
 
+// norms in front of the sublayers, streams that are mixed behind them
+int forward_pre_norm(Pass& f, Capture& cap, int n_rows, bool rows_identity) {
+    Model& m = f.m;
+    Layered& y = f.y;
+    const auto& c = m.cfg;
+    gptrs_stream_step base = {};
+    base.d_x = m.hidden.as<float>(); base.streams = std::max(y.cfg.streams, 1);
+    base.y_dtype = f.act_dt; base.eps = c.norm_eps;
+    base.d_h = y.h.p; base.h_dtype = f.act_dt; base.ldh = f.ldw;
+    base.d_status = m.d_status.as<int32_t>();
+    base.rows = f.T; base.dim = c.d_model;
+    auto launch = [&](const gptrs_stream_step& s) { ++m.launches; return gptrs_cuda_stream_step(&s, f.st); };
+    // what a sublayer reads
+    auto opens = [&](gptrs_stream_step& s, const LayeredLayer& L, int sub) {
+        s.d_in = f.fp(L.w->streams[sub].in);
+        s.d_gamma_in = f.fp(sub ? L.w->norm2 : L.w->norm1);
+    };
+    // the output of the sublayer that has just run
+    auto closing = [&](const LayeredLayer& L, int sub) {
+        gptrs_stream_step s = base;
+        s.d_mix = f.fp(L.w->streams[sub].mix); s.d_out = f.fp(L.w->streams[sub].out);
+        if (sub && L.cfg.mlp == GPTRS_MLP_EXPERTS) {
+            s.d_y = y.expert_y.p; s.ldy = L.w->down.n;
+            s.d_pair = y.pair.as<int32_t>(); s.d_pair_weight = y.pair_weight.as<float>(); s.top = L.moe.top;
+            if (L.cfg.shared_ff > 0) { s.d_add = y.y.p; s.ld_add = f.ldw; }
+        } else {
+            s.d_y = y.y.p; s.ldy = f.ldw;
+        }
+        return s;
+    };
+    gptrs_stream_step open = base;
+    open.d_embed = f.fp(m.tok_emb); open.embed_scale = y.cfg.embed_scale; open.d_tokens = m.d_tokens.as<int32_t>(); open.vocab = c.vocab;
+    opens(open, y.layers[0], 0);
+    int rc = launch(open);
+    if (rc) return rc;
+    for (int l = 0; l < c.n_layers; ++l) {
+        LayeredLayer& L = y.layers[l];
+        const bool last = l + 1 == c.n_layers, ff = L.cfg.mlp != GPTRS_MLP_NONE;
+        if ((rc = f.mixer(L))) return rc;
+        if (ff) {
+            gptrs_stream_step s = closing(L, 0);
+            opens(s, L, 1);
+            if ((rc = launch(s)) || (rc = f.feed_forward(L))) return rc;
+        }
+        gptrs_stream_step s = closing(L, ff ? 1 : 0);
+        if (!last || cap.buf.p) {
+            if (!last) opens(s, y.layers[l + 1], 0);
+            s.d_sum = cap.at(m, l, f.T);
+            if ((rc = launch(s))) return rc;
+        }
+        if (last) {
+            if (cap.buf.p) { s.d_y = s.d_add = nullptr; s.d_pair = nullptr; s.d_sum = nullptr; }   // the streams already hold it
+            s.d_gamma_in = f.fp(m.final_g);
+            s.d_rows = rows_identity ? nullptr : m.d_rows.as<int32_t>();
+            s.d_h = m.xn_rows.p;
+            s.rows = n_rows;
+            if ((rc = launch(s))) return rc;
+        }
+    }
+    return GPTRS_OK;
+}
+
 }  // namespace
 
 int layered_forward(Model& m, int T, int max_ctx, int n_rows, bool rows_identity, float temperature, bool skip_logits) {
@@ -909,7 +1080,10 @@ int layered_forward(Model& m, int T, int max_ctx, int n_rows, bool rows_identity
     cudaStream_t st = m.stream;
     Capture cap;
     int rc = cap.begin(m, T);
-    if (!rc) rc = y.cfg.block == GPTRS_BLOCK_SANDWICH ? forward_sandwich(f, cap, n_rows, rows_identity) : forward_output_norm(f, cap, n_rows, rows_identity);
+    if (!rc) {
+        const auto forward = y.cfg.block == GPTRS_BLOCK_SANDWICH ? forward_sandwich : y.cfg.block == GPTRS_BLOCK_PRE_NORM ? forward_pre_norm : forward_output_norm;
+        rc = forward(f, cap, n_rows, rows_identity);
+    }
     if (!rc) rc = cap.end(m);
     if (rc) return rc;
     const bool padded = y.head.n != c.vocab;

@@ -33,9 +33,9 @@ __host__ __device__ inline size_t w8_layout_b_bytes(int64_t n, int64_t k) {
 constexpr int kRedStride = kCtaN + 4; // row stride (floats) of the partial tile in shared memory
 
 // What a dense matmul does to an output element after the bias: xIELU (for z > 0 pos * z^2 + z / 2, else
-// neg * (exp(z) - 1 - z) + z / 2), then a soft cap c * tanh(z / c).
+// neg * (exp(z) - 1 - z) + z / 2) or a squared relu, then a soft cap c * tanh(z / c).
 struct DenseAct {
-    int kind;          // 0 none, 1 xIELU
+    int kind;          // 0 none, 1 xIELU, 2 max(z, 0)^2
     float pos, neg;
     float softcap;     // 0 = none
 };
@@ -55,9 +55,19 @@ __device__ __forceinline__ float dense_act(const DenseAct& a, float z) {
     if (a.kind == 1) {
         const float e = kFast ? expm1_minus_fast(fminf(z, 0.f)) : expm1f(z) - z;
         z = z > 0.f ? fmaf(a.pos * z, z, 0.5f * z) : fmaf(a.neg, e, 0.5f * z);
+    } else if (a.kind == 2) {
+        z = fmaxf(z, 0.f);
+        z *= z;
     }
     if (a.softcap > 0.f) z = a.softcap * tanhf(z / a.softcap);
     return z;
+}
+// Gate activations (GPTRS_GATE_*) for outputs that are rounded to bf16: z / (1 + exp(-z)), and tanh-gelu written the same way, since
+// (1 + tanh(t)) / 2 = 1 / (1 + exp(-2t)).
+__device__ __forceinline__ float silu_fast(float z) { return __fdividef(z, 1.f + __expf(-z)); }
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+    constexpr float k2 = 1.5957691216057308f;   // 2 sqrt(2 / pi)
+    return __fdividef(z, 1.f + __expf(-k2 * fmaf(0.044715f * z * z, z, z)));
 }
 
 struct MatmulParams {
@@ -331,10 +341,17 @@ __device__ __forceinline__ void split_reduce_finish(const MatmulParams& p, const
                 up.x *= r; up.y *= r; up.z *= r; up.w *= r;
             }
             float4 v;
-            v.x = gt.x / (1.f + expf(-gt.x)) * up.x;
-            v.y = gt.y / (1.f + expf(-gt.y)) * up.y;
-            v.z = gt.z / (1.f + expf(-gt.z)) * up.z;
-            v.w = gt.w / (1.f + expf(-gt.w)) * up.w;
+            if (kDense && p.swiglu == GPTRS_GATE_GELU_TANH) {
+                v.x = gelu_tanh_fast(gt.x) * up.x;
+                v.y = gelu_tanh_fast(gt.y) * up.y;
+                v.z = gelu_tanh_fast(gt.z) * up.z;
+                v.w = gelu_tanh_fast(gt.w) * up.w;
+            } else {
+                v.x = gt.x / (1.f + expf(-gt.x)) * up.x;
+                v.y = gt.y / (1.f + expf(-gt.y)) * up.y;
+                v.z = gt.z / (1.f + expf(-gt.z)) * up.z;
+                v.w = gt.w / (1.f + expf(-gt.w)) * up.w;
+            }
             if (p.out_f32) {
                 *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.y) + (size_t)m * NO + n_out) = v;
             } else {

@@ -1,6 +1,6 @@
 // Mixture of experts: which experts a row goes to, and the order of rows in which the grouped matmuls (dense_bf16.cu, dense_f32.cu)
 // find every expert's rows next to one another (no counterpart in gpt.rs).
-//   moe_choose_kernel   a warp per row: softmax over all experts, best groups, best experts of those; counts per expert
+//   moe_choose_kernel   a warp per row: softmax or sigmoid scores, best groups, best experts of those; counts per expert
 //   moe_plan            row offsets of the experts and the tile list of the grouped matmuls; with few rows the tail of the kernel above,
 //                       otherwise a kernel of its own
 //   moe_gather_kernel   copies every row to its places
@@ -13,6 +13,7 @@ namespace {
 struct Params {
     gptrs_moe a;
     const float* logits;
+    const float* correction;              // added to the scores that choose, or null
     int64_t ld;
     const unsigned char* h;
     unsigned char* sorted;
@@ -69,7 +70,7 @@ __device__ __forceinline__ void moe_plan(const Params& p, int* sh) {
     if (e == kWarps * 32 - 1) *p.n_tiles = t_end;
 }
 
-template <int VPL>
+template <int VPL, bool SIGMOID>
 __global__ void __launch_bounds__(kWarps * 32) moe_choose_kernel(const Params p) {
     __shared__ int hist[kMaxExperts], sh[32];
     extern __shared__ int mc_groups[];   // [warps][groups]: best score of every group, then whether it takes part
@@ -84,20 +85,37 @@ __global__ void __launch_bounds__(kWarps * 32) moe_choose_kernel(const Params p)
     for (int row = r_lo + warp; row < r_hi; row += kWarps) {
         constexpr int kNone = (int)0x80000000;
         float z[VPL];
-        int key[VPL];   // order of the logits; kNone: not to be chosen (any more)
+        int key[VPL];   // order of what chooses; kNone: not to be chosen (any more)
         float mx = -INFINITY;
 #pragma unroll
         for (int i = 0; i < VPL; ++i) {
             const int e = i * 32 + lane;
             z[i] = e < E ? p.logits[(size_t)row * p.ld + e] : -INFINITY;
-            key[i] = e < E ? max(order_of(z[i]), kNone + 1) : kNone;
             mx = fmaxf(mx, z[i]);
         }
         mx = warp_max(mx);
         float sum = 0.f;
+        if (SIGMOID) {
 #pragma unroll
-        for (int i = 0; i < VPL; ++i) sum += i * 32 + lane < E ? expf(z[i] - mx) : 0.f;
-        sum = warp_sum(sum);
+            for (int i = 0; i < VPL; ++i) z[i] = 1.f / (1.f + expf(-z[i]));
+        } else {
+#pragma unroll
+            for (int i = 0; i < VPL; ++i) {
+                const float w = i * 32 + lane < E ? expf(z[i] - mx) : 0.f;
+                sum += w;
+                if (p.correction) z[i] = w;   // scores choose in the same order as logits; a correction needs the scores themselves
+            }
+            sum = warp_sum(sum);
+            if (p.correction)
+#pragma unroll
+                for (int i = 0; i < VPL; ++i) z[i] /= sum;
+        }
+#pragma unroll
+        for (int i = 0; i < VPL; ++i) {
+            const int e = i * 32 + lane;
+            if (p.correction && e < E) z[i] += __ldg(p.correction + e);
+            key[i] = e < E ? max(order_of(z[i]), kNone + 1) : kNone;
+        }
         // largest key of `v` and the lowest index that has it
         auto best_of = [&](int v, int index, int* at) {
             const int best = __reduce_max_sync(0xffffffffu, v);
@@ -105,11 +123,28 @@ __global__ void __launch_bounds__(kWarps * 32) moe_choose_kernel(const Params p)
             return best;
         };
         if (p.a.keep < G) {
-            for (int g = lane; g < G; g += 32) gm[g] = kNone;
-            __syncwarp();
+            if (p.a.group_best == 2) {   // the sum of a group's two best
+                for (int g = 0; g < G; ++g) {
+                    const int e0 = g * size;
+                    int best = kNone, index = 0x7fffffff, second = kNone, at, at2;
 #pragma unroll
-            for (int i = 0; i < VPL; ++i)
-                if (i * 32 + lane < E) atomicMax(gm + (i * 32 + lane) / size, key[i]);
+                    for (int i = 0; i < VPL; ++i) {
+                        const int e = i * 32 + lane;
+                        if (e < e0 || e >= e0 + size) continue;
+                        if (key[i] > best) { second = best; best = key[i]; index = e; }
+                        else if (key[i] > second) second = key[i];
+                    }
+                    const int first = best_of(best, index, &at);
+                    const int next = best_of(index == at ? second : best, lane, &at2);
+                    if (lane == 0) gm[g] = min(order_of(value_of(first) + (size > 1 ? value_of(next) : 0.f)), 0x7ffffffe);
+                }
+            } else {
+                for (int g = lane; g < G; g += 32) gm[g] = kNone;
+                __syncwarp();
+#pragma unroll
+                for (int i = 0; i < VPL; ++i)
+                    if (i * 32 + lane < E) atomicMax(gm + (i * 32 + lane) / size, key[i]);
+            }
             __syncwarp();
             for (int n = 0; n < p.a.keep; ++n) {
                 int best = kNone, index = 0x7fffffff, at;
@@ -126,6 +161,7 @@ __global__ void __launch_bounds__(kWarps * 32) moe_choose_kernel(const Params p)
             __syncwarp();
         }
         int mine = 0, chosen = 0;   // lane k: the k-th choice (of the current 32)
+        float total = 0.f;          // this lane's scores
         for (int k = 0; k < p.a.top; ++k) {
             int best = kNone, index = 0x7fffffff, at;
 #pragma unroll
@@ -141,11 +177,19 @@ __global__ void __launch_bounds__(kWarps * 32) moe_choose_kernel(const Params p)
                 const int k0 = k & ~31;
                 if (lane <= k - k0) {
                     const size_t o = (size_t)row * p.a.top + k0 + lane;
-                    p.weight[o] = expf(value_of(mine) - mx) / sum;
+                    float w;
+                    if (SIGMOID) w = 1.f / (1.f + expf(-p.logits[(size_t)row * p.ld + chosen]));
+                    else w = expf((p.correction ? p.logits[(size_t)row * p.ld + chosen] : value_of(mine)) - mx) / sum;
+                    total += w;
+                    p.weight[o] = w;
                     p.id[o] = chosen;
                     p.place[o] = atomicAdd(hist + chosen, 1);
                 }
             }
+        }
+        if (p.a.weight_scale > 0.f) {   // in proportion; every lane changes what it has written itself
+            const float f = p.a.weight_scale / (warp_sum(total) + 1e-20f);
+            for (int k = lane; k < p.a.top; k += 32) p.weight[(size_t)row * p.a.top + k] *= f;
         }
     }
     __syncthreads();
@@ -183,27 +227,31 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const Params p) {
         for (int i = threadIdx.x * 4; i < p.row_bytes; i += 128 * 4) *reinterpret_cast<uint32_t*>(d + i) = *reinterpret_cast<const uint32_t*>(s + i);
 }
 
-struct PairParams { const float* x; float* y; int n; };
-__global__ void __launch_bounds__(128) swiglu_pairs_kernel(const PairParams p) {
+struct PairParams { const float* x; float* y; int n, gate; };
+__global__ void __launch_bounds__(128) gated_pairs_kernel(const PairParams p) {
     pdl_launch_dependents();
     pdl_wait();
     const float* x = p.x + (size_t)blockIdx.x * 2 * p.n;
     for (int i = threadIdx.x; i < p.n; i += 128) {
         const int c = (i >> 3) * 16 + (i & 7);
         const float g = x[c];
-        p.y[(size_t)blockIdx.x * p.n + i] = g / (1.f + expf(-g)) * x[c + 8];
+        const float a = p.gate == GPTRS_GATE_GELU_TANH ? 0.5f * g * (1.f + tanhf(0.7978845608028654f * fmaf(0.044715f * g * g, g, g))) : g / (1.f + expf(-g));
+        p.y[(size_t)blockIdx.x * p.n + i] = a * x[c + 8];
     }
 }
 
 template <int VPL>
 int launch_choose(const Params& p, int ctas, size_t smem, cudaStream_t st) {
-    if (smem > 40 * 1024) GPTRS_CUDA_OK(cudaFuncSetAttribute(moe_choose_kernel<VPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    return launch_kernel(moe_choose_kernel<VPL>, dim3((unsigned)ctas), dim3(kWarps * 32), smem, st, 1, p);
+    const auto kern = p.a.scores == GPTRS_ROUTE_SIGMOID ? moe_choose_kernel<VPL, true> : moe_choose_kernel<VPL, false>;
+    if (smem > 40 * 1024) GPTRS_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    return launch_kernel(kern, dim3((unsigned)ctas), dim3(kWarps * 32), smem, st, 1, p);
 }
 
 int check(const gptrs_moe* a) {
     GPTRS_REQUIRE(a && a->experts > 0 && a->top > 0 && a->groups > 0 && a->keep > 0 && a->tile_rows > 0, "experts: sizes must be positive");
     GPTRS_REQUIRE(a->experts % a->groups == 0 && a->keep <= a->groups && a->top <= a->keep * (a->experts / a->groups), "experts: groups must be equal and hold enough experts");
+    GPTRS_REQUIRE((a->scores == GPTRS_ROUTE_SOFTMAX || a->scores == GPTRS_ROUTE_SIGMOID) && a->group_best >= 0 && a->group_best <= 2 && a->weight_scale >= 0.f,
+                  "experts: scores, group score or weight scale");
     if (a->experts > kMaxExperts) return fail(GPTRS_UNIMPLEMENTED, "experts: more than 1024");
     return GPTRS_OK;
 }
@@ -223,7 +271,7 @@ int64_t gptrs_cuda_moe_max_tiles(const gptrs_moe* a, int64_t rows) {
 
 int64_t gptrs_cuda_moe_work_ints(const gptrs_moe* a, int64_t rows) { return a ? 2 * (int64_t)kMaxExperts + 2 * rows * a->top : 0; }
 
-int gptrs_cuda_moe_route(const gptrs_moe* a, const float* d_logits, int64_t ld, const void* d_h, int h_dtype, int64_t ldh, int32_t* d_pair, float* d_weight,
+int gptrs_cuda_moe_route(const gptrs_moe* a, const float* d_logits, int64_t ld, const float* d_correction, const void* d_h, int h_dtype, int64_t ldh, int32_t* d_pair, float* d_weight,
                          gptrs_row_tile* d_tiles, int32_t* d_n_tiles, void* d_sorted, int32_t* d_work, int64_t rows, void* stream) {
     int rc = check(a);
     if (rc) return rc;
@@ -232,7 +280,7 @@ int gptrs_cuda_moe_route(const gptrs_moe* a, const float* d_logits, int64_t ld, 
     GPTRS_REQUIRE(h_dtype == GPTRS_F32 || (h_dtype == GPTRS_BF16 && ldh % 2 == 0), "rows of f32, or of an even number of bf16");
     if (rows == 0) return GPTRS_OK;
     Params p = {};
-    p.a = *a; p.logits = d_logits; p.ld = ld;
+    p.a = *a; p.logits = d_logits; p.ld = ld; p.correction = d_correction;
     p.h = static_cast<const unsigned char*>(d_h); p.sorted = static_cast<unsigned char*>(d_sorted);
     p.row_bytes = (int)(ldh * (h_dtype == GPTRS_F32 ? 4 : 2));
     p.pair = d_pair; p.weight = d_weight; p.tiles = d_tiles; p.n_tiles = d_n_tiles;
@@ -254,12 +302,13 @@ int gptrs_cuda_moe_route(const gptrs_moe* a, const float* d_logits, int64_t ld, 
     return launch_kernel(moe_gather_kernel, dim3((unsigned)rows, (unsigned)a->top), dim3(128), 0, st, 1, p);
 }
 
-int gptrs_cuda_swiglu_pairs_f32(const float* d_gate_up, float* d_y, int64_t rows, int64_t n, void* stream) {
+int gptrs_cuda_gated_pairs_f32(const float* d_gate_up, float* d_y, int64_t rows, int64_t n, int gate, void* stream) {
     GPTRS_REQUIRE(d_gate_up && d_y, "null pointer");
     GPTRS_REQUIRE(rows >= 0 && rows < (1ll << 31) && n > 0 && n % 8 == 0 && n < (1ll << 30), "bad shape");
     if (rows == 0) return GPTRS_OK;
-    const PairParams p = {d_gate_up, d_y, (int)n};
-    return launch_kernel(swiglu_pairs_kernel, dim3((unsigned)rows), dim3(128), 0, as_stream(stream), 1, p);
+    GPTRS_REQUIRE(gate == GPTRS_GATE_SILU || gate == GPTRS_GATE_GELU_TANH, "unknown gate activation");
+    const PairParams p = {d_gate_up, d_y, (int)n, gate};
+    return launch_kernel(gated_pairs_kernel, dim3((unsigned)rows), dim3(128), 0, as_stream(stream), 1, p);
 }
 
 }  // extern "C"

@@ -21,8 +21,10 @@ from . import check, lib
 KIND_GPT, KIND_MINISTRAL, KIND_LAYERED = 0, 1, 2
 MODE_F32, MODE_W4A16, MODE_W8A16, MODE_BF16 = 0, 1, 2, 3
 MIXER_LATENT_ATTENTION, MIXER_GROUPED_ATTENTION, MIXER_CHANNEL_DELTA = 0, 1, 2
-MLP_NONE, MLP_DENSE_XIELU, MLP_EXPERTS = 0, 1, 2
-BLOCK_OUTPUT_NORM, BLOCK_SANDWICH = 0, 1
+MLP_NONE, MLP_DENSE_XIELU, MLP_EXPERTS, MLP_DENSE_GELU = 0, 1, 2, 3
+EXPERT_SWIGLU, EXPERT_RELU2 = 0, 1
+ROUTE_SOFTMAX, ROUTE_SIGMOID = 0, 1
+BLOCK_OUTPUT_NORM, BLOCK_SANDWICH, BLOCK_PRE_NORM = 0, 1, 2
 MASK_CAUSAL, MASK_WINDOW, MASK_CHUNK = 0, 1, 2
 
 
@@ -47,24 +49,28 @@ class _LayerConfig(ctypes.Structure):
         ("kv_heads", ctypes.c_int), ("mask", ctypes.c_int), ("mask_size", ctypes.c_int), ("distance_bias", ctypes.c_int), ("proj_bias", ctypes.c_int),
         ("softcap", ctypes.c_float), ("taps", ctypes.c_int), ("decay_rank", ctypes.c_int), ("gate_rank", ctypes.c_int),
         ("experts", ctypes.c_int), ("top", ctypes.c_int), ("groups", ctypes.c_int), ("keep", ctypes.c_int), ("weights_of", ctypes.c_int),
+        ("q_rank", ctypes.c_int), ("maps", ctypes.c_int), ("out_gate", ctypes.c_int), ("kv_from", ctypes.c_int), ("diff", ctypes.c_float),
+        ("expert_form", ctypes.c_int), ("shared_ff", ctypes.c_int), ("route", ctypes.c_int), ("group_best", ctypes.c_int), ("correction", ctypes.c_int),
+        ("weight_scale", ctypes.c_float),
     ]
 
 
 class _LayeredConfig(ctypes.Structure):
-    _fields_ = [("conv_taps", ctypes.c_int), ("logit_softcap", ctypes.c_float), ("block", ctypes.c_int), ("learned_positions", ctypes.c_int)]
+    _fields_ = [("conv_taps", ctypes.c_int), ("logit_softcap", ctypes.c_float), ("block", ctypes.c_int), ("learned_positions", ctypes.c_int),
+                ("streams", ctypes.c_int), ("embed_scale", ctypes.c_float)]
 
 
 @dataclass
 class LayerConfig:
-    """One layer of a model of the layered kind: its mixer and its feed-forward. Latent attention (in a sliding window) takes heads
-    .. rot_dims; attention with grouped key / value heads takes heads, dim, vdim, scale and kv_heads .. softcap; the delta rule takes
-    heads, dim, vdim, kv_heads and taps .. gate_rank. Experts have the size d_ff each."""
+    """One layer of a model of the layered kind: its mixer and its feed-forward. Latent attention (in a sliding window, or over
+    everything) takes heads .. rot_dims and q_rank; attention with grouped key / value heads takes heads, dim, vdim, scale, kv_heads ..
+    softcap and maps .. diff; the delta rule takes heads, dim, vdim, kv_heads and taps .. gate_rank. Experts have the size d_ff each."""
     heads: int
     dim: int            # query / key dimensions of a head (latent attention: those that are not rotated)
     rot_dim: int = 0    # and those that are (shared key part)
     vdim: int = 0
     kv_rank: int = 0
-    window: int = 0
+    window: int = 0     # 0 = none
     scale: float = 1.0
     rope_base: float = 10000.0
     rot_dims: int = 0   # rotated dimensions of the rot_dim part (0 = all)
@@ -85,30 +91,59 @@ class LayerConfig:
     groups: int = 1
     keep: int = 1
     weights_of: int = -1     # layer whose weights this one uses
+    q_rank: int = 0          # queries through a latent of this size
+    maps: int = 1            # 2: differential attention
+    out_gate: int = 0        # the heads' outputs are gated
+    kv_from: int = -1        # earlier layer whose keys and values this one reads
+    diff: float = 0.0        # constant of differential attention
+    expert_form: int = EXPERT_SWIGLU
+    shared_ff: int = 0       # size of a shared expert
+    route: int = ROUTE_SOFTMAX
+    group_best: int = 1      # experts that make a group's score
+    correction: int = 0      # a vector added to the scores that choose
+    weight_scale: float = 0.0   # > 0: the experts' weights are in proportion and sum to this
 
     def _struct(self):
         values = {f: getattr(self, f) for f, _ in _LayerConfig._fields_}
         values["rot_dims"] = self.rot_dims or self.rot_dim
         return _LayerConfig(**values)
 
-    def shapes(self, p: str, d: int, sandwich: bool, conv_taps: int) -> dict[str, tuple[int, ...]]:
+    def shapes(self, p: str, d: int, block: int, conv_taps: int, streams: int = 0) -> dict[str, tuple[int, ...]]:
         """Names and shapes of the layer's parameters (prefix `p`, width `d`)."""
         if self.weights_of >= 0:
             return {}
-        out: dict[str, tuple[int, ...]] = {f"{p}.norm1": (d,)}
-        out.update({f"{p}.norm1b": (d,)} if sandwich else {f"{p}.canon1": (d, conv_taps)})
+
+        def beside(n):   # a sublayer's norms and what the block form has beside them
+            out = {f"{p}.norm{n}": (d,)}
+            if block == BLOCK_SANDWICH:
+                out[f"{p}.norm{n}b"] = (d,)
+            elif block == BLOCK_OUTPUT_NORM:
+                out[f"{p}.canon{n}"] = (d, conv_taps)
+            elif streams:
+                out.update({f"{p}.hc{n}.in": (streams,), f"{p}.hc{n}.out": (streams,), f"{p}.hc{n}.mix": (streams, streams)})
+            return out
+
+        out: dict[str, tuple[int, ...]] = beside(1)
         x, qk, v = f"{p}.mix", self.heads * self.dim, self.heads * self.vdim
         if self.mixer == MIXER_LATENT_ATTENTION:
-            out.update({f"{x}.q": (self.heads * (self.dim + self.rot_dim), d), f"{x}.dkv": (self.kv_rank + self.rot_dim, d), f"{x}.dkv.norm": (self.kv_rank,),
+            rows = self.heads * (self.dim + self.rot_dim)
+            out.update({f"{x}.dq": (self.q_rank, d), f"{x}.dq.norm": (self.q_rank,), f"{x}.uq": (rows, self.q_rank)} if self.q_rank else {f"{x}.q": (rows, d)})
+            out.update({f"{x}.dkv": (self.kv_rank + self.rot_dim, d), f"{x}.dkv.norm": (self.kv_rank,),
                         f"{x}.uk": (qk, self.kv_rank), f"{x}.uv": (v, self.kv_rank), f"{x}.o": (d, v)})
         elif self.mixer == MIXER_GROUPED_ATTENTION:
-            rows = {"q": qk, "k": self.kv_heads * self.dim, "v": self.kv_heads * self.vdim}
+            rows = {"q": qk * self.maps}
+            if self.kv_from < 0:
+                rows.update(k=self.kv_heads * self.dim * self.maps, v=self.kv_heads * self.vdim)
             out.update({f"{x}.{n}": (r, d) for n, r in rows.items()})
             out[f"{x}.o"] = (d, v)
             if self.proj_bias:
                 out.update({f"{x}.{n}.b": (r,) for n, r in {**rows, "o": d}.items()})
             if self.distance_bias:
                 out.update({f"{x}.r1": (self.heads,), f"{x}.r2": (self.heads,)})
+            if self.out_gate:
+                out[f"{x}.g"] = (v, d)
+            if self.maps == 2:
+                out.update({f"{x}.{n}": (self.dim,) for n in ("lq1", "lk1", "lq2", "lk2")})
         else:
             kq = self.kv_heads * self.dim
             for n, r in (("q", kq), ("k", kq), ("v", v)):
@@ -118,14 +153,21 @@ class LayerConfig:
         if self.mlp == MLP_NONE:
             return out
         f = f"{p}.mlp"
-        out[f"{p}.norm2"] = (d,)
-        out.update({f"{p}.norm2b": (d,)} if sandwich else {f"{p}.canon2": (d, conv_taps)})
+        out.update(beside(2))
         if self.mlp == MLP_DENSE_XIELU:
             out.update({f"{f}.up": (self.d_ff, d), f"{f}.up.b": (self.d_ff,), f"{f}.down": (d, self.d_ff), f"{f}.down.b": (d,), f"{f}.act": (2,)})
+        elif self.mlp == MLP_DENSE_GELU:
+            out.update({f"{f}.gate": (self.d_ff, d), f"{f}.up": (self.d_ff, d), f"{f}.down": (d, self.d_ff)})
         else:
             for e in range(self.experts):
-                out.update({f"{f}.e{e}.gate": (self.d_ff, d), f"{f}.e{e}.up": (self.d_ff, d), f"{f}.e{e}.down": (d, self.d_ff)})
+                if self.expert_form == EXPERT_SWIGLU:
+                    out[f"{f}.e{e}.gate"] = (self.d_ff, d)
+                out.update({f"{f}.e{e}.up": (self.d_ff, d), f"{f}.e{e}.down": (d, self.d_ff)})
             out[f"{f}.router"] = (self.experts, d)
+            if self.correction:
+                out[f"{f}.correction"] = (self.experts,)
+            if self.shared_ff:
+                out.update({f"{f}.shared.up": (self.shared_ff, d), f"{f}.shared.down": (d, self.shared_ff)})
         return out
 
 
@@ -157,6 +199,8 @@ class ModelConfig:
     logit_softcap: float = 0.0
     block: int = BLOCK_OUTPUT_NORM
     learned_positions: int = 0     # position vectors added to the embedding
+    streams: int = 0               # copies of the residual that are mixed at every sublayer (BLOCK_PRE_NORM)
+    embed_scale: float = 1.0       # of the embedding (BLOCK_PRE_NORM)
 
     @staticmethod
     def layered(layers, d_model: int, vocab: int, context_length: int, norm_eps: float, conv_taps: int = 1, logit_softcap: float = 0.0, **kw):
@@ -217,14 +261,14 @@ class ModelConfig:
 
     def _layered_shapes(self) -> dict[str, tuple[int, ...]]:
         """Names and shapes of the layered kind; Linear weights are [out, in]."""
-        d, sandwich = self.d_model, self.block == BLOCK_SANDWICH
+        d = self.d_model
         out: dict[str, tuple[int, ...]] = {"embed": (self.vocab, d)}
-        if not sandwich:
+        if self.block == BLOCK_OUTPUT_NORM:
             out["embed.norm"] = (d,)
         if self.learned_positions:
             out["pos"] = (self.learned_positions, d)
         for l, c in enumerate(self.layers):
-            out.update(c.shapes(f"l{l}", d, sandwich, self.conv_taps))
+            out.update(c.shapes(f"l{l}", d, self.block, self.conv_taps, self.streams))
         out["final.norm"] = (d,)
         out["head"] = (self.vocab, d)
         return out
@@ -257,7 +301,7 @@ class LoadedModel:
         check(lib().gptrs_cuda_model_create(ctypes.byref(c), ctypes.byref(self._h)))
         if config.kind == KIND_LAYERED:
             rows = (_LayerConfig * len(config.layers))(*[l._struct() for l in config.layers])
-            common = _LayeredConfig(config.conv_taps, config.logit_softcap, config.block, config.learned_positions)
+            common = _LayeredConfig(config.conv_taps, config.logit_softcap, config.block, config.learned_positions, config.streams, config.embed_scale)
             check(lib().gptrs_cuda_model_set_layers(self._h, ctypes.byref(common), rows, len(config.layers)))
         self._finalized = False
 

@@ -385,6 +385,7 @@ def _status(dev, status):
 def _dense_epilogue(x, bias, xielu, softcap, strides, status):
     ep = _abi.DenseEpilogue()
     ep.d_bias = _ptr(bias)
+    ep.act = 2 if strides.pop("relu2", False) else 0
     if xielu is not None:
         ep.act, ep.act_pos, ep.act_neg = 1, *xielu
     ep.softcap = softcap
@@ -451,8 +452,8 @@ def post_norm_final(x, y, gamma, final_gamma, eps, rows=None, out_dtype=torch.fl
     return out
 
 
-def latent_layout(heads, dim, rot_dim, vdim, kv_rank, window, scale, rot_dims=None, bf16=True):
-    a = _abi.LatentAttention(BF16 if bf16 else F32, heads, dim, rot_dim, vdim, kv_rank, window, rot_dim if rot_dims is None else rot_dims, scale)
+def latent_layout(heads, dim, rot_dim, vdim, kv_rank, window, scale, rot_dims=None, bf16=True, q_rank=0):
+    a = _abi.LatentAttention(BF16 if bf16 else F32, heads, dim, rot_dim, vdim, kv_rank, window, rot_dim if rot_dims is None else rot_dims, scale, q_rank)
     check(lib().gptrs_cuda_latent_layout(ctypes.byref(a)))
     return a
 
@@ -460,6 +461,18 @@ def latent_layout(heads, dim, rot_dim, vdim, kv_rank, window, scale, rot_dims=No
 def latent_append(a, qkv, positions, slot, page_table, norm_w, eps, cos, sin, qa, pool):
     check(lib().gptrs_cuda_latent_append(ctypes.byref(a), _ptr(qkv), _ptr(positions), _ptr(slot), _ptr(page_table), page_table.shape[1], _ptr(norm_w), eps,
                                          _ptr(cos), _ptr(sin), _ptr(qa), _ptr(pool), qkv.shape[0], _stream()))
+
+
+def latent_append_keys(a, kv, positions, slot, page_table, norm_w, q_norm_w, eps, cos, sin, pool):
+    """Page write of the first projection's rows; returns the normed query latents."""
+    out = torch.empty((kv.shape[0], a.q_latent_row), dtype=kv.dtype, device=kv.device)
+    check(lib().gptrs_cuda_latent_append_keys(ctypes.byref(a), _ptr(kv), _ptr(positions), _ptr(slot), _ptr(page_table), page_table.shape[1], _ptr(norm_w),
+                                              _ptr(q_norm_w), eps, _ptr(cos), _ptr(sin), _ptr(out), _ptr(pool), kv.shape[0], _stream()))
+    return out
+
+
+def latent_rotate_queries(a, q, positions, cos, sin, qa):
+    check(lib().gptrs_cuda_latent_rotate_queries(ctypes.byref(a), _ptr(q), _ptr(positions), _ptr(cos), _ptr(sin), _ptr(qa), q.shape[0], _stream()))
 
 
 def latent_attention(a, qa, pool, page_table, slot, ctx_len, max_ctx_len, tiles=None, splits=None, status=None):
@@ -508,8 +521,38 @@ def norm_step(x, eps, y=None, gamma_out=None, gamma_in=None, pair=None, pair_wei
     return h
 
 
-def grouped_layout(heads, kv_heads, dim, vdim, mask, mask_size, scale, softcap=0.0, distance_bias=False, bf16=True):
-    a = _abi.GroupedAttention(BF16 if bf16 else F32, heads, kv_heads, dim, vdim, mask, mask_size, scale, softcap, int(distance_bias))
+def stream_step(x, eps, y=None, mix=None, w_out=None, w_in=None, gamma_in=None, pair=None, pair_weight=None, add=None, embed=None, embed_scale=1.0,
+                tokens=None, rows=None, want_sum=False, out_dtype=torch.float32, ldh=None, status=None):
+    """x [rows][streams][dim] (f32, in place) <- mixed streams + w_out y, or scaled embedding rows; returns (h = rms_norm of the streams' combination
+    w_in times gamma_in, or None; the sum of the new streams, or None)."""
+    dev, (n, streams, dim) = x.device, x.shape
+    s = _abi.StreamStep()
+    s.d_x, s.streams, s.eps, s.dim, s.d_status = _ptr(x), streams, eps, dim, _ptr(_status(dev, status))
+    s.rows = n if rows is None else rows.shape[0]
+    s.d_rows = _ptr(rows)
+    s.d_mix, s.d_out, s.d_in = _ptr(mix), _ptr(w_out), _ptr(w_in)
+    if y is not None:
+        s.d_y, s.y_dtype, s.ldy = _ptr(y), _dt(y), y.shape[1]
+    if pair is not None:
+        s.d_pair, s.d_pair_weight, s.top = _ptr(pair), _ptr(pair_weight), pair.shape[1]
+    if add is not None:
+        s.d_add, s.ld_add = _ptr(add), add.shape[1]
+    if embed is not None:
+        s.d_embed, s.embed_scale, s.d_tokens, s.vocab = _ptr(embed), embed_scale, _ptr(tokens), embed.shape[0]
+    total = torch.empty((n, dim), device=dev) if want_sum else None
+    s.d_sum = _ptr(total)
+    h = None
+    if gamma_in is not None:
+        h = torch.empty((s.rows, ldh or dim), dtype=out_dtype, device=dev)
+        s.d_gamma_in, s.d_h, s.h_dtype, s.ldh = _ptr(gamma_in), _ptr(h), _dt(h), h.shape[1]
+    check(lib().gptrs_cuda_stream_step(ctypes.byref(s), _stream()))
+    return h, total
+
+
+def grouped_layout(heads, kv_heads, dim, vdim, mask, mask_size, scale, softcap=0.0, distance_bias=False, bf16=True, maps=1, gate=False, shared_kv=False,
+                   lam=0.0, head_scale=1.0, head_eps=1e-5):
+    a = _abi.GroupedAttention(BF16 if bf16 else F32, heads, kv_heads, dim, vdim, mask, mask_size, scale, softcap, int(distance_bias), maps, int(gate),
+                              int(shared_kv), lam, head_scale, head_eps)
     check(lib().gptrs_cuda_grouped_layout(ctypes.byref(a)))
     return a
 
@@ -561,9 +604,9 @@ def delta_rule(a, proj, decay, gate, conv, a_log, dt_bias, norm, state, conv_sta
     return out
 
 
-def moe_route(experts, top, groups, keep, tile_rows, logits, h, work=None):
+def moe_route(experts, top, groups, keep, tile_rows, logits, h, work=None, sigmoid=False, group_best=1, weight_scale=0.0, correction=None):
     """Returns (pair, weight, tiles, n_tiles, sorted rows, most tiles): see gptrs_cuda_moe_route."""
-    a = _abi.Moe(experts, top, groups, keep, tile_rows)
+    a = _abi.Moe(experts, top, groups, keep, tile_rows, int(sigmoid), group_best, weight_scale)
     n, dev = logits.shape[0], logits.device
     most = lib().gptrs_cuda_moe_max_tiles(ctypes.byref(a), n)
     pair, weight = torch.empty((n, top), dtype=torch.int32, device=dev), torch.empty((n, top), device=dev)
@@ -571,12 +614,15 @@ def moe_route(experts, top, groups, keep, tile_rows, logits, h, work=None):
     out = torch.empty((n * top, h.shape[1]), dtype=h.dtype, device=dev)
     if work is None:
         work = torch.zeros(lib().gptrs_cuda_moe_work_ints(ctypes.byref(a), n), dtype=torch.int32, device=dev)
-    check(lib().gptrs_cuda_moe_route(ctypes.byref(a), _ptr(logits), logits.shape[1], _ptr(h), _dt(h), h.shape[1], _ptr(pair), _ptr(weight), _ptr(tiles),
+    check(lib().gptrs_cuda_moe_route(ctypes.byref(a), _ptr(logits), logits.shape[1], _ptr(correction), _ptr(h), _dt(h), h.shape[1], _ptr(pair), _ptr(weight), _ptr(tiles),
                                      _ptr(n_tiles), _ptr(out), _ptr(work), n, _stream()))
     return pair, weight, tiles, n_tiles, out, most
 
 
-def swiglu_pairs_f32(gate_up, n):
+GATE_SILU, GATE_GELU_TANH = 1, 2
+
+
+def gated_pairs_f32(gate_up, n, gate=GATE_SILU):
     out = torch.empty((gate_up.shape[0], n), device=gate_up.device)
-    check(lib().gptrs_cuda_swiglu_pairs_f32(_ptr(gate_up), _ptr(out), gate_up.shape[0], n, _stream()))
+    check(lib().gptrs_cuda_gated_pairs_f32(_ptr(gate_up), _ptr(out), gate_up.shape[0], n, gate, _stream()))
     return out

@@ -193,11 +193,12 @@ int gptrs_cuda_debug_matmul_fault(int starve, uint32_t spin_limit);
  * crates/gpt-rs/src/ops/functional/linalg.rs:109-127, tensor_ops.rs:42-56; the activations and the soft cap have no
  * counterpart in gpt.rs).
  * ============================================================================================ */
+enum { GPTRS_GATE_SILU = 1, GPTRS_GATE_GELU_TANH = 2 };   /* z / (1 + exp(-z)); z / 2 (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))) */
 typedef struct gptrs_row_tile { int32_t group, row0, rows, pad; } gptrs_row_tile;
 typedef struct {
     int out_dtype;             /* bf16 kernel: GPTRS_BF16 or GPTRS_F32 */
     const float* d_bias;       /* optional [n] */
-    int act;                   /* 0 = none, 1 = xIELU: z > 0: act_pos z^2 + z/2, else act_neg (exp(z) - 1 - z) + z/2 */
+    int act;                   /* 0 = none, 1 = xIELU: z > 0: act_pos z^2 + z/2, else act_neg (exp(z) - 1 - z) + z/2, 2 = max(z, 0)^2 */
     float act_pos, act_neg;
     float softcap;             /* > 0: y = softcap * tanh(y / softcap), after the activation */
     int64_t ldx, ldy;          /* row strides in elements (0 = k and n) */
@@ -214,7 +215,8 @@ typedef struct {
     const struct gptrs_row_tile* d_tiles;
     const int32_t* d_n_tiles;
     int64_t max_tiles, tile_rows;
-    int swiglu;                /* bf16 kernel: 16 channels = 8 gates, then their 8 partners; y[m][n / 2] = silu(gate) partner */
+    int swiglu;                /* bf16 kernel: 16 channels = 8 gates, then their 8 partners; y[m][n / 2] = act(gate) partner with
+                                * GPTRS_GATE_SILU or GPTRS_GATE_GELU_TANH; 0 = no gates */
 } gptrs_dense_epilogue;
 /* y[m][n] = act(x[m][k] . w[b][k][n] + bias), everything f32 (weights [in, out], nn/layers/linear.rs:14). */
 int gptrs_cuda_dense_f32(const float* d_x, const float* d_w, float* d_y, int64_t m, int64_t n, int64_t k,
@@ -269,15 +271,21 @@ int gptrs_cuda_post_norm_final(const float* d_x, const void* d_y, int y_dtype, i
  * Latent attention (no counterpart in gpt.rs): the cache holds one normed latent of kv_rank values and one rotated key part
  * of rot_dim values per token, shared by all heads; the per-head key and value projections are absorbed into the query
  * (W_uk^T q, a batched gptrs_cuda_dense_* in front) and the output (W_uv o, one behind). Sliding window: position i sees
- * i - window + 1 .. i. Pages of 16 tokens, addressed through page_table[slot][page index] like the KV pool below.
+ * i - window + 1 .. i (window 0: all of 0 .. i). Queries may come through a normed latent of their own (q_rank > 0): the first
+ * projection then gives [query latent | latent | rotated key], a second one the queries. Pages of 16 tokens, addressed through
+ * page_table[slot][page index] like the KV pool below.
  * ============================================================================================ */
 typedef struct {
     int dtype;                 /* GPTRS_F32 or GPTRS_BF16: activations and cache */
     int heads, dim, rot_dim, vdim, kv_rank, window;
     int rot_dims;              /* rotated dimensions of the rot_dim part: pairs (2i, 2i + 1) */
     float scale;
+    int q_rank;                /* 0 = queries are projected directly */
     /* filled in by gptrs_cuda_latent_layout (elements): */
-    int q_head_stride, q_rot_offset, dkv_offset, rot_offset, q_row; /* projection row: heads x [dim | rot], latent, rotated key */
+    int q_head_stride, q_rot_offset, dkv_offset, rot_offset, q_row; /* projection row: heads x [dim | rot], latent, rotated key; with
+                                                                       q_rank q_row is a row of queries alone */
+    int kv_row;                                                     /* row that holds the latent (q_row without q_rank) */
+    int q_latent_row;                                               /* with q_rank: row of normed query latents */
     int qa_head_stride, qa_rot_offset;                              /* absorbed query of a head: [kv_rank | rot] */
     int lat_head_stride;                                            /* attention output of a head, [kv_rank] */
     int out_head_stride;                                            /* the same after W_uv, [vdim] */
@@ -289,6 +297,13 @@ int gptrs_cuda_latent_layout(gptrs_latent_attention* a);
 int gptrs_cuda_latent_append(const gptrs_latent_attention* a, const void* d_qkv, const int32_t* d_positions, const int32_t* d_slot,
                              const int32_t* d_page_table, int64_t max_pages, const float* d_norm_w, float eps, const float* d_cos,
                              const float* d_sin, void* d_qa, void* d_pool, int64_t n_tokens, void* stream);
+/* With q_rank the same in two steps, before and after the second projection: first-projection rows [T][kv_row] -> page, and the query
+ * latents RMS-normed with d_q_norm_w -> d_q_latent [T][q_latent_row]; queries [T][q_row] -> rotated parts in d_qa. */
+int gptrs_cuda_latent_append_keys(const gptrs_latent_attention* a, const void* d_kv, const int32_t* d_positions, const int32_t* d_slot,
+                                  const int32_t* d_page_table, int64_t max_pages, const float* d_norm_w, const float* d_q_norm_w, float eps,
+                                  const float* d_cos, const float* d_sin, void* d_q_latent, void* d_pool, int64_t n_tokens, void* stream);
+int gptrs_cuda_latent_rotate_queries(const gptrs_latent_attention* a, const void* d_q, const int32_t* d_positions, const float* d_cos,
+                                     const float* d_sin, void* d_qa, int64_t n_tokens, void* stream);
 /* Tokens of a query tile of the tensor-core kernel (0: these sizes use the plain kernel), key splits for a launch, scratch. */
 int gptrs_cuda_latent_tile_tokens(const gptrs_latent_attention* a);
 int gptrs_cuda_latent_splits(const gptrs_latent_attention* a, int64_t n_tiles, int64_t max_ctx_len);
@@ -334,10 +349,54 @@ typedef struct {
 int gptrs_cuda_norm_step(const gptrs_norm_step* step, void* stream);
 
 /* ==============================================================================================
+ * Step between two sublayers of a model with a norm in front of every sublayer and `streams` copies of the residual (no counterpart
+ * in gpt.rs): for every row, from the old streams all at once,
+ *     x_t <- sum_s mix[s][t] x_s + out[t] y        h = rms(sum_s in[s] x_s) gamma_in
+ * where mix and out belong to the sublayer that has run and in to the one that comes. d_mix NULL: every stream keeps itself; d_out
+ * NULL: y enters every stream as it is; d_in NULL: the sum of the streams (one stream and no weights: the ordinary residual).
+ * d_embed set: every stream starts as embed_scale * embed[token]. d_y NULL: the streams stay. d_pair as in gptrs_norm_step; d_add:
+ * a second output added to y (a shared expert). d_rows set: row i of the launch is row d_rows[i] of x and y, h is compact, and x is
+ * not written (the end of the model).
+ * ============================================================================================ */
+enum { GPTRS_MAX_STREAMS = 16 };
+typedef struct {
+    float* d_x;                /* [rows][streams][dim] */
+    int streams;
+    const void* d_y;
+    int y_dtype;               /* of d_add too */
+    int64_t ldy;
+    const int32_t* d_pair;     /* [rows][top] */
+    const float* d_pair_weight;
+    int64_t top;
+    const void* d_add;         /* optional [rows][ld_add] */
+    int64_t ld_add;
+    const float* d_embed;
+    float embed_scale;
+    const int32_t* d_tokens;
+    int64_t vocab;
+    const float* d_mix;        /* [from][to] */
+    const float *d_out, *d_in; /* [streams] */
+    const float* d_gamma_in;   /* NULL: no h */
+    float eps;
+    const int32_t* d_rows;
+    void* d_h;
+    int h_dtype;
+    int64_t ldh;               /* columns past dim are zeroed */
+    float* d_sum;              /* optional [rows][dim]: the sum of the new streams */
+    int32_t* d_status;         /* receives 2 for a token id out of range */
+    int64_t rows, dim;
+} gptrs_stream_step;
+int gptrs_cuda_stream_step(const gptrs_stream_step* step, void* stream);
+
+/* ==============================================================================================
  * Attention with grouped key / value heads of any size over a paged cache (no counterpart in gpt.rs; the kernels further down
  * serve gpt.rs' own attention): query head h reads key / value head h / (heads / kv_heads); scores are soft-capped, then
  * r1[h] ln(1 + r2[h] (i - j)) is taken off; a mask says where the keys of position i begin. Pages of 16 tokens hold the
  * [value | key] rows of every kv head.
+ *   maps = 2 (differential attention): every query and key head has two parts, each an attention of its own over the same values;
+ *            the output is d = a1 - lambda a2, then d / sqrt(mean(d^2) + head_eps) head_scale over the values of the head.
+ *   gate     the output is multiplied by sigmoid(gate), a further part of the projection row.
+ *   shared_kv  the projection rows hold no keys and values: another layer has put them into the cache.
  * ============================================================================================ */
 enum { GPTRS_MASK_CAUSAL = 0, GPTRS_MASK_WINDOW = 1, GPTRS_MASK_CHUNK = 2 };   /* from 0; i - size + 1; floor(i / size) size */
 typedef struct {
@@ -346,8 +405,12 @@ typedef struct {
     int mask, mask_size;
     float scale, softcap;      /* softcap 0 = none */
     int distance_bias;         /* 1: r1 and r2 are given */
+    int maps, gate, shared_kv; /* maps 0 = 1 */
+    float lambda_, head_scale, head_eps;   /* two maps: lambda and the constants of the norm */
     /* filled in by gptrs_cuda_grouped_layout (elements): */
-    int q_head_stride, k_offset, k_head_stride, v_offset, v_head_stride, q_row;   /* projection row: queries, keys, values */
+    int q_head_stride, k_offset, k_head_stride, v_offset, v_head_stride, q_row;   /* projection row: queries, keys, values, gate */
+    int map_stride;            /* from a head's first map to its second */
+    int g_offset, g_head_stride;
     int out_head_stride;       /* attention output of a head */
     int64_t page_bytes;
 } gptrs_grouped_attention;
@@ -408,23 +471,29 @@ int gptrs_cuda_delta_rule(const gptrs_delta_rule* a, const gptrs_delta_step* ste
 
 /* ==============================================================================================
  * Mixture of experts: routing and the row order of the grouped matmuls (no counterpart in gpt.rs). Scores are the softmax of the
- * logits over all experts; the experts form `groups` equal groups of neighbours, those of the `keep` groups with the largest best
- * score may be chosen; a row goes to its `top` best experts with their scores as weights.
+ * logits over all experts, or their sigmoids; choices go by the scores plus an optional correction per expert. The experts form
+ * `groups` equal groups of neighbours, those of the `keep` best groups may be chosen (a group counts as much as its best expert, or as
+ * its two best together); a row goes to its `top` best experts with their scores (without the correction) as weights, as they are or
+ * in proportion.
  * ============================================================================================ */
+enum { GPTRS_ROUTE_SOFTMAX = 0, GPTRS_ROUTE_SIGMOID = 1 };
 typedef struct {
     int experts, top, groups, keep;
     int tile_rows;             /* rows of a tile of the grouped matmuls */
+    int scores;                /* GPTRS_ROUTE_* */
+    int group_best;            /* experts that make a group's score: 0 or 1 = its best, 2 = its two best */
+    float weight_scale;        /* 0 = the scores as they are; > 0: score / (sum of the chosen scores + 1e-20) * weight_scale */
 } gptrs_moe;
-/* logits [rows][ld] -> d_pair[rows][top]: the row of x_sorted that belongs to (row, k), sorted by expert; d_weight[rows][top]; the
+/* logits [rows][ld], d_correction [experts] or NULL -> d_pair[rows][top]: the row of x_sorted that belongs to (row, k), sorted by expert; d_weight[rows][top]; the
  * tiles of every expert's rows (at most gptrs_cuda_moe_max_tiles) and their number; d_work: gptrs_cuda_moe_work_ints ints, zeroed
  * before the first call (calls of different configurations may share it). h [rows][ldh] -> d_sorted [rows * top][ldh]. */
 int64_t gptrs_cuda_moe_max_tiles(const gptrs_moe* a, int64_t rows);
 int64_t gptrs_cuda_moe_work_ints(const gptrs_moe* a, int64_t rows);
-int gptrs_cuda_moe_route(const gptrs_moe* a, const float* d_logits, int64_t ld, const void* d_h, int h_dtype, int64_t ldh, int32_t* d_pair,
+int gptrs_cuda_moe_route(const gptrs_moe* a, const float* d_logits, int64_t ld, const float* d_correction, const void* d_h, int h_dtype, int64_t ldh, int32_t* d_pair,
                          float* d_weight, gptrs_row_tile* d_tiles, int32_t* d_n_tiles, void* d_sorted, int32_t* d_work, int64_t rows,
                          void* stream);
-/* f32 mode: y[r][i] = silu(gate) partner over rows of 2 n f32 in the order of the swiglu epilogue, for the first rows of d_tiles. */
-int gptrs_cuda_swiglu_pairs_f32(const float* d_gate_up, float* d_y, int64_t rows, int64_t n, void* stream);
+/* f32 mode: y[r][i] = act(gate) partner over rows of 2 n f32 in the order of the swiglu epilogue; gate = GPTRS_GATE_*. */
+int gptrs_cuda_gated_pairs_f32(const float* d_gate_up, float* d_y, int64_t rows, int64_t n, int gate, void* stream);
 
 /* ==============================================================================================
  * Paged bf16 KV cache and decode attention (split-K flash decoding).
@@ -703,25 +772,31 @@ typedef struct {
 } gptrs_model_config;
 
 /* Layered kind (no counterpart in gpt.rs): every layer has a configuration of its own, a mixer and an optional feed-forward, in
- * one of two block forms:
+ * one of three block forms:
  *   GPTRS_BLOCK_OUTPUT_NORM  norms on the outputs of the sublayers, x <- x + rms(mixer(h)), x <- x + rms(ff(h)); a sublayer reads
  *                            h = x + conv(x), a causal convolution over the last conv_taps positions of every channel whose last
  *                            conv_taps - 1 inputs are part of a sequence's state; the embedding is normed.
  *   GPTRS_BLOCK_SANDWICH     norms on both sides, x <- x + rms(mixer(rms(x))), x <- x + rms(ff(rms(x))); with learned_positions a
  *                            position vector is added to the embedding.
+ *   GPTRS_BLOCK_PRE_NORM     norms in front of the sublayers; the residual is `streams` copies that are mixed at every sublayer
+ *                            (gptrs_stream_step; streams 0: one, x <- x + f(rms(x))); the embedding is scaled by embed_scale.
  * The logits may be soft-capped. Of gptrs_model_config the fields n_layers, d_model, vocab, context_length, norm_eps, max_*,
  * kv_pages and use_pdl apply. Both weight modes keep the cache in pages; rows of a sequence must arrive in order. Pages that the
  * masks of all layers have passed return to the pool. A layer with weights_of >= 0 uses the weights of that layer (an equal
- * configuration) with a cache and state of its own. Parameter names ([out, in] weights): embed, embed.norm | pos,
- * l<i>.norm1, .norm2, .canon1, .canon2 | .norm1b, .norm2b, final.norm, head, and per mixer and feed-forward l<i>.mix. and l<i>.mlp.
- *   latent attention   q, dkv, dkv.norm, uk, uv, o
- *   grouped attention  q, q.b, k, k.b, v, v.b, r1, r2, o, o.b
+ * configuration) with a cache and state of its own; one with kv_from >= 0 (grouped attention) reads the cache of that earlier layer and
+ * projects no keys and values. Parameter names ([out, in] weights): embed, embed.norm | pos,
+ * l<i>.norm1, .norm2, .canon1, .canon2 | .norm1b, .norm2b | .hc1.in, .hc1.out, .hc1.mix, .hc2..., final.norm, head, and per mixer and
+ * feed-forward l<i>.mix. and l<i>.mlp.
+ *   latent attention   q | dq, dq.norm, uq; dkv, dkv.norm, uk, uv, o
+ *   grouped attention  q, q.b, k, k.b, v, v.b, r1, r2, g, lq1, lk1, lq2, lk2, o, o.b
  *   channel delta      q, q.conv, k, k.conv, v, v.conv, b, A_log, a1, a2, dt_bias, g1, g2, norm, o
  *   dense xIELU        up, up.b, down, down.b, act
- *   experts            e<j>.gate, e<j>.up, e<j>.down, router */
+ *   dense gated gelu   gate, up, down
+ *   experts            e<j>.gate, e<j>.up, e<j>.down, router, correction, shared.up, shared.down */
 enum { GPTRS_MIXER_LATENT_ATTENTION = 0, GPTRS_MIXER_GROUPED_ATTENTION = 1, GPTRS_MIXER_CHANNEL_DELTA = 2 };
-enum { GPTRS_MLP_NONE = 0, GPTRS_MLP_DENSE_XIELU = 1, GPTRS_MLP_EXPERTS = 2 };
-enum { GPTRS_BLOCK_OUTPUT_NORM = 0, GPTRS_BLOCK_SANDWICH = 1 };
+enum { GPTRS_MLP_NONE = 0, GPTRS_MLP_DENSE_XIELU = 1, GPTRS_MLP_EXPERTS = 2, GPTRS_MLP_DENSE_GELU = 3 };
+enum { GPTRS_BLOCK_OUTPUT_NORM = 0, GPTRS_BLOCK_SANDWICH = 1, GPTRS_BLOCK_PRE_NORM = 2 };
+enum { GPTRS_EXPERT_SWIGLU = 0, GPTRS_EXPERT_RELU2 = 1 };   /* W_down (silu(W_gate h) * (W_up h)); W_down max(W_up h, 0)^2 */
 typedef struct {
     int mixer;
     int heads, dim, rot_dim, rot_dims, vdim, kv_rank, window;
@@ -733,11 +808,19 @@ typedef struct {
     int taps, decay_rank, gate_rank;                           /* channel delta (kv_heads too) */
     int experts, top, groups, keep;                            /* experts of size d_ff */
     int weights_of;                                            /* -1 = weights of its own */
+    int q_rank;                                                /* latent attention: rank of the query latent, 0 = none */
+    int maps, out_gate, kv_from;                               /* grouped attention: 2 = differential; kv_from -1 = keys of its own */
+    float diff;                                                /* lambda = exp(lq1.lk1) - exp(lq2.lk2) + diff; head_scale = 1 - diff */
+    int expert_form, shared_ff;                                /* GPTRS_EXPERT_*; size of the shared expert, 0 = none */
+    int route, group_best, correction;                         /* as in gptrs_moe; correction 1 = a vector of that name */
+    float weight_scale;
 } gptrs_layer_config;
 typedef struct {
     int conv_taps;
     float logit_softcap;   /* 0 = none */
     int block, learned_positions;
+    int streams;           /* GPTRS_BLOCK_PRE_NORM */
+    float embed_scale;     /* GPTRS_BLOCK_PRE_NORM */
 } gptrs_layered_config;
 
 int gptrs_cuda_model_create(const gptrs_model_config* cfg, gptrs_model** out);

@@ -77,7 +77,7 @@ def test_latent_layout(dtype, want):
     a = _abi.LatentAttention(dtype, 3, 14, 6, 11, 21, 8, 6, 0.25)
     assert gptrs_b200.lib().gptrs_cuda_latent_layout(ctypes.byref(a)) == 0
     assert {k: getattr(a, k) for k in want} == want
-    for bad in (dict(window=0), dict(rot_dims=5), dict(rot_dims=8), dict(scale=0.0), dict(heads=0), dict(kv_rank=2000)):
+    for bad in (dict(window=-1), dict(rot_dims=5), dict(rot_dims=8), dict(scale=0.0), dict(heads=0), dict(kv_rank=2000)):
         b = _abi.LatentAttention(dtype, 3, 14, 6, 11, 21, 8, 6, 0.25)
         for k, v in bad.items():
             setattr(b, k, v)

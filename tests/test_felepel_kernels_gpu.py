@@ -150,7 +150,7 @@ def test_grouped_matmuls(cuda, rows, experts, top, w, f, tile):
         y = ops.dense_bf16(a, _dev(dn, cuda, dt), rows * top, wp, fp, out_f32=True, status=status, **kw)
     else:
         t = ops.dense_f32(srt, _dev(gu.transpose(0, 2, 1), cuda), rows * top, 2 * fp, wp, **kw)
-        a = ops.swiglu_pairs_f32(t, fp)
+        a = ops.gated_pairs_f32(t, fp)
         y = ops.dense_f32(a, _dev(dn.transpose(0, 2, 1), cuda), rows * top, wp, fp, **kw)
     assert int(status) == 0
     pair, a, y = pair.cpu().numpy(), a.float().cpu().numpy(), y.cpu().numpy()

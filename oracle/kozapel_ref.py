@@ -175,3 +175,143 @@ def forward(cfg, tensors, tokens, streams=False):
         after.append(x.sum(axis=0))
     logits = (rms(x.sum(axis=0), eps) * w["final.norm"]) @ w["head"].T
     return (logits, np.stack(after)) if streams else logits
+
+
+# ---- small models for the tests ---------------------------------------------------------------------------------------------
+def dense_mlp(ff=48):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(experts=6, top=2, count=3, keep=2, ff=24, scale=1.7, shared=40):
+    return {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": shared} if shared else None,
+            "router": {"experts": experts, "groups": {"count": count, "keep": keep}, "scale": scale, "top": top}}
+
+
+def latent_layer(heads=4, dim=16, rot_dim=8, vdim=12, kv_rank=24, q_rank=20, base=300.0, scale=None, mlp=dense_mlp()):
+    return {"type": "latent_attention", "mlp": mlp,
+            "mixer": {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "q_rank": q_rank,
+                      "rot": {"base": base, "dims": rot_dim}, "scale": float(scale if scale is not None else (dim + rot_dim) ** -0.5)}}
+
+
+def diff_layer(heads=4, kv_heads=2, dim=16, vdim=24, window=20, diff=0.4, scale=None, kv_from=None, mlp=dense_mlp()):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": window}, "diff": diff,
+         "scale": float(scale if scale is not None else dim ** -0.5)}
+    return {"type": "attention", "mlp": mlp, "mixer": m if kv_from is None else {**m, "kv_from": kv_from}}
+
+
+def model_config(layers, width=40, vocab=72, eps=1e-5, streams=2, embed_scale=3.0):
+    return {"architecture": "Kozapel", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": eps}, "streams": streams,
+            "embedding": {"scale": embed_scale}}
+
+
+def tensor_shapes(cfg):
+    n, v, s = cfg["width"], cfg["vocab"], cfg["streams"]
+    out = {"embed": (v, n)}
+    for i, layer in enumerate(cfg["layers"]):
+        m, p, mlp = layer["mixer"], f"l{i}.", layer["mlp"]
+        x, f = p + "mix.", p + "mlp."
+        for q in (1, 2) if mlp else (1,):
+            out.update({f"{p}norm{q}": (n,), f"{p}hc{q}.in": (s,), f"{p}hc{q}.out": (s,), f"{p}hc{q}.mix": (s, s)})
+        heads, dim, vdim = m["heads"], m["dim"], m["vdim"]
+        if layer["type"] == "latent_attention":
+            rank, rd, qr = m["kv_rank"], m["rot_dim"], m["q_rank"]
+            out.update({x + "dq": (qr, n), x + "dq.norm": (qr,), x + "uq": (heads * (dim + rd), qr), x + "dkv": (rank + rd, n), x + "dkv.norm": (rank,),
+                        x + "uk": (heads * dim, rank), x + "uv": (heads * vdim, rank)})
+        else:
+            out.update({x + "q": (heads * 2 * dim, n), x + "g": (heads * vdim, n), **{x + a: (dim,) for a in ("lq1", "lk1", "lq2", "lk2")}})
+            if "kv_from" not in m:
+                out.update({x + "k": (m["kv_heads"] * 2 * dim, n), x + "v": (m["kv_heads"] * vdim, n)})
+        out[x + "o"] = (n, heads * vdim)
+        if mlp and mlp["kind"] == "dense":
+            out.update({f + "gate": (mlp["ff"], n), f + "up": (mlp["ff"], n), f + "down": (n, mlp["ff"])})
+        elif mlp:
+            names = [f"e{e}." for e in range(mlp["router"]["experts"])]
+            for name, ff in [(a, mlp["expert"]["ff"]) for a in names] + ([("shared.", mlp["shared"]["ff"])] if mlp["shared"] else []):
+                out.update({f + name + "up": (ff, n), f + name + "down": (n, ff)})
+            out.update({f + "router": (mlp["router"]["experts"], n), f + "correction": (mlp["router"]["experts"],)})
+    out.update({"final.norm": (n,), "head": (v, n)})
+    return out
+
+
+def random_tensors(cfg, seed=0, sharp=1.0):
+    """bfloat16-valued weights; norm gains around 1, projections of unit output scale (queries times `sharp`), streams that differ, choices
+    that the correction changes (some of them negative)."""
+    rng = np.random.default_rng(seed)
+    out = {}
+    for name, shape in tensor_shapes(cfg).items():
+        last = name.rsplit(".", 1)[-1]
+        if "norm" in last:
+            w = 1.0 + 0.2 * rng.standard_normal(shape)
+        elif ".hc" in name:
+            w = 0.25 * rng.standard_normal(shape)
+            w += np.eye(*shape) if last == "mix" else 1.0 / shape[0] if last == "in" else 0.8
+        elif last in ("lq1", "lk1", "lq2", "lk2"):
+            w = 0.6 * rng.standard_normal(shape) / shape[0] ** 0.25
+        elif last == "correction":
+            w = rng.uniform(-0.9, 0.3, shape)
+        elif last == "router":
+            w = 2.0 * rng.standard_normal(shape) / np.sqrt(shape[-1])
+        elif name == "embed":
+            w = 0.4 * rng.standard_normal(shape)
+        else:
+            w = rng.standard_normal(shape) / np.sqrt(shape[-1]) * (sharp if last in ("q", "uq") else 1.0)
+        out[name] = to_bf16(w.astype(np.float32))
+    return out
+
+
+CODE = 8   # width reserved by `steady_routing`
+
+
+def steady_routing(cfg, tensors, seed=0, margin=0.02):
+    """Weights whose routers read the last CODE channels of the streams only, which no sublayer adds to, so that there every token keeps a
+    code of its own times a number that depends on the layer. Codes are drawn so that no choice of experts or groups is close, whatever
+    the norm makes of their size within a wide range: rounding then never changes an expert."""
+    rng = np.random.default_rng(seed)
+    t = {n: w.copy() for n, w in tensors.items()}
+    coef, routers = np.ones(cfg["streams"]), []
+    for i, layer in enumerate(cfg["layers"]):
+        t[f"l{i}.mix.o"][-CODE:] = 0
+        for n in t:
+            if n.startswith(f"l{i}.mlp.") and n.endswith("down"):
+                t[n][-CODE:] = 0
+        for q in (1, 2) if layer["mlp"] else (1,):
+            if q == 2 and layer["mlp"]["kind"] == "moe":
+                # inputs scaled so that the code arrives with the size of the embedding, whatever the mixing has made of it
+                w_in = t[f"l{i}.hc2.in"]
+                t[f"l{i}.hc2.in"] = to_bf16(w_in / np.float32(w_in @ coef)) if abs(w_in @ coef) > 0.2 else to_bf16(np.float32(coef / (coef @ coef)))
+                t[f"l{i}.norm2"][-CODE:] = 1
+                w = t[f"l{i}.mlp.router"]
+                w[:, :-CODE] = 0
+                w[:, -CODE:] = to_bf16((1.5 * rng.standard_normal((w.shape[0], CODE))).astype(np.float32))
+                routers.append((w[:, -CODE:].astype(D), t[f"l{i}.mlp.correction"].astype(D), layer["mlp"]["router"]))
+            coef = t[f"l{i}.hc{q}.mix"].astype(D).T @ coef
+
+    def picks(codes, w, corr, r):
+        """Chosen experts [N][E] (bool) and whether nothing was close."""
+        g = r["groups"]
+        choice = sigmoid(codes @ w.T) + corr
+        groups = choice.reshape(len(codes), g["count"], -1)
+        score = np.sort(groups, axis=2)[:, :, -2:].sum(axis=2)
+        order = np.sort(score, axis=1)[:, ::-1]
+        ok = order[:, g["keep"] - 1] - order[:, g["keep"]] > margin if g["keep"] < g["count"] else np.full(len(codes), True)
+        allowed = np.where((score >= order[:, [g["keep"] - 1]])[:, :, None], groups, -np.inf).reshape(len(codes), -1)
+        best = np.sort(allowed, axis=1)[:, ::-1]
+        if r["top"] < allowed.shape[1]:
+            ok &= best[:, r["top"] - 1] - best[:, r["top"]] > margin
+        return allowed >= best[:, [r["top"] - 1]], ok
+
+    drawn = rng.standard_normal((60000, CODE))
+    drawn *= 0.8 * CODE ** 0.5 / np.linalg.norm(drawn, axis=1, keepdims=True)
+    drawn = to_bf16(drawn.astype(np.float32))
+    good = np.full(len(drawn), True)
+    for w, corr, r in routers:
+        first = None
+        for size in (0.35, 0.5, 0.7, 1.0, 1.4, 2.0):
+            chosen, ok = picks(drawn * size, w, corr, r)
+            first = chosen if first is None else first
+            good &= ok & (chosen == first).all(axis=1)
+    codes = drawn[good]
+    if len(codes) < cfg["vocab"]:
+        raise ValueError(f"only {len(codes)} codes with this margin")
+    t["embed"][:, -CODE:] = to_bf16(codes[:cfg["vocab"]] * np.float32(1.5 / cfg["embedding"]["scale"]))
+    return t

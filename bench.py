@@ -307,6 +307,8 @@ def _random_model(gm, torch, dev, cfg, namespace):
         last = name.rsplit(".", 1)[-1]
         if name.endswith("gamma") or "norm" in last:
             t = torch.ones(shape, device=dev)
+        elif ".hc" in name:   # residual streams that keep themselves, read as their mean
+            t = torch.eye(shape[0], device=dev) if last == "mix" else torch.full(shape, 1.0 / shape[0] if last == "in" else 1.0, device=dev)
         elif last in ("r1", "r2", "dt_bias"):   # distance penalties are positive, decays slow
             t = torch.full(shape, -3.0 if last == "dt_bias" else 0.3, device=dev)
         else:
@@ -667,6 +669,186 @@ def run_felepel_kernels(args, out, ops, torch):
         if only is None:   # the like kernels of Bevosun
             rec["sizes"][name].update(like_decode=time_layered_kernels(ops, torch, dev, LAYERED_SIZES[name], BATCH),
                                       like_prefill=time_layered_kernels(ops, torch, dev, LAYERED_SIZES[name], 4 * PROMPT_LEN))
+        torch.cuda.empty_cache()
+    print(json.dumps(rec), file=out)
+
+
+# ---- Kozapel beside Felepel and Bevosun --------------------------------------------------------------------------------------------
+# name -> differential attention (heads, kv heads, dim of a part, vdim, window), latent attention (heads, dim, rot, vdim, kv rank, q rank),
+# experts (number, top, groups, kept groups, size, size of the shared one), dense size, streams; width and vocabulary as in LAYERED_SIZES
+KOZAPEL_SIZES = {
+    "w1024": ((8, 2, 64, 128, 1024), (16, 64, 32, 64, 128, 384), (16, 4, 4, 2, 768, 768), 3072, 4),
+    "w2048": ((16, 4, 64, 128, 2048), (16, 128, 64, 128, 256, 768), (32, 6, 4, 2, 1024, 1024), 6144, 4),
+    "w3072": ((32, 8, 64, 128, 4096), (32, 96, 32, 96, 256, 1024), (64, 6, 8, 4, 1536, 1536), 9216, 4),
+}
+
+
+def _kozapel_model(gm, torch, dev, name, n_layers, ctx, pdl, chunk, batch):
+    width, vocab = LAYERED_SIZES[name][0], LAYERED_SIZES[name][8]
+    (h, g, d, v, size), (lh, ld, lr, lv, rank, q_rank), (experts, top, groups, keep, eff, shared), ff, streams = KOZAPEL_SIZES[name]
+    dense = dict(mlp=gm.MLP_DENSE_GELU, d_ff=ff)
+    moe = dict(mlp=gm.MLP_EXPERTS, expert_form=gm.EXPERT_RELU2, d_ff=eff, experts=experts, top=top, groups=groups, keep=keep, route=gm.ROUTE_SIGMOID, group_best=2, correction=1,
+               weight_scale=2.0, shared_ff=shared)
+    att = dict(heads=h, kv_heads=g, dim=d, vdim=v, scale=d ** -0.5, mask=gm.MASK_WINDOW, mask_size=size, maps=2, out_gate=1, diff=0.5, mixer=gm.MIXER_GROUPED_ATTENTION)
+    lat = dict(heads=lh, dim=ld, rot_dim=lr, vdim=lv, kv_rank=rank, q_rank=q_rank, scale=(ld + lr) ** -0.5, rope_base=1e6, mixer=gm.MIXER_LATENT_ATTENTION)
+    layers = [gm.LayerConfig(**att, **dense), gm.LayerConfig(**lat, **moe), gm.LayerConfig(**att, kv_from=0, **moe), gm.LayerConfig(**lat, **dense)]
+    pages = (ctx + 15) // 16
+    cfg = gm.ModelConfig.layered([layers[i % 4] for i in range(n_layers)], width, vocab, ctx, 1e-6, block=gm.BLOCK_PRE_NORM, streams=streams, embed_scale=12.0, weight_mode=gm.MODE_BF16,
+                                 max_seqs=batch, max_tokens=chunk, max_logit_rows=batch, kv_pages=batch * pages + 8, max_pages_per_seq=pages, use_pdl=pdl)
+    return _random_model(gm, torch, dev, cfg, 74)
+
+
+def run_kozapel(args, out, gm, torch, np):
+    """Prefill and decode of Kozapel (differential and latent attention in turn, dense and expert feed-forwards, four residual streams;
+    random weights, bf16) beside Felepel and Bevosun of the same width and depth. Not the default line."""
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    n_layers, batch, prompt = 4, BATCH, PROMPT_LEN
+    ctx = prompt + args.steps + args.warmup + 32
+    rec = {"workload": "kozapel", "layers": n_layers, "batch": batch, "prompt_tokens": prompt, "steps": args.steps, "warmup": args.warmup, "data": "synthetic", "sizes": {}}
+    sampler = ClockSampler(None)
+    sampler.start()
+    for name in args.sizes.split(","):
+        row = {"kozapel": dict(zip(("attention", "latent", "experts", "ff", "streams"), KOZAPEL_SIZES[name])), "felepel": {}, "bevosun": {"width": LAYERED_SIZES[name][0]}}
+        builds = (("kozapel", lambda *a: _kozapel_model(gm, torch, dev, name, *a)), ("felepel", lambda *a: _felepel_model(gm, torch, dev, name, *a)),
+                  ("bevosun", lambda *a: _layered_model(gm, torch, dev, LAYERED_SIZES[name], *a)))
+        for kind, build in builds:
+            m = build(n_layers, ctx, args.pdl, 2048 if kind == "bevosun" else 8192, batch)
+            row[kind].update(_model_speed(gm, torch, np, dev, m, prompt, batch, args.steps, args.warmup))
+            m.close()
+            torch.cuda.empty_cache()
+        rec["sizes"][name] = row
+    rec["clocks"] = sampler.stop()
+    print(json.dumps(rec), file=out)
+
+
+def time_kozapel_kernels(ops, torch, dev, name, rows, ctx_len=PROMPT_LEN, only=None):
+    """Every kernel of Kozapel's layers by itself at `rows` tokens, as time_layered_kernels does it. Differential attention counts, per
+    visible pair and head, both scores and both sums over the values."""
+    w = LAYERED_SIZES[name][0]
+    (heads, kv, dim, vdim, size), (lh, ld, lr, lv, rank, q_rank), (experts, top, groups, keep, eff, shared), ff, streams = KOZAPEL_SIZES[name]
+    decode = rows <= 128
+    hbm, tf = _peaks()[0], _tensor_peak()
+    res = {}
+
+    def put(label, us, nbytes, flops):
+        t_mem, t_op = nbytes / hbm / 1e3, flops / tf / 1e6
+        res[label] = {"us": round(us, 2), "roofline_us": round(max(t_mem, t_op), 2), "bound": "hbm" if t_mem > t_op else "tensor", "frac": round(max(t_mem, t_op) / us, 3)}
+
+    bf, i32 = torch.bfloat16, torch.int32
+    status = torch.zeros(1, dtype=i32, device=dev)
+    want = lambda label: only is None or label in only  # noqa: E731
+
+    def gemm(label, n, k, batch=1, ldx=None, x_step=0, ldy=None, y_step=0, out_f32=False, gate=0, **kw):
+        if not want(label):
+            return
+        n8, k8 = (n + 7) // 8 * 8, (k + 7) // 8 * 8
+        per = batch * n8 * k8 * 2
+        mats = [torch.randn(batch, n8, k8, device=dev).mul_(k8 ** -0.5).to(bf) for _ in range(max(2, min(24, (300 << 20) // per)))]
+        x = torch.randn(rows, ldx or k8, device=dev).to(bf)
+        n_out = n8 // 2 if gate else n8
+        y = torch.empty(rows, ldy or n_out, device=dev, dtype=torch.float32 if out_f32 else bf)
+        st = dict(ldx=ldx or k8, ldy=ldy or n8, batch=batch, x_step=x_step, y_step=y_step) if batch > 1 else {"ldx": ldx} if ldx else {}
+        us = _graph_us(torch, [lambda m=m: ops.dense_bf16(x, m, rows, n8, k8, out=y, out_f32=out_f32, swiglu=gate, status=status, **st, **kw) for m in mats])
+        put(label, us, per + rows * batch * (k8 + n_out * (2 if out_f32 else 1)) * 2, 2.0 * rows * n8 * k8 * batch)
+
+    win = dict(maps=2, gate=True, lam=0.7, head_scale=0.5, head_eps=1e-6)
+    a, shared_a = (ops.grouped_layout(heads, kv, dim, vdim, 1, size, dim ** -0.5, shared_kv=f, **win) for f in (False, True))
+    b = ops.latent_layout(lh, ld, lr, lv, rank, 0, (ld + lr) ** -0.5, q_rank=q_rank)
+    gemm("qkvg", a.q_row, w)
+    gemm("qg", shared_a.q_row, w)
+    gemm("out", w, heads * a.out_head_stride)
+    gemm("latent_in", b.kv_row, w)
+    gemm("latent_uq", b.q_row, q_rank)
+    gemm("absorb_q", b.lat_head_stride, ld, lh, b.q_row, b.q_head_stride, lh * b.qa_head_stride, b.qa_head_stride)
+    gemm("absorb_v", b.out_head_stride, b.lat_head_stride, lh, lh * b.lat_head_stride, b.lat_head_stride, lh * b.out_head_stride, b.out_head_stride)
+    gemm("latent_out", w, lh * b.out_head_stride)
+    gemm("gated_up", 2 * ff, w, gate=ops.GATE_GELU_TANH)
+    gemm("down", w, ff)
+    gemm("shared_up", shared, w, relu2=True)
+    gemm("shared_down", w, shared)
+    gemm("router", experts, w, out_f32=True)
+
+    seqs = rows if decode else rows // ctx_len
+    per_seq, pages = rows // seqs, (ctx_len + 15) // 16
+    slot = torch.arange(seqs, dtype=i32, device=dev).repeat_interleave(per_seq).contiguous()
+    pos = (torch.full((rows,), ctx_len - 1, device=dev) if decode else torch.arange(ctx_len, device=dev).repeat(seqs)).to(i32)
+    ctx = (pos + 1).to(i32)
+    table = torch.randperm(seqs * pages, device=dev, dtype=i32).view(seqs, pages).contiguous()
+
+    def tiles(t):
+        first = torch.cat([torch.arange(0, per_seq, t, device=dev) + s * per_seq for s in range(seqs)]).to(i32)
+        return first, torch.minimum(torch.full_like(first, t), per_seq - first % per_seq).to(i32)
+
+    def pools(page_bytes):
+        return [torch.randn(seqs * pages * page_bytes // 2, device=dev).to(bf) for _ in range(4 if decode else 1)]
+
+    if want("attention") or want("append"):
+        qkv, store, ts = torch.randn(rows, a.q_row, device=dev).to(bf), pools(a.page_bytes), tiles(1 if decode else ops.grouped_tile_tokens(a))
+        us = _graph_us(torch, [lambda p=p: ops.grouped_attention(a, qkv, p, table, slot, ctx, ctx_len, tiles=ts, status=status) for p in store] * (4 if decode else 2))
+        seen = torch.minimum(ctx, torch.full_like(ctx, size)).double()
+        cache = float(seen.sum()) if decode else rows
+        put("attention", us, cache * kv * (2 * dim + vdim) * 2 + rows * heads * (2 * dim + 2 * vdim) * 2, 2.0 * heads * 2 * (dim + vdim) * float(seen.sum()))
+        us = _graph_us(torch, [lambda p=p: ops.grouped_append(a, qkv, pos, slot, table, p) for p in store] * 4)
+        put("append", us, rows * kv * (2 * dim + vdim) * 4, 0)
+        del store
+    if want("latent_attention") or want("latent_keys"):
+        qa, store, ts = torch.randn(rows, lh, b.qa_head_stride, device=dev).to(bf), pools(b.page_bytes), tiles(1 if decode else ops.latent_tile_tokens(b))
+        us = _graph_us(torch, [lambda p=p: ops.latent_attention(b, qa, p, table, slot, ctx, ctx_len, tiles=ts, status=status) for p in store] * (4 if decode else 2))
+        cache, pairs = (float(ctx.double().sum()) if decode else rows), float(ctx.double().sum())
+        put("latent_attention", us, cache * (rank + lr) * 2 + rows * lh * (2 * rank + lr) * 2, 2.0 * lh * (2 * rank + lr) * pairs)
+        kvr, q = torch.randn(rows, b.kv_row, device=dev).to(bf), torch.randn(rows, b.q_row, device=dev).to(bf)
+        cs, sn = torch.randn(ctx_len, lr // 2, device=dev), torch.randn(ctx_len, lr // 2, device=dev)
+        nw, qw = torch.ones(rank, device=dev), torch.ones(q_rank, device=dev)
+        us = _graph_us(torch, [lambda p=p: ops.latent_append_keys(b, kvr, pos, slot, table, nw, qw, 1e-6, cs, sn, p) for p in store] * 4)
+        put("latent_keys", us, rows * (b.kv_row + b.q_latent_row + rank + lr) * 2, 0)
+        us = _graph_us(torch, [lambda: ops.latent_rotate_queries(b, q, pos, cs, sn, qa)] * 8)
+        put("latent_queries", us, rows * lh * lr * 4, 0)
+        del store
+    x, y = torch.randn(rows, streams, w, device=dev), torch.randn(rows, w, device=dev).to(bf)
+    gamma, mix, vec = torch.ones(w, device=dev), torch.eye(streams, device=dev), torch.full((streams,), 0.25, device=dev)
+    if want("stream_step"):
+        us = _graph_us(torch, [lambda: ops.stream_step(x, 1e-6, y=y, mix=mix, w_out=vec, w_in=vec, gamma_in=gamma, out_dtype=bf, status=status)] * 8)
+        put("stream_step", us, rows * w * (8 * streams + 4), 0)
+    if want("experts") or want("route"):
+        mean = rows * top / experts
+        tile = 16 if mean <= 8 else 32 if mean <= 24 else 64 if mean <= 48 else 128
+        z, corr = torch.randn(rows, experts, device=dev), 0.1 * torch.randn(experts, device=dev)
+        route = dict(sigmoid=True, group_best=2, weight_scale=2.0, correction=corr)
+        us = _graph_us(torch, [lambda: ops.moe_route(experts, top, groups, keep, tile, z, y, **route)] * 4)
+        put("route", us, rows * experts * 4 + rows * w * 2 * (1 + top), 0)
+        pair, weight, row_tiles, n_tiles, srt, most = ops.moe_route(experts, top, groups, keep, tile, z, y, **route)
+        per = experts * 2 * eff * w * 2
+        active = int((torch.zeros(experts, device=dev).index_add_(0, row_tiles[:int(n_tiles), 0].long(), torch.ones(int(n_tiles), device=dev)) > 0).sum())
+        copies = 2 if per > (100 << 20) else 6
+        kw = dict(tiles=row_tiles, n_tiles=n_tiles, max_tiles=most, tile_rows=tile, batch=experts, status=status)
+        mid, ey = torch.empty(rows * top, eff, device=dev, dtype=bf), torch.empty(rows * top, w, device=dev, dtype=bf)
+        ups = [torch.randn(experts, eff, w, device=dev).mul_(w ** -0.5).to(bf) for _ in range(copies)]
+        us = _graph_us(torch, [lambda m=m: ops.dense_bf16(srt, m, rows * top, eff, w, out=mid, relu2=True, **kw) for m in ups] * 2)
+        put("experts_up", us, active * eff * w * 2 + rows * top * (w + eff) * 2, 2.0 * rows * top * eff * w)
+        del ups
+        downs = [torch.randn(experts, w, eff, device=dev).mul_(eff ** -0.5).to(bf) for _ in range(copies)]
+        us = _graph_us(torch, [lambda m=m: ops.dense_bf16(mid, m, rows * top, w, eff, out=ey, **kw) for m in downs] * 2)
+        put("experts_down", us, active * eff * w * 2 + rows * top * (w + eff) * 2, 2.0 * rows * top * eff * w)
+        del downs
+        us = _graph_us(torch, [lambda: ops.stream_step(x, 1e-6, y=ey, mix=mix, w_out=vec, w_in=vec, gamma_in=gamma, pair=pair, pair_weight=weight, add=y, out_dtype=bf, status=status)] * 4)
+        put("stream_step_experts", us, rows * w * (8 * streams + 2 * top + 2 + 2), 0)
+    assert int(status) == 0
+    return res
+
+
+def run_kozapel_kernels(args, out, ops, torch):
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    rec = {"microbench": "kozapel", "decode_rows": BATCH, "ctx": PROMPT_LEN, "prefill_rows": 4 * PROMPT_LEN, "sizes": {}}
+    only = args.only.split(",") if args.only else None
+    for name in args.sizes.split(","):
+        row = rec["sizes"][name] = {}
+        for phase, rows in (("decode", BATCH), ("prefill", 4 * PROMPT_LEN)):
+            row[phase] = time_kozapel_kernels(ops, torch, dev, name, rows, only=only)
+            if only is None:   # the like kernels of Felepel and Bevosun
+                row[f"felepel_{phase}"] = time_felepel_kernels(ops, torch, dev, name, rows)
+                row[f"bevosun_{phase}"] = time_layered_kernels(ops, torch, dev, LAYERED_SIZES[name], rows)
         torch.cuda.empty_cache()
     print(json.dumps(rec), file=out)
 
@@ -1096,17 +1278,17 @@ def _main(out):
     ap.add_argument("--pdl", type=int, default=int(os.environ.get("GPTRS_PDL", "1")))
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-extras", action="store_true", help="skip the kernel microbenchmarks")
-    ap.add_argument("--microbench", default=None, choices=["attention", "attention-ragged", "gemv", "gemv-lm-head", "gemm64", "quant-linear", "prefill", "prefill-attention", "layered", "felepel"],
+    ap.add_argument("--microbench", default=None, choices=["attention", "attention-ragged", "gemv", "gemv-lm-head", "gemm64", "quant-linear", "prefill", "prefill-attention", "layered", "felepel", "kozapel"],
                     help="run only one kernel microbenchmark (used for ncu captures) and print its JSON")
     ap.add_argument("--ctx", type=int, default=PROMPT_LEN + 20, help="context length for --microbench attention")
-    ap.add_argument("--workload", default="ministral3b-w4", choices=["ministral3b-w4", "gpt2-fp32", "dp512", "bevosun", "felepel"],
+    ap.add_argument("--workload", default="ministral3b-w4", choices=["ministral3b-w4", "gpt2-fp32", "dp512", "bevosun", "felepel", "kozapel"],
                     help="gpt2-fp32 = the reference's CPU-runnable case (one sequence, 32-token prompt, 64 greedy tokens); "
                          "dp512 = 512 requests with prompt lengths U{256..4096}, 256 decode steps each, partitioned over the ranks "
                          "(total work fixed: strong scaling; not the default line); "
                          "bevosun = prefill and decode of the layered kind at three sizes beside the Ministral-shaped model of equal size; "
-                         "felepel = the same for Felepel beside Bevosun")
-    ap.add_argument("--sizes", default="w1024,w2048,w3072", help="felepel: comma list of sizes")
-    ap.add_argument("--only", default="", help="--microbench felepel: comma list of kernels (attention, append, delta_rule, norm_step, experts, route, or a matmul)")
+                         "felepel = the same for Felepel beside Bevosun; kozapel = the same for Kozapel beside both")
+    ap.add_argument("--sizes", default="w1024,w2048,w3072", help="felepel, kozapel: comma list of sizes")
+    ap.add_argument("--only", default="", help="--microbench felepel, kozapel: comma list of kernels (attention, append, delta_rule, norm_step, experts, route, or a matmul)")
     ap.add_argument("--path", default="engine", choices=["engine", "run_program"],
                     help="gpt2-fp32 only: engine = the model-level ABI (default); run_program = every decode step one "
                          "PortableBackend::run_program call on the captured decode program")
@@ -1145,6 +1327,12 @@ def _main(out):
         return
     if args.microbench == "felepel":
         run_felepel_kernels(args, out, ops, torch)
+        return
+    if args.microbench == "kozapel":
+        run_kozapel_kernels(args, out, ops, torch)
+        return
+    if args.workload == "kozapel":
+        run_kozapel(args, out, gm, torch, np)
         return
     if args.workload == "felepel":
         run_felepel(args, out, gm, torch, np)

@@ -9,6 +9,7 @@
 // front of and behind the kernels of this file. Where queries come through a latent of their own, the first projection gives both
 // latents, and the kernel that writes the page also norms the query latent for the second projection:
 //   latent_append_kernel        norm of the latent(s), rotation of the shared key part and of the queries, page write
+//   latent_keys_kernel          its first half for bf16 rows with a query latent
 //   latent_attention_kernel     plain CUDA-core attention, f32 or bf16 cache, any sizes (the f32 path)
 //   flash_tc_kernel             tcgen05 flash attention (flash_tc.cuh), bf16, prompts and decode steps alike, kv_rank up to 256
 //
@@ -55,6 +56,7 @@ struct AppendParams {
     unsigned char* pool;
     int max_pages;
     float eps;
+    int rows;
 };
 
 constexpr int kAppendThreads = 128;
@@ -178,6 +180,89 @@ __global__ void __launch_bounds__(kAppendThreads) latent_append_kernel(const App
             const int h = j / g.rot, c = j % g.rot;
             rotate(q + h * g.q_head_stride + g.dim, reinterpret_cast<float*>(qa) + (size_t)h * g.qa_head_stride + g.qa_rot_off, c);
         }
+    }
+}
+
+// KEYS of a bf16 model alone, a warp per row with the row in registers: all loads are under way before the first one is needed (the norms'
+// gains before the kernel in front has ended), and no barrier is.
+constexpr int kKeyRows = 4;          // rows of a CTA
+constexpr int kLatChunks = 4;        // 16-byte chunks per lane: kv_rank up to 1024
+constexpr int kQueryChunks = 8;      // query latents of up to 2048 values
+__device__ __forceinline__ void unpack8(const uint4& u, float (&v)[8]) {
+    v[0] = bf16_lo(u.x); v[1] = bf16_hi(u.x); v[2] = bf16_lo(u.y); v[3] = bf16_hi(u.y);
+    v[4] = bf16_lo(u.z); v[5] = bf16_hi(u.z); v[6] = bf16_lo(u.w); v[7] = bf16_hi(u.w);
+}
+// eight values from column c0 on, of which those before n count: the sum of their squares; the normed values, zeros from n on
+__device__ __forceinline__ float squares8(const uint4& u, int c0, int n) {
+    float v[8], s = 0.f;
+    unpack8(u, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) s = c0 + e < n ? fmaf(v[e], v[e], s) : s;
+    return s;
+}
+__device__ __forceinline__ uint4 normed8(const uint4& u, int c0, int n, float inv, const float (&w)[8]) {
+    float v[8];
+    unpack8(u, v);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] = c0 + e < n ? v[e] * inv * w[e] : 0.f;
+    return pack8(v);
+}
+// eight gains from column c0 on (zeros from n on)
+__device__ __forceinline__ void gains8(const float* w, int c0, int n, float (&v)[8]) {
+    if (c0 + 8 <= n) {
+        const float4 a = __ldg(reinterpret_cast<const float4*>(w + c0)), b = __ldg(reinterpret_cast<const float4*>(w + c0) + 1);
+        v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+    } else {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) v[e] = c0 + e < n ? __ldg(w + c0 + e) : 0.f;
+    }
+}
+
+// LC, QC: chunks per lane of the latent and of the query latent
+template <int LC, int QC>
+__global__ void __launch_bounds__(kKeyRows * 32) latent_keys_kernel(const AppendParams p) {
+    const Geometry& g = p.g;
+    const int lane = threadIdx.x & 31, row = blockIdx.x * kKeyRows + (threadIdx.x >> 5);
+    pdl_launch_dependents();
+    float wl[LC][8], wq[QC][8];
+#pragma unroll
+    for (int i = 0; i < LC; ++i) gains8(p.norm_w, (i * 32 + lane) * 8, g.rank, wl[i]);
+#pragma unroll
+    for (int i = 0; i < QC; ++i) gains8(p.q_norm_w, (i * 32 + lane) * 8, g.q_rank, wq[i]);
+    pdl_wait();
+    if (row >= p.rows) return;
+    const int pos = p.pos[row], slot = p.slot[row];
+    const __nv_bfloat16* kv = static_cast<const __nv_bfloat16*>(p.kv) + (size_t)row * g.kv_row;
+    const uint4* lat = reinterpret_cast<const uint4*>(kv + g.dkv_off);
+    const int n_q = g.q_latent_row / 8, n_lat = up(g.rank, 8) / 8;
+    uint4 q[QC], l[LC];
+#pragma unroll
+    for (int i = 0; i < LC; ++i) l[i] = i * 32 + lane < n_lat ? lat[i * 32 + lane] : make_uint4(0, 0, 0, 0);
+#pragma unroll
+    for (int i = 0; i < QC; ++i) q[i] = i * 32 + lane < n_q ? reinterpret_cast<const uint4*>(kv)[i * 32 + lane] : make_uint4(0, 0, 0, 0);
+    unsigned char* page = p.pool + (size_t)p.page_table[(size_t)slot * p.max_pages + pos / kPageTok] * g.page_bytes;
+    const int t = pos % kPageTok;
+    for (int j = lane; j < (g.nb - g.nbc) * 8; j += 32) {
+        float v[8];
+        rotated8(kv + g.rot_off, j, g.rot, g.rot_pairs, p.cos_t + (size_t)pos * g.rot_pairs, p.sin_t + (size_t)pos * g.rot_pairs, v);
+        *reinterpret_cast<uint4*>(page + page_chunk(t, g.nbc * 8 + j, g.nb)) = pack8(v);
+    }
+    float sl = 0.f, sq = 0.f;
+#pragma unroll
+    for (int i = 0; i < LC; ++i) sl += squares8(l[i], (i * 32 + lane) * 8, g.rank);
+#pragma unroll
+    for (int i = 0; i < QC; ++i) sq += squares8(q[i], (i * 32 + lane) * 8, g.q_rank);
+    const float inv_l = 1.f / sqrtf(warp_sum(sl) / (float)g.rank + p.eps), inv_q = 1.f / sqrtf(warp_sum(sq) / (float)g.q_rank + p.eps);
+#pragma unroll
+    for (int i = 0; i < LC; ++i) {
+        const int j = i * 32 + lane;
+        if (j < g.nbc * 8) *reinterpret_cast<uint4*>(page + page_chunk(t, j, g.nb)) = normed8(l[i], j * 8, g.rank, inv_l, wl[i]);
+    }
+    uint4* ql = reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(p.q_latent) + (size_t)row * g.q_latent_row);
+#pragma unroll
+    for (int i = 0; i < QC; ++i) {
+        const int j = i * 32 + lane;
+        if (j < n_q) ql[j] = normed8(q[i], j * 8, g.q_rank, inv_q, wq[i]);
     }
 }
 
@@ -370,6 +455,14 @@ int gptrs_cuda_latent_append_keys(const gptrs_latent_attention* a, const void* d
     AppendParams p = {};
     p.g = geometry(*a); p.kv = d_kv; p.pos = d_positions; p.slot = d_slot; p.page_table = d_page_table; p.norm_w = d_norm_w; p.q_norm_w = d_q_norm_w;
     p.cos_t = d_cos; p.sin_t = d_sin; p.q_latent = d_q_latent; p.pool = static_cast<unsigned char*>(d_pool); p.max_pages = (int)max_pages; p.eps = eps;
+    const bool aligned = ((reinterpret_cast<uintptr_t>(d_norm_w) | reinterpret_cast<uintptr_t>(d_q_norm_w) | reinterpret_cast<uintptr_t>(d_kv) | reinterpret_cast<uintptr_t>(d_q_latent)) & 15) == 0;
+    p.rows = (int)n_tokens;
+    if (a->dtype == GPTRS_BF16 && aligned && a->q_rank <= kQueryChunks * 256) {
+        const dim3 grid((unsigned)ceil_div((int)n_tokens, kKeyRows));
+        void (*kern)(AppendParams) = a->kv_rank > 256 ? latent_keys_kernel<kLatChunks, kQueryChunks> : a->q_rank <= 512 ? latent_keys_kernel<1, 2>
+                                   : a->q_rank <= 1024 ? latent_keys_kernel<1, 4> : latent_keys_kernel<1, kQueryChunks>;
+        return launch_kernel(kern, grid, dim3(kKeyRows * 32), 0, as_stream(stream), 1, p);
+    }
     return launch_append<true, false>(a, p, n_tokens, stream);
 }
 

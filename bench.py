@@ -688,12 +688,12 @@ def _kozapel_model(gm, torch, dev, name, n_layers, ctx, pdl, chunk, batch):
     (h, g, d, v, size), (lh, ld, lr, lv, rank, q_rank), (experts, top, groups, keep, eff, shared), ff, streams = KOZAPEL_SIZES[name]
     dense = dict(mlp=gm.MLP_DENSE_GELU, d_ff=ff)
     moe = dict(mlp=gm.MLP_EXPERTS, expert_form=gm.EXPERT_RELU2, d_ff=eff, experts=experts, top=top, groups=groups, keep=keep, route=gm.ROUTE_SIGMOID, group_best=2, correction=1,
-               weight_scale=2.0, shared_ff=shared)
-    att = dict(heads=h, kv_heads=g, dim=d, vdim=v, scale=d ** -0.5, mask=gm.MASK_WINDOW, mask_size=size, maps=2, out_gate=1, diff=0.5, mixer=gm.MIXER_GROUPED_ATTENTION)
+               weight_scale=1.5, shared_ff=shared)
+    att = dict(heads=h, kv_heads=g, dim=d, vdim=v, scale=d ** -0.5, mask=gm.MASK_WINDOW, mask_size=size, maps=2, out_gate=1, diff=0.3, mixer=gm.MIXER_GROUPED_ATTENTION)
     lat = dict(heads=lh, dim=ld, rot_dim=lr, vdim=lv, kv_rank=rank, q_rank=q_rank, scale=(ld + lr) ** -0.5, rope_base=1e6, mixer=gm.MIXER_LATENT_ATTENTION)
     layers = [gm.LayerConfig(**att, **dense), gm.LayerConfig(**lat, **moe), gm.LayerConfig(**att, kv_from=0, **moe), gm.LayerConfig(**lat, **dense)]
     pages = (ctx + 15) // 16
-    cfg = gm.ModelConfig.layered([layers[i % 4] for i in range(n_layers)], width, vocab, ctx, 1e-6, block=gm.BLOCK_PRE_NORM, streams=streams, embed_scale=12.0, weight_mode=gm.MODE_BF16,
+    cfg = gm.ModelConfig.layered([layers[i % 4] for i in range(n_layers)], width, vocab, ctx, 1e-6, block=gm.BLOCK_PRE_NORM, streams=streams, embed_scale=8.0, weight_mode=gm.MODE_BF16,
                                  max_seqs=batch, max_tokens=chunk, max_logit_rows=batch, kv_pages=batch * pages + 8, max_pages_per_seq=pages, use_pdl=pdl)
     return _random_model(gm, torch, dev, cfg, 74)
 
@@ -814,7 +814,7 @@ def time_kozapel_kernels(ops, torch, dev, name, rows, ctx_len=PROMPT_LEN, only=N
         mean = rows * top / experts
         tile = 16 if mean <= 8 else 32 if mean <= 24 else 64 if mean <= 48 else 128
         z, corr = torch.randn(rows, experts, device=dev), 0.1 * torch.randn(experts, device=dev)
-        route = dict(sigmoid=True, group_best=2, weight_scale=2.0, correction=corr)
+        route = dict(sigmoid=True, group_best=2, weight_scale=1.5, correction=corr)
         us = _graph_us(torch, [lambda: ops.moe_route(experts, top, groups, keep, tile, z, y, **route)] * 4)
         put("route", us, rows * experts * 4 + rows * w * 2 * (1 + top), 0)
         pair, weight, row_tiles, n_tiles, srt, most = ops.moe_route(experts, top, groups, keep, tile, z, y, **route)

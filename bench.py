@@ -525,7 +525,7 @@ def _felepel_model(gm, torch, dev, name, n_layers, ctx, pdl, chunk, batch):
     width, vocab = LAYERED_SIZES[name][0], LAYERED_SIZES[name][8]
     (h, g, d, v, size), (dh, dg, dd, dv, taps, rank), (experts, top, groups, keep, ff) = FELEPEL_SIZES[name]
     moe = dict(mlp=gm.MLP_EXPERTS, d_ff=ff, experts=experts, top=top, groups=groups, keep=keep)
-    att = gm.LayerConfig(heads=h, kv_heads=g, dim=d, vdim=v, scale=d ** -0.5, softcap=30.0, mask=gm.MASK_CHUNK, mask_size=size, distance_bias=1, proj_bias=1,
+    att = gm.LayerConfig(heads=h, kv_heads=g, dim=d, vdim=v, scale=d ** -0.5, softcap=30.0, mask=gm.MASK_CHUNK, mask_size=size, distance_bias=gm.DISTANCE_LOG, proj_bias=1,
                          mixer=gm.MIXER_GROUPED_ATTENTION, **moe)
     delta = gm.LayerConfig(heads=dh, kv_heads=dg, dim=dd, vdim=dv, taps=taps, decay_rank=rank, gate_rank=rank, mixer=gm.MIXER_CHANNEL_DELTA, **moe)
     pages = (ctx + 15) // 16

@@ -90,19 +90,40 @@ class StreamStep(ctypes.Structure):
     ]
 
 
+class DepthStep(ctypes.Structure):
+    """gptrs_depth_step."""
+    _fields_ = [
+        ("d_x", ctypes.c_void_p), ("d_x_out", ctypes.c_void_p), ("d_y", ctypes.c_void_p), ("y_dtype", ctypes.c_int), ("ldy", ctypes.c_int64),
+        ("d_pair", ctypes.c_void_p), ("d_pair_weight", ctypes.c_void_p), ("top", ctypes.c_int64), ("d_add", ctypes.c_void_p), ("ld_add", ctypes.c_int64),
+        ("d_add_gate", ctypes.c_void_p), ("ld_add_gate", ctypes.c_int64), ("d_embed", ctypes.c_void_p), ("d_tokens", ctypes.c_void_p), ("vocab", ctypes.c_int64),
+        ("d_gamma_out", ctypes.c_void_p), ("mult", ctypes.c_float), ("groups", ctypes.c_int), ("eps", ctypes.c_float), ("d_states", ctypes.c_void_p),
+        ("state_stride", ctypes.c_int64), ("n_states", ctypes.c_int64), ("d_weights", ctypes.c_void_p), ("d_gamma_in", ctypes.c_void_p),
+        ("d_rows", ctypes.c_void_p), ("d_h", ctypes.c_void_p), ("h_dtype", ctypes.c_int), ("ldh", ctypes.c_int64), ("d_status", ctypes.c_void_p),
+        ("rows", ctypes.c_int64), ("dim", ctypes.c_int64),
+    ]
+
+
+class GroupedStep(ctypes.Structure):
+    """gptrs_grouped_step."""
+    _fields_ = [(n, ctypes.c_void_p) for n in ("d_qkv", "d_conv", "d_q_gain", "d_k_gain", "d_conv_state", "d_slot", "d_pos", "d_run_first", "d_run_last", "d_parity",
+                                               "d_page_table")] + \
+        [("max_pages", ctypes.c_int64), ("d_pool", ctypes.c_void_p), ("d_q", ctypes.c_void_p), ("rows", ctypes.c_int64)]
+
+
 class GroupedAttention(ctypes.Structure):
     """gptrs_grouped_attention."""
     _fields_ = [(n, ctypes.c_int) for n in ("dtype", "heads", "kv_heads", "dim", "vdim", "mask", "mask_size")] + \
         [("scale", ctypes.c_float), ("softcap", ctypes.c_float), ("distance_bias", ctypes.c_int)] + \
         [(n, ctypes.c_int) for n in ("maps", "gate", "shared_kv")] + [(n, ctypes.c_float) for n in ("lambda_", "head_scale", "head_eps")] + \
+        [(n, ctypes.c_int) for n in ("taps", "qk_norm", "tied")] + \
         [(n, ctypes.c_int) for n in ("q_head_stride", "k_offset", "k_head_stride", "v_offset", "v_head_stride", "q_row", "map_stride", "g_offset",
-                                     "g_head_stride", "out_head_stride")] + \
-        [("page_bytes", ctypes.c_int64)]
+                                     "g_head_stride", "out_head_stride", "query_row", "conv_channels")] + \
+        [("conv_floats", ctypes.c_int64), ("page_bytes", ctypes.c_int64)]
 
 
 class DeltaRule(ctypes.Structure):
     """gptrs_delta_rule."""
-    _fields_ = [(n, ctypes.c_int) for n in ("dtype", "heads", "kv_heads", "dim", "vdim", "taps", "decay_rank", "gate_rank")] + [("eps", ctypes.c_float)] + \
+    _fields_ = [(n, ctypes.c_int) for n in ("dtype", "heads", "kv_heads", "dim", "vdim", "taps", "decay_rank", "gate_rank")] + [("eps", ctypes.c_float), ("gate_silu", ctypes.c_int)] + \
         [(n, ctypes.c_int) for n in ("q_offset", "k_offset", "v_offset", "beta_offset", "a_offset", "g_offset", "row", "decay_row", "gate_row",
                                      "out_head_stride", "conv_channels")] + \
         [(n, ctypes.c_int64) for n in ("state_floats", "conv_floats")]

@@ -139,8 +139,8 @@ class CheckpointReader:
 
 
 # "architecture" of a model folder's config.json -> model kind of `engine_config`
-ARCHITECTURES = {"Bevosun": "bevosun", "Felepel": "felepel", "Kozapel": "kozapel"}
-LAYERED_KINDS = ("bevosun", "felepel", "kozapel")   # kinds whose layers are configured one by one
+ARCHITECTURES = {"Bevosun": "bevosun", "Felepel": "felepel", "Kozapel": "kozapel", "Domorax": "domorax"}
+LAYERED_KINDS = ("bevosun", "felepel", "kozapel", "domorax")   # kinds whose layers are configured one by one
 
 
 class ModelFolder:
@@ -332,6 +332,8 @@ def engine_config(model_config: dict, weight_mode: int = gm.MODE_F32, shapes: di
         return felepel_config(c, shapes, weight_mode=weight_mode, **engine_kw), None
     if kind == "kozapel":
         return kozapel_config(c, weight_mode=weight_mode, **engine_kw), None
+    if kind == "domorax":
+        return domorax_config(c, weight_mode=weight_mode, **engine_kw), None
     raise BackendError(2, f"model kind {kind!r} is not a decode model of this backend")
 
 
@@ -364,7 +366,7 @@ def felepel_config(c: dict, shapes: dict | None = None, context_length: int | No
                   weights_of=-1 if of is None else int(of))
         if layer["type"] == "attention":
             mask = m.get("mask")
-            kw.update(mixer=gm.MIXER_GROUPED_ATTENTION, scale=float(m["scale"]), softcap=float(m.get("softcap") or 0.0), distance_bias=1, proj_bias=1,
+            kw.update(mixer=gm.MIXER_GROUPED_ATTENTION, scale=float(m["scale"]), softcap=float(m.get("softcap") or 0.0), distance_bias=gm.DISTANCE_LOG, proj_bias=1,
                       mask=gm.MASK_CHUNK if mask else gm.MASK_CAUSAL, mask_size=int(mask["size"]) if mask else 0)
         elif layer["type"] == "channel_delta":
             owner = f"l{i if of is None else of}.mix."
@@ -421,6 +423,40 @@ def kozapel_config(c: dict, context_length: int = 4096, **engine_kw) -> gm.Model
         layers.append(gm.LayerConfig(**kw))
     return gm.ModelConfig.layered(layers, int(c["width"]), int(c["vocab"]), context_length, float(c["norm"]["eps"]), block=gm.BLOCK_PRE_NORM,
                                   streams=int(c.get("streams") or 0), embed_scale=float(c["embedding"]["scale"]), **engine_kw)
+
+
+def domorax_config(c: dict, context_length: int = 4096, **engine_kw) -> gm.ModelConfig:
+    """Domorax's config object -> the layered kind. The design bounds no context: `context_length` is the caller's."""
+    layers = []
+    for i, layer in enumerate(c["layers"]):
+        m, mlp = layer["mixer"], layer.get("mlp")
+        kw = dict(heads=int(m["heads"]), dim=int(m["dim"]), vdim=int(m["vdim"]), mlp=gm.MLP_NONE)
+        mask = m.get("mask")
+        if layer["type"] == "latent_attention":
+            rot = m["rot"]
+            kw.update(mixer=gm.MIXER_LATENT_ATTENTION, rot_dim=int(m["rot_dim"]), kv_rank=int(m["kv_rank"]), q_rank=int(m["q_rank"]), scale=float(m["scale"]),
+                      rope_base=float(rot["base"]), rot_dims=int(rot["dims"]), rope_halves=1, window=int(mask["size"]) if mask else 0, sink=1)
+            if rot.get("scaling"):
+                kw.update({"rope_" + k: float(rot["scaling"][k]) for k in ("factor", "original", "fast", "slow")})
+        elif layer["type"] == "attention":
+            kw.update(mixer=gm.MIXER_GROUPED_ATTENTION, kv_heads=int(m["kv_heads"]), scale=float(m["scale"]), taps=int(m["conv"]), qk_norm=1, tied=1,
+                      distance_bias=gm.DISTANCE_LINEAR, mask=gm.MASK_WINDOW if mask else gm.MASK_CAUSAL, mask_size=int(mask["size"]) if mask else 0)
+        elif layer["type"] == "delta":
+            kw.update(mixer=gm.MIXER_CHANNEL_DELTA, kv_heads=int(m["kv_heads"]), taps=int(m["conv"]), gate_silu=1)
+        else:
+            raise BackendError(2, f"layer {i}: mixer {layer['type']!r} is not built")
+        if mlp and mlp["kind"] == "dense":
+            kw.update(mlp=gm.MLP_DENSE_POLY, d_ff=int(mlp["ff"]))
+        elif mlp and mlp["kind"] == "moe":
+            r, shared = mlp["router"], mlp.get("shared")
+            kw.update(mlp=gm.MLP_EXPERTS, d_ff=int(mlp["expert"]["ff"]), experts=int(r["experts"]), top=int(r["top"]), weight_scale=1.0)   # softmax over the chosen
+            if shared:
+                kw.update(shared_ff=int(shared["ff"]), shared_gate=1)
+        elif mlp:
+            raise BackendError(2, f"layer {i}: feed-forward {mlp['kind']!r} is not built")
+        layers.append(gm.LayerConfig(**kw))
+    return gm.ModelConfig.layered(layers, int(c["width"]), int(c["vocab"]), context_length, float(c["norm"]["eps"]), block=gm.BLOCK_DEPTH,
+                                  residual_mult=float(c["residual_mult"]), norm_groups=int(c["norm"]["groups"]), **engine_kw)
 
 
 def load_model(path, weight_mode: int = gm.MODE_F32, namespace: int | None = None, **engine_kw) -> gm.LoadedModel:

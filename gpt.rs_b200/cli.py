@@ -127,6 +127,8 @@ def cmd_export_random(args) -> int:
             tensors[name] = np.ones(shape, np.float32)
         elif name.endswith(("beta", ".b", ".act", ".correction")) or ".b_" in name:
             tensors[name] = np.zeros(shape, np.float32)
+        elif name.endswith(".dwa"):   # what goes on is the layer's result alone
+            tensors[name] = np.eye(shape[0], dtype=np.float32)[-1]
         elif ".hc" in name:   # streams that stay as they are, read as their mean
             tensors[name] = np.eye(*shape, dtype=np.float32) if len(shape) == 2 else np.full(shape, 1.0 / shape[0] if name.endswith(".in") else 1.0, np.float32)
         else:
@@ -155,7 +157,7 @@ def main(argv=None) -> int:
     g.add_argument("--top-k", type=int, default=None)
     g.add_argument("--seed", type=int, default=0)
     g.add_argument("--weight-mode", default="f32", choices=["f32", "w4a16", "w8a16", "bf16"],
-                   help="w4a16 / w8a16 quantise the linear weights on the device while loading (ministral kind); bf16: the layered kinds, bevosun, felepel and kozapel")
+                   help="w4a16 / w8a16 quantise the linear weights on the device while loading (ministral kind); bf16: the layered kinds, bevosun, felepel, kozapel and domorax")
     g.add_argument("--no-graph", action="store_true", help="launch kernels one by one instead of replaying a CUDA graph")
     g.set_defaults(fn=cmd_generate)
     i = sub.add_parser("inspect", help="print the config and tensor index of a checkpoint")
@@ -163,7 +165,7 @@ def main(argv=None) -> int:
     i.set_defaults(fn=cmd_inspect)
     x = sub.add_parser("export-random", help="write a checkpoint with random weights for a config")
     x.add_argument("--out", required=True)
-    x.add_argument("--kind", required=True, choices=["gpt", "ministral", "bevosun", "felepel", "kozapel"])
+    x.add_argument("--kind", required=True, choices=["gpt", "ministral", "bevosun", "felepel", "kozapel", "domorax"])
     x.add_argument("--config", required=True, help="the model's config JSON object")
     x.add_argument("--seed", type=int, default=0)
     x.add_argument("--std", type=float, default=0.02)

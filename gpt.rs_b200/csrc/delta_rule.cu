@@ -1,4 +1,4 @@
-// Gated delta rule with a decay per key channel (no counterpart in gpt.rs). Per head and token
+// Gated delta rule with a decay per key channel, or one per head (no counterpart in gpt.rs). Per head and token
 //
 //   S <- g S (rows of S are key channels);   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
 //
@@ -31,11 +31,12 @@ struct Geo {
     int q_off, k_off, v_off, beta_off, row, decay_row, gate_row, out_stride, channels;
     int dp, vp;              // dim and vdim of the f32 planes, multiples of 4
     float eps, q_scale;
+    int head_decay, a_off, gate_silu;   // one decay per head: column a_off + head of the projection row
 };
 __host__ __device__ inline int pad4(int v) { return (v + 3) / 4 * 4; }
 Geo geo(const gptrs_delta_rule& a) {
     Geo g = {a.heads, a.kv_heads, a.heads / a.kv_heads, a.dim, a.vdim, a.taps, a.q_offset, a.k_offset, a.v_offset, a.beta_offset, a.row, a.decay_row, a.gate_row,
-             a.out_head_stride, a.conv_channels, pad4(a.dim), pad4(a.vdim), a.eps, 1.f / sqrtf((float)a.dim)};
+             a.out_head_stride, a.conv_channels, pad4(a.dim), pad4(a.vdim), a.eps, 1.f / sqrtf((float)a.dim), a.decay_rank == 0, a.a_offset, a.gate_silu};
     return g;
 }
 constexpr int kBlock = 4;        // tokens of a block
@@ -83,10 +84,17 @@ __device__ __forceinline__ float decay_fast(float x, float rate) {
     const float series = e * fmaf(e, fmaf(e, fmaf(e, -0.25f, 1.f / 3.f), -0.5f), 1.f);
     return __expf(rate * (fmaxf(x, 0.f) + (e < 0.02f ? series : __logf(1.f + e))));
 }
-__device__ __forceinline__ float decay_of(const Params& p, int row, int head, int d) {
-    const int c = head * p.g.dim + d;
-    return expf(-expf(p.s.d_a_log[head]) * softplus(p.s.d_decay[(size_t)row * p.g.decay_row + c] + p.s.d_dt_bias[c]));
+// what the softplus of a decay takes, without its bias; the bias
+template <typename T>
+__device__ __forceinline__ float decay_input(const Params& p, int row, int head, int d) {
+    return p.g.head_decay ? ld(static_cast<const T*>(p.s.d_proj) + (size_t)row * p.g.row + p.g.a_off + head) : p.s.d_decay[(size_t)row * p.g.decay_row + head * p.g.dim + d];
 }
+__device__ __forceinline__ float decay_bias(const Params& p, int head, int d) { return p.s.d_dt_bias[p.g.head_decay ? head : head * p.g.dim + d]; }
+template <typename T>
+__device__ __forceinline__ float decay_of(const Params& p, int row, int head, int d) {
+    return expf(-expf(p.s.d_a_log[head]) * softplus(decay_input<T>(p, row, head, d) + decay_bias(p, head, d)));
+}
+__device__ __forceinline__ float gate_of(const Geo& g, float z) { return g.gate_silu ? silu(z) : sigmoid(z); }
 
 // The convolution state that a single-token run reads and writes; place: where in the ring of taps - 1 inputs the last one lies.
 struct RowState { int pos, place; const float* old; float* fresh; };
@@ -262,7 +270,7 @@ __global__ void __launch_bounds__(kPrepThreads, NI <= 4 ? 4 : 1) delta_prepare_k
 #pragma unroll
             for (int t = 0; t < kBlock; ++t) {
                 const int d = i * 32 + lane;
-                dec[i][t] = t < b.n && d < g.dim ? p.s.d_decay[(size_t)(b.row + t) * g.decay_row + head * g.dim + d] : 0.f;
+                dec[i][t] = t < b.n && d < g.dim ? decay_input<T>(p, b.row + t, head, d) : 0.f;
             }
         float sums[8];
 #pragma unroll
@@ -297,7 +305,7 @@ __global__ void __launch_bounds__(kPrepThreads, NI <= 4 ? 4 : 1) delta_prepare_k
             const int d = i * 32 + lane;
             float gd[kBlock] = {1.f, 1.f, 1.f, 1.f};
             if (d < g.dim) {
-                const float bias = p.s.d_dt_bias[head * g.dim + d];
+                const float bias = decay_bias(p, head, d);
 #pragma unroll
                 for (int t = 0; t < kBlock; ++t)
                     if (t < b.n) {
@@ -544,8 +552,8 @@ __global__ void __launch_bounds__(256) delta_output_kernel(const Params p) {
             if (in) {
                 const uint2 gu = *reinterpret_cast<const uint2*>(gate + c);
                 const float4 w = *reinterpret_cast<const float4*>(p.s.d_norm + c);
-                *reinterpret_cast<uint2*>(out + c) = make_uint2(pack_bf16x2(v.x * inv * w.x * sigmoid(bf16_lo(gu.x)), v.y * inv * w.y * sigmoid(bf16_hi(gu.x))),
-                                                                pack_bf16x2(v.z * inv * w.z * sigmoid(bf16_lo(gu.y)), v.w * inv * w.w * sigmoid(bf16_hi(gu.y))));
+                *reinterpret_cast<uint2*>(out + c) = make_uint2(pack_bf16x2(v.x * inv * w.x * gate_of(g, bf16_lo(gu.x)), v.y * inv * w.y * gate_of(g, bf16_hi(gu.x))),
+                                                                pack_bf16x2(v.z * inv * w.z * gate_of(g, bf16_lo(gu.y)), v.w * inv * w.w * gate_of(g, bf16_hi(gu.y))));
             } else if (c < g.out_stride) {
                 *reinterpret_cast<uint2*>(out + c) = make_uint2(0, 0);
             }
@@ -555,7 +563,7 @@ __global__ void __launch_bounds__(256) delta_output_kernel(const Params p) {
     float ss = 0.f;
     for (int c = lane; c < g.vdim; c += 32) ss = fmaf(o[c], o[c], ss);
     const float inv = 1.f / sqrtf(warp_sum(ss) / (float)g.vdim + g.eps);
-    for (int c = lane; c < g.out_stride; c += 32) st(out + c, c < g.vdim ? o[c] * inv * p.s.d_norm[c] * sigmoid(ld(gate + c)) : 0.f);
+    for (int c = lane; c < g.out_stride; c += 32) st(out + c, c < g.vdim ? o[c] * inv * p.s.d_norm[c] * gate_of(g, ld(gate + c)) : 0.f);
 }
 
 // ---- decode: one token per sequence ----------------------------------------------------------------------------------------------
@@ -596,7 +604,7 @@ __global__ void __launch_bounds__(kDecThreads, NR * VEC <= 64 ? 2 : 1) delta_dec
     };
     load_state(0);   // travels while the vectors are prepared
     const float beta_raw = ld(static_cast<const T*>(p.s.d_proj) + (size_t)row * g.row + g.beta_off + head);
-    for (int d = tid; d < g.dim; d += kDecThreads) gd[d] = decay_of(p, row, head, d);
+    for (int d = tid; d < g.dim; d += kDecThreads) gd[d] = decay_of<T>(p, row, head, d);
     const bool own = head % g.group == 0;   // heads that share q and k: the first passes their convolution state on
     for (int i = tid; i < 2 * g.dim + g.vdim; i += kDecThreads) {
         if (i < g.dim) q[i] = conv_channel<T>(p, r, row, kvh * g.dim + i, g.q_off + kvh * g.dim + i, own);
@@ -676,7 +684,7 @@ __global__ void __launch_bounds__(kDecThreads, NR * VEC <= 64 ? 2 : 1) delta_dec
     const float inv = 1.f / sqrtf(ss / (float)g.vdim + g.eps);
     const T* gate = static_cast<const T*>(p.s.d_gate) + (size_t)row * g.gate_row + head * g.vdim;
     T* out = static_cast<T*>(p.s.d_out) + ((size_t)row * g.heads + head) * g.out_stride;
-    for (int c = tid; c < g.out_stride; c += kDecThreads) st(out + c, c < g.vdim ? o[c] * inv * p.s.d_norm[c] * sigmoid(ld(gate + c)) : 0.f);
+    for (int c = tid; c < g.out_stride; c += kDecThreads) st(out + c, c < g.vdim ? o[c] * inv * p.s.d_norm[c] * gate_of(g, ld(gate + c)) : 0.f);
 }
 
 template <int NI, int CPL, int LPC, int STAGES>
@@ -732,7 +740,7 @@ extern "C" {
 
 int gptrs_cuda_delta_layout(gptrs_delta_rule* a) {
     GPTRS_REQUIRE(a, "null pointer");
-    GPTRS_REQUIRE(a->heads > 0 && a->kv_heads > 0 && a->dim > 0 && a->vdim > 0 && a->taps > 0 && a->decay_rank > 0 && a->gate_rank > 0, "delta rule: sizes must be positive");
+    GPTRS_REQUIRE(a->heads > 0 && a->kv_heads > 0 && a->dim > 0 && a->vdim > 0 && a->taps > 0 && a->decay_rank >= 0 && a->gate_rank >= 0, "delta rule: sizes must be positive");
     GPTRS_REQUIRE(a->heads % a->kv_heads == 0, "delta rule: heads must be a multiple of the q/k heads");
     GPTRS_REQUIRE(a->dtype == GPTRS_F32 || a->dtype == GPTRS_BF16, "delta rule: f32 or bf16");
     if (a->dim > kMaxDim || a->vdim > 4096 || a->heads > 65535) return fail(GPTRS_UNIMPLEMENTED, "delta rule: dim above 512, vdim above 4096 or more than 65535 heads");
@@ -742,10 +750,10 @@ int gptrs_cuda_delta_layout(gptrs_delta_rule* a) {
     a->v_offset = a->k_offset + pad(a->kv_heads * a->dim);
     a->beta_offset = a->v_offset + pad(a->heads * a->vdim);
     a->a_offset = a->beta_offset + pad(a->heads);
-    a->g_offset = a->a_offset + pad(a->decay_rank);
-    a->row = a->g_offset + pad(a->gate_rank);
-    a->decay_row = pad(a->heads * a->dim);
-    a->gate_row = pad(a->heads * a->vdim);
+    a->g_offset = a->a_offset + pad(a->decay_rank > 0 ? a->decay_rank : a->heads);
+    a->row = a->g_offset + pad(a->gate_rank > 0 ? a->gate_rank : a->heads * a->vdim);
+    a->decay_row = a->decay_rank > 0 ? pad(a->heads * a->dim) : 0;
+    a->gate_row = a->gate_rank > 0 ? pad(a->heads * a->vdim) : a->row;
     a->out_head_stride = pad(a->vdim);
     a->conv_channels = 2 * a->kv_heads * a->dim + a->heads * a->vdim;
     a->state_floats = (int64_t)a->heads * a->dim * a->vdim;
@@ -762,12 +770,14 @@ int64_t gptrs_cuda_delta_scratch_floats(const gptrs_delta_rule* a, int64_t rows,
 int gptrs_cuda_delta_rule(const gptrs_delta_rule* a, const gptrs_delta_step* step, void* stream) {
     GPTRS_REQUIRE(a && step && a->row > 0, "null pointer, or layout not filled in");
     const gptrs_delta_step& s = *step;
-    GPTRS_REQUIRE(s.d_proj && s.d_decay && s.d_gate && s.d_conv && s.d_a_log && s.d_dt_bias && s.d_norm && s.d_state && (s.d_conv_state || a->taps == 1) && s.d_out, "null pointer");
+    GPTRS_REQUIRE((s.d_decay || a->decay_rank == 0) && (s.d_gate || a->gate_rank == 0), "null pointer");
+    GPTRS_REQUIRE(s.d_proj && s.d_conv && s.d_a_log && s.d_dt_bias && s.d_norm && s.d_state && (s.d_conv_state || a->taps == 1) && s.d_out, "null pointer");
     GPTRS_REQUIRE(s.d_slot && s.d_pos && s.d_run_first && s.d_run_last && s.d_parity, "null pointer");
     GPTRS_REQUIRE(s.rows >= 0 && s.rows < (1ll << 31) && s.n_runs >= 0 && s.n_runs <= s.rows && s.n_runs <= 65535, "delta rule: rows and runs");
     if (s.rows == 0) return GPTRS_OK;
     GPTRS_REQUIRE(s.n_runs == s.rows || (s.n_runs > 0 && s.d_runs && s.d_status && s.d_scratch && (reinterpret_cast<uintptr_t>(s.d_scratch) & 15) == 0), "delta rule: run list and scratch");
     Params p = {s, geo(*a), {}};
+    if (a->gate_rank == 0) p.s.d_gate = static_cast<const unsigned char*>(s.d_proj) + (size_t)a->g_offset * (a->dtype == GPTRS_BF16 ? 2 : 4);
     if (s.n_runs != s.rows) p.w = planes(p.g, s.d_scratch, s.rows, s.n_runs);
     return a->dtype == GPTRS_BF16 ? run<__nv_bfloat16>(p, as_stream(stream)) : run<float>(p, as_stream(stream));
 }

@@ -68,7 +68,10 @@ struct DenseWeight {   // [batch][n][k] bf16 with n and k padded to 8, or [batch
 // What a layer multiplies with; layers that reuse another one's weights share the object.
 struct LayerWeights {
     Tensor *norm1 = nullptr, *norm2 = nullptr, *norm1b = nullptr, *norm2b = nullptr, *conv1 = nullptr, *conv2 = nullptr, *latent_norm = nullptr;
-    Tensor *r1 = nullptr, *r2 = nullptr;                                                              // distance penalty
+    Tensor *r1 = nullptr, *r2 = nullptr;                                                              // distance penalty (linear: r1 alone, the slopes)
+    DevBuf reach;                                                                                     // of the kv heads, where norms bound the scores
+    Tensor *sink = nullptr, *dwa = nullptr, *act = nullptr;                                           // softmax sinks; average over depth; polynomial
+    Tensor *qk_conv = nullptr, *q_gain = nullptr, *k_gain = nullptr;                                  // grouped attention: convolutions, norms per head
     Tensor *q_norm = nullptr, *correction = nullptr;                                                  // query latent; experts' choice
     struct Streams { Tensor *in = nullptr, *out = nullptr, *mix = nullptr; } streams[2];              // of the two sublayers
     Tensor *delta_conv = nullptr, *a_log = nullptr, *dt_bias = nullptr, *delta_norm = nullptr;        // delta rule
@@ -76,7 +79,7 @@ struct LayerWeights {
     float act_pos = 0.f, act_neg = 0.f;
     float lambda = 0.f;   // differential attention
     ~LayerWeights() {
-        for (Tensor* t : {norm1, norm2, norm1b, norm2b, conv1, conv2, latent_norm, r1, r2, q_norm, correction, delta_conv, a_log, dt_bias, delta_norm}) tensor_release(t);
+        for (Tensor* t : {norm1, norm2, norm1b, norm2b, conv1, conv2, latent_norm, r1, r2, q_norm, correction, delta_conv, a_log, dt_bias, delta_norm, sink, dwa, act, qk_conv, q_gain, k_gain}) tensor_release(t);
         for (Streams& s : streams) for (Tensor* t : {s.in, s.out, s.mix}) tensor_release(t);
         for (DenseWeight* w : {&qkv, &uq, &uk, &uv, &out, &up, &down, &decay, &gate, &router, &shared_up, &shared_down}) { tensor_release(w->w); tensor_release(w->bias); }
     }
@@ -92,8 +95,9 @@ struct LayeredLayer {
     int rope = -1;         // index into Layered::ropes
     int tiles = -1;        // index into Layered::tile_sets, -1 = plain attention kernel
     int state1 = 0, state2 = 0;                      // convolution states of the two sublayers
-    size_t delta_state_off = 0, delta_conv_off = 0;  // floats
+    size_t delta_state_off = 0, mix_conv_off = 0;    // floats: delta rule's state, inputs of the mixer's convolutions
     bool attends() const { return cfg.mixer != GPTRS_MIXER_CHANNEL_DELTA; }
+    bool prepared() const { return cfg.mixer == GPTRS_MIXER_GROUPED_ATTENTION && (gatt.taps > 0 || gatt.qk_norm || gatt.tied); }   // queries in rows of their own
     // the first position that `pos` sees
     int first_visible(int pos) const {
         int f = 0;
@@ -113,7 +117,7 @@ struct Layered {
     std::vector<LayeredLayer> layers;
     Tensor* embed_norm = nullptr;
     DenseWeight head;
-    struct Rope { double base; int dims; DevBuf cos_t, sin_t; };
+    struct Rope { double base, factor, original, fast, slow; int dims; DevBuf cos_t, sin_t; };
     std::vector<std::unique_ptr<Rope>> ropes;
     // query tiles of the tensor-core attention: one list per distinct tile size (layers may differ in their head counts)
     struct TileSet { int tokens = 1, n = 0; DevBuf row, rows; };
@@ -121,7 +125,9 @@ struct Layered {
     int32_t* h_tiles = nullptr;   // pinned staging of one tile list (rows, then counts)
     DevBuf x2, h, qkv, q, q_latent, qa, lat, attn, up, y, logits_pad, state, scratch;
     DevBuf d_run_first, d_run_last, d_parity, d_runs;
-    DevBuf decay, gate, delta_state, delta_conv, delta_scratch;   // delta rule
+    DevBuf decay, gate, delta_state, delta_scratch;   // delta rule
+    DevBuf mix_conv;                                  // last inputs of the mixers' short convolutions
+    DevBuf states;                                    // GPTRS_BLOCK_DEPTH: the embedding and every layer's result [layers + 1][max_tokens][d_model]
     // experts: logits, sorted rows and what comes of them, the place of every (row, choice) among them, row tiles
     DevBuf router, sorted, gate_up, expert_y, pair, pair_weight, row_tiles, n_row_tiles, moe_work;
     std::vector<int> parity;      // per slot: the half of the convolution state the next step reads

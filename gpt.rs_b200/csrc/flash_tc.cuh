@@ -40,6 +40,9 @@ __device__ __forceinline__ int page_chunk(int t, int chunk, int nb) {
 // rows 0 .. 63 carry the first part of the queries, rows 64 .. 127 the second one, each with zeros in the columns of the other part, so
 // that one product with the whole key block gives the scores of both (an MMA of 64 rows would take as long as one of 128) and keys and
 // values are read once. At the end the halves of O meet in shared memory: difference, norm over the head, gate.
+// Linear distance bias and keys that are values times a number each (LINEAR): the numbers travel beside the pages and multiply the columns of
+// S, so that a block holds values only and is an operand of both products. Blocks are walked from the newest to the oldest: under a steep
+// bias the running maximum would otherwise move at every block.
 constexpr int kRows = 128;
 constexpr int kKeys = 64;
 constexpr int kTcThreads = 224;
@@ -61,6 +64,7 @@ struct FlashShape {
     int map_blocks;                    // query blocks of one part (query_blocks without a second one)
     uint32_t block_bytes;              // (page, kv head): 16 rows
     long long page_bytes;
+    int key_scales;                    // 1: 16 floats per kv head behind the blocks of a page, key = value x number
 };
 // What happens to the output of a head behind the softmax.
 struct HeadOutput {
@@ -96,7 +100,9 @@ struct TcParams {
     uint32_t tmem_cols, q_box_bytes, q_one_bytes;
     float scale_log2;                  // log2(e) scale; with a soft cap, 2 log2(e) scale / cap
     float cap_log2;                    // log2(e) cap, 0 = none
-    const float *r1, *r2;              // distance penalty r1[h] ln(1 + r2[h] d), or null
+    const float *r1, *r2;              // distance penalty r1[h] ln(1 + r2[h] d), or null; LINEAR: r1[h] d
+    const int* reach;                  // [kv heads] or null: keys further away than that weigh nothing
+    const float* sink;                 // [heads] or null: exp(sink) in the denominator
     HeadOutput head_out;
 };
 
@@ -214,16 +220,38 @@ __device__ __forceinline__ void score_log2(float (&s)[kKeys], float scale_log2, 
     }
 }
 
+// column j of the scores times c[j]
+__device__ __forceinline__ void scale_columns(float (&s)[kKeys], const float* c) {
+#pragma unroll
+    for (int j = 0; j < kKeys; j += 4) {
+        const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(c + j);
+        const float2 a = split(mul2(pair_of(s[j], s[j + 1]), v.x)), b = split(mul2(pair_of(s[j + 2], s[j + 3]), v.y));
+        s[j] = a.x; s[j + 1] = a.y; s[j + 2] = b.x; s[j + 3] = b.y;
+    }
+}
+// Raw products -> log2(e) (cap tanh(scale s / cap) - slope d)
+__device__ __forceinline__ void score_linear(float (&s)[kKeys], float scale_log2, float cap_log2, float slope, int d0) {
+    if (cap_log2 > 0.f) score_log2(s, scale_log2, cap_log2, 0.f, 0.f, 0);
+    const float c = slope * kLog2e, b0 = -c * (float)d0, mul = cap_log2 > 0.f ? 1.f : scale_log2;
+    const uint64_t m = pair_of(mul, mul);
+#pragma unroll
+    for (int j = 0; j < kKeys; j += 2) {
+        const float2 v = split(fma2(pair_of(s[j], s[j + 1]), m, pair_of(fmaf(c, (float)j, b0), fmaf(c, (float)(j + 1), b0))));
+        s[j] = v.x; s[j + 1] = v.y;
+    }
+}
+
 // GROUPED: kv heads of their own, soft cap, distance penalty; otherwise one latent row for all heads
 // kScores 2: two CTAs share an SM (tensor memory, shared memory and registers for half of one each), so that the softmax of one runs
 // under the waits of the other.
-// TWO: two query and key parts per head.
-template <bool GROUPED, int kScores, bool TWO = false>
+// TWO: two query and key parts per head. LINEAR: linear distance bias, keys by numbers.
+template <bool GROUPED, int kScores, bool TWO = false, bool LINEAR = false>
 __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_kernel(const __grid_constant__ TcParams p) {
     constexpr uint32_t kOCol = kScores * kKeys;
     constexpr int kTileRows = TWO ? kRows / 2 : kRows;
     extern __shared__ unsigned char smem_raw[];
     __shared__ __align__(8) uint64_t k_full[kMaxStages], k_empty[kMaxStages], s_full[kScores], p_full[kScores], q_full;
+    __shared__ __align__(16) float k_scale[LINEAR ? kMaxStages : 1][LINEAR ? kKeys : 4];
     __shared__ uint32_t tmem_holder;
     const FlashShape& g = p.g;
     const uint32_t smem = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -268,11 +296,14 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
     const int slot0 = p.slot[row0], cap = p.max_pages * kPageTok;
     const int hi = min(max(p.ctx_len[row0 + n_tok - 1], 0), cap);
     const int first_len = p.ctx_len[row0];
-    const int lo = (GROUPED ? first_visible(g.mask, g.mask_size, max(first_len - 1, 0)) : max(first_len - g.mask_size, 0)) & ~(kPageTok - 1);
+    int lo = GROUPED ? first_visible(g.mask, g.mask_size, max(first_len - 1, 0)) : max(first_len - g.mask_size, 0);
+    if (LINEAR && p.reach) lo = max(lo, first_len - 1 - p.reach[kvh]);
+    lo &= ~(kPageTok - 1);
     const int n_all = hi > lo ? (hi - lo + kKeys - 1) / kKeys : 0;
     const int kb0 = (int)((int64_t)n_all * blockIdx.y / p.splits), kb1 = (int)((int64_t)n_all * (blockIdx.y + 1) / p.splits);
     const int n_blocks = kb1 - kb0;
     const int key_base = lo + kb0 * kKeys;
+    auto key_of = [&](int it) { return key_base + (LINEAR ? n_blocks - 1 - it : it) * kKeys; };   // first key of the block that comes as number `it`
     bool failed = false;
     auto wait = [&](uint64_t* bar, uint32_t parity) {   // whole warp
         if (!failed && !mbar_wait_parked(smem_u32(bar), parity, kWaitLimit)) failed = true;
@@ -286,7 +317,7 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
         const uint32_t block_bytes = g.block_bytes;
         const unsigned char* pool = p.pool + (size_t)kvh * block_bytes;
         auto page_of = [&](int it) {   // lane j: the j-th page of block `it`
-            const int key0 = key_base + it * kKeys;
+            const int key0 = key_of(it);
             return it < n_blocks && lane < (min(kKeys, hi - key0) + kPageTok - 1) / kPageTok ? __ldg(pt + key0 / kPageTok + lane) : 0;
         };
         int n_req = 0, page_next = page_of(0);
@@ -323,13 +354,18 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
             const int page = page_next;
             page_next = page_of(it + 1);
             if (lap > 0 && !wait(&k_empty[st], (uint32_t)(lap - 1) & 1u)) break;
-            const int key0 = key_base + it * kKeys;
+            const int key0 = key_of(it);
             const int pages = (min(kKeys, hi - key0) + kPageTok - 1) / kPageTok;
             const uint32_t bar = smem_u32(&k_full[st]);
-            if (lane == 0) mbar_expect_tx_addr(bar, (uint32_t)pages * block_bytes);
+            const bool scales = LINEAR && g.key_scales;
+            if (lane == 0) mbar_expect_tx_addr(bar, (uint32_t)pages * (block_bytes + (scales ? kPageTok * 4u : 0u)));
             __syncwarp();
-            if (lane < pages)
+            if (lane < pages) {
                 bulk_g2s_addr(sK + st * stage_bytes + lane * block_bytes, pool + (size_t)page * g.page_bytes, block_bytes, bar);
+                if (scales)
+                    bulk_g2s_addr(smem_u32(&k_scale[st][0]) + lane * kPageTok * 4u, p.pool + (size_t)page * g.page_bytes + (size_t)g.kv_heads * block_bytes + kvh * (kPageTok * 4),
+                                  kPageTok * 4u, bar);
+            }
             __syncwarp();
             n_req = it + 1;
             if (it == 0) request_queries();   // behind the first pages, which come from further away
@@ -375,7 +411,7 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
         for (int it = 0; it < n_blocks; ++it) {
             const int st = it % p.stages;
             if (!wait(&p_full[it % kScores], (uint32_t)(it / kScores) & 1u)) break;
-            const int keys = hi - (key_base + it * kKeys);
+            const int keys = hi - key_of(it);
             if (keys < kKeys) {
                 // cache rows past the last visible key may hold anything; their weights are 0, but 0 x NaN is not
                 for (int r = keys; r < kKeys; ++r)
@@ -411,7 +447,7 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
         }
         const int my_lo = GROUPED ? first_visible(g.mask, g.mask_size, max(my_len - 1, 0)) : max(my_len - g.mask_size, 0);
         float r1 = 0.f, r2 = 0.f;
-        if (GROUPED && p.r1 && r < live) { r1 = p.r1[heads0 + r % heads_n]; r2 = p.r2[heads0 + r % heads_n]; }
+        if (GROUPED && p.r1 && r < live) { r1 = p.r1[heads0 + r % heads_n]; if (!LINEAR) r2 = p.r2[heads0 + r % heads_n]; }
         const uint32_t t_lane = tmem + ((uint32_t)(warp * 32) << 16);
         // capped scores of up to 60 in log2 units need no running maximum: every row sees itself at no distance, so its largest weight lies
         // between 2^-60 and 2^60
@@ -426,9 +462,17 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
                 float s[kKeys];
                 tmem_ld_32(t_s, *reinterpret_cast<float(*)[32]>(&s[0]));
                 tmem_ld_32(t_s + 32u, *reinterpret_cast<float(*)[32]>(&s[32]));
-                const int key0 = key_base + it * kKeys;
+                const int key0 = key_of(it);
                 const int v_lo = my_lo - key0, v_hi = my_len - key0;   // visible keys of this block: [v_lo, v_hi)
-                if constexpr (GROUPED) score_log2(s, p.scale_log2, p.cap_log2, r1, r2, my_len - 1 - key0);
+                if constexpr (LINEAR) {
+                    if (g.key_scales) {   // they have come with the pages; the wait is for this thread to see them
+                        if (!wait(&k_full[it % p.stages], (uint32_t)(it / p.stages) & 1u)) break;
+                        scale_columns(s, k_scale[it % p.stages]);
+                    }
+                    score_linear(s, p.scale_log2, p.cap_log2, r1, my_len - 1 - key0);
+                } else if constexpr (GROUPED) {
+                    score_log2(s, p.scale_log2, p.cap_log2, r1, r2, my_len - 1 - key0);
+                }
                 const float mul = GROUPED ? 1.f : p.scale_log2;
                 if (v_lo > 0 || v_hi < kKeys) {
 #pragma unroll
@@ -565,6 +609,7 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
                 const size_t token_head = (size_t)(row0 + r / heads_n) * g.heads + heads0 + r % heads_n;
                 const size_t part = (((size_t)tile * gridDim.z + hb) * p.splits + blockIdx.y) * kRows + (TWO ? tid : r);
                 if (p.splits > 1 && r < live) p.part_ml[part] = make_float2(m_run, failed ? 0.f : l_run);
+                if (!TWO && p.sink && p.splits == 1) l_run += ex2f(fmaf(p.sink[heads0 + r % heads_n], kLog2e, -m_run));   // infinite: the output is 0
                 const float inv = p.splits > 1 ? 1.f : l_run > 0.f ? 1.f / l_run : 0.f;
                 if (any)
 #pragma unroll 1
@@ -611,6 +656,7 @@ struct CombineParams {
     __nv_bfloat16* out;
     int heads, group, rows_per_token, head_blocks, splits, cols, out_stride, vdim;
     HeadOutput head_out;
+    const float* sink;
 };
 template <bool TWO>
 __global__ void __launch_bounds__(128) flash_combine_kernel(const CombineParams p) {
@@ -634,6 +680,7 @@ __global__ void __launch_bounds__(128) flash_combine_kernel(const CombineParams 
         for (int s = 0; s < p.splits; ++s) m = fmaxf(m, p.part_ml[part + (size_t)s * kRows].x);
         float l = 0.f;
         for (int s = 0; s < p.splits; ++s) { const float2 v = p.part_ml[part + (size_t)s * kRows]; l += v.y * ex2f(v.x - m); }
+        if (!TWO && p.sink) l += ex2f(fmaf(p.sink[head], kLog2e, -m));
         const float inv = (l > 0.f ? 1.f / l : 0.f) * (q ? -ho.lambda : 1.f);
         for (int s = 0; s < p.splits; ++s) {
             const float2 v = p.part_ml[part + (size_t)s * kRows];
@@ -688,7 +735,7 @@ size_t tc_scratch_bytes(int64_t n_tiles, int z_blocks, int splits, int value_blo
 }
 
 // Launches the kernel and, with key splits, the merge. The caller has filled in everything but the fields set here.
-template <bool GROUPED, int kScores, bool TWO = false>
+template <bool GROUPED, int kScores, bool TWO = false, bool LINEAR = false>
 int launch_flash(TcParams& p, int64_t n_tiles, void* d_scratch, cudaStream_t st) {
     constexpr int kTileRows = TWO ? kRows / 2 : kRows;
     const FlashShape& g = p.g;
@@ -701,11 +748,11 @@ int launch_flash(TcParams& p, int64_t n_tiles, void* d_scratch, cudaStream_t st)
     p.part_o = static_cast<float*>(d_scratch);
     p.part_ml = reinterpret_cast<float2*>(p.part_o + rows * (g.value_blocks * 64));
     static PerDeviceOnce attr_once;
-    if (attr_once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(flash_tc_kernel<GROUPED, kScores, TWO>, cudaFuncAttributeMaxDynamicSharedMemorySize, 221 * 1024));
+    if (attr_once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(flash_tc_kernel<GROUPED, kScores, TWO, LINEAR>, cudaFuncAttributeMaxDynamicSharedMemorySize, 221 * 1024));
     const size_t smem = (size_t)g.query_blocks * kRows * 128 + (size_t)p.stages * g.blocks * kKeys * 128 + 1024;
-    int rc = launch_kernel(flash_tc_kernel<GROUPED, kScores, TWO>, dim3((unsigned)n_tiles, (unsigned)p.splits, (unsigned)z), dim3(kTcThreads), smem, st, 1, p);
+    int rc = launch_kernel(flash_tc_kernel<GROUPED, kScores, TWO, LINEAR>, dim3((unsigned)n_tiles, (unsigned)p.splits, (unsigned)z), dim3(kTcThreads), smem, st, 1, p);
     if (rc || p.splits == 1) return rc;
-    CombineParams c = {p.part_o, p.part_ml, p.tile_row, p.tile_rows, p.out, g.heads, g.group, p.rows_per_token, p.head_blocks, p.splits, g.value_blocks * 64, g.out_stride, g.vdim, p.head_out};
+    CombineParams c = {p.part_o, p.part_ml, p.tile_row, p.tile_rows, p.out, g.heads, g.group, p.rows_per_token, p.head_blocks, p.splits, g.value_blocks * 64, g.out_stride, g.vdim, p.head_out, p.sink};
     // CTAs of four warps cover the rows of a tile
     return launch_kernel(flash_combine_kernel<TWO>, dim3((unsigned)n_tiles, kTileRows / 4, (unsigned)z), dim3(128), 0, st, 1, c);
 }

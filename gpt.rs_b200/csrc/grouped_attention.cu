@@ -7,8 +7,12 @@
 // A mask says where the keys of position i begin: at 0, at i - size + 1 (window) or at the last multiple of size (chunks).
 // Differential attention gives every query and key head two parts, each a softmax attention of its own over the same values; the output
 // of a head is their difference a1 - lambda a2, brought to unit root mean square. An output gate multiplies by sigmoid(gate). A layer may
-// read keys and values that another layer has put into the cache.
+// read keys and values that another layer has put into the cache. The penalty may be linear in the distance instead, r1_h (i - j). Queries and
+// keys may pass a short causal convolution over time and a norm per head, and the values may be the keys in front of that norm: then the
+// cache holds a vector and a number per key, and a key is their product.
 //   grouped_append_kernel       key / value part of a projection row -> the token's page
+//   grouped_prepare_kernel      convolutions with their state, norms, queries, page write: a warp per head and up to eight rows (bf16)
+//   grouped_prepare_any_kernel  the same for f32 and for sizes that the former does not take, a warp per head and row
 //   grouped_attention_kernel    plain CUDA-core attention, f32 or bf16 cache, any sizes (the f32 path)
 //   flash_tc_kernel<true>       tcgen05 flash attention (flash_tc.cuh), bf16, prompts and decode steps alike
 // A page holds, kv head by kv head, 16 rows of [value | key] or [value | key part 1 | key part 2]; in bf16 all are padded to whole
@@ -22,6 +26,7 @@ struct Shape {
     int heads, kv_heads, group, dim, vdim, mask, mask_size;
     int q_head_stride, k_off, k_head_stride, v_off, v_head_stride, q_row, out_stride;
     int maps, map_stride, g_off, g_head_stride;   // parts of a head; gate (g_head_stride 0: none)
+    int query_row, tied, width;   // row of queries; the cache holds values and numbers; columns of a cache row (f32)
     int nb, nbv, nbk;       // 64-column blocks of a cache row (bf16); of them values; of one key part
     long long page_bytes, block_bytes;
     float scale, softcap, lambda, head_scale, head_eps;
@@ -34,12 +39,19 @@ Shape shape_of(const gptrs_grouped_attention& a) {
     g.q_row = a.q_row; g.out_stride = a.out_head_stride;
     g.maps = a.maps > 1 ? a.maps : 1; g.map_stride = a.map_stride; g.g_off = a.g_offset; g.g_head_stride = a.g_head_stride;
     g.nbv = up(a.vdim, 64) / 64;
-    g.nbk = up(a.dim, 64) / 64;
+    g.tied = a.tied;
+    g.nbk = a.tied ? 0 : up(a.dim, 64) / 64;
     g.nb = g.nbv + g.maps * g.nbk;
-    g.page_bytes = a.page_bytes; g.block_bytes = a.page_bytes / a.kv_heads;
+    g.query_row = a.query_row; g.width = a.tied ? a.vdim : a.vdim + g.maps * a.dim;
+    g.page_bytes = a.page_bytes; g.block_bytes = (long long)kPageTok * (a.dtype == GPTRS_BF16 ? g.nb * 128 : g.width * 4);
     g.scale = a.scale; g.softcap = a.softcap;
     g.lambda = a.lambda_; g.head_scale = a.head_scale; g.head_eps = a.head_eps;
     return g;
+}
+
+// behind the blocks of a page: the numbers of its keys, [kv heads][16]
+__device__ __forceinline__ float* key_scale(const Shape& g, unsigned char* page, int kv_head, int t) {
+    return reinterpret_cast<float*>(page + g.kv_heads * g.block_bytes) + kv_head * kPageTok + t;
 }
 
 struct AppendParams {
@@ -91,6 +103,225 @@ __global__ void __launch_bounds__(kAppendThreads) grouped_append_kernel(const Ap
     }
 }
 
+// ---- convolutions, norms, queries, page write -----------------------------------------------------------------------------------
+struct PrepareParams {
+    Shape g;
+    gptrs_grouped_step s;
+    int taps, channels, norm;
+    float eps;
+};
+constexpr int kPrepareWarps = 4;
+
+// What a row needs of its sequence. Inputs in front of its run come from the half `old`, where the input of position q lies at q % (taps - 1).
+struct PrepareRow { int pos, first, last; const float* old; float* fresh; unsigned char* page; };
+__device__ __forceinline__ PrepareRow prepare_row(const PrepareParams& p, int pos, int slot, int first, int last, int parity) {
+    PrepareRow r;
+    r.pos = pos; r.first = first; r.last = last;
+    const size_t half = (size_t)(p.taps - 1) * p.channels;
+    float* state = p.s.d_conv_state + (size_t)slot * 2 * half;
+    r.old = state + (parity & 1) * half; r.fresh = state + ((parity & 1) ^ 1) * half;
+    r.page = static_cast<unsigned char*>(p.s.d_pool) + (size_t)p.s.d_page_table[(size_t)slot * p.s.max_pages + pos / kPageTok] * p.g.page_bytes;
+    return r;
+}
+
+// A lane holds the channels (i * 32 + lane) * 4 + e, i < NI, of a head; R rows one after another with the inputs before them in registers.
+template <int TAPS, int NI, int R>
+__global__ void __launch_bounds__(kPrepareWarps * 32) grouped_prepare_kernel(const PrepareParams p) {
+    constexpr int KEEP = TAPS - 1, HIST = KEEP > 0 ? KEEP : 1;
+    const Shape& g = p.g;
+    const int lane = threadIdx.x & 31, job = blockIdx.y * kPrepareWarps + (threadIdx.x >> 5);
+    pdl_launch_dependents();
+    const bool is_q = job < g.heads;
+    const int head = is_q ? job : job - g.heads, col0 = is_q ? head * g.q_head_stride : g.k_off + head * g.k_head_stride;
+    const bool live = job < g.heads + g.kv_heads, has_gain = p.norm && (is_q || !g.tied);
+    float w[TAPS][NI][4], gain[NI][4];
+#pragma unroll
+    for (int i = 0; i < NI; ++i) {   // constants: on their way before the kernel in front has ended
+        const int c = (i * 32 + lane) * 4;
+        const bool in = live && c < g.map_stride;
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+            const float4 v = in ? (p.s.d_conv ? __ldg(reinterpret_cast<const float4*>(p.s.d_conv + (size_t)j * p.channels + col0 + c)) : make_float4(1.f, 1.f, 1.f, 1.f))
+                                : make_float4(0.f, 0.f, 0.f, 0.f);
+            w[j][i][0] = v.x; w[j][i][1] = v.y; w[j][i][2] = v.z; w[j][i][3] = v.w;
+        }
+        const float* gp = is_q ? p.s.d_q_gain : p.s.d_k_gain;
+#pragma unroll
+        for (int e = 0; e < 4; ++e) gain[i][e] = in && has_gain && c + e < g.dim ? __ldg(gp + c + e) : 1.f;
+    }
+    pdl_wait();
+    if (!live) return;
+    const int row0 = blockIdx.x * R, rows = min(R, (int)p.s.rows - row0);
+    int v_pos = 0, v_slot = 0, v_first = 0, v_last = 0, v_par = 0;
+    if (lane < rows) {
+        v_pos = p.s.d_pos[row0 + lane]; v_slot = p.s.d_slot[row0 + lane];
+        v_first = p.s.d_run_first[row0 + lane]; v_last = p.s.d_run_last[row0 + lane]; v_par = p.s.d_parity[row0 + lane];
+    }
+    const __nv_bfloat16* x = static_cast<const __nv_bfloat16*>(p.s.d_qkv) + (size_t)row0 * g.q_row + col0;
+    uint2 cur[R][NI];
+#pragma unroll
+    for (int r = 0; r < R; ++r)
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int c = (i * 32 + lane) * 4;
+            cur[r][i] = r < rows && c < g.map_stride ? *reinterpret_cast<const uint2*>(x + (size_t)r * g.q_row + c) : make_uint2(0, 0);
+        }
+    float hist[HIST][NI][4];   // hist[k]: the input k + 1 positions back
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+        if (r >= rows) break;
+        const int row = row0 + r;
+        const PrepareRow q = prepare_row(p, __shfl_sync(0xffffffffu, v_pos, r), __shfl_sync(0xffffffffu, v_slot, r), __shfl_sync(0xffffffffu, v_first, r),
+                                         __shfl_sync(0xffffffffu, v_last, r), __shfl_sync(0xffffffffu, v_par, r));
+        if (KEEP > 0 && (r == 0 || row == q.first)) {
+#pragma unroll
+            for (int k = 0; k < KEEP; ++k)
+#pragma unroll
+                for (int i = 0; i < NI; ++i) {
+                    const int c = (i * 32 + lane) * 4, at = q.pos - 1 - k;
+                    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+                    if (c < g.map_stride) {
+                        if (row - 1 - k >= q.first) {
+                            const uint2 u = *reinterpret_cast<const uint2*>(x + (int64_t)(r - 1 - k) * g.q_row + c);
+                            v = make_float4(bf16_lo(u.x), bf16_hi(u.x), bf16_lo(u.y), bf16_hi(u.y));
+                        } else if (at >= 0) {
+                            v = *reinterpret_cast<const float4*>(q.old + (size_t)(at % HIST) * p.channels + col0 + c);
+                        }
+                    }
+                    hist[k][i][0] = v.x; hist[k][i][1] = v.y; hist[k][i][2] = v.z; hist[k][i][3] = v.w;
+                }
+        }
+        float y[NI][4], ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const float now[4] = {bf16_lo(cur[r][i].x), bf16_hi(cur[r][i].x), bf16_lo(cur[r][i].y), bf16_hi(cur[r][i].y)};
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                float a = 0.f;
+#pragma unroll
+                for (int k = KEEP - 1; k >= 0; --k) a = fmaf(w[KEEP - 1 - k][i][e], hist[k][i][e], a);
+                y[i][e] = fmaf(w[KEEP][i][e], now[e], a);
+                ss = fmaf(y[i][e], y[i][e], ss);
+            }
+            if constexpr (KEEP > 0) {
+                const int c = (i * 32 + lane) * 4;
+                if (q.last - row < KEEP && c < g.map_stride) {   // the inputs that the sequence's next step needs
+                    float* f = q.fresh + col0 + c;
+                    *reinterpret_cast<float4*>(f + (size_t)(q.pos % HIST) * p.channels) = make_float4(now[0], now[1], now[2], now[3]);
+                    if (row == q.first)   // a run shorter than the state: what it does not push out stays
+#pragma unroll
+                        for (int k = 0; k < KEEP - 1; ++k)
+                            if (q.pos - 1 - k >= 0 && k + 1 + q.last - row < KEEP)
+                                *reinterpret_cast<float4*>(f + (size_t)((q.pos - 1 - k) % HIST) * p.channels) = make_float4(hist[k][i][0], hist[k][i][1], hist[k][i][2], hist[k][i][3]);
+                }
+#pragma unroll
+                for (int k = KEEP - 1; k > 0; --k)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) hist[k][i][e] = hist[k - 1][i][e];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) hist[0][i][e] = now[e];
+            }
+        }
+        const float inv = p.norm ? 1.f / sqrtf(warp_sum(ss) / (float)g.dim + p.eps) : 1.f;
+        if (is_q) {
+            __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.s.d_q) + (size_t)row * g.query_row + col0;
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const int c = (i * 32 + lane) * 4;
+                if (c < g.map_stride)
+                    *reinterpret_cast<uint2*>(dst + c) = make_uint2(pack_bf16x2(y[i][0] * inv * gain[i][0], y[i][1] * inv * gain[i][1]),
+                                                                    pack_bf16x2(y[i][2] * inv * gain[i][2], y[i][3] * inv * gain[i][3]));
+            }
+            continue;
+        }
+        const int t = q.pos % kPageTok;
+        unsigned char* block = q.page + head * g.block_bytes;
+        const float f = g.tied ? 1.f : inv;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {   // the columns of the last block that hold no data get zeros
+            const int c = (i * 32 + lane) * 4, at = c + (g.tied ? 0 : g.nbv * 64);
+            if (c < up(g.dim, 64))
+                *reinterpret_cast<uint2*>(block + page_chunk(t, at >> 3, g.nb) + (at & 7) * 2) =
+                    make_uint2(pack_bf16x2(y[i][0] * f * gain[i][0], y[i][1] * f * gain[i][1]), pack_bf16x2(y[i][2] * f * gain[i][2], y[i][3] * f * gain[i][3]));
+        }
+        if (g.tied) {
+            if (lane == 0) *key_scale(g, q.page, head, t) = inv;
+        } else {
+            const __nv_bfloat16* v = static_cast<const __nv_bfloat16*>(p.s.d_qkv) + (size_t)row * g.q_row + g.v_off + head * g.v_head_stride;
+            for (int c = lane * 4; c < g.nbv * 64; c += 128)
+                *reinterpret_cast<uint2*>(block + page_chunk(t, c >> 3, g.nb) + (c & 7) * 2) = c < g.v_head_stride ? *reinterpret_cast<const uint2*>(v + c) : make_uint2(0, 0);
+        }
+    }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kPrepareWarps * 32) grouped_prepare_any_kernel(const PrepareParams p) {
+    constexpr bool BF16 = sizeof(T) == 2;
+    const Shape& g = p.g;
+    const int lane = threadIdx.x & 31, job = blockIdx.y * kPrepareWarps + (threadIdx.x >> 5), row = blockIdx.x, keep = p.taps - 1;
+    pdl_launch_dependents();
+    pdl_wait();
+    if (job >= g.heads + g.kv_heads) return;
+    const bool is_q = job < g.heads;
+    const int head = is_q ? job : job - g.heads, col0 = is_q ? head * g.q_head_stride : g.k_off + head * g.k_head_stride;
+    const PrepareRow q = prepare_row(p, p.s.d_pos[row], p.s.d_slot[row], p.s.d_run_first[row], p.s.d_run_last[row], p.s.d_parity[row]);
+    auto value = [](T v) -> float { if constexpr (sizeof(T) == 2) return __bfloat162float(v); else return v; };
+    auto put = [](T* dst, float v) { if constexpr (sizeof(T) == 2) *dst = __float2bfloat16_rn(v); else *dst = v; };
+    const T* x = static_cast<const T*>(p.s.d_qkv) + (size_t)row * g.q_row;
+    auto input = [&](int k, int c) -> float {   // k positions back
+        if (row - k >= q.first) return value(x[col0 + c - (int64_t)k * g.q_row]);
+        const int at = q.pos - k;
+        return at >= 0 ? q.old[(size_t)(at % keep) * p.channels + col0 + c] : 0.f;
+    };
+    auto conv = [&](int c) -> float {
+        if (!p.s.d_conv) return input(0, c);
+        float a = 0.f;
+        for (int k = keep; k >= 0; --k) a = fmaf(p.s.d_conv[(size_t)(keep - k) * p.channels + col0 + c], input(k, c), a);
+        return a;
+    };
+    float inv = 1.f;
+    if (p.norm) {
+        float ss = 0.f;
+        for (int c = lane; c < g.dim; c += 32) { const float v = conv(c); ss = fmaf(v, v, ss); }
+        inv = 1.f / sqrtf(warp_sum(ss) / (float)g.dim + p.eps);
+    }
+    const float* gp = p.norm && (is_q || !g.tied) ? (is_q ? p.s.d_q_gain : p.s.d_k_gain) : nullptr;
+    const int t = q.pos % kPageTok;
+    unsigned char* block = q.page + head * g.block_bytes;
+    auto cell = [&](int c) -> T* {   // column c of the token's cache row, values first
+        if constexpr (BF16) return reinterpret_cast<T*>(block + page_chunk(t, c >> 3, g.nb) + (c & 7) * 2);
+        else return reinterpret_cast<T*>(block) + (size_t)t * g.width + c;
+    };
+    const int key0 = g.tied ? 0 : BF16 ? g.nbv * 64 : g.vdim, key_cols = BF16 ? up(g.dim, 64) : g.dim, val_cols = BF16 ? g.nbv * 64 : g.vdim;
+    for (int c = lane; c < (is_q ? g.map_stride : key_cols); c += 32) {
+        const float f = !is_q && g.tied ? 1.f : inv;
+        const float v = c < g.dim ? conv(c) * f * (gp ? gp[c] : 1.f) : 0.f;
+        put(is_q ? static_cast<T*>(p.s.d_q) + (size_t)row * g.query_row + col0 + c : cell(key0 + c), v);
+    }
+    if (!is_q && g.tied && lane == 0) *key_scale(g, q.page, head, t) = inv;
+    if (!is_q && !g.tied)
+        for (int c = lane; c < val_cols; c += 32) put(cell(c), c < g.vdim ? value(x[g.v_off + head * g.v_head_stride + c]) : 0.f);
+    if (keep > 0 && q.last - row < keep)
+        for (int c = lane; c < g.map_stride; c += 32) {
+            float* f = q.fresh + col0 + c;
+            f[(size_t)(q.pos % keep) * p.channels] = input(0, c);
+            if (row == q.first)
+                for (int k = 1; k < keep; ++k)
+                    if (q.pos - k >= 0 && k + q.last - row < keep) f[(size_t)((q.pos - k) % keep) * p.channels] = input(k, c);
+        }
+}
+
+template <int TAPS, int NI>
+int launch_prepare_rows(const PrepareParams& p, cudaStream_t st) {
+    const unsigned jobs = (unsigned)ceil_div(p.g.heads + p.g.kv_heads, kPrepareWarps);
+    if (p.s.rows <= 256) return launch_kernel(grouped_prepare_kernel<TAPS, NI, 1>, dim3((unsigned)p.s.rows, jobs), dim3(kPrepareWarps * 32), 0, st, 1, p);
+    return launch_kernel(grouped_prepare_kernel<TAPS, NI, 8>, dim3((unsigned)ceil_div((int)p.s.rows, 8), jobs), dim3(kPrepareWarps * 32), 0, st, 1, p);
+}
+template <int NI>
+int launch_prepare(const PrepareParams& p, cudaStream_t st) {
+    return p.taps == 1 ? launch_prepare_rows<1, NI>(p, st) : p.taps == 2 ? launch_prepare_rows<2, NI>(p, st) : p.taps == 3 ? launch_prepare_rows<3, NI>(p, st) : launch_prepare_rows<4, NI>(p, st);
+}
+
 // ---- plain attention: one CTA per (head, row) ---------------------------------------------------------------------------------
 struct AttnParams {
     Shape g;
@@ -98,6 +329,7 @@ struct AttnParams {
     const unsigned char* pool;
     const int *page_table, *slot, *ctx_len;
     const float *r1, *r2;
+    const int* reach;
     void* out;
     int* status;
     int max_pages;
@@ -119,14 +351,15 @@ __global__ void __launch_bounds__(kPlainThreads) grouped_attention_kernel(const 
     pdl_wait();
     int len = p.ctx_len[row];
     if (len < 0 || len > p.max_pages * kPageTok) { if (tid == 0) atomicExch(p.status, 2); len = len < 0 ? 0 : p.max_pages * kPageTok; }
-    const int lo = first_visible(g.mask, g.mask_size, max(len - 1, 0));
-    const int kvh = head / g.group, width = g.vdim + g.maps * g.dim;
+    const int kvh = head / g.group, width = g.width;
+    int lo = first_visible(g.mask, g.mask_size, max(len - 1, 0));
+    if (p.reach) lo = max(lo, len - 1 - p.reach[kvh]);
     const int* pt = p.page_table + (size_t)p.slot[row] * p.max_pages;
-    const float r1 = p.r1 ? p.r1[head] : 0.f, r2 = p.r1 ? p.r2[head] : 0.f;
+    const float r1 = p.r1 ? p.r1[head] : 0.f, r2 = p.r2 ? p.r2[head] : 0.f;
     float o[kPlainCols], acc[kPlainCols];
     float m, l;
     for (int part = 0; part < g.maps; ++part) {
-        const size_t qo = (size_t)row * g.q_row + (size_t)head * g.q_head_stride + (size_t)part * g.map_stride;
+        const size_t qo = (size_t)row * g.query_row + (size_t)head * g.q_head_stride + (size_t)part * g.map_stride;
         for (int c = tid; c < dim_pad; c += kPlainThreads) {
             float v = 0.f;
             if (c < g.dim) v = BF16 ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.qkv)[qo + c]) : static_cast<const float*>(p.qkv)[qo + c];
@@ -141,13 +374,13 @@ __global__ void __launch_bounds__(kPlainThreads) grouped_attention_kernel(const 
             float s = -INFINITY;
             if (tid < n) {
                 const int j = j0 + tid;
-                const long long base = (long long)pt[j / kPageTok] * g.page_bytes + kvh * g.block_bytes;
+                const long long page = (long long)pt[j / kPageTok] * g.page_bytes, base = page + kvh * g.block_bytes;
                 s_row[tid] = base;
                 s = 0.f;
                 if constexpr (BF16) {
                     const unsigned char* pg = p.pool + base;
                     for (int k = 0; k < dim_pad / 8; ++k) {
-                        const uint4 u = __ldg(reinterpret_cast<const uint4*>(pg + page_chunk(j % kPageTok, (g.nbv + part * g.nbk) * 8 + k, g.nb)));
+                        const uint4 u = __ldg(reinterpret_cast<const uint4*>(pg + page_chunk(j % kPageTok, (g.tied ? 0 : g.nbv + part * g.nbk) * 8 + k, g.nb)));
                         const float* qk = qs + k * 8;
                         s = fmaf(qk[0], bf16_lo(u.x), s); s = fmaf(qk[1], bf16_hi(u.x), s);
                         s = fmaf(qk[2], bf16_lo(u.y), s); s = fmaf(qk[3], bf16_hi(u.y), s);
@@ -155,12 +388,13 @@ __global__ void __launch_bounds__(kPlainThreads) grouped_attention_kernel(const 
                         s = fmaf(qk[6], bf16_lo(u.w), s); s = fmaf(qk[7], bf16_hi(u.w), s);
                     }
                 } else {
-                    const float* kv = reinterpret_cast<const float*>(p.pool + base) + (size_t)(j % kPageTok) * width + g.vdim + part * g.dim;
+                    const float* kv = reinterpret_cast<const float*>(p.pool + base) + (size_t)(j % kPageTok) * width + (g.tied ? 0 : g.vdim + part * g.dim);
                     for (int c = 0; c < g.dim; ++c) s = fmaf(qs[c], __ldg(kv + c), s);
                 }
+                if (g.tied) s *= __ldg(reinterpret_cast<const float*>(p.pool + page + g.kv_heads * g.block_bytes) + kvh * kPageTok + j % kPageTok);
                 s *= g.scale;
                 if (g.softcap > 0.f) s = g.softcap * tanhf(s / g.softcap);
-                if (p.r1) s -= r1 * log1pf(r2 * (float)(len - 1 - j));
+                if (p.r1) s -= r1 * (p.r2 ? log1pf(r2 * (float)(len - 1 - j)) : (float)(len - 1 - j));
             }
             const float wm = warp_max(s);
             if ((tid & 31) == 0) sh[tid >> 5] = wm;
@@ -230,7 +464,7 @@ int encode_queries(const void* qkv, const Shape& g, int64_t n_tokens, int heads,
     EncodeTiledFn enc = encode_fn();
     if (!enc) return fail(GPTRS_EXECUTION, "cuTensorMapEncodeTiled is not available");
     cuuint64_t dims[4] = {(cuuint64_t)g.map_stride, (cuuint64_t)g.maps, (cuuint64_t)g.heads, (cuuint64_t)n_tokens};
-    cuuint64_t strides[3] = {(cuuint64_t)g.map_stride * 2, (cuuint64_t)g.q_head_stride * 2, (cuuint64_t)g.q_row * 2};
+    cuuint64_t strides[3] = {(cuuint64_t)g.map_stride * 2, (cuuint64_t)g.q_head_stride * 2, (cuuint64_t)g.query_row * 2};
     cuuint32_t box[4] = {64, 1, (cuuint32_t)heads, (cuuint32_t)tokens};
     cuuint32_t estr[4] = {1, 1, 1, 1};
     CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 4, const_cast<void*>(qkv), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
@@ -240,6 +474,7 @@ int encode_queries(const void* qkv, const Shape& g, int64_t n_tokens, int heads,
 }
 
 int tile_rows(const Shape& g) { return g.maps > 1 ? kRows / 2 : kRows; }   // rows of a tile that are (token, head) pairs of their own
+int query_blocks(const Shape& g) { return g.tied ? g.nbv : g.nb - g.nbv; }
 int tile_tokens(const Shape& g) { return g.group >= tile_rows(g) ? 1 : tile_rows(g) / g.group; }
 
 }  // namespace
@@ -260,15 +495,25 @@ int gptrs_cuda_grouped_layout(gptrs_grouped_attention* a) {
     if (a->vdim > kPlainThreads * kPlainCols || a->dim > 8192) return fail(GPTRS_UNIMPLEMENTED, "grouped attention: vdim above 1024 or dim above 8192");
     const bool bf16 = a->dtype == GPTRS_BF16;
     const int maps = a->maps > 1 ? a->maps : 1;
+    const bool prepared = a->taps > 0 || a->qk_norm || a->tied;
+    GPTRS_REQUIRE(a->distance_bias >= GPTRS_DISTANCE_NONE && a->distance_bias <= GPTRS_DISTANCE_LINEAR && a->taps >= 0, "grouped attention: distance penalty or taps");
+    GPTRS_REQUIRE(!a->tied || (a->dim == a->vdim && a->distance_bias != GPTRS_DISTANCE_LOG), "grouped attention: values that are keys have the keys' size and no logarithmic penalty");
+    if (maps > 1 && (prepared || a->distance_bias == GPTRS_DISTANCE_LINEAR)) return fail(GPTRS_UNIMPLEMENTED, "grouped attention: two parts with convolutions, norms or a linear penalty");
+    if (prepared && (a->gate || a->shared_kv)) return fail(GPTRS_UNIMPLEMENTED, "grouped attention: convolutions or norms with a gate or shared keys");
     a->map_stride = bf16 ? up(a->dim, 8) : a->dim;
     a->q_head_stride = a->k_head_stride = maps * a->map_stride;
     a->v_head_stride = a->out_head_stride = bf16 ? up(a->vdim, 8) : a->vdim;
     a->k_offset = a->heads * a->q_head_stride;
     a->v_offset = a->k_offset + (a->shared_kv ? 0 : a->kv_heads * a->k_head_stride);
-    a->g_offset = a->v_offset + (a->shared_kv ? 0 : a->kv_heads * a->v_head_stride);
+    a->g_offset = a->v_offset + (a->shared_kv || a->tied ? 0 : a->kv_heads * a->v_head_stride);
     a->g_head_stride = a->gate ? a->out_head_stride : 0;
     a->q_row = a->g_offset + a->heads * a->g_head_stride;
-    a->page_bytes = (int64_t)a->kv_heads * kPageTok * (bf16 ? (maps * up(a->dim, 64) + up(a->vdim, 64)) * 2 : (maps * a->dim + a->vdim) * 4);
+    a->query_row = prepared ? a->heads * a->q_head_stride : a->q_row;
+    a->conv_channels = a->v_offset;
+    a->conv_floats = a->taps > 1 ? (int64_t)2 * (a->taps - 1) * a->conv_channels : 0;
+    const int key_parts = a->tied ? 0 : maps;
+    a->page_bytes = (int64_t)a->kv_heads * kPageTok * (bf16 ? (key_parts * up(a->dim, 64) + up(a->vdim, 64)) * 2 : (key_parts * a->dim + a->vdim) * 4);
+    if (a->tied) a->page_bytes = (a->page_bytes + (int64_t)a->kv_heads * kPageTok * 4 + 127) / 128 * 128;
     return GPTRS_OK;
 }
 
@@ -277,6 +522,7 @@ int gptrs_cuda_grouped_append(const gptrs_grouped_attention* a, const void* d_qk
     GPTRS_REQUIRE(a && d_qkv && d_positions && d_slot && d_page_table && d_pool, "null pointer");
     GPTRS_REQUIRE(a->q_row > 0 && max_pages > 0, "grouped attention: layout not filled in");
     GPTRS_REQUIRE(!a->shared_kv, "grouped attention: these rows hold no keys and values");
+    GPTRS_REQUIRE(a->taps == 0 && !a->qk_norm && !a->tied, "grouped attention: these rows go through gptrs_cuda_grouped_prepare");
     if (n_tokens == 0) return GPTRS_OK;
     AppendParams p = {shape_of(*a), d_qkv, d_positions, d_slot, d_page_table, static_cast<unsigned char*>(d_pool), (int)max_pages};
     const dim3 grid((unsigned)n_tokens);
@@ -284,10 +530,29 @@ int gptrs_cuda_grouped_append(const gptrs_grouped_attention* a, const void* d_qk
                                   : launch_kernel(grouped_append_kernel<false>, grid, dim3(kAppendThreads), 0, as_stream(stream), 1, p);
 }
 
+int gptrs_cuda_grouped_prepare(const gptrs_grouped_attention* a, const gptrs_grouped_step* step, void* stream) {
+    GPTRS_REQUIRE(a && step && a->q_row > 0, "null pointer, or layout not filled in");
+    const gptrs_grouped_step& s = *step;
+    GPTRS_REQUIRE(a->taps > 0 || a->qk_norm || a->tied, "grouped attention: these rows go through gptrs_cuda_grouped_append");
+    GPTRS_REQUIRE(s.d_qkv && s.d_slot && s.d_pos && s.d_run_first && s.d_run_last && s.d_parity && s.d_page_table && s.d_pool && s.d_q && s.max_pages > 0, "null pointer");
+    GPTRS_REQUIRE((a->taps == 0 || s.d_conv) && (a->taps <= 1 || s.d_conv_state) && (!a->qk_norm || (s.d_q_gain && (a->tied || s.d_k_gain))), "null pointer");
+    GPTRS_REQUIRE(s.rows >= 0 && s.rows < (1ll << 31) && a->heads + a->kv_heads <= 65535 * kPrepareWarps, "bad shape");
+    if (s.rows == 0) return GPTRS_OK;
+    PrepareParams p = {shape_of(*a), s, a->taps > 0 ? a->taps : 1, a->conv_channels, a->qk_norm, a->head_eps};
+    if (a->taps == 0) p.s.d_conv = nullptr;
+    cudaStream_t st = as_stream(stream);
+    const uintptr_t ptrs = reinterpret_cast<uintptr_t>(s.d_qkv) | reinterpret_cast<uintptr_t>(s.d_conv) | reinterpret_cast<uintptr_t>(s.d_conv_state) |
+                           reinterpret_cast<uintptr_t>(s.d_pool) | reinterpret_cast<uintptr_t>(s.d_q);
+    if (a->dtype == GPTRS_BF16 && p.taps <= 4 && a->dim <= 256 && (ptrs & 15) == 0) return a->dim <= 128 ? launch_prepare<1>(p, st) : launch_prepare<2>(p, st);
+    const dim3 grid((unsigned)s.rows, (unsigned)ceil_div(a->heads + a->kv_heads, kPrepareWarps));
+    return a->dtype == GPTRS_BF16 ? launch_kernel(grouped_prepare_any_kernel<__nv_bfloat16>, grid, dim3(kPrepareWarps * 32), 0, st, 1, p)
+                                  : launch_kernel(grouped_prepare_any_kernel<float>, grid, dim3(kPrepareWarps * 32), 0, st, 1, p);
+}
+
 int gptrs_cuda_grouped_tile_tokens(const gptrs_grouped_attention* a) {
     if (!a || a->dtype != GPTRS_BF16 || a->heads < 1) return 0;
     const Shape g = shape_of(*a);
-    return tc_fits(g.nb - g.nbv, g.nbv, g.nb) ? tile_tokens(g) : 0;
+    return tc_fits(query_blocks(g), g.nbv, g.nb) ? tile_tokens(g) : 0;
 }
 
 int gptrs_cuda_grouped_splits(const gptrs_grouped_attention* a, int64_t n_tiles, int64_t max_ctx_len) {
@@ -297,7 +562,7 @@ int gptrs_cuda_grouped_splits(const gptrs_grouped_attention* a, int64_t n_tiles,
     const int64_t span = max_ctx_len < limit ? max_ctx_len : limit;
     const int64_t blocks = (span + kPageTok - 1 + kKeys - 1) / kKeys;
     const Shape g = shape_of(*a);
-    int64_t s = (tc_fits_twice(g.nb - g.nbv, g.nbv, g.nb) ? 2 : 1) * sm_count() / (n_tiles * a->kv_heads * ceil_div(g.group, tile_rows(g)));
+    int64_t s = (tc_fits_twice(query_blocks(g), g.nbv, g.nb) ? 2 : 1) * sm_count() / (n_tiles * a->kv_heads * ceil_div(g.group, tile_rows(g)));
     if (s > blocks) s = blocks;
     return (int)(s < 1 ? 1 : s);
 }
@@ -309,19 +574,19 @@ size_t gptrs_cuda_grouped_scratch_bytes(const gptrs_grouped_attention* a, int64_
 }
 
 int gptrs_cuda_grouped_attention(const gptrs_grouped_attention* a, const void* d_qkv, const void* d_pool, const int32_t* d_page_table, int64_t max_pages,
-                                 const int32_t* d_slot, const int32_t* d_ctx_len, const float* d_r1, const float* d_r2, const int32_t* d_tile_row,
+                                 const int32_t* d_slot, const int32_t* d_ctx_len, const float* d_r1, const float* d_r2, const int32_t* d_reach, const int32_t* d_tile_row,
                                  const int32_t* d_tile_rows, int64_t n_tiles, int splits, void* d_out, void* d_scratch, size_t scratch_bytes,
                                  int32_t* d_status, int64_t n_tokens, void* stream) {
     GPTRS_REQUIRE(a && d_qkv && d_pool && d_page_table && d_slot && d_ctx_len && d_out && d_status, "null pointer");
-    GPTRS_REQUIRE(!a->distance_bias || (d_r1 && d_r2), "grouped attention: distance penalty without its numbers");
+    GPTRS_REQUIRE(a->distance_bias == GPTRS_DISTANCE_NONE || (d_r1 && (d_r2 || a->distance_bias == GPTRS_DISTANCE_LINEAR)), "grouped attention: distance penalty without its numbers");
     GPTRS_REQUIRE(a->q_row > 0 && max_pages > 0 && max_pages * kPageTok < ((int64_t)1 << 30), "grouped attention: layout not filled in, or a bad page table");
     if (n_tokens == 0) return GPTRS_OK;
     const Shape g = shape_of(*a);
     cudaStream_t st = as_stream(stream);
-    const float *r1 = a->distance_bias ? d_r1 : nullptr, *r2 = a->distance_bias ? d_r2 : nullptr;
+    const float *r1 = a->distance_bias != GPTRS_DISTANCE_NONE ? d_r1 : nullptr, *r2 = a->distance_bias == GPTRS_DISTANCE_LOG ? d_r2 : nullptr;
     if (n_tiles <= 0) {   // plain kernel: every row by itself
         GPTRS_REQUIRE(n_tokens <= 65535, "grouped attention: too many rows in one launch");
-        AttnParams p = {g, d_qkv, static_cast<const unsigned char*>(d_pool), d_page_table, d_slot, d_ctx_len, r1, r2, d_out, d_status, (int)max_pages};
+        AttnParams p = {g, d_qkv, static_cast<const unsigned char*>(d_pool), d_page_table, d_slot, d_ctx_len, r1, r2, d_reach, d_out, d_status, (int)max_pages};
         const size_t smem = ((size_t)up(g.dim, 8) + kPlainThreads) * 4;
         const dim3 grid((unsigned)g.heads, (unsigned)n_tokens);
         return a->dtype == GPTRS_BF16 ? launch_kernel(grouped_attention_kernel<true>, grid, dim3(kPlainThreads), smem, st, 1, p)
@@ -343,10 +608,11 @@ int gptrs_cuda_grouped_attention(const gptrs_grouped_attention* a, const void* d
     p.q_one_bytes = (uint32_t)box_heads * 128u;
     FlashShape& f = p.g;
     f.heads = g.heads; f.kv_heads = g.kv_heads; f.group = g.group;
-    f.blocks = g.nb; f.value_blocks = f.key_block = g.nbv; f.query_blocks = g.nb - g.nbv;
-    f.map_blocks = g.nbk;
+    f.blocks = g.nb; f.value_blocks = g.nbv; f.key_block = g.tied ? 0 : g.nbv; f.query_blocks = query_blocks(g);
+    f.map_blocks = f.query_blocks / g.maps;
+    f.key_scales = g.tied;
     for (int b = 0; b < f.query_blocks; ++b) {
-        const int left = g.dim - b % g.nbk * 64;
+        const int left = g.dim - b % f.map_blocks * 64;
         f.steps[b] = left >= 64 ? 4 : (left + 15) / 16;
     }
     f.mask = g.mask; f.mask_size = g.mask_size;
@@ -357,12 +623,13 @@ int gptrs_cuda_grouped_attention(const gptrs_grouped_attention* a, const void* d
     p.out = static_cast<__nv_bfloat16*>(d_out);
     p.status = d_status;
     p.max_pages = (int)max_pages; p.splits = splits;
-    p.r1 = r1; p.r2 = r2;
+    p.r1 = r1; p.r2 = r2; p.reach = d_reach;
     p.scale_log2 = g.softcap > 0.f ? 2.f * kLog2e * g.scale / g.softcap : kLog2e * g.scale;
     p.cap_log2 = g.softcap > 0.f ? kLog2e * g.softcap : 0.f;
     p.head_out = {g.lambda, g.head_scale, g.head_eps, g.g_head_stride > 0 ? static_cast<const __nv_bfloat16*>(d_qkv) + g.g_off : nullptr, g.q_row, g.g_head_stride};
     const bool twice = tc_fits_twice(f.query_blocks, f.value_blocks, f.blocks);
     if (g.maps > 1) return twice ? launch_flash<true, 2, true>(p, n_tiles, d_scratch, st) : launch_flash<true, 3, true>(p, n_tiles, d_scratch, st);
+    if (g.tied || a->distance_bias == GPTRS_DISTANCE_LINEAR) return twice ? launch_flash<true, 2, false, true>(p, n_tiles, d_scratch, st) : launch_flash<true, 3, false, true>(p, n_tiles, d_scratch, st);
     return twice ? launch_flash<true, 2>(p, n_tiles, d_scratch, st) : launch_flash<true, 3>(p, n_tiles, d_scratch, st);
 }
 

@@ -5,8 +5,8 @@
 //   score(i, j, h) = ((W_uk,h^T q_ih) . c_j + rot(q'_ih) . k'_j) * scale,      o_ih = W_uv,h (sum_j p_ijh c_j)
 //
 // so attention itself is multi-query attention with kv_rank + rot_dim key dimensions whose values are the first kv_rank of
-// them, over a sliding window (position i sees i - window + 1 .. i) or all of 0 .. i. The two absorbed products are batched matmuls in
-// front of and behind the kernels of this file. Where queries come through a latent of their own, the first projection gives both
+// them, over a sliding window (position i sees i - window + 1 .. i) or all of 0 .. i; a sink per head adds exp(sink) to the denominator
+// of the softmax. The two absorbed products are batched matmuls in front of and behind the kernels of this file. Where queries come through a latent of their own, the first projection gives both
 // latents, and the kernel that writes the page also norms the query latent for the second projection:
 //   latent_append_kernel        norm of the latent(s), rotation of the shared key part and of the queries, page write
 //   latent_keys_kernel          its first half for bf16 rows with a query latent
@@ -272,6 +272,7 @@ struct AttnParams {
     const void* qa;
     const unsigned char* pool;
     const int *page_table, *slot, *ctx_len;
+    const float* sink;          // [heads] or null
     void* out;                  // [T][heads][lat_stride]
     int* status;
     int max_pages;
@@ -357,6 +358,7 @@ __global__ void __launch_bounds__(kPlainThreads) latent_attention_kernel(const A
         __syncthreads();
     }
     const size_t oo = ((size_t)row * g.heads + head) * g.lat_stride;
+    if (p.sink) l += expf(p.sink[head] - m);   // infinite where the sink outweighs everything: the output is 0
     const float inv = l > 0.f ? 1.f / l : 0.f;
 #pragma unroll
     for (int i = 0; i < kPlainCols; ++i) {
@@ -496,7 +498,7 @@ size_t gptrs_cuda_latent_scratch_bytes(const gptrs_latent_attention* a, int64_t 
 }
 
 int gptrs_cuda_latent_attention(const gptrs_latent_attention* a, const void* d_qa, const void* d_pool, const int32_t* d_page_table, int64_t max_pages,
-                                const int32_t* d_slot, const int32_t* d_ctx_len, const int32_t* d_tile_row, const int32_t* d_tile_rows, int64_t n_tiles,
+                                const int32_t* d_slot, const int32_t* d_ctx_len, const float* d_sink, const int32_t* d_tile_row, const int32_t* d_tile_rows, int64_t n_tiles,
                                 int splits, void* d_out, void* d_scratch, size_t scratch_bytes, int32_t* d_status, int64_t n_tokens, void* stream) {
     GPTRS_REQUIRE(a && d_qa && d_pool && d_page_table && d_slot && d_ctx_len && d_out && d_status, "null pointer");
     GPTRS_REQUIRE(a->q_row > 0 && max_pages > 0 && max_pages * kPageTok < ((int64_t)1 << 30), "latent attention: layout not filled in, or a bad page table");
@@ -505,7 +507,7 @@ int gptrs_cuda_latent_attention(const gptrs_latent_attention* a, const void* d_q
     cudaStream_t st = as_stream(stream);
     if (n_tiles <= 0) {   // plain kernel: every row by itself
         GPTRS_REQUIRE(n_tokens <= 65535 && a->heads <= 0x7fffffff, "latent attention: too many rows in one launch");
-        AttnParams p = {g, d_qa, static_cast<const unsigned char*>(d_pool), d_page_table, d_slot, d_ctx_len, d_out, d_status, (int)max_pages};
+        AttnParams p = {g, d_qa, static_cast<const unsigned char*>(d_pool), d_page_table, d_slot, d_ctx_len, d_sink, d_out, d_status, (int)max_pages};
         const size_t smem = ((size_t)g.qa_head_stride + kPlainThreads) * 4;
         const dim3 grid((unsigned)g.heads, (unsigned)n_tokens);
         return a->dtype == GPTRS_BF16 ? launch_kernel(latent_attention_kernel<true>, grid, dim3(kPlainThreads), smem, st, 1, p)
@@ -536,6 +538,7 @@ int gptrs_cuda_latent_attention(const gptrs_latent_attention* a, const void* d_q
     p.status = d_status;
     p.max_pages = (int)max_pages; p.splits = splits;
     p.scale_log2 = kLog2e * g.scale;
+    p.sink = d_sink;
     return launch_flash<false, 3>(p, n_tiles, d_scratch, st);
 }
 

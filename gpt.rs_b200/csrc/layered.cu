@@ -1,9 +1,10 @@
 // Models whose layers are configured one by one (engine kind "layered"): weight packing, cache and state set-up and the forward
 // pass. A layer is a mixer (latent attention, latent_attention.cu; attention with grouped key / value heads, grouped_attention.cu; a
-// gated delta rule, delta_rule.cu) and an optional feed-forward (dense xIELU or gated gelu; a mixture of experts, moe_route.cu). The step
-// between two sublayers is post_norm_conv.cu (output norm, residual sum, short convolution with its per-sequence state), norm_step.cu
-// (norms on both sides of a sublayer) or stream_step.cu (norms in front, several residual streams), the matmuls are dense_bf16.cu or, in f32 mode, dense_f32.cu. Slots, pages, graphs, sampling and the
-// generator are the engine's.
+// gated delta rule, delta_rule.cu) and an optional feed-forward (dense xIELU, gated gelu or a polynomial of normed powers; a mixture of
+// experts, moe_route.cu). The step between two sublayers is post_norm_conv.cu (output norm, residual sum, short convolution with its
+// per-sequence state), norm_step.cu (norms on both sides of a sublayer), stream_step.cu (norms in front, several residual streams) or
+// depth_step.cu (output norms in groups, an average over all layers' results), the matmuls are dense_bf16.cu or, in f32 mode,
+// dense_f32.cu. Slots, pages, graphs, sampling and the generator are the engine's.
 #include <cmath>
 #include <cstdlib>
 #include <cstring>
@@ -46,6 +47,7 @@ struct Piece {
     int64_t col, col_b;         // first input column, step between batches
     int64_t mat_b;              // step between batches in whole matrices (1: a batch entry is a matrix of its own)
     int64_t mat = 0;            // matrix of the first batch entry
+    int64_t row_n = 1;          // step between packed rows
 };
 struct Leaf {
     std::string name;
@@ -119,7 +121,7 @@ int pack_weight(Model& m, const std::vector<Leaf>& leaves, int64_t batch, int64_
             pp.dst = static_cast<unsigned char*>(w->w->data) + (p.mat * w->n * w->k + p.row * dn + p.col * dk) * (bf16 ? 2 : 4);
             pp.n = p.n; pp.k = p.k; pp.total = p.batch * p.n * p.k;
             pp.sb = p.sb; pp.sn = p.sn; pp.sk = p.sk;
-            pp.db = p.row_b * dn + p.col_b * dk + p.mat_b * w->n * w->k; pp.dn = dn; pp.dk = dk;
+            pp.db = p.row_b * dn + p.col_b * dk + p.mat_b * w->n * w->k; pp.dn = p.row_n * dn; pp.dk = dk;
             pp.bf16 = bf16;
             if ((rc = launch_pack(m, pp))) break;
         }
@@ -184,7 +186,7 @@ int expert_tile_rows(const Model& m, const gptrs_moe& a, int64_t rows) {
 struct Widths {
     int64_t qkv = 0, q = 0, q_latent = 0, qa = 0, lat = 0, attn = 0, up = 0, gate_up = 0, decay = 0, gate = 0;
     int64_t delta_scratch = 0, router = 0, sorted = 0, expert_y = 0, top = 0, work = 0, row_tiles = 0;
-    size_t pool = 0, delta_state = 0, delta_conv = 0;
+    size_t pool = 0, delta_state = 0, mix_conv = 0;
     int n_state = 0;
 };
 
@@ -195,14 +197,23 @@ int build_latent(Model& m, LayeredLayer& L, const std::string& x, std::vector<st
     int rc;
     if ((rc = get_raw(m, x + "dkv.norm", {rank}, &w.latent_norm))) return rc;
     // queries (or the query latent) and the down-projection in one weight, laid out as the attention kernels expect a projection row
-    auto queries = [&](const char* name, int64_t k) {
-        return Leaf{x + name, {H * (dim + rot), k}, {{H, dim, k, 0, (dim + rot) * k, k, 1, 0, a.q_head_stride, 0, 0, 0},
-                                                    {H, rot, k, dim * k, (dim + rot) * k, k, 1, a.q_rot_offset, a.q_head_stride, 0, 0, 0}}, ""};
+    // the rotated part, pairs next to one another whichever layout the design has
+    auto rotated = [&](std::vector<Piece>* to, int64_t batch, int64_t k, int64_t src, int64_t sb, int64_t row, int64_t row_b) {
+        const int64_t half = L.cfg.rope_halves ? a.rot_dims / 2 : 0, done = 2 * half;
+        for (int64_t i = 0; i < 2 && half > 0; ++i) to->push_back({batch, half, k, src + i * half * k, sb, k, 1, row + i, row_b, 0, 0, 0, 0, 2});
+        if (rot > done) to->push_back({batch, rot - done, k, src + done * k, sb, k, 1, row + done, row_b, 0, 0, 0});
     };
-    if ((rc = pack_weight(m, {a.q_rank > 0 ? rows_of(x + "dq", a.q_rank, W, 0) : queries("q", W),
-                              {x + "dkv", {rank + rot, W}, {{1, rank, W, 0, 0, W, 1, a.dkv_offset, 0, 0, 0, 0}, {1, rot, W, rank * W, 0, W, 1, a.rot_offset, 0, 0, 0, 0}}, ""}},
-                          1, a.kv_row, W, "latent_qkv", &w.qkv, used))) return rc;
-    if (a.q_rank > 0 && ((rc = get_raw(m, x + "dq.norm", {a.q_rank}, &w.q_norm)) || (rc = pack_weight(m, {queries("uq", a.q_rank)}, 1, a.q_row, a.q_rank, "latent_uq", &w.uq, used)))) return rc;
+    auto queries = [&](const char* name, int64_t k) {
+        Leaf l = {x + name, {H * (dim + rot), k}, {{H, dim, k, 0, (dim + rot) * k, k, 1, 0, a.q_head_stride, 0, 0, 0}}, ""};
+        rotated(&l.pieces, H, k, dim * k, (dim + rot) * k, a.q_rot_offset, a.q_head_stride);
+        return l;
+    };
+    Leaf down = {x + "dkv", {rank + rot, W}, {{1, rank, W, 0, 0, W, 1, a.dkv_offset, 0, 0, 0, 0}}, ""};
+    rotated(&down.pieces, 1, W, rank * W, 0, a.rot_offset, 0);
+    const std::string order = L.cfg.rope_halves ? "_halves" + std::to_string(a.rot_dims) : "";   // part of what the packed layout is memoised under
+    if (L.cfg.sink && (rc = get_raw(m, x + "sink", {H}, &w.sink))) return rc;
+    if ((rc = pack_weight(m, {a.q_rank > 0 ? rows_of(x + "dq", a.q_rank, W, 0) : queries("q", W), down}, 1, a.kv_row, W, "latent_qkv" + order, &w.qkv, used))) return rc;
+    if (a.q_rank > 0 && ((rc = get_raw(m, x + "dq.norm", {a.q_rank}, &w.q_norm)) || (rc = pack_weight(m, {queries("uq", a.q_rank)}, 1, a.q_row, a.q_rank, "latent_uq" + order, &w.uq, used)))) return rc;
     // absorbed query: per head [rank] <- [dim], the stored key projection transposed
     if ((rc = pack_weight(m, {{x + "uk", {H * dim, rank}, {{H, rank, dim, 0, dim * rank, 1, rank, 0, 0, 0, 0, 1}}, ""}}, H, rank, dim, "latent_uk", &w.uk, used))) return rc;
     if ((rc = pack_weight(m, {{x + "uv", {H * vd, rank}, {{H, vd, rank, 0, vd * rank, rank, 1, 0, 0, 0, 0, 1}}, ""}}, H, vd, rank, "latent_uv", &w.uv, used))) return rc;
@@ -228,19 +239,87 @@ int read_lambda(Model& m, const std::string& x, int64_t dim, float diff, float* 
     return GPTRS_OK;
 }
 
+int read_floats(Model& m, const std::string& name, int64_t n, std::vector<float>* v) {
+    Tensor* t = nullptr;
+    const int rc = get_raw(m, name, {n}, &t);
+    if (rc) return rc;
+    v->resize(n);
+    const cudaError_t e = cudaMemcpy(v->data(), t->data, (size_t)n * 4, cudaMemcpyDeviceToHost);
+    tensor_release(t);
+    GPTRS_CUDA_OK(e);
+    return GPTRS_OK;
+}
+int write_floats(const std::vector<float>& v, Tensor** t) {
+    int64_t d[1] = {(int64_t)v.size()};
+    const int rc = tensor_alloc(GPTRS_F32, 1, d, false, t);
+    if (rc) return rc;
+    GPTRS_CUDA_OK(cudaMemcpy((*t)->data, v.data(), v.size() * 4, cudaMemcpyHostToDevice));
+    return GPTRS_OK;
+}
+
+// Short convolutions and norms of queries and keys, slopes of a linear distance bias, and how far its heads can see at all: the norms bound a
+// score by scale dim max |gain_q gain_k|, so a key at distance d weighs at most exp(2 bound - slope d) times as much as the position itself.
+int build_grouped_prepare(Model& m, LayeredLayer& L, const std::string& x) {
+    const gptrs_grouped_attention& a = L.gatt;
+    LayerWeights& w = *L.w;
+    int rc;
+    if (a.taps > 0) {
+        int64_t cd[2] = {a.taps, a.conv_channels};
+        if ((rc = tensor_alloc(GPTRS_F32, 2, cd, true, &w.qk_conv))) return rc;
+        if (cudaDeviceSynchronize() != cudaSuccess) return fail(GPTRS_EXECUTION, "packing a convolution failed");   // the zero fill is done
+        for (int part = 0; part < 2; ++part) {
+            const int heads = part ? a.kv_heads : a.heads;
+            Tensor* t = nullptr;
+            if ((rc = get_raw(m, x + (part ? "k.conv" : "q.conv"), {(int64_t)heads * a.dim, a.taps}, &t))) return rc;
+            PackParams pp = {};
+            pp.src = static_cast<const float*>(t->data); pp.dst = static_cast<float*>(w.qk_conv->data) + (part ? a.k_offset : 0);
+            pp.n = a.dim; pp.k = a.taps; pp.total = (int64_t)heads * a.dim * a.taps;
+            pp.sb = (int64_t)a.dim * a.taps; pp.sn = a.taps; pp.sk = 1;
+            pp.db = a.q_head_stride; pp.dn = 1; pp.dk = a.conv_channels;
+            rc = launch_pack(m, pp);
+            if (cudaStreamSynchronize(m.stream) != cudaSuccess && !rc) rc = fail(GPTRS_EXECUTION, "packing a convolution failed");
+            tensor_release(t);
+            if (rc) return rc;
+        }
+    }
+    std::vector<float> gq, gk;
+    if (a.qk_norm) {
+        if ((rc = read_floats(m, x + "q.norm", a.dim, &gq)) || (rc = read_floats(m, x + "k.norm", a.dim, &gk))) return rc;
+        std::vector<float> both(gq);
+        for (size_t i = 0; i < both.size(); ++i) both[i] *= gk[i];
+        if ((rc = write_floats(a.tied ? both : gq, &w.q_gain)) || (!a.tied && (rc = write_floats(gk, &w.k_gain)))) return rc;
+    }
+    if (a.distance_bias != GPTRS_DISTANCE_LINEAR) return GPTRS_OK;
+    std::vector<float> slope(a.heads);
+    for (int h = 0; h < a.heads; ++h) slope[h] = (float)std::exp2(-8.0 * (h + 1) / a.heads);
+    if ((rc = write_floats(slope, &w.r1)) || !a.qk_norm) return rc;
+    double bound = 0.;
+    for (int i = 0; i < a.dim; ++i) bound = std::max(bound, std::fabs((double)gq[i] * gk[i]));
+    bound *= 1.02 * a.scale * a.dim;   // queries and keys that are rounded to bf16 may be a little longer
+    std::vector<int32_t> reach(a.kv_heads);
+    for (int g = 0; g < a.kv_heads; ++g) {
+        const double least = slope[(g + 1) * (a.heads / a.kv_heads) - 1];   // slopes fall with the head
+        reach[g] = (int32_t)std::min(std::ceil((2. * bound + 32.) / least), 1e9);
+    }
+    if ((rc = w.reach.alloc(reach.size() * 4))) return rc;
+    GPTRS_CUDA_OK(cudaMemcpy(w.reach.p, reach.data(), reach.size() * 4, cudaMemcpyHostToDevice));
+    return GPTRS_OK;
+}
+
 int build_grouped(Model& m, LayeredLayer& L, const std::string& x, std::vector<std::string>* used) {
     const gptrs_grouped_attention& a = L.gatt;
     LayerWeights& w = *L.w;
     const int64_t W = m.cfg.d_model, H = a.heads, G = a.kv_heads;
     auto bias = [&](const char* n) { return L.cfg.proj_bias ? x + n + ".b" : std::string(); };
     int rc;
-    if (a.distance_bias && ((rc = get_raw(m, x + "r1", {H}, &w.r1)) || (rc = get_raw(m, x + "r2", {H}, &w.r2)))) return rc;
+    if (a.distance_bias == GPTRS_DISTANCE_LOG && ((rc = get_raw(m, x + "r1", {H}, &w.r1)) || (rc = get_raw(m, x + "r2", {H}, &w.r2)))) return rc;
+    if ((rc = build_grouped_prepare(m, L, x))) return rc;
     const int64_t maps = a.maps > 1 ? a.maps : 1;
     if (maps > 1 && (rc = read_lambda(m, x, a.dim, L.cfg.diff, &w.lambda))) return rc;
     std::vector<Leaf> in = {heads_of(x + "q", H * maps, a.dim, W, 0, a.map_stride, bias("q"))};
     if (!a.shared_kv) {
         in.push_back(heads_of(x + "k", G * maps, a.dim, W, a.k_offset, a.map_stride, bias("k")));
-        in.push_back(heads_of(x + "v", G, a.vdim, W, a.v_offset, a.v_head_stride, bias("v")));
+        if (!a.tied) in.push_back(heads_of(x + "v", G, a.vdim, W, a.v_offset, a.v_head_stride, bias("v")));
     }
     if (a.gate) in.push_back(heads_of(x + "g", H, a.vdim, W, a.g_offset, a.g_head_stride));
     if ((rc = pack_weight(m, in, 1, a.q_row, W, "grouped_qkv", &w.qkv, used))) return rc;
@@ -265,10 +344,12 @@ int build_delta(Model& m, LayeredLayer& L, const std::string& x, std::vector<std
     LayerWeights& w = *L.w;
     const int64_t W = m.cfg.d_model, H = a.heads, kq = (int64_t)a.kv_heads * a.dim, hv = H * a.vdim, hd = H * a.dim;
     int rc;
-    if ((rc = get_raw(m, x + "A_log", {H}, &w.a_log)) || (rc = get_raw(m, x + "dt_bias", {hd}, &w.dt_bias)) || (rc = get_raw(m, x + "norm", {a.vdim}, &w.delta_norm))) return rc;
+    if ((rc = get_raw(m, x + "A_log", {H}, &w.a_log)) || (rc = get_raw(m, x + "dt_bias", {a.decay_rank > 0 ? hd : H}, &w.dt_bias)) || (rc = get_raw(m, x + "norm", {a.vdim}, &w.delta_norm))) return rc;
     if ((rc = pack_weight(m, {rows_of(x + "q", kq, W, a.q_offset), rows_of(x + "k", kq, W, a.k_offset), rows_of(x + "v", hv, W, a.v_offset), rows_of(x + "b", H, W, a.beta_offset),
-                              rows_of(x + "a1", a.decay_rank, W, a.a_offset), rows_of(x + "g1", a.gate_rank, W, a.g_offset)}, 1, a.row, W, "delta_proj", &w.qkv, used))) return rc;
-    if ((rc = pack_plain(m, x + "a2", hd, a.decay_rank, "", &w.decay, used)) || (rc = pack_plain(m, x + "g2", hv, a.gate_rank, "", &w.gate, used))) return rc;
+                              a.decay_rank > 0 ? rows_of(x + "a1", a.decay_rank, W, a.a_offset) : rows_of(x + "a", H, W, a.a_offset),
+                              a.gate_rank > 0 ? rows_of(x + "g1", a.gate_rank, W, a.g_offset) : rows_of(x + "g", hv, W, a.g_offset)}, 1, a.row, W, "delta_proj", &w.qkv, used))) return rc;
+    if (a.decay_rank > 0 && (rc = pack_plain(m, x + "a2", hd, a.decay_rank, "", &w.decay, used))) return rc;
+    if (a.gate_rank > 0 && (rc = pack_plain(m, x + "g2", hv, a.gate_rank, "", &w.gate, used))) return rc;
     if ((rc = pack_weight(m, {{x + "o", {W, hv}, {{H, W, a.vdim, 0, a.vdim, hv, 1, 0, 0, 0, a.out_head_stride, 0}}, ""}}, 1, W, H * a.out_head_stride, "heads_o", &w.out, used))) return rc;
     // the three convolutions behind one another
     int64_t cd[2] = {a.conv_channels, a.taps};
@@ -309,9 +390,18 @@ int build_experts(Model& m, LayeredLayer& L, const std::string& x, std::vector<s
     int rc;
     if ((rc = pack_weight(m, up, E, gated ? 2 * Fp : F, W, "experts_up", &w.up, used)) ||
         (rc = pack_weight(m, down, E, W, gated ? Fp : F, "experts_down", &w.down, used))) return rc;
-    if (S > 0 && ((rc = pack_plain(m, x + "shared.up", S, W, "", &w.shared_up, used)) || (rc = pack_plain(m, x + "shared.down", W, S, "", &w.shared_down, used)))) return rc;
+    if (S > 0 && gated) {
+        std::vector<Leaf> shared;
+        add_gated(&shared, x + "shared.", S, W, 0);
+        if ((rc = pack_weight(m, shared, 1, 2 * pad8(S), W, "gated_up", &w.shared_up, used)) ||
+            (rc = pack_weight(m, {rows_of(x + "shared.down", W, S, 0)}, 1, W, pad8(S), "gated_down", &w.shared_down, used))) return rc;
+    } else if (S > 0 && ((rc = pack_plain(m, x + "shared.up", S, W, "", &w.shared_up, used)) || (rc = pack_plain(m, x + "shared.down", W, S, "", &w.shared_down, used)))) {
+        return rc;
+    }
     if (L.cfg.correction && (rc = get_raw(m, x + "correction", {E}, &w.correction))) return rc;
-    return pack_plain(m, x + "router", E, W, "", &w.router, used);
+    if (!L.cfg.shared_gate) return pack_plain(m, x + "router", E, W, "", &w.router, used);
+    // the shared expert's gate is one more row of the router
+    return pack_weight(m, {rows_of(x + "router", E, W, 0), rows_of(x + "shared.sg", 1, W, E)}, 1, E + 1, W, "router_gate", &w.router, used);
 }
 
 // what stands beside the norms of a sublayer (0: mixer, 1: feed-forward), depending on the block form
@@ -322,6 +412,7 @@ int build_block(Model& m, LayerWeights& w, const std::string& p, int sub) {
     int rc;
     if ((rc = get_raw(m, p + "norm" + n, {W}, sub ? &w.norm2 : &w.norm1))) return rc;
     if (c.block == GPTRS_BLOCK_SANDWICH) return get_raw(m, p + "norm" + n + "b", {W}, sub ? &w.norm2b : &w.norm1b);
+    if (c.block == GPTRS_BLOCK_DEPTH) return GPTRS_OK;
     if (c.block == GPTRS_BLOCK_OUTPUT_NORM) return get_raw(m, p + "canon" + n, {W, c.conv_taps}, sub ? &w.conv2 : &w.conv1);
     if (c.streams == 0) return GPTRS_OK;
     const std::string h = p + "hc" + n + ".";
@@ -338,6 +429,7 @@ int build_weights(Model& m, LayeredLayer& L, int l, bool drop_leaves) {
     std::vector<std::string> used;
     int rc;
     if ((rc = build_block(m, w, p, 0))) return rc;
+    if (m.lay->cfg.block == GPTRS_BLOCK_DEPTH && (rc = get_raw(m, p + "dwa", {l + 2}, &w.dwa))) return rc;
     if (L.cfg.mixer == GPTRS_MIXER_LATENT_ATTENTION) rc = build_latent(m, L, x, &used);
     else if (L.cfg.mixer == GPTRS_MIXER_GROUPED_ATTENTION) rc = build_grouped(m, L, x, &used);
     else rc = build_delta(m, L, x, &used);
@@ -361,6 +453,9 @@ int build_weights(Model& m, LayeredLayer& L, int l, bool drop_leaves) {
         add_gated(&up, f, F, W, 0);
         if ((rc = pack_weight(m, up, 1, 2 * pad8(F), W, "gated_up", &w.up, &used)) ||
             (rc = pack_weight(m, {rows_of(f + "down", W, F, 0)}, 1, W, pad8(F), "gated_down", &w.down, &used))) return rc;
+    } else if (L.cfg.mlp == GPTRS_MLP_DENSE_POLY) {
+        const int64_t F = L.cfg.d_ff;
+        if ((rc = get_raw(m, f + "act", {4}, &w.act)) || (rc = pack_plain(m, f + "up", F, W, "", &w.up, &used)) || (rc = pack_plain(m, f + "down", W, F, "", &w.down, &used))) return rc;
     } else if (L.cfg.mlp == GPTRS_MLP_EXPERTS) {
         if ((rc = build_experts(m, L, f, &used))) return rc;
     }
@@ -372,23 +467,40 @@ int build_weights(Model& m, LayeredLayer& L, int l, bool drop_leaves) {
     return GPTRS_OK;
 }
 
-// rotation tables, one pair per distinct (base, dims); angles in double, rounded once
+// Rotation tables, one pair per distinct rotation; angles in double, rounded once. With YaRN scaling (Peng et al., "YaRN: Efficient Context Window
+// Extension of Large Language Models") dimensions that turn less than `slow` times over `original` positions are slowed down by `factor`,
+// those that turn more than `fast` times stay, those in between are blended; cos and sin grow by 0.1 ln(factor) + 1.
 int add_rope(Model& m, LayeredLayer& L) {
     Layered& y = *m.lay;
     const auto& c = m.cfg;
     const gptrs_latent_attention& a = L.att;
     for (size_t i = 0; i < y.ropes.size(); ++i)
-        if (y.ropes[i]->base == L.cfg.rope_base && y.ropes[i]->dims == a.rot_dims) L.rope = (int)i;
+        if (const Layered::Rope& o = *y.ropes[i]; o.base == L.cfg.rope_base && o.dims == a.rot_dims && o.factor == L.cfg.rope_factor && o.original == L.cfg.rope_original &&
+                                                  o.fast == L.cfg.rope_fast && o.slow == L.cfg.rope_slow) L.rope = (int)i;
     if (L.rope >= 0) return GPTRS_OK;
     auto r = std::make_unique<Layered::Rope>();
     r->base = L.cfg.rope_base; r->dims = a.rot_dims;
+    r->factor = L.cfg.rope_factor; r->original = L.cfg.rope_original; r->fast = L.cfg.rope_fast; r->slow = L.cfg.rope_slow;
     const int half = a.rot_dims / 2;
+    const bool scaled = r->factor > 0. && half > 0;
+    double lo = 0., hi = 0., mag = 1.;
+    if (scaled) {
+        constexpr double kTwoPi = 6.283185307179586;
+        auto turning = [&](double turns) { return r->dims * std::log(r->original / (kTwoPi * turns)) / (2. * std::log(r->base)); };   // the dimension that turns so often
+        lo = std::max(std::floor(turning(r->fast)), 0.);
+        hi = std::min(std::ceil(turning(r->slow)), r->dims - 1.);
+        mag = 0.1 * std::log(r->factor) + 1.;
+    }
     std::vector<float> cs((size_t)c.context_length * half), sn(cs.size());
     for (int i = 0; i < half; ++i) {
-        const double f = std::pow(r->base, -2.0 * i / a.rot_dims);
+        double f = std::pow(r->base, -2.0 * i / a.rot_dims);
+        if (scaled) {
+            const double slowed = std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.), 1.);
+            f = f / r->factor * slowed + f * (1. - slowed);
+        }
         for (int q = 0; q < c.context_length; ++q) {
-            cs[(size_t)q * half + i] = (float)std::cos(q * f);
-            sn[(size_t)q * half + i] = (float)std::sin(q * f);
+            cs[(size_t)q * half + i] = (float)(std::cos(q * f) * mag);
+            sn[(size_t)q * half + i] = (float)(std::sin(q * f) * mag);
         }
     }
     int rc;
@@ -440,23 +552,27 @@ void count_widths(const Model& m, LayeredLayer& L, Widths* n) {
     } else if (L.cfg.mixer == GPTRS_MIXER_GROUPED_ATTENTION) {
         if (L.cfg.kv_from >= 0) L.pool_off = m.lay->layers[L.cfg.kv_from].pool_off;
         else n->pool += (size_t)c.kv_pages * L.gatt.page_bytes;
+        if (L.prepared()) n->q = std::max(n->q, (int64_t)L.gatt.query_row);
+        L.mix_conv_off = n->mix_conv;
+        n->mix_conv += (size_t)c.max_seqs * L.gatt.conv_floats;
     } else {
         n->decay = std::max(n->decay, (int64_t)L.delta.decay_row);
         n->gate = std::max(n->gate, (int64_t)L.delta.gate_row);
         // a pass that is not one token per sequence: at most one run per slot
         n->delta_scratch = std::max(n->delta_scratch, gptrs_cuda_delta_scratch_floats(&L.delta, c.max_tokens, std::min(c.max_seqs, c.max_tokens - 1)));
         L.delta_state_off = n->delta_state;
-        L.delta_conv_off = n->delta_conv;
+        L.mix_conv_off = n->mix_conv;
         n->delta_state += (size_t)c.max_seqs * L.delta.state_floats;
-        n->delta_conv += (size_t)c.max_seqs * L.delta.conv_floats;
+        n->mix_conv += (size_t)c.max_seqs * L.delta.conv_floats;
     }
     n->pool = (n->pool + 255) / 256 * 256;
     n->delta_state = (n->delta_state + 63) / 64 * 64;
+    n->mix_conv = (n->mix_conv + 63) / 64 * 64;
     if (m.lay->cfg.block == GPTRS_BLOCK_OUTPUT_NORM) {
         L.state1 = n->n_state++;
         if (L.cfg.mlp != GPTRS_MLP_NONE) L.state2 = n->n_state++;
     }
-    if (L.cfg.mlp == GPTRS_MLP_DENSE_XIELU) n->up = std::max(n->up, w.up.n);
+    if (L.cfg.mlp == GPTRS_MLP_DENSE_XIELU || L.cfg.mlp == GPTRS_MLP_DENSE_POLY) n->up = std::max(n->up, w.up.n);
     if (L.cfg.mlp == GPTRS_MLP_DENSE_GELU) {
         n->up = std::max(n->up, w.up.n / 2);
         n->gate_up = std::max(n->gate_up, w.up.n);
@@ -467,8 +583,8 @@ void count_widths(const Model& m, LayeredLayer& L, Widths* n) {
         n->router = std::max(n->router, w.router.n);
         n->sorted = std::max(n->sorted, top * w.up.k);
         const bool gated = L.cfg.expert_form == GPTRS_EXPERT_SWIGLU;
-        n->up = std::max({n->up, gated ? top * w.up.n / 2 : top * w.up.n, w.shared_up.n});
-        if (gated) n->gate_up = std::max(n->gate_up, top * w.up.n);
+        n->up = std::max({n->up, gated ? top * w.up.n / 2 : top * w.up.n, gated ? w.shared_up.n / 2 : w.shared_up.n});
+        if (gated) n->gate_up = std::max({n->gate_up, top * w.up.n, w.shared_up.n});
         n->expert_y = std::max(n->expert_y, top * w.down.n);
         n->work = std::max(n->work, gptrs_cuda_moe_work_ints(&L.moe, T));
         gptrs_moe smallest = L.moe;   // most tiles: the smallest tile that a launch of this many rows, or of one, may get
@@ -482,7 +598,8 @@ bool same_shape(const gptrs_layer_config& a, const gptrs_layer_config& b) {
         return std::make_tuple(std::make_tuple(c.mixer, c.heads, c.dim, c.rot_dim, c.rot_dims, c.vdim, c.kv_rank, c.window, c.scale, c.rope_base, c.mlp, c.d_ff),
                                std::make_tuple(c.kv_heads, c.mask, c.mask_size, c.distance_bias, c.proj_bias, c.softcap, c.taps, c.decay_rank, c.gate_rank),
                                std::make_tuple(c.experts, c.top, c.groups, c.keep, c.expert_form, c.shared_ff, c.route, c.group_best, c.correction, c.weight_scale),
-                               std::make_tuple(c.q_rank, c.maps, c.out_gate, c.kv_from, c.diff));
+                               std::make_tuple(c.q_rank, c.maps, c.out_gate, c.kv_from, c.diff, c.sink, c.rope_halves, c.qk_norm, c.tied, c.gate_silu, c.shared_gate),
+                               std::make_tuple(c.rope_factor, c.rope_original, c.rope_fast, c.rope_slow));
     };
     return key(a) == key(b);
 }
@@ -499,7 +616,8 @@ int layered_check_config(const gptrs_model_config& c) {
 
 int layered_set_layers(Model& m, const gptrs_layered_config& common, const gptrs_layer_config* layers) {
     const int n = m.cfg.n_layers;
-    GPTRS_REQUIRE(common.block == GPTRS_BLOCK_OUTPUT_NORM || common.block == GPTRS_BLOCK_SANDWICH || common.block == GPTRS_BLOCK_PRE_NORM, "unknown block form");
+    GPTRS_REQUIRE(common.block == GPTRS_BLOCK_OUTPUT_NORM || common.block == GPTRS_BLOCK_SANDWICH || common.block == GPTRS_BLOCK_PRE_NORM || common.block == GPTRS_BLOCK_DEPTH, "unknown block form");
+    GPTRS_REQUIRE(common.block != GPTRS_BLOCK_DEPTH || (common.norm_groups >= 1 && m.cfg.d_model % common.norm_groups == 0), "norm groups: equal parts of the width");
     GPTRS_REQUIRE(common.streams >= 0 && (common.streams == 0 || common.block == GPTRS_BLOCK_PRE_NORM), "residual streams: for the block form with norms in front");
     if (common.streams > GPTRS_MAX_STREAMS) return fail(GPTRS_UNIMPLEMENTED, "more than 16 residual streams");
     GPTRS_REQUIRE(common.block != GPTRS_BLOCK_OUTPUT_NORM || (common.conv_taps >= 1 && common.conv_taps <= 16), "short convolutions of 1 to 16 taps");
@@ -513,6 +631,8 @@ int layered_set_layers(Model& m, const gptrs_layered_config& common, const gptrs
         const gptrs_layer_config& c = layers[l];
         GPTRS_REQUIRE(c.mlp == GPTRS_MLP_NONE || c.d_ff > 0, "feed-forward size");
         GPTRS_REQUIRE(c.weights_of < n && (c.weights_of < 0 || layers[c.weights_of].weights_of < 0), "weights_of names a layer that has weights of its own");
+        GPTRS_REQUIRE(common.block != GPTRS_BLOCK_DEPTH || c.weights_of < 0, "a layer whose output is averaged over depth has weights of its own");
+        GPTRS_REQUIRE(!(c.rope_factor > 0.) || (c.rope_original > 0. && c.rope_fast > 0. && c.rope_slow > 0.), "rotation scaling: constants must be positive");
         LayeredLayer& L = m.lay->layers[l];
         L.cfg = c;
         int rc;
@@ -527,6 +647,7 @@ int layered_set_layers(Model& m, const gptrs_layered_config& common, const gptrs
             L.gatt.scale = c.scale; L.gatt.softcap = c.softcap; L.gatt.distance_bias = c.distance_bias;
             L.gatt.maps = c.maps; L.gatt.gate = c.out_gate; L.gatt.shared_kv = c.kv_from >= 0;
             L.gatt.head_scale = 1.f - c.diff; L.gatt.head_eps = m.cfg.norm_eps;
+            L.gatt.taps = c.taps; L.gatt.qk_norm = c.qk_norm; L.gatt.tied = c.tied;
             if (c.kv_from >= 0) {
                 GPTRS_REQUIRE(c.kv_from < l && !c.proj_bias, "kv_from names an earlier layer (projections without biases)");
                 const gptrs_layer_config& o = layers[c.kv_from];
@@ -537,22 +658,23 @@ int layered_set_layers(Model& m, const gptrs_layered_config& common, const gptrs
         } else if (c.mixer == GPTRS_MIXER_CHANNEL_DELTA) {
             L.delta.dtype = dtype;
             L.delta.heads = c.heads; L.delta.kv_heads = c.kv_heads; L.delta.dim = c.dim; L.delta.vdim = c.vdim; L.delta.taps = c.taps;
-            L.delta.decay_rank = c.decay_rank; L.delta.gate_rank = c.gate_rank; L.delta.eps = m.cfg.norm_eps;
+            L.delta.decay_rank = c.decay_rank; L.delta.gate_rank = c.gate_rank; L.delta.eps = m.cfg.norm_eps; L.delta.gate_silu = c.gate_silu;
             rc = gptrs_cuda_delta_layout(&L.delta);
         } else {
             return fail(GPTRS_UNIMPLEMENTED, "unknown mixer");
         }
         if (rc) return rc;
         if (c.mlp == GPTRS_MLP_EXPERTS) {
-            GPTRS_REQUIRE(common.block != GPTRS_BLOCK_OUTPUT_NORM, "experts: for the block forms with norms in front of the sublayers");
-            GPTRS_REQUIRE(c.shared_ff >= 0 && (c.shared_ff == 0 || (common.block == GPTRS_BLOCK_PRE_NORM && c.expert_form == GPTRS_EXPERT_RELU2)),
-                          "shared expert: of squared-relu form, for the block form with norms in front only");
+            GPTRS_REQUIRE(common.block != GPTRS_BLOCK_OUTPUT_NORM, "experts: for the block forms without short convolutions between the sublayers");
+            GPTRS_REQUIRE(c.shared_ff >= 0 && (c.shared_ff == 0 || common.block == GPTRS_BLOCK_PRE_NORM || common.block == GPTRS_BLOCK_DEPTH),
+                          "shared expert: for the block forms with norms on one side only");
+            GPTRS_REQUIRE(!c.shared_gate || (c.shared_ff > 0 && common.block == GPTRS_BLOCK_DEPTH), "gated shared expert: for the block form with an average over depth");
             GPTRS_REQUIRE(c.expert_form == GPTRS_EXPERT_SWIGLU || c.expert_form == GPTRS_EXPERT_RELU2, "unknown form of the experts");
             L.moe = {c.experts, c.top, c.groups, c.keep, 16, c.route, c.group_best, c.weight_scale};
             GPTRS_REQUIRE(c.experts > 0 && c.top > 0 && c.groups > 0 && c.keep > 0 && c.experts % c.groups == 0 && c.keep <= c.groups &&
                               c.top <= c.keep * (c.experts / c.groups), "experts: groups must be equal and hold enough experts");
             if (c.experts > 1024) return fail(GPTRS_UNIMPLEMENTED, "experts: more than 1024");
-        } else if (c.mlp != GPTRS_MLP_NONE && c.mlp != GPTRS_MLP_DENSE_XIELU && c.mlp != GPTRS_MLP_DENSE_GELU) {
+        } else if (c.mlp != GPTRS_MLP_NONE && c.mlp != GPTRS_MLP_DENSE_XIELU && c.mlp != GPTRS_MLP_DENSE_GELU && c.mlp != GPTRS_MLP_DENSE_POLY) {
             return fail(GPTRS_UNIMPLEMENTED, "unknown feed-forward kind");
         }
     }
@@ -598,7 +720,8 @@ int layered_finalize(Model& m, bool drop_leaves) {
         (rc = y.lat.alloc(T * n.lat * act, true)) || (rc = y.attn.alloc(T * n.attn * act, true)) || (rc = y.up.alloc(T * n.up * act, true)) ||
         (rc = m.xn_rows.alloc(rows * Wp * act, true)) || (rc = m.logits.alloc(rows * V * 4, true))) return rc;
     if ((rc = y.decay.alloc(T * n.decay * 4, true)) || (rc = y.gate.alloc(T * n.gate * act, true)) || (rc = y.delta_scratch.alloc(n.delta_scratch * 4, true)) ||
-        (rc = y.delta_state.alloc(n.delta_state * 4, true)) || (rc = y.delta_conv.alloc(n.delta_conv * 4, true))) return rc;
+        (rc = y.delta_state.alloc(n.delta_state * 4, true)) || (rc = y.mix_conv.alloc(n.mix_conv * 4, true))) return rc;
+    if (y.cfg.block == GPTRS_BLOCK_DEPTH && (rc = y.states.alloc((size_t)(c.n_layers + 1) * T * W * 4, true))) return rc;
     if ((rc = y.router.alloc(T * n.router * 4, true)) || (rc = y.sorted.alloc(T * n.sorted * act, true)) || (rc = y.gate_up.alloc(m.f32() ? T * n.gate_up * 4 : 0, true)) ||
         (rc = y.expert_y.alloc(T * n.expert_y * act, true)) || (rc = y.pair.alloc(T * n.top * 4, true)) || (rc = y.pair_weight.alloc(T * n.top * 4, true)) ||
         (rc = y.row_tiles.alloc(n.row_tiles * sizeof(gptrs_row_tile), true)) || (rc = y.n_row_tiles.alloc(4, true)) || (rc = y.moe_work.alloc(n.work * 4, true))) return rc;
@@ -769,7 +892,7 @@ struct Pass {
         const Layered::TileSet* t = L.tiles >= 0 ? y.tile_sets[L.tiles].get() : nullptr;
         const int splits = t ? gptrs_cuda_latent_splits(&a, t->n, max_ctx) : 1;
         m.launches += splits > 1 ? 2 : 1;
-        if ((rc = gptrs_cuda_latent_attention(&a, y.qa.p, pool(L), pages(), m.cfg.max_pages_per_seq, slot(), m.d_ctx.as<int32_t>(),
+        if ((rc = gptrs_cuda_latent_attention(&a, y.qa.p, pool(L), pages(), m.cfg.max_pages_per_seq, slot(), m.d_ctx.as<int32_t>(), fp(w.sink),
                                               t ? t->row.as<int32_t>() : nullptr, t ? t->rows.as<int32_t>() : nullptr, t ? t->n : 0, splits, y.lat.p, y.scratch.p,
                                               y.scratch.n, m.d_status.as<int32_t>(), T, st))) return rc;
         DenseOpts ov;
@@ -784,11 +907,23 @@ struct Pass {
         int rc;
         if ((rc = dense(m, w.qkv, y.h.p, y.qkv.p, T, {}))) return rc;
         if (!a.shared_kv) ++m.launches;
-        if (!a.shared_kv && (rc = gptrs_cuda_grouped_append(&a, y.qkv.p, pos(), slot(), pages(), m.cfg.max_pages_per_seq, pool(L), T, st))) return rc;
+        const void* q = y.qkv.p;
+        if (L.prepared()) {
+            gptrs_grouped_step s = {};
+            s.d_qkv = y.qkv.p; s.d_conv = fp(w.qk_conv); s.d_q_gain = fp(w.q_gain); s.d_k_gain = fp(w.k_gain);
+            s.d_conv_state = y.mix_conv.as<float>() + L.mix_conv_off;
+            s.d_slot = slot(); s.d_pos = pos();
+            s.d_run_first = y.d_run_first.as<int32_t>(); s.d_run_last = y.d_run_last.as<int32_t>(); s.d_parity = y.d_parity.as<int32_t>();
+            s.d_page_table = pages(); s.max_pages = m.cfg.max_pages_per_seq; s.d_pool = pool(L); s.d_q = y.q.p; s.rows = T;
+            if ((rc = gptrs_cuda_grouped_prepare(&a, &s, st))) return rc;
+            q = y.q.p;
+        } else if (!a.shared_kv && (rc = gptrs_cuda_grouped_append(&a, y.qkv.p, pos(), slot(), pages(), m.cfg.max_pages_per_seq, pool(L), T, st))) {
+            return rc;
+        }
         const Layered::TileSet* t = L.tiles >= 0 ? y.tile_sets[L.tiles].get() : nullptr;
         const int splits = t ? gptrs_cuda_grouped_splits(&a, t->n, max_ctx) : 1;
         m.launches += splits > 1 ? 2 : 1;
-        if ((rc = gptrs_cuda_grouped_attention(&a, y.qkv.p, pool(L), pages(), m.cfg.max_pages_per_seq, slot(), m.d_ctx.as<int32_t>(), fp(w.r1), fp(w.r2),
+        if ((rc = gptrs_cuda_grouped_attention(&a, q, pool(L), pages(), m.cfg.max_pages_per_seq, slot(), m.d_ctx.as<int32_t>(), fp(w.r1), fp(w.r2), w.reach.as<int32_t>(),
                                                t ? t->row.as<int32_t>() : nullptr, t ? t->rows.as<int32_t>() : nullptr, t ? t->n : 0, splits, y.attn.p, y.scratch.p,
                                                y.scratch.n, m.d_status.as<int32_t>(), T, st))) return rc;
         return dense(m, w.out, y.attn.p, y.y.p, T, {});
@@ -803,15 +938,15 @@ struct Pass {
         auto column = [&](int off) { return y.qkv.as<unsigned char>() + off * act; };
         DenseOpts od;
         od.out_f32 = true; od.ldx = w.qkv.n; od.ldy = a.decay_row;
-        if ((rc = dense(m, w.decay, column(a.a_offset), y.decay.p, T, od))) return rc;
+        if (a.decay_rank > 0 && (rc = dense(m, w.decay, column(a.a_offset), y.decay.p, T, od))) return rc;
         DenseOpts og;
         og.ldx = w.qkv.n; og.ldy = a.gate_row;
-        if ((rc = dense(m, w.gate, column(a.g_offset), y.gate.p, T, og))) return rc;
+        if (a.gate_rank > 0 && (rc = dense(m, w.gate, column(a.g_offset), y.gate.p, T, og))) return rc;
         gptrs_delta_step s = {};
         s.d_proj = y.qkv.p; s.d_decay = y.decay.as<float>(); s.d_gate = y.gate.p;
         s.d_conv = fp(w.delta_conv); s.d_a_log = fp(w.a_log); s.d_dt_bias = fp(w.dt_bias); s.d_norm = fp(w.delta_norm);
         s.d_state = y.delta_state.as<float>() + L.delta_state_off;
-        s.d_conv_state = y.delta_conv.as<float>() + L.delta_conv_off;
+        s.d_conv_state = y.mix_conv.as<float>() + L.mix_conv_off;
         s.d_slot = slot(); s.d_pos = pos();
         s.d_run_first = y.d_run_first.as<int32_t>(); s.d_run_last = y.d_run_last.as<int32_t>(); s.d_parity = y.d_parity.as<int32_t>();
         s.d_runs = y.d_runs.as<int32_t>(); s.n_runs = y.n_runs;
@@ -830,7 +965,8 @@ struct Pass {
         if (L.cfg.shared_ff > 0) {   // its output is a second one for the step behind
             DenseOpts os;
             os.act = 2;
-            if ((rc = dense(m, w.shared_up, y.h.p, y.up.p, T, os)) || (rc = dense(m, w.shared_down, y.up.p, y.y.p, T, {}))) return rc;
+            rc = L.cfg.expert_form == GPTRS_EXPERT_SWIGLU ? gated(w.shared_up, y.h.p, T, GPTRS_GATE_SILU, {}) : dense(m, w.shared_up, y.h.p, y.up.p, T, os);
+            if (rc || (rc = dense(m, w.shared_down, y.up.p, y.y.p, T, {}))) return rc;
         }
         DenseOpts orr;
         orr.out_f32 = true;
@@ -872,6 +1008,13 @@ struct Pass {
         if (L.cfg.mlp == GPTRS_MLP_DENSE_GELU) {
             const int rg = gated(L.w->up, y.h.p, T, GPTRS_GATE_GELU_TANH, {});
             return rg ? rg : dense(m, L.w->down, y.up.p, y.y.p, T, {});
+        }
+        if (L.cfg.mlp == GPTRS_MLP_DENSE_POLY) {
+            const LayerWeights& w = *L.w;
+            int rp = dense(m, w.up, y.h.p, y.up.p, T, {});
+            ++m.launches;
+            if (!rp) rp = gptrs_cuda_poly_norm(y.up.p, fp(w.act), m.cfg.norm_eps, y.up.p, act_dt, T, L.cfg.d_ff, w.up.n, st);
+            return rp ? rp : dense(m, w.down, y.up.p, y.y.p, T, {});
         }
         DenseOpts ou;
         ou.act = 1; ou.pos = L.w->act_pos; ou.neg = L.w->act_neg;
@@ -1071,6 +1214,68 @@ int forward_pre_norm(Pass& f, Capture& cap, int n_rows, bool rows_identity) {
     return GPTRS_OK;
 }
 
+// norms on the outputs in groups, a weighted average of all results so far behind every layer
+int forward_depth(Pass& f, Capture& cap, int n_rows, bool rows_identity) {
+    Model& m = f.m;
+    Layered& y = f.y;
+    const auto& c = m.cfg;
+    float *x = y.states.as<float>(), *running = m.hidden.as<float>();   // the first layer reads the embedding
+    gptrs_depth_step base = {};
+    base.y_dtype = f.act_dt; base.mult = y.cfg.residual_mult; base.groups = y.cfg.norm_groups; base.eps = c.norm_eps;
+    base.d_states = y.states.as<float>(); base.state_stride = (int64_t)c.max_tokens * c.d_model;
+    base.d_h = y.h.p; base.h_dtype = f.act_dt; base.ldh = f.ldw;
+    base.d_status = m.d_status.as<int32_t>();
+    base.rows = f.T; base.dim = c.d_model;
+    auto launch = [&](const gptrs_depth_step& s) { ++m.launches; return gptrs_cuda_depth_step(&s, f.st); };
+    // the output of the sublayer that has just run
+    auto closing = [&](const LayeredLayer& L, int sub) {
+        gptrs_depth_step s = base;
+        s.d_x = x; s.d_x_out = running;
+        s.d_gamma_out = f.fp(sub ? L.w->norm2 : L.w->norm1);
+        if (sub && L.cfg.mlp == GPTRS_MLP_EXPERTS) {
+            s.d_y = y.expert_y.p; s.ldy = L.w->down.n;
+            s.d_pair = y.pair.as<int32_t>(); s.d_pair_weight = y.pair_weight.as<float>(); s.top = L.moe.top;
+            if (L.cfg.shared_ff > 0) { s.d_add = y.y.p; s.ld_add = f.ldw; }
+            if (L.cfg.shared_gate) { s.d_add_gate = y.router.as<float>() + L.moe.experts; s.ld_add_gate = L.w->router.n; }
+        } else {
+            s.d_y = y.y.p; s.ldy = f.ldw;
+        }
+        return s;
+    };
+    gptrs_depth_step open = base;
+    open.d_embed = f.fp(m.tok_emb); open.d_tokens = m.d_tokens.as<int32_t>(); open.vocab = c.vocab;
+    open.d_x_out = x;
+    int rc = launch(open);
+    if (rc) return rc;
+    for (int l = 0; l < c.n_layers; ++l) {
+        LayeredLayer& L = y.layers[l];
+        const bool last = l + 1 == c.n_layers, ff = L.cfg.mlp != GPTRS_MLP_NONE;
+        if ((rc = f.mixer(L))) return rc;
+        if (ff) {
+            if ((rc = launch(closing(L, 0)))) return rc;
+            x = running;
+            if ((rc = f.feed_forward(L))) return rc;
+        }
+        gptrs_depth_step s = closing(L, ff ? 1 : 0);
+        s.d_weights = f.fp(L.w->dwa); s.n_states = l + 1;
+        if (!last || cap.buf.p) {
+            if (last) s.d_h = nullptr;
+            if ((rc = launch(s)) || (rc = cap.take(m, l, running, f.T))) return rc;
+            x = running;
+        }
+        if (last) {
+            if (cap.buf.p) { s.d_x = running; s.d_y = s.d_add = nullptr; s.d_pair = nullptr; s.d_weights = nullptr; }   // the stream already holds it
+            s.d_gamma_in = f.fp(m.final_g);
+            s.d_rows = rows_identity ? nullptr : m.d_rows.as<int32_t>();
+            if (rows_identity) s.d_x_out = nullptr;
+            s.d_h = m.xn_rows.p;
+            s.rows = n_rows;
+            if ((rc = launch(s))) return rc;
+        }
+    }
+    return GPTRS_OK;
+}
+
 }  // namespace
 
 int layered_forward(Model& m, int T, int max_ctx, int n_rows, bool rows_identity, float temperature, bool skip_logits) {
@@ -1081,7 +1286,8 @@ int layered_forward(Model& m, int T, int max_ctx, int n_rows, bool rows_identity
     Capture cap;
     int rc = cap.begin(m, T);
     if (!rc) {
-        const auto forward = y.cfg.block == GPTRS_BLOCK_SANDWICH ? forward_sandwich : y.cfg.block == GPTRS_BLOCK_PRE_NORM ? forward_pre_norm : forward_output_norm;
+        const auto forward = y.cfg.block == GPTRS_BLOCK_SANDWICH ? forward_sandwich : y.cfg.block == GPTRS_BLOCK_PRE_NORM ? forward_pre_norm
+                           : y.cfg.block == GPTRS_BLOCK_DEPTH ? forward_depth : forward_output_norm;
         rc = forward(f, cap, n_rows, rows_identity);
     }
     if (!rc) rc = cap.end(m);

@@ -21,11 +21,12 @@ from . import check, lib
 KIND_GPT, KIND_MINISTRAL, KIND_LAYERED = 0, 1, 2
 MODE_F32, MODE_W4A16, MODE_W8A16, MODE_BF16 = 0, 1, 2, 3
 MIXER_LATENT_ATTENTION, MIXER_GROUPED_ATTENTION, MIXER_CHANNEL_DELTA = 0, 1, 2
-MLP_NONE, MLP_DENSE_XIELU, MLP_EXPERTS, MLP_DENSE_GELU = 0, 1, 2, 3
+MLP_NONE, MLP_DENSE_XIELU, MLP_EXPERTS, MLP_DENSE_GELU, MLP_DENSE_POLY = 0, 1, 2, 3, 4
 EXPERT_SWIGLU, EXPERT_RELU2 = 0, 1
 ROUTE_SOFTMAX, ROUTE_SIGMOID = 0, 1
-BLOCK_OUTPUT_NORM, BLOCK_SANDWICH, BLOCK_PRE_NORM = 0, 1, 2
+BLOCK_OUTPUT_NORM, BLOCK_SANDWICH, BLOCK_PRE_NORM, BLOCK_DEPTH = 0, 1, 2, 3
 MASK_CAUSAL, MASK_WINDOW, MASK_CHUNK = 0, 1, 2
+DISTANCE_NONE, DISTANCE_LOG, DISTANCE_LINEAR = 0, 1, 2
 
 
 class _ModelConfig(ctypes.Structure):
@@ -52,19 +53,23 @@ class _LayerConfig(ctypes.Structure):
         ("q_rank", ctypes.c_int), ("maps", ctypes.c_int), ("out_gate", ctypes.c_int), ("kv_from", ctypes.c_int), ("diff", ctypes.c_float),
         ("expert_form", ctypes.c_int), ("shared_ff", ctypes.c_int), ("route", ctypes.c_int), ("group_best", ctypes.c_int), ("correction", ctypes.c_int),
         ("weight_scale", ctypes.c_float),
+        ("sink", ctypes.c_int), ("rope_halves", ctypes.c_int), ("rope_factor", ctypes.c_double), ("rope_original", ctypes.c_double),
+        ("rope_fast", ctypes.c_double), ("rope_slow", ctypes.c_double), ("qk_norm", ctypes.c_int), ("tied", ctypes.c_int), ("gate_silu", ctypes.c_int),
+        ("shared_gate", ctypes.c_int),
     ]
 
 
 class _LayeredConfig(ctypes.Structure):
     _fields_ = [("conv_taps", ctypes.c_int), ("logit_softcap", ctypes.c_float), ("block", ctypes.c_int), ("learned_positions", ctypes.c_int),
-                ("streams", ctypes.c_int), ("embed_scale", ctypes.c_float)]
+                ("streams", ctypes.c_int), ("embed_scale", ctypes.c_float), ("residual_mult", ctypes.c_float), ("norm_groups", ctypes.c_int)]
 
 
 @dataclass
 class LayerConfig:
     """One layer of a model of the layered kind: its mixer and its feed-forward. Latent attention (in a sliding window, or over
-    everything) takes heads .. rot_dims and q_rank; attention with grouped key / value heads takes heads, dim, vdim, scale, kv_heads ..
-    softcap and maps .. diff; the delta rule takes heads, dim, vdim, kv_heads and taps .. gate_rank. Experts have the size d_ff each."""
+    everything) takes heads .. rot_dims, q_rank and sink .. rope_slow; attention with grouped key / value heads takes heads, dim, vdim, scale,
+    kv_heads .. taps, maps .. diff, qk_norm and tied; the delta rule takes heads, dim, vdim, kv_heads, taps .. gate_rank and gate_silu.
+    Experts have the size d_ff each."""
     heads: int
     dim: int            # query / key dimensions of a head (latent attention: those that are not rotated)
     rot_dim: int = 0    # and those that are (shared key part)
@@ -80,12 +85,12 @@ class LayerConfig:
     kv_heads: int = 0
     mask: int = MASK_CAUSAL
     mask_size: int = 0
-    distance_bias: int = 0   # a penalty r1 ln(1 + r2 distance) per head
+    distance_bias: int = DISTANCE_NONE   # a penalty per head: r1 ln(1 + r2 distance), or 2^(-8 (h + 1) / heads) distance
     proj_bias: int = 0       # biases on the four projections
     softcap: float = 0.0     # of the scores
-    taps: int = 0
-    decay_rank: int = 0
-    gate_rank: int = 0
+    taps: int = 0            # of the short convolutions (grouped attention: 0 = none)
+    decay_rank: int = 0      # 0: one decay per head
+    gate_rank: int = 0       # 0: a gate projected at once
     experts: int = 0
     top: int = 0
     groups: int = 1
@@ -102,6 +107,16 @@ class LayerConfig:
     group_best: int = 1      # experts that make a group's score
     correction: int = 0      # a vector added to the scores that choose
     weight_scale: float = 0.0   # > 0: the experts' weights are in proportion and sum to this
+    sink: int = 0            # exp(sink) per head in the denominator of the softmax
+    rope_halves: int = 0     # rotated pairs are (i, i + rot_dims / 2) instead of (2i, 2i + 1)
+    rope_factor: float = 0.0    # YaRN scaling of the rotation (0 = none)
+    rope_original: float = 0.0
+    rope_fast: float = 0.0
+    rope_slow: float = 0.0
+    qk_norm: int = 0         # norms per head on queries and keys
+    tied: int = 0            # values are the keys in front of their norm
+    gate_silu: int = 0       # the delta rule's gate: silu instead of sigmoid
+    shared_gate: int = 0     # the shared expert's output times sigmoid(shared.sg h)
 
     def _struct(self):
         values = {f: getattr(self, f) for f, _ in _LayerConfig._fields_}
@@ -119,7 +134,7 @@ class LayerConfig:
                 out[f"{p}.norm{n}b"] = (d,)
             elif block == BLOCK_OUTPUT_NORM:
                 out[f"{p}.canon{n}"] = (d, conv_taps)
-            elif streams:
+            elif block == BLOCK_PRE_NORM and streams:
                 out.update({f"{p}.hc{n}.in": (streams,), f"{p}.hc{n}.out": (streams,), f"{p}.hc{n}.mix": (streams, streams)})
             return out
 
@@ -130,15 +145,24 @@ class LayerConfig:
             out.update({f"{x}.dq": (self.q_rank, d), f"{x}.dq.norm": (self.q_rank,), f"{x}.uq": (rows, self.q_rank)} if self.q_rank else {f"{x}.q": (rows, d)})
             out.update({f"{x}.dkv": (self.kv_rank + self.rot_dim, d), f"{x}.dkv.norm": (self.kv_rank,),
                         f"{x}.uk": (qk, self.kv_rank), f"{x}.uv": (v, self.kv_rank), f"{x}.o": (d, v)})
+            if self.sink:
+                out[f"{x}.sink"] = (self.heads,)
         elif self.mixer == MIXER_GROUPED_ATTENTION:
             rows = {"q": qk * self.maps}
             if self.kv_from < 0:
-                rows.update(k=self.kv_heads * self.dim * self.maps, v=self.kv_heads * self.vdim)
+                rows["k"] = self.kv_heads * self.dim * self.maps
+                if not self.tied:
+                    rows["v"] = self.kv_heads * self.vdim
             out.update({f"{x}.{n}": (r, d) for n, r in rows.items()})
+            for n in "qk":
+                if self.taps:
+                    out[f"{x}.{n}.conv"] = (rows[n], self.taps)
+                if self.qk_norm:
+                    out[f"{x}.{n}.norm"] = (self.dim,)
             out[f"{x}.o"] = (d, v)
             if self.proj_bias:
                 out.update({f"{x}.{n}.b": (r,) for n, r in {**rows, "o": d}.items()})
-            if self.distance_bias:
+            if self.distance_bias == DISTANCE_LOG:
                 out.update({f"{x}.r1": (self.heads,), f"{x}.r2": (self.heads,)})
             if self.out_gate:
                 out[f"{x}.g"] = (v, d)
@@ -148,8 +172,10 @@ class LayerConfig:
             kq = self.kv_heads * self.dim
             for n, r in (("q", kq), ("k", kq), ("v", v)):
                 out.update({f"{x}.{n}": (r, d), f"{x}.{n}.conv": (r, self.taps)})
-            out.update({f"{x}.b": (self.heads, d), f"{x}.A_log": (self.heads,), f"{x}.a1": (self.decay_rank, d), f"{x}.a2": (qk, self.decay_rank),
-                        f"{x}.dt_bias": (qk,), f"{x}.g1": (self.gate_rank, d), f"{x}.g2": (v, self.gate_rank), f"{x}.norm": (self.vdim,), f"{x}.o": (d, v)})
+            out.update({f"{x}.b": (self.heads, d), f"{x}.A_log": (self.heads,), f"{x}.norm": (self.vdim,), f"{x}.o": (d, v)})
+            out.update({f"{x}.a1": (self.decay_rank, d), f"{x}.a2": (qk, self.decay_rank), f"{x}.dt_bias": (qk,)} if self.decay_rank else
+                       {f"{x}.a": (self.heads, d), f"{x}.dt_bias": (self.heads,)})
+            out.update({f"{x}.g1": (self.gate_rank, d), f"{x}.g2": (v, self.gate_rank)} if self.gate_rank else {f"{x}.g": (v, d)})
         if self.mlp == MLP_NONE:
             return out
         f = f"{p}.mlp"
@@ -158,6 +184,8 @@ class LayerConfig:
             out.update({f"{f}.up": (self.d_ff, d), f"{f}.up.b": (self.d_ff,), f"{f}.down": (d, self.d_ff), f"{f}.down.b": (d,), f"{f}.act": (2,)})
         elif self.mlp == MLP_DENSE_GELU:
             out.update({f"{f}.gate": (self.d_ff, d), f"{f}.up": (self.d_ff, d), f"{f}.down": (d, self.d_ff)})
+        elif self.mlp == MLP_DENSE_POLY:
+            out.update({f"{f}.up": (self.d_ff, d), f"{f}.down": (d, self.d_ff), f"{f}.act": (4,)})
         else:
             for e in range(self.experts):
                 if self.expert_form == EXPERT_SWIGLU:
@@ -166,6 +194,10 @@ class LayerConfig:
             out[f"{f}.router"] = (self.experts, d)
             if self.correction:
                 out[f"{f}.correction"] = (self.experts,)
+            if self.shared_ff and self.expert_form == EXPERT_SWIGLU:
+                out[f"{f}.shared.gate"] = (self.shared_ff, d)
+            if self.shared_gate:
+                out[f"{f}.shared.sg"] = (1, d)
             if self.shared_ff:
                 out.update({f"{f}.shared.up": (self.shared_ff, d), f"{f}.shared.down": (d, self.shared_ff)})
         return out
@@ -201,6 +233,8 @@ class ModelConfig:
     learned_positions: int = 0     # position vectors added to the embedding
     streams: int = 0               # copies of the residual that are mixed at every sublayer (BLOCK_PRE_NORM)
     embed_scale: float = 1.0       # of the embedding (BLOCK_PRE_NORM)
+    residual_mult: float = 1.0     # of the sublayers' normed outputs (BLOCK_DEPTH)
+    norm_groups: int = 1           # equal parts of a row, each with a norm of its own (BLOCK_DEPTH)
 
     @staticmethod
     def layered(layers, d_model: int, vocab: int, context_length: int, norm_eps: float, conv_taps: int = 1, logit_softcap: float = 0.0, **kw):
@@ -269,6 +303,8 @@ class ModelConfig:
             out["pos"] = (self.learned_positions, d)
         for l, c in enumerate(self.layers):
             out.update(c.shapes(f"l{l}", d, self.block, self.conv_taps, self.streams))
+            if self.block == BLOCK_DEPTH:
+                out[f"l{l}.dwa"] = (l + 2,)
         out["final.norm"] = (d,)
         out["head"] = (self.vocab, d)
         return out
@@ -301,7 +337,8 @@ class LoadedModel:
         check(lib().gptrs_cuda_model_create(ctypes.byref(c), ctypes.byref(self._h)))
         if config.kind == KIND_LAYERED:
             rows = (_LayerConfig * len(config.layers))(*[l._struct() for l in config.layers])
-            common = _LayeredConfig(config.conv_taps, config.logit_softcap, config.block, config.learned_positions, config.streams, config.embed_scale)
+            common = _LayeredConfig(config.conv_taps, config.logit_softcap, config.block, config.learned_positions, config.streams, config.embed_scale,
+                                    config.residual_mult, config.norm_groups)
             check(lib().gptrs_cuda_model_set_layers(self._h, ctypes.byref(common), rows, len(config.layers)))
         self._finalized = False
 

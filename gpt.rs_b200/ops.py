@@ -475,7 +475,7 @@ def latent_rotate_queries(a, q, positions, cos, sin, qa):
     check(lib().gptrs_cuda_latent_rotate_queries(ctypes.byref(a), _ptr(q), _ptr(positions), _ptr(cos), _ptr(sin), _ptr(qa), q.shape[0], _stream()))
 
 
-def latent_attention(a, qa, pool, page_table, slot, ctx_len, max_ctx_len, tiles=None, splits=None, status=None):
+def latent_attention(a, qa, pool, page_table, slot, ctx_len, max_ctx_len, tiles=None, splits=None, status=None, sink=None):
     """out [T][heads][lat_head_stride]; `tiles` = (first rows, row counts) for the tensor-core kernel, None for the plain one."""
     status = _status(qa.device, status)
     n = slot.shape[0]
@@ -485,7 +485,7 @@ def latent_attention(a, qa, pool, page_table, slot, ctx_len, max_ctx_len, tiles=
         splits = lib().gptrs_cuda_latent_splits(ctypes.byref(a), n_tiles, max_ctx_len) if n_tiles else 1
     nbytes = lib().gptrs_cuda_latent_scratch_bytes(ctypes.byref(a), n_tiles, splits)
     scratch = torch.empty(max(nbytes, 1), dtype=torch.uint8, device=qa.device)
-    check(lib().gptrs_cuda_latent_attention(ctypes.byref(a), _ptr(qa), _ptr(pool), _ptr(page_table), page_table.shape[1], _ptr(slot), _ptr(ctx_len),
+    check(lib().gptrs_cuda_latent_attention(ctypes.byref(a), _ptr(qa), _ptr(pool), _ptr(page_table), page_table.shape[1], _ptr(slot), _ptr(ctx_len), _ptr(sink),
                                             None if tiles is None else _ptr(tiles[0]), None if tiles is None else _ptr(tiles[1]), n_tiles, splits, _ptr(out),
                                             _ptr(scratch), nbytes, _ptr(status), n, _stream()))
     return out, status
@@ -549,10 +549,46 @@ def stream_step(x, eps, y=None, mix=None, w_out=None, w_in=None, gamma_in=None, 
     return h, total
 
 
+def depth_step(groups, eps, mult=1.0, x=None, x_out=None, y=None, gamma_out=None, pair=None, pair_weight=None, add=None, add_gate=None, embed=None, tokens=None,
+               states=None, weights=None, gamma_in=None, rows=None, want_h=True, out_dtype=torch.float32, ldh=None, status=None):
+    """r = x + mult N(y) gamma_out (or embedding rows); with `weights` [n + 1] r becomes state n of `states` [n + 1][rows][dim] and x' = their weighted sum,
+    otherwise x' = r. x' goes to `x_out`; returns h = x' or N(x') gamma_in. `add_gate` [rows][k]: its first column gates `add`."""
+    s = _abi.DepthStep()
+    dev = (x if x is not None else embed).device
+    n, dim = (tokens.shape[0], embed.shape[1]) if embed is not None else x.shape
+    s.d_x, s.d_x_out, s.dim, s.groups, s.eps, s.mult, s.d_status = _ptr(x), _ptr(x_out), dim, groups, eps, mult, _ptr(_status(dev, status))
+    s.rows = n if rows is None else rows.shape[0]
+    s.d_rows = _ptr(rows)
+    if y is not None:
+        s.d_y, s.y_dtype, s.ldy, s.d_gamma_out = _ptr(y), _dt(y), y.shape[1], _ptr(gamma_out)
+    if pair is not None:
+        s.d_pair, s.d_pair_weight, s.top = _ptr(pair), _ptr(pair_weight), pair.shape[1]
+    if add is not None:
+        s.d_add, s.ld_add = _ptr(add), add.shape[1]
+    if add_gate is not None:
+        s.d_add_gate, s.ld_add_gate = _ptr(add_gate), add_gate.shape[1]
+    if embed is not None:
+        s.d_embed, s.d_tokens, s.vocab = _ptr(embed), _ptr(tokens), embed.shape[0]
+    if weights is not None:
+        s.d_states, s.state_stride, s.n_states, s.d_weights = _ptr(states), states.stride(0), weights.shape[0] - 1, _ptr(weights)
+    h = None
+    if want_h:
+        h = torch.empty((s.rows, ldh or dim), dtype=out_dtype, device=dev)
+        s.d_gamma_in, s.d_h, s.h_dtype, s.ldh = _ptr(gamma_in), _ptr(h), _dt(h), h.shape[1]
+    check(lib().gptrs_cuda_depth_step(ctypes.byref(s), _stream()))
+    return h
+
+
+def poly_norm(z, act, eps, n, out=None):
+    out = torch.empty_like(z) if out is None else out
+    check(lib().gptrs_cuda_poly_norm(_ptr(z), _ptr(act), eps, _ptr(out), _dt(z), z.shape[0], n, z.shape[1], _stream()))
+    return out
+
+
 def grouped_layout(heads, kv_heads, dim, vdim, mask, mask_size, scale, softcap=0.0, distance_bias=False, bf16=True, maps=1, gate=False, shared_kv=False,
-                   lam=0.0, head_scale=1.0, head_eps=1e-5):
+                   lam=0.0, head_scale=1.0, head_eps=1e-5, taps=0, qk_norm=False, tied=False):
     a = _abi.GroupedAttention(BF16 if bf16 else F32, heads, kv_heads, dim, vdim, mask, mask_size, scale, softcap, int(distance_bias), maps, int(gate),
-                              int(shared_kv), lam, head_scale, head_eps)
+                              int(shared_kv), lam, head_scale, head_eps, taps, int(qk_norm), int(tied))
     check(lib().gptrs_cuda_grouped_layout(ctypes.byref(a)))
     return a
 
@@ -562,11 +598,23 @@ def grouped_append(a, qkv, positions, slot, page_table, pool):
                                           qkv.shape[0], _stream()))
 
 
+def grouped_prepare(a, qkv, conv, q_gain, k_gain, conv_state, runs, page_table, pool):
+    """Convolutions, norms, page write; returns the queries. `runs` = (slot, pos, run_first, run_last, parity) per row."""
+    n = qkv.shape[0]
+    out = torch.empty((n, a.query_row), dtype=qkv.dtype, device=qkv.device)
+    s = _abi.GroupedStep()
+    s.d_qkv, s.d_conv, s.d_q_gain, s.d_k_gain, s.d_conv_state, s.d_page_table, s.d_pool, s.d_q = (_ptr(t) for t in (qkv, conv, q_gain, k_gain, conv_state, page_table, pool, out))
+    s.d_slot, s.d_pos, s.d_run_first, s.d_run_last, s.d_parity = (_ptr(t) for t in runs)
+    s.max_pages, s.rows = page_table.shape[1], n
+    check(lib().gptrs_cuda_grouped_prepare(ctypes.byref(a), ctypes.byref(s), _stream()))
+    return out
+
+
 def grouped_tile_tokens(a) -> int:
     return lib().gptrs_cuda_grouped_tile_tokens(ctypes.byref(a))
 
 
-def grouped_attention(a, qkv, pool, page_table, slot, ctx_len, max_ctx_len, r1=None, r2=None, tiles=None, splits=None, status=None):
+def grouped_attention(a, qkv, pool, page_table, slot, ctx_len, max_ctx_len, r1=None, r2=None, tiles=None, splits=None, status=None, reach=None):
     """out [T][heads][out_head_stride]; `tiles` = (first rows, row counts) for the tensor-core kernel, None for the plain one."""
     status = _status(qkv.device, status)
     n = slot.shape[0]
@@ -577,13 +625,13 @@ def grouped_attention(a, qkv, pool, page_table, slot, ctx_len, max_ctx_len, r1=N
     nbytes = lib().gptrs_cuda_grouped_scratch_bytes(ctypes.byref(a), n_tiles, splits)
     scratch = torch.empty(max(nbytes, 1), dtype=torch.uint8, device=qkv.device)
     check(lib().gptrs_cuda_grouped_attention(ctypes.byref(a), _ptr(qkv), _ptr(pool), _ptr(page_table), page_table.shape[1], _ptr(slot), _ptr(ctx_len), _ptr(r1),
-                                             _ptr(r2), None if tiles is None else _ptr(tiles[0]), None if tiles is None else _ptr(tiles[1]), n_tiles, splits,
+                                             _ptr(r2), _ptr(reach), None if tiles is None else _ptr(tiles[0]), None if tiles is None else _ptr(tiles[1]), n_tiles, splits,
                                              _ptr(out), _ptr(scratch), nbytes, _ptr(status), n, _stream()))
     return out, status
 
 
-def delta_layout(heads, kv_heads, dim, vdim, taps, decay_rank, gate_rank, eps, bf16=True):
-    a = _abi.DeltaRule(BF16 if bf16 else F32, heads, kv_heads, dim, vdim, taps, decay_rank, gate_rank, eps)
+def delta_layout(heads, kv_heads, dim, vdim, taps, decay_rank, gate_rank, eps, bf16=True, gate_silu=False):
+    a = _abi.DeltaRule(BF16 if bf16 else F32, heads, kv_heads, dim, vdim, taps, decay_rank, gate_rank, eps, int(gate_silu))
     check(lib().gptrs_cuda_delta_layout(ctypes.byref(a)))
     return a
 

@@ -272,13 +272,14 @@ int gptrs_cuda_post_norm_final(const float* d_x, const void* d_y, int y_dtype, i
  * of rot_dim values per token, shared by all heads; the per-head key and value projections are absorbed into the query
  * (W_uk^T q, a batched gptrs_cuda_dense_* in front) and the output (W_uv o, one behind). Sliding window: position i sees
  * i - window + 1 .. i (window 0: all of 0 .. i). Queries may come through a normed latent of their own (q_rank > 0): the first
- * projection then gives [query latent | latent | rotated key], a second one the queries. Pages of 16 tokens, addressed through
- * page_table[slot][page index] like the KV pool below.
+ * projection then gives [query latent | latent | rotated key], a second one the queries. A sink per head may add exp(sink) to the
+ * denominator of the softmax. Pages of 16 tokens, addressed through page_table[slot][page index] like the KV pool below.
  * ============================================================================================ */
 typedef struct {
     int dtype;                 /* GPTRS_F32 or GPTRS_BF16: activations and cache */
     int heads, dim, rot_dim, vdim, kv_rank, window;
-    int rot_dims;              /* rotated dimensions of the rot_dim part: pairs (2i, 2i + 1) */
+    int rot_dims;              /* rotated dimensions of the rot_dim part: pairs (2i, 2i + 1). Scores do not depend on the order of columns, so a
+                                * design that pairs i with i + rot_dims / 2 packs the rows of its projections in this order */
     float scale;
     int q_rank;                /* 0 = queries are projected directly */
     /* filled in by gptrs_cuda_latent_layout (elements): */
@@ -308,10 +309,10 @@ int gptrs_cuda_latent_rotate_queries(const gptrs_latent_attention* a, const void
 int gptrs_cuda_latent_tile_tokens(const gptrs_latent_attention* a);
 int gptrs_cuda_latent_splits(const gptrs_latent_attention* a, int64_t n_tiles, int64_t max_ctx_len);
 size_t gptrs_cuda_latent_scratch_bytes(const gptrs_latent_attention* a, int64_t n_tiles, int splits);
-/* out[T][heads][lat_head_stride] = softmax over the visible cache rows . latents. n_tiles = 0: the plain kernel; else tile i
- * is the rows tile_row[i] .. + tile_rows[i] (at most gptrs_cuda_latent_tile_tokens, consecutive positions of one sequence). */
+/* out[T][heads][lat_head_stride] = softmax over the visible cache rows . latents; d_sink [heads] or NULL. n_tiles = 0: the plain kernel; else
+ * tile i is the rows tile_row[i] .. + tile_rows[i] (at most gptrs_cuda_latent_tile_tokens, consecutive positions of one sequence). */
 int gptrs_cuda_latent_attention(const gptrs_latent_attention* a, const void* d_qa, const void* d_pool, const int32_t* d_page_table,
-                                int64_t max_pages, const int32_t* d_slot, const int32_t* d_ctx_len, const int32_t* d_tile_row,
+                                int64_t max_pages, const int32_t* d_slot, const int32_t* d_ctx_len, const float* d_sink, const int32_t* d_tile_row,
                                 const int32_t* d_tile_rows, int64_t n_tiles, int splits, void* d_out, void* d_scratch,
                                 size_t scratch_bytes, int32_t* d_status, int64_t n_tokens, void* stream);
 
@@ -389,44 +390,119 @@ typedef struct {
 int gptrs_cuda_stream_step(const gptrs_stream_step* step, void* stream);
 
 /* ==============================================================================================
+ * Step between two sublayers of a model with norms on the sublayers' outputs only and a weighted average over depth (no counterpart in
+ * gpt.rs). For every row, with N dividing each of `groups` equal consecutive parts of a row by its own sqrt(mean(part^2) + eps),
+ *     r = x + mult N(y) gamma_out
+ *     x' = sum_{j < n_states} weights[j] state_j + weights[n_states] r        state_(n_states) = r      (d_weights NULL: x' = r)
+ *     h = x'                                                                                           (d_gamma_in: h = N(x') gamma_in)
+ * d_embed set: r = embed[token] instead. d_y NULL: r = x. d_pair as in gptrs_norm_step; d_add: a second output added to y, times
+ * sigmoid(add_gate[row]) where that is given (a shared expert). d_rows set: row i of the launch is row d_rows[i] of everything that is
+ * read, h is compact, and neither x' nor r is written (the end of the model).
+ * ============================================================================================ */
+typedef struct {
+    const float* d_x;
+    float* d_x_out;            /* NULL: x' is not kept; may be d_x */
+    const void* d_y;
+    int y_dtype;               /* of d_add too */
+    int64_t ldy;
+    const int32_t* d_pair;     /* [rows][top] */
+    const float* d_pair_weight;
+    int64_t top;
+    const void* d_add;         /* optional [rows][ld_add] */
+    int64_t ld_add;
+    const float* d_add_gate;   /* optional, one number every ld_add_gate */
+    int64_t ld_add_gate;
+    const float* d_embed;
+    const int32_t* d_tokens;
+    int64_t vocab;
+    const float* d_gamma_out;
+    float mult;
+    int groups;
+    float eps;
+    float* d_states;           /* state j of a row at d_states + j state_stride + row dim */
+    int64_t state_stride;
+    int64_t n_states;
+    const float* d_weights;    /* [n_states + 1] */
+    const float* d_gamma_in;
+    const int32_t* d_rows;
+    void* d_h;                 /* NULL: no h */
+    int h_dtype;
+    int64_t ldh;               /* columns past dim are zeroed */
+    int32_t* d_status;         /* receives 2 for a token id out of range */
+    int64_t rows, dim;
+} gptrs_depth_step;
+int gptrs_cuda_depth_step(const gptrs_depth_step* step, void* stream);
+/* y = act[0] N(z) + act[1] N(z^2) + act[2] N(z^3) + act[3] for every row, with powers element by element and N dividing a row of n values
+ * by the root of its mean square plus eps. z and y may be the same; columns from n up to ld are zeroed. */
+int gptrs_cuda_poly_norm(const void* d_z, const float* d_act, float eps, void* d_y, int dtype, int64_t rows, int64_t n, int64_t ld, void* stream);
+
+/* ==============================================================================================
  * Attention with grouped key / value heads of any size over a paged cache (no counterpart in gpt.rs; the kernels further down
  * serve gpt.rs' own attention): query head h reads key / value head h / (heads / kv_heads); scores are soft-capped, then
- * r1[h] ln(1 + r2[h] (i - j)) is taken off; a mask says where the keys of position i begin. Pages of 16 tokens hold the
+ * r1[h] ln(1 + r2[h] (i - j)) or r1[h] (i - j) is taken off; a mask says where the keys of position i begin. Pages of 16 tokens hold the
  * [value | key] rows of every kv head.
  *   maps = 2 (differential attention): every query and key head has two parts, each an attention of its own over the same values;
  *            the output is d = a1 - lambda a2, then d / sqrt(mean(d^2) + head_eps) head_scale over the values of the head.
  *   gate     the output is multiplied by sigmoid(gate), a further part of the projection row.
  *   shared_kv  the projection rows hold no keys and values: another layer has put them into the cache.
+ *   taps     queries and keys pass a short causal convolution over time per channel.
+ *   qk_norm  queries and keys are RMS-normed per head, times a gain.
+ *   tied     the values are the keys as they were in front of the norm. The cache then holds them once, with one number per key that
+ *            turns a value into its normed key (16 floats per kv head behind the rows of a page); the keys' gain goes into the queries.
+ * With any of the last three, gptrs_cuda_grouped_prepare takes the place of gptrs_cuda_grouped_append and leaves the queries in rows
+ * of their own.
  * ============================================================================================ */
 enum { GPTRS_MASK_CAUSAL = 0, GPTRS_MASK_WINDOW = 1, GPTRS_MASK_CHUNK = 2 };   /* from 0; i - size + 1; floor(i / size) size */
+enum { GPTRS_DISTANCE_NONE = 0, GPTRS_DISTANCE_LOG = 1, GPTRS_DISTANCE_LINEAR = 2 };   /* r1 ln(1 + r2 d); r1 d */
 typedef struct {
     int dtype;                 /* GPTRS_F32 or GPTRS_BF16: activations and cache */
     int heads, kv_heads, dim, vdim;
     int mask, mask_size;
     float scale, softcap;      /* softcap 0 = none */
-    int distance_bias;         /* 1: r1 and r2 are given */
+    int distance_bias;         /* GPTRS_DISTANCE_* */
     int maps, gate, shared_kv; /* maps 0 = 1 */
-    float lambda_, head_scale, head_eps;   /* two maps: lambda and the constants of the norm */
+    float lambda_, head_scale, head_eps;   /* two maps: lambda and the constants of the norm; qk_norm: head_eps */
+    int taps, qk_norm, tied;   /* taps 0 = no convolution */
     /* filled in by gptrs_cuda_grouped_layout (elements): */
     int q_head_stride, k_offset, k_head_stride, v_offset, v_head_stride, q_row;   /* projection row: queries, keys, values, gate */
     int map_stride;            /* from a head's first map to its second */
     int g_offset, g_head_stride;
     int out_head_stride;       /* attention output of a head */
+    int query_row;             /* row that attention reads its queries from (q_row without gptrs_cuda_grouped_prepare) */
+    int conv_channels;         /* columns of a projection row that pass the convolutions (queries and keys, with padding) */
+    int64_t conv_floats;       /* convolution state of a slot: 2 (taps - 1) conv_channels */
     int64_t page_bytes;
 } gptrs_grouped_attention;
 int gptrs_cuda_grouped_layout(gptrs_grouped_attention* a);
 /* Keys and values of projection rows -> the tokens' pages. */
 int gptrs_cuda_grouped_append(const gptrs_grouped_attention* a, const void* d_qkv, const int32_t* d_positions, const int32_t* d_slot,
                               const int32_t* d_page_table, int64_t max_pages, void* d_pool, int64_t n_tokens, void* stream);
+/* Projection rows -> convolutions with their state, norms -> queries in d_q [rows][query_row], keys and values in the tokens' pages.
+ * Rows come in runs of consecutive positions of one sequence; the last taps - 1 inputs of a sequence have two halves (run_first, run_last
+ * and parity as in gptrs_conv_step). */
+typedef struct {
+    const void* d_qkv;
+    const float* d_conv;       /* [taps][conv_channels], the newest input under the last tap */
+    const float *d_q_gain, *d_k_gain;   /* [dim]; tied: d_q_gain is the product of both gains, d_k_gain is not read */
+    float* d_conv_state;       /* [slots][2][taps - 1][conv_channels] */
+    const int32_t *d_slot, *d_pos, *d_run_first, *d_run_last, *d_parity;
+    const int32_t* d_page_table;
+    int64_t max_pages;
+    void* d_pool;
+    void* d_q;
+    int64_t rows;
+} gptrs_grouped_step;
+int gptrs_cuda_grouped_prepare(const gptrs_grouped_attention* a, const gptrs_grouped_step* step, void* stream);
 /* As for latent attention above: tokens of a query tile of the tensor-core kernel (0: these sizes use the plain kernel), key
  * splits, scratch. */
 int gptrs_cuda_grouped_tile_tokens(const gptrs_grouped_attention* a);
 int gptrs_cuda_grouped_splits(const gptrs_grouped_attention* a, int64_t n_tiles, int64_t max_ctx_len);
 size_t gptrs_cuda_grouped_scratch_bytes(const gptrs_grouped_attention* a, int64_t n_tiles, int splits);
-/* out[T][heads][out_head_stride]; n_tiles = 0: the plain kernel. d_ctx_len[t] = position + 1. */
+/* out[T][heads][out_head_stride]; n_tiles = 0: the plain kernel. d_ctx_len[t] = position + 1. d_reach [kv_heads] or NULL: keys further away
+ * than that are known to weigh nothing and may be left out. */
 int gptrs_cuda_grouped_attention(const gptrs_grouped_attention* a, const void* d_qkv, const void* d_pool, const int32_t* d_page_table,
                                  int64_t max_pages, const int32_t* d_slot, const int32_t* d_ctx_len, const float* d_r1, const float* d_r2,
-                                 const int32_t* d_tile_row, const int32_t* d_tile_rows, int64_t n_tiles, int splits, void* d_out,
+                                 const int32_t* d_reach, const int32_t* d_tile_row, const int32_t* d_tile_rows, int64_t n_tiles, int splits, void* d_out,
                                  void* d_scratch, size_t scratch_bytes, int32_t* d_status, int64_t n_tokens, void* stream);
 
 /* ==============================================================================================
@@ -434,16 +510,19 @@ int gptrs_cuda_grouped_attention(const gptrs_grouped_attention* a, const void* d
  *     S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
  * q, k (kv_heads x dim, shared by heads / kv_heads heads) and v come from short causal convolutions over time with silu; q and k
  * are unit vectors, q times dim^(-1/2); g = exp(-exp(A_log_h) softplus(a + dt_bias)) per head and key channel; the output is
- * o / rms(o) * norm * sigmoid(gate). Rows come in runs of consecutive positions of one sequence (run_first / run_last as above).
+ * o / rms(o) * norm * sigmoid(gate). decay_rank 0: one decay per head (a and dt_bias too), a being a part of the projection row; gate_rank 0:
+ * the gate is a part of the projection row; gate_silu: silu(gate) instead. Rows come in runs of consecutive positions of one sequence
+ * (run_first / run_last as above).
  * The recurrent state is updated in place, the taps - 1 last inputs of the convolutions have two halves (parity as above).
  * ============================================================================================ */
 typedef struct {
     int dtype;                 /* GPTRS_F32 or GPTRS_BF16: projections and output */
     int heads, kv_heads, dim, vdim, taps, decay_rank, gate_rank;
     float eps;
+    int gate_silu;
     /* filled in by gptrs_cuda_delta_layout (elements): */
     int q_offset, k_offset, v_offset, beta_offset, a_offset, g_offset, row;   /* projection row: q, k, v, beta, decay and gate bottlenecks */
-    int decay_row, gate_row;   /* rows of the expanded decay (f32) and gate */
+    int decay_row, gate_row;   /* rows of the expanded decay (f32; 0: none) and gate (row where the gate is a part of it) */
     int out_head_stride;
     int conv_channels;         /* 2 kv_heads dim + heads vdim: rows of d_conv, channels of the convolution state */
     int64_t state_floats;      /* recurrent state of a slot: heads dim vdim */
@@ -453,8 +532,8 @@ int gptrs_cuda_delta_layout(gptrs_delta_rule* a);
 int64_t gptrs_cuda_delta_scratch_floats(const gptrs_delta_rule* a, int64_t rows, int64_t n_runs);
 typedef struct {
     const void* d_proj;        /* [T][row] */
-    const float* d_decay;      /* [T][decay_row] */
-    const void* d_gate;        /* [T][gate_row] */
+    const float* d_decay;      /* [T][decay_row]; not read with decay_rank 0 */
+    const void* d_gate;        /* [T][gate_row]; not read with gate_rank 0 */
     const float* d_conv;       /* [conv_channels][taps], the newest input under the last tap */
     const float *d_a_log, *d_dt_bias, *d_norm;
     float* d_state;            /* [slots][heads][dim][vdim] */
@@ -772,7 +851,7 @@ typedef struct {
 } gptrs_model_config;
 
 /* Layered kind (no counterpart in gpt.rs): every layer has a configuration of its own, a mixer and an optional feed-forward, in
- * one of three block forms:
+ * one of four block forms:
  *   GPTRS_BLOCK_OUTPUT_NORM  norms on the outputs of the sublayers, x <- x + rms(mixer(h)), x <- x + rms(ff(h)); a sublayer reads
  *                            h = x + conv(x), a causal convolution over the last conv_taps positions of every channel whose last
  *                            conv_taps - 1 inputs are part of a sequence's state; the embedding is normed.
@@ -780,22 +859,26 @@ typedef struct {
  *                            position vector is added to the embedding.
  *   GPTRS_BLOCK_PRE_NORM     norms in front of the sublayers; the residual is `streams` copies that are mixed at every sublayer
  *                            (gptrs_stream_step; streams 0: one, x <- x + f(rms(x))); the embedding is scaled by embed_scale.
+ *   GPTRS_BLOCK_DEPTH        norms in norm_groups parts on the outputs of the sublayers, x <- x + residual_mult norm(f(x)); behind every layer x
+ *                            becomes a weighted sum of the embedding and the results of all layers so far (gptrs_depth_step).
  * The logits may be soft-capped. Of gptrs_model_config the fields n_layers, d_model, vocab, context_length, norm_eps, max_*,
  * kv_pages and use_pdl apply. Both weight modes keep the cache in pages; rows of a sequence must arrive in order. Pages that the
  * masks of all layers have passed return to the pool. A layer with weights_of >= 0 uses the weights of that layer (an equal
  * configuration) with a cache and state of its own; one with kv_from >= 0 (grouped attention) reads the cache of that earlier layer and
  * projects no keys and values. Parameter names ([out, in] weights): embed, embed.norm | pos,
- * l<i>.norm1, .norm2, .canon1, .canon2 | .norm1b, .norm2b | .hc1.in, .hc1.out, .hc1.mix, .hc2..., final.norm, head, and per mixer and
+ * l<i>.norm1, .norm2, .canon1, .canon2 | .norm1b, .norm2b | .hc1.in, .hc1.out, .hc1.mix, .hc2... | .dwa, final.norm, head, and per mixer and
  * feed-forward l<i>.mix. and l<i>.mlp.
- *   latent attention   q | dq, dq.norm, uq; dkv, dkv.norm, uk, uv, o
- *   grouped attention  q, q.b, k, k.b, v, v.b, r1, r2, g, lq1, lk1, lq2, lk2, o, o.b
- *   channel delta      q, q.conv, k, k.conv, v, v.conv, b, A_log, a1, a2, dt_bias, g1, g2, norm, o
+ *   latent attention   q | dq, dq.norm, uq; dkv, dkv.norm, uk, uv, sink, o
+ *   grouped attention  q, q.b, q.conv, q.norm, k, k.b, k.conv, k.norm, v, v.b, r1, r2, g, lq1, lk1, lq2, lk2, o, o.b
+ *   channel delta      q, q.conv, k, k.conv, v, v.conv, b, A_log, a1, a2 | a, dt_bias, g1, g2 | g, norm, o
  *   dense xIELU        up, up.b, down, down.b, act
  *   dense gated gelu   gate, up, down
- *   experts            e<j>.gate, e<j>.up, e<j>.down, router, correction, shared.up, shared.down */
+ *   dense poly norm    up, down, act
+ *   experts            e<j>.gate, e<j>.up, e<j>.down, router, correction, shared.gate, shared.up, shared.down, shared.sg
+ * A linear distance bias has no tensor: the slope of head h is 2^(-8 (h + 1) / heads). */
 enum { GPTRS_MIXER_LATENT_ATTENTION = 0, GPTRS_MIXER_GROUPED_ATTENTION = 1, GPTRS_MIXER_CHANNEL_DELTA = 2 };
-enum { GPTRS_MLP_NONE = 0, GPTRS_MLP_DENSE_XIELU = 1, GPTRS_MLP_EXPERTS = 2, GPTRS_MLP_DENSE_GELU = 3 };
-enum { GPTRS_BLOCK_OUTPUT_NORM = 0, GPTRS_BLOCK_SANDWICH = 1, GPTRS_BLOCK_PRE_NORM = 2 };
+enum { GPTRS_MLP_NONE = 0, GPTRS_MLP_DENSE_XIELU = 1, GPTRS_MLP_EXPERTS = 2, GPTRS_MLP_DENSE_GELU = 3, GPTRS_MLP_DENSE_POLY = 4 };
+enum { GPTRS_BLOCK_OUTPUT_NORM = 0, GPTRS_BLOCK_SANDWICH = 1, GPTRS_BLOCK_PRE_NORM = 2, GPTRS_BLOCK_DEPTH = 3 };
 enum { GPTRS_EXPERT_SWIGLU = 0, GPTRS_EXPERT_RELU2 = 1 };   /* W_down (silu(W_gate h) * (W_up h)); W_down max(W_up h, 0)^2 */
 typedef struct {
     int mixer;
@@ -805,7 +888,7 @@ typedef struct {
     int mlp, d_ff;
     int kv_heads, mask, mask_size, distance_bias, proj_bias;   /* grouped attention */
     float softcap;
-    int taps, decay_rank, gate_rank;                           /* channel delta (kv_heads too) */
+    int taps, decay_rank, gate_rank;                           /* channel delta (kv_heads too); grouped attention: taps 0 = no convolution */
     int experts, top, groups, keep;                            /* experts of size d_ff */
     int weights_of;                                            /* -1 = weights of its own */
     int q_rank;                                                /* latent attention: rank of the query latent, 0 = none */
@@ -814,6 +897,11 @@ typedef struct {
     int expert_form, shared_ff;                                /* GPTRS_EXPERT_*; size of the shared expert, 0 = none */
     int route, group_best, correction;                         /* as in gptrs_moe; correction 1 = a vector of that name */
     float weight_scale;
+    int sink, rope_halves;                                     /* latent attention: a sink per head; dimension i is paired with i + rot_dims / 2 */
+    double rope_factor, rope_original, rope_fast, rope_slow;   /* YaRN scaling of the rotation; factor 0 = none */
+    int qk_norm, tied;                                         /* grouped attention */
+    int gate_silu;                                             /* channel delta */
+    int shared_gate;                                           /* the shared expert's output times sigmoid(shared.sg h) */
 } gptrs_layer_config;
 typedef struct {
     int conv_taps;
@@ -821,6 +909,8 @@ typedef struct {
     int block, learned_positions;
     int streams;           /* GPTRS_BLOCK_PRE_NORM */
     float embed_scale;     /* GPTRS_BLOCK_PRE_NORM */
+    float residual_mult;   /* GPTRS_BLOCK_DEPTH */
+    int norm_groups;       /* GPTRS_BLOCK_DEPTH */
 } gptrs_layered_config;
 
 int gptrs_cuda_model_create(const gptrs_model_config* cfg, gptrs_model** out);

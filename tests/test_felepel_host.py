@@ -110,7 +110,7 @@ def test_delta_layout(dtype, want):
     rc, a = layout()
     assert rc == 0 and {k: getattr(a, k) for k in want} == want
     assert (a.state_floats, a.conv_floats) == (6 * 7 * 9, 2 * 3 * 96)
-    for bad in (dict(kv_heads=4), dict(taps=0), dict(dim=1000), dict(decay_rank=0), dict(vdim=0)):
+    for bad in (dict(kv_heads=4), dict(taps=0), dict(dim=1000), dict(decay_rank=-1), dict(vdim=0)):
         assert layout(**bad)[0] != 0, bad
 
 

@@ -178,3 +178,143 @@ def forward(cfg, tensors, tokens, streams=False):
         after.append(x)
     logits = (group_rms(x, groups, eps) * w["final.norm"]) @ w["head"].T
     return (logits, np.stack(after)) if streams else logits
+
+
+# ---- small models for the tests -----------------------------------------------------------------------------------------------
+def dense_mlp(ff=48):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(experts=6, top=2, ff=24, shared=40):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}, **({"shared": {"ff": shared}} if shared else {})}
+
+
+def latent_layer(heads=4, dim=16, rot_dim=8, vdim=12, kv_rank=24, q_rank=20, window=20, base=300.0, scaling=(4.0, 64, 8.0, 1.0), scale=None, mlp=dense_mlp()):
+    """scaling: (factor, original, fast, slow) or None."""
+    rot = {"base": base, "dims": rot_dim}
+    if scaling:
+        rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    m = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "q_rank": q_rank, "rot": rot,
+         "scale": float(scale if scale is not None else (dim + rot_dim) ** -0.5)}
+    return {"type": "latent_attention", "mlp": mlp, "mixer": {**m, "mask": {"size": window}} if window else m}
+
+
+def attention_layer(heads=4, kv_heads=2, dim=16, conv=3, scale=None, mlp=dense_mlp()):
+    return {"type": "attention", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "conv": conv,
+                                                      "scale": float(scale if scale is not None else dim ** -0.5)}}
+
+
+def delta_layer(heads=4, kv_heads=2, dim=16, vdim=24, conv=4, mlp=dense_mlp()):
+    return {"type": "delta", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "conv": conv}}
+
+
+def model_config(layers, width=40, vocab=72, eps=1e-5, groups=2, mult=0.6):
+    return {"architecture": "Domorax", "vocab": vocab, "width": width, "layers": layers, "norm": {"eps": eps, "groups": groups}, "residual_mult": mult}
+
+
+def tensor_shapes(cfg):
+    n, v = cfg["width"], cfg["vocab"]
+    out = {"embed": (v, n)}
+    for i, layer in enumerate(cfg["layers"]):
+        m, p, mlp = layer["mixer"], f"l{i}.", layer["mlp"]
+        x, f = p + "mix.", p + "mlp."
+        heads, dim, vdim, kv = m["heads"], m["dim"], m["vdim"], m.get("kv_heads")
+        out.update({p + "norm1": (n,), p + "dwa": (i + 2,), x + "o": (n, heads * vdim)})
+        if layer["type"] == "latent_attention":
+            rank, rd, qr = m["kv_rank"], m["rot_dim"], m["q_rank"]
+            out.update({x + "dq": (qr, n), x + "dq.norm": (qr,), x + "uq": (heads * (dim + rd), qr), x + "dkv": (rank + rd, n), x + "dkv.norm": (rank,),
+                        x + "uk": (heads * dim, rank), x + "uv": (heads * vdim, rank), x + "sink": (heads,)})
+        elif layer["type"] == "attention":
+            for name, rows in (("q", heads * dim), ("k", kv * dim)):
+                out.update({x + name: (rows, n), x + name + ".conv": (rows, m["conv"]), x + name + ".norm": (dim,)})
+        else:
+            for name, rows in (("q", kv * dim), ("k", kv * dim), ("v", heads * vdim)):
+                out.update({x + name: (rows, n), x + name + ".conv": (rows, m["conv"])})
+            out.update({x + "b": (heads, n), x + "a": (heads, n), x + "A_log": (heads,), x + "dt_bias": (heads,), x + "g": (heads * vdim, n), x + "norm": (vdim,)})
+        if not mlp:
+            continue
+        out[p + "norm2"] = (n,)
+        if mlp["kind"] == "dense":
+            out.update({f + "up": (mlp["ff"], n), f + "down": (n, mlp["ff"]), f + "act": (4,)})
+            continue
+        names = [(f"e{e}.", mlp["expert"]["ff"]) for e in range(mlp["router"]["experts"])]
+        if mlp.get("shared"):
+            names.append(("shared.", mlp["shared"]["ff"]))
+            out[f + "shared.sg"] = (1, n)
+        for name, ff in names:
+            out.update({f + name + "gate": (ff, n), f + name + "up": (ff, n), f + name + "down": (n, ff)})
+        out[f + "router"] = (mlp["router"]["experts"], n)
+    out.update({"final.norm": (n,), "head": (v, n)})
+    return out
+
+
+def random_tensors(cfg, seed=0, sharp=1.0):
+    """bfloat16-valued weights; norm gains around 1, projections of unit output scale (what makes scores larger times `sharp`), sinks that take a
+    share of the softmax, decays between quick and slow, averages over depth that lean on the newest result."""
+    rng = np.random.default_rng(seed)
+    out = {}
+    for name, shape in tensor_shapes(cfg).items():
+        last = name.rsplit(".", 1)[-1]
+        if "norm" in last:
+            w = (1.0 + 0.2 * rng.standard_normal(shape)) * (sharp if name.endswith("q.norm") and not name.endswith("dq.norm") else 1.0)
+        elif last == "conv":
+            w = 0.5 * rng.standard_normal(shape)
+            w[:, -1] += 0.7
+        elif last == "sink":
+            w = rng.uniform(0.5, 3.0, shape)
+        elif last == "dwa":
+            w = 0.25 * rng.standard_normal(shape)
+            w[-1] += 0.8
+        elif last == "act":
+            w = rng.uniform(0.3, 1.0, shape) * np.array([1, 1, -1, 1])
+        elif last == "A_log":
+            w = np.log(rng.uniform(0.3, 3.0, shape))
+        elif last == "dt_bias":
+            w = rng.uniform(-6.0, 0.0, shape)
+        elif last == "router":
+            w = 2.0 * rng.standard_normal(shape) / np.sqrt(shape[-1])
+        elif name == "embed":
+            w = rng.standard_normal(shape)
+        else:
+            w = rng.standard_normal(shape) / np.sqrt(shape[-1]) * (sharp if last == "uq" else 1.0)
+        out[name] = to_bf16(w.astype(np.float32))
+    return out
+
+
+CODE = 8   # width reserved by `steady_routing`
+
+
+def steady_routing(cfg, tensors, seed=0, margin=0.12):
+    """Weights whose routers read the last CODE channels of the stream only, which no sublayer adds to: there every token keeps a code of its
+    own times a number that depends on the layer. Codes are drawn so that no choice is close: rounding then never changes an expert."""
+    rng = np.random.default_rng(seed)
+    t = {n: w.copy() for n, w in tensors.items()}
+    routers, states, now = [], [1.0], 1.0   # what the averages over depth have made of a code of 1
+    for i, layer in enumerate(cfg["layers"]):
+        t[f"l{i}.norm1"][-CODE:] = 0
+        if layer["mlp"]:
+            t[f"l{i}.norm2"][-CODE:] = 0
+        if layer["mlp"] and layer["mlp"]["kind"] == "moe":
+            w = t[f"l{i}.mlp.router"]
+            w[:, :-CODE] = 0
+            w[:, -CODE:] = to_bf16(rng.standard_normal((w.shape[0], CODE)).astype(np.float32))
+            routers.append((w[:, -CODE:].astype(D) * now, layer["mlp"]["router"]["top"]))
+        states.append(now)
+        now = float(np.dot(t[f"l{i}.dwa"].astype(D), states))
+        if abs(now) < 0.3:   # codes would fade: lean on the newest result
+            t[f"l{i}.dwa"] = to_bf16(np.eye(i + 2)[-1].astype(np.float32))
+            now = states[-1]
+
+    def decided(z, top):
+        order = np.sort(z)[::-1]
+        return top == len(z) or order[top - 1] - order[top] >= margin * np.abs(z).max()
+
+    for v in range(cfg["vocab"]):
+        for _ in range(20000):
+            code = to_bf16((1.5 * rng.standard_normal(CODE)).astype(np.float32))
+            if all(decided(w @ code, top) for w, top in routers):
+                break
+        else:
+            raise ValueError("no code with this margin")
+        t["embed"][v, -CODE:] = code
+    return t

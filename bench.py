@@ -26,6 +26,7 @@ from __future__ import annotations
 
 import argparse
 import json
+import math
 import os
 import subprocess
 import sys
@@ -309,6 +310,9 @@ def _random_model(gm, torch, dev, cfg, namespace):
             t = torch.ones(shape, device=dev)
         elif ".hc" in name:   # residual streams that keep themselves, read as their mean
             t = torch.eye(shape[0], device=dev) if last == "mix" else torch.full(shape, 1.0 / shape[0] if last == "in" else 1.0, device=dev)
+        elif last == "dwa":   # averages over depth that lean on the newest result
+            t = torch.full(shape, 0.1, device=dev)
+            t[-1] = 0.9
         elif last in ("r1", "r2", "dt_bias"):   # distance penalties are positive, decays slow
             t = torch.full(shape, -3.0 if last == "dt_bias" else 0.3, device=dev)
         else:
@@ -853,6 +857,221 @@ def run_kozapel_kernels(args, out, ops, torch):
     print(json.dumps(rec), file=out)
 
 
+# ---- Domorax beside Kozapel, Felepel and Bevosun ----------------------------------------------------------------------------------
+# name -> latent attention (heads, dim, rot, vdim, kv rank, q rank, window), attention (heads, kv heads, dim, taps), delta rule (heads, q/k heads,
+# dim, vdim, taps), experts (number, top, size, size of the shared one), dense size; width and vocabulary as in LAYERED_SIZES
+DOMORAX_SIZES = {
+    "w1024": ((16, 64, 32, 64, 128, 384, 1024), (8, 2, 128, 4), (8, 8, 128, 128, 4), (16, 4, 768, 768), 3072),
+    "w2048": ((16, 128, 64, 128, 256, 768, 4096), (16, 4, 128, 4), (16, 16, 128, 128, 4), (32, 6, 1024, 1024), 6144),
+    "w3072": ((32, 96, 32, 96, 256, 1024, 4096), (32, 8, 128, 4), (24, 24, 128, 128, 4), (64, 6, 1536, 1536), 9216),
+}
+DOMORAX_GROUPS = 2
+
+
+def _domorax_model(gm, torch, dev, name, n_layers, ctx, pdl, chunk, batch):
+    width, vocab = LAYERED_SIZES[name][0], LAYERED_SIZES[name][8]
+    (lh, ld, lr, lv, rank, q_rank, window), (h, g, d, taps), (dh, dg, dd, dv, dtaps), (experts, top, eff, shared), ff = DOMORAX_SIZES[name]
+    dense = dict(mlp=gm.MLP_DENSE_POLY, d_ff=ff)
+    moe = dict(mlp=gm.MLP_EXPERTS, d_ff=eff, experts=experts, top=top, weight_scale=1.0, shared_ff=shared, shared_gate=1)
+    lat = dict(heads=lh, dim=ld, rot_dim=lr, vdim=lv, kv_rank=rank, q_rank=q_rank, window=window, scale=(ld + lr) ** -0.5, rope_base=1e6, rope_halves=1, rope_factor=4.0,
+               rope_original=4096.0, rope_fast=32.0, rope_slow=1.0, sink=1, mixer=gm.MIXER_LATENT_ATTENTION)
+    att = dict(heads=h, kv_heads=g, dim=d, vdim=d, scale=d ** -0.5, taps=taps, qk_norm=1, tied=1, distance_bias=gm.DISTANCE_LINEAR, mixer=gm.MIXER_GROUPED_ATTENTION)
+    delta = dict(heads=dh, kv_heads=dg, dim=dd, vdim=dv, taps=dtaps, gate_silu=1, mixer=gm.MIXER_CHANNEL_DELTA)
+    layers = [gm.LayerConfig(**lat, **dense), gm.LayerConfig(**att, **moe), gm.LayerConfig(**delta, **moe), gm.LayerConfig(**lat, **moe)]
+    pages = (ctx + 15) // 16
+    cfg = gm.ModelConfig.layered([layers[i % 4] for i in range(n_layers)], width, vocab, ctx, 1e-6, block=gm.BLOCK_DEPTH, residual_mult=0.3, norm_groups=DOMORAX_GROUPS,
+                                 weight_mode=gm.MODE_BF16, max_seqs=batch, max_tokens=chunk, max_logit_rows=batch, kv_pages=batch * pages + 8, max_pages_per_seq=pages, use_pdl=pdl)
+    return _random_model(gm, torch, dev, cfg, 75)
+
+
+def run_domorax(args, out, gm, torch, np):
+    """Prefill and decode of Domorax (latent attention, attention whose values are keys, delta rule, latent attention; a dense feed-forward and
+    experts; random weights, bf16) beside Kozapel, Felepel and Bevosun of the same width and depth. Not the default line."""
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    n_layers, batch, prompt = 4, BATCH, PROMPT_LEN
+    ctx = prompt + args.steps + args.warmup + 32
+    rec = {"workload": "domorax", "layers": n_layers, "batch": batch, "prompt_tokens": prompt, "steps": args.steps, "warmup": args.warmup, "data": "synthetic", "sizes": {}}
+    sampler = ClockSampler(None)
+    sampler.start()
+    for name in args.sizes.split(","):
+        row = {"domorax": dict(zip(("latent", "attention", "delta", "experts", "ff"), DOMORAX_SIZES[name])), "kozapel": {}, "felepel": {}, "bevosun": {"width": LAYERED_SIZES[name][0]}}
+        builds = (("domorax", lambda *a: _domorax_model(gm, torch, dev, name, *a)), ("kozapel", lambda *a: _kozapel_model(gm, torch, dev, name, *a)),
+                  ("felepel", lambda *a: _felepel_model(gm, torch, dev, name, *a)), ("bevosun", lambda *a: _layered_model(gm, torch, dev, LAYERED_SIZES[name], *a)))
+        for kind, build in builds:
+            m = build(n_layers, ctx, args.pdl, 2048 if kind == "bevosun" else 8192, batch)
+            row[kind].update(_model_speed(gm, torch, np, dev, m, prompt, batch, args.steps, args.warmup))
+            m.close()
+            torch.cuda.empty_cache()
+        rec["sizes"][name] = row
+    rec["clocks"] = sampler.stop()
+    print(json.dumps(rec), file=out)
+
+
+def time_domorax_kernels(ops, torch, dev, name, rows, ctx_len=PROMPT_LEN, only=None):
+    """Every kernel of Domorax's layers by itself at `rows` tokens, as time_layered_kernels does it. Attention counts the keys within the reach
+    that unit gains give the heads of a kv head; the delta rule as in time_felepel_kernels."""
+    w = LAYERED_SIZES[name][0]
+    (lh, ld, lr, lv, rank, q_rank, window), (heads, kv, dim, taps), (dh, dg, dd, dv, dtaps), (experts, top, eff, shared), ff = DOMORAX_SIZES[name]
+    decode = rows <= 128
+    hbm, tf, f32_tf = _peaks()[0], _tensor_peak(), 148 * 128 * 2 * 1.965e-3
+    res = {}
+
+    def put(label, us, nbytes, flops, peak=tf):
+        t_mem, t_op = nbytes / hbm / 1e3, flops / peak / 1e6
+        res[label] = {"us": round(us, 2), "roofline_us": round(max(t_mem, t_op), 2), "bound": "hbm" if t_mem > t_op else ("f32" if peak == f32_tf else "tensor"),
+                      "frac": round(max(t_mem, t_op) / us, 3)}
+
+    bf, i32 = torch.bfloat16, torch.int32
+    status = torch.zeros(1, dtype=i32, device=dev)
+    want = lambda label: only is None or label in only  # noqa: E731
+
+    def gemm(label, n, k, batch=1, ldx=None, x_step=0, ldy=None, y_step=0, out_f32=False, gate=0, **kw):
+        if not want(label):
+            return
+        n8, k8 = (n + 7) // 8 * 8, (k + 7) // 8 * 8
+        per = batch * n8 * k8 * 2
+        mats = [torch.randn(batch, n8, k8, device=dev).mul_(k8 ** -0.5).to(bf) for _ in range(max(2, min(24, (300 << 20) // per)))]
+        x = torch.randn(rows, ldx or k8, device=dev).to(bf)
+        n_out = n8 // 2 if gate else n8
+        y = torch.empty(rows, ldy or n_out, device=dev, dtype=torch.float32 if out_f32 else bf)
+        st = dict(ldx=ldx or k8, ldy=ldy or n8, batch=batch, x_step=x_step, y_step=y_step) if batch > 1 else {"ldx": ldx} if ldx else {}
+        us = _graph_us(torch, [lambda m=m: ops.dense_bf16(x, m, rows, n8, k8, out=y, out_f32=out_f32, swiglu=gate, status=status, **st, **kw) for m in mats])
+        put(label, us, per + rows * batch * (k8 + n_out * (2 if out_f32 else 1)) * 2, 2.0 * rows * n8 * k8 * batch)
+
+    a = ops.grouped_layout(heads, kv, dim, dim, 0, 0, dim ** -0.5, 0.0, 2, head_eps=1e-6, taps=taps, qk_norm=True, tied=True)
+    b = ops.latent_layout(lh, ld, lr, lv, rank, window, (ld + lr) ** -0.5, q_rank=q_rank)
+    d = ops.delta_layout(dh, dg, dd, dv, dtaps, 0, 0, 1e-6, gate_silu=True)
+    gemm("qk", a.q_row, w)
+    gemm("out", w, heads * a.out_head_stride)
+    gemm("latent_in", b.kv_row, w)
+    gemm("latent_uq", b.q_row, q_rank)
+    gemm("absorb_q", b.lat_head_stride, ld, lh, b.q_row, b.q_head_stride, lh * b.qa_head_stride, b.qa_head_stride)
+    gemm("absorb_v", b.out_head_stride, b.lat_head_stride, lh, lh * b.lat_head_stride, b.lat_head_stride, lh * b.out_head_stride, b.out_head_stride)
+    gemm("latent_out", w, lh * b.out_head_stride)
+    gemm("delta_proj", d.row, w)
+    gemm("delta_out", w, dh * d.out_head_stride)
+    gemm("up", ff, w)
+    gemm("down", w, ff)
+    gemm("shared_up", 2 * shared, w, gate=ops.GATE_SILU)
+    gemm("shared_down", w, shared)
+    gemm("router", experts + 1, w, out_f32=True)
+
+    seqs = rows if decode else rows // ctx_len
+    per_seq, pages = rows // seqs, (ctx_len + 15) // 16
+    slot = torch.arange(seqs, dtype=i32, device=dev).repeat_interleave(per_seq).contiguous()
+    pos = (torch.full((rows,), ctx_len - 1, device=dev) if decode else torch.arange(ctx_len, device=dev).repeat(seqs)).to(i32)
+    ctx = (pos + 1).to(i32)
+    table = torch.randperm(seqs * pages, device=dev, dtype=i32).view(seqs, pages).contiguous()
+    lo = torch.arange(rows, device=dev) // per_seq * per_seq
+    runs = (slot, pos, lo.to(i32), (lo + per_seq - 1).to(i32), torch.zeros_like(slot))
+
+    def tiles(t):
+        first = torch.cat([torch.arange(0, per_seq, t, device=dev) + s * per_seq for s in range(seqs)]).to(i32)
+        return first, torch.minimum(torch.full_like(first, t), per_seq - first % per_seq).to(i32)
+
+    def pools(page_bytes):
+        return [torch.randn(seqs * pages * page_bytes // 2, device=dev).to(bf) for _ in range(4 if decode else 1)]
+
+    if want("attention") or want("prepare"):
+        store, ts = pools(a.page_bytes), tiles(1 if decode else ops.grouped_tile_tokens(a))
+        data = kv * 16 * ((dim + 63) // 64) * 64
+        for p in store:   # behind the rows of a page: one float per key
+            p.view(seqs * pages, -1)[:, data:data + kv * 32] = torch.ones(kv * 16, device=dev).view(bf)
+        q, qk = torch.randn(rows, a.query_row, device=dev).to(bf), torch.randn(rows, a.q_row, device=dev).to(bf)
+        slope = [2.0 ** (-8.0 * (h + 1) / heads) for h in range(heads)]
+        reach = [min(1 << 30, math.ceil((2 * 1.02 * dim ** 0.5 + 32) / slope[(g + 1) * (heads // kv) - 1])) for g in range(kv)]
+        r1, d_reach = torch.tensor(slope, device=dev), torch.tensor(reach, dtype=i32, device=dev)
+        us = _graph_us(torch, [lambda p=p: ops.grouped_attention(a, q, p, table, slot, ctx, ctx_len, r1, reach=d_reach, tiles=ts, status=status) for p in store] * (4 if decode else 2))
+        seen = [float(torch.minimum(ctx, torch.full_like(ctx, r + 1)).double().sum()) for r in reach]
+        put("attention", us, (sum(seen) if decode else rows * kv) * (dim * 2 + 4) + rows * heads * 2 * dim * 2, 2.0 * (heads // kv) * 2 * dim * sum(seen))
+        us = _graph_us(torch, [lambda p=p: ops.grouped_attention(a, q, p, table, slot, ctx, ctx_len, r1, tiles=ts, status=status) for p in store] * (4 if decode else 2))
+        every = kv * float(ctx.double().sum())
+        put("attention_all_keys", us, (every if decode else rows * kv) * (dim * 2 + 4) + rows * heads * 2 * dim * 2, 2.0 * (heads // kv) * 2 * dim * every)
+        conv, gain = torch.randn(taps, a.conv_channels, device=dev), torch.ones(dim, device=dev)
+        state = torch.zeros(seqs, max(a.conv_floats, 1), device=dev)
+        us = _graph_us(torch, [lambda p=p: ops.grouped_prepare(a, qk, conv, gain, None, state, runs, table, p) for p in store] * 4)
+        put("prepare", us, rows * (a.q_row + a.query_row + kv * (dim + 2)) * 2 + seqs * a.conv_floats * 4, 0)
+        del store
+    if want("latent_attention") or want("latent_keys"):
+        qa, store, ts, sink = torch.randn(rows, lh, b.qa_head_stride, device=dev).to(bf), pools(b.page_bytes), tiles(1 if decode else ops.latent_tile_tokens(b)), torch.zeros(lh, device=dev)
+        us = _graph_us(torch, [lambda p=p: ops.latent_attention(b, qa, p, table, slot, ctx, ctx_len, tiles=ts, status=status, sink=sink) for p in store] * (4 if decode else 2))
+        pairs = float(torch.minimum(ctx, torch.full_like(ctx, window)).double().sum())
+        put("latent_attention", us, (pairs if decode else rows) * (rank + lr) * 2 + rows * lh * (2 * rank + lr) * 2, 2.0 * lh * (2 * rank + lr) * pairs)
+        kvr, q = torch.randn(rows, b.kv_row, device=dev).to(bf), torch.randn(rows, b.q_row, device=dev).to(bf)
+        cs, sn = torch.randn(ctx_len, lr // 2, device=dev), torch.randn(ctx_len, lr // 2, device=dev)
+        nw, qw = torch.ones(rank, device=dev), torch.ones(q_rank, device=dev)
+        us = _graph_us(torch, [lambda p=p: ops.latent_append_keys(b, kvr, pos, slot, table, nw, qw, 1e-6, cs, sn, p) for p in store] * 4)
+        put("latent_keys", us, rows * (b.kv_row + b.q_latent_row + rank + lr) * 2, 0)
+        us = _graph_us(torch, [lambda: ops.latent_rotate_queries(b, q, pos, cs, sn, qa)] * 8)
+        put("latent_queries", us, rows * lh * lr * 4, 0)
+        del store
+    if want("delta_rule"):
+        starts = (torch.arange(seqs, device=dev) * per_seq).to(i32)
+        proj = torch.randn(rows, d.row, device=dev).to(bf)
+        consts = [torch.randn(d.conv_channels, dtaps, device=dev), torch.zeros(dh, device=dev), torch.full((dh,), -3.0, device=dev), torch.ones(dv, device=dev)]
+        states = [(torch.zeros(seqs, d.state_floats, device=dev), torch.zeros(seqs, max(d.conv_floats, 1), device=dev)) for _ in range(4 if decode else 1)]
+        us = _graph_us(torch, [lambda s=s: ops.delta_rule(d, proj, None, None, *consts, *s, runs, starts) for s in states] * (4 if decode else 1))
+        nbytes = seqs * (d.state_floats * 8 + d.conv_floats * 4) + rows * (d.row + dh * dv) * 2
+        put("delta_rule", us, nbytes, 8.0 * rows * dh * dd * dv, f32_tf)
+        res["delta_rule"]["frac_hbm"] = round(nbytes / hbm / 1e3 / us, 3)
+        del states
+    x, y, gamma = torch.randn(rows, w, device=dev), torch.randn(rows, w, device=dev).to(bf), torch.ones(w, device=dev)
+    hist, avg = torch.randn(4, rows, w, device=dev), torch.tensor([0.1, 0.1, 0.1, 0.7], device=dev)
+    end = dict(states=hist, weights=avg, out_dtype=bf, status=status)
+    if want("depth_step"):
+        us = _graph_us(torch, [lambda: ops.depth_step(DOMORAX_GROUPS, 1e-6, 0.3, x, x, y, gamma, out_dtype=bf, status=status)] * 8)
+        put("depth_step", us, rows * w * (4 + 2 + 4 + 2), 0)
+        us = _graph_us(torch, [lambda: ops.depth_step(DOMORAX_GROUPS, 1e-6, 0.3, x, x, y, gamma, **end)] * 8)
+        put("depth_step_end", us, rows * w * (4 + 2 + 3 * 4 + 4 + 4 + 2), 0)
+    if want("poly_norm"):
+        zs, act = [torch.randn(rows, ff, device=dev).to(bf) for _ in range(max(2, min(24, (300 << 20) // (rows * ff * 2))))], torch.ones(4, device=dev)
+        us = _graph_us(torch, [lambda z=z: ops.poly_norm(z, act, 1e-6, ff, out=z) for z in zs])
+        put("poly_norm", us, rows * ff * 4, 0)
+    if want("experts") or want("route"):
+        mean = rows * top / experts
+        tile = 16 if mean <= 8 else 32 if mean <= 24 else 64 if mean <= 48 else 128
+        z = torch.randn(rows, experts + 1, device=dev)
+        zr = z[:, :experts].contiguous()
+        us = _graph_us(torch, [lambda: ops.moe_route(experts, top, 1, 1, tile, zr, y, weight_scale=1.0)] * 4)
+        put("route", us, rows * experts * 4 + rows * w * 2 * (1 + top), 0)
+        pair, weight, row_tiles, n_tiles, srt, most = ops.moe_route(experts, top, 1, 1, tile, zr, y, weight_scale=1.0)
+        per = experts * 3 * eff * w * 2
+        active = int((torch.zeros(experts, device=dev).index_add_(0, row_tiles[:int(n_tiles), 0].long(), torch.ones(int(n_tiles), device=dev)) > 0).sum())
+        copies = 2 if per > (100 << 20) else 6
+        kw = dict(tiles=row_tiles, n_tiles=n_tiles, max_tiles=most, tile_rows=tile, batch=experts, status=status)
+        mid, ey = torch.empty(rows * top, eff, device=dev, dtype=bf), torch.empty(rows * top, w, device=dev, dtype=bf)
+        ups = [torch.randn(experts, 2 * eff, w, device=dev).mul_(w ** -0.5).to(bf) for _ in range(copies)]
+        us = _graph_us(torch, [lambda m=m: ops.dense_bf16(srt, m, rows * top, 2 * eff, w, out=mid, swiglu=1, **kw) for m in ups] * 2)
+        put("experts_up", us, active * 2 * eff * w * 2 + rows * top * (w + eff) * 2, 4.0 * rows * top * eff * w)
+        del ups
+        downs = [torch.randn(experts, w, eff, device=dev).mul_(eff ** -0.5).to(bf) for _ in range(copies)]
+        us = _graph_us(torch, [lambda m=m: ops.dense_bf16(mid, m, rows * top, w, eff, out=ey, **kw) for m in downs] * 2)
+        put("experts_down", us, active * eff * w * 2 + rows * top * (w + eff) * 2, 2.0 * rows * top * eff * w)
+        del downs
+        us = _graph_us(torch, [lambda: ops.depth_step(DOMORAX_GROUPS, 1e-6, 0.3, x, x, ey, gamma, pair, weight, y, z, **end)] * 4)
+        put("depth_step_experts", us, rows * w * (4 + 2 * top + 2 + 3 * 4 + 4 + 4 + 2), 0)
+    assert int(status) == 0
+    return res
+
+
+def run_domorax_kernels(args, out, ops, torch):
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+    rec = {"microbench": "domorax", "decode_rows": BATCH, "ctx": PROMPT_LEN, "prefill_rows": 4 * PROMPT_LEN, "sizes": {}}
+    only = args.only.split(",") if args.only else None
+    for name in args.sizes.split(","):
+        row = rec["sizes"][name] = {}
+        for phase, rows in (("decode", BATCH), ("prefill", 4 * PROMPT_LEN)):
+            row[phase] = time_domorax_kernels(ops, torch, dev, name, rows, only=only)
+            if only is None:   # the like kernels of the other layered designs
+                row[f"kozapel_{phase}"] = time_kozapel_kernels(ops, torch, dev, name, rows)
+                row[f"felepel_{phase}"] = time_felepel_kernels(ops, torch, dev, name, rows)
+                row[f"bevosun_{phase}"] = time_layered_kernels(ops, torch, dev, LAYERED_SIZES[name], rows)
+        torch.cuda.empty_cache()
+    print(json.dumps(rec), file=out)
+
+
 def run_reference_arm(args):
     """CPU arm: the gpt.rs C backend's kernel library (oracle/_ref) driving the restated f32 decode
     step on the host. The reference's kernels are single-threaded and requests are independent, so one
@@ -1278,17 +1497,18 @@ def _main(out):
     ap.add_argument("--pdl", type=int, default=int(os.environ.get("GPTRS_PDL", "1")))
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-extras", action="store_true", help="skip the kernel microbenchmarks")
-    ap.add_argument("--microbench", default=None, choices=["attention", "attention-ragged", "gemv", "gemv-lm-head", "gemm64", "quant-linear", "prefill", "prefill-attention", "layered", "felepel", "kozapel"],
+    ap.add_argument("--microbench", default=None, choices=["attention", "attention-ragged", "gemv", "gemv-lm-head", "gemm64", "quant-linear", "prefill", "prefill-attention", "layered", "felepel", "kozapel",
+                                                           "domorax"],
                     help="run only one kernel microbenchmark (used for ncu captures) and print its JSON")
     ap.add_argument("--ctx", type=int, default=PROMPT_LEN + 20, help="context length for --microbench attention")
-    ap.add_argument("--workload", default="ministral3b-w4", choices=["ministral3b-w4", "gpt2-fp32", "dp512", "bevosun", "felepel", "kozapel"],
+    ap.add_argument("--workload", default="ministral3b-w4", choices=["ministral3b-w4", "gpt2-fp32", "dp512", "bevosun", "felepel", "kozapel", "domorax"],
                     help="gpt2-fp32 = the reference's CPU-runnable case (one sequence, 32-token prompt, 64 greedy tokens); "
                          "dp512 = 512 requests with prompt lengths U{256..4096}, 256 decode steps each, partitioned over the ranks "
                          "(total work fixed: strong scaling; not the default line); "
                          "bevosun = prefill and decode of the layered kind at three sizes beside the Ministral-shaped model of equal size; "
-                         "felepel = the same for Felepel beside Bevosun; kozapel = the same for Kozapel beside both")
-    ap.add_argument("--sizes", default="w1024,w2048,w3072", help="felepel, kozapel: comma list of sizes")
-    ap.add_argument("--only", default="", help="--microbench felepel, kozapel: comma list of kernels (attention, append, delta_rule, norm_step, experts, route, or a matmul)")
+                         "felepel = the same for Felepel beside Bevosun; kozapel = the same for Kozapel beside both; domorax = the same for Domorax beside all three")
+    ap.add_argument("--sizes", default="w1024,w2048,w3072", help="felepel, kozapel, domorax: comma list of sizes")
+    ap.add_argument("--only", default="", help="--microbench felepel, kozapel, domorax: comma list of kernels (attention, append, delta_rule, norm_step, experts, route, or a matmul)")
     ap.add_argument("--path", default="engine", choices=["engine", "run_program"],
                     help="gpt2-fp32 only: engine = the model-level ABI (default); run_program = every decode step one "
                          "PortableBackend::run_program call on the captured decode program")
@@ -1330,6 +1550,12 @@ def _main(out):
         return
     if args.microbench == "kozapel":
         run_kozapel_kernels(args, out, ops, torch)
+        return
+    if args.microbench == "domorax":
+        run_domorax_kernels(args, out, ops, torch)
+        return
+    if args.workload == "domorax":
+        run_domorax(args, out, gm, torch, np)
         return
     if args.workload == "kozapel":
         run_kozapel(args, out, gm, torch, np)

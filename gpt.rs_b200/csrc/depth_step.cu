@@ -228,60 +228,83 @@ struct PolyParams {
     float eps;
     int bf16, n, ld;
 };
-__device__ __forceinline__ float3 power_scales(const PolyParams& p, float s2, float s4, float s6) {
-    const float n = (float)p.n;
-    return make_float3(p.act[0] / sqrtf(s2 / n + p.eps), p.act[1] / sqrtf(s4 / n + p.eps), p.act[2] / sqrtf(s6 / n + p.eps));
-}
-// sums of three numbers over the CTA
+// Sums of z^2, z^4, z^6 over the CTA -> act[i] / sqrt(mean + eps); the first warp adds up what the warps have.
 template <int THREADS>
-__device__ __forceinline__ float3 row_sum3(float a, float b, float c, float (*sh)[3]) {
-    a = warp_sum(a); b = warp_sum(b); c = warp_sum(c);
-    if ((threadIdx.x & 31) == 0) { float* s = sh[threadIdx.x >> 5]; s[0] = a; s[1] = b; s[2] = c; }
+__device__ __forceinline__ float3 power_scales(const PolyParams& p, float s2, float s4, float s6, float (*sh)[3], float* scale) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    s2 = warp_sum(s2); s4 = warp_sum(s4); s6 = warp_sum(s6);
+    if (lane == 0) { sh[warp][0] = s2; sh[warp][1] = s4; sh[warp][2] = s6; }
     __syncthreads();
-    float3 t = make_float3(0.f, 0.f, 0.f);
+    if (threadIdx.x < 3) {
+        float t = 0.f;
 #pragma unroll
-    for (int w = 0; w < THREADS / 32; ++w) { t.x += sh[w][0]; t.y += sh[w][1]; t.z += sh[w][2]; }
-    return t;
+        for (int w = 0; w < THREADS / 32; ++w) t += sh[w][lane];
+        scale[lane] = p.act[lane] / sqrtf(t / (float)p.n + p.eps);
+    }
+    __syncthreads();
+    return make_float3(scale[0], scale[1], scale[2]);
 }
 
-// A thread holds the columns (i * THREADS + tid) * 4 + e, i < N.
-template <int THREADS, int N>
+// A thread holds the columns (i * THREADS + tid) * 8 + e, i < N, of a row whose length in memory is a multiple of 8.
+template <bool BF16>
+__device__ __forceinline__ void load8(const void* base, size_t i, float (&v)[8]) {
+    if constexpr (BF16) {
+        const uint4 u = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(base) + i);
+        v[0] = bf16_lo(u.x); v[1] = bf16_hi(u.x); v[2] = bf16_lo(u.y); v[3] = bf16_hi(u.y);
+        v[4] = bf16_lo(u.z); v[5] = bf16_hi(u.z); v[6] = bf16_lo(u.w); v[7] = bf16_hi(u.w);
+    } else {
+        const float4* q = reinterpret_cast<const float4*>(static_cast<const float*>(base) + i);
+        const float4 a = q[0], b = q[1];
+        v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+    }
+}
+template <int THREADS, int N, bool BF16>
 __global__ void __launch_bounds__(THREADS) poly_norm_kernel(const PolyParams p) {
-    __shared__ float sh[THREADS / 32][3];
+    __shared__ float sh[THREADS / 32][3], scale[3];
     const int tid = threadIdx.x;
     const size_t base = (size_t)blockIdx.x * p.ld;
     pdl_launch_dependents();
+    const float shift = __ldg(p.act + 3);
     pdl_wait();
-    float z[N][4], s2 = 0.f, s4 = 0.f, s6 = 0.f;
+    float z[N][8], s2 = 0.f, s4 = 0.f, s6 = 0.f;
 #pragma unroll
     for (int i = 0; i < N; ++i) {
-        const int c = (i * THREADS + tid) * 4;
+        const int c = (i * THREADS + tid) * 8;
+        if (c < p.n) load8<BF16>(p.z, base + c, z[i]);
+    }
 #pragma unroll
-        for (int e = 0; e < 4; ++e) z[i][e] = 0.f;
-        if (c >= p.n) continue;
-        load_act<4>(p.z, base + c, p.bf16, z[i]);
+    for (int i = 0; i < N; ++i) {
+        const int left = p.n - (i * THREADS + tid) * 8;
 #pragma unroll
-        for (int e = 0; e < 4; ++e) {
-            if (c + e >= p.n) z[i][e] = 0.f;
+        for (int e = 0; e < 8; ++e) {
+            if (e >= left) z[i][e] = 0.f;
             const float q = z[i][e] * z[i][e], f = q * q;
-            s2 += q; s4 += f; s6 = fmaf(f, q, s6);
+            s2 += q; s4 = fmaf(q, q, s4); s6 = fmaf(f, q, s6);
         }
     }
-    const float3 s = row_sum3<THREADS>(s2, s4, s6, sh), k = power_scales(p, s.x, s.y, s.z);
-    const float shift = p.act[3];
+    const float3 k = power_scales<THREADS>(p, s2, s4, s6, sh, scale);
 #pragma unroll
     for (int i = 0; i < N; ++i) {
-        const int c = (i * THREADS + tid) * 4;
+        const int c = (i * THREADS + tid) * 8, left = p.n - c;
         if (c >= p.ld) continue;
-        float y[4];
+        float y[8];
 #pragma unroll
-        for (int e = 0; e < 4; ++e) y[e] = c + e < p.n ? fmaf(z[i][e], fmaf(z[i][e], fmaf(z[i][e], k.z, k.y), k.x), shift) : 0.f;
-        store_act<4>(p.y, base + c, p.bf16, y);
+        for (int e = 0; e < 8; ++e) y[e] = e < left ? fmaf(z[i][e], fmaf(z[i][e], fmaf(z[i][e], k.z, k.y), k.x), shift) : 0.f;
+        if constexpr (BF16) {
+            *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(p.y) + base + c) = make_uint4(pack_bf16x2(y[0], y[1]), pack_bf16x2(y[2], y[3]), pack_bf16x2(y[4], y[5]), pack_bf16x2(y[6], y[7]));
+        } else {
+            float4* d = reinterpret_cast<float4*>(static_cast<float*>(p.y) + base + c);
+            d[0] = make_float4(y[0], y[1], y[2], y[3]); d[1] = make_float4(y[4], y[5], y[6], y[7]);
+        }
     }
+}
+template <int THREADS, int N>
+int launch_poly(const PolyParams& p, dim3 grid, cudaStream_t st) {
+    return p.bf16 ? launch_kernel(poly_norm_kernel<THREADS, N, true>, grid, dim3(THREADS), 0, st, 1, p) : launch_kernel(poly_norm_kernel<THREADS, N, false>, grid, dim3(THREADS), 0, st, 1, p);
 }
 
 __global__ void __launch_bounds__(kAnyThreads) poly_norm_any_kernel(const PolyParams p) {
-    __shared__ float sh[kAnyThreads / 32][3];
+    __shared__ float sh[kAnyThreads / 32][3], scale[3];
     const int tid = threadIdx.x;
     const size_t base = (size_t)blockIdx.x * p.ld;
     pdl_launch_dependents();
@@ -293,7 +316,7 @@ __global__ void __launch_bounds__(kAnyThreads) poly_norm_any_kernel(const PolyPa
         const float q = z[0] * z[0], f = q * q;
         s2 += q; s4 += f; s6 = fmaf(f, q, s6);
     }
-    const float3 s = row_sum3<kAnyThreads>(s2, s4, s6, sh), k = power_scales(p, s.x, s.y, s.z);
+    const float3 k = power_scales<kAnyThreads>(p, s2, s4, s6, sh, scale);
     for (int c = tid; c < p.ld; c += kAnyThreads) {   // the columns that this thread has read
         float z[1] = {0.f}, y[1] = {0.f};
         if (c < p.n) {
@@ -348,13 +371,15 @@ int gptrs_cuda_poly_norm(const void* d_z, const float* d_act, float eps, void* d
     const PolyParams p = {d_z, d_act, d_y, eps, dtype == GPTRS_BF16, (int)n, (int)ld};
     const dim3 grid((unsigned)rows);
     cudaStream_t st = as_stream(stream);
-    if (ld % 4 == 0) {
-        if (ld <= 512) return launch_kernel(poly_norm_kernel<128, 1>, grid, dim3(128), 0, st, 1, p);
-        if (ld <= 1024) return launch_kernel(poly_norm_kernel<256, 1>, grid, dim3(256), 0, st, 1, p);
-        if (ld <= 2048) return launch_kernel(poly_norm_kernel<256, 2>, grid, dim3(256), 0, st, 1, p);
-        if (ld <= 4096) return launch_kernel(poly_norm_kernel<256, 4>, grid, dim3(256), 0, st, 1, p);
-        if (ld <= 8192) return launch_kernel(poly_norm_kernel<512, 4>, grid, dim3(512), 0, st, 1, p);
-        if (ld <= 16384) return launch_kernel(poly_norm_kernel<512, 8>, grid, dim3(512), 0, st, 1, p);
+    if (ld % 8 == 0) {
+        if (ld <= 1024) return launch_poly<128, 1>(p, grid, st);
+        if (ld <= 2048) return launch_poly<128, 2>(p, grid, st);
+        if (ld <= 3072) return launch_poly<128, 3>(p, grid, st);
+        if (ld <= 4096) return launch_poly<256, 2>(p, grid, st);
+        if (ld <= 6144) return launch_poly<256, 3>(p, grid, st);
+        if (ld <= 9216) return launch_poly<384, 3>(p, grid, st);
+        if (ld <= 12288) return launch_poly<512, 3>(p, grid, st);
+        if (ld <= 16384) return launch_poly<512, 4>(p, grid, st);
     }
     return launch_kernel(poly_norm_any_kernel, grid, dim3(kAnyThreads), 0, st, 1, p);
 }

@@ -124,7 +124,25 @@ __device__ __forceinline__ PrepareRow prepare_row(const PrepareParams& p, int po
     return r;
 }
 
-// A lane holds the channels (i * 32 + lane) * 4 + e, i < NI, of a head; R rows one after another with the inputs before them in registers.
+// Sums of R values over the warp, R a power of two up to 32: lane i gets the sum of v[i mod R].
+template <int R>
+__device__ __forceinline__ float transpose_sum(float (&v)[R]) {
+    const int lane = threadIdx.x & 31;
+#pragma unroll
+    for (int h = R / 2; h >= 1; h >>= 1)
+#pragma unroll
+        for (int i = 0; i < h; ++i) {
+            const float give = (lane & h) ? v[i] : v[i + h], keep = (lane & h) ? v[i + h] : v[i];
+            v[i] = keep + __shfl_xor_sync(0xffffffffu, give, h);
+        }
+#pragma unroll
+    for (int h = R; h < 32; h <<= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], h);
+    return v[0];
+}
+__device__ __forceinline__ void unpack4(const uint2& u, float (&v)[4]) { v[0] = bf16_lo(u.x); v[1] = bf16_hi(u.x); v[2] = bf16_lo(u.y); v[3] = bf16_hi(u.y); }
+
+// A lane holds the channels (i * 32 + lane) * 4 + e, i < NI, of a head for R rows, with the inputs in front of them. Rows away from the ends of
+// their run (nearly all of a prompt's) need nothing but rows of this pass.
 template <int TAPS, int NI, int R>
 __global__ void __launch_bounds__(kPrepareWarps * 32) grouped_prepare_kernel(const PrepareParams p) {
     constexpr int KEEP = TAPS - 1, HIST = KEEP > 0 ? KEEP : 1;
@@ -134,7 +152,7 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) grouped_prepare_kernel(con
     const bool is_q = job < g.heads;
     const int head = is_q ? job : job - g.heads, col0 = is_q ? head * g.q_head_stride : g.k_off + head * g.k_head_stride;
     const bool live = job < g.heads + g.kv_heads, has_gain = p.norm && (is_q || !g.tied);
-    float w[TAPS][NI][4], gain[NI][4];
+    float w[TAPS][NI][4];
 #pragma unroll
     for (int i = 0; i < NI; ++i) {   // constants: on their way before the kernel in front has ended
         const int c = (i * 32 + lane) * 4;
@@ -145,9 +163,6 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) grouped_prepare_kernel(con
                                 : make_float4(0.f, 0.f, 0.f, 0.f);
             w[j][i][0] = v.x; w[j][i][1] = v.y; w[j][i][2] = v.z; w[j][i][3] = v.w;
         }
-        const float* gp = is_q ? p.s.d_q_gain : p.s.d_k_gain;
-#pragma unroll
-        for (int e = 0; e < 4; ++e) gain[i][e] = in && has_gain && c + e < g.dim ? __ldg(gp + c + e) : 1.f;
     }
     pdl_wait();
     if (!live) return;
@@ -158,96 +173,142 @@ __global__ void __launch_bounds__(kPrepareWarps * 32) grouped_prepare_kernel(con
         v_first = p.s.d_run_first[row0 + lane]; v_last = p.s.d_run_last[row0 + lane]; v_par = p.s.d_parity[row0 + lane];
     }
     const __nv_bfloat16* x = static_cast<const __nv_bfloat16*>(p.s.d_qkv) + (size_t)row0 * g.q_row + col0;
-    uint2 cur[R][NI];
+    uint2 raw[KEEP + R][NI];   // rows row0 - KEEP .. row0 + R - 1
 #pragma unroll
-    for (int r = 0; r < R; ++r)
+    for (int r = 0; r < KEEP + R; ++r)
 #pragma unroll
         for (int i = 0; i < NI; ++i) {
             const int c = (i * 32 + lane) * 4;
-            cur[r][i] = r < rows && c < g.map_stride ? *reinterpret_cast<const uint2*>(x + (size_t)r * g.q_row + c) : make_uint2(0, 0);
+            raw[r][i] = r < KEEP + rows && row0 + r >= KEEP && c < g.map_stride ? *reinterpret_cast<const uint2*>(x + (int64_t)(r - KEEP) * g.q_row + c) : make_uint2(0, 0);
         }
-    float hist[HIST][NI][4];   // hist[k]: the input k + 1 positions back
+    const int first = __shfl_sync(0xffffffffu, v_first, 0), last = __shfl_sync(0xffffffffu, v_last, 0);
+    const bool inner = R > 1 && rows == R && row0 - KEEP >= first && row0 + R - 1 + KEEP <= last;
+    float y[R][NI][4], ss[R];
 #pragma unroll
-    for (int r = 0; r < R; ++r) {
-        if (r >= rows) break;
-        const int row = row0 + r;
-        const PrepareRow q = prepare_row(p, __shfl_sync(0xffffffffu, v_pos, r), __shfl_sync(0xffffffffu, v_slot, r), __shfl_sync(0xffffffffu, v_first, r),
-                                         __shfl_sync(0xffffffffu, v_last, r), __shfl_sync(0xffffffffu, v_par, r));
-        if (KEEP > 0 && (r == 0 || row == q.first)) {
+    for (int r = 0; r < R; ++r) ss[r] = 0.f;
+    if (inner || KEEP == 0) {
 #pragma unroll
-            for (int k = 0; k < KEEP; ++k)
+        for (int r = 0; r < R; ++r)
 #pragma unroll
-                for (int i = 0; i < NI; ++i) {
-                    const int c = (i * 32 + lane) * 4, at = q.pos - 1 - k;
-                    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-                    if (c < g.map_stride) {
-                        if (row - 1 - k >= q.first) {
-                            const uint2 u = *reinterpret_cast<const uint2*>(x + (int64_t)(r - 1 - k) * g.q_row + c);
-                            v = make_float4(bf16_lo(u.x), bf16_hi(u.x), bf16_lo(u.y), bf16_hi(u.y));
-                        } else if (at >= 0) {
-                            v = *reinterpret_cast<const float4*>(q.old + (size_t)(at % HIST) * p.channels + col0 + c);
+            for (int i = 0; i < NI; ++i) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) y[r][i][e] = 0.f;
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) {
+                    float v[4];
+                    unpack4(raw[r + j][i], v);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) y[r][i][e] = fmaf(w[j][i][e], v[e], y[r][i][e]);
+                }
+            }
+    } else {
+        float hist[HIST][NI][4];   // hist[k]: the input k + 1 positions back
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            if (r >= rows) break;
+            const int row = row0 + r, pos = __shfl_sync(0xffffffffu, v_pos, r), r_first = __shfl_sync(0xffffffffu, v_first, r), r_last = __shfl_sync(0xffffffffu, v_last, r);
+            const size_t half = (size_t)KEEP * p.channels;
+            const int par = __shfl_sync(0xffffffffu, v_par, r) & 1;
+            float* state = p.s.d_conv_state + (size_t)__shfl_sync(0xffffffffu, v_slot, r) * 2 * half + col0;
+            const float* old = state + par * half;
+            float* fresh = state + (par ^ 1) * half;
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                const int c = (i * 32 + lane) * 4;
+                const bool in = c < g.map_stride;
+                if (r == 0 || row == r_first) {
+#pragma unroll
+                    for (int k = 0; k < KEEP; ++k) {
+                        const int at = pos - 1 - k;
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) hist[k][i][e] = 0.f;
+                        if (row - 1 - k >= r_first) {
+                            unpack4(raw[r + KEEP - 1 - k][i], hist[k][i]);
+                        } else if (at >= 0 && in) {
+                            const float4 v = *reinterpret_cast<const float4*>(old + (size_t)(at % HIST) * p.channels + c);
+                            hist[k][i][0] = v.x; hist[k][i][1] = v.y; hist[k][i][2] = v.z; hist[k][i][3] = v.w;
                         }
                     }
-                    hist[k][i][0] = v.x; hist[k][i][1] = v.y; hist[k][i][2] = v.z; hist[k][i][3] = v.w;
                 }
-        }
-        float y[NI][4], ss = 0.f;
+                float now[4];
+                unpack4(raw[r + KEEP][i], now);
 #pragma unroll
-        for (int i = 0; i < NI; ++i) {
-            const float now[4] = {bf16_lo(cur[r][i].x), bf16_hi(cur[r][i].x), bf16_lo(cur[r][i].y), bf16_hi(cur[r][i].y)};
+                for (int e = 0; e < 4; ++e) {
+                    float a = 0.f;
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                float a = 0.f;
-#pragma unroll
-                for (int k = KEEP - 1; k >= 0; --k) a = fmaf(w[KEEP - 1 - k][i][e], hist[k][i][e], a);
-                y[i][e] = fmaf(w[KEEP][i][e], now[e], a);
-                ss = fmaf(y[i][e], y[i][e], ss);
-            }
-            if constexpr (KEEP > 0) {
-                const int c = (i * 32 + lane) * 4;
-                if (q.last - row < KEEP && c < g.map_stride) {   // the inputs that the sequence's next step needs
-                    float* f = q.fresh + col0 + c;
-                    *reinterpret_cast<float4*>(f + (size_t)(q.pos % HIST) * p.channels) = make_float4(now[0], now[1], now[2], now[3]);
-                    if (row == q.first)   // a run shorter than the state: what it does not push out stays
+                    for (int k = KEEP - 1; k >= 0; --k) a = fmaf(w[KEEP - 1 - k][i][e], hist[k][i][e], a);
+                    y[r][i][e] = fmaf(w[KEEP][i][e], now[e], a);
+                }
+                if (r_last - row < KEEP && in) {   // the inputs that the sequence's next step needs
+                    *reinterpret_cast<float4*>(fresh + (size_t)(pos % HIST) * p.channels + c) = make_float4(now[0], now[1], now[2], now[3]);
+                    if (row == r_first)   // a run shorter than the state: what it does not push out stays
 #pragma unroll
                         for (int k = 0; k < KEEP - 1; ++k)
-                            if (q.pos - 1 - k >= 0 && k + 1 + q.last - row < KEEP)
-                                *reinterpret_cast<float4*>(f + (size_t)((q.pos - 1 - k) % HIST) * p.channels) = make_float4(hist[k][i][0], hist[k][i][1], hist[k][i][2], hist[k][i][3]);
+                            if (pos - 1 - k >= 0 && k + 1 + r_last - row < KEEP)
+                                *reinterpret_cast<float4*>(fresh + (size_t)((pos - 1 - k) % HIST) * p.channels + c) = make_float4(hist[k][i][0], hist[k][i][1], hist[k][i][2], hist[k][i][3]);
                 }
 #pragma unroll
-                for (int k = KEEP - 1; k > 0; --k)
+                for (int e = 0; e < 4; ++e) {
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) hist[k][i][e] = hist[k - 1][i][e];
-#pragma unroll
-                for (int e = 0; e < 4; ++e) hist[0][i][e] = now[e];
+                    for (int k = KEEP - 1; k > 0; --k) hist[k][i][e] = hist[k - 1][i][e];
+                    hist[0][i][e] = now[e];
+                }
             }
         }
-        const float inv = p.norm ? 1.f / sqrtf(warp_sum(ss) / (float)g.dim + p.eps) : 1.f;
-        if (is_q) {
-            __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.s.d_q) + (size_t)row * g.query_row + col0;
+    }
+    float my_inv = 1.f;   // of row lane mod R
+    if (p.norm) {
+#pragma unroll
+        for (int r = 0; r < R; ++r)
+            if (r < rows)
+#pragma unroll
+                for (int i = 0; i < NI; ++i)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) ss[r] = fmaf(y[r][i][e], y[r][i][e], ss[r]);
+        my_inv = 1.f / sqrtf(transpose_sum(ss) / (float)g.dim + p.eps);
+    }
+    float gain[NI][4];
+#pragma unroll
+    for (int i = 0; i < NI; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int c = (i * 32 + lane) * 4 + e;
+            gain[i][e] = has_gain && c < g.dim ? __ldg((is_q ? p.s.d_q_gain : p.s.d_k_gain) + c) : 1.f;
+        }
+    if (is_q) {
+        __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.s.d_q) + (size_t)row0 * g.query_row + col0;
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            if (r >= rows) break;
+            const float inv = __shfl_sync(0xffffffffu, my_inv, r);
 #pragma unroll
             for (int i = 0; i < NI; ++i) {
                 const int c = (i * 32 + lane) * 4;
                 if (c < g.map_stride)
-                    *reinterpret_cast<uint2*>(dst + c) = make_uint2(pack_bf16x2(y[i][0] * inv * gain[i][0], y[i][1] * inv * gain[i][1]),
-                                                                    pack_bf16x2(y[i][2] * inv * gain[i][2], y[i][3] * inv * gain[i][3]));
+                    *reinterpret_cast<uint2*>(dst + (size_t)r * g.query_row + c) = make_uint2(pack_bf16x2(y[r][i][0] * inv * gain[i][0], y[r][i][1] * inv * gain[i][1]),
+                                                                                              pack_bf16x2(y[r][i][2] * inv * gain[i][2], y[r][i][3] * inv * gain[i][3]));
             }
-            continue;
         }
-        const int t = q.pos % kPageTok;
-        unsigned char* block = q.page + head * g.block_bytes;
-        const float f = g.tied ? 1.f : inv;
+        return;
+    }
+    long long v_page = 0;
+    if (lane < rows) v_page = (long long)p.s.d_page_table[(size_t)v_slot * p.s.max_pages + v_pos / kPageTok] * g.page_bytes;
+    if (g.tied && lane < rows) *key_scale(g, static_cast<unsigned char*>(p.s.d_pool) + v_page, head, v_pos % kPageTok) = my_inv;
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+        if (r >= rows) break;
+        const int t = __shfl_sync(0xffffffffu, v_pos, r) % kPageTok;
+        unsigned char* block = static_cast<unsigned char*>(p.s.d_pool) + __shfl_sync(0xffffffffu, v_page, r) + head * g.block_bytes;
+        const float f = g.tied ? 1.f : __shfl_sync(0xffffffffu, my_inv, r);
 #pragma unroll
         for (int i = 0; i < NI; ++i) {   // the columns of the last block that hold no data get zeros
             const int c = (i * 32 + lane) * 4, at = c + (g.tied ? 0 : g.nbv * 64);
             if (c < up(g.dim, 64))
                 *reinterpret_cast<uint2*>(block + page_chunk(t, at >> 3, g.nb) + (at & 7) * 2) =
-                    make_uint2(pack_bf16x2(y[i][0] * f * gain[i][0], y[i][1] * f * gain[i][1]), pack_bf16x2(y[i][2] * f * gain[i][2], y[i][3] * f * gain[i][3]));
+                    make_uint2(pack_bf16x2(y[r][i][0] * f * gain[i][0], y[r][i][1] * f * gain[i][1]), pack_bf16x2(y[r][i][2] * f * gain[i][2], y[r][i][3] * f * gain[i][3]));
         }
-        if (g.tied) {
-            if (lane == 0) *key_scale(g, q.page, head, t) = inv;
-        } else {
-            const __nv_bfloat16* v = static_cast<const __nv_bfloat16*>(p.s.d_qkv) + (size_t)row * g.q_row + g.v_off + head * g.v_head_stride;
+        if (!g.tied) {
+            const __nv_bfloat16* v = static_cast<const __nv_bfloat16*>(p.s.d_qkv) + (size_t)(row0 + r) * g.q_row + g.v_off + head * g.v_head_stride;
             for (int c = lane * 4; c < g.nbv * 64; c += 128)
                 *reinterpret_cast<uint2*>(block + page_chunk(t, c >> 3, g.nb) + (c & 7) * 2) = c < g.v_head_stride ? *reinterpret_cast<const uint2*>(v + c) : make_uint2(0, 0);
         }

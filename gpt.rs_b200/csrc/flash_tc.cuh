@@ -652,11 +652,12 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
 struct CombineParams {
     const float* part_o;
     const float2* part_ml;
-    const int *tile_row, *tile_rows;
+    const int *tile_row, *tile_rows;   // tile_rows null: one row each
     __nv_bfloat16* out;
     int heads, group, rows_per_token, head_blocks, splits, cols, out_stride, vdim;
     HeadOutput head_out;
     const float* sink;
+    int part_rows;                     // rows of a part
 };
 template <bool TWO>
 __global__ void __launch_bounds__(128) flash_combine_kernel(const CombineParams p) {
@@ -666,7 +667,7 @@ __global__ void __launch_bounds__(128) flash_combine_kernel(const CombineParams 
     const int tile = blockIdx.x, hb = blockIdx.z, r = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     const int kvh = hb / p.head_blocks, head_block = hb % p.head_blocks;
     const int heads_n = min(p.rows_per_token, p.group - head_block * kTileRows), heads0 = kvh * p.group + head_block * kTileRows;
-    if (r >= p.tile_rows[tile] * heads_n) return;
+    if (r >= (p.tile_rows ? p.tile_rows[tile] : 1) * heads_n) return;
     const int row = p.tile_row[tile] + r / heads_n, head = heads0 + r % heads_n;
     const HeadOutput& ho = p.head_out;
     constexpr int kSteps = 4;   // 64-column steps: values of up to 256 columns
@@ -675,18 +676,18 @@ __global__ void __launch_bounds__(128) flash_combine_kernel(const CombineParams 
     for (int i = 0; i < kSteps; ++i) acc[i] = make_float2(0.f, 0.f);
 #pragma unroll
     for (int q = 0; q < kParts; ++q) {
-        const size_t part = ((size_t)tile * gridDim.z + hb) * p.splits * kRows + q * (kRows / 2) + r;
+        const size_t part = ((size_t)tile * gridDim.z + hb) * p.splits * p.part_rows + q * (kRows / 2) + r;
         float m = -1e30f;
-        for (int s = 0; s < p.splits; ++s) m = fmaxf(m, p.part_ml[part + (size_t)s * kRows].x);
+        for (int s = 0; s < p.splits; ++s) m = fmaxf(m, p.part_ml[part + (size_t)s * p.part_rows].x);
         float l = 0.f;
-        for (int s = 0; s < p.splits; ++s) { const float2 v = p.part_ml[part + (size_t)s * kRows]; l += v.y * ex2f(v.x - m); }
+        for (int s = 0; s < p.splits; ++s) { const float2 v = p.part_ml[part + (size_t)s * p.part_rows]; l += v.y * ex2f(v.x - m); }
         if (!TWO && p.sink) l += ex2f(fmaf(p.sink[head], kLog2e, -m));
         const float inv = (l > 0.f ? 1.f / l : 0.f) * (q ? -ho.lambda : 1.f);
         for (int s = 0; s < p.splits; ++s) {
-            const float2 v = p.part_ml[part + (size_t)s * kRows];
+            const float2 v = p.part_ml[part + (size_t)s * p.part_rows];
             if (v.y == 0.f) continue;   // a split without a visible key left no output
             const float w = ex2f(v.x - m) * inv;
-            const float* src = p.part_o + (part + (size_t)s * kRows) * p.cols + lane * 2;
+            const float* src = p.part_o + (part + (size_t)s * p.part_rows) * p.cols + lane * 2;
 #pragma unroll
             for (int i = 0; i < kSteps; ++i)
                 if (i * 64 < p.cols) {
@@ -752,7 +753,7 @@ int launch_flash(TcParams& p, int64_t n_tiles, void* d_scratch, cudaStream_t st)
     const size_t smem = (size_t)g.query_blocks * kRows * 128 + (size_t)p.stages * g.blocks * kKeys * 128 + 1024;
     int rc = launch_kernel(flash_tc_kernel<GROUPED, kScores, TWO, LINEAR>, dim3((unsigned)n_tiles, (unsigned)p.splits, (unsigned)z), dim3(kTcThreads), smem, st, 1, p);
     if (rc || p.splits == 1) return rc;
-    CombineParams c = {p.part_o, p.part_ml, p.tile_row, p.tile_rows, p.out, g.heads, g.group, p.rows_per_token, p.head_blocks, p.splits, g.value_blocks * 64, g.out_stride, g.vdim, p.head_out, p.sink};
+    CombineParams c = {p.part_o, p.part_ml, p.tile_row, p.tile_rows, p.out, g.heads, g.group, p.rows_per_token, p.head_blocks, p.splits, g.value_blocks * 64, g.out_stride, g.vdim, p.head_out, p.sink, kRows};
     // CTAs of four warps cover the rows of a tile
     return launch_kernel(flash_combine_kernel<TWO>, dim3((unsigned)n_tiles, kTileRows / 4, (unsigned)z), dim3(128), 0, st, 1, c);
 }

@@ -15,9 +15,10 @@
 //   grouped_prepare_any_kernel  the same for f32 and for sizes that the former does not take, a warp per head and row
 //   grouped_attention_kernel    plain CUDA-core attention, f32 or bf16 cache, any sizes (the f32 path)
 //   flash_tc_kernel<true>       tcgen05 flash attention (flash_tc.cuh), bf16, prompts and decode steps alike
+//   grouped_decode_kernel       decode steps with few heads per kv head, bf16 (grouped_decode.cuh; GPTRS_GROUPED_DECODE=0 keeps the former)
 // A page holds, kv head by kv head, 16 rows of [value | key] or [value | key part 1 | key part 2]; in bf16 all are padded to whole
 // 64-column blocks in the layout of flash_tc.cuh, in f32 the rows are plain.
-#include "flash_tc.cuh"
+#include "grouped_decode.cuh"
 
 namespace gptrs {
 namespace {
@@ -536,6 +537,11 @@ int encode_queries(const void* qkv, const Shape& g, int64_t n_tokens, int heads,
 
 int tile_rows(const Shape& g) { return g.maps > 1 ? kRows / 2 : kRows; }   // rows of a tile that are (token, head) pairs of their own
 int query_blocks(const Shape& g) { return g.tied ? g.nbv : g.nb - g.nbv; }
+uint32_t decode_stage_bytes(const Shape& g) { return (uint32_t)g.block_bytes + (g.tied ? kPageTok * 4u : 0u); }
+bool decode_fits(const Shape& g) {
+    static const bool on = [] { const char* e = getenv("GPTRS_GROUPED_DECODE"); return !e || atoi(e) != 0; }();
+    return on && g.maps == 1 && g.g_head_stride == 0 && g.group <= kDecHeads && g.nbv <= 2 && query_blocks(g) <= 2 && decode_stages(decode_stage_bytes(g)) >= 2;
+}
 int tile_tokens(const Shape& g) { return g.group >= tile_rows(g) ? 1 : tile_rows(g) / g.group; }
 
 }  // namespace
@@ -616,13 +622,18 @@ int gptrs_cuda_grouped_tile_tokens(const gptrs_grouped_attention* a) {
     return tc_fits(query_blocks(g), g.nbv, g.nb) ? tile_tokens(g) : 0;
 }
 
-int gptrs_cuda_grouped_splits(const gptrs_grouped_attention* a, int64_t n_tiles, int64_t max_ctx_len) {
+int gptrs_cuda_grouped_splits(const gptrs_grouped_attention* a, int64_t n_tokens, int64_t n_tiles, int64_t max_ctx_len) {
     const int tokens = gptrs_cuda_grouped_tile_tokens(a);
     if (n_tiles <= 0 || tokens == 0) return 1;
     const int64_t limit = a->mask == GPTRS_MASK_CAUSAL ? max_ctx_len : (int64_t)a->mask_size + tokens - 1;
     const int64_t span = max_ctx_len < limit ? max_ctx_len : limit;
     const int64_t blocks = (span + kPageTok - 1 + kKeys - 1) / kKeys;
     const Shape g = shape_of(*a);
+    if (n_tiles == n_tokens && decode_fits(g)) {   // about two waves, at least 16 pages each
+        int64_t s = ceil_div((int)(2 * kDecCtas * sm_count()), (int)(n_tiles * a->kv_heads));
+        if (s > (span + 16 * kPageTok - 1) / (16 * kPageTok)) s = (span + 16 * kPageTok - 1) / (16 * kPageTok);
+        return (int)(s < 1 ? 1 : s);
+    }
     int64_t s = (tc_fits_twice(query_blocks(g), g.nbv, g.nb) ? 2 : 1) * sm_count() / (n_tiles * a->kv_heads * ceil_div(g.group, tile_rows(g)));
     if (s > blocks) s = blocks;
     return (int)(s < 1 ? 1 : s);
@@ -658,8 +669,24 @@ int gptrs_cuda_grouped_attention(const gptrs_grouped_attention* a, const void* d
     GPTRS_REQUIRE(d_tile_row && d_tile_rows && splits >= 1 && splits <= 65535, "grouped attention: tile list");
     GPTRS_REQUIRE((reinterpret_cast<uintptr_t>(d_pool) & 15) == 0 && (reinterpret_cast<uintptr_t>(d_qkv) & 15) == 0 && (reinterpret_cast<uintptr_t>(d_out) & 15) == 0,
                   "grouped attention: 16-byte alignment");
-    const size_t need = gptrs_cuda_grouped_scratch_bytes(a, n_tiles, splits);
+    const bool decode = n_tiles == n_tokens && decode_fits(g);   // every row is a tile
+    const size_t need = decode ? (splits > 1 ? (size_t)n_tiles * g.kv_heads * splits * kDecHeads * (g.nbv * 256 + 8) : 0) : gptrs_cuda_grouped_scratch_bytes(a, n_tiles, splits);
     GPTRS_REQUIRE(need == 0 || (d_scratch && scratch_bytes >= need), "grouped attention: scratch too small");
+    if (decode) {
+        DecodeParams p = {};
+        FlashShape& f = p.g;
+        f.heads = g.heads; f.kv_heads = g.kv_heads; f.group = g.group; f.blocks = g.nb; f.key_block = g.tied ? 0 : g.nbv; f.mask = g.mask; f.mask_size = g.mask_size;
+        f.out_stride = g.out_stride; f.vdim = g.vdim; f.key_scales = g.tied; f.page_bytes = g.page_bytes; f.block_bytes = (uint32_t)g.block_bytes;
+        p.q = static_cast<const __nv_bfloat16*>(d_qkv); p.q_row = g.query_row; p.q_head_stride = g.q_head_stride; p.q_cols = g.map_stride;
+        p.pool = static_cast<const unsigned char*>(d_pool);
+        p.page_table = d_page_table; p.slot = d_slot; p.ctx_len = d_ctx_len; p.tile_row = d_tile_row;
+        p.out = static_cast<__nv_bfloat16*>(d_out); p.status = d_status;
+        p.max_pages = (int)max_pages; p.splits = splits; p.stage_bytes = (int)decode_stage_bytes(g); p.stages = decode_stages(decode_stage_bytes(g));
+        p.scale = g.scale; p.cap = g.softcap; p.r1 = r1; p.r2 = r2; p.reach = d_reach;
+        const bool k2 = query_blocks(g) == 2, v2 = g.nbv == 2;
+        return k2 ? (v2 ? launch_decode<2, 2>(p, n_tiles, d_scratch, st) : launch_decode<2, 1>(p, n_tiles, d_scratch, st))
+                  : (v2 ? launch_decode<1, 2>(p, n_tiles, d_scratch, st) : launch_decode<1, 1>(p, n_tiles, d_scratch, st));
+    }
     TcParams p = {};
     const int box_heads = g.group < tile_rows(g) ? g.group : tile_rows(g);
     int rc = encode_queries(d_qkv, g, n_tokens, box_heads, tokens, &p.q_map);

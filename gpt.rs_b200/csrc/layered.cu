@@ -921,7 +921,7 @@ struct Pass {
             return rc;
         }
         const Layered::TileSet* t = L.tiles >= 0 ? y.tile_sets[L.tiles].get() : nullptr;
-        const int splits = t ? gptrs_cuda_grouped_splits(&a, t->n, max_ctx) : 1;
+        const int splits = t ? gptrs_cuda_grouped_splits(&a, T, t->n, max_ctx) : 1;
         m.launches += splits > 1 ? 2 : 1;
         if ((rc = gptrs_cuda_grouped_attention(&a, q, pool(L), pages(), m.cfg.max_pages_per_seq, slot(), m.d_ctx.as<int32_t>(), fp(w.r1), fp(w.r2), w.reach.as<int32_t>(),
                                                t ? t->row.as<int32_t>() : nullptr, t ? t->rows.as<int32_t>() : nullptr, t ? t->n : 0, splits, y.attn.p, y.scratch.p,

@@ -621,7 +621,7 @@ def grouped_attention(a, qkv, pool, page_table, slot, ctx_len, max_ctx_len, r1=N
     out = torch.empty((n, a.heads, a.out_head_stride), dtype=qkv.dtype, device=qkv.device)
     n_tiles = 0 if tiles is None else tiles[0].shape[0]
     if splits is None:
-        splits = lib().gptrs_cuda_grouped_splits(ctypes.byref(a), n_tiles, max_ctx_len) if n_tiles else 1
+        splits = lib().gptrs_cuda_grouped_splits(ctypes.byref(a), n, n_tiles, max_ctx_len) if n_tiles else 1
     nbytes = lib().gptrs_cuda_grouped_scratch_bytes(ctypes.byref(a), n_tiles, splits)
     scratch = torch.empty(max(nbytes, 1), dtype=torch.uint8, device=qkv.device)
     check(lib().gptrs_cuda_grouped_attention(ctypes.byref(a), _ptr(qkv), _ptr(pool), _ptr(page_table), page_table.shape[1], _ptr(slot), _ptr(ctx_len), _ptr(r1),

@@ -494,9 +494,9 @@ typedef struct {
 } gptrs_grouped_step;
 int gptrs_cuda_grouped_prepare(const gptrs_grouped_attention* a, const gptrs_grouped_step* step, void* stream);
 /* As for latent attention above: tokens of a query tile of the tensor-core kernel (0: these sizes use the plain kernel), key
- * splits, scratch. */
+ * splits, scratch. Where every row is a tile of its own (a decode step), sizes with few heads per kv head use a kernel for that. */
 int gptrs_cuda_grouped_tile_tokens(const gptrs_grouped_attention* a);
-int gptrs_cuda_grouped_splits(const gptrs_grouped_attention* a, int64_t n_tiles, int64_t max_ctx_len);
+int gptrs_cuda_grouped_splits(const gptrs_grouped_attention* a, int64_t n_tokens, int64_t n_tiles, int64_t max_ctx_len);
 size_t gptrs_cuda_grouped_scratch_bytes(const gptrs_grouped_attention* a, int64_t n_tiles, int splits);
 /* out[T][heads][out_head_stride]; n_tiles = 0: the plain kernel. d_ctx_len[t] = position + 1. d_reach [kv_heads] or NULL: keys further away
  * than that are known to weigh nothing and may be left out. */

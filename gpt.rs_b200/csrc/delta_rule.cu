@@ -11,7 +11,8 @@
 //   S4  = p_3 S0 + sum_t c_t u_t^T,   c_t = k_t (decays of t+1 .. 3)
 //
 // so that a block costs 13 multiply-adds per element of S instead of 16 and one reduction over the key channels instead of four.
-// Every factor is a product of decays, at most 1.
+// Every factor is a product of decays, at most 1. With one decay per head (HEAD) the decays leave the sums: r_t = p_t (S0^T k_t), c_t u_t^T =
+// k_t (decay u_t)^T, so a block is the vectors k_t and q_t and eight numbers more.
 //   delta_prepare_kernel   prompts: a CTA per block, a warp per head: convolutions with their state, unit norms, decays, the vectors
 //                          p_t k_t, p_t q_t, c_t, p_3 and the numbers A, B of the block
 //   delta_scan_kernel      prompts: a warp keeps a few columns of a head's S in registers over a whole run (packed pairs of key channels,
@@ -40,19 +41,21 @@ Geo geo(const gptrs_delta_rule& a) {
     return g;
 }
 constexpr int kBlock = 4;        // tokens of a block
-constexpr int kVecs = 13;        // per block, head and key channel: p_t k_t (4), p_t q_t (4), c_t (4), p_3
-constexpr int kNums = 24;        // per block and head: beta (4), A10 A20 A21 A30 A31 A32 (+ 2), B00 B10 B11 B20 B21 B22 B30 .. B33 (+ 2)
-// Scratch of a prompt's blocks: vectors [block][head][13][dp], values [block][head][4][vp], numbers [block][head][24]; then the
+// per block, head and key channel: p_t k_t (4), p_t q_t (4), c_t (4), p_3; HEAD: k_t (4), q_t (4)
+__host__ __device__ constexpr int vecs_of(bool head_decay) { return head_decay ? 8 : 13; }
+// per block and head: beta (4), A10 A20 A21 A30 A31 A32 (+ 2), B00 B10 B11 B20 B21 B22 B30 .. B33 (+ 2); HEAD: p_t (4), decays of t+1 .. 3 (4)
+__host__ __device__ constexpr int nums_of(bool head_decay) { return head_decay ? 32 : 24; }
+// Scratch of a prompt's blocks: vectors [block][head][vecs][dp], values [block][head][4][vp], numbers [block][head][nums]; then the
 // read-outs [row][head][vp]. Run i with first row r keeps its blocks from number r / 4 + i on.
 struct Planes { float *vec, *v, *num, *o; };
-int64_t block_floats(const Geo& g) { return (int64_t)g.heads * (kVecs * g.dp + kBlock * g.vp + kNums); }
+int64_t block_floats(const Geo& g) { return (int64_t)g.heads * (vecs_of(g.head_decay) * g.dp + kBlock * g.vp + nums_of(g.head_decay)); }
 int64_t max_blocks(int64_t rows, int64_t runs) { return rows / kBlock + runs; }
 Planes planes(const Geo& g, float* s, int64_t rows, int64_t runs) {
     const int64_t n = max_blocks(rows, runs);
     Planes p;
-    p.vec = s; s += n * g.heads * kVecs * g.dp;
+    p.vec = s; s += n * g.heads * vecs_of(g.head_decay) * g.dp;
     p.v = s; s += n * g.heads * kBlock * g.vp;
-    p.num = s; s += n * g.heads * kNums;
+    p.num = s; s += n * g.heads * nums_of(g.head_decay);
     p.o = s;
     return p;
 }
@@ -220,8 +223,9 @@ __device__ __forceinline__ float transpose_sum(float (&v)[N]) {
 }
 
 // NI: groups of 32 key channels
-template <typename T, int NI, int TAPS>
+template <typename T, int NI, int TAPS, bool HEAD>
 __global__ void __launch_bounds__(kPrepThreads, NI <= 4 ? 4 : 1) delta_prepare_kernel(const Params p) {
+    constexpr int kVecs = vecs_of(HEAD), kNums = nums_of(HEAD), ND = HEAD ? 1 : NI;
     const Geo& g = p.g;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, blk = blockIdx.x;
     pdl_launch_dependents();
@@ -264,12 +268,12 @@ __global__ void __launch_bounds__(kPrepThreads, NI <= 4 ? 4 : 1) delta_prepare_k
         }
         const int head = job, kvh = head / g.group;
         const bool own = head % g.group == 0;   // heads that share q and k: the first passes their convolution state on
-        float q[NI][kBlock], k[NI][kBlock], dec[NI][kBlock];
+        float q[NI][kBlock], k[NI][kBlock], dec[ND][kBlock];
 #pragma unroll
-        for (int i = 0; i < NI; ++i)   // travels while the convolutions are computed
+        for (int i = 0; i < ND; ++i)   // travels while the convolutions are computed
 #pragma unroll
             for (int t = 0; t < kBlock; ++t) {
-                const int d = i * 32 + lane;
+                const int d = HEAD ? 0 : i * 32 + lane;
                 dec[i][t] = t < b.n && d < g.dim ? decay_input<T>(p, b.row + t, head, d) : 0.f;
             }
         float sums[8];
@@ -300,10 +304,10 @@ __global__ void __launch_bounds__(kPrepThreads, NI <= 4 ? 4 : 1) delta_prepare_k
         float num[16];   // A in 0 .. 5, B in 6 .. 15
 #pragma unroll
         for (int i = 0; i < 16; ++i) num[i] = 0.f;
+        float gd[kBlock];
+        auto decays = [&](int i, int d) {
 #pragma unroll
-        for (int i = 0; i < NI; ++i) {
-            const int d = i * 32 + lane;
-            float gd[kBlock] = {1.f, 1.f, 1.f, 1.f};
+            for (int t = 0; t < kBlock; ++t) gd[t] = 1.f;
             if (d < g.dim) {
                 const float bias = decay_bias(p, head, d);
 #pragma unroll
@@ -313,6 +317,12 @@ __global__ void __launch_bounds__(kPrepThreads, NI <= 4 ? 4 : 1) delta_prepare_k
                         gd[t] = sizeof(T) == 2 ? decay_fast(x, rate) : expf(rate * softplus(x));
                     }
             }
+        };
+        if (HEAD) decays(0, 0);
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int d = i * 32 + lane;
+            if (!HEAD) decays(HEAD ? 0 : i, d);
             const float g10 = gd[1], g21 = gd[2], g32 = gd[3], g20 = g21 * g10, g31 = g32 * g21, g30 = g31 * g10;   // decays of s+1 .. t
             const float* kk = k[i];
             const float* qq = q[i];
@@ -333,8 +343,13 @@ __global__ void __launch_bounds__(kPrepThreads, NI <= 4 ? 4 : 1) delta_prepare_k
             num[14] = fmaf(qq[3] * kk[2], g32, num[14]);
             num[15] = fmaf(qq[3], kk[3], num[15]);
             if (d < g.dp) {
-                const float p0 = gd[0], p1 = p0 * gd[1], p2 = p1 * gd[2], p3 = p2 * gd[3];
                 float* o = vec + d;
+                if constexpr (HEAD) {
+#pragma unroll
+                    for (int t = 0; t < kBlock; ++t) { o[t * g.dp] = kk[t]; o[(kBlock + t) * g.dp] = qq[t]; }
+                    continue;
+                }
+                const float p0 = gd[0], p1 = p0 * gd[1], p2 = p1 * gd[2], p3 = p2 * gd[3];
                 o[0] = p0 * kk[0]; o[g.dp] = p1 * kk[1]; o[2 * g.dp] = p2 * kk[2]; o[3 * g.dp] = p3 * kk[3];
                 o[4 * g.dp] = p0 * qq[0]; o[5 * g.dp] = p1 * qq[1]; o[6 * g.dp] = p2 * qq[2]; o[7 * g.dp] = p3 * qq[3];
                 o[8 * g.dp] = kk[0] * g30; o[9 * g.dp] = kk[1] * g31; o[10 * g.dp] = kk[2] * g32; o[11 * g.dp] = kk[3];
@@ -344,6 +359,11 @@ __global__ void __launch_bounds__(kPrepThreads, NI <= 4 ? 4 : 1) delta_prepare_k
         const float mine = transpose_sum(num);
         float* dst = p.w.num + ((size_t)blk * g.heads + head) * kNums;
         if (lane < 16) dst[lane < 6 ? 4 + lane : 6 + lane] = mine;
+        if (HEAD && lane == 0) {
+            const float p1 = gd[0] * gd[1], p2 = p1 * gd[2];
+            *reinterpret_cast<float4*>(dst + 24) = make_float4(gd[0], p1, p2, p2 * gd[3]);
+            *reinterpret_cast<float4*>(dst + 28) = make_float4(gd[1] * gd[2] * gd[3], gd[2] * gd[3], gd[3], 1.f);
+        }
         if (lane < kBlock)
             dst[lane] = lane < b.n ? sigmoid(ld(static_cast<const T*>(p.s.d_proj) + (size_t)(b.row + lane) * g.row + g.beta_off + head)) : 0.f;
     }
@@ -354,8 +374,9 @@ constexpr int kScanWarps = 8;
 
 // LPC lanes share a column: lane l holds the channels (LPC i + l) 4 + e, i < NI, of CPL neighbouring columns; 32 / LPC such groups
 // make a warp. dim <= 4 LPC NI. 
-template <int NI, int CPL, int LPC, int STAGES>
+template <int NI, int CPL, int LPC, int STAGES, bool HEAD>
 __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Params p) {
+    constexpr int kVecs = vecs_of(HEAD), kNums = nums_of(HEAD);
     constexpr int W = 4 * LPC * NI;                                 // channels with padding
     constexpr int GROUPS = 32 / LPC, COLS = kScanWarps * GROUPS * CPL;
     constexpr int kStage = kVecs * W + kBlock * COLS + kNums;       // floats
@@ -421,7 +442,8 @@ __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Param
         if (!failed && !mbar_wait_relaxed(&full[b % STAGES], (uint32_t)(b / STAGES) & 1u)) failed = true;   // bounded: reported below
         const float* sm = ds_smem + (b % STAGES) * kStage;
         const float* lanes = sm + l * 4;
-        uint64_t acc[8][CPL];     // p_t k_t, then p_t q_t
+        uint64_t acc[8][CPL];     // p_t k_t, then p_t q_t (HEAD: without p_t)
+        uint64_t kv[HEAD ? NI : 1][kBlock][2];
 #pragma unroll
         for (int x = 0; x < 8; ++x)
 #pragma unroll
@@ -431,6 +453,7 @@ __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Param
 #pragma unroll
             for (int x = 0; x < 8; ++x) {
                 const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(lanes + x * W + 4 * LPC * i);
+                if (HEAD && x < kBlock) { kv[HEAD ? i : 0][x & 3][0] = v.x; kv[HEAD ? i : 0][x & 3][1] = v.y; }
 #pragma unroll
                 for (int j = 0; j < CPL; ++j) acc[x][j] = fma2(S[i][1][j], v.y, fma2(S[i][0][j], v.x, acc[x][j]));
             }
@@ -474,6 +497,14 @@ __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Param
         const float* num = sm + kVecs * W + kBlock * COLS;
         const float4 beta = *reinterpret_cast<const float4*>(num), a0 = *reinterpret_cast<const float4*>(num + 4), a1 = *reinterpret_cast<const float4*>(num + 8);
         const float* vs = sm + kVecs * W + col0 - c_blk + j_mine;
+        float4 tail = make_float4(1.f, 1.f, 1.f, 1.f);
+        uint64_t whole = 0;       // the decay of the block
+        if constexpr (HEAD) {
+            const float4 pt = *reinterpret_cast<const float4*>(num + 24);
+            tail = *reinterpret_cast<const float4*>(num + 28);
+            y[0] *= pt.x; y[1] *= pt.y; y[2] *= pt.z; y[3] *= pt.w;
+            whole = pair_of(pt.w, pt.w);
+        }
         float u[kBlock];          // meaningful in the lanes of the k sums
         u[0] = beta.x * (vs[0] - y[0]);
         u[1] = beta.y * (vs[COLS] - fmaf(a0.x, u[0], y[1]));
@@ -484,7 +515,8 @@ __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Param
         for (int j = 0; j < CPL; ++j)
 #pragma unroll
             for (int t = 0; t < kBlock; ++t) {
-                const float x = __shfl_sync(0xffffffffu, u[t], (lane & ~(LPC - 1)) + ((2 * j) << SH));
+                float x = __shfl_sync(0xffffffffu, u[t], (lane & ~(LPC - 1)) + ((2 * j) << SH));
+                if (HEAD) x *= t == 0 ? tail.x : t == 1 ? tail.y : t == 2 ? tail.z : 1.f;
                 uu[j][t] = pair_of(x, x);
             }
         float uo[kBlock];
@@ -492,12 +524,16 @@ __global__ void __launch_bounds__(kScanWarps * 32) delta_scan_kernel(const Param
         for (int t = 0; t < kBlock; ++t) uo[t] = __shfl_xor_sync(0xffffffffu, u[t], 1 << SH);
 #pragma unroll
         for (int i = 0; i < NI; ++i) {
-            const ulonglong2 gv = *reinterpret_cast<const ulonglong2*>(lanes + 12 * W + 4 * LPC * i);
+            ulonglong2 gv;
+            if constexpr (HEAD) gv = make_ulonglong2(whole, whole);
+            else gv = *reinterpret_cast<const ulonglong2*>(lanes + 12 * W + 4 * LPC * i);
 #pragma unroll
             for (int j = 0; j < CPL; ++j) { S[i][0][j] = mul2(S[i][0][j], gv.x); S[i][1][j] = mul2(S[i][1][j], gv.y); }
 #pragma unroll
             for (int t = 0; t < kBlock; ++t) {
-                const ulonglong2 c = *reinterpret_cast<const ulonglong2*>(lanes + (8 + t) * W + 4 * LPC * i);
+                ulonglong2 c;
+                if constexpr (HEAD) c = make_ulonglong2(kv[i][t][0], kv[i][t][1]);
+                else c = *reinterpret_cast<const ulonglong2*>(lanes + (8 + t) * W + 4 * LPC * i);
 #pragma unroll
                 for (int j = 0; j < CPL; ++j) { S[i][0][j] = fma2(c.x, uu[j][t], S[i][0][j]); S[i][1][j] = fma2(c.y, uu[j][t], S[i][1][j]); }
             }
@@ -687,20 +723,31 @@ __global__ void __launch_bounds__(kDecThreads, NR * VEC <= 64 ? 2 : 1) delta_dec
     for (int c = tid; c < g.out_stride; c += kDecThreads) st(out + c, c < g.vdim ? o[c] * inv * p.s.d_norm[c] * gate_of(g, ld(gate + c)) : 0.f);
 }
 
+template <int NI, int CPL, int LPC, int STAGES, bool HEAD>
+int launch_scan_of(const Params& p, cudaStream_t s) {
+    constexpr int cols = kScanWarps * 32 / LPC * CPL;
+    constexpr size_t smem = (size_t)STAGES * (vecs_of(HEAD) * 4 * LPC * NI + kBlock * cols + nums_of(HEAD)) * 4;
+    static PerDeviceOnce once;
+    if (once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(delta_scan_kernel<NI, CPL, LPC, STAGES, HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    return launch_kernel(delta_scan_kernel<NI, CPL, LPC, STAGES, HEAD>, dim3((unsigned)ceil_div(p.g.vdim, cols), (unsigned)p.g.heads, (unsigned)p.s.n_runs), dim3(kScanWarps * 32), smem,
+                         s, 1, p);
+}
 template <int NI, int CPL, int LPC, int STAGES>
 int launch_scan(const Params& p, cudaStream_t s) {
-    constexpr int cols = kScanWarps * 32 / LPC * CPL;
-    constexpr size_t smem = (size_t)STAGES * (kVecs * 4 * LPC * NI + kBlock * cols + kNums) * 4;
-    static PerDeviceOnce once;
-    if (once.first_time()) GPTRS_CUDA_OK(cudaFuncSetAttribute(delta_scan_kernel<NI, CPL, LPC, STAGES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    return launch_kernel(delta_scan_kernel<NI, CPL, LPC, STAGES>, dim3((unsigned)ceil_div(p.g.vdim, cols), (unsigned)p.g.heads, (unsigned)p.s.n_runs), dim3(kScanWarps * 32), smem,
-                         s, 1, p);
+    // a run is a chain of blocks: while there are SMs to spare, fewer columns per warp make its links shorter
+    if constexpr (CPL > 1 && LPC == 16) {
+        constexpr int cols = kScanWarps * 32 / LPC * CPL;
+        if ((int64_t)ceil_div(p.g.vdim, cols) * p.g.heads * p.s.n_runs * 2 <= sm_count()) return launch_scan<NI, CPL / 2, LPC, STAGES>(p, s);
+    }
+    return p.g.head_decay ? launch_scan_of<NI, CPL, LPC, STAGES, true>(p, s) : launch_scan_of<NI, CPL, LPC, STAGES, false>(p, s);
 }
 template <typename T, int NI>
 int launch_prepare(const Params& p, cudaStream_t s) {
     const dim3 grid((unsigned)max_blocks(p.s.rows, p.s.n_runs));
-    if (p.g.taps == 4) return launch_kernel(delta_prepare_kernel<T, NI, 4>, grid, dim3(kPrepThreads), 0, s, 1, p);
-    return launch_kernel(delta_prepare_kernel<T, NI, 0>, grid, dim3(kPrepThreads), 0, s, 1, p);
+    constexpr int kTaps = NI <= 8 ? 4 : 0;   // convolutions of four taps are unrolled
+    void (*kern)(Params) = p.g.head_decay ? (p.g.taps == kTaps ? delta_prepare_kernel<T, NI, kTaps, true> : delta_prepare_kernel<T, NI, 0, true>)
+                                          : (p.g.taps == kTaps ? delta_prepare_kernel<T, NI, kTaps, false> : delta_prepare_kernel<T, NI, 0, false>);
+    return launch_kernel(kern, grid, dim3(kPrepThreads), 0, s, 1, p);
 }
 template <typename T, int NR, int VEC>
 int launch_decode(const Params& p, cudaStream_t s) {

@@ -404,7 +404,8 @@ def test_latent_attention_with_sinks(cuda, mode, heads, rank, rot, window):
 
 # ---- delta rule with a decay per head --------------------------------------------------------------------------------------
 @pytest.mark.parametrize("heads,kv,dim,vdim,taps", [(1, 1, 8, 8, 4), (4, 2, 16, 24, 3), (6, 6, 32, 64, 4), (3, 1, 5, 7, 2), (2, 2, 64, 40, 1), (4, 4, 128, 128, 4), (2, 1, 100, 130, 5),
-                                                    (2, 2, 200, 260, 4), (1, 1, 300, 33, 7), (12, 3, 32, 20, 4)])
+                                                    (2, 2, 200, 260, 4), (1, 1, 300, 33, 7), (12, 3, 32, 20, 4),
+                                                    (16, 8, 72, 24, 4), (30, 10, 72, 24, 4)])   # columns per warp depend on the number of heads and runs
 @pytest.mark.parametrize("bf16", [False, True])
 def test_delta_rule_with_head_decays_over_any_cut(cuda, heads, kv, dim, vdim, taps, bf16):
     rng = np.random.default_rng(dim + vdim)

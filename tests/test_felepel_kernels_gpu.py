@@ -330,7 +330,8 @@ def _runs(parts, parity, cuda):
 
 DELTA_SHAPES = [  # heads, q/k heads, dim, vdim, taps, decay rank, gate rank
     (1, 1, 8, 8, 4, 8, 8), (4, 2, 16, 24, 3, 10, 6), (6, 6, 32, 64, 4, 24, 40), (3, 1, 5, 7, 2, 3, 1), (2, 2, 64, 40, 1, 8, 8), (4, 4, 128, 128, 4, 16, 16),
-    (2, 1, 100, 130, 5, 16, 16), (2, 2, 200, 260, 4, 8, 8), (1, 1, 300, 33, 7, 8, 8)]
+    (2, 1, 100, 130, 5, 16, 16), (2, 2, 200, 260, 4, 8, 8), (1, 1, 300, 33, 7, 8, 8),
+    (16, 8, 40, 24, 4, 8, 8), (30, 10, 40, 24, 4, 8, 8)]   # columns per warp depend on the number of heads and runs
 
 
 @pytest.mark.parametrize("shape", DELTA_SHAPES)

@@ -272,7 +272,7 @@ __global__ void __launch_bounds__(kTcThreads, kScores == 2 ? 2 : 1) flash_tc_ker
     }
     pdl_wait();
     const int tile = (int)gridDim.x - 1 - (int)blockIdx.x;   // long contexts come last in a token list: start them first
-    const int row0 = p.tile_row[tile], n_tok = p.tile_rows[tile], hb = blockIdx.z;
+    const int row0 = p.tile_row[tile], n_tok = p.tile_rows[tile], hb = LINEAR ? (int)gridDim.z - 1 - (int)blockIdx.z : (int)blockIdx.z;   // later kv heads reach further
     const int kvh = GROUPED ? hb / p.head_blocks : 0, head_block = GROUPED ? hb % p.head_blocks : hb;
     const int heads_n = min(p.rows_per_token, g.group - head_block * kTileRows);   // heads of this CTA per token
     const int heads0 = kvh * g.group + head_block * kTileRows;
@@ -677,24 +677,36 @@ __global__ void __launch_bounds__(128) flash_combine_kernel(const CombineParams 
 #pragma unroll
     for (int q = 0; q < kParts; ++q) {
         const size_t part = ((size_t)tile * gridDim.z + hb) * p.splits * p.part_rows + q * (kRows / 2) + r;
-        float m = -1e30f;
-        for (int s = 0; s < p.splits; ++s) m = fmaxf(m, p.part_ml[part + (size_t)s * p.part_rows].x);
-        float l = 0.f;
-        for (int s = 0; s < p.splits; ++s) { const float2 v = p.part_ml[part + (size_t)s * p.part_rows]; l += v.y * ex2f(v.x - m); }
+        // a lane per split, 32 at a time
+        auto part_of = [&](int s) { return s < p.splits ? p.part_ml[part + (size_t)s * p.part_rows] : make_float2(-1e30f, 0.f); };
+        float m = -1e30f, l = 0.f;
+        int best = 0;
+        for (int s0 = 0; s0 < p.splits; s0 += 32) {
+            const float2 v = part_of(s0 + lane);
+            const float top = warp_max(v.y == 0.f ? -1e30f : v.x);
+            if (top > m) { m = top; best = s0 + __ffs(__ballot_sync(0xffffffffu, v.y != 0.f && v.x == top)) - 1; }
+        }
+        for (int s0 = 0; s0 < p.splits; s0 += 32) { const float2 v = part_of(s0 + lane); l += v.y * ex2f(v.x - m); }
+        l = warp_sum(l);
         if (!TWO && p.sink) l += ex2f(fmaf(p.sink[head], kLog2e, -m));
         const float inv = (l > 0.f ? 1.f / l : 0.f) * (q ? -ho.lambda : 1.f);
-        for (int s = 0; s < p.splits; ++s) {
-            const float2 v = p.part_ml[part + (size_t)s * p.part_rows];
-            if (v.y == 0.f) continue;   // a split without a visible key left no output
-            const float w = ex2f(v.x - m) * inv;
-            const float* src = p.part_o + (part + (size_t)s * p.part_rows) * p.cols + lane * 2;
+        for (int s0 = 0; s0 < p.splits; s0 += 32) {
+            const float2 v = part_of(s0 + lane);
+            const float mine = v.y == 0.f ? 0.f : ex2f(v.x - m) * inv;
+            const int n = min(32, p.splits - s0);
+#pragma unroll 4
+            for (int k = 0; k < n; ++k) {
+                const float w = __shfl_sync(0xffffffffu, mine, k);
+                const int s = w != 0.f ? s0 + k : best;   // a split without a visible key left no output
+                const float* src = p.part_o + (part + (size_t)s * p.part_rows) * p.cols + lane * 2;
 #pragma unroll
-            for (int i = 0; i < kSteps; ++i)
-                if (i * 64 < p.cols) {
-                    const float2 o = *reinterpret_cast<const float2*>(src + i * 64);
-                    acc[i].x = fmaf(w, o.x, acc[i].x);
-                    acc[i].y = fmaf(w, o.y, acc[i].y);
-                }
+                for (int i = 0; i < kSteps; ++i)
+                    if (i * 64 < p.cols) {
+                        const float2 o = *reinterpret_cast<const float2*>(src + i * 64);
+                        acc[i].x = fmaf(w, o.x, acc[i].x);
+                        acc[i].y = fmaf(w, o.y, acc[i].y);
+                    }
+            }
         }
     }
     float f = 1.f;

@@ -629,11 +629,7 @@ int gptrs_cuda_grouped_splits(const gptrs_grouped_attention* a, int64_t n_tokens
     const int64_t span = max_ctx_len < limit ? max_ctx_len : limit;
     const int64_t blocks = (span + kPageTok - 1 + kKeys - 1) / kKeys;
     const Shape g = shape_of(*a);
-    if (n_tiles == n_tokens && decode_fits(g)) {   // about two waves, at least 16 pages each
-        int64_t s = ceil_div((int)(2 * kDecCtas * sm_count()), (int)(n_tiles * a->kv_heads));
-        if (s > (span + 16 * kPageTok - 1) / (16 * kPageTok)) s = (span + 16 * kPageTok - 1) / (16 * kPageTok);
-        return (int)(s < 1 ? 1 : s);
-    }
+    if (n_tiles == n_tokens && decode_fits(g)) return decode_splits(n_tiles * a->kv_heads, span);
     int64_t s = (tc_fits_twice(query_blocks(g), g.nbv, g.nb) ? 2 : 1) * sm_count() / (n_tiles * a->kv_heads * ceil_div(g.group, tile_rows(g)));
     if (s > blocks) s = blocks;
     return (int)(s < 1 ? 1 : s);

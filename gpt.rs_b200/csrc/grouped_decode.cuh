@@ -40,7 +40,7 @@ __global__ void __launch_bounds__(kDecWarps * 32, kDecCtas) grouped_decode_kerne
     __shared__ float2 s_ml[kDecWarps][kDecHeads];
     const FlashShape& g = p.g;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, gi = lane >> 2, t = lane & 3;
-    const int kvh = blockIdx.z, group = g.group;
+    const int kvh = (int)gridDim.z - 1 - (int)blockIdx.z, group = g.group;   // later kv heads reach further: start them first
     unsigned char* ring = gd_smem + warp * p.stages * p.stage_bytes;
     if (lane == 0) {
         for (int i = 0; i < p.stages; ++i) mbar_init(&full[warp][i], 1);
@@ -222,6 +222,16 @@ __global__ void __launch_bounds__(kDecWarps * 32, kDecCtas) grouped_decode_kerne
             *reinterpret_cast<uint2*>(p.out + ((size_t)row * g.heads + kvh * group + r) * g.out_stride + c) = make_uint2(pack_bf16x2(a.x * inv, a.y * inv), pack_bf16x2(a.z * inv, a.w * inv));
         }
     }
+}
+
+// Key splits of a decode step: a wave of CTAs (three where sequences are long, since heads with a reach end early), but not so many that the
+// merge, which takes their parts one after another, weighs more than the pages a warp then does not have to walk.
+inline int decode_splits(int64_t ctas, int64_t span) {
+    const int64_t pages = span / kPageTok + 1, slots = (int64_t)kDecCtas * sm_count() * (pages >= 512 ? 3 : 1);
+    int64_t s = (2 * slots + ctas) / (2 * ctas), most = (int64_t)(0.7 * sqrt((double)pages));
+    if (most > pages / 16) most = pages / 16;
+    if (s > most) s = most;
+    return (int)(s < 1 ? 1 : s);
 }
 
 // stages of a warp's ring (0: these sizes do not fit)

@@ -351,7 +351,7 @@ def test_decode_equals_prompt_rows(cuda):
     r1 = _slopes(a)
     whole = c.attend(q, slot, pos, r1, "tc", 1)
     for pick in ([5], [299, 376], [0, 300, 64, 169, 310, 170, 171, 299]):
-        for splits in (1, 2, 3, 4, 9):
+        for splits in (1, 2, 3, 4, 9, 40):
             got = c.attend(q[pick].contiguous(), [slot[i] for i in pick], [pos[i] for i in pick], r1, "tc", splits)
             assert np.abs(got - whole[pick]).max() < 2 ** -7 * np.abs(whole).max()
 

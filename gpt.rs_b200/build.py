@@ -22,7 +22,7 @@ NVCC_FLAGS = [
     "-O3", "-std=c++17", "-lineinfo",
     "-Xcompiler", "-fPIC,-Wall,-Wno-unused-function",
     "--expt-relaxed-constexpr",
-    "-DGPTRS_BUILDING=1", "--split-compile=4",
+    "-DGPTRS_BUILDING=1",
 ]
 
 

@@ -13,7 +13,7 @@
 // so that a block costs 13 multiply-adds per element of S instead of 16 and one reduction over the key channels instead of four.
 // Every factor is a product of decays, at most 1. With one decay per head (HEAD) the decays leave the sums: r_t = p_t (S0^T k_t), c_t u_t^T =
 // k_t (decay u_t)^T, so a block is the vectors k_t and q_t and eight numbers more.
-//   delta_prepare_kernel   prompts: a CTA per block, a warp per head: convolutions with their state, unit norms, decays, the vectors
+//   delta_prepare_kernel   (delta_prepare.cu) prompts: a CTA per block, a warp per head: convolutions with their state, unit norms, decays, the vectors
 //                          p_t k_t, p_t q_t, c_t, p_3 and the numbers A, B of the block
 //   delta_scan_kernel      prompts: a warp keeps a few columns of a head's S in registers over a whole run (packed pairs of key channels,
 //                          fma.rn.f32x2); blocks arrive by bulk copies in a ring of shared-memory stages (bounded waits, status 3); the sums meet in a transposing reduction
@@ -22,82 +22,13 @@
 //                          written once
 // Everything that enters the recurrence, and S itself, is f32. S is updated in place (one CTA owns a column of a slot's state);
 // the convolution state has two halves like the one of post_norm_conv.cu.
-#include "umma_common.cuh"
+#include "delta_rule.cuh"
 
 namespace gptrs {
+namespace delta {
 namespace {
 
-struct Geo {
-    int heads, kv_heads, group, dim, vdim, taps;
-    int q_off, k_off, v_off, beta_off, row, decay_row, gate_row, out_stride, channels;
-    int dp, vp;              // dim and vdim of the f32 planes, multiples of 4
-    float eps, q_scale;
-    int head_decay, a_off, gate_silu;   // one decay per head: column a_off + head of the projection row
-};
-__host__ __device__ inline int pad4(int v) { return (v + 3) / 4 * 4; }
-Geo geo(const gptrs_delta_rule& a) {
-    Geo g = {a.heads, a.kv_heads, a.heads / a.kv_heads, a.dim, a.vdim, a.taps, a.q_offset, a.k_offset, a.v_offset, a.beta_offset, a.row, a.decay_row, a.gate_row,
-             a.out_head_stride, a.conv_channels, pad4(a.dim), pad4(a.vdim), a.eps, 1.f / sqrtf((float)a.dim), a.decay_rank == 0, a.a_offset, a.gate_silu};
-    return g;
-}
-constexpr int kBlock = 4;        // tokens of a block
-// per block, head and key channel: p_t k_t (4), p_t q_t (4), c_t (4), p_3; HEAD: k_t (4), q_t (4)
-__host__ __device__ constexpr int vecs_of(bool head_decay) { return head_decay ? 8 : 13; }
-// per block and head: beta (4), A10 A20 A21 A30 A31 A32 (+ 2), B00 B10 B11 B20 B21 B22 B30 .. B33 (+ 2); HEAD: p_t (4), decays of t+1 .. 3 (4)
-__host__ __device__ constexpr int nums_of(bool head_decay) { return head_decay ? 32 : 24; }
-// Scratch of a prompt's blocks: vectors [block][head][vecs][dp], values [block][head][4][vp], numbers [block][head][nums]; then the
-// read-outs [row][head][vp]. Run i with first row r keeps its blocks from number r / 4 + i on.
-struct Planes { float *vec, *v, *num, *o; };
-int64_t block_floats(const Geo& g) { return (int64_t)g.heads * (vecs_of(g.head_decay) * g.dp + kBlock * g.vp + nums_of(g.head_decay)); }
-int64_t max_blocks(int64_t rows, int64_t runs) { return rows / kBlock + runs; }
-Planes planes(const Geo& g, float* s, int64_t rows, int64_t runs) {
-    const int64_t n = max_blocks(rows, runs);
-    Planes p;
-    p.vec = s; s += n * g.heads * vecs_of(g.head_decay) * g.dp;
-    p.v = s; s += n * g.heads * kBlock * g.vp;
-    p.num = s; s += n * g.heads * nums_of(g.head_decay);
-    p.o = s;
-    return p;
-}
-
-struct Params {
-    gptrs_delta_step s;
-    Geo g;
-    Planes w;
-};
-
-__device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
-__device__ __forceinline__ float sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
-__device__ __forceinline__ float softplus(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
-template <typename T>
-__device__ __forceinline__ float ld(const T* p) {
-    if constexpr (sizeof(T) == 2) return __bfloat162float(*p);
-    else return *p;
-}
-template <typename T>
-__device__ __forceinline__ void st(T* p, float v) {
-    if constexpr (sizeof(T) == 2) *p = __float2bfloat16_rn(v);
-    else *p = v;
-}
-// silu of a convolution that is rounded to bf16 anyway; exp(rate softplus(x)) with the hardware's exponential and logarithm, the latter
-// as the series of ln(1 + e) where 1 + e would lose e
-__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f + __expf(-x)); }
-__device__ __forceinline__ float decay_fast(float x, float rate) {
-    const float e = __expf(-fabsf(x));
-    const float series = e * fmaf(e, fmaf(e, fmaf(e, -0.25f, 1.f / 3.f), -0.5f), 1.f);
-    return __expf(rate * (fmaxf(x, 0.f) + (e < 0.02f ? series : __logf(1.f + e))));
-}
-// what the softplus of a decay takes, without its bias; the bias
-template <typename T>
-__device__ __forceinline__ float decay_input(const Params& p, int row, int head, int d) {
-    return p.g.head_decay ? ld(static_cast<const T*>(p.s.d_proj) + (size_t)row * p.g.row + p.g.a_off + head) : p.s.d_decay[(size_t)row * p.g.decay_row + head * p.g.dim + d];
-}
-__device__ __forceinline__ float decay_bias(const Params& p, int head, int d) { return p.s.d_dt_bias[p.g.head_decay ? head : head * p.g.dim + d]; }
-template <typename T>
-__device__ __forceinline__ float decay_of(const Params& p, int row, int head, int d) {
-    return expf(-expf(p.s.d_a_log[head]) * softplus(decay_input<T>(p, row, head, d) + decay_bias(p, head, d)));
-}
-__device__ __forceinline__ float gate_of(const Geo& g, float z) { return g.gate_silu ? silu(z) : sigmoid(z); }
+constexpr int kMaxDim = 512;
 
 // The convolution state that a single-token run reads and writes; place: where in the ring of taps - 1 inputs the last one lies.
 struct RowState { int pos, place; const float* old; float* fresh; };
@@ -151,222 +82,6 @@ __device__ __forceinline__ float conv_channel(const Params& p, const RowState& r
     }
     if (keep_state) r.fresh[(size_t)(r.pos % keep) * p.g.channels + ch] = now;
     return silu(fmaf(w[keep], now, acc));
-}
-
-constexpr int kMaxDim = 512;
-constexpr int kPrepThreads = 256;
-
-// What a block's channels need: the first row of the block, its live tokens, the convolution state of the sequence.
-struct BlockState { bool inner; int row, n, first, last, pos; const float* old; float* fresh; };
-// silu(convolution) of channel `ch` (column `col` of the projection rows) for the tokens of a block; tokens that are not there give 0.
-// TAPS 0: any number. `keep_state`: this thread also passes the channel's inputs on to the next step.
-template <typename T, int TAPS>
-__device__ __forceinline__ void conv_block(const Params& p, const BlockState& b, int ch, int col, bool keep_state, float (&out)[kBlock]) {
-    const int taps = TAPS ? TAPS : p.g.taps, keep = taps - 1;
-    const T* x = static_cast<const T*>(p.s.d_proj) + (size_t)b.row * p.g.row + col;
-    const float* w = p.s.d_conv + (size_t)ch * taps;
-    auto input = [&](int k) -> float {   // k rows after the block's first one (k < 0: before it)
-        if (b.row + k >= b.first) return ld(x + (int64_t)k * p.g.row);
-        const int at = b.pos + k;
-        return at >= 0 ? b.old[(size_t)(at % keep) * p.g.channels + ch] : 0.f;
-    };
-    if constexpr (TAPS > 0) {
-        float in[TAPS - 1 + kBlock], wt[TAPS];
-#pragma unroll
-        for (int j = 0; j < TAPS; ++j) wt[j] = __ldg(w + j);
-        if (b.inner) {   // a whole block away from the start of its run: all inputs are rows of this pass
-#pragma unroll
-            for (int k = 0; k < TAPS - 1 + kBlock; ++k) in[k] = ld(x + (int64_t)(k - (TAPS - 1)) * p.g.row);
-        } else {
-#pragma unroll
-            for (int k = 0; k < TAPS - 1 + kBlock; ++k) in[k] = k - (TAPS - 1) < b.n ? input(k - (TAPS - 1)) : 0.f;
-        }
-#pragma unroll
-        for (int t = 0; t < kBlock; ++t) {
-            float acc = 0.f;
-#pragma unroll
-            for (int j = 0; j < TAPS; ++j) acc = fmaf(wt[j], in[t + j], acc);
-            out[t] = t < b.n ? (sizeof(T) == 2 ? silu_fast(acc) : silu(acc)) : 0.f;
-        }
-    } else {
-        for (int t = 0; t < kBlock; ++t) {
-            float acc = 0.f;
-            if (t < b.n)
-                for (int j = 0; j < taps; ++j) acc = fmaf(w[j], input(t + j - keep), acc);
-            out[t] = t < b.n ? silu(acc) : 0.f;
-        }
-    }
-    if (!keep_state || keep == 0 || (b.inner && b.last - (b.row + kBlock - 1) >= keep)) return;
-    if (b.row == b.first)   // a run shorter than the state: what it does not push out stays
-        for (int k = 1; k <= keep; ++k) {
-            const int at = b.pos - k;
-            if (at >= 0 && at > b.pos + (b.last - b.row) - keep) b.fresh[(size_t)(at % keep) * p.g.channels + ch] = b.old[(size_t)(at % keep) * p.g.channels + ch];
-        }
-    for (int t = 0; t < b.n; ++t)
-        if (b.last - (b.row + t) < keep) b.fresh[(size_t)((b.pos + t) % keep) * p.g.channels + ch] = ld(x + (int64_t)t * p.g.row);
-}
-
-// sums of N values over the warp: lane i gets the sum of v[i mod N]
-template <int N>
-__device__ __forceinline__ float transpose_sum(float (&v)[N]) {
-    const int lane = threadIdx.x & 31;
-#pragma unroll
-    for (int h = N / 2; h >= 1; h >>= 1)
-#pragma unroll
-        for (int i = 0; i < h; ++i) {
-            const float give = (lane & h) ? v[i] : v[i + h], keep = (lane & h) ? v[i + h] : v[i];
-            v[i] = keep + __shfl_xor_sync(0xffffffffu, give, h);
-        }
-#pragma unroll
-    for (int h = N; h < 32; h <<= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], h);
-    return v[0];
-}
-
-// NI: groups of 32 key channels
-template <typename T, int NI, int TAPS, bool HEAD>
-__global__ void __launch_bounds__(kPrepThreads, NI <= 4 ? 4 : 1) delta_prepare_kernel(const Params p) {
-    constexpr int kVecs = vecs_of(HEAD), kNums = nums_of(HEAD), ND = HEAD ? 1 : NI;
-    const Geo& g = p.g;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, blk = blockIdx.x;
-    pdl_launch_dependents();
-    pdl_wait();
-    int run = 0;   // the last run whose blocks start at or before this one
-    for (int lo = 0, hi = (int)p.s.n_runs; lo < hi;) {
-        const int mid = (lo + hi) / 2;
-        if (p.s.d_runs[mid] / kBlock + mid <= blk) { run = mid; lo = mid + 1; }
-        else hi = mid;
-    }
-    BlockState b;
-    b.first = p.s.d_runs[run];
-    b.last = p.s.d_run_last[b.first];
-    b.row = b.first + (blk - (b.first / kBlock + run)) * kBlock;
-    if (b.row > b.last) return;
-    b.n = min(kBlock, b.last - b.row + 1);
-    b.pos = p.s.d_pos[b.row];
-    b.inner = b.n == kBlock && b.row - b.first >= g.taps - 1;
-    {
-        const size_t half = (size_t)(g.taps - 1) * g.channels;
-        float* state = p.s.d_conv_state + (size_t)p.s.d_slot[b.row] * 2 * half;
-        const int par = p.s.d_parity[b.row] & 1;
-        b.old = state + par * half; b.fresh = state + (par ^ 1) * half;
-    }
-    const int v_groups = (g.vp + 127) / 128;   // of 128 value columns of a head
-    for (int job = warp; job < g.heads * (1 + v_groups); job += kPrepThreads / 32) {
-        if (job >= g.heads) {
-            const int h = (job - g.heads) / v_groups, c0 = (job - g.heads) % v_groups * 128 + lane;
-#pragma unroll
-            for (int i = 0; i < 4; ++i) {
-                const int c = c0 + i * 32;
-                if (c >= g.vp) break;
-                float v[kBlock] = {0.f, 0.f, 0.f, 0.f};
-                if (c < g.vdim) conv_block<T, TAPS>(p, b, 2 * g.kv_heads * g.dim + h * g.vdim + c, g.v_off + h * g.vdim + c, true, v);
-                float* dst = p.w.v + ((size_t)blk * g.heads + h) * kBlock * g.vp + c;
-#pragma unroll
-                for (int t = 0; t < kBlock; ++t) dst[(size_t)t * g.vp] = v[t];
-            }
-            continue;
-        }
-        const int head = job, kvh = head / g.group;
-        const bool own = head % g.group == 0;   // heads that share q and k: the first passes their convolution state on
-        float q[NI][kBlock], k[NI][kBlock], dec[ND][kBlock];
-#pragma unroll
-        for (int i = 0; i < ND; ++i)   // travels while the convolutions are computed
-#pragma unroll
-            for (int t = 0; t < kBlock; ++t) {
-                const int d = HEAD ? 0 : i * 32 + lane;
-                dec[i][t] = t < b.n && d < g.dim ? decay_input<T>(p, b.row + t, head, d) : 0.f;
-            }
-        float sums[8];
-#pragma unroll
-        for (int i = 0; i < 8; ++i) sums[i] = 0.f;
-#pragma unroll
-        for (int i = 0; i < NI; ++i) {
-            const int d = i * 32 + lane;
-#pragma unroll
-            for (int t = 0; t < kBlock; ++t) q[i][t] = k[i][t] = 0.f;
-            if (d < g.dim) {
-                conv_block<T, TAPS>(p, b, kvh * g.dim + d, g.q_off + kvh * g.dim + d, own, q[i]);
-                conv_block<T, TAPS>(p, b, (g.kv_heads + kvh) * g.dim + d, g.k_off + kvh * g.dim + d, own, k[i]);
-            }
-#pragma unroll
-            for (int t = 0; t < kBlock; ++t) { sums[t] = fmaf(q[i][t], q[i][t], sums[t]); sums[4 + t] = fmaf(k[i][t], k[i][t], sums[4 + t]); }
-        }
-        float norm = 1.f / sqrtf(transpose_sum(sums) + 1e-6f);
-        if (lane < 4) norm *= g.q_scale;
-#pragma unroll
-        for (int t = 0; t < kBlock; ++t) {
-            const float qs = __shfl_sync(0xffffffffu, norm, t), ks = __shfl_sync(0xffffffffu, norm, 4 + t);
-#pragma unroll
-            for (int i = 0; i < NI; ++i) { q[i][t] *= qs; k[i][t] *= ks; }
-        }
-        const float rate = -expf(p.s.d_a_log[head]);
-        float* vec = p.w.vec + ((size_t)blk * g.heads + head) * kVecs * g.dp;
-        float num[16];   // A in 0 .. 5, B in 6 .. 15
-#pragma unroll
-        for (int i = 0; i < 16; ++i) num[i] = 0.f;
-        float gd[kBlock];
-        auto decays = [&](int i, int d) {
-#pragma unroll
-            for (int t = 0; t < kBlock; ++t) gd[t] = 1.f;
-            if (d < g.dim) {
-                const float bias = decay_bias(p, head, d);
-#pragma unroll
-                for (int t = 0; t < kBlock; ++t)
-                    if (t < b.n) {
-                        const float x = dec[i][t] + bias;
-                        gd[t] = sizeof(T) == 2 ? decay_fast(x, rate) : expf(rate * softplus(x));
-                    }
-            }
-        };
-        if (HEAD) decays(0, 0);
-#pragma unroll
-        for (int i = 0; i < NI; ++i) {
-            const int d = i * 32 + lane;
-            if (!HEAD) decays(HEAD ? 0 : i, d);
-            const float g10 = gd[1], g21 = gd[2], g32 = gd[3], g20 = g21 * g10, g31 = g32 * g21, g30 = g31 * g10;   // decays of s+1 .. t
-            const float* kk = k[i];
-            const float* qq = q[i];
-            num[0] = fmaf(kk[1] * kk[0], g10, num[0]);
-            num[1] = fmaf(kk[2] * kk[0], g20, num[1]);
-            num[2] = fmaf(kk[2] * kk[1], g21, num[2]);
-            num[3] = fmaf(kk[3] * kk[0], g30, num[3]);
-            num[4] = fmaf(kk[3] * kk[1], g31, num[4]);
-            num[5] = fmaf(kk[3] * kk[2], g32, num[5]);
-            num[6] = fmaf(qq[0], kk[0], num[6]);
-            num[7] = fmaf(qq[1] * kk[0], g10, num[7]);
-            num[8] = fmaf(qq[1], kk[1], num[8]);
-            num[9] = fmaf(qq[2] * kk[0], g20, num[9]);
-            num[10] = fmaf(qq[2] * kk[1], g21, num[10]);
-            num[11] = fmaf(qq[2], kk[2], num[11]);
-            num[12] = fmaf(qq[3] * kk[0], g30, num[12]);
-            num[13] = fmaf(qq[3] * kk[1], g31, num[13]);
-            num[14] = fmaf(qq[3] * kk[2], g32, num[14]);
-            num[15] = fmaf(qq[3], kk[3], num[15]);
-            if (d < g.dp) {
-                float* o = vec + d;
-                if constexpr (HEAD) {
-#pragma unroll
-                    for (int t = 0; t < kBlock; ++t) { o[t * g.dp] = kk[t]; o[(kBlock + t) * g.dp] = qq[t]; }
-                    continue;
-                }
-                const float p0 = gd[0], p1 = p0 * gd[1], p2 = p1 * gd[2], p3 = p2 * gd[3];
-                o[0] = p0 * kk[0]; o[g.dp] = p1 * kk[1]; o[2 * g.dp] = p2 * kk[2]; o[3 * g.dp] = p3 * kk[3];
-                o[4 * g.dp] = p0 * qq[0]; o[5 * g.dp] = p1 * qq[1]; o[6 * g.dp] = p2 * qq[2]; o[7 * g.dp] = p3 * qq[3];
-                o[8 * g.dp] = kk[0] * g30; o[9 * g.dp] = kk[1] * g31; o[10 * g.dp] = kk[2] * g32; o[11 * g.dp] = kk[3];
-                o[12 * g.dp] = p3;
-            }
-        }
-        const float mine = transpose_sum(num);
-        float* dst = p.w.num + ((size_t)blk * g.heads + head) * kNums;
-        if (lane < 16) dst[lane < 6 ? 4 + lane : 6 + lane] = mine;
-        if (HEAD && lane == 0) {
-            const float p1 = gd[0] * gd[1], p2 = p1 * gd[2];
-            *reinterpret_cast<float4*>(dst + 24) = make_float4(gd[0], p1, p2, p2 * gd[3]);
-            *reinterpret_cast<float4*>(dst + 28) = make_float4(gd[1] * gd[2] * gd[3], gd[2] * gd[3], gd[3], 1.f);
-        }
-        if (lane < kBlock)
-            dst[lane] = lane < b.n ? sigmoid(ld(static_cast<const T*>(p.s.d_proj) + (size_t)(b.row + lane) * g.row + g.beta_off + head)) : 0.f;
-    }
 }
 
 // ---- the scan ------------------------------------------------------------------------------------------------------------------
@@ -741,14 +456,6 @@ int launch_scan(const Params& p, cudaStream_t s) {
     }
     return p.g.head_decay ? launch_scan_of<NI, CPL, LPC, STAGES, true>(p, s) : launch_scan_of<NI, CPL, LPC, STAGES, false>(p, s);
 }
-template <typename T, int NI>
-int launch_prepare(const Params& p, cudaStream_t s) {
-    const dim3 grid((unsigned)max_blocks(p.s.rows, p.s.n_runs));
-    constexpr int kTaps = NI <= 8 ? 4 : 0;   // convolutions of four taps are unrolled
-    void (*kern)(Params) = p.g.head_decay ? (p.g.taps == kTaps ? delta_prepare_kernel<T, NI, kTaps, true> : delta_prepare_kernel<T, NI, 0, true>)
-                                          : (p.g.taps == kTaps ? delta_prepare_kernel<T, NI, kTaps, false> : delta_prepare_kernel<T, NI, 0, false>);
-    return launch_kernel(kern, grid, dim3(kPrepThreads), 0, s, 1, p);
-}
 template <typename T, int NR, int VEC>
 int launch_decode(const Params& p, cudaStream_t s) {
     const size_t smem = ((size_t)3 * p.g.dp + 2 * p.g.vp + kDecWarps * 2 * 32 * VEC) * 4;
@@ -768,20 +475,23 @@ int run(const Params& p, cudaStream_t s) {
         if (g.dim <= 128) return launch_decode<T, 16, 1>(p, s);
         return launch_decode<T, 64, 1>(p, s);
     }
-    int rc = GPTRS_OK;
-    if (g.dim <= 32) { if (!(rc = launch_prepare<T, 1>(p, s))) rc = launch_scan<1, 2, 8, 4>(p, s); }
-    else if (g.dim <= 64) { if (!(rc = launch_prepare<T, 2>(p, s))) rc = launch_scan<1, 4, 16, 4>(p, s); }
-    else if (g.dim <= 128) { if (!(rc = launch_prepare<T, 4>(p, s))) rc = launch_scan<2, 4, 16, 4>(p, s); }
-    else if (g.dim <= 256) { if (!(rc = launch_prepare<T, 8>(p, s))) rc = launch_scan<4, 4, 16, 4>(p, s); }
-    else { if (!(rc = launch_prepare<T, 16>(p, s))) rc = launch_scan<8, 2, 16, 4>(p, s); }
+    int rc = launch_prepare(p, sizeof(T) == 2, s);
+    if (rc) return rc;
+    if (g.dim <= 32) rc = launch_scan<1, 2, 8, 4>(p, s);
+    else if (g.dim <= 64) rc = launch_scan<1, 4, 16, 4>(p, s);
+    else if (g.dim <= 128) rc = launch_scan<2, 4, 16, 4>(p, s);
+    else if (g.dim <= 256) rc = launch_scan<4, 4, 16, 4>(p, s);
+    else rc = launch_scan<8, 2, 16, 4>(p, s);
     if (rc) return rc;
     return launch_kernel(delta_output_kernel<T>, dim3((unsigned)ceil_div(p.s.rows * g.heads, 8)), dim3(256), 0, s, 1, p);
 }
 
 }  // namespace
+}  // namespace delta
 }  // namespace gptrs
 
 using namespace gptrs;
+using namespace gptrs::delta;
 
 extern "C" {
 
